@@ -138,8 +138,9 @@ PYBIND11_MODULE(_engine, m) {
   py::class_<EngineCoreRequest>(m, "EngineCoreRequest")
       .def(py::init<>())
       .def(py::init([](std::string id, std::vector<int32_t> toks, SamplingParams sp,
-                       std::optional<int32_t> eos, double arrival, int priority) {
+                       std::optional<int32_t> eos, double arrival, int priority, bool input_open) {
              EngineCoreRequest r;
+             r.input_open = input_open;
              r.request_id = std::move(id);
              r.prompt_token_ids = std::move(toks);
              r.sampling_params = std::move(sp);
@@ -150,7 +151,8 @@ PYBIND11_MODULE(_engine, m) {
            }),
            py::arg("request_id"), py::arg("prompt_token_ids"), py::arg("sampling_params"),
            py::arg("eos_token_id") = std::nullopt, py::arg("arrival_time") = 0.0,
-           py::arg("priority") = 0)
+           py::arg("priority") = 0, py::arg("input_open") = false)
+      .def_readwrite("input_open", &EngineCoreRequest::input_open)
       .def_readwrite("request_id", &EngineCoreRequest::request_id)
       .def_readwrite("prompt_token_ids", &EngineCoreRequest::prompt_token_ids)
       .def_readwrite("sampling_params", &EngineCoreRequest::sampling_params)
@@ -191,6 +193,7 @@ PYBIND11_MODULE(_engine, m) {
       .def_readonly("sampling_params", &NewRequestData::sampling_params)
       .def_readonly("block_ids", &NewRequestData::block_ids)
       .def_readonly("num_computed_tokens", &NewRequestData::num_computed_tokens)
+      .def_readonly("input_open", &NewRequestData::input_open)
       .def_readonly("num_prompt_tokens", &NewRequestData::num_prompt_tokens);
   py::class_<CachedRequestData>(m, "CachedRequestData")
       .def_readonly("req_ids", &CachedRequestData::req_ids)
@@ -299,6 +302,7 @@ PYBIND11_MODULE(_engine, m) {
       .def_readwrite("block_size", &KVCacheSpec::block_size)
       .def_readwrite("num_kv_heads", &KVCacheSpec::num_kv_heads)
       .def_readwrite("head_size", &KVCacheSpec::head_size)
+      .def_readwrite("head_size_v", &KVCacheSpec::head_size_v)
       .def_readwrite("dtype_bytes", &KVCacheSpec::dtype_bytes)
       .def_readwrite("sliding_window", &KVCacheSpec::sliding_window)
       .def_readwrite("attention_chunk_size", &KVCacheSpec::attention_chunk_size)
@@ -397,6 +401,8 @@ PYBIND11_MODULE(_engine, m) {
         s.add_request(req);
         return req;
       })
+      .def("append_input", &Scheduler::append_input, py::arg("request_id"), py::arg("tokens"),
+           py::arg("close") = false)
       .def("schedule", &Scheduler::schedule)
       .def("update_from_output", &Scheduler::update_from_output)
       .def("finish_requests", &Scheduler::finish_requests)
@@ -492,7 +498,8 @@ PYBIND11_MODULE(_engine, m) {
   // ---- worker-side input preparation
   py::class_<StepLayout>(m, "StepLayout")
       .def_static("make", &StepLayout::make, py::arg("max_tokens"), py::arg("max_reqs"),
-                  py::arg("max_blocks"), py::arg("num_groups"), py::arg("max_spec") = 0)
+                  py::arg("max_blocks"), py::arg("num_groups"), py::arg("max_spec") = 0,
+                  py::arg("max_score") = 0)
       .def_readonly("max_logits", &StepLayout::max_logits)
       .def_readonly("max_tokens", &StepLayout::max_tokens)
       .def_readonly("max_reqs", &StepLayout::max_reqs)
@@ -535,6 +542,9 @@ PYBIND11_MODULE(_engine, m) {
       .def_readonly("produces_token", &StepInfo::produces_token)
       .def_readonly("num_draft", &StepInfo::num_draft)
       .def_readonly("logits_row0", &StepInfo::logits_row0)
+      .def_readonly("num_score", &StepInfo::num_score)
+      .def_readonly("score_req_ids", &StepInfo::score_req_ids)
+      .def_readonly("score_positions", &StepInfo::score_positions)
       .def_readonly("max_logprobs", &StepInfo::max_logprobs);
   py::class_<InputBatch>(m, "InputBatch")
       .def(py::init<int, int, int, std::vector<int>>())
@@ -544,6 +554,7 @@ PYBIND11_MODULE(_engine, m) {
         return b.prepare(so, l, reinterpret_cast<uint8_t*>(buf), async_mode);
       }, py::arg("scheduler_output"), py::arg("layout"), py::arg("buffer_ptr"),
            py::arg("async_mode") = false)
+      .def("set_score_positions", &InputBatch::set_score_positions)
       .def("propose_ngram", &InputBatch::propose_ngram)
       .def("num_tokens", [](const InputBatch& b, const std::string& id) {
         const CachedRequestState* s = b.get(id);

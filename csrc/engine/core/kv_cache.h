@@ -26,6 +26,7 @@ struct KVCacheSpec {
   int block_size = 16;
   int num_kv_heads = 1;
   int head_size = 128;
+  int head_size_v = 0;           // values of another width than the keys (0: the same)
   int dtype_bytes = 2;
   int sliding_window = 0;        // kSlidingWindow
   int attention_chunk_size = 0;  // kChunkedLocal
@@ -35,7 +36,7 @@ struct KVCacheSpec {
   int64_t page_size_bytes() const {
     if (kind == KVSpecKind::kMamba) return mamba_state_bytes;
     if (kind == KVSpecKind::kMLA) return (int64_t)block_size * head_size * dtype_bytes;
-    return 2ll * block_size * num_kv_heads * head_size * dtype_bytes;
+    return (int64_t)block_size * num_kv_heads * (head_size + (head_size_v ? head_size_v : head_size)) * dtype_bytes;
   }
   // Worst-case bytes one request of max_model_len tokens needs in this group.
   int64_t max_memory_usage_bytes(int max_model_len) const;

@@ -65,6 +65,18 @@ void Scheduler::add_request(const RequestPtr& req) {
   waiting_.add(req);
 }
 
+void Scheduler::append_input(const std::string& id, const std::vector<int32_t>& tokens, bool close) {
+  RequestPtr r = get_request(id);
+  if (!r || !r->input_open) throw std::invalid_argument("request " + id + " takes no further input");
+  if (close && tokens.empty()) throw std::invalid_argument("the input is closed with its last tokens");
+  if (r->num_tokens() + (int)tokens.size() >= cfg_.max_model_len)
+    throw std::invalid_argument("request " + id + " would exceed max_model_len");
+  r->prompt_token_ids.insert(r->prompt_token_ids.end(), tokens.begin(), tokens.end());
+  r->all_token_ids.insert(r->all_token_ids.end(), tokens.begin(), tokens.end());
+  r->appended_input = true;
+  if (close) r->input_open = false;
+}
+
 void Scheduler::preempt_request(const RequestPtr& req) {
   kv_->free(*req);
   req->status = RequestStatus::kPreempted;
@@ -259,6 +271,7 @@ SchedulerOutput Scheduler::schedule() {
     d.block_ids = new_blocks_of[r->request_id].block_ids();
     d.num_computed_tokens = r->num_computed_tokens;
     d.num_prompt_tokens = r->num_prompt_tokens();
+    d.input_open = r->input_open;
     return d;
   };
   for (auto& r : new_reqs) out.scheduled_new_reqs.push_back(as_new(r));
@@ -270,14 +283,18 @@ SchedulerOutput Scheduler::schedule() {
     // tokens the worker has not seen yet: everything sampled after what it has computed
     int n_sched = sched_tokens[r->request_id];
     int lo = r->num_computed_tokens;
-    int hi = std::min(r->num_tokens(), lo + n_sched);
+    // (all of them after an appended portion: the worker tells from its count whether a step
+    // reaches the end of the known tokens)
+    int hi = r->appended_input ? r->num_tokens() : std::min(r->num_tokens(), lo + n_sched);
     std::vector<int32_t> toks;
-    if (lo < hi && lo >= r->num_prompt_tokens())
+    if (lo < hi && (lo >= r->num_prompt_tokens() || r->appended_input))
       toks.assign(r->all_token_ids.begin() + lo, r->all_token_ids.begin() + hi);
     c.new_token_ids.push_back(std::move(toks));
     c.new_block_ids.push_back(new_blocks_of[r->request_id].block_ids());
     c.num_computed_tokens.push_back(r->num_computed_tokens);
     c.num_output_tokens.push_back(r->num_output_tokens());
+    c.input_open.push_back(r->input_open ? 1 : 0);
+    c.num_prompt_tokens.push_back(r->num_prompt_tokens());
   }
   for (auto& r : preempted) out.preempted_req_ids.push_back(r->request_id);
   for (auto& p : out.num_scheduled_tokens) {
@@ -504,7 +521,7 @@ void AsyncScheduler::update_after_schedule(const SchedulerOutput& so) {
   for (auto& p : so.num_scheduled_tokens) {
     Request& r = *requests_[p.first];
     // This step computes the request's last known token: a new token will come out of it.
-    if (r.num_computed_tokens == r.num_tokens() + r.num_output_placeholders)
+    if (!r.input_open && r.num_computed_tokens == r.num_tokens() + r.num_output_placeholders)
       r.num_output_placeholders += 1;
   }
 }

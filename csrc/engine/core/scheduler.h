@@ -86,6 +86,9 @@ class Scheduler {
   virtual ~Scheduler() = default;
 
   void add_request(const RequestPtr& req);
+  // Further prompt tokens of a request whose input is open; `close` ends the input, after which
+  // the request generates like any other. Throws for an unknown or closed request.
+  void append_input(const std::string& id, const std::vector<int32_t>& tokens, bool close);
   virtual SchedulerOutput schedule();
   // Returns one EngineCoreOutputs (single client).
   virtual EngineCoreOutputs update_from_output(const SchedulerOutput& so,

@@ -46,7 +46,8 @@ void SamplingParams::post_init() {
 Request::Request(const EngineCoreRequest& r)
     : request_id(r.request_id), prompt_token_ids(r.prompt_token_ids),
       sampling_params(r.sampling_params), eos_token_id(r.eos_token_id),
-      arrival_time(r.arrival_time), priority(r.priority), cache_salt(r.cache_salt) {
+      arrival_time(r.arrival_time), priority(r.priority), cache_salt(r.cache_salt),
+      input_open(r.input_open) {
   all_token_ids = prompt_token_ids;
   max_tokens = sampling_params.max_tokens ? *sampling_params.max_tokens : (1 << 30);
   use_structured_output = sampling_params.structured_outputs && sampling_params.structured_outputs->any();

@@ -120,6 +120,9 @@ struct EngineCoreRequest {
   double arrival_time = 0.0;
   int priority = 0;
   std::optional<std::string> cache_salt;
+  // The prompt arrives in portions (Scheduler::append_input): the request computes what it has
+  // and keeps its blocks, but samples nothing until its input is closed.
+  bool input_open = false;
 };
 
 // Stop reason: either a token id or a stop string.
@@ -152,6 +155,8 @@ struct Request {
   void* structured_state = nullptr;        // owned by the structured-output manager
   std::vector<BlockHash> block_hashes;     // chained hashes of the full blocks seen so far
   int num_nans_in_logits = 0;
+  bool input_open = false;                 // more prompt tokens may follow; nothing is sampled
+  bool appended_input = false;             // prompt tokens were added after the first portion
 
   explicit Request(const EngineCoreRequest& r);
   int num_prompt_tokens() const { return (int)prompt_token_ids.size(); }
@@ -177,6 +182,7 @@ struct NewRequestData {
   std::vector<std::vector<int32_t>> block_ids;  // per KV-cache group
   int num_computed_tokens = 0;
   int num_prompt_tokens = 0;
+  bool input_open = false;
 };
 
 struct CachedRequestData {
@@ -186,6 +192,8 @@ struct CachedRequestData {
   std::vector<std::vector<std::vector<int32_t>>> new_block_ids;  // per request, per group
   std::vector<int> num_computed_tokens;
   std::vector<int> num_output_tokens;
+  std::vector<uint8_t> input_open;
+  std::vector<int> num_prompt_tokens;                            // grows with appended input
   size_t size() const { return req_ids.size(); }
 };
 

@@ -9,9 +9,9 @@ namespace b200 {
 static size_t align_up(size_t v, size_t a) { return (v + a - 1) / a * a; }
 
 StepLayout StepLayout::make(int max_tokens, int max_reqs, int max_blocks, int num_groups,
-                            int max_spec) {
+                            int max_spec, int max_score) {
   StepLayout l;
-  l.max_logits = max_reqs * (1 + (max_spec > 0 ? max_spec : 0));
+  l.max_logits = max_reqs * (1 + (max_spec > 0 ? max_spec : 0)) + max_score;
   l.max_tokens = max_tokens;
   l.max_reqs = max_reqs;
   l.max_blocks = max_blocks;
@@ -101,17 +101,18 @@ bool InputBatch::plain_greedy(const std::string& id) const {
 }
 
 void InputBatch::update_states(const SchedulerOutput& so) {
-  auto drop = [&](const std::string& id) {
+  auto drop = [&](const std::string& id, bool forget) {
     auto it = reqs_.find(id);
     if (it == reqs_.end()) return;
     if (it->second.state_slot >= 0) free_state_slots_.push_back(it->second.state_slot);
+    if (forget) score_.erase(id);
     reqs_.erase(it);
     last_rows_.erase(id);
   };
-  for (auto& id : so.finished_req_ids) drop(id);
-  for (auto& id : so.preempted_req_ids) drop(id);
+  for (auto& id : so.finished_req_ids) drop(id, true);
+  for (auto& id : so.preempted_req_ids) drop(id, false);
   for (auto& n : so.scheduled_new_reqs) {
-    drop(n.req_id);  // a resumed request replaces whatever was left
+    drop(n.req_id, false);  // a resumed request replaces whatever was left
     CachedRequestState s;
     s.req_id = n.req_id;
     s.token_ids = n.prompt_token_ids;
@@ -119,6 +120,7 @@ void InputBatch::update_states(const SchedulerOutput& so) {
     s.num_computed_tokens = n.num_computed_tokens;
     s.block_ids = n.block_ids;
     s.sampling_params = n.sampling_params;
+    s.input_open = n.input_open;
     s.state_slot = alloc_state_slot();
     s.sample_step = (uint64_t)std::max(0, (int)n.prompt_token_ids.size() - n.num_prompt_tokens);
     reqs_.emplace(n.req_id, std::move(s));
@@ -129,6 +131,8 @@ void InputBatch::update_states(const SchedulerOutput& so) {
     if (it == reqs_.end()) throw std::runtime_error("cached request unknown to the worker: " + c.req_ids[i]);
     CachedRequestState& s = it->second;
     s.num_computed_tokens = c.num_computed_tokens[i];
+    s.input_open = c.input_open[i] != 0;
+    s.num_prompt_tokens = c.num_prompt_tokens[i];
     auto& nt = c.new_token_ids[i];
     if (!nt.empty()) {
       size_t lo = (size_t)s.num_computed_tokens;
@@ -140,6 +144,12 @@ void InputBatch::update_states(const SchedulerOutput& so) {
     for (size_t g = 0; g < nb.size(); ++g)
       s.block_ids[g].insert(s.block_ids[g].end(), nb[g].begin(), nb[g].end());
   }
+}
+
+void InputBatch::set_score_positions(const std::string& id, const std::vector<int>& positions) {
+  auto& v = score_[id];
+  v.insert(v.end(), positions.begin(), positions.end());
+  std::sort(v.begin(), v.end());
 }
 
 void InputBatch::append_sampled(const std::string& req_id, const std::vector<int32_t>& toks) {
@@ -195,6 +205,7 @@ StepInfo InputBatch::prepare(const SchedulerOutput& so, const StepLayout& L, uin
   qs[0] = 0;
   pqs[0] = 0;
   std::unordered_map<std::string, int> new_rows;
+  std::vector<int> score_rows;
   for (size_t r = 0; r < items.size(); ++r) {
     CachedRequestState& s = *items[r].s;
     const int n = items[r].n;
@@ -263,7 +274,20 @@ StepInfo InputBatch::prepare(const SchedulerOutput& so, const StepLayout& L, uin
     rep[r] = (float)sp.repetition_penalty;
     freq[r] = (float)sp.frequency_penalty;
     pres[r] = (float)sp.presence_penalty;
-    const bool produces = lo + n >= (int)s.token_ids.size();
+    if (!score_.empty()) {
+      auto sc = score_.find(s.req_id);
+      if (sc != score_.end()) {
+        auto& v = sc->second;
+        auto b = std::lower_bound(v.begin(), v.end(), lo), e = std::lower_bound(v.begin(), v.end(), lo + n);
+        for (auto p = b; p != e; ++p) {
+          score_rows.push_back(qs[r] + *p - lo);
+          info.score_req_ids.push_back(s.req_id);
+          info.score_positions.push_back(*p);
+        }
+        v.erase(b, e);
+      }
+    }
+    const bool produces = !s.input_open && lo + n >= (int)s.token_ids.size();
     info.produces_token.push_back(produces ? 1 : 0);
     // drafts verified this step: the scheduled positions beyond the known tokens
     // (positions beyond the known tokens without a draft are in-flight tokens of async scheduling)
@@ -297,6 +321,9 @@ StepInfo InputBatch::prepare(const SchedulerOutput& so, const StepLayout& L, uin
     s.batch_row = (int)r;
     new_rows[s.req_id] = (int)r;
   }
+  if (info.num_logits + (int)score_rows.size() > L.max_logits)
+    throw std::runtime_error("more positions to score than the layout has logits rows");
+  for (int row : score_rows) logits_idx[info.num_logits + info.num_score++] = row;
   info.num_reqs = (int)items.size();
   info.num_tokens = tok;
   last_rows_.swap(new_rows);

@@ -31,6 +31,7 @@ struct CachedRequestState {
   int state_slot = -1;   // recurrent-state slot (GDN / Mamba), stable for the request's life
   uint64_t sample_step = 0;
   int batch_row = -1;    // row in the last prepared batch (for device-resident sampled ids)
+  bool input_open = false;  // prompt still arriving: no token is sampled
 };
 
 // Byte offsets of each array inside the packed step buffer.
@@ -60,8 +61,9 @@ struct StepLayout {
   size_t sample_rows = 0;     // int32 [max_reqs] batch row of each logits row (rows that sample)
   size_t total_bytes = 0;
   // max_spec: draft tokens a request may verify per step (each adds a logits row).
+  // max_score: logits rows per step beyond those that sample (InputBatch::set_score_positions).
   static StepLayout make(int max_tokens, int max_reqs, int max_blocks, int num_groups,
-                         int max_spec = 0);
+                         int max_spec = 0, int max_score = 0);
 };
 
 struct StepInfo {
@@ -82,6 +84,10 @@ struct StepInfo {
   std::vector<int> max_logprobs;           // per request (-1 = none)
   std::vector<int> num_draft;              // per request: draft tokens verified this step
   std::vector<int> logits_row0;            // per request: its first logits row (-1 = none)
+  // rows num_logits .. num_logits + num_score - 1: positions whose logits were asked for
+  int num_score = 0;
+  std::vector<std::string> score_req_ids;
+  std::vector<int> score_positions;
 };
 
 class InputBatch {
@@ -97,6 +103,10 @@ class InputBatch {
   // Sync mode: record sampled tokens (the scheduler also sends them back as new_token_ids).
   void append_sampled(const std::string& req_id, const std::vector<int32_t>& toks);
   const CachedRequestState* get(const std::string& id) const;
+  // Positions of a request whose logits are wanted besides the sampled ones. A step that computes
+  // some of them lists their rows after the sampling rows (StepInfo::num_score). May be called
+  // before the request reaches the worker.
+  void set_score_positions(const std::string& id, const std::vector<int>& positions);
   // Prompt-lookup drafting (reference: include/vllm/v1/spec_decode/ngram_proposer.h): the longest
   // suffix of between min_n and max_n tokens that occurred earlier in the request (latest
   // occurrence first); returns up to k tokens that followed it. Empty if none.
@@ -122,6 +132,7 @@ class InputBatch {
   std::vector<int> block_sizes_;
   std::unordered_map<std::string, CachedRequestState> reqs_;
   std::vector<int> free_state_slots_;
+  std::unordered_map<std::string, std::vector<int>> score_;  // ascending positions still to come
   std::unordered_map<std::string, int> last_rows_;  // req id -> row in the previous batch
 };
 

@@ -171,6 +171,59 @@ typedef struct B200MoeScatter {
   const void* op_counter;
 } B200MoeScatter;
 
+// Attention with a per-head distance bias, mixed heads and an optional null softmax entry over pages
+// [block_size][kw] keys | [block_size][G * vdim] values (attn_bias.cu). q rows carry the score scale;
+// every head reads the whole key row. bias: fp32 [H, bias_len], the entry of distance
+// min(i - j, bias_len - 1), or null. Decode: one row per request. Prefill: q_start [num_reqs + 1]
+// and the 128-row tile list. f32: fp32 q / out / cache instead of bf16.
+typedef struct B200BiasAttn {
+  const void* q;
+  long long ldq;
+  void* out;
+  long long ldo;
+  const void* cache;
+  long long num_blocks;
+  const void* block_table;
+  const void* seq_lens;
+  const void* q_start;
+  const void* bias;
+  void* tmp_o;                 // decode, splits > 1: fp32 [rows, H, splits, vdim]
+  void* tmp_lse;               // fp32 [rows, H, splits]
+  const void* tile_req;
+  const void* tile_q0;
+  int max_blocks, num_reqs, rows;
+  int H, G, kw, vdim, block_size;
+  int bias_len, null_entry, f32, splits, num_tiles;
+} B200BiasAttn;
+
+// fp32 residual stream update + RMSNorm in one pass per row (stream.cu):
+//   start:  stream = table[ids] * scale        (ids non-null)
+//   else:   stream += a + sum_j w_j y[pair_pos[j]]   (a, y each optional; pair_w null: w = 1)
+//   out = stream / rms(stream) * (norm_w + norm_offset)
+// Rows are `width` values in storage padded to `cols` (a multiple of 8, zeros). norm_w: fp32.
+typedef struct B200StreamNorm {
+  float* stream;
+  const void* ids;             // int64 [T]
+  const void* table;
+  const void* a;
+  const void* y;
+  const void* pair_pos;        // int32 [T, k], < 0: skipped
+  const float* pair_w;
+  const float* norm_w;
+  void* out;
+  long long lds, lda, ldy, ldo, vocab;
+  int T, width, cols, k;
+  int f32, a_f32;              // element type of table / y / out, and of a
+  float scale, eps, norm_offset;
+} B200StreamNorm;
+
+// Activation of a gated pair with clamps: g = min(gate, limit), u = clamp(up, -limit, limit),
+// g * sigmoid(alpha g) * (u + up_offset); gate and up are first multiplied by row_w[row] (null: 1).
+typedef struct B200ClampedGate {
+  float limit, alpha, up_offset;
+  const float* row_w;
+} B200ClampedGate;
+
 // A fused-chain program (recipe.cu): rows x width bf16 values, up to four shared-memory row
 // registers, a list of steps over them. Operand rows are addressed as
 // ptr + (row / heads) * ld + (row % heads) * width + col, in elements of the operand's type
@@ -202,6 +255,11 @@ int b200_attn_decode_merge(const void* tmp_o, const void* tmp_lse, void* out, in
 int b200_merge_attn_states(const void* a, const void* lse_a, const void* b, const void* lse_b, void* out, void* lse_out, int T, int H, int D, cudaStream_t stream);
 // ---- attn_decode_tc.cu
 int b200_attn_decode_tc(const void* q, int ldq, void* out, int ldo, const void* kv_cache, int64_t num_blocks, int block_size, int Hq, int Hkv, int D, const void* block_table, int max_blocks, const void* seq_lens, int B, float scale, float softcap, int window, int splits, void* tmp_o, void* tmp_lse, cudaStream_t stream);
+// ---- attn_bias.cu
+int b200_head_mix_kv(const void* qkv, long long ld, const void* mix, void* q_out, long long ldq, const void* slots, void* cache, int H, int G, int dim, int vdim, int block_size, int T, int f32, cudaStream_t stream);
+int b200_bias_attn_kernel(const B200BiasAttn* a, int phase);
+int b200_bias_attn_decode(const B200BiasAttn* a, int any_size, cudaStream_t stream);
+int b200_bias_attn_prefill(const B200BiasAttn* a, int any_size, cudaStream_t stream);
 // ---- attn_prefill.cu
 int b200_attn_prefill(const void* q, int ldq, void* out, int ldo, void* lse, const void* kv_cache, int64_t num_blocks, int block_size, int Hq, int Hkv, int D, const void* block_table, int max_blocks, const void* seq_lens, const void* q_start, const void* tile_req, const void* tile_q0, int num_tiles, int total_q, float scale, float softcap, int window, int causal, cudaStream_t stream);
 // ---- common.cu
@@ -251,6 +309,8 @@ int b200_moe_sort(const void* topk_ids, int T, int k, int e0, int e1, void* meta
 int b200_moe_gather(const void* x, int ldx, const void* sorted_token, const void* meta, int E, void* xs, int H, int max_rows, cudaStream_t stream);
 int b200_moe_grouped_gemm(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, cudaStream_t stream);
 int b200_moe_grouped_gemm_gated(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, int kind, cudaStream_t stream);
+int b200_moe_grouped_gemm_clamped(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, const B200ClampedGate* act, cudaStream_t stream);
+int b200_moe_row_weights(const void* pair_pos, const void* topk_w, int P, void* row_w, cudaStream_t stream);
 int b200_moe_combine(const void* y, const void* pair_pos, const void* topk_w, int T, int k, int H, const void* shared, const void* shared_gate, void* out, const B200MoeScatter* sc, cudaStream_t stream);
 int b200_shared_gate(const void* x, int ldx, const void* w, int T, int H, void* out, cudaStream_t stream);
 // ---- norm_act.cu
@@ -263,6 +323,11 @@ int b200_cast_bf16_f32(const void* a, void* out, size_t n, cudaStream_t stream);
 int b200_cast_f32_bf16(const void* a, void* out, size_t n, cudaStream_t stream);
 int b200_embedding(const void* ids, const void* table, void* out, int T, int H, int64_t vocab_start, int64_t vocab_rows, int64_t vocab_total, float scale, cudaStream_t stream);
 int b200_gather_rows(const void* x, const void* idx, void* out, int n_out, int n_src, int row_bytes, cudaStream_t stream);
+// ---- stream.cu
+int b200_stream_norm(const B200StreamNorm* a, cudaStream_t stream);
+int b200_gemm_f32(const void* A, int lda, const void* W, int ldw, void* out, int ldo, const void* bias, int M, int N, int K, cudaStream_t stream);
+int b200_moe_grouped_gemm_f32(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, cudaStream_t stream);
+int b200_clamped_gate_f32(const void* gate_up, void* out, const void* meta, int E, int max_rows, int I, const B200ClampedGate* act, cudaStream_t stream);
 // ---- rope_cache.cu
 int b200_rope_kv(void* qkv, int ld, int q_off, int k_off, int v_off, int q_head_stride, int Hq, int Hkv, int D, int rot, const void* positions, const void* cos_sin, const void* q_norm_w, const void* k_norm_w, float eps, int gemma, int neox, const void* slot_mapping, void* kv_cache, int block_size, void* q_out, int T, cudaStream_t stream);
 int b200_reshape_and_cache(const void* k, int ldk, const void* v, int ldv, const void* slots, void* cache, int block_size, int Hkv, int D, int T, cudaStream_t stream);

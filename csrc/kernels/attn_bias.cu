@@ -1,0 +1,954 @@
+// Attention whose scores carry a per-head distance bias and a mix of the heads, with an optional
+// null entry in the softmax, over a paged cache with separate key and value widths.
+//
+//   s[h, i, j] = sum_g M[h, g] (q_g(i) . k_g(j)) + bias[h, min(i - j, L - 1)]
+//   p[h, i, j] = exp(s) / (null + sum_j exp(s)),   o[h, i] = sum_j p[h, i, j] v_{h / R}(j)
+//
+// A mix of heads before the softmax is linear in the queries, so it moves to the query side: head h
+// gets the query row  q'_h = [ sum_{g in group 0} M[h, g] q_g | sum_{g in group 1} ... ]  over the
+// concatenated key heads, one key row per token serves every head (b200_head_mix_kv builds the
+// rows and writes the cache), and the score is one dot product of the full key row.
+//
+// Cache of a layer: [num_blocks] pages of  [block_size][kw] keys | [block_size][vw] values,
+// kw = key row, vw = value row (all key / value heads), one element type.
+//
+// Three kernels:
+//   bias_attn_any_kernel      any sizes, float or bf16 storage, one CTA per (query row, 4 heads)
+//   bias_attn_decode_kernel   bf16, one query row per request: key / value rows arrive by bulk copies
+//                             in a shared-memory ring, all heads of a request share them, products on
+//                             mma.sync (the kernel is bound by the cache read), split-KV
+//   bias_attn_prefill_kernel  bf16, 128-row query tiles on tcgen05 / TMEM
+#include <float.h>
+
+#include <mutex>
+#include <unordered_map>
+
+#include "api.h"
+#include "sm100.cuh"
+
+namespace b200 {
+
+static constexpr float kLog2e = 1.4426950408889634f;
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
+// ------------------------------------------------------------------------- query mix + cache write
+struct MixParams {
+  const float* qkv;      // [T, ld]: q heads (H * dim) | key heads (G * dim) | value heads (G * vdim)
+  long long ld;
+  const float* mix;      // [H, H]
+  void* q_out;           // [T, H * kw], kw = G * dim
+  long long ldq;
+  const int64_t* slots;  // [T], < 0: no cache write
+  void* cache;
+  int H, G, dim, vdim, block_size, T;
+};
+
+static constexpr int kMixHeads = 8; // output heads per CTA (blockIdx.y)
+
+// kMixTok: tokens per CTA (each loaded mix coefficient serves that many)
+template <typename TO, int kMixTok>
+__global__ void __launch_bounds__(256) head_mix_kv_kernel(MixParams p) {
+  extern __shared__ float mix_smem[];     // [kMixHeads][H] mix rows, then [kMixTok][H * dim] queries
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t0 = blockIdx.x * kMixTok, h0 = blockIdx.y * kMixHeads;
+  const int nt = min(kMixTok, p.T - t0), nh = min(kMixHeads, p.H - h0);
+  const int qw = p.H * p.dim, kw = p.G * p.dim, vw = p.G * p.vdim, R = p.H / p.G;
+  float* sm = mix_smem;
+  float* sq = mix_smem + kMixHeads * p.H;
+  for (int i = threadIdx.x; i < kMixHeads * p.H; i += blockDim.x)
+    sm[i] = i < nh * p.H ? p.mix[(size_t)h0 * p.H + i] : 0.f;
+  for (int t = 0; t < kMixTok; ++t)
+    for (int i = threadIdx.x; i < qw; i += blockDim.x)
+      sq[t * qw + i] = t < nt ? p.qkv[(size_t)(t0 + t) * p.ld + i] : 0.f;
+  __syncthreads();
+  TO* qo = reinterpret_cast<TO*>(p.q_out);
+  for (int c = threadIdx.x; c < kw; c += blockDim.x) {
+    const int g = c / p.dim, d = c - g * p.dim;
+    float acc[kMixHeads][kMixTok];
+#pragma unroll
+    for (int h = 0; h < kMixHeads; ++h)
+#pragma unroll
+      for (int t = 0; t < kMixTok; ++t) acc[h][t] = 0.f;
+    for (int r = 0; r < R; ++r) {
+      const int gh = g * R + r;
+      float q[kMixTok];
+#pragma unroll
+      for (int t = 0; t < kMixTok; ++t) q[t] = sq[t * qw + gh * p.dim + d];
+#pragma unroll
+      for (int h = 0; h < kMixHeads; ++h) {
+        const float m = sm[h * p.H + gh];
+#pragma unroll
+        for (int t = 0; t < kMixTok; ++t) acc[h][t] = fmaf(m, q[t], acc[h][t]);
+      }
+    }
+    for (int h = 0; h < nh; ++h)
+      for (int t = 0; t < nt; ++t) qo[(size_t)(t0 + t) * p.ldq + (size_t)(h0 + h) * kw + c] = from_f<TO>(acc[h][t]);
+  }
+  if (blockIdx.y == 0) {
+    TO* cache = reinterpret_cast<TO*>(p.cache);
+    for (int t = 0; t < nt; ++t) {
+      const int64_t slot = p.slots[t0 + t];
+      if (slot < 0) continue;
+      const int64_t blk = slot / p.block_size, off = slot % p.block_size;
+      const float* src = p.qkv + (size_t)(t0 + t) * p.ld + qw;
+      TO* page = cache + blk * p.block_size * (int64_t)(kw + vw);
+      TO* kd = page + off * kw;
+      TO* vd = page + (int64_t)p.block_size * kw + off * vw;
+      for (int i = threadIdx.x; i < kw; i += blockDim.x) kd[i] = from_f<TO>(src[i]);
+      for (int i = threadIdx.x; i < vw; i += blockDim.x) vd[i] = from_f<TO>(src[kw + i]);
+    }
+  }
+}
+
+// -------------------------------------------------------------------------------- shared parameters
+struct BiasAttnParams {
+  const void* q;            // [rows, H * kw]
+  long long ldq;
+  void* out;                // [rows, H * vdim]
+  long long ldo;
+  const void* cache;
+  const int32_t* block_table;
+  int max_blocks;
+  const int32_t* seq_lens;
+  const int32_t* q_start;   // [num_reqs + 1] first row of each request; null: one row per request
+  int num_reqs, rows;
+  int H, G, kw, vdim, block_size;
+  const float* bias;        // [H, bias_len] or null
+  int bias_len;
+  int null_entry;           // softmax counts one entry of score 0 without a value
+  // decode
+  int splits;
+  float* tmp_o;             // [B, H, splits, vdim]
+  float* tmp_lse;           // [B, H, splits]
+  int kwp, vwp, mt, stages, hp;
+  // prefill
+  const int32_t* tile_req;
+  const int32_t* tile_q0;
+  int k_slots, bias_smem;
+  int* status;
+};
+
+// ------------------------------------------------------------------------------- any-size attention
+static constexpr int kAnyHeads = 4;
+static constexpr int kAnyKeys = 128;
+static constexpr int kAnyAcc = 16;     // outputs per thread: kAnyHeads * vdim <= 128 * kAnyAcc
+
+template <typename T>
+__global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
+  extern __shared__ float any_smem[];
+  float* sq = any_smem;                                  // [kAnyHeads][kw]
+  float* sc = sq + kAnyHeads * p.kw;                     // [kAnyHeads][kAnyKeys]
+  __shared__ long long krow[kAnyKeys], vrow[kAnyKeys];
+  __shared__ float s_alpha[kAnyHeads], s_l[kAnyHeads];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row = blockIdx.x, h0 = blockIdx.y * kAnyHeads, nh = min(kAnyHeads, p.H - h0);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int vw = p.G * p.vdim, R = p.H / p.G;
+  int req = row, pos;
+  if (p.q_start) {
+    int lo = 0, hi = p.num_reqs - 1;                     // last request whose first row is <= row
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (p.q_start[mid] <= row) lo = mid; else hi = mid - 1;
+    }
+    req = lo;
+    pos = p.seq_lens[req] - (p.q_start[req + 1] - row);
+  } else {
+    pos = p.seq_lens[req] - 1;
+  }
+  const T* q = reinterpret_cast<const T*>(p.q) + (size_t)row * p.ldq + (size_t)h0 * p.kw;
+  for (int i = tid; i < nh * p.kw; i += blockDim.x) sq[i] = to_f(q[i]);
+  const T* cache = reinterpret_cast<const T*>(p.cache);
+  const int32_t* bt = p.block_table + (size_t)req * p.max_blocks;
+  float acc[kAnyAcc];
+#pragma unroll
+  for (int a = 0; a < kAnyAcc; ++a) acc[a] = 0.f;
+  // warp w owns the softmax state of head h0 + w
+  float m = p.null_entry ? 0.f : -INFINITY, l = p.null_entry ? 1.f : 0.f;
+  for (int base = 0; base <= pos; base += kAnyKeys) {
+    const int key = base + tid;
+    const bool valid = key <= pos;
+    __syncthreads();
+    if (valid) {
+      const long long page = (long long)bt[key / p.block_size] * p.block_size * (p.kw + vw);
+      const int off = key % p.block_size;
+      krow[tid] = page + (long long)off * p.kw;
+      vrow[tid] = page + (long long)p.block_size * p.kw + (long long)off * vw;
+      float s[kAnyHeads];
+#pragma unroll
+      for (int h = 0; h < kAnyHeads; ++h) s[h] = 0.f;
+      const T* k = cache + krow[tid];
+      for (int i = 0; i < p.kw; ++i) {
+        const float kv = to_f(k[i]);
+#pragma unroll
+        for (int h = 0; h < kAnyHeads; ++h) s[h] = fmaf(sq[h * p.kw + i], kv, s[h]);
+      }
+      for (int h = 0; h < nh; ++h)
+        sc[h * kAnyKeys + tid] =
+            s[h] + (p.bias ? p.bias[(size_t)(h0 + h) * p.bias_len + min(pos - key, p.bias_len - 1)] : 0.f);
+    } else {
+      for (int h = 0; h < nh; ++h) sc[h * kAnyKeys + tid] = -INFINITY;
+    }
+    __syncthreads();
+    if (warp < nh) {
+      float v[kAnyKeys / 32], mx = m;
+#pragma unroll
+      for (int i = 0; i < kAnyKeys / 32; ++i) {
+        v[i] = sc[warp * kAnyKeys + i * 32 + lane];
+        mx = fmaxf(mx, v[i]);
+      }
+      mx = warp_max_f32(mx);
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < kAnyKeys / 32; ++i) {
+        const float e = expf(v[i] - mx);
+        sc[warp * kAnyKeys + i * 32 + lane] = e;
+        sum += e;
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      const float a = m == -INFINITY ? 0.f : expf(m - mx);
+      l = l * a + sum;
+      m = mx;
+      if (lane == 0) s_alpha[warp] = a;
+    }
+    __syncthreads();
+    const int nk = min(kAnyKeys, pos + 1 - base);
+#pragma unroll
+    for (int a = 0; a < kAnyAcc; ++a) {
+      const int e = tid + a * 128;
+      if (e < nh * p.vdim) {
+        const int h = e / p.vdim, d = e - h * p.vdim;
+        const T* v = cache + (size_t)((h0 + h) / R) * p.vdim + d;
+        float x = acc[a] * s_alpha[h];
+        for (int kk = 0; kk < nk; ++kk) x = fmaf(sc[h * kAnyKeys + kk], to_f(v[vrow[kk]]), x);
+        acc[a] = x;
+      }
+    }
+  }
+  if (warp < nh && lane == 0) s_l[warp] = l;
+  __syncthreads();
+  T* o = reinterpret_cast<T*>(p.out) + (size_t)row * p.ldo + (size_t)h0 * p.vdim;
+#pragma unroll
+  for (int a = 0; a < kAnyAcc; ++a) {
+    const int e = tid + a * 128;
+    if (e < nh * p.vdim) {
+      const float ls = s_l[e / p.vdim];
+      o[e] = from_f<T>(ls > 0.f ? acc[a] / ls : 0.f);
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------- decode (bf16)
+__device__ __forceinline__ void ldsm_x4(uint32_t* r, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm_x2(uint32_t* r, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];"
+               : "=r"(r[0]), "=r"(r[1]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm_x4_trans(uint32_t* r, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma_bf16_16816(float* d, const uint32_t* a, const uint32_t* b) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+      "{%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+}
+// Untiled bulk copy global -> shared (16-byte aligned, a multiple of 16 bytes), counted on `bar`.
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+               ::"r"(smem_u32(dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
+}
+
+static constexpr int kDecKeys = 32;      // keys per tile
+static constexpr int kDecWarps = 8;
+static constexpr int kDecMaxStages = 4;
+
+struct DecodeSmem {                      // byte offsets
+  int q, k, v, s, p, stat, bars, total;
+};
+__host__ __device__ inline DecodeSmem decode_smem(int hp, int kwp, int vwp, int prow, int stages) {
+  DecodeSmem d;
+  int o = 0;
+  d.q = o; o += hp * (kwp + 8) * 2;
+  d.k = o; o += stages * kDecKeys * (kwp + 8) * 2;
+  d.v = o; o += stages * kDecKeys * (vwp + 8) * 2;
+  d.s = o; o += hp * (kDecKeys + 1) * 4;
+  o = (o + 15) & ~15;
+  d.p = o; o += prow * (kDecKeys + 8) * 2;
+  d.stat = o; o += 3 * hp * 4;
+  o = (o + 15) & ~15;
+  d.bars = o; o += kDecMaxStages * 8;
+  d.total = o;
+  return d;
+}
+
+// grid (request, split). MAXI: 16 x 8 output tiles a warp keeps in registers.
+template <int MAXI>
+__global__ void __launch_bounds__(kDecWarps * 32, 1) bias_attn_decode_kernel(BiasAttnParams p) {
+  extern __shared__ __align__(16) uint8_t dec_smem[];
+  const int prow = p.G * p.mt * 16;
+  const DecodeSmem L = decode_smem(p.hp, p.kwp, p.vwp, prow, p.stages);
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(dec_smem + L.q);
+  __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(dec_smem + L.k);
+  __nv_bfloat16* sV = reinterpret_cast<__nv_bfloat16*>(dec_smem + L.v);
+  float* sS = reinterpret_cast<float*>(dec_smem + L.s);
+  __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(dec_smem + L.p);
+  float* s_alpha = reinterpret_cast<float*>(dec_smem + L.stat);
+  float* s_m = s_alpha + p.hp;
+  float* s_l = s_m + p.hp;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(dec_smem + L.bars);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int b = blockIdx.x, split = blockIdx.y;
+  const int H = p.H, R = H / p.G, vw = p.G * p.vdim;
+  const int ks = p.kwp + 8, vs = p.vwp + 8, ps = kDecKeys + 8, ss = kDecKeys + 1;
+
+  // everything a product may read and no copy fills has to be finite: clear it once
+  for (int i = tid; i < L.s / 16; i += blockDim.x) reinterpret_cast<uint4*>(dec_smem)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < prow * ps / 8; i += blockDim.x) reinterpret_cast<uint4*>(sP)[i] = make_uint4(0, 0, 0, 0);
+  if (tid == 0) {
+    for (int i = 0; i < p.stages; ++i) mbar_init(&bars[i], 1);
+    mbar_fence_init();
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  const int seq_len = p.seq_lens[b], pos = seq_len - 1;
+  int chunk = (seq_len + p.splits - 1) / p.splits;
+  chunk = (chunk + kDecKeys - 1) / kDecKeys * kDecKeys;
+  const int t0 = split * chunk, t1 = min(seq_len, t0 + chunk);
+  const int ntiles = t1 > t0 ? (t1 - t0 + kDecKeys - 1) / kDecKeys : 0;
+  const bool counts_null = p.null_entry && split == 0;
+  for (int h = tid; h < p.hp; h += blockDim.x) {
+    s_m[h] = counts_null ? 0.f : -INFINITY;              // log2 domain
+    s_l[h] = counts_null ? 1.f : 0.f;
+  }
+  fence_proxy_async_smem();          // the clears are ordered before the copies that follow
+  __syncthreads();
+
+  const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(p.cache);
+  const int32_t* bt = p.block_table + (size_t)b * p.max_blocks;
+  auto load_tile = [&](int it) {     // warp 0: one key and one value row per lane
+    const int st = it % p.stages, tok0 = t0 + it * kDecKeys, n = min(kDecKeys, t1 - tok0);
+    if (lane == 0) mbar_expect_tx(&bars[st], (uint32_t)n * (p.kw + vw) * 2);
+    __syncwarp();
+    if (lane < n) {
+      const int tok = tok0 + lane;
+      const __nv_bfloat16* page = cache + (size_t)bt[tok / p.block_size] * p.block_size * (p.kw + vw);
+      const int off = tok % p.block_size;
+      bulk_load(sK + (size_t)(st * kDecKeys + lane) * ks, page + (size_t)off * p.kw, p.kw * 2, &bars[st]);
+      bulk_load(sV + (size_t)(st * kDecKeys + lane) * vs, page + (size_t)p.block_size * p.kw + (size_t)off * vw,
+                vw * 2, &bars[st]);
+    }
+  };
+  if (warp == 0)
+    for (int it = 0; it < min(p.stages, ntiles); ++it) load_tile(it);
+  {
+    const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(p.q) + (size_t)b * p.ldq;
+    const int n8 = p.kw / 8;
+    for (int h = warp; h < H; h += kDecWarps)
+      for (int i = lane; i < n8; i += 32)
+        *reinterpret_cast<uint4*>(sQ + (size_t)h * ks + i * 8) =
+            *reinterpret_cast<const uint4*>(q + (size_t)h * p.kw + i * 8);
+  }
+  __syncthreads();
+
+  const int n_vt = p.vdim / 8, items = p.G * p.mt * n_vt;
+  const int per_warp = (items + kDecWarps - 1) / kDecWarps;
+  const int i0 = warp * per_warp, cnt = max(0, min(items - i0, per_warp));
+  float o[MAXI][4];
+#pragma unroll
+  for (int i = 0; i < MAXI; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  const int s_tiles = (p.hp / 16) * (kDecKeys / 8);
+  bool ok = true;
+
+  for (int it = 0; it < ntiles; ++it) {
+    const int st = it % p.stages, tok0 = t0 + it * kDecKeys;
+    ok = mbar_wait(&bars[st], (it / p.stages) & 1, p.status);
+    if (!__syncthreads_and(ok)) { ok = false; break; }
+    // ---- scores: 16 heads x 8 keys per warp step
+    for (int x = warp; x < s_tiles; x += kDecWarps) {
+      const int mtile = x / (kDecKeys / 8), ntile = x % (kDecKeys / 8);
+      const uint32_t qa = smem_u32(sQ + (size_t)(mtile * 16 + (lane & 15)) * ks + (lane >> 4) * 8);
+      const uint32_t ka = smem_u32(sK + (size_t)(st * kDecKeys + ntile * 8 + (lane & 7)) * ks + ((lane >> 3) & 1) * 8);
+      float d0[4] = {0.f, 0.f, 0.f, 0.f}, d1[4] = {0.f, 0.f, 0.f, 0.f};
+      const int nk = p.kwp / 16;
+      int kk = 0;
+      for (; kk + 1 < nk; kk += 2) {
+        uint32_t a0[4], a1[4], b0[2], b1[2];
+        ldsm_x4(a0, qa + kk * 32);
+        ldsm_x2(b0, ka + kk * 32);
+        ldsm_x4(a1, qa + kk * 32 + 32);
+        ldsm_x2(b1, ka + kk * 32 + 32);
+        mma_bf16_16816(d0, a0, b0);
+        mma_bf16_16816(d1, a1, b1);
+      }
+      if (kk < nk) {
+        uint32_t a0[4], b0[2];
+        ldsm_x4(a0, qa + kk * 32);
+        ldsm_x2(b0, ka + kk * 32);
+        mma_bf16_16816(d0, a0, b0);
+      }
+      float* s0 = sS + (size_t)(mtile * 16 + (lane >> 2)) * ss + ntile * 8 + (lane & 3) * 2;
+      s0[0] = d0[0] + d1[0];
+      s0[1] = d0[1] + d1[1];
+      s0[8 * ss] = d0[2] + d1[2];
+      s0[8 * ss + 1] = d0[3] + d1[3];
+    }
+    __syncthreads();
+    // ---- softmax: one warp per head, one key per lane
+    for (int h = warp; h < H; h += kDecWarps) {
+      const int key = tok0 + lane;
+      float x = -INFINITY;
+      if (key < t1) {
+        x = sS[(size_t)h * ss + lane];
+        if (p.bias) x += __ldg(p.bias + (size_t)h * p.bias_len + min(pos - key, p.bias_len - 1));
+        x *= kLog2e;
+      }
+      const float mo = s_m[h], mn = fmaxf(mo, warp_max_f32(x));
+      const float e = exp2f(x - mn);
+      float sum = e;
+#pragma unroll
+      for (int k2 = 16; k2 > 0; k2 >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, k2);
+      const int g = h / R, r = h - g * R;
+      sP[(size_t)(g * p.mt * 16 + r) * ps + lane] = __float2bfloat16(e);
+      if (lane == 0) {
+        const float a = mo == -INFINITY ? 0.f : exp2f(mo - mn);
+        s_alpha[h] = a;
+        s_m[h] = mn;
+        s_l[h] = s_l[h] * a + sum;
+      }
+    }
+    __syncthreads();
+    // ---- outputs: each warp keeps its 16 x 8 tiles
+    uint32_t pa[2][4];
+    float al0 = 1.f, al1 = 1.f;
+    int cur = -1;
+#pragma unroll
+    for (int i = 0; i < MAXI; ++i) {
+      if (i < cnt) {
+        const int item = i0 + i, gm = item / n_vt, nt = item - gm * n_vt;
+        const int g = gm / p.mt, mi = gm - g * p.mt;
+        if (gm != cur) {
+          cur = gm;
+          const uint32_t a = smem_u32(sP + (size_t)(gm * 16 + (lane & 15)) * ps + (lane >> 4) * 8);
+          ldsm_x4(pa[0], a);
+          ldsm_x4(pa[1], a + 32);
+          const int r0 = mi * 16 + (lane >> 2);
+          al0 = r0 < R ? s_alpha[g * R + r0] : 0.f;
+          al1 = r0 + 8 < R ? s_alpha[g * R + r0 + 8] : 0.f;
+        }
+        uint32_t vb[4];
+        ldsm_x4_trans(vb, smem_u32(sV + (size_t)(st * kDecKeys + lane) * vs + g * p.vdim + nt * 8));
+        o[i][0] *= al0; o[i][1] *= al0; o[i][2] *= al1; o[i][3] *= al1;
+        mma_bf16_16816(o[i], pa[0], vb);
+        mma_bf16_16816(o[i], pa[1], vb + 2);
+      }
+    }
+    __syncthreads();
+    if (warp == 0 && it + p.stages < ntiles) load_tile(it + p.stages);
+  }
+  if (!ok) return;
+#pragma unroll
+  for (int i = 0; i < MAXI; ++i) {
+    if (i < cnt) {
+      const int item = i0 + i, gm = item / n_vt, nt = item - gm * n_vt;
+      const int g = gm / p.mt, mi = gm - g * p.mt;
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int r = mi * 16 + (lane >> 2) + half * 8;
+        if (r < R) {
+          const int h = g * R + r, d = nt * 8 + (lane & 3) * 2;
+          const float l = s_l[h], inv = l > 0.f ? 1.f / l : 0.f;
+          const float x0 = o[i][half * 2] * inv, x1 = o[i][half * 2 + 1] * inv;
+          if (p.splits == 1) {
+            *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)b * p.ldo +
+                                         (size_t)h * p.vdim + d) = pack_bf16x2(x0, x1);
+          } else {
+            float* t = p.tmp_o + (((size_t)b * H + h) * p.splits + split) * p.vdim + d;
+            t[0] = x0;
+            t[1] = x1;
+          }
+        }
+      }
+    }
+  }
+  if (p.splits > 1)
+    for (int h = tid; h < H; h += blockDim.x)
+      p.tmp_lse[((size_t)b * H + h) * p.splits + split] = s_l[h] > 0.f ? s_m[h] + log2f(s_l[h]) : -INFINITY;
+}
+
+// --------------------------------------------------------------------------------- prefill (bf16)
+// One CTA = one 128-row query tile of one request and one head. The query tile (all 64-wide chunks
+// of the query row) stays in shared memory; key tiles arrive chunk by chunk (64 keys x 64 dims) in a
+// ring, value tiles in a second ring of two. S is double-buffered in TMEM, O accumulates there.
+// Warps: 0 TMA producer, 1 MMA issuer + TMEM owner, 2..5 softmax (one thread per query row).
+static constexpr int kBQ = 128, kBKeys = 64, kChunkBytes = kBKeys * 128, kQChunkBytes = kBQ * 128;
+static constexpr int kVSlots = 2, kMaxKSlots = 8;
+
+struct alignas(8) BiasPrefillBars {
+  uint64_t q_full, k_full[kMaxKSlots], k_empty[kMaxKSlots], v_full[kVSlots], v_empty[kVSlots];
+  uint64_t s_full[2], s_empty[2], p_full, p_empty, o_full;
+  uint32_t tmem_base;
+};
+
+__device__ __forceinline__ float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+__global__ void __launch_bounds__(192)
+    bias_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+                             const __grid_constant__ CUtensorMap tmV, BiasAttnParams p) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int nkc = (p.kw + 63) / 64, nvc = (p.vdim + 63) / 64;
+  uint8_t* sQ = smem;
+  uint8_t* sK = sQ + nkc * kQChunkBytes;
+  uint8_t* sV = sK + p.k_slots * kChunkBytes;
+  uint8_t* sP = sV + kVSlots * nvc * kChunkBytes;
+  float* sB = reinterpret_cast<float*>(sP + kQChunkBytes);
+  BiasPrefillBars* bars =
+      reinterpret_cast<BiasPrefillBars*>(reinterpret_cast<uint8_t*>(sB) + ((p.bias_smem * 4 + 15) & ~15));
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int tile = blockIdx.x, h = blockIdx.y, hkv = h / (p.H / p.G);
+  const int req = p.tile_req[tile], q0 = p.tile_q0[tile];
+  const int q_begin = p.q_start[req], q_len = p.q_start[req + 1] - q_begin;
+  const int seq_len = p.seq_lens[req], ctx_off = seq_len - q_len;
+  const int rows = min(kBQ, q_len - q0);
+  const int ntiles = (ctx_off + q0 + rows - 1) / kBKeys + 1;
+  const uint32_t tmem_cols = p.vdim > 128 ? 512 : 256;
+
+  if (threadIdx.x == 0) {
+    mbar_init(&bars->q_full, 1);
+    for (int i = 0; i < p.k_slots; ++i) { mbar_init(&bars->k_full[i], 1); mbar_init(&bars->k_empty[i], 1); }
+    for (int i = 0; i < kVSlots; ++i) { mbar_init(&bars->v_full[i], 1); mbar_init(&bars->v_empty[i], 1); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&bars->s_full[i], 1); mbar_init(&bars->s_empty[i], 4); }
+    mbar_init(&bars->p_full, 4);
+    mbar_init(&bars->p_empty, 1);
+    mbar_init(&bars->o_full, 1);
+    mbar_fence_init();
+  }
+  if (warp == 1) { tmem_alloc(&bars->tmem_base, tmem_cols); tmem_relinquish(); }
+  const float* bias = p.bias ? p.bias + (size_t)h * p.bias_len : nullptr;
+  for (int i = threadIdx.x; i < p.bias_smem; i += blockDim.x) sB[i] = bias[i] * kLog2e;
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem_base = bars->tmem_base, tmem_s0 = tmem_base, tmem_o = tmem_base + 128;
+
+  if (warp == 0) {
+    if (lane == 0) {
+      tma_prefetch_desc(&tmQ);
+      tma_prefetch_desc(&tmK);
+      tma_prefetch_desc(&tmV);
+      mbar_expect_tx(&bars->q_full, nkc * kQChunkBytes);
+      for (int c = 0; c < nkc; ++c)
+        tma_load_2d(sQ + c * kQChunkBytes, &tmQ, &bars->q_full, h * p.kw + c * 64, q_begin + q0);
+      const int32_t* bt = p.block_table + (size_t)req * p.max_blocks;
+      const int nblk = (seq_len + p.block_size - 1) / p.block_size;
+      const int rpl = min(p.block_size, kBKeys), loads = kBKeys / rpl;
+      uint32_t kc = 0;
+      bool ok = true;
+      // Order K0 K1 V0 K2 V1 ... K(n-1) V(n-2) V(n-1): the order in which the MMA warp consumes them.
+      for (int j = 0; j <= ntiles && ok; ++j) {
+        if (j < ntiles) {
+          for (int c = 0; c < nkc && ok; ++c, ++kc) {
+            const int sl = kc % p.k_slots;
+            if (!mbar_wait(&bars->k_empty[sl], ((kc / p.k_slots) & 1) ^ 1, p.status)) { ok = false; break; }
+            mbar_expect_tx(&bars->k_full[sl], kChunkBytes);
+            for (int l = 0; l < loads; ++l) {
+              const int tk = j * kBKeys + l * rpl, bi = tk / p.block_size;
+              const int blk = max(bi < nblk ? bt[bi] : bt[0], 0);
+              tma_load_3d(sK + sl * kChunkBytes + l * rpl * 128, &tmK, &bars->k_full[sl], c * 64,
+                          tk % p.block_size, blk);
+            }
+          }
+        }
+        if (j >= 1 && ok) {
+          const int i = j - 1, sl = i % kVSlots;
+          if (!mbar_wait(&bars->v_empty[sl], ((i / kVSlots) & 1) ^ 1, p.status)) { ok = false; break; }
+          mbar_expect_tx(&bars->v_full[sl], nvc * kChunkBytes);
+          for (int l = 0; l < loads; ++l) {
+            const int tk = i * kBKeys + l * rpl, bi = tk / p.block_size;
+            const int blk = max(bi < nblk ? bt[bi] : bt[0], 0);
+            for (int c = 0; c < nvc; ++c)
+              tma_load_3d(sV + (sl * nvc + c) * kChunkBytes + l * rpl * 128, &tmV, &bars->v_full[sl],
+                          hkv * p.vdim + c * 64, tk % p.block_size, blk);
+          }
+        }
+      }
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      const uint32_t idesc_qk = umma_idesc_bf16(kBQ, kBKeys, 0, 0);
+      const uint32_t idesc_pv = umma_idesc_bf16(kBQ, (p.vdim + 15) & ~15, 0, 1);
+      bool ok = mbar_wait(&bars->q_full, 0, p.status);
+      const uint32_t q_addr = smem_u32(sQ), k_addr0 = smem_u32(sK), v_addr0 = smem_u32(sV), p_addr = smem_u32(sP);
+      uint32_t kc = 0;
+      for (int j = 0; j <= ntiles && ok; ++j) {
+        if (j < ntiles) {
+          const int sb = j & 1;
+          if (!mbar_wait(&bars->s_empty[sb], ((j >> 1) & 1) ^ 1, p.status)) { ok = false; break; }
+          for (int c = 0; c < nkc; ++c, ++kc) {
+            const int sl = kc % p.k_slots;
+            if (!mbar_wait(&bars->k_full[sl], (kc / p.k_slots) & 1, p.status)) { ok = false; break; }
+            tc_fence_after_sync();
+            const int steps = min(4, (p.kw - c * 64 + 15) / 16);
+            for (int kk = 0; kk < steps; ++kk)
+              umma_bf16_ss(tmem_s0 + sb * kBKeys, umma_desc_k_sw128(q_addr + c * kQChunkBytes + kk * 32, 1024),
+                           umma_desc_k_sw128(k_addr0 + sl * kChunkBytes + kk * 32, 1024), idesc_qk, (c | kk) != 0);
+            umma_commit(&bars->k_empty[sl]);
+          }
+          if (!ok) break;
+          umma_commit(&bars->s_full[sb]);
+        }
+        if (j >= 1) {
+          const int i = j - 1, sl = i % kVSlots;
+          if (!mbar_wait(&bars->v_full[sl], (i / kVSlots) & 1, p.status)) { ok = false; break; }
+          if (!mbar_wait(&bars->p_full, i & 1, p.status)) { ok = false; break; }
+          tc_fence_after_sync();
+          const uint32_t v_addr = v_addr0 + sl * nvc * kChunkBytes;
+#pragma unroll
+          for (int kk = 0; kk < kBKeys / 16; ++kk)
+            umma_bf16_ss(tmem_o, umma_desc_k_sw128(p_addr + kk * 32, 1024),
+                         umma_desc_mn_sw128(v_addr + kk * 2048, kChunkBytes, 1024), idesc_pv, (i | kk) != 0);
+          umma_commit(&bars->v_empty[sl]);
+          umma_commit(&bars->o_full);
+          umma_commit(&bars->p_empty);
+        }
+      }
+    }
+  } else {
+    const int quarter = warp & 3, r = quarter * 32 + lane;
+    const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
+    const int q_pos = ctx_off + q0 + r, hi = min(q_pos, seq_len - 1);
+    const int warp_pos0 = ctx_off + q0 + quarter * 32;       // position of the warp's first row
+    // m: reference maximum in the log2 domain, raised lazily (by more than 2^8). The null entry
+    // is the state before the first key: score 0, weight 1.
+    float m = p.null_entry ? 0.f : -INFINITY, l = p.null_entry ? 1.f : 0.f;
+    const float far = bias ? bias[p.bias_len - 1] * kLog2e : 0.f;
+    bool ok = true;
+    uint8_t* prow = sP + r * 128;
+    const int vcols = (p.vdim + 31) / 32;
+    for (int j = 0; j < ntiles && ok; ++j) {
+      const int sb = j & 1, kbase = j * kBKeys;
+      ok = __all_sync(0xffffffffu, mbar_wait(&bars->s_full[sb], (j >> 1) & 1, p.status));
+      if (!ok) break;
+      tc_fence_after_sync();
+      const uint32_t s_addr = tmem_s0 + sb * kBKeys + lane_off;
+      uint32_t s0[32], s1[32];
+      tmem_ld_32x32b_x32(s_addr, s0);
+      tmem_ld_32x32b_x32(s_addr + 32, s1);
+      tmem_ld_wait();
+      tc_fence_before_sync();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars->s_empty[sb]);
+      const bool need_mask = kbase + kBKeys - 1 > warp_pos0;                    // warp-uniform
+      const bool near = bias && warp_pos0 - (kbase + kBKeys - 1) < p.bias_len - 1;
+      if (near || need_mask) {
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          const int ka = kbase + i, kb = ka + 32;
+          float ba = far, bb = far;
+          if (near) {
+            const int da = min(max(q_pos - ka, 0), p.bias_len - 1), db = min(max(q_pos - kb, 0), p.bias_len - 1);
+            ba = p.bias_smem ? sB[da] : __ldg(bias + da) * kLog2e;
+            bb = p.bias_smem ? sB[db] : __ldg(bias + db) * kLog2e;
+          }
+          const float a = fmaf(__uint_as_float(s0[i]), kLog2e, ba), b = fmaf(__uint_as_float(s1[i]), kLog2e, bb);
+          s0[i] = __float_as_uint(ka > hi ? -INFINITY : a);
+          s1[i] = __float_as_uint(kb > hi ? -INFINITY : b);
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          s0[i] = __float_as_uint(fmaf(__uint_as_float(s0[i]), kLog2e, far));
+          s1[i] = __float_as_uint(fmaf(__uint_as_float(s1[i]), kLog2e, far));
+        }
+      }
+      float mx0 = -INFINITY, mx1 = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        mx0 = fmaxf(mx0, __uint_as_float(s0[i]));
+        mx1 = fmaxf(mx1, __uint_as_float(s1[i]));
+      }
+      const float tile_max = fmaxf(mx0, mx1);
+      float alpha = 1.f;
+      bool rescale = false;
+      if (tile_max > m + 8.f) {
+        if (m != -INFINITY) { alpha = ex2_approx(m - tile_max); rescale = j > 0; }
+        m = tile_max;
+      }
+      const float m_use = m == -INFINITY ? 0.f : m;
+      ok = __all_sync(0xffffffffu, mbar_wait(&bars->p_empty, (j & 1) ^ 1, p.status));
+      if (!ok) break;
+      if (__any_sync(0xffffffffu, rescale)) {
+        tc_fence_after_sync();
+        for (int c = 0; c < vcols; ++c) {
+          uint32_t rr[32];
+          tmem_ld_32x32b_x32(tmem_o + lane_off + c * 32, rr);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) rr[i] = __float_as_uint(__uint_as_float(rr[i]) * alpha);
+          tmem_st_32x32b_x32(tmem_o + lane_off + c * 32, rr);
+        }
+        tmem_st_wait();
+      }
+      float rs0 = 0.f, rs1 = 0.f;
+#pragma unroll
+      for (int c = 0; c < 8; ++c) {
+        uint32_t pk[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int i = (c & 3) * 8 + e * 2;
+          const float x0 = __uint_as_float(c < 4 ? s0[i] : s1[i]), x1 = __uint_as_float(c < 4 ? s0[i + 1] : s1[i + 1]);
+          const float p0 = ex2_approx(x0 - m_use), p1 = ex2_approx(x1 - m_use);
+          rs0 += p0;
+          rs1 += p1;
+          pk[e] = pack_bf16x2(p0, p1);
+        }
+        *reinterpret_cast<uint4*>(prow + ((c ^ (r & 7)) << 4)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+      }
+      l = l * alpha + (rs0 + rs1);
+      fence_proxy_async_smem();
+      tc_fence_before_sync();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars->p_full);
+    }
+    if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->o_full, (ntiles - 1) & 1, p.status));
+    if (ok) {
+      tc_fence_after_sync();
+      const float inv = l > 0.f ? 1.f / l : 0.f;
+      __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(q_begin + q0 + r) * p.ldo + (size_t)h * p.vdim;
+      for (int c = 0; c < vcols; ++c) {
+        uint32_t rr[32];
+        tmem_ld_32x32b_x32(tmem_o + lane_off + c * 32, rr);
+        tmem_ld_wait();
+        if (r < rows) {
+#pragma unroll
+          for (int i = 0; i < 32; i += 8) {
+            if (c * 32 + i < p.vdim) {
+              uint4 w;
+              w.x = pack_bf16x2(__uint_as_float(rr[i + 0]) * inv, __uint_as_float(rr[i + 1]) * inv);
+              w.y = pack_bf16x2(__uint_as_float(rr[i + 2]) * inv, __uint_as_float(rr[i + 3]) * inv);
+              w.z = pack_bf16x2(__uint_as_float(rr[i + 4]) * inv, __uint_as_float(rr[i + 5]) * inv);
+              w.w = pack_bf16x2(__uint_as_float(rr[i + 6]) * inv, __uint_as_float(rr[i + 7]) * inv);
+              *reinterpret_cast<uint4*>(dst + c * 32 + i) = w;
+            }
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  if (warp == 1) tmem_dealloc(tmem_base, tmem_cols);
+}
+
+// ------------------------------------------------------------------------------------ host helpers
+static bool decode_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem, int& maxi) {
+  if (a->f32 || (a->kw & 7) || (a->vdim & 7) || (a->ldq & 7) || (a->ldo & 1)) return false;
+  if (((uintptr_t)a->q | (uintptr_t)a->cache) & 15) return false;
+  const int R = a->H / a->G;
+  p.kwp = (a->kw + 15) & ~15;
+  p.vwp = a->G * a->vdim;
+  p.mt = (R + 15) / 16;
+  p.hp = (a->H + 15) & ~15;
+  const int per_warp = (a->G * p.mt * (a->vdim / 8) + kDecWarps - 1) / kDecWarps;
+  if (per_warp > 32) return false;
+  maxi = per_warp <= 4 ? 4 : per_warp <= 8 ? 8 : per_warp <= 16 ? 16 : 32;
+  for (p.stages = kDecMaxStages; p.stages >= 2; --p.stages) {
+    smem = (size_t)decode_smem(p.hp, p.kwp, p.vwp, a->G * p.mt * 16, p.stages).total;
+    if (smem <= 225 * 1024) return true;
+  }
+  return false;
+}
+
+static bool prefill_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem) {
+  if (a->f32 || !a->tile_req || (a->kw & 7) || (a->vdim & 7) || a->vdim > 256 || (a->ldq & 7) || (a->ldo & 7)) return false;
+  if (((uintptr_t)a->q | (uintptr_t)a->cache | (uintptr_t)a->out) & 15) return false;
+  const int bs = a->block_size;
+  if (bs < 8 || (bs & 7) || (bs < kBKeys && kBKeys % bs) || (bs > kBKeys && bs % kBKeys)) return false;
+  const int nkc = (a->kw + 63) / 64, nvc = (a->vdim + 63) / 64;
+  p.bias_smem = a->bias && a->bias_len <= 1024 ? a->bias_len : 0;
+  const size_t fixed = (size_t)nkc * kQChunkBytes + kVSlots * nvc * kChunkBytes + kQChunkBytes +
+                       ((p.bias_smem * 4 + 15) & ~15) + sizeof(BiasPrefillBars) + 1024;
+  const size_t limit = 226 * 1024;
+  if (fixed + 2 * kChunkBytes > limit) return false;
+  // two CTAs on an SM where the query rows are short enough, else as deep a key ring as fits
+  int slots = fixed + 3 * kChunkBytes <= 112 * 1024 ? (int)((112 * 1024 - fixed) / kChunkBytes)
+                                                    : (int)((limit - fixed) / kChunkBytes);
+  p.k_slots = slots > kMaxKSlots ? kMaxKSlots : slots;
+  smem = fixed + (size_t)p.k_slots * kChunkBytes;
+  return true;
+}
+
+struct PageMapKey {
+  const void* base;
+  uint64_t blocks;
+  int bs, kw, vw;
+  bool operator==(const PageMapKey& o) const {
+    return base == o.base && blocks == o.blocks && bs == o.bs && kw == o.kw && vw == o.vw;
+  }
+};
+struct PageMapHash {
+  size_t operator()(const PageMapKey& k) const {
+    return reinterpret_cast<size_t>(k.base) ^ (k.blocks * 0x9e3779b97f4a7c15ull) ^ ((size_t)k.bs << 40) ^
+           ((size_t)k.kw << 20) ^ (size_t)k.vw;
+  }
+};
+
+// Tensor maps of the key and the value part of a page, built once per cache.
+static bool page_maps(const B200BiasAttn* a, CUtensorMap* mk, CUtensorMap* mv) {
+  static std::mutex mu;
+  static std::unordered_map<PageMapKey, std::pair<CUtensorMap, CUtensorMap>, PageMapHash> maps;
+  const int vw = a->G * a->vdim;
+  PageMapKey key{a->cache, (uint64_t)a->num_blocks, a->block_size, a->kw, vw};
+  std::lock_guard<std::mutex> lock(mu);
+  auto it = maps.find(key);
+  if (it == maps.end()) {
+    if (maps.size() > 4096) maps.clear();
+    const uint64_t page = (uint64_t)a->block_size * (a->kw + vw) * 2;
+    const uint32_t rows = a->block_size < kBKeys ? a->block_size : kBKeys;
+    const uint8_t* base = reinterpret_cast<const uint8_t*>(a->cache);
+    CUtensorMap k, v;
+    if (!encode_tmap_3d(&k, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a->kw, a->block_size, a->num_blocks,
+                        (uint64_t)a->kw * 2, page, 64, rows, 1, CU_TENSOR_MAP_SWIZZLE_128B) ||
+        !encode_tmap_3d(&v, base + (size_t)a->block_size * a->kw * 2, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, vw,
+                        a->block_size, a->num_blocks, (uint64_t)vw * 2, page, 64, rows, 1, CU_TENSOR_MAP_SWIZZLE_128B))
+      return false;
+    it = maps.emplace(key, std::make_pair(k, v)).first;
+  }
+  *mk = it->second.first;
+  *mv = it->second.second;
+  return true;
+}
+
+static BiasAttnParams common_params(const B200BiasAttn* a) {
+  BiasAttnParams p{};
+  p.q = a->q; p.ldq = a->ldq; p.out = a->out; p.ldo = a->ldo; p.cache = a->cache;
+  p.block_table = (const int32_t*)a->block_table; p.max_blocks = a->max_blocks;
+  p.seq_lens = (const int32_t*)a->seq_lens; p.q_start = (const int32_t*)a->q_start;
+  p.num_reqs = a->num_reqs; p.rows = a->rows;
+  p.H = a->H; p.G = a->G; p.kw = a->kw; p.vdim = a->vdim; p.block_size = a->block_size;
+  p.bias = (const float*)a->bias; p.bias_len = a->bias_len; p.null_entry = a->null_entry;
+  p.splits = a->splits < 1 ? 1 : a->splits; p.tmp_o = (float*)a->tmp_o; p.tmp_lse = (float*)a->tmp_lse;
+  p.tile_req = (const int32_t*)a->tile_req; p.tile_q0 = (const int32_t*)a->tile_q0;
+  p.status = device_status_word();
+  return p;
+}
+
+template <typename T>
+static int launch_any(const BiasAttnParams& p, cudaStream_t stream) {
+  if ((long)kAnyHeads * p.vdim > 128l * kAnyAcc) return -4;
+  const size_t smem = (size_t)kAnyHeads * (p.kw + kAnyKeys) * 4;
+  if (smem > 200 * 1024) return -4;
+  static PerDeviceOnce once;
+  if (once.first()) cudaFuncSetAttribute(bias_attn_any_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+  dim3 grid(p.rows, (p.H + kAnyHeads - 1) / kAnyHeads);
+  return launch_pdl(bias_attn_any_kernel<T>, grid, dim3(128), smem, stream, p) == cudaSuccess ? 0 : -2;
+}
+
+template <int MAXI>
+static int launch_decode_mma(const BiasAttnParams& p, size_t smem, cudaStream_t stream) {
+  static PerDeviceOnce once;
+  if (once.first()) cudaFuncSetAttribute(bias_attn_decode_kernel<MAXI>, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024);
+  return launch_pdl(bias_attn_decode_kernel<MAXI>, dim3(p.rows, p.splits), dim3(kDecWarps * 32), smem, stream, p) ==
+                 cudaSuccess ? 0 : -2;
+}
+
+template <typename TO, int TOK>
+static int launch_mix(const MixParams& p, int gy, cudaStream_t stream) {
+  const size_t smem = ((size_t)kMixHeads * p.H + (size_t)TOK * p.H * p.dim) * 4;
+  if (smem > 220 * 1024) return -4;
+  static PerDeviceOnce once;
+  if (once.first())
+    cudaFuncSetAttribute(head_mix_kv_kernel<TO, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+  return launch_pdl(head_mix_kv_kernel<TO, TOK>, dim3((p.T + TOK - 1) / TOK, gy), dim3(256), smem, stream, p) ==
+                 cudaSuccess ? 0 : -2;
+}
+
+static bool valid_args(const B200BiasAttn* a) {
+  return a->H > 0 && a->G > 0 && a->H % a->G == 0 && a->kw > 0 && a->vdim > 0 && a->block_size > 0 &&
+         (!a->bias || a->bias_len > 0);
+}
+
+}  // namespace b200
+
+using namespace b200;
+
+extern "C" {
+
+int b200_head_mix_kv(const void* qkv, long long ld, const void* mix, void* q_out, long long ldq, const void* slots,
+                     void* cache, int H, int G, int dim, int vdim, int block_size, int T, int f32, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || block_size <= 0) return -1;
+  MixParams p{(const float*)qkv, ld, (const float*)mix, q_out, ldq, (const int64_t*)slots, cache, H, G, dim, vdim,
+              block_size, T};
+  // few tokens: one per CTA, so that more SMs take part
+  const int gy = (H + kMixHeads - 1) / kMixHeads;
+  const size_t wide = ((size_t)kMixHeads * H + 4 * (size_t)H * dim) * 4;
+  const bool narrow = wide > 220 * 1024 || (long)((T + 3) / 4) * gy < 2l * b200_num_sms();
+  if (f32) return narrow ? launch_mix<float, 1>(p, gy, stream) : launch_mix<float, 4>(p, gy, stream);
+  return narrow ? launch_mix<__nv_bfloat16, 1>(p, gy, stream) : launch_mix<__nv_bfloat16, 4>(p, gy, stream);
+}
+
+// 2: tensor-core kernels for this shape, 1: the any-size kernel only. phase 0 decode, 1 prefill.
+int b200_bias_attn_kernel(const B200BiasAttn* a, int phase) {
+  BiasAttnParams p{};
+  size_t smem;
+  int maxi;
+  if (!valid_args(a)) return 0;
+  return (phase == 0 ? decode_plan(a, p, smem, maxi) : prefill_plan(a, p, smem)) ? 2 : 1;
+}
+
+int b200_bias_attn_decode(const B200BiasAttn* a, int any_size, cudaStream_t stream) {
+  if (a->rows <= 0) return 0;
+  if (!valid_args(a)) return -1;
+  BiasAttnParams p = common_params(a);
+  p.q_start = nullptr;
+  size_t smem;
+  int maxi;
+  if (any_size || !decode_plan(a, p, smem, maxi))
+    return a->f32 ? launch_any<float>(p, stream) : launch_any<__nv_bfloat16>(p, stream);
+  if (p.splits > 1 && (!p.tmp_o || !p.tmp_lse)) return -1;
+  const int rc = maxi == 4 ? launch_decode_mma<4>(p, smem, stream) : maxi == 8 ? launch_decode_mma<8>(p, smem, stream)
+               : maxi == 16 ? launch_decode_mma<16>(p, smem, stream) : launch_decode_mma<32>(p, smem, stream);
+  if (rc || p.splits == 1) return rc;
+  return b200_attn_decode_merge(p.tmp_o, p.tmp_lse, p.out, (int)p.ldo, p.rows, p.H, p.vdim, p.splits, stream);
+}
+
+int b200_bias_attn_prefill(const B200BiasAttn* a, int any_size, cudaStream_t stream) {
+  if (a->rows <= 0) return 0;
+  if (!valid_args(a) || !a->q_start) return -1;
+  BiasAttnParams p = common_params(a);
+  size_t smem;
+  if (any_size || !prefill_plan(a, p, smem))
+    return a->f32 ? launch_any<float>(p, stream) : launch_any<__nv_bfloat16>(p, stream);
+  if (a->num_tiles <= 0) return 0;
+  CUtensorMap tmQ, tmK, tmV;
+  if (!encode_tmap_2d(&tmQ, a->q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)a->rows, (uint64_t)a->H * a->kw,
+                      (uint64_t)a->ldq, kBQ, 64, CU_TENSOR_MAP_SWIZZLE_128B) ||
+      !page_maps(a, &tmK, &tmV))
+    return -3;
+  static PerDeviceOnce once;
+  if (once.first()) cudaFuncSetAttribute(bias_attn_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+  bias_attn_prefill_kernel<<<dim3(a->num_tiles, a->H), 192, smem, stream>>>(tmQ, tmK, tmV, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+
+}  // extern "C"

@@ -247,6 +247,13 @@ __global__ void __launch_bounds__(128)
   for (int i = threadIdx.x; i < (H >> 3); i += blockDim.x) d[i] = s[i];
 }
 
+// row_w[pos] = weight of the (token, expert) pair that was sorted to pos
+__global__ void moe_row_weights_kernel(const int32_t* __restrict__ pair_pos, const float* __restrict__ topk_w, int P,
+                                       float* row_w) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < P && pair_pos[i] >= 0) row_w[pair_pos[i]] = topk_w[i];
+}
+
 // ------------------------------------------------------------------------------ grouped GEMM
 static constexpr int kGBM = 128, kGBK = 64, kGMaxStages = 8;
 struct GroupedParams {
@@ -264,6 +271,7 @@ struct GroupedParams {
   // merged projection never reaches memory. Both values are rounded to bf16 first, as the separate
   // activation kernel would see them.
   int act_fuse;
+  B200ClampedGate clamp;    // act_fuse == 4: clamped pair, applied to the fp32 accumulators
   int* status;
 };
 struct alignas(8) GroupedBars {
@@ -346,7 +354,27 @@ __global__ void __launch_bounds__(192, 1)
     const int n = tn * kGBM + quarter * 32 + lane;        // output column of this thread
     const uint32_t ta = tmem_base + ((uint32_t)(quarter * 32) << 16);
     const int kind = p.act_fuse - 1;
-    if (ok) {
+    if (ok && kind == 3) {
+      for (int c = 0; c < np / 16; ++c) {
+        uint32_t g[16], u[16];
+        tmem_ld_32x32b_x16(ta + c * 16, g);
+        tmem_ld_32x32b_x16(ta + 256 + c * 16, u);
+        tmem_ld_wait();
+        if (n < half_n) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            const int m = c * 16 + i;
+            if (m < rows) {
+              const float w = p.clamp.row_w ? __ldg(p.clamp.row_w + row0 + m) : 1.f;
+              const float gg = fminf(__uint_as_float(g[i]) * w, p.clamp.limit);
+              const float uu = fminf(fmaxf(__uint_as_float(u[i]) * w, -p.clamp.limit), p.clamp.limit);
+              p.out[(size_t)(row0 + m) * half_n + n] =
+                  __float2bfloat16(gg / (1.f + __expf(-p.clamp.alpha * gg)) * (uu + p.clamp.up_offset));
+            }
+          }
+        }
+      }
+    } else if (ok) {
       for (int c = 0; c < np / 16; ++c) {
         uint32_t g[16], u[16];
         tmem_ld_32x32b_x16(ta + c * 16, g);
@@ -551,10 +579,11 @@ int b200_moe_gather(const void* x, int ldx, const void* sorted_token, const void
 static int moe_grouped_gemm_impl(const void* xs, int max_rows, const void* W, int E, int N, int K,
                                  void* out, const void* chunk_expert, const void* chunk_row0,
                                  const void* chunk_n, const void* meta, int max_chunks, int act_fuse,
-                                 cudaStream_t stream) {
+                                 cudaStream_t stream, const B200ClampedGate* clamp = nullptr) {
   if (max_rows <= 0) return 0;
   if ((K & 7) || (N & 7)) return -1;
-  if (act_fuse && ((N & 1) || ((N / 2) & 7) || act_fuse < 1 || act_fuse > 3)) return -1;
+  if (act_fuse && ((N & 1) || ((N / 2) & 7) || act_fuse < 1 || act_fuse > 4 || (act_fuse == 4) != (clamp != nullptr)))
+    return -1;
   static std::mutex mu;
   CUtensorMap tmW, tmX;
   if (!encode_tmap_3d(&tmW, W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)K, (uint64_t)N,
@@ -574,6 +603,7 @@ static int moe_grouped_gemm_impl(const void* xs, int max_rows, const void* W, in
   const int nkb = (K + kGBK - 1) / kGBK;
   if (stages > nkb) stages = nkb < 2 ? 2 : nkb;
   p.stages = stages; p.act_fuse = act_fuse; p.status = device_status_word();
+  if (clamp) p.clamp = *clamp;
   const size_t smem = (size_t)stages * stage + 1024 + sizeof(GroupedBars);
   static PerDeviceOnce attr_once;
   if (attr_once.first()) {
@@ -600,6 +630,22 @@ int b200_moe_grouped_gemm_gated(const void* xs, int max_rows, const void* W, int
                                 cudaStream_t stream) {
   return moe_grouped_gemm_impl(xs, max_rows, W, E, N, K, out, chunk_expert, chunk_row0, chunk_n, meta, max_chunks,
                                kind + 1, stream);
+}
+// Same with the clamped pair as the activation (B200ClampedGate); a routing weight that scales the
+// expert's input is applied here, to the accumulators: W (w x) = w (W x).
+int b200_moe_grouped_gemm_clamped(const void* xs, int max_rows, const void* W, int E, int N, int K,
+                                  void* out, const void* chunk_expert, const void* chunk_row0,
+                                  const void* chunk_n, const void* meta, int max_chunks,
+                                  const B200ClampedGate* act, cudaStream_t stream) {
+  if (!act) return -1;
+  return moe_grouped_gemm_impl(xs, max_rows, W, E, N, K, out, chunk_expert, chunk_row0, chunk_n, meta, max_chunks, 4,
+                               stream, act);
+}
+int b200_moe_row_weights(const void* pair_pos, const void* topk_w, int P, void* row_w, cudaStream_t stream) {
+  if (P <= 0) return 0;
+  moe_row_weights_kernel<<<(P + 255) / 256, 256, 0, stream>>>((const int32_t*)pair_pos, (const float*)topk_w, P,
+                                                            (float*)row_w);
+  RETL;
 }
 
 

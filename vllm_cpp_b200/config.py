@@ -41,6 +41,33 @@ class RopeConfig:
 
 
 @dataclass
+class AttentionSpec:
+    """Mixer of one decoder block: grouped heads with separate key and value sizes, a distance bias
+    that saturates at ``bias_max``."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    bias_max: int
+
+
+@dataclass
+class ExpertSpec:
+    """Feed-forward of one decoder block: ``top`` of ``experts`` clamped gated units."""
+    experts: int
+    top: int
+    ff: int
+    limit: float
+
+
+@dataclass
+class BlockSpec:
+    attention: AttentionSpec
+    mlp: Optional[ExpertSpec] = None
+
+
+@dataclass
 class ModelConfig:
     architecture: str = "LlamaForCausalLM"
     vocab_size: int = 32000
@@ -106,6 +133,8 @@ class ModelConfig:
     dtype: str = "bfloat16"
     eos_token_id: Optional[int] = None
     bos_token_id: Optional[int] = None
+    # block-by-block sizes of the families whose config.json lists every layer (None: uniform)
+    blocks: Optional[list] = None
     raw: dict = field(default_factory=dict)
 
     @property
@@ -268,9 +297,70 @@ def model_config_from_hf(cfg: dict) -> ModelConfig:
     return m
 
 
+def model_config_from_blocks(cfg: dict) -> ModelConfig:
+    """ModelConfig of a config.json that names one ``architecture`` and lists its ``layers``, each
+    with a mixer and a feed-forward (or null)."""
+    arch = cfg["architecture"]
+    if arch != "Nufusun":
+        raise ValueError(f"no reader for the layer list of architecture {arch!r}")
+    blocks = []
+    for i, l in enumerate(cfg["layers"]):
+        if l["type"] != "attention":
+            raise ValueError(f"layer {i}: unknown mixer {l['type']!r}")
+        m = l["mixer"]
+        att = AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
+                            vdim=int(m["vdim"]), scale=float(m["scale"]), bias_max=int(m["bias_max"]))
+        if att.heads % att.kv_heads:
+            raise ValueError(f"layer {i}: {att.heads} heads do not divide into {att.kv_heads} groups")
+        mlp = None
+        if l.get("mlp") is not None:
+            f = l["mlp"]
+            if f["kind"] != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward {f['kind']!r}")
+            mlp = ExpertSpec(experts=int(f["router"]["experts"]), top=int(f["router"]["top"]),
+                             ff=int(f["expert"]["ff"]), limit=float(f["expert"]["limit"]))
+            if not 1 <= mlp.top <= mlp.experts:
+                raise ValueError(f"layer {i}: {mlp.top} of {mlp.experts} experts")
+        blocks.append(BlockSpec(att, mlp))
+    return model_config_of_blocks(arch, blocks, vocab=int(cfg["vocab"]), width=int(cfg["width"]),
+                                  eps=float(cfg["norm"]["eps"]), embed_scale=float(cfg["embedding"]["scale"]), raw=cfg)
+
+
+def model_config_of_blocks(arch: str, blocks: list, *, vocab: int, width: int, eps: float, embed_scale: float,
+                           max_position: int = 32768, raw: Optional[dict] = None) -> ModelConfig:
+    att, moe = [b.attention for b in blocks], [b.mlp for b in blocks if b.mlp is not None]
+    return ModelConfig(
+        architecture=arch, vocab_size=vocab, hidden_size=width, num_layers=len(blocks),
+        intermediate_size=max([m.ff * m.top for m in moe], default=0), num_heads=max(a.heads for a in att),
+        num_kv_heads=max(a.kv_heads for a in att), head_dim=max(a.dim for a in att),
+        v_head_dim=max(a.vdim for a in att), rms_norm_eps=eps, embed_scale=embed_scale, gemma_norm=True,
+        attention_bias=True, hidden_act="clamped_gate", scoring_func="sigmoid", norm_topk_prob=False,
+        num_experts=max([m.experts for m in moe], default=0), num_experts_per_tok=max([m.top for m in moe], default=0),
+        moe_intermediate_size=max([m.ff for m in moe], default=0), max_position_embeddings=max_position,
+        blocks=blocks, raw=raw or {})
+
+
+def block_config_dict(cfg: ModelConfig) -> dict:
+    """config.json of a ModelConfig with ``blocks`` (the inverse of model_config_from_blocks)."""
+    layers = []
+    for b in cfg.blocks:
+        a, m = b.attention, b.mlp
+        layers.append({
+            "type": "attention",
+            "mixer": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale,
+                      "bias_max": a.bias_max},
+            "mlp": None if m is None else {"kind": "moe", "router": {"experts": m.experts, "top": m.top},
+                                           "expert": {"ff": m.ff, "limit": m.limit}}})
+    return {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_size,
+            "norm": {"eps": cfg.rms_norm_eps}, "embedding": {"scale": cfg.embed_scale}, "layers": layers}
+
+
 def load_model_config(model_dir: str) -> ModelConfig:
     with open(os.path.join(model_dir, "config.json")) as f:
-        return model_config_from_hf(json.load(f))
+        raw = json.load(f)
+    if "architecture" in raw and "layers" in raw:
+        return model_config_from_blocks(raw)
+    return model_config_from_hf(raw)
 
 
 # ------------------------------------------------------------------ named synthetic shapes
@@ -329,6 +419,17 @@ def synthetic_config(name: str) -> ModelConfig:
                            linear_num_key_heads=16, linear_num_value_heads=48,
                            linear_key_head_dim=128, linear_value_head_dim=128,
                            linear_conv_kernel_dim=4, quant="nvfp4")
+    if n in ("nufusun-30b-a3b",):
+        # the layer sizes of qwen3-coder-30b-a3b
+        b = BlockSpec(AttentionSpec(heads=32, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, bias_max=1024),
+                      ExpertSpec(experts=128, top=8, ff=768, limit=7.0))
+        return model_config_of_blocks("Nufusun", [b] * 48, vocab=151936, width=2048, eps=1e-6, embed_scale=1.0,
+                                      max_position=262144)
+    if n == "tiny-nufusun":
+        b = BlockSpec(AttentionSpec(heads=6, kv_heads=3, dim=32, vdim=48, scale=0.2, bias_max=60),
+                      ExpertSpec(experts=5, top=2, ff=64, limit=2.0))
+        return model_config_of_blocks("Nufusun", [b, BlockSpec(b.attention), b], vocab=500, width=192, eps=1e-5,
+                                      embed_scale=2.0, max_position=2048)
     if n.startswith("tiny"):
         # small shapes for tests: tiny-dense, tiny-moe, tiny-mla, tiny-gdn
         base = dict(vocab_size=512, hidden_size=256, intermediate_size=512, num_layers=2,
@@ -433,6 +534,11 @@ class EngineArgs:
     # the packed form (integer block dot products); None keeps bf16 weights
     cpu_weight_quant: Optional[str] = None
     enable_cuda_graphs: bool = True
+    # "auto": the checkpoint's type (bf16). "float32": weights, activations, cache and products in
+    # 32 bits, for the models that support it
+    dtype: str = "auto"
+    # logits rows per step for positions asked for with LLM.score_positions (besides the sampled ones)
+    max_score_rows: int = 0
     seed: int = 0
     device: str = "cuda"
     parallel: ParallelConfig = field(default_factory=ParallelConfig)

@@ -76,6 +76,12 @@ class LLM:
         max_len = args.max_model_len or cfg.max_position_embeddings
         self.max_model_len = max_len
         _, cls = registry.resolve(cfg.architecture)
+        if args.dtype != "auto":
+            if args.dtype not in cls.DTYPES:
+                raise ValueError(f"{cfg.architecture} runs in {', '.join(cls.DTYPES)}, not in {args.dtype}")
+            cfg.dtype = args.dtype
+        if args.max_score_rows and par.tensor_parallel_size > 1:
+            raise ValueError("scored positions need the whole vocabulary on one rank")
         self.model = cls(cfg, device=device, parallel=par, comm=self.comm, max_position=max_len)
         if torch.device(device).type == "cpu" and args.cpu_backend == "native":
             from ..models.backend import CpuNativeBackend
@@ -133,7 +139,8 @@ class LLM:
         self.runner = ModelRunner(self.model, block_size=args.block_size, num_blocks=num_blocks,
                                   max_num_seqs=args.max_num_seqs, max_num_batched_tokens=budget,
                                   max_model_len=max_len, enable_cuda_graphs=args.enable_cuda_graphs,
-                                  async_mode=use_async, speculative_config=spec, step_channel=channel)
+                                  async_mode=use_async, speculative_config=spec, step_channel=channel,
+                                  max_score_rows=args.max_score_rows)
         if spec is not None and spec.method == "mtp":
             from ..models.gdn_mtp import Qwen35MTP
             mtp = Qwen35MTP(self.model, getattr(cfg, "mtp_num_hidden_layers", 1) or 1)
@@ -182,6 +189,7 @@ class LLM:
         self.use_async = use_async
         self._counter = itertools.count()
         self._states: dict[str, RequestOutput] = {}
+        self._open: set[str] = set()          # requests whose input is still open
         self.eos_token_id = cfg.eos_token_id
         self.step_times: list = []
 
@@ -261,7 +269,8 @@ class LLM:
     # ------------------------------------------------------------------ LLMEngine surface
     def add_request(self, prompt_token_ids: Sequence[int], params: "E.SamplingParams",
                     request_id: Optional[str] = None, priority: int = 0,
-                    prompt: Optional[str] = None) -> str:
+                    prompt: Optional[str] = None, input_open: bool = False) -> str:
+        """``input_open``: the prompt arrives in portions, see :meth:`extend_request`."""
         if not self.is_driver:
             raise RuntimeError("this rank owns no scheduler: requests go to rank 0")
         rid = request_id or f"req-{next(self._counter)}"
@@ -269,12 +278,16 @@ class LLM:
         if len(toks) >= self.max_model_len:
             raise ValueError(f"prompt ({len(toks)} tokens) is longer than max_model_len "
                              f"({self.max_model_len})")
-        req = E.EngineCoreRequest(rid, toks, params, self.eos_token_id, time.monotonic(), priority)
+        if not toks:
+            raise ValueError("empty prompt")
+        req = E.EngineCoreRequest(rid, toks, params, self.eos_token_id, time.monotonic(), priority, input_open)
         self.runner.set_eos(rid, self.eos_token_id)
         if self.structured is not None and params.structured_outputs is not None \
                 and params.structured_outputs.any():
             self.structured.validate(params.structured_outputs)    # raises on a bad constraint
         self.core.add_request(req)
+        if input_open:
+            self._open.add(rid)
         st = RequestOutput(rid, toks, [CompletionOutput()], prompt=prompt)
         if self.tokenizer is not None and params.detokenize:
             st.detok = E.IncrementalDetokenizer(self.tokenizer, toks, params.skip_special_tokens,
@@ -284,9 +297,34 @@ class LLM:
         self._states[rid] = st
         return rid
 
+    def extend_request(self, request_id: str, tokens: Sequence[int], close: bool = False) -> None:
+        """Further prompt tokens of a request that was added with ``input_open=True``. Its steps compute
+        what has arrived and keep the cache; it samples once its input is closed (with the last
+        tokens). ``abort_request`` gives back what it holds."""
+        toks = list(tokens)
+        self.core.scheduler().append_input(request_id, toks, close)
+        if close:
+            self._open.discard(request_id)
+        st = self._states.get(request_id)
+        if st is not None:
+            st.prompt_token_ids.extend(toks)
+
+    def score_positions(self, request_id: str, positions: Sequence[int]) -> None:
+        """Asks for the logits of positions of a request that no step has computed yet (the request
+        may still be unknown); they are collected by :meth:`take_scores`. A request that is scored
+        should set ``prompt_logprobs``, so that no position is taken from the prefix cache."""
+        if not self.args.max_score_rows:
+            raise ValueError("EngineArgs.max_score_rows is 0")
+        self.runner.batch.set_score_positions(request_id, list(positions))
+
+    def take_scores(self) -> dict:
+        """request id -> [(position, fp32 logits)] of the scored positions computed since the last call."""
+        return self.runner.take_scores()
+
     def abort_request(self, request_id: str) -> None:
         self.core.abort_requests([request_id])
         self._states.pop(request_id, None)
+        self._open.discard(request_id)
 
     def has_unfinished_requests(self) -> bool:
         return self.core.has_work()
@@ -356,6 +394,8 @@ class LLM:
             order.append(self.add_request(p, sp, prompt=text))
         results: dict[str, RequestOutput] = {}
         while self.has_unfinished_requests():
+            if self._open and not any(r in self._states for r in order):
+                break               # what is left waits for further input
             for st in self.step():
                 if st.finished:
                     results[st.request_id] = st

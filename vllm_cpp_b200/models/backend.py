@@ -269,6 +269,26 @@ class CpuBackend(FusedLinearMixin):
             return out
         return y
 
+    # ---- fp32 residual stream, mixed-head attention with a distance bias, clamped experts
+    def stream_norm(self, stream, norm_w, eps, out, **kw):
+        from ..ops.stream import ref_stream_norm
+        return ref_stream_norm(stream, norm_w, eps, out, **kw)
+
+    def head_mix_kv(self, qkv, mix, q_out, slots, cache, **kw):
+        from ..ops.bias_attn import ref_head_mix_kv
+        ref_head_mix_kv(qkv, mix, q_out, slots, cache, **kw)
+
+    def bias_attention(self, q, cache, ctx, group, *, out, **kw):
+        from ..ops.bias_attn import ref_bias_attention
+        return ref_bias_attention(q, cache, out, block_table=ctx.block_table[group], seq_lens=ctx.seq_lens,
+                                  q_start=ctx.query_start, **kw)
+
+    def clamped_experts(self, x, logits, w_gate_up, w_down, ws, *, top, limit, alpha, up_offset):
+        from ..ops import moe as M
+        ids, w = M.ref_router_topk(logits, top, renorm=False, scoring="sigmoid")
+        y = M.ref_clamped_experts(x, ids, w, w_gate_up, w_down, limit=limit, alpha=alpha, up_offset=up_offset)
+        return y, torch.arange(ids.numel(), dtype=torch.int32).view_as(ids)
+
     def add(self, a, b):
         return (a.float() + b.float()).to(a.dtype)
 
@@ -441,7 +461,13 @@ class GpuBackend(FusedLinearMixin):
 
     def gemm(self, a, w, bias=None, residual=None, out=None, out_dtype=torch.bfloat16):
         """``w`` is always a model weight here (never written by a kernel of the step), which
-        lets the GEMM start fetching it before the previous kernel has finished."""
+        lets the GEMM start fetching it before the previous kernel has finished. fp32 operands
+        are multiplied in fp32."""
+        if a.dtype == torch.float32:
+            from ..ops.stream import gemm_f32
+            if residual is not None:
+                raise ValueError("the fp32 product takes no residual")
+            return gemm_f32(a, w, bias=bias, out=out)
         if isinstance(w, Fp8Weight):
             from ..ops import quant as Q
             N, K = w.shape
@@ -541,6 +567,35 @@ class GpuBackend(FusedLinearMixin):
                                   block_size=block_size, scale=scale, out=out[nd:],
                                   softcap=softcap, window=window)
         return out
+
+    def stream_norm(self, stream, norm_w, eps, out, **kw):
+        from ..ops.stream import stream_norm
+        return stream_norm(stream, norm_w, eps, out, **kw)
+
+    def head_mix_kv(self, qkv, mix, q_out, slots, cache, **kw):
+        from ..ops.bias_attn import head_mix_kv
+        head_mix_kv(qkv, mix, q_out, slots, cache, **kw)
+
+    def bias_attention(self, q, cache, ctx, group, *, out, **kw):
+        """Decode rows first (one token per request), then the prompt portions."""
+        from ..ops import bias_attn as A
+        nd, bt = ctx.num_decodes, ctx.block_table[group]
+        if nd > 0:
+            A.decode(q[:nd], cache, out[:nd], block_table=bt[:nd], seq_lens=ctx.seq_lens[:nd],
+                     splits=ctx.decode_splits, tmp=ctx.extra.get("decode_tmp"), **kw)
+        if ctx.num_prefills > 0:
+            A.prefill(q[nd:], cache, out[nd:], block_table=bt[nd:], seq_lens=ctx.seq_lens[nd:],
+                      q_start=ctx.prefill_q_start, num_reqs=ctx.num_prefills, tile_req=ctx.tile_req[:ctx.num_tiles],
+                      tile_q0=ctx.tile_q0[:ctx.num_tiles], **kw)
+        return out
+
+    def clamped_experts(self, x, logits, w_gate_up, w_down, ws, *, top, limit, alpha, up_offset):
+        """Sigmoid router over ``logits``, the ``top`` experts of each token applied to the weighted
+        input. -> (expert outputs in sorted order, the row of each (token, choice) pair [T, top])."""
+        from ..ops import moe as M
+        ids, w = M.router_topk(logits, top, renorm=False, scoring="sigmoid")
+        y = M.clamped_experts(x, ids, w, w_gate_up, w_down, ws, limit=limit, alpha=alpha, up_offset=up_offset)
+        return y, ws.pair_pos[: ids.numel()].view_as(ids)
 
     def add(self, a, b):
         return self.ops.add(a, b)

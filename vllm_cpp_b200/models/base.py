@@ -70,15 +70,17 @@ class BufferPool:
             from .. import ops
             ops.init_device(torch.device(device))
 
-    def get(self, name: str, rows: int, cols: int, dtype=torch.bfloat16) -> torch.Tensor:
+    def get(self, name: str, rows: int, cols: int, dtype=torch.bfloat16, zero: bool = False) -> torch.Tensor:
+        """``zero``: a new buffer starts as zeros (columns no kernel writes stay zero)."""
         b = self._bufs.get(name)
         if b is None or b.shape[0] < rows or b.shape[1] != cols or b.dtype != dtype:
             cap = rows if b is None else max(rows, b.shape[0])
             if b is not None:
                 self._retired.append(b)
-            b = torch.empty((cap, cols), dtype=dtype, device=self.device)
+            make = torch.zeros if zero else torch.empty
+            b = make((cap, cols), dtype=dtype, device=self.device)
             self._bufs[name] = b
         return b[:rows]
 
-    def reserve(self, name: str, rows: int, cols: int, dtype=torch.bfloat16) -> None:
-        self.get(name, rows, cols, dtype)
+    def reserve(self, name: str, rows: int, cols: int, dtype=torch.bfloat16, zero: bool = False) -> None:
+        self.get(name, rows, cols, dtype, zero)

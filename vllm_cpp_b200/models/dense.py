@@ -26,6 +26,8 @@ ACT_KIND = {"silu": 0, "gelu_tanh": 1, "gelu_pytorch_tanh": 1, "gelu": 2}
 
 
 class DenseModel:
+    DTYPES = ("bfloat16",)         # types the family's kernels run in (EngineArgs.dtype)
+
     def __init__(self, cfg: ModelConfig, device="cuda", parallel: ParallelConfig | None = None,
                  comm=None, max_position: int | None = None):
         from ..parallel.comm import SingleComm

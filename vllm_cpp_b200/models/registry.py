@@ -18,6 +18,7 @@ _REGISTRY.update({
     "Qwen3_5MoeForConditionalGeneration": ("gdn", "Qwen35Model"),
     "Qwen3NextForCausalLM": ("gdn", "Qwen35Model"),
     "OPTForCausalLM": ("opt", "OPTModel"),
+    "Nufusun": ("nufusun", "NufusunModel"),
 })
 
 

@@ -1,0 +1,177 @@
+"""Attention with a per-head distance bias, heads mixed before the softmax and an optional null
+softmax entry, over pages ``[block_size, kw] keys | [block_size, G * vdim] values``.
+
+The mix of the heads is moved to the query side (``head_mix_kv``): head ``h`` reads the whole key
+row of a token with the query row ``[sum_{g in group 0} M[h, g] q_g | sum_{g in group 1} ... ]``."""
+from __future__ import annotations
+
+import ctypes
+import math
+
+import torch
+
+from . import _lib
+from ._lib import check, lib, ptr, stream_ptr
+
+_P, _L, _I = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int
+
+
+class BiasAttnArgs(ctypes.Structure):
+    _fields_ = [("q", _P), ("ldq", _L), ("out", _P), ("ldo", _L), ("cache", _P), ("num_blocks", _L),
+                ("block_table", _P), ("seq_lens", _P), ("q_start", _P), ("bias", _P), ("tmp_o", _P),
+                ("tmp_lse", _P), ("tile_req", _P), ("tile_q0", _P),
+                ("max_blocks", _I), ("num_reqs", _I), ("rows", _I), ("H", _I), ("G", _I), ("kw", _I), ("vdim", _I),
+                ("block_size", _I), ("bias_len", _I), ("null_entry", _I), ("f32", _I), ("splits", _I),
+                ("num_tiles", _I)]
+
+
+_declared = False
+
+
+def _declare():
+    global _declared
+    if _declared:
+        return
+    P, I, L = _lib.P, _lib.I, ctypes.c_longlong
+    A = ctypes.POINTER(BiasAttnArgs)
+    _lib.declare("b200_head_mix_kv", [P, L, P, P, L, P, P, I, I, I, I, I, I, I, P], I)
+    _lib.declare("b200_bias_attn_kernel", [A, I], I)
+    _lib.declare("b200_bias_attn_decode", [A, I, P], I)
+    _lib.declare("b200_bias_attn_prefill", [A, I, P], I)
+    lib()
+    _declared = True
+
+
+def head_mix_kv(qkv, mix, q_out, slots, cache, *, H, G, dim, vdim, block_size):
+    """fp32 ``qkv`` rows ``[q | k | v]`` -> mixed query rows ``q_out`` [T, H * G * dim] and this
+    step's keys and values in ``cache`` (slot < 0: none), in the type of ``q_out``."""
+    _declare()
+    assert qkv.dtype == torch.float32 and mix.dtype == torch.float32 and q_out.dtype == cache.dtype
+    check(lib().b200_head_mix_kv(ptr(qkv), qkv.stride(0), ptr(mix), ptr(q_out), q_out.stride(0), ptr(slots),
+                                 ptr(cache), H, G, dim, vdim, block_size, qkv.shape[0],
+                                 int(q_out.dtype == torch.float32), stream_ptr()), "head_mix_kv")
+
+
+def _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry) -> BiasAttnArgs:
+    a = BiasAttnArgs()
+    a.q, a.ldq, a.out, a.ldo = ptr(q), q.stride(0), ptr(out), out.stride(0)
+    a.cache, a.num_blocks = ptr(cache), cache.shape[0]
+    a.block_table, a.max_blocks, a.seq_lens = ptr(block_table), block_table.stride(0), ptr(seq_lens)
+    a.bias, a.bias_len = ptr(bias), bias.shape[1] if bias is not None else 0
+    a.rows, a.num_reqs = q.shape[0], q.shape[0]
+    a.H, a.G, a.kw, a.vdim, a.block_size = H, G, kw, vdim, block_size
+    a.null_entry, a.f32, a.splits = int(null_entry), int(q.dtype == torch.float32), 1
+    return a
+
+
+def decode(q, cache, out, *, block_table, seq_lens, H, G, kw, vdim, block_size, bias=None, null_entry=False,
+           splits=1, tmp=None, any_size=False):
+    """One query row per request, at its last position."""
+    _declare()
+    a = _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry)
+    if splits > 1:
+        if tmp is None:
+            tmp = (torch.empty(a.rows * H * splits * vdim, dtype=torch.float32, device=q.device),
+                   torch.empty(a.rows * H * splits, dtype=torch.float32, device=q.device))
+        assert tmp[0].numel() >= a.rows * H * splits * vdim and tmp[1].numel() >= a.rows * H * splits
+        a.splits, a.tmp_o, a.tmp_lse = splits, ptr(tmp[0]), ptr(tmp[1])
+    check(lib().b200_bias_attn_decode(ctypes.byref(a), int(any_size), stream_ptr()), "bias_attn_decode")
+    return out
+
+
+def prefill(q, cache, out, *, block_table, seq_lens, q_start, num_reqs, tile_req, tile_q0, H, G, kw, vdim,
+            block_size, bias=None, null_entry=False, any_size=False):
+    """Portions of prompts; ``tile_req`` / ``tile_q0`` list their 128-row query tiles."""
+    _declare()
+    a = _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry)
+    a.q_start, a.num_reqs = ptr(q_start), num_reqs
+    a.tile_req, a.tile_q0, a.num_tiles = ptr(tile_req), ptr(tile_q0), tile_req.numel()
+    check(lib().b200_bias_attn_prefill(ctypes.byref(a), int(any_size), stream_ptr()), "bias_attn_prefill")
+    return out
+
+
+def kernel_kind(phase: str, q, cache, *, H, G, kw, vdim, block_size) -> str:
+    """Which kernel serves a shape: "tensor-core" or "any-size"."""
+    _declare()
+    a = BiasAttnArgs()
+    a.q, a.ldq, a.out, a.ldo, a.cache = ptr(q), q.stride(0), ptr(q), H * vdim, ptr(cache)
+    a.H, a.G, a.kw, a.vdim, a.block_size = H, G, kw, vdim, block_size
+    a.f32, a.tile_req = int(q.dtype == torch.float32), ptr(q)
+    return {2: "tensor-core", 1: "any-size"}[lib().b200_bias_attn_kernel(ctypes.byref(a), int(phase == "prefill"))]
+
+
+def decode_splits(batch: int, max_seq_len: int, num_sms: int) -> int:
+    """KV splits of the decode kernel (one CTA per request and split, one CTA per SM at real sizes;
+    fixed per batch size, because the count is baked into a captured graph)."""
+    return max(1, min(num_sms // max(1, batch), -(-max_seq_len // 128), 32))
+
+
+# ------------------------------------------------------------------------- tables built at load time
+def bucket_of_distance(n: int, num_buckets: int, max_distance: int) -> int:
+    """Distances below half the table have a bucket each; beyond, buckets are spaced evenly in the
+    logarithm up to ``max_distance``, and the last bucket takes the rest."""
+    half = num_buckets // 2
+    if n < half:
+        return n
+    if max_distance <= half or n >= max_distance:
+        return num_buckets - 1
+    # (an exact boundary must not fall into the bucket below through the rounding of the logarithms)
+    x = math.log(n / half) / math.log(max_distance / half) * (num_buckets - half)
+    return min(num_buckets - 1, half + int(math.floor(x + 1e-9)))
+
+
+def distance_bias_table(rel: torch.Tensor, max_distance: int) -> torch.Tensor:
+    """``rel`` [buckets, H] -> fp32 [H, L]: the bias of every distance up to the first from which
+    it no longer changes (the last column)."""
+    B = rel.shape[0]
+    idx = [bucket_of_distance(n, B, max_distance) for n in range(max(max_distance, B // 2) + 1)]
+    while len(idx) > 1 and idx[-2] == idx[-1] == B - 1:
+        idx.pop()
+    return rel.float()[torch.tensor(idx, device=rel.device)].t().contiguous()
+
+
+# ------------------------------------------------------------------------------ restatements
+def page_views(cache, block_size, kw):
+    """(keys [num_blocks, block_size, kw], values [num_blocks, block_size, vw]) of a page tensor."""
+    nb = cache.shape[0]
+    flat = cache.view(nb, -1)
+    k = flat[:, : block_size * kw].view(nb, block_size, kw)
+    v = flat[:, block_size * kw:].view(nb, block_size, -1)
+    return k, v
+
+
+def ref_head_mix_kv(qkv, mix, q_out, slots, cache, *, H, G, dim, vdim, block_size):
+    T, kw, vw = qkv.shape[0], G * dim, G * vdim
+    q = qkv[:, : H * dim].float().view(T, G, H // G, dim)
+    m = torch.einsum("hgr,tgrd->thgd", mix.view(H, G, H // G), q)
+    q_out[:T, : H * kw] = m.reshape(T, H * kw).to(q_out.dtype)
+    keys, vals = page_views(cache, block_size, kw)
+    ok = slots >= 0
+    b, o = slots[ok] // block_size, slots[ok] % block_size
+    keys[b, o] = qkv[ok, H * dim: H * dim + kw].to(cache.dtype)
+    vals[b, o] = qkv[ok, H * dim + kw: H * dim + kw + vw].to(cache.dtype)
+
+
+def ref_bias_attention(q, cache, out, *, block_table, seq_lens, q_start, H, G, kw, vdim, block_size, bias=None,
+                       null_entry=False):
+    keys, vals = page_views(cache, block_size, kw)
+    qs = q_start.tolist()
+    for r, sl in enumerate(seq_lens.tolist()):
+        t0, t1 = qs[r], qs[r + 1]
+        if t1 <= t0 or sl <= 0:
+            continue
+        blocks = block_table[r, : (sl + block_size - 1) // block_size].long()
+        k = keys[blocks].reshape(-1, kw)[:sl].float()
+        v = vals[blocks].reshape(-1, G, vdim)[:sl].float().repeat_interleave(H // G, 1)
+        s = torch.einsum("qhd,kd->hqk", q[t0:t1, : H * kw].float().view(t1 - t0, H, kw), k)
+        dist = torch.arange(sl - (t1 - t0), sl)[:, None] - torch.arange(sl)[None]
+        if bias is not None:
+            s = s + bias[:, dist.clamp(0, bias.shape[1] - 1)]
+        s = s.masked_fill(dist < 0, -math.inf)
+        m = s.amax(-1, keepdim=True)
+        if null_entry:
+            m = m.clamp(min=0)
+        e = torch.exp(s - m)
+        den = e.sum(-1, keepdim=True) + (torch.exp(-m) if null_entry else 0.0)
+        out[t0:t1, : H * vdim] = torch.einsum("hqk,khd->qhd", e / den, v).reshape(t1 - t0, H * vdim).to(out.dtype)
+    return out

@@ -8,6 +8,7 @@ import torch
 
 from . import _lib
 from ._lib import check, lib, ptr, stream_ptr
+from .stream import ClampedGate
 
 
 class B200MoeScatter(ctypes.Structure):
@@ -32,6 +33,11 @@ def _declare():
     _lib.declare("b200_moe_grouped_gemm_gated", [P, I, P, I, I, I, P, P, P, P, P, I, I, P], I)
     _lib.declare("b200_moe_combine", [P, P, P, I, I, I, P, P, P, ctypes.POINTER(B200MoeScatter), P], I)
     _lib.declare("b200_shared_gate", [P, I, P, I, I, P, P], I)
+    C = ctypes.POINTER(ClampedGate)
+    _lib.declare("b200_moe_grouped_gemm_clamped", [P, I, P, I, I, I, P, P, P, P, P, I, C, P], I)
+    _lib.declare("b200_moe_row_weights", [P, P, I, P, P], I)
+    _lib.declare("b200_moe_grouped_gemm_f32", [P, I, P, I, I, I, P, P, P, P, P, I, P], I)
+    _lib.declare("b200_clamped_gate_f32", [P, P, P, I, I, I, C, P], I)
     lib()
     _declared = True
 
@@ -55,7 +61,7 @@ class MoeWorkspace:
     """Persistent buffers of one MoE layer shape (sized for ``max_tokens``)."""
 
     def __init__(self, device, max_tokens: int, k: int, num_local_experts: int, hidden: int,
-                 inter: int):
+                 inter: int, dtype=torch.bfloat16):
         P = max_tokens * k
         E = num_local_experts
         self.max_pairs = P
@@ -67,7 +73,8 @@ class MoeWorkspace:
         self.chunk_expert = torch.zeros(self.max_chunks, **i32)
         self.chunk_row0 = torch.zeros(self.max_chunks, **i32)
         self.chunk_n = torch.zeros(self.max_chunks, **i32)
-        bf = dict(dtype=torch.bfloat16, device=device)
+        self.row_w = torch.zeros(P, dtype=torch.float32, device=device)   # routing weight of a sorted row
+        bf = dict(dtype=dtype, device=device)
         self.xs = torch.zeros((P + 256, hidden), **bf)
         self.gu = torch.zeros((P + 256, 2 * inter), **bf)
         self.act = torch.zeros((P + 256, inter), **bf)
@@ -84,8 +91,9 @@ def moe_sort(topk_ids: torch.Tensor, e0: int, e1: int, ws: MoeWorkspace):
 
 def moe_gather(x: torch.Tensor, ws: MoeWorkspace, num_local_experts: int, max_rows: int):
     _declare()
-    check(lib().b200_moe_gather(ptr(x), x.stride(0), ptr(ws.sorted_token), ptr(ws.meta),
-                                num_local_experts, ptr(ws.xs), x.shape[1], max_rows,
+    w = x.element_size() // 2                   # the kernel copies rows as 16-bit values
+    check(lib().b200_moe_gather(ptr(x), x.stride(0) * w, ptr(ws.sorted_token), ptr(ws.meta),
+                                num_local_experts, ptr(ws.xs), x.shape[1] * w, max_rows,
                                 stream_ptr()), "moe_gather")
 
 
@@ -113,6 +121,34 @@ def grouped_gemm_gated(xs: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Ten
                                             ptr(ws.meta), max_chunks or ws.max_chunks, kind, stream_ptr()),
           "moe_grouped_gemm_gated")
     return out
+
+
+def clamped_experts(x, ids, w, w_gate_up, w_down, ws: MoeWorkspace, *, limit, alpha, up_offset):
+    """Expert outputs in sorted order, ``ws.y[ws.pair_pos[t * k + j]]`` = W_down a(w_tj W_gate_up x_t)
+    with the clamped pair ``a`` (see :class:`ops.stream.ClampedGate`); the routing weight scales the
+    expert's input. bf16: tcgen05 grouped GEMMs, the weight and the activation in the epilogue of the
+    first; fp32: fp32 products."""
+    T, k = ids.shape
+    E, P = w_gate_up.shape[0], T * k
+    chunks = min(ws.max_chunks, E + (P + 255) // 256)
+    moe_sort(ids, 0, E, ws)
+    moe_gather(x, ws, E, P)
+    check(lib().b200_moe_row_weights(ptr(ws.pair_pos), ptr(w), P, ptr(ws.row_w), stream_ptr()), "moe_row_weights")
+    act = ClampedGate(limit, alpha, up_offset, ptr(ws.row_w))
+    N, K = w_gate_up.shape[1:]
+    args = (ptr(ws.chunk_expert), ptr(ws.chunk_row0), ptr(ws.chunk_n), ptr(ws.meta), chunks)
+    if x.dtype == torch.bfloat16:
+        check(lib().b200_moe_grouped_gemm_clamped(ptr(ws.xs), P, ptr(w_gate_up), E, N, K, ptr(ws.act), *args,
+                                                  ctypes.byref(act), stream_ptr()), "moe_grouped_gemm_clamped")
+        grouped_gemm(ws.act, w_down, ws.y, ws, P, chunks)
+        return ws.y
+    check(lib().b200_moe_grouped_gemm_f32(ptr(ws.xs), P, ptr(w_gate_up), E, N, K, ptr(ws.gu), *args, stream_ptr()),
+          "moe_grouped_gemm_f32")
+    check(lib().b200_clamped_gate_f32(ptr(ws.gu), ptr(ws.act), ptr(ws.meta), E, P, N // 2, ctypes.byref(act),
+                                      stream_ptr()), "clamped_gate_f32")
+    check(lib().b200_moe_grouped_gemm_f32(ptr(ws.act), P, ptr(w_down), E, w_down.shape[1], N // 2, ptr(ws.y), *args,
+                                          stream_ptr()), "moe_grouped_gemm_f32")
+    return ws.y
 
 
 def combine(y: torch.Tensor, ws: MoeWorkspace, topk_w: torch.Tensor, out: torch.Tensor | None,
@@ -163,6 +199,20 @@ def ref_router_topk(logits, k, renorm=True, scoring="softmax", e_bias=None, n_gr
         d = w.sum(-1, keepdim=True)
         w = w / torch.where(d > 0, d, torch.ones_like(d))
     return ids.int(), w * routed_scale
+
+
+def ref_clamped_experts(x, ids, w, w_gate_up, w_down, *, limit, alpha, up_offset):
+    """-> outputs [T * k, H] in pair order (token-major), in the type of ``x``."""
+    from .stream import ref_clamped_gate
+    T, k = ids.shape
+    y = torch.zeros((T * k, x.shape[1]), dtype=x.dtype, device=x.device)
+    flat, wt = ids.reshape(-1).long(), w.reshape(-1)
+    for e in flat.unique().tolist():
+        rows = (flat == e).nonzero().flatten()
+        gu = (x[rows // k].float() @ w_gate_up[e].float().t()) * wt[rows, None]
+        a = ref_clamped_gate(gu, limit, alpha, up_offset).to(x.dtype)
+        y[rows] = (a.float() @ w_down[e].float().t()).to(x.dtype)
+    return y
 
 
 def ref_moe_block(x, topk_ids, topk_w, w_gate_up, w_down, e0=0):

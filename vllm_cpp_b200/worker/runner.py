@@ -36,7 +36,8 @@ _DT = {"input_ids": (torch.int64, 8), "positions": (torch.int64, 8), "slot_mappi
 STEP_INFO_FIELDS = ("num_reqs", "num_tokens", "num_decodes", "num_prefills", "num_prefill_tokens",
                     "num_tiles", "max_query_len", "max_seq_len", "num_logits", "num_splice", "all_greedy",
                     "any_penalties", "any_top_k_top_p", "any_min_p", "any_logprobs", "any_logit_edits",
-                    "req_ids", "produces_token", "max_logprobs", "num_draft", "logits_row0")
+                    "req_ids", "produces_token", "max_logprobs", "num_draft", "logits_row0", "num_score",
+                    "score_req_ids", "score_positions")
 
 
 def _plain(v):
@@ -58,7 +59,7 @@ def decode_graph_sizes(max_num_seqs: int) -> list[int]:
 class ModelRunner(E.ModelRunnerBase):
     def __init__(self, model, *, block_size: int, num_blocks: int, max_num_seqs: int,
                  max_num_batched_tokens: int, max_model_len: int, enable_cuda_graphs: bool = True,
-                 async_mode: bool = False, speculative_config=None, step_channel=None):
+                 async_mode: bool = False, speculative_config=None, step_channel=None, max_score_rows: int = 0):
         super().__init__()
         # Multi-rank serving: the rank that owns the scheduler publishes every step (the packed
         # step buffer and what the sampler needs) on this channel; the other ranks run
@@ -93,7 +94,7 @@ class ModelRunner(E.ModelRunnerBase):
         self.num_groups = len(self.groups)
         self.max_blocks = (max_model_len + block_size - 1) // block_size + 1
         self.layout = E.StepLayout.make(self.max_tokens, max_num_seqs, self.max_blocks,
-                                        self.num_groups, self.max_spec)
+                                        self.num_groups, self.max_spec, max_score_rows)
         self.off = self.layout.offsets()
         nbytes = self.layout.total_bytes
         # two pinned staging buffers: with a step in flight its copy may not have run yet when
@@ -123,6 +124,8 @@ class ModelRunner(E.ModelRunnerBase):
         self.graph_sizes = decode_graph_sizes(max_num_seqs) if self.enable_graphs else []
         self._info = None
         self._logits = None
+        # logits of the positions asked for with ``batch.set_score_positions``: rows of the last step
+        self._scored: list = []          # (request id, position, fp32 row), see take_scores
         self._eos: dict[str, int] = {}
         self.h2d_bytes = 0
         self.d2h_bytes = 0
@@ -204,6 +207,8 @@ class ModelRunner(E.ModelRunnerBase):
         if not self.is_cuda:
             return 1, None
         key = batch
+        if key not in self._decode_tmp and hasattr(self.model, "decode_workspace"):
+            self._decode_tmp[key] = self.model.decode_workspace(batch, self.max_model_len, self.block_size)
         if key not in self._decode_tmp:
             s = self.ops.attn_decode_splits(batch, self._Hkv, self._Hq // self._Hkv, self._D,
                                             self.max_model_len, self.block_size)
@@ -225,7 +230,7 @@ class ModelRunner(E.ModelRunnerBase):
             num_decodes=nd, num_prefills=0 if padded is not None else info.num_prefills,
             num_prefill_tokens=0 if padded is not None else info.num_prefill_tokens,
             num_tiles=0 if padded is not None else info.num_tiles,
-            num_logits=T if padded is not None else info.num_logits,
+            num_logits=T if padded is not None else info.num_logits + info.num_score,
             input_ids=v["input_ids"], positions=v["positions"], slot_mapping=v["slot_mapping"],
             query_start=v["query_start"], seq_lens=v["seq_lens"], block_table=v["block_table"],
             logits_indices=v["logits_indices"], tile_req=v["tile_req"], tile_q0=v["tile_q0"],
@@ -380,19 +385,44 @@ class ModelRunner(E.ModelRunnerBase):
             _l.LAUNCHES[0] += g[2]  # launcher calls folded into the replayed graph
             self._logits = g[1][:R] if g[1] is not None else None
             self._graph_sampled = True
+            # the graph has one row per request; requests whose input is still open sample nothing
+            rows = self.views["logits_indices"]
+            self._graph_ids = self.sampled if info.num_logits == R else self.sampled[rows[: info.num_logits].long()]
+            if info.num_score:
+                self._keep_scores(info, self._logits[rows[info.num_logits: info.num_logits + info.num_score].long()])
         else:
             ctx = self._context(info)
             self._last_ctx = ctx
-            if plain_greedy and self._model_samples_greedy:
+            if plain_greedy and self._model_samples_greedy and not info.num_score:
                 # the model writes the argmax ids itself (tensor parallel: candidates per vocabulary
                 # shard are exchanged instead of the logits)
                 ctx.extra["greedy_out"] = self.sampled
             with nvtx.range(f"forward T={T} R={R}"):
                 self._logits = self.model.forward(ctx)
             self._graph_sampled = self._logits is None
+            self._graph_ids = self.sampled
+            if info.num_score and self._logits is not None:
+                self._keep_scores(info, self._logits[info.num_logits:])
+                self._logits = self._logits[: info.num_logits]
         self.num_kernel_steps += 1
         if getattr(self.model, "eplb", None) is not None:
             self.model.eplb_end_step()         # closes the load window of the step; rebalances on schedule
+
+    def _keep_scores(self, info, rows) -> None:
+        self._scored.append((list(info.score_req_ids), list(info.score_positions), rows.clone()))
+
+    def take_scores(self) -> dict:
+        """Logits of the scored positions computed since the last call: request id -> [(position,
+        fp32 row on the host)], in position order."""
+        out: dict = {}
+        scored, self._scored = self._scored, []
+        for ids, positions, rows in scored:
+            rows = rows.float().cpu()
+            for i, (rid, p) in enumerate(zip(ids, positions)):
+                out.setdefault(rid, []).append((p, rows[i]))
+        if self.is_cuda:
+            self._check_status(int(self._status_dev.cpu()[0]))
+        return out
 
     def _sample_device(self, info, grammar) -> torch.Tensor:
         """Runs the sampler pipeline on the logits of this step; returns int64 ids [num_logits]."""
@@ -400,7 +430,7 @@ class ModelRunner(E.ModelRunnerBase):
         logits = self._logits
         v = self.views
         if self._graph_sampled:
-            return self.sampled[:n]
+            return self._graph_ids[:n]
         edits = self._pending_edits
         if edits is None:
             edits = self._host_sampler_edits(info, grammar)
