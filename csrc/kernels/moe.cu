@@ -63,7 +63,11 @@ __global__ void __launch_bounds__(256)
     for (int i = threadIdx.x; i < E; i += blockDim.x) score[i] = 1.f / (1.f + expf(-x[i]));
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < E; i += blockDim.x) sel[i] = score[i] + (e_bias ? e_bias[i] : 0.f);
+  // plain sigmoid scores are ranked by their logits: the same order, without the ties that fp32
+  // scores near 1 round to
+  const bool by_logit = scoring == 1 && !e_bias && n_group <= 1;
+  for (int i = threadIdx.x; i < E; i += blockDim.x)
+    sel[i] = by_logit ? x[i] : score[i] + (e_bias ? e_bias[i] : 0.f);
   __syncthreads();
   if (n_group > 1 && topk_group < n_group) {
     // thread g scores group g (n_group is small), thread 0 masks the losers

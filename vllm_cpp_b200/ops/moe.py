@@ -178,7 +178,9 @@ def ref_router_topk(logits, k, renorm=True, scoring="softmax", e_bias=None, n_gr
                     topk_group=1, routed_scale=1.0):
     x = logits.float()
     score = torch.softmax(x, -1) if scoring == "softmax" else torch.sigmoid(x)
-    sel = score + (e_bias.float() if e_bias is not None else 0.0)
+    # (plain sigmoid scores are ranked by their logits, which do not tie where fp32 scores round to 1)
+    by_logit = scoring != "softmax" and e_bias is None and n_group <= 1
+    sel = x if by_logit else score + (e_bias.float() if e_bias is not None else 0.0)
     T, E = x.shape
     if n_group > 1 and topk_group < n_group:
         g = sel.view(T, n_group, E // n_group)
