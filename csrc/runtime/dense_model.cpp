@@ -34,7 +34,9 @@ DenseConfig DenseConfig::from_hf(const Json& cfg_in) {
     for (auto& kv : cfg_in["text_config"].members()) t[kv.first] = kv.second;
   DenseConfig c;
   const auto& archs = t["architectures"];
-  c.architecture = archs.size() ? archs[0].as_string() : "LlamaForCausalLM";
+  // (layer-list checkpoints name one "architecture")
+  c.architecture = archs.size() ? archs[0].as_string()
+                   : t.contains("architecture") ? t["architecture"].as_string() : "LlamaForCausalLM";
   static const char* kSupported[] = {"LlamaForCausalLM", "MistralForCausalLM", "Qwen3ForCausalLM",
                                      "Qwen3MoeForCausalLM"};
   bool ok = false;

@@ -322,8 +322,10 @@ def model_config_from_blocks(cfg: dict) -> ModelConfig:
             if not 1 <= mlp.top <= mlp.experts:
                 raise ValueError(f"layer {i}: {mlp.top} of {mlp.experts} experts")
         blocks.append(BlockSpec(att, mlp))
-    return model_config_of_blocks(arch, blocks, vocab=int(cfg["vocab"]), width=int(cfg["width"]),
-                                  eps=float(cfg["norm"]["eps"]), embed_scale=float(cfg["embedding"]["scale"]), raw=cfg)
+    m = model_config_of_blocks(arch, blocks, vocab=int(cfg["vocab"]), width=int(cfg["width"]),
+                               eps=float(cfg["norm"]["eps"]), embed_scale=float(cfg["embedding"]["scale"]), raw=cfg)
+    m.eos_token_id, m.bos_token_id = cfg.get("eos_token_id"), cfg.get("bos_token_id")
+    return m
 
 
 def model_config_of_blocks(arch: str, blocks: list, *, vocab: int, width: int, eps: float, embed_scale: float,

@@ -13,7 +13,10 @@ def main(argv=None) -> int:
     ap = argparse.ArgumentParser("vllm_cpp_b200 cli")
     ap.add_argument("--model", required=True)
     ap.add_argument("--tokenizer-config", dest="tokenizer", default=None)
-    ap.add_argument("--prompt", required=True)
+    ap.add_argument("--prompt", default=None)
+    ap.add_argument("--prompt-ids", default=None, metavar="ID,ID,...",
+                    help="token ids instead of text (models without a tokenizer); prints the generated ids")
+    ap.add_argument("--dtype", default="auto", choices=["auto", "bfloat16", "float32"])
     ap.add_argument("--max-tokens", type=int, default=64)
     ap.add_argument("--temperature", type=float, default=0.0)
     ap.add_argument("--top-p", type=float, default=1.0)
@@ -24,6 +27,8 @@ def main(argv=None) -> int:
     ap.add_argument("--max-model-len", type=int, default=0)
     ap.add_argument("--tokenize-only", action="store_true")
     a = ap.parse_args(argv)
+    if (a.prompt is None) == (a.prompt_ids is None):
+        ap.error("one of --prompt and --prompt-ids")
     if a.tokenize_only:
         from ..loader import load_tokenizer
         tok = load_tokenizer(a.tokenizer or a.model)
@@ -35,11 +40,15 @@ def main(argv=None) -> int:
     from ..engine import LLM, SamplingParams
     from .async_llm import AsyncLLM
     llm = LLM(EngineArgs(model=a.model, tokenizer=a.tokenizer, device=a.device, max_model_len=a.max_model_len,
-                         max_num_seqs=1))
+                         max_num_seqs=1, dtype=a.dtype))
     kw = dict(temperature=a.temperature, top_p=a.top_p, top_k=a.top_k, max_tokens=a.max_tokens)
     if a.seed is not None:
         kw["seed"] = a.seed
     sp = SamplingParams(**kw)
+    if a.prompt_ids is not None:
+        out = llm.generate([[int(x) for x in a.prompt_ids.split(",")]], sp)[0]
+        print(",".join(map(str, out.outputs[0].token_ids)))
+        return 0
     if not a.stream:
         out = llm.generate([a.prompt], sp)[0]
         print(out.outputs[0].text)

@@ -24,14 +24,15 @@ MAX_REQUESTS = 4
 
 
 class TraceReplay:
-    def __init__(self, model: str, dtype: str, max_tokens: int, device: str = "cuda", max_requests: int = MAX_REQUESTS):
+    def __init__(self, model: str, dtype: str, max_tokens: int, device: str = "cuda", max_requests: int = MAX_REQUESTS,
+                 page: int = PAGE):
         from ..config import EngineArgs
         from ..engine import LLM
-        pages = (max_tokens + PAGE - 1) // PAGE
+        pages = (max_tokens + page - 1) // page
         # one page beyond the pool is the block pool's null page
-        self.llm = LLM(EngineArgs(model=model, dtype=dtype, device=device, block_size=PAGE, num_blocks=pages + 1,
-                                  max_model_len=pages * PAGE + 2, max_num_seqs=max_requests,
-                                  max_num_batched_tokens=pages * PAGE, max_score_rows=pages * PAGE,
+        self.llm = LLM(EngineArgs(model=model, dtype=dtype, device=device, block_size=page, num_blocks=pages + 1,
+                                  max_model_len=pages * page + 2, max_num_seqs=max_requests,
+                                  max_num_batched_tokens=pages * page, max_score_rows=pages * page,
                                   enable_prefix_caching=False))
         self.length: dict[str, int] = {}
 

@@ -19,7 +19,7 @@ from typing import Iterator, Optional
 
 import torch
 
-from ..config import ModelConfig, load_model_config, model_config_from_hf
+from ..config import ModelConfig, block_config_dict, load_model_config, model_config_from_hf
 from .safetensors import SafetensorsFile, open_shards, save_file  # noqa: F401
 
 # e2m1 code -> value (sign in bit 3)
@@ -195,7 +195,8 @@ def synthetic_tokenizer_json(vocab_size: int, specials=("<|endoftext|>", "<|im_s
 
 
 def hf_config_dict(cfg: ModelConfig) -> dict:
-    """config.json for a ModelConfig of the dense / Qwen3-MoE families."""
+    """config.json for a ModelConfig of the dense / Qwen3-MoE families (``config.block_config_dict`` is
+    the one of layer-list models)."""
     d = {
         "architectures": [cfg.architecture], "hidden_size": cfg.hidden_size,
         "num_hidden_layers": cfg.num_layers, "num_attention_heads": cfg.num_heads,
@@ -233,7 +234,7 @@ def write_synthetic_checkpoint(out_dir: str, cfg: ModelConfig, seed: int = 0, st
     model.load_weights = capture
     model.init_random(seed, std) if "std" in model.init_random.__code__.co_varnames else model.init_random(seed)
     save_file(captured, os.path.join(out_dir, "model.safetensors"), {"format": "pt"})
-    hf = hf_config_dict(cfg)
+    hf = block_config_dict(cfg) if cfg.blocks else hf_config_dict(cfg)
     if with_tokenizer:
         hf["eos_token_id"] = cfg.vocab_size - 3      # <|endoftext|> in the synthetic tokenizer
     with open(os.path.join(out_dir, "config.json"), "w") as f:
