@@ -1,0 +1,236 @@
+"""Throughput of the Nufusun design beside the closest other model of this package (Qwen3-MoE) at equal
+layer sizes, and its kernels beside the like kernels of that model, each against its roofline.
+
+``bench.py --design nufusun`` runs it and prints one JSON line. Random weights; device time (CUDA
+events); kernels are timed with an L2 flush between iterations, median of several."""
+from __future__ import annotations
+
+import json
+import os
+
+import torch
+
+# name -> width, heads, kv heads, head size, experts, top, expert size, layers
+SIZES = {
+    "30b-a3b layers": (2048, 32, 4, 128, 128, 8, 768, 4),
+    "small layers": (1024, 16, 4, 64, 32, 4, 512, 6),
+    "8 kv heads": (2048, 32, 8, 64, 64, 4, 1024, 4),
+    "wide layers": (4096, 32, 8, 128, 16, 2, 2048, 3),
+}
+
+
+def configs(size):
+    from ..config import AttentionSpec, BlockSpec, ExpertSpec, ModelConfig, RopeConfig, model_config_of_blocks
+    W, H, G, D, E, top, ff, layers = size
+    block = BlockSpec(AttentionSpec(heads=H, kv_heads=G, dim=D, vdim=D, scale=D ** -0.5, bias_max=1024),
+                      ExpertSpec(experts=E, top=top, ff=ff, limit=7.0))
+    mine = model_config_of_blocks("Nufusun", [block] * layers, vocab=32000, width=W, eps=1e-6, embed_scale=1.0)
+    other = ModelConfig(architecture="Qwen3MoeForCausalLM", vocab_size=32000, hidden_size=W, intermediate_size=3 * W,
+                        num_layers=layers, num_heads=H, num_kv_heads=G, head_dim=D, max_position_embeddings=32768,
+                        qk_norm=True, rope=RopeConfig(theta=1e6), num_experts=E, num_experts_per_tok=top,
+                        moe_intermediate_size=ff, norm_topk_prob=True)
+    return {"nufusun": mine, "qwen3-moe": other}
+
+
+def throughput(cfg, prompt: int, batch: int, decode_steps: int, prompt_steps: int) -> dict:
+    """Prompt tokens/s over full-budget steps and decoded tokens/s of a full batch, device time."""
+    from ..config import EngineArgs
+    from ..engine import LLM, SamplingParams
+    budget, block = 8192, 32
+    max_len = prompt + decode_steps + 64
+    llm = LLM(EngineArgs(model_config=cfg, device="cuda", block_size=block, max_model_len=max_len, max_num_seqs=batch,
+                         max_num_batched_tokens=budget, num_blocks=batch * (max_len // block + 2) + 8,
+                         enable_prefix_caching=False))
+    llm.runner.warmup_graphs([s for s in llm.runner.graph_sizes if s >= batch][:1])
+    g = torch.Generator().manual_seed(1)
+    rng = lambda n: torch.randint(0, cfg.vocab_size, (n,), generator=g).tolist()      # noqa: E731
+
+    def run(n_req, out, skip):
+        for _ in range(n_req):
+            llm.add_request(rng(prompt), SamplingParams(temperature=0.0, max_tokens=out, ignore_eos=True))
+        for _ in range(skip):
+            llm.step()
+
+    per_step = max(1, budget // prompt)
+    run(per_step * 3, 1, 3)                                         # warm-up
+    run(per_step * prompt_steps, 1, 0)
+    llm.runner.device_step_ms()
+    llm.runner.time_steps = True
+    tokens = 0
+    while llm.has_unfinished_requests():
+        llm.step()
+        tokens += llm.step_stats()["scheduled_tokens"]
+    prefill = tokens / llm.runner.device_step_ms() * 1e3
+    llm.runner.time_steps = False
+    run(batch, decode_steps + 8, -(-batch * prompt // budget) + 4)  # prompts in, a few decode steps
+    llm.runner.device_step_ms()
+    llm.runner.time_steps = True
+    for _ in range(decode_steps - 8):
+        llm.step()
+    ms = llm.runner.device_step_ms() / (decode_steps - 8)
+    status = llm.runner.ops.read_status()
+    return {"prefill_tok_s": round(prefill), "decode_tok_s": round(batch / ms * 1e3), "decode_step_ms": round(ms, 4),
+            "status": status}
+
+
+# ------------------------------------------------------------------------------ kernels
+def _peaks():
+    root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+    try:
+        with open(os.path.join(root, "MEASURED_PEAKS.json")) as f:
+            p = json.load(f)
+        return p["hbm_gbs"], p["bf16_tflops"], "measured"
+    except (OSError, KeyError, ValueError):
+        return 6650.0, 1590.0, "fallback"
+
+
+class KernelBench:
+    def __init__(self, size):
+        self.W, self.H, self.G, self.D, self.E, self.top, self.ff, _ = size
+        self.dev = torch.device("cuda")
+        self.hbm, self.tflops, _ = _peaks()
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device=self.dev)
+        self.rows: list = []
+
+    def time(self, fn, iters=9):
+        from ..ops.bench import _time
+        return _time(fn, iters=iters, warmup=3, flush=self.flush)
+
+    def add(self, name, whose, fn, nbytes=0.0, flops=0.0, note=None):
+        """The roofline is the slower of the bytes at the measured copy rate and the tensor FLOPs at
+        the measured GEMM rate."""
+        ms = self.time(fn)
+        best = max(nbytes / (self.hbm * 1e6), flops / (self.tflops * 1e9))
+        row = {"kernel": name, "model": whose, "us": round(ms * 1e3, 1), "roofline_us": round(best * 1e3, 1),
+               "fraction": round(best / ms, 3)}
+        if note:
+            row["note"] = note
+        self.rows.append(row)
+
+    def rnd(self, *shape, dtype=torch.bfloat16, s=1.0):
+        return (torch.randn(*shape, device=self.dev, dtype=torch.float32) * s).to(dtype)
+
+    def i32(self, x):
+        return torch.tensor(x, dtype=torch.int32, device=self.dev)
+
+    def attention(self, B, prompt, decode_batch, ctx, bs=32):
+        from .. import ops
+        from ..ops import bias_attn as A
+        from ..ops.reference import build_prefill_tiles
+        H, G, D, kw = self.H, self.G, self.D, self.G * self.D
+        bias = self.rnd(H, 1024, dtype=torch.float32)
+        # ---- prompts of equal length
+        nb, T = prompt // bs, B * prompt
+        bt = torch.arange(1, B * nb + 1, device=self.dev, dtype=torch.int32).view(B, nb)
+        sl, qs = self.i32([prompt] * B), self.i32([i * prompt for i in range(B + 1)])
+        tr, tq = (self.i32(x) for x in build_prefill_tiles([prompt] * B))
+        pairs = B * prompt * (prompt + 1) / 2
+        flops = 2 * pairs * H * 2 * D
+        q = self.rnd(T, H * kw, s=kw ** -0.5)
+        pages = self.rnd(B * nb + 1, bs * 2 * kw)
+        out = torch.empty(T, H * D, dtype=torch.bfloat16, device=self.dev)
+        shape = dict(H=H, G=G, kw=kw, vdim=D, block_size=bs)
+        kind = A.kernel_kind("prefill", q, pages, **shape)
+        self.add(f"attention, {B} x {prompt} prompt", "nufusun",
+                 lambda: A.prefill(q, pages, out, block_table=bt, seq_lens=sl, q_start=qs, num_reqs=B, tile_req=tr,
+                                   tile_q0=tq, bias=bias, null_entry=True, **shape), flops=flops,
+                 note=f"{kind}; multiplies {kw} + {D} wide, {(kw + D) / (2 * D):.2f} x the counted FLOPs")
+        q2, kv = self.rnd(T, H * D), self.rnd(B * nb + 1, 2, bs, G, D)
+        self.add(f"attention, {B} x {prompt} prompt", "qwen3-moe",
+                 lambda: ops.attn_prefill(q2, kv, block_table=bt, seq_lens=sl, q_start=qs, tile_req=tr, tile_q0=tq,
+                                          num_q_heads=H, num_kv_heads=G, head_dim=D, block_size=bs, scale=D ** -0.5,
+                                          out=out), flops=flops)
+        # ---- head mix + cache write against qk-norm + rotation + cache write
+        qkv = self.rnd(T, (H + 2 * G) * D, dtype=torch.float32)
+        slots = (bt.long()[:, :, None] * bs + torch.arange(bs, device=self.dev)).reshape(-1)
+        mix = self.rnd(H, H, dtype=torch.float32)
+        self.add(f"query preparation + cache write, {T} tokens", "nufusun",
+                 lambda: A.head_mix_kv(qkv, mix, q, slots, pages, H=H, G=G, dim=D, vdim=D, block_size=bs),
+                 nbytes=T * ((H + 2 * G) * D * 4 + (H * kw + 2 * G * D) * 2))
+        qkvb, pos = qkv.to(torch.bfloat16), torch.arange(T, device=self.dev) % prompt
+        table = self.rnd(prompt, D, dtype=torch.float32)
+        nw = self.rnd(D)
+        self.add(f"query preparation + cache write, {T} tokens", "qwen3-moe",
+                 lambda: ops.rope_kv(qkvb, pos, table, num_q_heads=H, num_kv_heads=G, head_dim=D, q_norm=nw, k_norm=nw,
+                                     slot_mapping=slots, kv_cache=kv, block_size=bs),
+                 nbytes=T * ((H + 2 * G) * D * 2 + (H + 4 * G) * D * 2 - 2 * G * D))
+        # ---- decode
+        B, nb = decode_batch, ctx // bs
+        bt = torch.arange(1, B * nb + 1, device=self.dev, dtype=torch.int32).view(B, nb)
+        sl = self.i32([ctx] * B)
+        pages, kv = self.rnd(B * nb + 1, bs * 2 * kw), self.rnd(B * nb + 1, 2, bs, G, D)
+        q, q2 = self.rnd(B, H * kw, s=kw ** -0.5), self.rnd(B, H * D)
+        nbytes = B * ctx * 2 * kw * 2
+        splits = A.decode_splits(B, ctx, ops.num_sms())
+        out = torch.empty(B, H * D, dtype=torch.bfloat16, device=self.dev)
+        self.add(f"attention, decode {B} x {ctx}", "nufusun",
+                 lambda: A.decode(q, pages, out, block_table=bt, seq_lens=sl, bias=bias, null_entry=True, splits=splits,
+                                  **shape), nbytes=nbytes, note=A.kernel_kind("decode", q, pages, **shape))
+        self.add(f"attention, decode {B} x {ctx}", "qwen3-moe",
+                 lambda: ops.attn_decode(q2, kv, block_table=bt, seq_lens=sl, num_q_heads=H, num_kv_heads=G, head_dim=D,
+                                         block_size=bs, scale=D ** -0.5, out=out), nbytes=nbytes)
+
+    def rest(self, T):
+        from .. import ops
+        from ..ops import moe as M
+        from ..ops.stream import stream_norm
+        W, E, top, ff = self.W, self.E, self.top, self.ff
+        P = T * top
+        ws = M.MoeWorkspace(self.dev, T, top, E, W, ff)
+        x, wgu, wd = self.rnd(T, W), self.rnd(E, 2 * ff, W, s=0.05), self.rnd(E, W, ff, s=0.05)
+        logits = self.rnd(T, E, dtype=torch.float32)
+        ids, w = M.router_topk(logits, top, renorm=False, scoring="sigmoid")
+        used = min(E, int(ids.unique().numel()))
+        chunks = min(ws.max_chunks, E + (P + 255) // 256)
+        M.moe_sort(ids, 0, E, ws)
+        M.moe_gather(x, ws, E, P)
+        act = M.ClampedGate(7.0, 1.702, 1.0, M.ptr(ws.row_w))
+        nbytes = used * 2 * ff * W * 2 + P * (W + ff) * 2
+        args = (M.ptr(ws.chunk_expert), M.ptr(ws.chunk_row0), M.ptr(ws.chunk_n), M.ptr(ws.meta), chunks)
+        import ctypes
+        self.add(f"gated expert products, {T} tokens", "nufusun",
+                 lambda: M.check(M.lib().b200_moe_grouped_gemm_clamped(M.ptr(ws.xs), P, M.ptr(wgu), E, 2 * ff, W, M.ptr(ws.act),
+                                                                       *args, ctypes.byref(act), M.stream_ptr()), "clamped"),
+                 nbytes=nbytes, flops=2.0 * P * 2 * ff * W)
+        self.add(f"gated expert products, {T} tokens", "qwen3-moe",
+                 lambda: M.grouped_gemm_gated(ws.xs, wgu, ws.act, ws, P, chunks), nbytes=nbytes, flops=2.0 * P * 2 * ff * W)
+        out, stream = torch.empty_like(x), self.rnd(T, W, dtype=torch.float32)
+        a, nw = self.rnd(T, W, dtype=torch.float32), self.rnd(W, dtype=torch.float32)
+        pos = ws.pair_pos[:P].view(T, top)
+        self.add(f"expert sum + residual + norm, {T} tokens", "nufusun",
+                 lambda: stream_norm(stream, nw, 1e-6, out, width=W, a=a, y=ws.y, pair_pos=pos),
+                 nbytes=T * W * (4 + 4 + 4 + 2 * top + 2))
+        o2, res, nwb = torch.empty_like(x), self.rnd(T, W), nw.to(torch.bfloat16)
+
+        def two():
+            M.combine(ws.y, ws, w, o2)
+            ops.rmsnorm(o2, nwb, 1e-6, residual=res, out=out)
+        self.add(f"expert sum + residual + norm, {T} tokens", "qwen3-moe", two, nbytes=T * W * 2 * (top + 1 + 1 + 2 + 1),
+                 note="two kernels")
+
+
+def run(sizes=None, kernels=True) -> dict:
+    hbm, tf, how = _peaks()
+    res = {"metric": "design_layer_throughput", "unit": "tok/s", "impl": "ours", "dtype": "bf16",
+           "data": "synthetic (uniform-random prompt ids, random-init weights)",
+           "roofline": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": how}, "models": {}, "kernels": {}}
+    for name, size in SIZES.items():
+        if sizes and name not in sizes:
+            continue
+        res["models"][name] = {"layers": dict(zip(("width", "heads", "kv_heads", "head", "experts", "top", "expert", "layers"), size))}
+        for prompt, batch in ((1024, 64), (4096, 16)):
+            r = {}
+            for who, cfg in configs(size).items():
+                r[who] = throughput(cfg, prompt, batch, decode_steps=40, prompt_steps=4)
+                torch.cuda.empty_cache()
+            res["models"][name][f"prompt {prompt}, decode batch {batch}"] = r
+        if kernels:
+            k = KernelBench(size)
+            k.attention(B=4, prompt=2048, decode_batch=64, ctx=4096)
+            k.attention(B=8, prompt=1024, decode_batch=8, ctx=16384)
+            for T in (64, 8192):
+                k.rest(T)
+            res["kernels"][name] = k.rows
+            del k
+            torch.cuda.empty_cache()
+    return res

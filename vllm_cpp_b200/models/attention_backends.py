@@ -38,6 +38,13 @@ REGISTRY: list[AttentionBackend] = [
                      lambda head_dim, **_: head_dim in (64, 128, 256)),
     AttentionBackend("tcgen05-prefill", "prefill", "paged", 0, "b200_attn_prefill",
                      lambda head_dim, block_size, **_: head_dim in (64, 128, 256) and _pages_tile(block_size, 64)),
+    AttentionBackend("mma-bias-decode", "decode", "bias", 0, "b200_bias_attn_decode",
+                     lambda head_dim, v_head_dim, f32=False, **_: not f32 and head_dim % 8 == 0 and v_head_dim % 8 == 0),
+    AttentionBackend("tcgen05-bias-prefill", "prefill", "bias", 0, "b200_bias_attn_prefill",
+                     lambda head_dim, v_head_dim, block_size, f32=False, **_: not f32 and head_dim % 8 == 0
+                     and v_head_dim % 8 == 0 and v_head_dim <= 256 and _pages_tile(block_size, 64)),
+    AttentionBackend("any-size-bias-decode", "decode", "bias", 1, "b200_bias_attn_decode", lambda **_: True),
+    AttentionBackend("any-size-bias-prefill", "prefill", "bias", 1, "b200_bias_attn_prefill", lambda **_: True),
     AttentionBackend("mla-absorbed-decode", "decode", "mla", 0, "b200_mla_decode",
                      lambda num_heads, block_size, **_: 1 <= num_heads <= 16 and _pages_tile(block_size, 128)),
     AttentionBackend("mla-expanded-prefill", "prefill", "mla", 0, "b200_attn_prefill (head_dim 256 over expanded K/V)",
