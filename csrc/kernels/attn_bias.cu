@@ -87,8 +87,11 @@ __global__ void __launch_bounds__(256) head_mix_kv_kernel(MixParams p) {
         for (int t = 0; t < kMixTok; ++t) acc[h][t] = fmaf(m, q[t], acc[h][t]);
       }
     }
-    for (int h = 0; h < nh; ++h)
-      for (int t = 0; t < nt; ++t) qo[(size_t)(t0 + t) * p.ldq + (size_t)(h0 + h) * kw + c] = from_f<TO>(acc[h][t]);
+#pragma unroll
+    for (int h = 0; h < kMixHeads; ++h)
+#pragma unroll
+      for (int t = 0; t < kMixTok; ++t)
+        if (h < nh && t < nt) qo[(size_t)(t0 + t) * p.ldq + (size_t)(h0 + h) * kw + c] = from_f<TO>(acc[h][t]);
   }
   if (blockIdx.y == 0) {
     TO* cache = reinterpret_cast<TO*>(p.cache);
@@ -102,6 +105,71 @@ __global__ void __launch_bounds__(256) head_mix_kv_kernel(MixParams p) {
       TO* vd = page + (int64_t)p.block_size * kw + off * vw;
       for (int i = threadIdx.x; i < kw; i += blockDim.x) kd[i] = from_f<TO>(src[i]);
       for (int i = threadIdx.x; i < vw; i += blockDim.x) vd[i] = from_f<TO>(src[kw + i]);
+    }
+  }
+}
+
+// Head size a multiple of 4 and RR = heads per group known: a thread takes four consecutive dims of one
+// group of one token, holds the RR query values of each in registers and runs over this block's output
+// heads; the mix rows lie in shared memory in groups of RR. blockIdx.y: slice of output heads, the last
+// slice writes the cache instead.
+template <typename TO> struct Store4;
+template <> struct Store4<float> {
+  static __device__ __forceinline__ void put(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+};
+template <> struct Store4<__nv_bfloat16> {
+  static __device__ __forceinline__ void put(__nv_bfloat16* p, const float* v) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+  }
+};
+
+template <typename TO, int RR>
+__global__ void __launch_bounds__(256) head_mix_kv_vec_kernel(MixParams p, int heads_per_block) {
+  extern __shared__ float mix_smem[];     // [heads_per_block][H]
+  pdl_wait();
+  pdl_launch_dependents();
+  const int kw = p.G * p.dim, vw = p.G * p.vdim, kw4 = kw / 4, vw4 = vw / 4, d4 = p.dim / 4;
+  const size_t stride = (size_t)gridDim.x * blockDim.x, first = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (blockIdx.y + 1 == gridDim.y) {
+    TO* cache = reinterpret_cast<TO*>(p.cache);
+    const int row4 = kw4 + vw4;
+    for (size_t x = first; x < (size_t)p.T * row4; x += stride) {
+      const int t = (int)(x / row4), i = (int)(x - (size_t)t * row4);
+      const int64_t slot = p.slots[t];
+      if (slot < 0) continue;
+      const int64_t blk = slot / p.block_size, off = slot % p.block_size;
+      TO* page = cache + blk * p.block_size * (int64_t)(kw + vw);
+      TO* dst = i < kw4 ? page + off * kw + i * 4 : page + (int64_t)p.block_size * kw + off * vw + (i - kw4) * 4;
+      const float4 v = *reinterpret_cast<const float4*>(p.qkv + (size_t)t * p.ld + (size_t)p.H * p.dim + i * 4);
+      const float f[4] = {v.x, v.y, v.z, v.w};
+      Store4<TO>::put(dst, f);
+    }
+    return;
+  }
+  const int h0 = blockIdx.y * heads_per_block, nh = min(heads_per_block, p.H - h0);
+  for (int i = threadIdx.x; i < nh * p.H; i += blockDim.x) mix_smem[i] = p.mix[(size_t)h0 * p.H + i];
+  __syncthreads();
+  for (size_t x = first; x < (size_t)p.T * kw4; x += stride) {
+    const int t = (int)(x / kw4), c = (int)(x - (size_t)t * kw4), g = c / d4, d = (c - g * d4) * 4;
+    const float* src = p.qkv + (size_t)t * p.ld + (size_t)g * RR * p.dim + d;
+    float q[RR][4];
+#pragma unroll
+    for (int r = 0; r < RR; ++r) {
+      const float4 v = *reinterpret_cast<const float4*>(src + r * p.dim);
+      q[r][0] = v.x; q[r][1] = v.y; q[r][2] = v.z; q[r][3] = v.w;
+    }
+    TO* dst = reinterpret_cast<TO*>(p.q_out) + (size_t)t * p.ldq + (size_t)h0 * kw + (size_t)c * 4;
+    const float* m = mix_smem + g * RR;
+#pragma unroll 2
+    for (int h = 0; h < nh; ++h, m += p.H, dst += kw) {
+      float a[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int r = 0; r < RR; ++r) {
+        const float w = m[r];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) a[e] = fmaf(w, q[r][e], a[e]);
+      }
+      Store4<TO>::put(dst, a);
     }
   }
 }
@@ -550,6 +618,17 @@ __global__ void __launch_bounds__(192)
   const uint32_t tmem_base = bars->tmem_base, tmem_s0 = tmem_base, tmem_o = tmem_base + 128;
 
   if (warp == 0) {
+    // A 64-key tile spans up to eight pages; lane l fetches the rows of the l-th one, so the page
+    // look-ups of a tile run side by side.
+    const int rpl = min(p.block_size, kBKeys), loads = kBKeys / rpl;
+    const int32_t* bt = p.block_table + (size_t)req * p.max_blocks;
+    const int nblk = (seq_len + p.block_size - 1) / p.block_size;
+    auto page_of = [&](int j) {
+      const int bi = (j * kBKeys + lane * rpl) / p.block_size;
+      return max(lane < loads && bi < nblk ? bt[bi] : bt[0], 0);
+    };
+    const int row_in_page = (lane * rpl) % p.block_size;            // block_size <= 64
+    const int dst_off = lane * rpl * 128;
     if (lane == 0) {
       tma_prefetch_desc(&tmQ);
       tma_prefetch_desc(&tmK);
@@ -557,39 +636,39 @@ __global__ void __launch_bounds__(192)
       mbar_expect_tx(&bars->q_full, nkc * kQChunkBytes);
       for (int c = 0; c < nkc; ++c)
         tma_load_2d(sQ + c * kQChunkBytes, &tmQ, &bars->q_full, h * p.kw + c * 64, q_begin + q0);
-      const int32_t* bt = p.block_table + (size_t)req * p.max_blocks;
-      const int nblk = (seq_len + p.block_size - 1) / p.block_size;
-      const int rpl = min(p.block_size, kBKeys), loads = kBKeys / rpl;
-      uint32_t kc = 0;
-      bool ok = true;
-      // Order K0 K1 V0 K2 V1 ... K(n-1) V(n-2) V(n-1): the order in which the MMA warp consumes them.
-      for (int j = 0; j <= ntiles && ok; ++j) {
-        if (j < ntiles) {
-          for (int c = 0; c < nkc && ok; ++c, ++kc) {
-            const int sl = kc % p.k_slots;
-            if (!mbar_wait(&bars->k_empty[sl], ((kc / p.k_slots) & 1) ^ 1, p.status)) { ok = false; break; }
-            mbar_expect_tx(&bars->k_full[sl], kChunkBytes);
-            for (int l = 0; l < loads; ++l) {
-              const int tk = j * kBKeys + l * rpl, bi = tk / p.block_size;
-              const int blk = max(bi < nblk ? bt[bi] : bt[0], 0);
-              tma_load_3d(sK + sl * kChunkBytes + l * rpl * 128, &tmK, &bars->k_full[sl], c * 64,
-                          tk % p.block_size, blk);
-            }
-          }
-        }
-        if (j >= 1 && ok) {
-          const int i = j - 1, sl = i % kVSlots;
-          if (!mbar_wait(&bars->v_empty[sl], ((i / kVSlots) & 1) ^ 1, p.status)) { ok = false; break; }
-          mbar_expect_tx(&bars->v_full[sl], nvc * kChunkBytes);
-          for (int l = 0; l < loads; ++l) {
-            const int tk = i * kBKeys + l * rpl, bi = tk / p.block_size;
-            const int blk = max(bi < nblk ? bt[bi] : bt[0], 0);
-            for (int c = 0; c < nvc; ++c)
-              tma_load_3d(sV + (sl * nvc + c) * kChunkBytes + l * rpl * 128, &tmV, &bars->v_full[sl],
-                          hkv * p.vdim + c * 64, tk % p.block_size, blk);
-          }
+    }
+    int sl = 0, blk = page_of(0), blk_prev = 0;
+    uint32_t ph = 1;
+    bool ok = true;
+    // Order K0 K1 V0 K2 V1 ... K(n-1) V(n-2) V(n-1): the order in which the MMA warp consumes them.
+    for (int j = 0; j <= ntiles && ok; ++j) {
+      const int next = j + 1 < ntiles ? page_of(j + 1) : 0;
+      if (j < ntiles) {
+        const int row = p.block_size > kBKeys ? (j * kBKeys) % p.block_size : row_in_page;
+        for (int c = 0; c < nkc; ++c) {
+          ok = __all_sync(0xffffffffu, mbar_wait(&bars->k_empty[sl], ph, p.status));
+          if (!ok) break;
+          if (lane == 0) mbar_expect_tx(&bars->k_full[sl], kChunkBytes);
+          __syncwarp();
+          if (lane < loads)
+            tma_load_3d(sK + sl * kChunkBytes + dst_off, &tmK, &bars->k_full[sl], c * 64, row, blk);
+          if (++sl == p.k_slots) { sl = 0; ph ^= 1; }
         }
       }
+      if (j >= 1 && ok) {
+        const int i = j - 1, vs = i % kVSlots;
+        const int row = p.block_size > kBKeys ? (i * kBKeys) % p.block_size : row_in_page;
+        ok = __all_sync(0xffffffffu, mbar_wait(&bars->v_empty[vs], ((i / kVSlots) & 1) ^ 1, p.status));
+        if (!ok) break;
+        if (lane == 0) mbar_expect_tx(&bars->v_full[vs], nvc * kChunkBytes);
+        __syncwarp();
+        if (lane < loads)
+          for (int c = 0; c < nvc; ++c)
+            tma_load_3d(sV + (vs * nvc + c) * kChunkBytes + dst_off, &tmV, &bars->v_full[vs], hkv * p.vdim + c * 64,
+                        row, blk_prev);
+      }
+      blk_prev = blk;
+      blk = next;
     }
   } else if (warp == 1) {
     if (lane == 0) {
@@ -597,20 +676,30 @@ __global__ void __launch_bounds__(192)
       const uint32_t idesc_pv = umma_idesc_bf16(kBQ, (p.vdim + 15) & ~15, 0, 1);
       bool ok = mbar_wait(&bars->q_full, 0, p.status);
       const uint32_t q_addr = smem_u32(sQ), k_addr0 = smem_u32(sK), v_addr0 = smem_u32(sV), p_addr = smem_u32(sP);
-      uint32_t kc = 0;
+      // descriptors advance by plain adds: 16 k elements are 32 bytes = 2 address units
+      const uint64_t qd0 = umma_desc_k_sw128(q_addr, 1024), kd0 = umma_desc_k_sw128(k_addr0, 1024);
+      const int tail = (p.kw - (nkc - 1) * 64 + 15) / 16;          // instructions of the last chunk
+      int ksl = 0;
+      uint32_t kph = 0;
       for (int j = 0; j <= ntiles && ok; ++j) {
         if (j < ntiles) {
           const int sb = j & 1;
+          const uint32_t d = tmem_s0 + sb * kBKeys;
           if (!mbar_wait(&bars->s_empty[sb], ((j >> 1) & 1) ^ 1, p.status)) { ok = false; break; }
-          for (int c = 0; c < nkc; ++c, ++kc) {
-            const int sl = kc % p.k_slots;
-            if (!mbar_wait(&bars->k_full[sl], (kc / p.k_slots) & 1, p.status)) { ok = false; break; }
+          for (int c = 0; c < nkc; ++c) {
+            if (!mbar_wait(&bars->k_full[ksl], kph, p.status)) { ok = false; break; }
             tc_fence_after_sync();
-            const int steps = min(4, (p.kw - c * 64 + 15) / 16);
-            for (int kk = 0; kk < steps; ++kk)
-              umma_bf16_ss(tmem_s0 + sb * kBKeys, umma_desc_k_sw128(q_addr + c * kQChunkBytes + kk * 32, 1024),
-                           umma_desc_k_sw128(k_addr0 + sl * kChunkBytes + kk * 32, 1024), idesc_qk, (c | kk) != 0);
-            umma_commit(&bars->k_empty[sl]);
+            const uint64_t qd = qd0 + c * (kQChunkBytes >> 4), kd = kd0 + ksl * (kChunkBytes >> 4);
+            umma_bf16_ss(d, qd, kd, idesc_qk, c != 0);
+            if (c + 1 < nkc || tail == 4) {
+              umma_bf16_ss(d, qd + 2, kd + 2, idesc_qk, 1);
+              umma_bf16_ss(d, qd + 4, kd + 4, idesc_qk, 1);
+              umma_bf16_ss(d, qd + 6, kd + 6, idesc_qk, 1);
+            } else {
+              for (int kk = 1; kk < tail; ++kk) umma_bf16_ss(d, qd + 2 * kk, kd + 2 * kk, idesc_qk, 1);
+            }
+            umma_commit(&bars->k_empty[ksl]);
+            if (++ksl == p.k_slots) { ksl = 0; kph ^= 1; }
           }
           if (!ok) break;
           umma_commit(&bars->s_full[sb]);
@@ -882,6 +971,43 @@ static int launch_mix(const MixParams& p, int gy, cudaStream_t stream) {
                  cudaSuccess ? 0 : -2;
 }
 
+template <typename TO, int RR>
+static int launch_mix_vec(const MixParams& p, cudaStream_t stream) {
+  const int sms = b200_num_sms();
+  const long threads = (long)p.T * p.G * p.dim / 4;
+  int slices = 1;                          // few tokens: the output heads are dealt out to more blocks
+  while (slices < p.H && slices < 16 && (threads + 255) / 256 * slices < 2l * sms) slices *= 2;
+  int hpb = (p.H + slices - 1) / slices;
+  slices = (p.H + hpb - 1) / hpb;
+  const size_t smem = (size_t)hpb * p.H * 4;
+  if (smem > 96 * 1024) return -5;         // (the caller takes the other kernel)
+  static PerDeviceOnce once;
+  if (once.first())
+    cudaFuncSetAttribute(head_mix_kv_vec_kernel<TO, RR>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
+  long gx = (threads + 255) / 256;
+  if (gx > 16l * sms) gx = 16l * sms;
+  return launch_pdl(head_mix_kv_vec_kernel<TO, RR>, dim3((unsigned)gx, slices + 1), dim3(256), smem, stream, p, hpb) ==
+                 cudaSuccess ? 0 : -2;
+}
+template <typename TO>
+static int launch_mix_vec(const MixParams& p, cudaStream_t stream) {
+  const size_t es = sizeof(TO);
+  if ((p.dim & 3) || (p.vdim & 3) || (p.ld & 3) || (p.ldq & 3) || ((uintptr_t)p.qkv & 15) ||
+      ((uintptr_t)p.q_out & (4 * es - 1)) || ((uintptr_t)p.cache & (4 * es - 1)))
+    return -5;
+  switch (p.H / p.G) {
+    case 1: return launch_mix_vec<TO, 1>(p, stream);
+    case 2: return launch_mix_vec<TO, 2>(p, stream);
+    case 3: return launch_mix_vec<TO, 3>(p, stream);
+    case 4: return launch_mix_vec<TO, 4>(p, stream);
+    case 6: return launch_mix_vec<TO, 6>(p, stream);
+    case 8: return launch_mix_vec<TO, 8>(p, stream);
+    case 12: return launch_mix_vec<TO, 12>(p, stream);
+    case 16: return launch_mix_vec<TO, 16>(p, stream);
+    default: return -5;
+  }
+}
+
 static bool valid_args(const B200BiasAttn* a) {
   return a->H > 0 && a->G > 0 && a->H % a->G == 0 && a->kw > 0 && a->vdim > 0 && a->block_size > 0 &&
          (!a->bias || a->bias_len > 0);
@@ -899,6 +1025,8 @@ int b200_head_mix_kv(const void* qkv, long long ld, const void* mix, void* q_out
   if (H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || block_size <= 0) return -1;
   MixParams p{(const float*)qkv, ld, (const float*)mix, q_out, ldq, (const int64_t*)slots, cache, H, G, dim, vdim,
               block_size, T};
+  const int rc = f32 ? launch_mix_vec<float>(p, stream) : launch_mix_vec<__nv_bfloat16>(p, stream);
+  if (rc != -5) return rc;
   // few tokens: one per CTA, so that more SMs take part
   const int gy = (H + kMixHeads - 1) / kMixHeads;
   const size_t wide = ((size_t)kMixHeads * H + 4 * (size_t)H * dim) * 4;

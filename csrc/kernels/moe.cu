@@ -281,6 +281,7 @@ struct GroupedParams {
 struct alignas(8) GroupedBars {
   uint64_t full[kGMaxStages], empty[kGMaxStages], acc_full;
   uint32_t tmem_base;
+  float row_w[256];        // clamped pair: routing weights of the chunk's rows
 };
 
 // grid: (N / 128, max_chunks). A CTA whose chunk index is past the device-side count exits.
@@ -353,6 +354,11 @@ __global__ void __launch_bounds__(192, 1)
     }
   } else if (gated) {
     const int quarter = warp & 3;
+    if (p.act_fuse == 4) {
+      for (int i = threadIdx.x - 64; i < 256; i += 128)
+        bars->row_w[i] = p.clamp.row_w && i < rows ? p.clamp.row_w[row0 + i] : 1.f;
+      asm volatile("bar.sync 1, 128;" ::: "memory");      // the four epilogue warps
+    }
     bool ok = __all_sync(0xffffffffu, mbar_wait(&bars->acc_full, 0, p.status));
     tc_fence_after_sync();
     const int n = tn * kGBM + quarter * 32 + lane;        // output column of this thread
@@ -369,11 +375,11 @@ __global__ void __launch_bounds__(192, 1)
           for (int i = 0; i < 16; ++i) {
             const int m = c * 16 + i;
             if (m < rows) {
-              const float w = p.clamp.row_w ? __ldg(p.clamp.row_w + row0 + m) : 1.f;
+              const float w = bars->row_w[m];
               const float gg = fminf(__uint_as_float(g[i]) * w, p.clamp.limit);
               const float uu = fminf(fmaxf(__uint_as_float(u[i]) * w, -p.clamp.limit), p.clamp.limit);
               p.out[(size_t)(row0 + m) * half_n + n] =
-                  __float2bfloat16(gg / (1.f + __expf(-p.clamp.alpha * gg)) * (uu + p.clamp.up_offset));
+                  __float2bfloat16(__fdividef(gg, 1.f + __expf(-p.clamp.alpha * gg)) * (uu + p.clamp.up_offset));
             }
           }
         }
