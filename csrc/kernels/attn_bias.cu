@@ -198,7 +198,7 @@ struct BiasAttnParams {
   // prefill
   const int32_t* tile_req;
   const int32_t* tile_q0;
-  int k_slots, bias_smem;
+  int k_slots, v_slots, q_stream;
   int* status;
 };
 
@@ -558,17 +558,25 @@ __global__ void __launch_bounds__(kDecWarps * 32, 1) bias_attn_decode_kernel(Bia
 }
 
 // --------------------------------------------------------------------------------- prefill (bf16)
-// One CTA = one 128-row query tile of one request and one head. The query tile (all 64-wide chunks
-// of the query row) stays in shared memory; key tiles arrive chunk by chunk (64 keys x 64 dims) in a
-// ring, value tiles in a second ring of two. S is double-buffered in TMEM, O accumulates there.
-// Warps: 0 TMA producer, 1 MMA issuer + TMEM owner, 2..5 softmax (one thread per query row).
-static constexpr int kBQ = 128, kBKeys = 64, kChunkBytes = kBKeys * 128, kQChunkBytes = kBQ * 128;
-static constexpr int kVSlots = 2, kMaxKSlots = 8;
+// One CTA = one 128-row query tile of one request and one head, key tiles of 128. The query row of a
+// head is as wide as all key heads together (kw), so the score product is cut into 64-wide chunks that
+// arrive in a ring; the query tile stays in shared memory when it fits (else its chunks ride in the
+// ring beside the keys'). S is double-buffered in TMEM, P goes back to TMEM as bf16 and is the A operand
+// of P V, O accumulates in TMEM (lazy reference maximum, in-place rescale).
+// Warps: 0 TMA producer, 1 MMA issuer + TMEM owner, 2..9 softmax, two threads per query row (64 keys
+// each) that exchange their row maximum through shared memory.
+// The bias of a warp's 32 rows and 128 keys depends on 159 distances only: the pair of warps keeps
+// that window of the table in shared memory, filled one tile ahead.
+static constexpr int kBQ = 128, kBKeys = 128, kChunkBytes = 128 * 128;   // chunk: 128 rows x 64 bf16
+static constexpr int kMaxKSlots = 8, kMinKSlots = 3, kWin = 160;
+static constexpr int kPrefillThreads = 320;
 
 struct alignas(8) BiasPrefillBars {
-  uint64_t q_full, k_full[kMaxKSlots], k_empty[kMaxKSlots], v_full[kVSlots], v_empty[kVSlots];
-  uint64_t s_full[2], s_empty[2], p_full, p_empty, o_full;
+  uint64_t q_full, k_full[kMaxKSlots], k_empty[kMaxKSlots], v_full[2], v_empty[2];
+  uint64_t s_full[2], s_empty[2], p_full[2], p_empty[2], o_full;
   uint32_t tmem_base;
+  float row_max[2][2][kBQ];          // [tile parity][half][row]
+  float window[2][4][kWin];          // [tile parity][quarter]: log2-domain bias by distance
 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
@@ -576,20 +584,21 @@ __device__ __forceinline__ float ex2_approx(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+__device__ __forceinline__ void pair_sync(int quarter) {             // the two warps of a row quarter
+  asm volatile("bar.sync %0, 64;" ::"r"(quarter + 1) : "memory");
+}
 
-__global__ void __launch_bounds__(192)
+__global__ void __launch_bounds__(kPrefillThreads, 1)
     bias_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                              const __grid_constant__ CUtensorMap tmV, BiasAttnParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int nkc = (p.kw + 63) / 64, nvc = (p.vdim + 63) / 64;
+  const int slot_bytes = p.q_stream ? 2 * kChunkBytes : kChunkBytes;      // [keys | queries]
   uint8_t* sQ = smem;
-  uint8_t* sK = sQ + nkc * kQChunkBytes;
-  uint8_t* sV = sK + p.k_slots * kChunkBytes;
-  uint8_t* sP = sV + kVSlots * nvc * kChunkBytes;
-  float* sB = reinterpret_cast<float*>(sP + kQChunkBytes);
-  BiasPrefillBars* bars =
-      reinterpret_cast<BiasPrefillBars*>(reinterpret_cast<uint8_t*>(sB) + ((p.bias_smem * 4 + 15) & ~15));
+  uint8_t* sK = sQ + (p.q_stream ? 0 : nkc * kChunkBytes);
+  uint8_t* sV = sK + p.k_slots * slot_bytes;
+  BiasPrefillBars* bars = reinterpret_cast<BiasPrefillBars*>(sV + p.v_slots * nvc * kChunkBytes);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int tile = blockIdx.x, h = blockIdx.y, hkv = h / (p.H / p.G);
   const int req = p.tile_req[tile], q0 = p.tile_q0[tile];
@@ -597,28 +606,32 @@ __global__ void __launch_bounds__(192)
   const int seq_len = p.seq_lens[req], ctx_off = seq_len - q_len;
   const int rows = min(kBQ, q_len - q0);
   const int ntiles = (ctx_off + q0 + rows - 1) / kBKeys + 1;
-  const uint32_t tmem_cols = p.vdim > 128 ? 512 : 256;
+  // TMEM columns: S buffers (128 each), then O, then two P buffers (64 each)
+  const int s_bufs = p.vdim > 128 ? 1 : 2;
+  const int o_cols = p.vdim > 128 ? 256 : 128;
 
   if (threadIdx.x == 0) {
     mbar_init(&bars->q_full, 1);
     for (int i = 0; i < p.k_slots; ++i) { mbar_init(&bars->k_full[i], 1); mbar_init(&bars->k_empty[i], 1); }
-    for (int i = 0; i < kVSlots; ++i) { mbar_init(&bars->v_full[i], 1); mbar_init(&bars->v_empty[i], 1); }
-    for (int i = 0; i < 2; ++i) { mbar_init(&bars->s_full[i], 1); mbar_init(&bars->s_empty[i], 4); }
-    mbar_init(&bars->p_full, 4);
-    mbar_init(&bars->p_empty, 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&bars->v_full[i], 1);
+      mbar_init(&bars->v_empty[i], 1);
+      mbar_init(&bars->s_full[i], 1);
+      mbar_init(&bars->s_empty[i], 8);
+      mbar_init(&bars->p_full[i], 8);
+      mbar_init(&bars->p_empty[i], 1);
+    }
     mbar_init(&bars->o_full, 1);
     mbar_fence_init();
   }
-  if (warp == 1) { tmem_alloc(&bars->tmem_base, tmem_cols); tmem_relinquish(); }
-  const float* bias = p.bias ? p.bias + (size_t)h * p.bias_len : nullptr;
-  for (int i = threadIdx.x; i < p.bias_smem; i += blockDim.x) sB[i] = bias[i] * kLog2e;
+  if (warp == 1) { tmem_alloc(&bars->tmem_base, 512); tmem_relinquish(); }
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
-  const uint32_t tmem_base = bars->tmem_base, tmem_s0 = tmem_base, tmem_o = tmem_base + 128;
+  const uint32_t tmem_s = bars->tmem_base, tmem_o = tmem_s + s_bufs * kBKeys, tmem_p = tmem_o + o_cols;
 
   if (warp == 0) {
-    // A 64-key tile spans up to eight pages; lane l fetches the rows of the l-th one, so the page
+    // A 128-key tile spans up to 16 pages; lane l fetches the rows of the l-th one, so the page
     // look-ups of a tile run side by side.
     const int rpl = min(p.block_size, kBKeys), loads = kBKeys / rpl;
     const int32_t* bt = p.block_table + (size_t)req * p.max_blocks;
@@ -627,15 +640,17 @@ __global__ void __launch_bounds__(192)
       const int bi = (j * kBKeys + lane * rpl) / p.block_size;
       return max(lane < loads && bi < nblk ? bt[bi] : bt[0], 0);
     };
-    const int row_in_page = (lane * rpl) % p.block_size;            // block_size <= 64
+    const int row_in_page = (lane * rpl) % p.block_size;
     const int dst_off = lane * rpl * 128;
     if (lane == 0) {
       tma_prefetch_desc(&tmQ);
       tma_prefetch_desc(&tmK);
       tma_prefetch_desc(&tmV);
-      mbar_expect_tx(&bars->q_full, nkc * kQChunkBytes);
-      for (int c = 0; c < nkc; ++c)
-        tma_load_2d(sQ + c * kQChunkBytes, &tmQ, &bars->q_full, h * p.kw + c * 64, q_begin + q0);
+      if (!p.q_stream) {
+        mbar_expect_tx(&bars->q_full, nkc * kChunkBytes);
+        for (int c = 0; c < nkc; ++c)
+          tma_load_2d(sQ + c * kChunkBytes, &tmQ, &bars->q_full, h * p.kw + c * 64, q_begin + q0);
+      }
     }
     int sl = 0, blk = page_of(0), blk_prev = 0;
     uint32_t ph = 1;
@@ -648,17 +663,21 @@ __global__ void __launch_bounds__(192)
         for (int c = 0; c < nkc; ++c) {
           ok = __all_sync(0xffffffffu, mbar_wait(&bars->k_empty[sl], ph, p.status));
           if (!ok) break;
-          if (lane == 0) mbar_expect_tx(&bars->k_full[sl], kChunkBytes);
+          uint8_t* dst = sK + sl * slot_bytes;
+          if (lane == 0) {
+            mbar_expect_tx(&bars->k_full[sl], slot_bytes);
+            if (p.q_stream)
+              tma_load_2d(dst + kChunkBytes, &tmQ, &bars->k_full[sl], h * p.kw + c * 64, q_begin + q0);
+          }
           __syncwarp();
-          if (lane < loads)
-            tma_load_3d(sK + sl * kChunkBytes + dst_off, &tmK, &bars->k_full[sl], c * 64, row, blk);
+          if (lane < loads) tma_load_3d(dst + dst_off, &tmK, &bars->k_full[sl], c * 64, row, blk);
           if (++sl == p.k_slots) { sl = 0; ph ^= 1; }
         }
       }
       if (j >= 1 && ok) {
-        const int i = j - 1, vs = i % kVSlots;
+        const int i = j - 1, vs = i % p.v_slots;
         const int row = p.block_size > kBKeys ? (i * kBKeys) % p.block_size : row_in_page;
-        ok = __all_sync(0xffffffffu, mbar_wait(&bars->v_empty[vs], ((i / kVSlots) & 1) ^ 1, p.status));
+        ok = __all_sync(0xffffffffu, mbar_wait(&bars->v_empty[vs], ((i / p.v_slots) & 1) ^ 1, p.status));
         if (!ok) break;
         if (lane == 0) mbar_expect_tx(&bars->v_full[vs], nvc * kChunkBytes);
         __syncwarp();
@@ -674,22 +693,23 @@ __global__ void __launch_bounds__(192)
     if (lane == 0) {
       const uint32_t idesc_qk = umma_idesc_bf16(kBQ, kBKeys, 0, 0);
       const uint32_t idesc_pv = umma_idesc_bf16(kBQ, (p.vdim + 15) & ~15, 0, 1);
-      bool ok = mbar_wait(&bars->q_full, 0, p.status);
-      const uint32_t q_addr = smem_u32(sQ), k_addr0 = smem_u32(sK), v_addr0 = smem_u32(sV), p_addr = smem_u32(sP);
+      bool ok = p.q_stream || mbar_wait(&bars->q_full, 0, p.status);
       // descriptors advance by plain adds: 16 k elements are 32 bytes = 2 address units
-      const uint64_t qd0 = umma_desc_k_sw128(q_addr, 1024), kd0 = umma_desc_k_sw128(k_addr0, 1024);
+      const uint64_t qd0 = umma_desc_k_sw128(smem_u32(sQ), 1024), kd0 = umma_desc_k_sw128(smem_u32(sK), 1024);
+      const uint64_t vd0 = umma_desc_mn_sw128(smem_u32(sV), kChunkBytes, 1024);
       const int tail = (p.kw - (nkc - 1) * 64 + 15) / 16;          // instructions of the last chunk
       int ksl = 0;
       uint32_t kph = 0;
       for (int j = 0; j <= ntiles && ok; ++j) {
         if (j < ntiles) {
-          const int sb = j & 1;
-          const uint32_t d = tmem_s0 + sb * kBKeys;
-          if (!mbar_wait(&bars->s_empty[sb], ((j >> 1) & 1) ^ 1, p.status)) { ok = false; break; }
+          const int sb = j % s_bufs;
+          const uint32_t d = tmem_s + sb * kBKeys;
+          if (!mbar_wait(&bars->s_empty[sb], ((j / s_bufs) & 1) ^ 1, p.status)) { ok = false; break; }
           for (int c = 0; c < nkc; ++c) {
             if (!mbar_wait(&bars->k_full[ksl], kph, p.status)) { ok = false; break; }
             tc_fence_after_sync();
-            const uint64_t qd = qd0 + c * (kQChunkBytes >> 4), kd = kd0 + ksl * (kChunkBytes >> 4);
+            const uint64_t kd = kd0 + ksl * (slot_bytes >> 4);
+            const uint64_t qd = p.q_stream ? kd + (kChunkBytes >> 4) : qd0 + c * (kChunkBytes >> 4);
             umma_bf16_ss(d, qd, kd, idesc_qk, c != 0);
             if (c + 1 < nkc || tail == 4) {
               umma_bf16_ss(d, qd + 2, kd + 2, idesc_qk, 1);
@@ -705,61 +725,67 @@ __global__ void __launch_bounds__(192)
           umma_commit(&bars->s_full[sb]);
         }
         if (j >= 1) {
-          const int i = j - 1, sl = i % kVSlots;
-          if (!mbar_wait(&bars->v_full[sl], (i / kVSlots) & 1, p.status)) { ok = false; break; }
-          if (!mbar_wait(&bars->p_full, i & 1, p.status)) { ok = false; break; }
+          const int i = j - 1, vs = i % p.v_slots, pb = i & 1;
+          if (!mbar_wait(&bars->v_full[vs], (i / p.v_slots) & 1, p.status)) { ok = false; break; }
+          if (!mbar_wait(&bars->p_full[pb], (i >> 1) & 1, p.status)) { ok = false; break; }
           tc_fence_after_sync();
-          const uint32_t v_addr = v_addr0 + sl * nvc * kChunkBytes;
+          const uint64_t vd = vd0 + vs * nvc * (kChunkBytes >> 4);
 #pragma unroll
-          for (int kk = 0; kk < kBKeys / 16; ++kk)
-            umma_bf16_ss(tmem_o, umma_desc_k_sw128(p_addr + kk * 32, 1024),
-                         umma_desc_mn_sw128(v_addr + kk * 2048, kChunkBytes, 1024), idesc_pv, (i | kk) != 0);
-          umma_commit(&bars->v_empty[sl]);
-          umma_commit(&bars->o_full);
-          umma_commit(&bars->p_empty);
+          for (int kk = 0; kk < kBKeys / 16; ++kk)                  // 16 keys: 8 columns of P, 2048 B of V
+            umma_bf16_ts(tmem_o, tmem_p + pb * 64 + kk * 8, vd + kk * 128, idesc_pv, (i | kk) != 0);
+          umma_commit(&bars->v_empty[vs]);
+          umma_commit(&bars->p_empty[pb]);
+          if (i == ntiles - 1) umma_commit(&bars->o_full);
         }
       }
     }
   } else {
-    const int quarter = warp & 3, r = quarter * 32 + lane;
+    const int quarter = warp & 3, half = (warp - 2) >> 2, r = quarter * 32 + lane;
     const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
     const int q_pos = ctx_off + q0 + r, hi = min(q_pos, seq_len - 1);
     const int warp_pos0 = ctx_off + q0 + quarter * 32;       // position of the warp's first row
-    // m: reference maximum in the log2 domain, raised lazily (by more than 2^8). The null entry
-    // is the state before the first key: score 0, weight 1.
-    float m = p.null_entry ? 0.f : -INFINITY, l = p.null_entry ? 1.f : 0.f;
-    const float far = bias ? bias[p.bias_len - 1] * kLog2e : 0.f;
+    const int key0 = half * 64;                              // this thread's keys inside a tile
+    const float* bias = p.bias ? p.bias + (size_t)h * p.bias_len : nullptr;
+    const int last = p.bias_len - 1;
+    const float far = bias ? bias[last] * kLog2e : 0.f;
+    // Window entry e of tile j holds the bias of distance d0 - e, d0 = warp_pos0 + 31 - j * 128; key k
+    // of the tile is entry 31 - lane + k for this row. Tiles that lie wholly beyond the table need none.
+    auto tile_near = [&](int j) { return bias && warp_pos0 - (j * kBKeys + kBKeys - 1) < last; };
+    auto fill_window = [&](int j) {
+      const int d0 = warp_pos0 + 31 - j * kBKeys;
+#pragma unroll
+      for (int i = 0; i < 3; ++i) {
+        const int e = half * 32 + lane + i * 64;
+        if (e < kWin) bars->window[j & 1][quarter][e] = bias[min(max(d0 - e, 0), last)] * kLog2e;
+      }
+    };
+    // m: reference maximum of the row in the log2 domain (the same in both threads of a row), raised
+    // lazily, by more than 2^8. The null entry is the state before the first key: score 0, weight 1.
+    float m = p.null_entry ? 0.f : -INFINITY, l = p.null_entry && half == 0 ? 1.f : 0.f;
     bool ok = true;
-    uint8_t* prow = sP + r * 128;
     const int vcols = (p.vdim + 31) / 32;
-    for (int j = 0; j < ntiles && ok; ++j) {
-      const int sb = j & 1, kbase = j * kBKeys;
-      ok = __all_sync(0xffffffffu, mbar_wait(&bars->s_full[sb], (j >> 1) & 1, p.status));
-      if (!ok) break;
+    if (tile_near(0)) fill_window(0);
+    pair_sync(quarter);
+    for (int j = 0; j < ntiles; ++j) {
+      const int sb = j % s_bufs, pb = j & 1, kbase = j * kBKeys + key0;
+      // after a wait that ran out the warp goes through the motions without waiting, so that its
+      // partner is never left at a barrier
+      ok = ok && __all_sync(0xffffffffu, mbar_wait(&bars->s_full[sb], (j / s_bufs) & 1, p.status));
       tc_fence_after_sync();
-      const uint32_t s_addr = tmem_s0 + sb * kBKeys + lane_off;
       uint32_t s0[32], s1[32];
+      const uint32_t s_addr = tmem_s + sb * kBKeys + key0 + lane_off;
       tmem_ld_32x32b_x32(s_addr, s0);
       tmem_ld_32x32b_x32(s_addr + 32, s1);
       tmem_ld_wait();
       tc_fence_before_sync();
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->s_empty[sb]);
-      const bool need_mask = kbase + kBKeys - 1 > warp_pos0;                    // warp-uniform
-      const bool near = bias && warp_pos0 - (kbase + kBKeys - 1) < p.bias_len - 1;
-      if (near || need_mask) {
+      if (tile_near(j)) {
+        const float* w = bars->window[j & 1][quarter] + 31 - lane + key0;
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          const int ka = kbase + i, kb = ka + 32;
-          float ba = far, bb = far;
-          if (near) {
-            const int da = min(max(q_pos - ka, 0), p.bias_len - 1), db = min(max(q_pos - kb, 0), p.bias_len - 1);
-            ba = p.bias_smem ? sB[da] : __ldg(bias + da) * kLog2e;
-            bb = p.bias_smem ? sB[db] : __ldg(bias + db) * kLog2e;
-          }
-          const float a = fmaf(__uint_as_float(s0[i]), kLog2e, ba), b = fmaf(__uint_as_float(s1[i]), kLog2e, bb);
-          s0[i] = __float_as_uint(ka > hi ? -INFINITY : a);
-          s1[i] = __float_as_uint(kb > hi ? -INFINITY : b);
+          s0[i] = __float_as_uint(fmaf(__uint_as_float(s0[i]), kLog2e, w[i]));
+          s1[i] = __float_as_uint(fmaf(__uint_as_float(s1[i]), kLog2e, w[i + 32]));
         }
       } else {
 #pragma unroll
@@ -768,13 +794,24 @@ __global__ void __launch_bounds__(192)
           s1[i] = __float_as_uint(fmaf(__uint_as_float(s1[i]), kLog2e, far));
         }
       }
+      if (kbase + 63 > min(warp_pos0, seq_len - 1)) {                    // (warp-uniform)
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          if (kbase + i > hi) s0[i] = __float_as_uint(-INFINITY);
+          if (kbase + 32 + i > hi) s1[i] = __float_as_uint(-INFINITY);
+        }
+      }
       float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
       for (int i = 0; i < 32; ++i) {
         mx0 = fmaxf(mx0, __uint_as_float(s0[i]));
         mx1 = fmaxf(mx1, __uint_as_float(s1[i]));
       }
-      const float tile_max = fmaxf(mx0, mx1);
+      float tile_max = fmaxf(mx0, mx1);
+      bars->row_max[pb][half][r] = tile_max;
+      if (j + 1 < ntiles && tile_near(j + 1)) fill_window(j + 1);
+      pair_sync(quarter);
+      tile_max = fmaxf(tile_max, bars->row_max[pb][half ^ 1][r]);
       float alpha = 1.f;
       bool rescale = false;
       if (tile_max > m + 8.f) {
@@ -782,11 +819,12 @@ __global__ void __launch_bounds__(192)
         m = tile_max;
       }
       const float m_use = m == -INFINITY ? 0.f : m;
-      ok = __all_sync(0xffffffffu, mbar_wait(&bars->p_empty, (j & 1) ^ 1, p.status));
-      if (!ok) break;
+      // the P buffer is free once the product of two tiles ago has run
+      ok = ok && __all_sync(0xffffffffu, mbar_wait(&bars->p_empty[pb], ((j >> 1) & 1) ^ 1, p.status));
       if (__any_sync(0xffffffffu, rescale)) {
+        ok = ok && __all_sync(0xffffffffu, mbar_wait(&bars->p_empty[pb ^ 1], ((j - 1) >> 1) & 1, p.status));
         tc_fence_after_sync();
-        for (int c = 0; c < vcols; ++c) {
+        for (int c = half; c < vcols; c += 2) {
           uint32_t rr[32];
           tmem_ld_32x32b_x32(tmem_o + lane_off + c * 32, rr);
           tmem_ld_wait();
@@ -794,35 +832,39 @@ __global__ void __launch_bounds__(192)
           for (int i = 0; i < 32; ++i) rr[i] = __float_as_uint(__uint_as_float(rr[i]) * alpha);
           tmem_st_32x32b_x32(tmem_o + lane_off + c * 32, rr);
         }
-        tmem_st_wait();
       }
+      tc_fence_after_sync();
       float rs0 = 0.f, rs1 = 0.f;
 #pragma unroll
-      for (int c = 0; c < 8; ++c) {
-        uint32_t pk[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int i = (c & 3) * 8 + e * 2;
-          const float x0 = __uint_as_float(c < 4 ? s0[i] : s1[i]), x1 = __uint_as_float(c < 4 ? s0[i + 1] : s1[i + 1]);
-          const float p0 = ex2_approx(x0 - m_use), p1 = ex2_approx(x1 - m_use);
-          rs0 += p0;
-          rs1 += p1;
-          pk[e] = pack_bf16x2(p0, p1);
-        }
-        *reinterpret_cast<uint4*>(prow + ((c ^ (r & 7)) << 4)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+      for (int i = 0; i < 16; ++i) {
+        const float a0 = ex2_approx(__uint_as_float(s0[2 * i]) - m_use), a1 = ex2_approx(__uint_as_float(s0[2 * i + 1]) - m_use);
+        rs0 += a0;
+        rs1 += a1;
+        s0[i] = pack_bf16x2(a0, a1);
       }
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const float a0 = ex2_approx(__uint_as_float(s1[2 * i]) - m_use), a1 = ex2_approx(__uint_as_float(s1[2 * i + 1]) - m_use);
+        rs0 += a0;
+        rs1 += a1;
+        s0[16 + i] = pack_bf16x2(a0, a1);
+      }
+      tmem_st_32x32b_x32(tmem_p + pb * 64 + half * 32 + lane_off, s0);
+      tmem_st_wait();
       l = l * alpha + (rs0 + rs1);
-      fence_proxy_async_smem();
       tc_fence_before_sync();
       __syncwarp();
-      if (lane == 0) mbar_arrive(&bars->p_full);
+      if (lane == 0) mbar_arrive(&bars->p_full[pb]);
     }
-    if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->o_full, (ntiles - 1) & 1, p.status));
+    bars->row_max[ntiles & 1][half][r] = l;       // (the slot read in the last tile has the other parity)
+    pair_sync(quarter);
+    l += bars->row_max[ntiles & 1][half ^ 1][r];
+    if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->o_full, 0, p.status));
     if (ok) {
       tc_fence_after_sync();
       const float inv = l > 0.f ? 1.f / l : 0.f;
       __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(q_begin + q0 + r) * p.ldo + (size_t)h * p.vdim;
-      for (int c = 0; c < vcols; ++c) {
+      for (int c = half; c < vcols; c += 2) {
         uint32_t rr[32];
         tmem_ld_32x32b_x32(tmem_o + lane_off + c * 32, rr);
         tmem_ld_wait();
@@ -845,7 +887,7 @@ __global__ void __launch_bounds__(192)
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
-  if (warp == 1) tmem_dealloc(tmem_base, tmem_cols);
+  if (warp == 1) tmem_dealloc(bars->tmem_base, 512);
 }
 
 // ------------------------------------------------------------------------------------ host helpers
@@ -873,17 +915,21 @@ static bool prefill_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem)
   const int bs = a->block_size;
   if (bs < 8 || (bs & 7) || (bs < kBKeys && kBKeys % bs) || (bs > kBKeys && bs % kBKeys)) return false;
   const int nkc = (a->kw + 63) / 64, nvc = (a->vdim + 63) / 64;
-  p.bias_smem = a->bias && a->bias_len <= 1024 ? a->bias_len : 0;
-  const size_t fixed = (size_t)nkc * kQChunkBytes + kVSlots * nvc * kChunkBytes + kQChunkBytes +
-                       ((p.bias_smem * 4 + 15) & ~15) + sizeof(BiasPrefillBars) + 1024;
-  const size_t limit = 226 * 1024;
-  if (fixed + 2 * kChunkBytes > limit) return false;
-  // two CTAs on an SM where the query rows are short enough, else as deep a key ring as fits
-  int slots = fixed + 3 * kChunkBytes <= 112 * 1024 ? (int)((112 * 1024 - fixed) / kChunkBytes)
-                                                    : (int)((limit - fixed) / kChunkBytes);
-  p.k_slots = slots > kMaxKSlots ? kMaxKSlots : slots;
-  smem = fixed + (size_t)p.k_slots * kChunkBytes;
-  return true;
+  const int limit = 227 * 1024, fixed = (int)sizeof(BiasPrefillBars) + 1024;
+  // the query tile stays in shared memory if enough of the key ring fits beside it
+  for (p.q_stream = 0; p.q_stream < 2; ++p.q_stream) {
+    const int slot = (p.q_stream ? 2 : 1) * kChunkBytes, resident = p.q_stream ? 0 : nkc * kChunkBytes;
+    for (p.v_slots = 2; p.v_slots >= 1; --p.v_slots) {
+      const int left = limit - fixed - resident - p.v_slots * nvc * kChunkBytes;
+      p.k_slots = left < 0 ? 0 : left / slot;
+      if (p.k_slots > kMaxKSlots) p.k_slots = kMaxKSlots;
+      if (p.k_slots >= (p.v_slots == 2 ? kMinKSlots + 1 : kMinKSlots)) {
+        smem = (size_t)fixed + resident + p.v_slots * nvc * kChunkBytes + p.k_slots * slot;
+        return true;
+      }
+    }
+  }
+  return false;
 }
 
 struct PageMapKey {
@@ -1075,7 +1121,7 @@ int b200_bias_attn_prefill(const B200BiasAttn* a, int any_size, cudaStream_t str
     return -3;
   static PerDeviceOnce once;
   if (once.first()) cudaFuncSetAttribute(bias_attn_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
-  bias_attn_prefill_kernel<<<dim3(a->num_tiles, a->H), 192, smem, stream>>>(tmQ, tmK, tmV, p);
+  bias_attn_prefill_kernel<<<dim3(a->num_tiles, a->H), kPrefillThreads, smem, stream>>>(tmQ, tmK, tmV, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 

@@ -42,7 +42,7 @@ REGISTRY: list[AttentionBackend] = [
                      lambda head_dim, v_head_dim, f32=False, **_: not f32 and head_dim % 8 == 0 and v_head_dim % 8 == 0),
     AttentionBackend("tcgen05-bias-prefill", "prefill", "bias", 0, "b200_bias_attn_prefill",
                      lambda head_dim, v_head_dim, block_size, f32=False, **_: not f32 and head_dim % 8 == 0
-                     and v_head_dim % 8 == 0 and v_head_dim <= 256 and _pages_tile(block_size, 64)),
+                     and v_head_dim % 8 == 0 and v_head_dim <= 256 and _pages_tile(block_size, 128)),
     AttentionBackend("any-size-bias-decode", "decode", "bias", 1, "b200_bias_attn_decode", lambda **_: True),
     AttentionBackend("any-size-bias-prefill", "prefill", "bias", 1, "b200_bias_attn_prefill", lambda **_: True),
     AttentionBackend("mla-absorbed-decode", "decode", "mla", 0, "b200_mla_decode",
