@@ -14,9 +14,9 @@
 //
 // Three kernels:
 //   bias_attn_any_kernel      any sizes, float or bf16 storage, one CTA per (query row, 4 heads)
-//   bias_attn_decode_kernel   bf16, one query row per request: key / value rows arrive by bulk copies
-//                             in a shared-memory ring, all heads of a request share them, products on
-//                             mma.sync (the kernel is bound by the cache read), split-KV
+//   bias_attn_decode_kernel   bf16, one query row per request: key / value tiles arrive by TMA in two
+//                             rings, all heads of a request share them, products on mma.sync (few
+//                             query rows per key: the kernel is bound by the cache read), split-KV
 //   bias_attn_prefill_kernel  bf16, 128-row query tiles on tcgen05 / TMEM
 #include <float.h>
 
@@ -194,7 +194,7 @@ struct BiasAttnParams {
   int splits;
   float* tmp_o;             // [B, H, splits, vdim]
   float* tmp_lse;           // [B, H, splits]
-  int kwp, vwp, mt, stages, hp;
+  int mt, hp, ksplit;
   // prefill
   const int32_t* tile_req;
   const int32_t* tile_q0;
@@ -319,8 +319,8 @@ __device__ __forceinline__ void ldsm_x4(uint32_t* r, uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
-__device__ __forceinline__ void ldsm_x2(uint32_t* r, uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];"
+__device__ __forceinline__ void ldsm_x2_trans(uint32_t* r, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0, %1}, [%2];"
                : "=r"(r[0]), "=r"(r[1]) : "r"(addr) : "memory");
 }
 __device__ __forceinline__ void ldsm_x4_trans(uint32_t* r, uint32_t addr) {
@@ -334,211 +334,271 @@ __device__ __forceinline__ void mma_bf16_16816(float* d, const uint32_t* a, cons
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
 }
-// Untiled bulk copy global -> shared (16-byte aligned, a multiple of 16 bytes), counted on `bar`.
-__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
-  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-               ::"r"(smem_u32(dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
-}
+static constexpr int kDecWarps = 16;     // compute warps; one more feeds the rings
+static constexpr int kDecThreads = (kDecWarps + 1) * 32;
+static constexpr int kDecMaxSlots = 4, kDecHeads = 8;   // kDecHeads * kDecWarps heads at most
 
-static constexpr int kDecKeys = 32;      // keys per tile
-static constexpr int kDecWarps = 8;
-static constexpr int kDecMaxStages = 4;
-
-struct DecodeSmem {                      // byte offsets
-  int q, k, v, s, p, stat, bars, total;
+struct DecodeSmem {                      // byte offsets; the rings are 1024-byte aligned
+  int k, v, q, s, p, stat, bars, total;
 };
-__host__ __device__ inline DecodeSmem decode_smem(int hp, int kwp, int vwp, int prow, int stages) {
+__host__ __device__ inline DecodeSmem decode_smem(int tk, int hp, int nkc, int nvc, int prow, int ksplit, int k_slots,
+                                                  int v_slots) {
   DecodeSmem d;
   int o = 0;
-  d.q = o; o += hp * (kwp + 8) * 2;
-  d.k = o; o += stages * kDecKeys * (kwp + 8) * 2;
-  d.v = o; o += stages * kDecKeys * (vwp + 8) * 2;
-  d.s = o; o += hp * (kDecKeys + 1) * 4;
+  d.k = o; o += k_slots * nkc * tk * 128;
+  d.v = o; o += v_slots * nvc * tk * 128;
+  d.q = o; o += hp * (nkc * 64 + 8) * 2;
+  d.s = o; o += ksplit * hp * (tk + 1) * 4;
   o = (o + 15) & ~15;
-  d.p = o; o += prow * (kDecKeys + 8) * 2;
-  d.stat = o; o += 3 * hp * 4;
+  d.p = o; o += prow * (tk + 8) * 2;
+  d.stat = o; o += 2 * hp * 4;
   o = (o + 15) & ~15;
-  d.bars = o; o += kDecMaxStages * 8;
+  d.bars = o; o += 4 * kDecMaxSlots * 8;
   d.total = o;
   return d;
 }
 
-// grid (request, split). MAXI: 16 x 8 output tiles a warp keeps in registers.
-template <int MAXI>
-__global__ void __launch_bounds__(kDecWarps * 32, 1) bias_attn_decode_kernel(BiasAttnParams p) {
-  extern __shared__ __align__(16) uint8_t dec_smem[];
-  const int prow = p.G * p.mt * 16;
-  const DecodeSmem L = decode_smem(p.hp, p.kwp, p.vwp, prow, p.stages);
-  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(dec_smem + L.q);
-  __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(dec_smem + L.k);
-  __nv_bfloat16* sV = reinterpret_cast<__nv_bfloat16*>(dec_smem + L.v);
-  float* sS = reinterpret_cast<float*>(dec_smem + L.s);
-  __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(dec_smem + L.p);
-  float* s_alpha = reinterpret_cast<float*>(dec_smem + L.stat);
-  float* s_m = s_alpha + p.hp;
-  float* s_l = s_m + p.hp;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(dec_smem + L.bars);
+// grid (request, split). TK keys per tile; MAXI: 16 x 8 output tiles a warp keeps in registers. Key and
+// value rows arrive by TMA in 128-byte swizzled chunks of 64 columns. Per tile two barriers: the scores
+// of tile t run beside the output product of tile t - 1, then the softmax of tile t.
+template <int TK, int MAXI>
+__global__ void __launch_bounds__(kDecThreads, 1)
+    bias_attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
+                            BiasAttnParams p) {
+  extern __shared__ uint8_t dec_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(dec_raw) + 1023) & ~uintptr_t(1023));
+  const int nkc = (p.kw + 63) / 64, vw = p.G * p.vdim, nvc = (vw + 63) / 64, prow = p.G * p.mt * 16;
+  const DecodeSmem L = decode_smem(TK, p.hp, nkc, nvc, prow, p.ksplit, p.k_slots, p.v_slots);
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem + L.q);
+  float* sS = reinterpret_cast<float*>(smem + L.s);
+  __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(smem + L.p);
+  float* s_alpha = reinterpret_cast<float*>(smem + L.stat);
+  float* s_l = s_alpha + p.hp;
+  uint64_t* k_full = reinterpret_cast<uint64_t*>(smem + L.bars);
+  uint64_t *k_empty = k_full + kDecMaxSlots, *v_full = k_empty + kDecMaxSlots, *v_empty = v_full + kDecMaxSlots;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int b = blockIdx.x, split = blockIdx.y;
-  const int H = p.H, R = H / p.G, vw = p.G * p.vdim;
-  const int ks = p.kwp + 8, vs = p.vwp + 8, ps = kDecKeys + 8, ss = kDecKeys + 1;
+  const int H = p.H, R = H / p.G, qs = nkc * 64 + 8, ps = TK + 8, ss = TK + 1;
+  const int k_slot_bytes = nkc * TK * 128, v_slot_bytes = nvc * TK * 128;
 
-  // everything a product may read and no copy fills has to be finite: clear it once
-  for (int i = tid; i < L.s / 16; i += blockDim.x) reinterpret_cast<uint4*>(dec_smem)[i] = make_uint4(0, 0, 0, 0);
-  for (int i = tid; i < prow * ps / 8; i += blockDim.x) reinterpret_cast<uint4*>(sP)[i] = make_uint4(0, 0, 0, 0);
+  // what a product may read and nothing fills has to be finite
+  for (int i = tid; i < p.hp * qs / 8; i += kDecThreads) reinterpret_cast<uint4*>(sQ)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < prow * ps / 8; i += kDecThreads) reinterpret_cast<uint4*>(sP)[i] = make_uint4(0, 0, 0, 0);
   if (tid == 0) {
-    for (int i = 0; i < p.stages; ++i) mbar_init(&bars[i], 1);
+    for (int i = 0; i < kDecMaxSlots; ++i) {
+      mbar_init(&k_full[i], 1);
+      mbar_init(&v_full[i], 1);
+      mbar_init(&k_empty[i], kDecWarps);
+      mbar_init(&v_empty[i], kDecWarps);
+    }
     mbar_fence_init();
   }
   pdl_wait();
   pdl_launch_dependents();
   const int seq_len = p.seq_lens[b], pos = seq_len - 1;
   int chunk = (seq_len + p.splits - 1) / p.splits;
-  chunk = (chunk + kDecKeys - 1) / kDecKeys * kDecKeys;
+  chunk = (chunk + TK - 1) / TK * TK;
   const int t0 = split * chunk, t1 = min(seq_len, t0 + chunk);
-  const int ntiles = t1 > t0 ? (t1 - t0 + kDecKeys - 1) / kDecKeys : 0;
-  const bool counts_null = p.null_entry && split == 0;
-  for (int h = tid; h < p.hp; h += blockDim.x) {
-    s_m[h] = counts_null ? 0.f : -INFINITY;              // log2 domain
-    s_l[h] = counts_null ? 1.f : 0.f;
-  }
-  fence_proxy_async_smem();          // the clears are ordered before the copies that follow
+  const int ntiles = t1 > t0 ? (t1 - t0 + TK - 1) / TK : 0;
   __syncthreads();
 
-  const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(p.cache);
-  const int32_t* bt = p.block_table + (size_t)b * p.max_blocks;
-  auto load_tile = [&](int it) {     // warp 0: one key and one value row per lane
-    const int st = it % p.stages, tok0 = t0 + it * kDecKeys, n = min(kDecKeys, t1 - tok0);
-    if (lane == 0) mbar_expect_tx(&bars[st], (uint32_t)n * (p.kw + vw) * 2);
-    __syncwarp();
-    if (lane < n) {
-      const int tok = tok0 + lane;
-      const __nv_bfloat16* page = cache + (size_t)bt[tok / p.block_size] * p.block_size * (p.kw + vw);
-      const int off = tok % p.block_size;
-      bulk_load(sK + (size_t)(st * kDecKeys + lane) * ks, page + (size_t)off * p.kw, p.kw * 2, &bars[st]);
-      bulk_load(sV + (size_t)(st * kDecKeys + lane) * vs, page + (size_t)p.block_size * p.kw + (size_t)off * vw,
-                vw * 2, &bars[st]);
+  if (warp == kDecWarps) {
+    // ---------------- producer: lane l fetches chunks of the page part l & (loads - 1) of a tile
+    const int rpl = min(p.block_size, TK), loads = TK / rpl, part = lane & (loads - 1);
+    const int32_t* bt = p.block_table + (size_t)b * p.max_blocks;
+    const int nblk = (seq_len + p.block_size - 1) / p.block_size;
+    auto page_of = [&](int t) {
+      const int bi = (t0 + t * TK + part * rpl) / p.block_size;
+      return max(bi < nblk ? bt[bi] : bt[0], 0);
+    };
+    bool ok = true;
+    int blk = ntiles > 0 ? page_of(0) : 0, blk_prev = 0;
+    for (int t = 0; t <= ntiles && ntiles > 0 && ok; ++t) {
+      const int next = t + 1 < ntiles ? page_of(t + 1) : 0;
+      if (t < ntiles) {
+        const int sl = t % p.k_slots, row = (t0 + t * TK + part * rpl) % p.block_size;
+        ok = __all_sync(0xffffffffu, mbar_wait(&k_empty[sl], ((t / p.k_slots) & 1) ^ 1, p.status));
+        if (!ok) break;
+        if (lane == 0) mbar_expect_tx(&k_full[sl], k_slot_bytes);
+        __syncwarp();
+        for (int x = lane; x < nkc * loads; x += 32) {
+          const int c = x / loads;
+          tma_load_3d(smem + L.k + sl * k_slot_bytes + c * TK * 128 + part * rpl * 128, &tmK, &k_full[sl], c * 64, row, blk);
+        }
+      }
+      if (t > 0) {
+        const int i = t - 1, sl = i % p.v_slots, row = (t0 + i * TK + part * rpl) % p.block_size;
+        ok = __all_sync(0xffffffffu, mbar_wait(&v_empty[sl], ((i / p.v_slots) & 1) ^ 1, p.status));
+        if (!ok) break;
+        if (lane == 0) mbar_expect_tx(&v_full[sl], v_slot_bytes);
+        __syncwarp();
+        for (int x = lane; x < nvc * loads; x += 32) {
+          const int c = x / loads;
+          tma_load_3d(smem + L.v + sl * v_slot_bytes + c * TK * 128 + part * rpl * 128, &tmV, &v_full[sl], c * 64, row, blk_prev);
+        }
+      }
+      blk_prev = blk;
+      blk = next;
     }
-  };
-  if (warp == 0)
-    for (int it = 0; it < min(p.stages, ntiles); ++it) load_tile(it);
+    return;
+  }
+  auto compute_sync = [] { asm volatile("bar.sync 1, %0;" ::"n"(kDecWarps * 32) : "memory"); };
   {
     const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(p.q) + (size_t)b * p.ldq;
     const int n8 = p.kw / 8;
     for (int h = warp; h < H; h += kDecWarps)
       for (int i = lane; i < n8; i += 32)
-        *reinterpret_cast<uint4*>(sQ + (size_t)h * ks + i * 8) =
-            *reinterpret_cast<const uint4*>(q + (size_t)h * p.kw + i * 8);
+        *reinterpret_cast<uint4*>(sQ + (size_t)h * qs + i * 8) = *reinterpret_cast<const uint4*>(q + (size_t)h * p.kw + i * 8);
   }
-  __syncthreads();
-
-  const int n_vt = p.vdim / 8, items = p.G * p.mt * n_vt;
-  const int per_warp = (items + kDecWarps - 1) / kDecWarps;
-  const int i0 = warp * per_warp, cnt = max(0, min(items - i0, per_warp));
+  // this warp's output tiles: consecutive 8-column pieces in (group, 16-head tile, column) order
+  const int n_vt = p.vdim / 8, items = p.G * p.mt * n_vt, per_warp = (items + kDecWarps - 1) / kDecWarps;
+  const int i0 = warp * per_warp, cnt = max(0, min(items - i0, per_warp)), gm0 = i0 / n_vt, nt0 = i0 - gm0 * n_vt;
   float o[MAXI][4];
 #pragma unroll
   for (int i = 0; i < MAXI; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  const int s_tiles = (p.hp / 16) * (kDecKeys / 8);
-  bool ok = true;
-
-  for (int it = 0; it < ntiles; ++it) {
-    const int st = it % p.stages, tok0 = t0 + it * kDecKeys;
-    ok = mbar_wait(&bars[st], (it / p.stages) & 1, p.status);
-    if (!__syncthreads_and(ok)) { ok = false; break; }
-    // ---- scores: 16 heads x 8 keys per warp step
-    for (int x = warp; x < s_tiles; x += kDecWarps) {
-      const int mtile = x / (kDecKeys / 8), ntile = x % (kDecKeys / 8);
-      const uint32_t qa = smem_u32(sQ + (size_t)(mtile * 16 + (lane & 15)) * ks + (lane >> 4) * 8);
-      const uint32_t ka = smem_u32(sK + (size_t)(st * kDecKeys + ntile * 8 + (lane & 7)) * ks + ((lane >> 3) & 1) * 8);
-      float d0[4] = {0.f, 0.f, 0.f, 0.f}, d1[4] = {0.f, 0.f, 0.f, 0.f};
-      const int nk = p.kwp / 16;
-      int kk = 0;
-      for (; kk + 1 < nk; kk += 2) {
-        uint32_t a0[4], a1[4], b0[2], b1[2];
-        ldsm_x4(a0, qa + kk * 32);
-        ldsm_x2(b0, ka + kk * 32);
-        ldsm_x4(a1, qa + kk * 32 + 32);
-        ldsm_x2(b1, ka + kk * 32 + 32);
-        mma_bf16_16816(d0, a0, b0);
-        mma_bf16_16816(d1, a1, b1);
-      }
-      if (kk < nk) {
-        uint32_t a0[4], b0[2];
-        ldsm_x4(a0, qa + kk * 32);
-        ldsm_x2(b0, ka + kk * 32);
-        mma_bf16_16816(d0, a0, b0);
-      }
-      float* s0 = sS + (size_t)(mtile * 16 + (lane >> 2)) * ss + ntile * 8 + (lane & 3) * 2;
-      s0[0] = d0[0] + d1[0];
-      s0[1] = d0[1] + d1[1];
-      s0[8 * ss] = d0[2] + d1[2];
-      s0[8 * ss + 1] = d0[3] + d1[3];
-    }
-    __syncthreads();
-    // ---- softmax: one warp per head, one key per lane
-    for (int h = warp; h < H; h += kDecWarps) {
-      const int key = tok0 + lane;
-      float x = -INFINITY;
-      if (key < t1) {
-        x = sS[(size_t)h * ss + lane];
-        if (p.bias) x += __ldg(p.bias + (size_t)h * p.bias_len + min(pos - key, p.bias_len - 1));
-        x *= kLog2e;
-      }
-      const float mo = s_m[h], mn = fmaxf(mo, warp_max_f32(x));
-      const float e = exp2f(x - mn);
-      float sum = e;
+  // softmax state of heads warp, warp + 16, ...: the maximum (log2 domain) is uniform, the sum per lane
+  const bool counts_null = p.null_entry && split == 0;
+  float m[kDecHeads], l[kDecHeads];
 #pragma unroll
-      for (int k2 = 16; k2 > 0; k2 >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, k2);
-      const int g = h / R, r = h - g * R;
-      sP[(size_t)(g * p.mt * 16 + r) * ps + lane] = __float2bfloat16(e);
-      if (lane == 0) {
-        const float a = mo == -INFINITY ? 0.f : exp2f(mo - mn);
-        s_alpha[h] = a;
-        s_m[h] = mn;
-        s_l[h] = s_l[h] * a + sum;
-      }
-    }
-    __syncthreads();
-    // ---- outputs: each warp keeps its 16 x 8 tiles
-    uint32_t pa[2][4];
-    float al0 = 1.f, al1 = 1.f;
-    int cur = -1;
-#pragma unroll
-    for (int i = 0; i < MAXI; ++i) {
-      if (i < cnt) {
-        const int item = i0 + i, gm = item / n_vt, nt = item - gm * n_vt;
-        const int g = gm / p.mt, mi = gm - g * p.mt;
-        if (gm != cur) {
-          cur = gm;
-          const uint32_t a = smem_u32(sP + (size_t)(gm * 16 + (lane & 15)) * ps + (lane >> 4) * 8);
-          ldsm_x4(pa[0], a);
-          ldsm_x4(pa[1], a + 32);
-          const int r0 = mi * 16 + (lane >> 2);
-          al0 = r0 < R ? s_alpha[g * R + r0] : 0.f;
-          al1 = r0 + 8 < R ? s_alpha[g * R + r0 + 8] : 0.f;
-        }
-        uint32_t vb[4];
-        ldsm_x4_trans(vb, smem_u32(sV + (size_t)(st * kDecKeys + lane) * vs + g * p.vdim + nt * 8));
-        o[i][0] *= al0; o[i][1] *= al0; o[i][2] *= al1; o[i][3] *= al1;
-        mma_bf16_16816(o[i], pa[0], vb);
-        mma_bf16_16816(o[i], pa[1], vb + 2);
-      }
-    }
-    __syncthreads();
-    if (warp == 0 && it + p.stages < ntiles) load_tile(it + p.stages);
+  for (int i = 0; i < kDecHeads; ++i) {
+    m[i] = counts_null ? 0.f : -INFINITY;
+    l[i] = counts_null && lane == 0 ? 1.f : 0.f;
   }
+  constexpr int kNT = TK / 8;
+  const int s_tiles = (p.hp / 16) * kNT, cper = (nkc + p.ksplit - 1) / p.ksplit;
+  const uint32_t k_base = smem_u32(smem + L.k), v_base = smem_u32(smem + L.v);
+  int ksl = 0, vsl = 0;
+  uint32_t kph = 0, vph = 0;
+  bool ok = true;       // after a wait that ran out the warp goes on without waiting (barriers stay matched)
+  compute_sync();
+
+  for (int t = 0; t <= ntiles && ntiles > 0; ++t) {
+    const int tok0 = t0 + t * TK;
+    float bv[kDecHeads];
+#pragma unroll
+    for (int i = 0; i < kDecHeads; ++i) {
+      const int h = warp + i * kDecWarps;
+      bv[i] = 0.f;
+      if (h < H && p.bias && t < ntiles)
+        bv[i] = __ldg(p.bias + (size_t)h * p.bias_len + min(max(pos - tok0 - lane, 0), p.bias_len - 1));
+    }
+    if (t < ntiles) {
+      ok = ok && __all_sync(0xffffffffu, mbar_wait(&k_full[ksl], kph, p.status));
+      for (int x = warp; x < s_tiles * p.ksplit; x += kDecWarps) {
+        const int kpart = x / s_tiles, y = x - kpart * s_tiles, mtile = y / kNT, ntile = y % kNT;
+        const int c0 = kpart * cper, c1 = min(nkc, c0 + cper);
+        const uint32_t qa = smem_u32(sQ + (size_t)(mtile * 16 + (lane & 15)) * qs + (lane >> 4) * 8);
+        const uint32_t ka = k_base + ksl * k_slot_bytes + (ntile * 8 + (lane & 7)) * 128;
+        const uint32_t u0 = (((lane >> 3)) ^ (lane & 7)) << 4, u1 = ((4 + (lane >> 3)) ^ (lane & 7)) << 4;
+        float d0[4] = {0.f, 0.f, 0.f, 0.f}, d1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 2
+        for (int c = c0; c < c1; ++c) {
+          uint32_t a[4][4], kb[8];
+          ldsm_x4(kb, ka + c * TK * 128 + u0);
+          ldsm_x4(kb + 4, ka + c * TK * 128 + u1);
+#pragma unroll
+          for (int kk = 0; kk < 4; ++kk) ldsm_x4(a[kk], qa + c * 128 + kk * 32);
+          mma_bf16_16816(d0, a[0], kb);
+          mma_bf16_16816(d1, a[1], kb + 2);
+          mma_bf16_16816(d0, a[2], kb + 4);
+          mma_bf16_16816(d1, a[3], kb + 6);
+        }
+        float* s0 = sS + (size_t)(kpart * p.hp + mtile * 16 + (lane >> 2)) * ss + ntile * 8 + (lane & 3) * 2;
+        s0[0] = d0[0] + d1[0];
+        s0[1] = d0[1] + d1[1];
+        s0[8 * ss] = d0[2] + d1[2];
+        s0[8 * ss + 1] = d0[3] + d1[3];
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&k_empty[ksl]);
+      if (++ksl == p.k_slots) { ksl = 0; kph ^= 1; }
+    }
+    if (t > 0) {
+      ok = ok && __all_sync(0xffffffffu, mbar_wait(&v_full[vsl], vph, p.status));
+      uint32_t pa[TK / 16][4];
+      float al0 = 0.f, al1 = 0.f;
+      int gm = gm0, nt = nt0, g = gm0 / p.mt, mi = gm0 - g * p.mt;
+      bool fresh = true;
+      const int row = lane & (TK - 1);
+      const uint32_t va = v_base + vsl * v_slot_bytes + row * 128;
+#pragma unroll
+      for (int i = 0; i < MAXI; ++i) {
+        if (i < cnt) {
+          if (fresh) {
+            const uint32_t a = smem_u32(sP + (size_t)(gm * 16 + (lane & 15)) * ps + (lane >> 4) * 8);
+#pragma unroll
+            for (int kk = 0; kk < TK / 16; ++kk) ldsm_x4(pa[kk], a + kk * 32);
+            const int r0 = mi * 16 + (lane >> 2);
+            al0 = r0 < R ? s_alpha[g * R + r0] : 0.f;
+            al1 = r0 + 8 < R ? s_alpha[g * R + r0 + 8] : 0.f;
+          }
+          const int u = (g * p.vdim >> 3) + nt;             // 16-byte unit of the value row
+          const uint32_t addr = va + (u >> 3) * (TK * 128) + (((u & 7) ^ (row & 7)) << 4);
+          uint32_t vb[4];
+          if (TK == 32) ldsm_x4_trans(vb, addr); else ldsm_x2_trans(vb, addr);
+          o[i][0] *= al0; o[i][1] *= al0; o[i][2] *= al1; o[i][3] *= al1;
+#pragma unroll
+          for (int kk = 0; kk < TK / 16; ++kk) mma_bf16_16816(o[i], pa[kk], vb + 2 * kk);
+          fresh = ++nt == n_vt;
+          if (fresh) {
+            nt = 0;
+            ++gm;
+            if (++mi == p.mt) { mi = 0; ++g; }
+          }
+        }
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&v_empty[vsl]);
+      if (++vsl == p.v_slots) { vsl = 0; vph ^= 1; }
+    }
+    compute_sync();
+    if (t == ntiles) break;
+    // ---- softmax: one key per lane
+#pragma unroll
+    for (int i = 0; i < kDecHeads; ++i) {
+      const int h = warp + i * kDecWarps;
+      if (h < H) {
+        float x = -INFINITY;
+        if (lane < TK && tok0 + lane < t1) {
+          x = sS[(size_t)h * ss + lane];
+          for (int kpart = 1; kpart < p.ksplit; ++kpart) x += sS[(size_t)(kpart * p.hp + h) * ss + lane];
+          x = (x + bv[i]) * kLog2e;
+        }
+        const float mn = fmaxf(m[i], warp_max_f32(x)), e = exp2f(x - mn);
+        const float a = m[i] == -INFINITY ? 0.f : exp2f(m[i] - mn);
+        m[i] = mn;
+        l[i] = l[i] * a + e;
+        const int g = h / R;
+        if (lane < TK) sP[(size_t)(g * p.mt * 16 + h - g * R) * ps + lane] = __float2bfloat16(e);
+        if (lane == 0) s_alpha[h] = a;
+      }
+    }
+    compute_sync();
+  }
+#pragma unroll
+  for (int i = 0; i < kDecHeads; ++i) {
+    const int h = warp + i * kDecWarps;
+    if (h < H) {
+#pragma unroll
+      for (int k2 = 16; k2 > 0; k2 >>= 1) l[i] += __shfl_xor_sync(0xffffffffu, l[i], k2);
+      if (lane == 0) {
+        s_l[h] = l[i];
+        if (p.splits > 1) p.tmp_lse[((size_t)b * H + h) * p.splits + split] = l[i] > 0.f ? m[i] + log2f(l[i]) : -INFINITY;
+      }
+    }
+  }
+  compute_sync();
   if (!ok) return;
+  int nt = nt0, g = gm0 / p.mt, mi = gm0 - g * p.mt;
 #pragma unroll
   for (int i = 0; i < MAXI; ++i) {
     if (i < cnt) {
-      const int item = i0 + i, gm = item / n_vt, nt = item - gm * n_vt;
-      const int g = gm / p.mt, mi = gm - g * p.mt;
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int r = mi * 16 + (lane >> 2) + half * 8;
         if (r < R) {
           const int h = g * R + r, d = nt * 8 + (lane & 3) * 2;
-          const float l = s_l[h], inv = l > 0.f ? 1.f / l : 0.f;
+          const float inv = s_l[h] > 0.f ? 1.f / s_l[h] : 0.f;
           const float x0 = o[i][half * 2] * inv, x1 = o[i][half * 2 + 1] * inv;
           if (p.splits == 1) {
             *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)b * p.ldo +
@@ -550,11 +610,12 @@ __global__ void __launch_bounds__(kDecWarps * 32, 1) bias_attn_decode_kernel(Bia
           }
         }
       }
+      if (++nt == n_vt) {
+        nt = 0;
+        if (++mi == p.mt) { mi = 0; ++g; }
+      }
     }
   }
-  if (p.splits > 1)
-    for (int h = tid; h < H; h += blockDim.x)
-      p.tmp_lse[((size_t)b * H + h) * p.splits + split] = s_l[h] > 0.f ? s_m[h] + log2f(s_l[h]) : -INFINITY;
 }
 
 // --------------------------------------------------------------------------------- prefill (bf16)
@@ -891,20 +952,28 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
 }
 
 // ------------------------------------------------------------------------------------ host helpers
-static bool decode_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem, int& maxi) {
+// Shapes the decode kernel serves: tk keys per tile, maxi output tiles per warp.
+static bool decode_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem, int& tk, int& maxi) {
   if (a->f32 || (a->kw & 7) || (a->vdim & 7) || (a->ldq & 7) || (a->ldo & 1)) return false;
   if (((uintptr_t)a->q | (uintptr_t)a->cache) & 15) return false;
-  const int R = a->H / a->G;
-  p.kwp = (a->kw + 15) & ~15;
-  p.vwp = a->G * a->vdim;
+  if (a->H > kDecWarps * kDecHeads) return false;
+  const int R = a->H / a->G, nkc = (a->kw + 63) / 64, nvc = (a->G * a->vdim + 63) / 64;
   p.mt = (R + 15) / 16;
   p.hp = (a->H + 15) & ~15;
   const int per_warp = (a->G * p.mt * (a->vdim / 8) + kDecWarps - 1) / kDecWarps;
-  if (per_warp > 32) return false;
-  maxi = per_warp <= 4 ? 4 : per_warp <= 8 ? 8 : per_warp <= 16 ? 16 : 32;
-  for (p.stages = kDecMaxStages; p.stages >= 2; --p.stages) {
-    smem = (size_t)decode_smem(p.hp, p.kwp, p.vwp, a->G * p.mt * 16, p.stages).total;
-    if (smem <= 225 * 1024) return true;
+  if (per_warp > 16) return false;
+  maxi = per_warp <= 4 ? 4 : per_warp <= 8 ? 8 : 16;
+  for (tk = 32; tk >= 16; tk -= 16) {
+    if (a->block_size < 8 || (a->block_size < tk ? tk % a->block_size : a->block_size % tk)) continue;
+    // the score product is cut along the key row until every warp has a piece
+    p.ksplit = 1;
+    while (p.hp / 16 * (tk / 8) * p.ksplit < kDecWarps && 2 * p.ksplit <= nkc && p.ksplit < 4) p.ksplit *= 2;
+    for (int n = 2 * kDecMaxSlots; n >= 4; --n) {         // slots of both rings together
+      p.k_slots = (n + 1) / 2;
+      p.v_slots = n / 2;
+      smem = (size_t)decode_smem(tk, p.hp, nkc, nvc, a->G * p.mt * 16, p.ksplit, p.k_slots, p.v_slots).total + 1024;
+      if (smem <= 227 * 1024) return true;
+    }
   }
   return false;
 }
@@ -935,30 +1004,31 @@ static bool prefill_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem)
 struct PageMapKey {
   const void* base;
   uint64_t blocks;
-  int bs, kw, vw;
+  int bs, kw, vw, rows;
   bool operator==(const PageMapKey& o) const {
-    return base == o.base && blocks == o.blocks && bs == o.bs && kw == o.kw && vw == o.vw;
+    return base == o.base && blocks == o.blocks && bs == o.bs && kw == o.kw && vw == o.vw && rows == o.rows;
   }
 };
 struct PageMapHash {
   size_t operator()(const PageMapKey& k) const {
     return reinterpret_cast<size_t>(k.base) ^ (k.blocks * 0x9e3779b97f4a7c15ull) ^ ((size_t)k.bs << 40) ^
-           ((size_t)k.kw << 20) ^ (size_t)k.vw;
+           ((size_t)k.kw << 20) ^ ((size_t)k.vw << 4) ^ (size_t)k.rows;
   }
 };
 
-// Tensor maps of the key and the value part of a page, built once per cache.
-static bool page_maps(const B200BiasAttn* a, CUtensorMap* mk, CUtensorMap* mv) {
+// Tensor maps of the key and the value part of a page, built once per cache; a load brings up to
+// `keys` rows of one page.
+static bool page_maps(const B200BiasAttn* a, int keys, CUtensorMap* mk, CUtensorMap* mv) {
   static std::mutex mu;
   static std::unordered_map<PageMapKey, std::pair<CUtensorMap, CUtensorMap>, PageMapHash> maps;
   const int vw = a->G * a->vdim;
-  PageMapKey key{a->cache, (uint64_t)a->num_blocks, a->block_size, a->kw, vw};
+  const uint32_t rows = a->block_size < keys ? a->block_size : keys;
+  PageMapKey key{a->cache, (uint64_t)a->num_blocks, a->block_size, a->kw, vw, (int)rows};
   std::lock_guard<std::mutex> lock(mu);
   auto it = maps.find(key);
   if (it == maps.end()) {
     if (maps.size() > 4096) maps.clear();
     const uint64_t page = (uint64_t)a->block_size * (a->kw + vw) * 2;
-    const uint32_t rows = a->block_size < kBKeys ? a->block_size : kBKeys;
     const uint8_t* base = reinterpret_cast<const uint8_t*>(a->cache);
     CUtensorMap k, v;
     if (!encode_tmap_3d(&k, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a->kw, a->block_size, a->num_blocks,
@@ -998,12 +1068,15 @@ static int launch_any(const BiasAttnParams& p, cudaStream_t stream) {
   return launch_pdl(bias_attn_any_kernel<T>, grid, dim3(128), smem, stream, p) == cudaSuccess ? 0 : -2;
 }
 
-template <int MAXI>
-static int launch_decode_mma(const BiasAttnParams& p, size_t smem, cudaStream_t stream) {
+template <int TK, int MAXI>
+static int launch_decode_mma(const B200BiasAttn* a, const BiasAttnParams& p, size_t smem, cudaStream_t stream) {
+  CUtensorMap tmK, tmV;
+  if (!page_maps(a, TK, &tmK, &tmV)) return -3;
   static PerDeviceOnce once;
-  if (once.first()) cudaFuncSetAttribute(bias_attn_decode_kernel<MAXI>, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024);
-  return launch_pdl(bias_attn_decode_kernel<MAXI>, dim3(p.rows, p.splits), dim3(kDecWarps * 32), smem, stream, p) ==
-                 cudaSuccess ? 0 : -2;
+  if (once.first())
+    cudaFuncSetAttribute(bias_attn_decode_kernel<TK, MAXI>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+  return launch_pdl(bias_attn_decode_kernel<TK, MAXI>, dim3(p.rows, p.splits), dim3(kDecThreads), smem, stream, tmK, tmV,
+                    p) == cudaSuccess ? 0 : -2;
 }
 
 template <typename TO, int TOK>
@@ -1085,9 +1158,9 @@ int b200_head_mix_kv(const void* qkv, long long ld, const void* mix, void* q_out
 int b200_bias_attn_kernel(const B200BiasAttn* a, int phase) {
   BiasAttnParams p{};
   size_t smem;
-  int maxi;
+  int tk, maxi;
   if (!valid_args(a)) return 0;
-  return (phase == 0 ? decode_plan(a, p, smem, maxi) : prefill_plan(a, p, smem)) ? 2 : 1;
+  return (phase == 0 ? decode_plan(a, p, smem, tk, maxi) : prefill_plan(a, p, smem)) ? 2 : 1;
 }
 
 int b200_bias_attn_decode(const B200BiasAttn* a, int any_size, cudaStream_t stream) {
@@ -1096,12 +1169,16 @@ int b200_bias_attn_decode(const B200BiasAttn* a, int any_size, cudaStream_t stre
   BiasAttnParams p = common_params(a);
   p.q_start = nullptr;
   size_t smem;
-  int maxi;
-  if (any_size || !decode_plan(a, p, smem, maxi))
+  int tk, maxi;
+  if (any_size || !decode_plan(a, p, smem, tk, maxi))
     return a->f32 ? launch_any<float>(p, stream) : launch_any<__nv_bfloat16>(p, stream);
   if (p.splits > 1 && (!p.tmp_o || !p.tmp_lse)) return -1;
-  const int rc = maxi == 4 ? launch_decode_mma<4>(p, smem, stream) : maxi == 8 ? launch_decode_mma<8>(p, smem, stream)
-               : maxi == 16 ? launch_decode_mma<16>(p, smem, stream) : launch_decode_mma<32>(p, smem, stream);
+  const int rc = tk == 32 ? (maxi == 4   ? launch_decode_mma<32, 4>(a, p, smem, stream)
+                             : maxi == 8 ? launch_decode_mma<32, 8>(a, p, smem, stream)
+                                         : launch_decode_mma<32, 16>(a, p, smem, stream))
+                          : (maxi == 4   ? launch_decode_mma<16, 4>(a, p, smem, stream)
+                             : maxi == 8 ? launch_decode_mma<16, 8>(a, p, smem, stream)
+                                         : launch_decode_mma<16, 16>(a, p, smem, stream));
   if (rc || p.splits == 1) return rc;
   return b200_attn_decode_merge(p.tmp_o, p.tmp_lse, p.out, (int)p.ldo, p.rows, p.H, p.vdim, p.splits, stream);
 }
@@ -1117,7 +1194,7 @@ int b200_bias_attn_prefill(const B200BiasAttn* a, int any_size, cudaStream_t str
   CUtensorMap tmQ, tmK, tmV;
   if (!encode_tmap_2d(&tmQ, a->q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)a->rows, (uint64_t)a->H * a->kw,
                       (uint64_t)a->ldq, kBQ, 64, CU_TENSOR_MAP_SWIZZLE_128B) ||
-      !page_maps(a, &tmK, &tmV))
+      !page_maps(a, kBKeys, &tmK, &tmV))
     return -3;
   static PerDeviceOnce once;
   if (once.first()) cudaFuncSetAttribute(bias_attn_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
