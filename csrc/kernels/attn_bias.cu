@@ -328,68 +328,74 @@ __device__ __forceinline__ void ldsm_x4_trans(uint32_t* r, uint32_t addr) {
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 __device__ __forceinline__ void mma_bf16_16816(float* d, const uint32_t* a, const uint32_t* b) {
-  asm volatile(
+  asm(
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
       "{%0, %1, %2, %3};"
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
 }
-static constexpr int kDecWarps = 16;     // compute warps; one more feeds the rings
-static constexpr int kDecThreads = (kDecWarps + 1) * 32;
-static constexpr int kDecMaxSlots = 4, kDecHeads = 8;   // kDecHeads * kDecWarps heads at most
+__device__ __forceinline__ float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+static constexpr int kDecWarps = 8;      // 255 registers each
+static constexpr int kDecThreads = kDecWarps * 32;
+static constexpr int kDecMaxSlots = 4;
 
 struct DecodeSmem {                      // byte offsets; the rings are 1024-byte aligned
   int k, v, q, s, p, stat, bars, total;
 };
 __host__ __device__ inline DecodeSmem decode_smem(int tk, int hp, int nkc, int nvc, int prow, int ksplit, int k_slots,
-                                                  int v_slots) {
+                                                  int v_slots, bool q_smem) {
   DecodeSmem d;
   int o = 0;
   d.k = o; o += k_slots * nkc * tk * 128;
   d.v = o; o += v_slots * nvc * tk * 128;
-  d.q = o; o += hp * (nkc * 64 + 8) * 2;
-  d.s = o; o += ksplit * hp * (tk + 1) * 4;
+  d.q = o; o += q_smem ? hp * (nkc * 64 + 8) * 2 : 0;
+  d.s = o; o += 2 * ksplit * hp * (tk + 8) * 4;
   o = (o + 15) & ~15;
-  d.p = o; o += prow * (tk + 8) * 2;
-  d.stat = o; o += 2 * hp * 4;
+  d.p = o; o += 2 * prow * (tk + 8) * 2;
+  d.stat = o; o += 3 * hp * 4;
   o = (o + 15) & ~15;
-  d.bars = o; o += 4 * kDecMaxSlots * 8;
+  d.bars = o; o += 2 * kDecMaxSlots * 8;
   d.total = o;
   return d;
 }
 
-// grid (request, split). TK keys per tile; MAXI: 16 x 8 output tiles a warp keeps in registers. Key and
-// value rows arrive by TMA in 128-byte swizzled chunks of 64 columns. Per tile two barriers: the scores
-// of tile t run beside the output product of tile t - 1, then the softmax of tile t.
-template <int TK, int MAXI>
+// grid (request, split). TK keys per tile; MAXI: 16 x 8 output tiles a warp keeps in registers; CPW:
+// 64-wide chunks of the query rows it keeps there (0: the queries stay in shared memory); HPW: heads per
+// warp in the softmax. (Shared memory leaves next to no L1 cache: nothing may spill.) Key and value
+// rows arrive by TMA in 128-byte swizzled chunks of 64 columns. Three tiles are in work at a time, with
+// one barrier per round: the scores of tile t + 1 (each warp a slice of the key row, partial sums in
+// shared memory), the softmax of tile t, the output product of tile t - 1.
+template <int TK, int MAXI, int CPW, int HPW>
 __global__ void __launch_bounds__(kDecThreads, 1)
     bias_attn_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                             BiasAttnParams p) {
   extern __shared__ uint8_t dec_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(dec_raw) + 1023) & ~uintptr_t(1023));
   const int nkc = (p.kw + 63) / 64, vw = p.G * p.vdim, nvc = (vw + 63) / 64, prow = p.G * p.mt * 16;
-  const DecodeSmem L = decode_smem(TK, p.hp, nkc, nvc, prow, p.ksplit, p.k_slots, p.v_slots);
+  const DecodeSmem L = decode_smem(TK, p.hp, nkc, nvc, prow, p.ksplit, p.k_slots, p.v_slots, CPW == 0);
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem + L.q);
   float* sS = reinterpret_cast<float*>(smem + L.s);
   __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(smem + L.p);
   float* s_alpha = reinterpret_cast<float*>(smem + L.stat);
-  float* s_l = s_alpha + p.hp;
+  float* s_l = s_alpha + 2 * p.hp;
   uint64_t* k_full = reinterpret_cast<uint64_t*>(smem + L.bars);
-  uint64_t *k_empty = k_full + kDecMaxSlots, *v_full = k_empty + kDecMaxSlots, *v_empty = v_full + kDecMaxSlots;
+  uint64_t* v_full = k_full + kDecMaxSlots;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int b = blockIdx.x, split = blockIdx.y;
-  const int H = p.H, R = H / p.G, qs = nkc * 64 + 8, ps = TK + 8, ss = TK + 1;
+  const int H = p.H, R = H / p.G, ps = TK + 8, ss = TK + 8, s_buf = p.ksplit * p.hp * ss, p_buf = prow * ps;
   const int k_slot_bytes = nkc * TK * 128, v_slot_bytes = nvc * TK * 128;
 
   // what a product may read and nothing fills has to be finite
-  for (int i = tid; i < p.hp * qs / 8; i += kDecThreads) reinterpret_cast<uint4*>(sQ)[i] = make_uint4(0, 0, 0, 0);
-  for (int i = tid; i < prow * ps / 8; i += kDecThreads) reinterpret_cast<uint4*>(sP)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < 2 * p_buf / 8; i += kDecThreads) reinterpret_cast<uint4*>(sP)[i] = make_uint4(0, 0, 0, 0);
   if (tid == 0) {
     for (int i = 0; i < kDecMaxSlots; ++i) {
-      mbar_init(&k_full[i], 1);
-      mbar_init(&v_full[i], 1);
-      mbar_init(&k_empty[i], kDecWarps);
-      mbar_init(&v_empty[i], kDecWarps);
+      mbar_init(&k_full[i], kDecWarps);
+      mbar_init(&v_full[i], kDecWarps);
     }
     mbar_fence_init();
   }
@@ -402,181 +408,258 @@ __global__ void __launch_bounds__(kDecThreads, 1)
   const int ntiles = t1 > t0 ? (t1 - t0 + TK - 1) / TK : 0;
   __syncthreads();
 
-  if (warp == kDecWarps) {
-    // ---------------- producer: lane l fetches chunks of the page part l & (loads - 1) of a tile
-    const int rpl = min(p.block_size, TK), loads = TK / rpl, part = lane & (loads - 1);
-    const int32_t* bt = p.block_table + (size_t)b * p.max_blocks;
-    const int nblk = (seq_len + p.block_size - 1) / p.block_size;
-    auto page_of = [&](int t) {
-      const int bi = (t0 + t * TK + part * rpl) / p.block_size;
-      return max(bi < nblk ? bt[bi] : bt[0], 0);
-    };
-    bool ok = true;
-    int blk = ntiles > 0 ? page_of(0) : 0, blk_prev = 0;
-    for (int t = 0; t <= ntiles && ntiles > 0 && ok; ++t) {
-      const int next = t + 1 < ntiles ? page_of(t + 1) : 0;
-      if (t < ntiles) {
-        const int sl = t % p.k_slots, row = (t0 + t * TK + part * rpl) % p.block_size;
-        ok = __all_sync(0xffffffffu, mbar_wait(&k_empty[sl], ((t / p.k_slots) & 1) ^ 1, p.status));
-        if (!ok) break;
-        if (lane == 0) mbar_expect_tx(&k_full[sl], k_slot_bytes);
-        __syncwarp();
-        for (int x = lane; x < nkc * loads; x += 32) {
-          const int c = x / loads;
-          tma_load_3d(smem + L.k + sl * k_slot_bytes + c * TK * 128 + part * rpl * 128, &tmK, &k_full[sl], c * 64, row, blk);
-        }
-      }
-      if (t > 0) {
-        const int i = t - 1, sl = i % p.v_slots, row = (t0 + i * TK + part * rpl) % p.block_size;
-        ok = __all_sync(0xffffffffu, mbar_wait(&v_empty[sl], ((i / p.v_slots) & 1) ^ 1, p.status));
-        if (!ok) break;
-        if (lane == 0) mbar_expect_tx(&v_full[sl], v_slot_bytes);
-        __syncwarp();
-        for (int x = lane; x < nvc * loads; x += 32) {
-          const int c = x / loads;
-          tma_load_3d(smem + L.v + sl * v_slot_bytes + c * TK * 128 + part * rpl * 128, &tmV, &v_full[sl], c * 64, row, blk_prev);
-        }
-      }
-      blk_prev = blk;
-      blk = next;
+  // Every warp fetches its share of a tile's 64-wide chunks (one copy per chunk and page part of rpl
+  // rows; lane l looks up the page of part l, lane 0 issues). In a slot: [part][chunk][rpl rows][64]. A
+  // slot is free once the round that used it has passed its barrier.
+  const int rpl = min(p.block_size, TK), loads = TK / rpl;
+  const int32_t* bt = p.block_table + (size_t)b * p.max_blocks;
+  const int nblk = (seq_len + p.block_size - 1) / p.block_size;
+  auto page_of = [&](int t) {
+    const int bi = (t0 + t * TK + lane * rpl) / p.block_size;
+    return max(t < ntiles && lane < loads && bi < nblk ? bt[bi] : 0, 0);
+  };
+  auto load = [&](const CUtensorMap* map, uint64_t* bar, int ring, int chunks, int first, int t, int blk) {
+    const int row = p.block_size > TK ? (t0 + t * TK) % p.block_size : 0;
+    const int n = first < chunks ? (chunks - first + kDecWarps - 1) / kDecWarps : 0;
+    if (lane == 0) mbar_expect_tx(bar, n * TK * 128);
+    for (int l = 0; l < loads; ++l) {
+      const int page = __shfl_sync(0xffffffffu, blk, l);
+      if (lane == 0)
+        for (int c = first; c < chunks; c += kDecWarps)
+          tma_load_3d(smem + ring + (l * chunks + c) * rpl * 128, map, bar, c * 64, row, page);
     }
-    return;
+  };
+  const int v_first = (warp + kDecWarps - nkc % kDecWarps) % kDecWarps;   // value chunks go on where the key chunks end
+  if (ntiles > 0) {
+    if (tid == 0) { tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV); }
+    for (int i = 0; i < min(p.k_slots, ntiles); ++i)
+      load(&tmK, &k_full[i], L.k + i * k_slot_bytes, nkc, warp, i, page_of(i));
+    for (int i = 0; i < min(p.v_slots, ntiles); ++i)
+      load(&tmV, &v_full[i], L.v + i * v_slot_bytes, nvc, v_first, i, page_of(i));
   }
-  auto compute_sync = [] { asm volatile("bar.sync 1, %0;" ::"n"(kDecWarps * 32) : "memory"); };
+  // pages of the next tile of each ring, looked up one round ahead
+  int k_page = page_of(p.k_slots), v_page = page_of(p.v_slots);
+  // scores: this warp's 16 heads, slice of the key row (chunks c0 ..) and 8-key columns npart, npart + nsplit ..
+  constexpr int kNT = TK / 8;
+  const int mtiles = p.hp / 16, cper = (nkc + p.ksplit - 1) / p.ksplit;
+  const int mtile = warp % mtiles, kpart = (warp / mtiles) % p.ksplit, npart = warp / (mtiles * p.ksplit);
+  int nsplit = 1;                          // a power of two
+  while (2 * nsplit <= kNT && 2 * nsplit * mtiles * p.ksplit <= kDecWarps) nsplit *= 2;
+  const int c0 = kpart * cper, nc = npart < nsplit ? min(cper, nkc - c0) : 0;
+  const int qs = nkc * 64 + 8;
+  uint32_t qa[CPW > 0 ? CPW : 1][4][4];
   {
     const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(p.q) + (size_t)b * p.ldq;
-    const int n8 = p.kw / 8;
-    for (int h = warp; h < H; h += kDecWarps)
-      for (int i = lane; i < n8; i += 32)
-        *reinterpret_cast<uint4*>(sQ + (size_t)h * qs + i * 8) = *reinterpret_cast<const uint4*>(q + (size_t)h * p.kw + i * 8);
+    if (CPW == 0) {
+      for (int h = warp; h < p.hp; h += kDecWarps)
+        for (int i = lane; i < qs / 8; i += 32)
+          *reinterpret_cast<uint4*>(sQ + h * qs + i * 8) =
+              h < H && i * 8 < p.kw ? *reinterpret_cast<const uint4*>(q + (size_t)h * p.kw + i * 8) : make_uint4(0, 0, 0, 0);
+      __syncthreads();
+    } else {
+#pragma unroll
+      for (int c = 0; c < CPW; ++c)
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk)
+#pragma unroll
+          for (int x = 0; x < 4; ++x) {
+            const int h = mtile * 16 + (lane >> 2) + (x & 1) * 8, k = (c0 + c) * 64 + kk * 16 + (lane & 3) * 2 + (x >> 1) * 8;
+            qa[c][kk][x] = h < H && c < nc && k < p.kw ? *reinterpret_cast<const uint32_t*>(q + (size_t)h * p.kw + k) : 0u;
+          }
+    }
   }
-  // this warp's output tiles: consecutive 8-column pieces in (group, 16-head tile, column) order
+  const uint32_t q_addr = smem_u32(sQ + (mtile * 16 + (lane & 15)) * qs + (lane >> 4) * 8) + c0 * 128;
+  const uint32_t k_off = c0 * rpl * 128 + (lane & 7) * 128;
+  uint32_t n_off[kNT];                     // where the 8 keys of a column start in a slot
+#pragma unroll
+  for (int n = 0; n < kNT; ++n) n_off[n] = n * 8 / rpl * (nkc * rpl * 128) + n * 8 % rpl * 128;
+  const uint32_t u0 = ((lane >> 3) ^ (lane & 7)) << 4, u1 = ((4 + (lane >> 3)) ^ (lane & 7)) << 4;
+  float* s_dst = sS + (size_t)(kpart * p.hp + mtile * 16 + (lane >> 2)) * ss + (lane & 3) * 2;
+  // outputs: consecutive 8-column pieces in (group, 16-head tile, column) order
   const int n_vt = p.vdim / 8, items = p.G * p.mt * n_vt, per_warp = (items + kDecWarps - 1) / kDecWarps;
   const int i0 = warp * per_warp, cnt = max(0, min(items - i0, per_warp)), gm0 = i0 / n_vt, nt0 = i0 - gm0 * n_vt;
+  const bool one_tile = nt0 + cnt <= n_vt;
+  const int g0 = gm0 / p.mt, mi0 = gm0 - g0 * p.mt, v_row = lane & (TK - 1);
   float o[MAXI][4];
 #pragma unroll
   for (int i = 0; i < MAXI; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  // softmax state of heads warp, warp + 16, ...: the maximum (log2 domain) is uniform, the sum per lane
+  // softmax state of heads warp, warp + 8, ...: the maximum (log2 domain) is uniform, the sum per lane
   const bool counts_null = p.null_entry && split == 0;
-  float m[kDecHeads], l[kDecHeads];
+  const int last = p.bias_len - 1;
+  float m[HPW], l[HPW], far[HPW];
+  int p_off[HPW];
 #pragma unroll
-  for (int i = 0; i < kDecHeads; ++i) {
+  for (int i = 0; i < HPW; ++i) {
+    const int h = min(warp + i * kDecWarps, H - 1), g = h / R;
     m[i] = counts_null ? 0.f : -INFINITY;
     l[i] = counts_null && lane == 0 ? 1.f : 0.f;
+    far[i] = p.bias ? p.bias[(size_t)h * p.bias_len + last] * kLog2e : 0.f;
+    p_off[i] = (g * p.mt * 16 + h - g * R) * ps + lane;
   }
-  constexpr int kNT = TK / 8;
-  const int s_tiles = (p.hp / 16) * kNT, cper = (nkc + p.ksplit - 1) / p.ksplit;
+  const uint32_t v_off = v_row / rpl * (nvc * rpl * 128) + v_row % rpl * 128;
   const uint32_t k_base = smem_u32(smem + L.k), v_base = smem_u32(smem + L.v);
-  int ksl = 0, vsl = 0;
+  int ksl = 0, vsl = 0, k_free = 0, v_free = 0;
   uint32_t kph = 0, vph = 0;
   bool ok = true;       // after a wait that ran out the warp goes on without waiting (barriers stay matched)
-  compute_sync();
 
-  for (int t = 0; t <= ntiles && ntiles > 0; ++t) {
-    const int tok0 = t0 + t * TK;
-    float bv[kDecHeads];
-#pragma unroll
-    for (int i = 0; i < kDecHeads; ++i) {
-      const int h = warp + i * kDecWarps;
-      bv[i] = 0.f;
-      if (h < H && p.bias && t < ntiles)
-        bv[i] = __ldg(p.bias + (size_t)h * p.bias_len + min(max(pos - tok0 - lane, 0), p.bias_len - 1));
+  for (int t = -1; t <= ntiles && ntiles > 0; ++t) {
+    // the last round used key tile t and value tile t - 2
+    if (t >= 0 && t + p.k_slots < ntiles) {
+      load(&tmK, &k_full[k_free], L.k + k_free * k_slot_bytes, nkc, warp, t + p.k_slots, k_page);
+      k_page = page_of(t + 1 + p.k_slots);
+      if (++k_free == p.k_slots) k_free = 0;
     }
-    if (t < ntiles) {
-      ok = ok && __all_sync(0xffffffffu, mbar_wait(&k_full[ksl], kph, p.status));
-      for (int x = warp; x < s_tiles * p.ksplit; x += kDecWarps) {
-        const int kpart = x / s_tiles, y = x - kpart * s_tiles, mtile = y / kNT, ntile = y % kNT;
-        const int c0 = kpart * cper, c1 = min(nkc, c0 + cper);
-        const uint32_t qa = smem_u32(sQ + (size_t)(mtile * 16 + (lane & 15)) * qs + (lane >> 4) * 8);
-        const uint32_t ka = k_base + ksl * k_slot_bytes + (ntile * 8 + (lane & 7)) * 128;
-        const uint32_t u0 = (((lane >> 3)) ^ (lane & 7)) << 4, u1 = ((4 + (lane >> 3)) ^ (lane & 7)) << 4;
-        float d0[4] = {0.f, 0.f, 0.f, 0.f}, d1[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 2
-        for (int c = c0; c < c1; ++c) {
-          uint32_t a[4][4], kb[8];
-          ldsm_x4(kb, ka + c * TK * 128 + u0);
-          ldsm_x4(kb + 4, ka + c * TK * 128 + u1);
+    if (t >= 2 && t - 2 + p.v_slots < ntiles) {
+      load(&tmV, &v_full[v_free], L.v + v_free * v_slot_bytes, nvc, v_first, t - 2 + p.v_slots, v_page);
+      v_page = page_of(t - 1 + p.v_slots);
+      if (++v_free == p.v_slots) v_free = 0;
+    }
+    // bias of this round's softmax, asked for before the scores
+    const bool near = p.bias && pos - (t0 + t * TK + TK - 1) < last;
+    float bias[HPW];
 #pragma unroll
-          for (int kk = 0; kk < 4; ++kk) ldsm_x4(a[kk], qa + c * 128 + kk * 32);
-          mma_bf16_16816(d0, a[0], kb);
-          mma_bf16_16816(d1, a[1], kb + 2);
-          mma_bf16_16816(d0, a[2], kb + 4);
-          mma_bf16_16816(d1, a[3], kb + 6);
+    for (int i = 0; i < HPW; ++i) {
+      bias[i] = far[i];
+      if (near && t >= 0 && warp + i * kDecWarps < H)
+        bias[i] = __ldg(p.bias + (size_t)(warp + i * kDecWarps) * p.bias_len + min(max(pos - t0 - t * TK - lane, 0), last)) * kLog2e;
+    }
+    if (t + 1 < ntiles) {
+      // ---- scores of tile t + 1
+      ok = ok && __all_sync(0xffffffffu, mbar_wait(&k_full[ksl], kph, p.status));
+      const uint32_t ka = k_base + ksl * k_slot_bytes + k_off;
+      float* sd = s_dst + ((t + 1) & 1) * s_buf;
+      if (nc > 0) {
+        float d[kNT][4];
+#pragma unroll
+        for (int n = 0; n < kNT; ++n) d[n][0] = d[n][1] = d[n][2] = d[n][3] = 0.f;
+        auto chunk_products = [&](int c, const uint32_t (&a)[4][4]) {
+#pragma unroll
+          for (int n = 0; n < kNT; ++n) {
+            if ((n & (nsplit - 1)) != npart) continue;
+            uint32_t kb[8];
+            ldsm_x4(kb, ka + c * rpl * 128 + n_off[n] + u0);
+            ldsm_x4(kb + 4, ka + c * rpl * 128 + n_off[n] + u1);
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk) mma_bf16_16816(d[n], a[kk], kb + 2 * kk);
+          }
+        };
+        if (CPW == 0) {
+          for (int c = 0; c < nc; ++c) {
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk) ldsm_x4(qa[0][kk], q_addr + c * 128 + kk * 32);
+            chunk_products(c, qa[0]);
+          }
+        } else {
+#pragma unroll
+          for (int c = 0; c < CPW; ++c)
+            if (c < nc) chunk_products(c, qa[c]);
         }
-        float* s0 = sS + (size_t)(kpart * p.hp + mtile * 16 + (lane >> 2)) * ss + ntile * 8 + (lane & 3) * 2;
-        s0[0] = d0[0] + d1[0];
-        s0[1] = d0[1] + d1[1];
-        s0[8 * ss] = d0[2] + d1[2];
-        s0[8 * ss + 1] = d0[3] + d1[3];
+#pragma unroll
+        for (int n = 0; n < kNT; ++n) {
+          if ((n & (nsplit - 1)) != npart) continue;
+          *reinterpret_cast<float2*>(sd + n * 8) = make_float2(d[n][0], d[n][1]);
+          *reinterpret_cast<float2*>(sd + 8 * ss + n * 8) = make_float2(d[n][2], d[n][3]);
+        }
       }
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&k_empty[ksl]);
       if (++ksl == p.k_slots) { ksl = 0; kph ^= 1; }
     }
-    if (t > 0) {
+    if (t >= 0 && t < ntiles) {
+      // ---- softmax of tile t: one key per lane
+      const int tok0 = t0 + t * TK;
+      const bool mine = lane < TK && tok0 + lane < t1;
+      const float* ssrc = sS + (t & 1) * s_buf + (lane & (TK - 1));
+      __nv_bfloat16* pd = sP + (t & 1) * p_buf;
+      float x[HPW];
+#pragma unroll
+      for (int i = 0; i < HPW; ++i) x[i] = warp + i * kDecWarps < H ? ssrc[(warp + i * kDecWarps) * ss] : 0.f;
+      for (int k = 1; k < p.ksplit; ++k) {
+#pragma unroll
+        for (int i = 0; i < HPW; ++i)
+          if (warp + i * kDecWarps < H) x[i] += ssrc[(k * p.hp + warp + i * kDecWarps) * ss];
+      }
+#pragma unroll
+      for (int i = 0; i < HPW; ++i) {
+        const int h = warp + i * kDecWarps;
+        if (h < H) {
+          x[i] = mine ? fmaf(x[i], kLog2e, bias[i]) : -INFINITY;
+          const float mn = fmaxf(m[i], warp_max_f32(x[i])), e = ex2_approx(x[i] - mn);
+          const float a = m[i] == -INFINITY ? 0.f : ex2_approx(m[i] - mn);
+          m[i] = mn;
+          l[i] = fmaf(l[i], a, e);
+          if (lane < TK) pd[p_off[i]] = __float2bfloat16(e);
+          if (lane == 0) s_alpha[(t & 1) * p.hp + h] = a;
+        }
+      }
+    }
+    if (t >= 1) {
+      // ---- output product of tile t - 1
       ok = ok && __all_sync(0xffffffffu, mbar_wait(&v_full[vsl], vph, p.status));
+      const __nv_bfloat16* pp = sP + ((t - 1) & 1) * p_buf + (size_t)(lane & 15) * ps + (lane >> 4) * 8;
+      const float* al = s_alpha + ((t - 1) & 1) * p.hp;
+      const uint32_t va = v_base + vsl * v_slot_bytes + v_off;
       uint32_t pa[TK / 16][4];
       float al0 = 0.f, al1 = 0.f;
-      int gm = gm0, nt = nt0, g = gm0 / p.mt, mi = gm0 - g * p.mt;
-      bool fresh = true;
-      const int row = lane & (TK - 1);
-      const uint32_t va = v_base + vsl * v_slot_bytes + row * 128;
+      int gm = gm0, nt = nt0, g = g0, mi = mi0, u = (g0 * p.vdim >> 3) + nt0;   // u: 16-byte unit of the value row
+      if (cnt > 0 && one_tile) {      // (a warp without pieces has no place in P either)
+        // every piece belongs to the same 16 heads: all loads first
+#pragma unroll
+        for (int kk = 0; kk < TK / 16; ++kk) ldsm_x4(pa[kk], smem_u32(pp + gm * 16 * ps + kk * 16));
+        const int r0 = mi * 16 + (lane >> 2);
+        al0 = r0 < R ? al[g * R + r0] : 0.f;
+        al1 = r0 + 8 < R ? al[g * R + r0 + 8] : 0.f;
+#pragma unroll
+        for (int i4 = 0; i4 < MAXI; i4 += 4) {
+          uint32_t vb[4][4];
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const int uu = u + i4 + i;
+            const uint32_t addr = va + (uu >> 3) * (rpl * 128) + (((uu & 7) ^ (v_row & 7)) << 4);
+            if (i4 + i < cnt) { if (TK == 32) ldsm_x4_trans(vb[i], addr); else ldsm_x2_trans(vb[i], addr); }
+          }
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            if (i4 + i < cnt) {
+              float* d = o[i4 + i];
+              d[0] *= al0; d[1] *= al0; d[2] *= al1; d[3] *= al1;
+#pragma unroll
+              for (int kk = 0; kk < TK / 16; ++kk) mma_bf16_16816(d, pa[kk], vb[i] + 2 * kk);
+            }
+          }
+        }
+      } else {
+        bool fresh = true;
 #pragma unroll
       for (int i = 0; i < MAXI; ++i) {
         if (i < cnt) {
-          if (fresh) {
-            const uint32_t a = smem_u32(sP + (size_t)(gm * 16 + (lane & 15)) * ps + (lane >> 4) * 8);
-#pragma unroll
-            for (int kk = 0; kk < TK / 16; ++kk) ldsm_x4(pa[kk], a + kk * 32);
-            const int r0 = mi * 16 + (lane >> 2);
-            al0 = r0 < R ? s_alpha[g * R + r0] : 0.f;
-            al1 = r0 + 8 < R ? s_alpha[g * R + r0 + 8] : 0.f;
-          }
-          const int u = (g * p.vdim >> 3) + nt;             // 16-byte unit of the value row
-          const uint32_t addr = va + (u >> 3) * (TK * 128) + (((u & 7) ^ (row & 7)) << 4);
           uint32_t vb[4];
+          const uint32_t addr = va + (u >> 3) * (rpl * 128) + (((u & 7) ^ (v_row & 7)) << 4);
           if (TK == 32) ldsm_x4_trans(vb, addr); else ldsm_x2_trans(vb, addr);
+          if (fresh) {
+#pragma unroll
+            for (int kk = 0; kk < TK / 16; ++kk) ldsm_x4(pa[kk], smem_u32(pp + gm * 16 * ps + kk * 16));
+            const int r0 = mi * 16 + (lane >> 2);
+            al0 = r0 < R ? al[g * R + r0] : 0.f;
+            al1 = r0 + 8 < R ? al[g * R + r0 + 8] : 0.f;
+          }
           o[i][0] *= al0; o[i][1] *= al0; o[i][2] *= al1; o[i][3] *= al1;
 #pragma unroll
           for (int kk = 0; kk < TK / 16; ++kk) mma_bf16_16816(o[i], pa[kk], vb + 2 * kk);
+          ++u;
           fresh = ++nt == n_vt;
           if (fresh) {
             nt = 0;
             ++gm;
-            if (++mi == p.mt) { mi = 0; ++g; }
+            if (++mi == p.mt) { mi = 0; ++g; } else { u -= n_vt; }
           }
         }
       }
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&v_empty[vsl]);
+      }
       if (++vsl == p.v_slots) { vsl = 0; vph ^= 1; }
     }
-    compute_sync();
-    if (t == ntiles) break;
-    // ---- softmax: one key per lane
-#pragma unroll
-    for (int i = 0; i < kDecHeads; ++i) {
-      const int h = warp + i * kDecWarps;
-      if (h < H) {
-        float x = -INFINITY;
-        if (lane < TK && tok0 + lane < t1) {
-          x = sS[(size_t)h * ss + lane];
-          for (int kpart = 1; kpart < p.ksplit; ++kpart) x += sS[(size_t)(kpart * p.hp + h) * ss + lane];
-          x = (x + bv[i]) * kLog2e;
-        }
-        const float mn = fmaxf(m[i], warp_max_f32(x)), e = exp2f(x - mn);
-        const float a = m[i] == -INFINITY ? 0.f : exp2f(m[i] - mn);
-        m[i] = mn;
-        l[i] = l[i] * a + e;
-        const int g = h / R;
-        if (lane < TK) sP[(size_t)(g * p.mt * 16 + h - g * R) * ps + lane] = __float2bfloat16(e);
-        if (lane == 0) s_alpha[h] = a;
-      }
-    }
-    compute_sync();
+    __syncthreads();
   }
 #pragma unroll
-  for (int i = 0; i < kDecHeads; ++i) {
+  for (int i = 0; i < HPW; ++i) {
     const int h = warp + i * kDecWarps;
     if (h < H) {
 #pragma unroll
@@ -587,9 +670,9 @@ __global__ void __launch_bounds__(kDecThreads, 1)
       }
     }
   }
-  compute_sync();
+  __syncthreads();
   if (!ok) return;
-  int nt = nt0, g = gm0 / p.mt, mi = gm0 - g * p.mt;
+  int nt = nt0, g = g0, mi = mi0;
 #pragma unroll
   for (int i = 0; i < MAXI; ++i) {
     if (i < cnt) {
@@ -640,11 +723,6 @@ struct alignas(8) BiasPrefillBars {
   float window[2][4][kWin];          // [tile parity][quarter]: log2-domain bias by distance
 };
 
-__device__ __forceinline__ float ex2_approx(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 __device__ __forceinline__ void pair_sync(int quarter) {             // the two warps of a row quarter
   asm volatile("bar.sync %0, 64;" ::"r"(quarter + 1) : "memory");
 }
@@ -692,7 +770,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
   const uint32_t tmem_s = bars->tmem_base, tmem_o = tmem_s + s_bufs * kBKeys, tmem_p = tmem_o + o_cols;
 
   if (warp == 0) {
-    // A 128-key tile spans up to 16 pages; lane l fetches the rows of the l-th one, so the page
+    // A 128-key tile spans up to 16 pages; lane l looks up and fetches the l-th one, so that the
     // look-ups of a tile run side by side.
     const int rpl = min(p.block_size, kBKeys), loads = kBKeys / rpl;
     const int32_t* bt = p.block_table + (size_t)req * p.max_blocks;
@@ -701,8 +779,6 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
       const int bi = (j * kBKeys + lane * rpl) / p.block_size;
       return max(lane < loads && bi < nblk ? bt[bi] : bt[0], 0);
     };
-    const int row_in_page = (lane * rpl) % p.block_size;
-    const int dst_off = lane * rpl * 128;
     if (lane == 0) {
       tma_prefetch_desc(&tmQ);
       tma_prefetch_desc(&tmK);
@@ -720,7 +796,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
     for (int j = 0; j <= ntiles && ok; ++j) {
       const int next = j + 1 < ntiles ? page_of(j + 1) : 0;
       if (j < ntiles) {
-        const int row = p.block_size > kBKeys ? (j * kBKeys) % p.block_size : row_in_page;
+        const int row = p.block_size > kBKeys ? (j * kBKeys) % p.block_size : 0;
         for (int c = 0; c < nkc; ++c) {
           ok = __all_sync(0xffffffffu, mbar_wait(&bars->k_empty[sl], ph, p.status));
           if (!ok) break;
@@ -731,21 +807,21 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
               tma_load_2d(dst + kChunkBytes, &tmQ, &bars->k_full[sl], h * p.kw + c * 64, q_begin + q0);
           }
           __syncwarp();
-          if (lane < loads) tma_load_3d(dst + dst_off, &tmK, &bars->k_full[sl], c * 64, row, blk);
+          if (lane < loads) tma_load_3d(dst + lane * rpl * 128, &tmK, &bars->k_full[sl], c * 64, row, blk);
           if (++sl == p.k_slots) { sl = 0; ph ^= 1; }
         }
       }
       if (j >= 1 && ok) {
         const int i = j - 1, vs = i % p.v_slots;
-        const int row = p.block_size > kBKeys ? (i * kBKeys) % p.block_size : row_in_page;
+        const int row = p.block_size > kBKeys ? (i * kBKeys) % p.block_size : 0;
         ok = __all_sync(0xffffffffu, mbar_wait(&bars->v_empty[vs], ((i / p.v_slots) & 1) ^ 1, p.status));
         if (!ok) break;
         if (lane == 0) mbar_expect_tx(&bars->v_full[vs], nvc * kChunkBytes);
         __syncwarp();
         if (lane < loads)
           for (int c = 0; c < nvc; ++c)
-            tma_load_3d(sV + (vs * nvc + c) * kChunkBytes + dst_off, &tmV, &bars->v_full[vs], hkv * p.vdim + c * 64,
-                        row, blk_prev);
+            tma_load_3d(sV + (vs * nvc + c) * kChunkBytes + lane * rpl * 128, &tmV, &bars->v_full[vs],
+                        hkv * p.vdim + c * 64, row, blk_prev);
       }
       blk_prev = blk;
       blk = next;
@@ -952,27 +1028,34 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
 }
 
 // ------------------------------------------------------------------------------------ host helpers
-// Shapes the decode kernel serves: tk keys per tile, maxi output tiles per warp.
-static bool decode_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem, int& tk, int& maxi) {
+// Shapes the decode kernel serves. tk: keys per tile; cls: register class (0: 8 output tiles, 2 query
+// chunks and 4 heads per warp, 1: 16 tiles, 8 heads, queries in shared memory).
+static bool decode_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem, int& tk, int& cls) {
   if (a->f32 || (a->kw & 7) || (a->vdim & 7) || (a->ldq & 7) || (a->ldo & 1)) return false;
   if (((uintptr_t)a->q | (uintptr_t)a->cache) & 15) return false;
-  if (a->H > kDecWarps * kDecHeads) return false;
   const int R = a->H / a->G, nkc = (a->kw + 63) / 64, nvc = (a->G * a->vdim + 63) / 64;
   p.mt = (R + 15) / 16;
   p.hp = (a->H + 15) & ~15;
+  const int mtiles = p.hp / 16, heads = p.hp / kDecWarps;         // heads: per warp
   const int per_warp = (a->G * p.mt * (a->vdim / 8) + kDecWarps - 1) / kDecWarps;
-  if (per_warp > 16) return false;
-  maxi = per_warp <= 4 ? 4 : per_warp <= 8 ? 8 : 16;
+  if (heads > 8 || per_warp > 16) return false;
+  // The key row is cut into slices (a power of two, then without empty ones), as many as there are warps
+  // for and as the partial sums leave room for.
+  int most = 1;
+  while (mtiles * most * 2 <= kDecWarps && most * 2 <= nkc) most *= 2;
   for (tk = 32; tk >= 16; tk -= 16) {
     if (a->block_size < 8 || (a->block_size < tk ? tk % a->block_size : a->block_size % tk)) continue;
-    // the score product is cut along the key row until every warp has a piece
-    p.ksplit = 1;
-    while (p.hp / 16 * (tk / 8) * p.ksplit < kDecWarps && 2 * p.ksplit <= nkc && p.ksplit < 4) p.ksplit *= 2;
-    for (int n = 2 * kDecMaxSlots; n >= 4; --n) {         // slots of both rings together
-      p.k_slots = (n + 1) / 2;
-      p.v_slots = n / 2;
-      smem = (size_t)decode_smem(tk, p.hp, nkc, nvc, a->G * p.mt * 16, p.ksplit, p.k_slots, p.v_slots).total + 1024;
-      if (smem <= 227 * 1024) return true;
+    for (int slices = most; slices >= 1; slices /= 2) {
+      const int cper = (nkc + slices - 1) / slices;
+      p.ksplit = (nkc + cper - 1) / cper;
+      cls = per_warp <= 8 && cper <= 2 && heads <= 4 ? 0 : 1;
+      for (int n = 2 * kDecMaxSlots; n >= 4; --n) {         // slots of both rings together
+        p.k_slots = (n + 1) / 2;
+        p.v_slots = n / 2;
+        smem = (size_t)decode_smem(tk, p.hp, nkc, nvc, a->G * p.mt * 16, p.ksplit, p.k_slots, p.v_slots, cls == 1).total +
+               1024;
+        if (smem <= 227 * 1024) return true;
+      }
     }
   }
   return false;
@@ -1068,14 +1151,14 @@ static int launch_any(const BiasAttnParams& p, cudaStream_t stream) {
   return launch_pdl(bias_attn_any_kernel<T>, grid, dim3(128), smem, stream, p) == cudaSuccess ? 0 : -2;
 }
 
-template <int TK, int MAXI>
+template <int TK, int MAXI, int CPW, int HPW>
 static int launch_decode_mma(const B200BiasAttn* a, const BiasAttnParams& p, size_t smem, cudaStream_t stream) {
   CUtensorMap tmK, tmV;
   if (!page_maps(a, TK, &tmK, &tmV)) return -3;
   static PerDeviceOnce once;
   if (once.first())
-    cudaFuncSetAttribute(bias_attn_decode_kernel<TK, MAXI>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
-  return launch_pdl(bias_attn_decode_kernel<TK, MAXI>, dim3(p.rows, p.splits), dim3(kDecThreads), smem, stream, tmK, tmV,
+    cudaFuncSetAttribute(bias_attn_decode_kernel<TK, MAXI, CPW, HPW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+  return launch_pdl(bias_attn_decode_kernel<TK, MAXI, CPW, HPW>, dim3(p.rows, p.splits), dim3(kDecThreads), smem, stream, tmK, tmV,
                     p) == cudaSuccess ? 0 : -2;
 }
 
@@ -1158,9 +1241,9 @@ int b200_head_mix_kv(const void* qkv, long long ld, const void* mix, void* q_out
 int b200_bias_attn_kernel(const B200BiasAttn* a, int phase) {
   BiasAttnParams p{};
   size_t smem;
-  int tk, maxi;
+  int tk, cls;
   if (!valid_args(a)) return 0;
-  return (phase == 0 ? decode_plan(a, p, smem, tk, maxi) : prefill_plan(a, p, smem)) ? 2 : 1;
+  return (phase == 0 ? decode_plan(a, p, smem, tk, cls) : prefill_plan(a, p, smem)) ? 2 : 1;
 }
 
 int b200_bias_attn_decode(const B200BiasAttn* a, int any_size, cudaStream_t stream) {
@@ -1169,16 +1252,14 @@ int b200_bias_attn_decode(const B200BiasAttn* a, int any_size, cudaStream_t stre
   BiasAttnParams p = common_params(a);
   p.q_start = nullptr;
   size_t smem;
-  int tk, maxi;
-  if (any_size || !decode_plan(a, p, smem, tk, maxi))
+  int tk, cls;
+  if (any_size || !decode_plan(a, p, smem, tk, cls))
     return a->f32 ? launch_any<float>(p, stream) : launch_any<__nv_bfloat16>(p, stream);
   if (p.splits > 1 && (!p.tmp_o || !p.tmp_lse)) return -1;
-  const int rc = tk == 32 ? (maxi == 4   ? launch_decode_mma<32, 4>(a, p, smem, stream)
-                             : maxi == 8 ? launch_decode_mma<32, 8>(a, p, smem, stream)
-                                         : launch_decode_mma<32, 16>(a, p, smem, stream))
-                          : (maxi == 4   ? launch_decode_mma<16, 4>(a, p, smem, stream)
-                             : maxi == 8 ? launch_decode_mma<16, 8>(a, p, smem, stream)
-                                         : launch_decode_mma<16, 16>(a, p, smem, stream));
+  const int rc = tk == 32 ? (cls == 0 ? launch_decode_mma<32, 8, 2, 4>(a, p, smem, stream)
+                                      : launch_decode_mma<32, 16, 0, 8>(a, p, smem, stream))
+                          : (cls == 0 ? launch_decode_mma<16, 8, 2, 4>(a, p, smem, stream)
+                                      : launch_decode_mma<16, 16, 0, 8>(a, p, smem, stream));
   if (rc || p.splits == 1) return rc;
   return b200_attn_decode_merge(p.tmp_o, p.tmp_lse, p.out, (int)p.ldo, p.rows, p.H, p.vdim, p.splits, stream);
 }
