@@ -194,7 +194,7 @@ struct BiasAttnParams {
   int splits;
   float* tmp_o;             // [B, H, splits, vdim]
   float* tmp_lse;           // [B, H, splits]
-  int mt, hp, ksplit;
+  int mt, hp, ksplit, zslices;
   // prefill
   const int32_t* tile_req;
   const int32_t* tile_q0;
@@ -364,7 +364,7 @@ __host__ __device__ inline DecodeSmem decode_smem(int tk, int hp, int nkc, int n
   return d;
 }
 
-// grid (request, split). TK keys per tile; MAXI: 16 x 8 output tiles a warp keeps in registers; CPW:
+// grid (request, split, slice of the kv groups). TK keys per tile; MAXI: 16 x 8 output tiles a warp keeps in registers; CPW:
 // 64-wide chunks of the query rows it keeps there (0: the queries stay in shared memory); HPW: heads per
 // warp in the softmax. (Shared memory leaves next to no L1 cache: nothing may spill.) Key and value
 // rows arrive by TMA in 128-byte swizzled chunks of 64 columns. Three tiles are in work at a time, with
@@ -376,7 +376,9 @@ __global__ void __launch_bounds__(kDecThreads, 1)
                             BiasAttnParams p) {
   extern __shared__ uint8_t dec_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(dec_raw) + 1023) & ~uintptr_t(1023));
-  const int nkc = (p.kw + 63) / 64, vw = p.G * p.vdim, nvc = (vw + 63) / 64, prow = p.G * p.mt * 16;
+  // this CTA's heads: the groups of its z slice
+  const int G = p.G / gridDim.z, H = p.H / gridDim.z, h_base = blockIdx.z * H, v_col = blockIdx.z * G * p.vdim;
+  const int nkc = (p.kw + 63) / 64, nvc = (G * p.vdim + 63) / 64, prow = G * p.mt * 16;
   const DecodeSmem L = decode_smem(TK, p.hp, nkc, nvc, prow, p.ksplit, p.k_slots, p.v_slots, CPW == 0);
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem + L.q);
   float* sS = reinterpret_cast<float*>(smem + L.s);
@@ -387,7 +389,7 @@ __global__ void __launch_bounds__(kDecThreads, 1)
   uint64_t* v_full = k_full + kDecMaxSlots;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int b = blockIdx.x, split = blockIdx.y;
-  const int H = p.H, R = H / p.G, ps = TK + 8, ss = TK + 8, s_buf = p.ksplit * p.hp * ss, p_buf = prow * ps;
+  const int R = H / G, ps = TK + 8, ss = TK + 8, s_buf = p.ksplit * p.hp * ss, p_buf = prow * ps;
   const int k_slot_bytes = nkc * TK * 128, v_slot_bytes = nvc * TK * 128;
 
   // what a product may read and nothing fills has to be finite
@@ -418,7 +420,7 @@ __global__ void __launch_bounds__(kDecThreads, 1)
     const int bi = (t0 + t * TK + lane * rpl) / p.block_size;
     return max(t < ntiles && lane < loads && bi < nblk ? bt[bi] : 0, 0);
   };
-  auto load = [&](const CUtensorMap* map, uint64_t* bar, int ring, int chunks, int first, int t, int blk) {
+  auto load = [&](const CUtensorMap* map, uint64_t* bar, int ring, int chunks, int col, int first, int t, int blk) {
     const int row = p.block_size > TK ? (t0 + t * TK) % p.block_size : 0;
     const int n = first < chunks ? (chunks - first + kDecWarps - 1) / kDecWarps : 0;
     if (lane == 0) mbar_expect_tx(bar, n * TK * 128);
@@ -426,16 +428,16 @@ __global__ void __launch_bounds__(kDecThreads, 1)
       const int page = __shfl_sync(0xffffffffu, blk, l);
       if (lane == 0)
         for (int c = first; c < chunks; c += kDecWarps)
-          tma_load_3d(smem + ring + (l * chunks + c) * rpl * 128, map, bar, c * 64, row, page);
+          tma_load_3d(smem + ring + (l * chunks + c) * rpl * 128, map, bar, col + c * 64, row, page);
     }
   };
   const int v_first = (warp + kDecWarps - nkc % kDecWarps) % kDecWarps;   // value chunks go on where the key chunks end
   if (ntiles > 0) {
     if (tid == 0) { tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV); }
     for (int i = 0; i < min(p.k_slots, ntiles); ++i)
-      load(&tmK, &k_full[i], L.k + i * k_slot_bytes, nkc, warp, i, page_of(i));
+      load(&tmK, &k_full[i], L.k + i * k_slot_bytes, nkc, 0, warp, i, page_of(i));
     for (int i = 0; i < min(p.v_slots, ntiles); ++i)
-      load(&tmV, &v_full[i], L.v + i * v_slot_bytes, nvc, v_first, i, page_of(i));
+      load(&tmV, &v_full[i], L.v + i * v_slot_bytes, nvc, v_col, v_first, i, page_of(i));
   }
   // pages of the next tile of each ring, looked up one round ahead
   int k_page = page_of(p.k_slots), v_page = page_of(p.v_slots);
@@ -449,7 +451,7 @@ __global__ void __launch_bounds__(kDecThreads, 1)
   const int qs = nkc * 64 + 8;
   uint32_t qa[CPW > 0 ? CPW : 1][4][4];
   {
-    const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(p.q) + (size_t)b * p.ldq;
+    const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(p.q) + (size_t)b * p.ldq + (size_t)h_base * p.kw;
     if (CPW == 0) {
       for (int h = warp; h < p.hp; h += kDecWarps)
         for (int i = lane; i < qs / 8; i += 32)
@@ -476,7 +478,7 @@ __global__ void __launch_bounds__(kDecThreads, 1)
   const uint32_t u0 = ((lane >> 3) ^ (lane & 7)) << 4, u1 = ((4 + (lane >> 3)) ^ (lane & 7)) << 4;
   float* s_dst = sS + (size_t)(kpart * p.hp + mtile * 16 + (lane >> 2)) * ss + (lane & 3) * 2;
   // outputs: consecutive 8-column pieces in (group, 16-head tile, column) order
-  const int n_vt = p.vdim / 8, items = p.G * p.mt * n_vt, per_warp = (items + kDecWarps - 1) / kDecWarps;
+  const int n_vt = p.vdim / 8, items = G * p.mt * n_vt, per_warp = (items + kDecWarps - 1) / kDecWarps;
   const int i0 = warp * per_warp, cnt = max(0, min(items - i0, per_warp)), gm0 = i0 / n_vt, nt0 = i0 - gm0 * n_vt;
   const bool one_tile = nt0 + cnt <= n_vt;
   const int g0 = gm0 / p.mt, mi0 = gm0 - g0 * p.mt, v_row = lane & (TK - 1);
@@ -493,7 +495,7 @@ __global__ void __launch_bounds__(kDecThreads, 1)
     const int h = min(warp + i * kDecWarps, H - 1), g = h / R;
     m[i] = counts_null ? 0.f : -INFINITY;
     l[i] = counts_null && lane == 0 ? 1.f : 0.f;
-    far[i] = p.bias ? p.bias[(size_t)h * p.bias_len + last] * kLog2e : 0.f;
+    far[i] = p.bias ? p.bias[(size_t)(h_base + h) * p.bias_len + last] * kLog2e : 0.f;
     p_off[i] = (g * p.mt * 16 + h - g * R) * ps + lane;
   }
   const uint32_t v_off = v_row / rpl * (nvc * rpl * 128) + v_row % rpl * 128;
@@ -505,12 +507,12 @@ __global__ void __launch_bounds__(kDecThreads, 1)
   for (int t = -1; t <= ntiles && ntiles > 0; ++t) {
     // the last round used key tile t and value tile t - 2
     if (t >= 0 && t + p.k_slots < ntiles) {
-      load(&tmK, &k_full[k_free], L.k + k_free * k_slot_bytes, nkc, warp, t + p.k_slots, k_page);
+      load(&tmK, &k_full[k_free], L.k + k_free * k_slot_bytes, nkc, 0, warp, t + p.k_slots, k_page);
       k_page = page_of(t + 1 + p.k_slots);
       if (++k_free == p.k_slots) k_free = 0;
     }
     if (t >= 2 && t - 2 + p.v_slots < ntiles) {
-      load(&tmV, &v_full[v_free], L.v + v_free * v_slot_bytes, nvc, v_first, t - 2 + p.v_slots, v_page);
+      load(&tmV, &v_full[v_free], L.v + v_free * v_slot_bytes, nvc, v_col, v_first, t - 2 + p.v_slots, v_page);
       v_page = page_of(t - 1 + p.v_slots);
       if (++v_free == p.v_slots) v_free = 0;
     }
@@ -521,7 +523,7 @@ __global__ void __launch_bounds__(kDecThreads, 1)
     for (int i = 0; i < HPW; ++i) {
       bias[i] = far[i];
       if (near && t >= 0 && warp + i * kDecWarps < H)
-        bias[i] = __ldg(p.bias + (size_t)(warp + i * kDecWarps) * p.bias_len + min(max(pos - t0 - t * TK - lane, 0), last)) * kLog2e;
+        bias[i] = __ldg(p.bias + (size_t)(h_base + warp + i * kDecWarps) * p.bias_len + min(max(pos - t0 - t * TK - lane, 0), last)) * kLog2e;
     }
     if (t + 1 < ntiles) {
       // ---- scores of tile t + 1
@@ -666,7 +668,7 @@ __global__ void __launch_bounds__(kDecThreads, 1)
       for (int k2 = 16; k2 > 0; k2 >>= 1) l[i] += __shfl_xor_sync(0xffffffffu, l[i], k2);
       if (lane == 0) {
         s_l[h] = l[i];
-        if (p.splits > 1) p.tmp_lse[((size_t)b * H + h) * p.splits + split] = l[i] > 0.f ? m[i] + log2f(l[i]) : -INFINITY;
+        if (p.splits > 1) p.tmp_lse[((size_t)b * p.H + h_base + h) * p.splits + split] = l[i] > 0.f ? m[i] + log2f(l[i]) : -INFINITY;
       }
     }
   }
@@ -685,9 +687,9 @@ __global__ void __launch_bounds__(kDecThreads, 1)
           const float x0 = o[i][half * 2] * inv, x1 = o[i][half * 2 + 1] * inv;
           if (p.splits == 1) {
             *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)b * p.ldo +
-                                         (size_t)h * p.vdim + d) = pack_bf16x2(x0, x1);
+                                         (size_t)(h_base + h) * p.vdim + d) = pack_bf16x2(x0, x1);
           } else {
-            float* t = p.tmp_o + (((size_t)b * H + h) * p.splits + split) * p.vdim + d;
+            float* t = p.tmp_o + (((size_t)b * p.H + h_base + h) * p.splits + split) * p.vdim + d;
             t[0] = x0;
             t[1] = x1;
           }
@@ -1033,28 +1035,35 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
 static bool decode_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem, int& tk, int& cls) {
   if (a->f32 || (a->kw & 7) || (a->vdim & 7) || (a->ldq & 7) || (a->ldo & 1)) return false;
   if (((uintptr_t)a->q | (uintptr_t)a->cache) & 15) return false;
-  const int R = a->H / a->G, nkc = (a->kw + 63) / 64, nvc = (a->G * a->vdim + 63) / 64;
+  const int R = a->H / a->G, nkc = (a->kw + 63) / 64;
   p.mt = (R + 15) / 16;
-  p.hp = (a->H + 15) & ~15;
-  const int mtiles = p.hp / 16, heads = p.hp / kDecWarps;         // heads: per warp
-  const int per_warp = (a->G * p.mt * (a->vdim / 8) + kDecWarps - 1) / kDecWarps;
-  if (heads > 8 || per_warp > 16) return false;
-  // The key row is cut into slices (a power of two, then without empty ones), as many as there are warps
-  // for and as the partial sums leave room for.
-  int most = 1;
-  while (mtiles * most * 2 <= kDecWarps && most * 2 <= nkc) most *= 2;
-  for (tk = 32; tk >= 16; tk -= 16) {
-    if (a->block_size < 8 || (a->block_size < tk ? tk % a->block_size : a->block_size % tk)) continue;
-    for (int slices = most; slices >= 1; slices /= 2) {
-      const int cper = (nkc + slices - 1) / slices;
-      p.ksplit = (nkc + cper - 1) / cper;
-      cls = per_warp <= 8 && cper <= 2 && heads <= 4 ? 0 : 1;
-      for (int n = 2 * kDecMaxSlots; n >= 4; --n) {         // slots of both rings together
-        p.k_slots = (n + 1) / 2;
-        p.v_slots = n / 2;
-        smem = (size_t)decode_smem(tk, p.hp, nkc, nvc, a->G * p.mt * 16, p.ksplit, p.k_slots, p.v_slots, cls == 1).total +
-               1024;
-        if (smem <= 227 * 1024) return true;
+  // All heads of a request in one CTA read each key once; where they do not fit its registers and shared
+  // memory, CTAs share them by kv groups (the keys then come out of L2 for all but the first).
+  for (int z = 1; z <= a->G; ++z) {
+    if (a->G % z) continue;
+    const int G = a->G / z, H = a->H / z, nvc = (G * a->vdim + 63) / 64;
+    p.zslices = z;
+    p.hp = (H + 15) & ~15;
+    const int mtiles = p.hp / 16, heads = p.hp / kDecWarps;         // heads: per warp
+    const int per_warp = (G * p.mt * (a->vdim / 8) + kDecWarps - 1) / kDecWarps;
+    if (heads > 8 || per_warp > 16) continue;
+    // The key row is cut into slices (a power of two, then without empty ones), as many as there are
+    // warps for and as the partial sums leave room for.
+    int most = 1;
+    while (mtiles * most * 2 <= kDecWarps && most * 2 <= nkc) most *= 2;
+    for (tk = 32; tk >= 16; tk -= 16) {
+      if (a->block_size < 8 || (a->block_size < tk ? tk % a->block_size : a->block_size % tk)) continue;
+      for (int slices = most; slices >= 1; slices /= 2) {
+        const int cper = (nkc + slices - 1) / slices;
+        p.ksplit = (nkc + cper - 1) / cper;
+        cls = per_warp <= 8 && cper <= 2 && heads <= 4 ? 0 : 1;
+        for (int n = 2 * kDecMaxSlots; n >= 4; --n) {         // slots of both rings together
+          p.k_slots = (n + 1) / 2;
+          p.v_slots = n / 2;
+          smem = (size_t)decode_smem(tk, p.hp, nkc, nvc, G * p.mt * 16, p.ksplit, p.k_slots, p.v_slots, cls == 1).total +
+                 1024;
+          if (smem <= 227 * 1024) return true;
+        }
       }
     }
   }
@@ -1158,7 +1167,7 @@ static int launch_decode_mma(const B200BiasAttn* a, const BiasAttnParams& p, siz
   static PerDeviceOnce once;
   if (once.first())
     cudaFuncSetAttribute(bias_attn_decode_kernel<TK, MAXI, CPW, HPW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
-  return launch_pdl(bias_attn_decode_kernel<TK, MAXI, CPW, HPW>, dim3(p.rows, p.splits), dim3(kDecThreads), smem, stream, tmK, tmV,
+  return launch_pdl(bias_attn_decode_kernel<TK, MAXI, CPW, HPW>, dim3(p.rows, p.splits, p.zslices), dim3(kDecThreads), smem, stream, tmK, tmV,
                     p) == cudaSuccess ? 0 : -2;
 }
 

@@ -82,6 +82,12 @@ def route(h, w_router, top):
     return s.topk(top, -1).indices, s.topk(top, -1).values
 
 
+def router_margin(h, w_router, top):
+    """[T]: distance of the router logits on the two sides of the choice (inf: all are chosen)."""
+    z = linear(h, w_router).sort(-1, descending=True).values
+    return z[:, top - 1] - z[:, top] if z.shape[1] > top else torch.full_like(z[:, 0], math.inf)
+
+
 def experts(h, w, c):
     """The routing weight scales what goes into an expert."""
     ids, wt = route(h, w("router"), c["router"]["top"])
@@ -94,9 +100,9 @@ def experts(h, w, c):
     return out
 
 
-def forward(config, tensors, tokens, dtype=torch.float64, trace=None):
+def forward(config, tensors, tokens, dtype=torch.float64, trace=None, margins=None):
     """Logits [T, vocab] of one sequence. ``trace``: a list that receives the stream after every
-    layer."""
+    layer; ``margins``: one that receives every layer's router margins."""
     t = lambda n: tensors[n].to(dtype)                               # noqa: E731
     eps = config["norm"]["eps"]
     x = t("embed")[torch.tensor(tokens)] * config["embedding"]["scale"]
@@ -105,6 +111,8 @@ def forward(config, tensors, tokens, dtype=torch.float64, trace=None):
         d = attention(h, lambda n: t(f"l{l}.mix.{n}"), c["mixer"])
         if c.get("mlp"):
             d = d + experts(h, lambda n: t(f"l{l}.mlp.{n}"), c["mlp"])
+            if margins is not None:
+                margins.append(router_margin(h, t(f"l{l}.mlp.router"), c["mlp"]["router"]["top"]))
         x = x + d
         if trace is not None:
             trace.append(x)

@@ -19,7 +19,8 @@ def _status():
 
 # (H, G, dim, vdim, block_size, bias_max)
 SHAPES = [(8, 4, 32, 48, 16, 40), (4, 1, 64, 64, 32, 200), (6, 3, 16, 24, 8, 30), (12, 2, 72, 136, 64, 90),
-          (32, 4, 128, 128, 32, 1024), (20, 1, 96, 256, 128, 64), (5, 5, 20, 12, 16, 50), (3, 1, 7, 11, 16, 33)]
+          (32, 4, 128, 128, 32, 1024), (20, 1, 96, 256, 128, 64),
+          (96, 6, 40, 40, 32, 50), (16, 16, 64, 64, 64, 70), (24, 8, 160, 16, 32, 300), (40, 2, 64, 128, 16, 100), (5, 5, 20, 12, 16, 50), (3, 1, 7, 11, 16, 33)]
 
 
 def _case(shape, lens, seed, dtype):

@@ -19,6 +19,7 @@ DEVICES = ["cpu", pytest.param("cuda", marks=pytest.mark.gpu)]
 TOL = {"float32": 2e-5, "bfloat16": 4e-2}
 both = pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 device = pytest.mark.parametrize("dev", DEVICES)
+CLOSE_CALL = 0.05       # router margin below which rounding to bf16 may change the chosen experts
 _logits: dict = {}
 
 
@@ -31,8 +32,23 @@ def oracle(name, toks, seed=0):
     key = (name, tuple(toks), seed)
     if key not in _logits:
         cfg, w = C.case(name, seed)
-        _logits[key] = R.forward(cfg, w, toks, dtype=torch.float64)
-    return _logits[key]
+        margins = []
+        lg = R.forward(cfg, w, toks, dtype=torch.float64, margins=margins)
+        _logits[key] = lg, torch.stack(margins).min(0).values
+    return _logits[key][0]
+
+
+def agrees(got, name, toks, dtype):
+    """The logits of every position agree; in bf16, of every position whose experts are no close call
+    (there are few of those)."""
+    want, margin = oracle(name, toks), _logits[name, tuple(toks), 0][1]
+    if dtype == "bfloat16":
+        clear = margin > CLOSE_CALL
+        assert clear.float().mean() > 0.8 or len(toks) < 20
+        got, want = got[clear], want[clear]
+        if not len(want):
+            return
+    assert rel(got, want) < TOL[dtype]
 
 
 @pytest.fixture(scope="module")
@@ -90,7 +106,7 @@ class Replay:
 def test_whole_prompt(folder, name, dtype, dev):
     toks = tokens(150, C.CASES[name][0]["vocab"], 1)
     got = Replay(folder(name), dtype, dev, 160).run({"a": toks}, [[("a", len(toks))]])["a"]
-    assert rel(got, oracle(name, toks)) < TOL[dtype]
+    agrees(got, name, toks, dtype)
 
 
 @device
@@ -99,7 +115,7 @@ def test_whole_prompt(folder, name, dtype, dev):
 def test_token_by_token(folder, name, dtype, dev):
     toks = tokens(70, C.CASES[name][0]["vocab"], 2)
     got = Replay(folder(name), dtype, dev, 80).run({"a": toks}, [[("a", 1)]] * len(toks))["a"]
-    assert rel(got, oracle(name, toks)) < TOL[dtype]
+    agrees(got, name, toks, dtype)
 
 
 @device
@@ -109,7 +125,7 @@ def test_first_tokens(folder, dtype, dev):
         toks = tokens(n, 96, 3 + n)
         for steps in ([[("a", n)]], [[("a", 1)]] * n):
             got = Replay(folder("aligned"), dtype, dev, 8).run({"a": toks}, steps)["a"]
-            assert rel(got, oracle("aligned", toks)) < TOL[dtype]
+            agrees(got, "aligned", toks, dtype)
 
 
 @device
@@ -123,7 +139,7 @@ def test_portions(folder, sizes, dtype, dev):
         steps.append([("a", n)])
         left, i = left - n, i + 1
     got = Replay(folder("aligned"), dtype, dev, 160).run({"a": toks}, steps)["a"]
-    assert rel(got, oracle("aligned", toks)) < TOL[dtype]
+    agrees(got, "aligned", toks, dtype)
 
 
 @device
@@ -221,7 +237,7 @@ def test_mixed_batches(folder, name, dtype, dev):
             steps.append(step)
     got = Replay(folder(name), dtype, dev, 176).run(prompts, steps)
     for r, p in prompts.items():
-        assert rel(got[r], oracle(name, p)) < TOL[dtype], r
+        agrees(got[r], name, p, dtype)
 
 
 @device
@@ -247,7 +263,7 @@ def test_pages_and_slots_are_used_again(folder, dtype, dev):
         steps = [[(x, 9), (y, ny - 5)], [(x, 1), (y, 1)], [(y, 2), (x, 25)], [(x, 5), (y, 2)]]
         got = r.run(prompts, steps)
         for k, p in prompts.items():
-            assert rel(got[k], oracle("aligned", p)) < TOL[dtype], k
+            agrees(got[k], "aligned", p, dtype)
     r.r.step([], [])
     assert r.free_pages() == total
 
@@ -267,9 +283,13 @@ def greedy(n, **kw):
 
 
 def check_greedy(name, prompt, out, margin):
-    """Every generated token is the oracle's choice, or within ``margin`` of it."""
+    """Every generated token is the oracle's choice, or within ``margin`` of it (with a bf16-sized
+    margin: except where the choice of experts is a close call)."""
     lg = oracle(name, prompt + out)
+    clear = _logits[name, tuple(prompt + out), 0][1] > (CLOSE_CALL if margin > 1e-3 else 0.0)
     for i, t in enumerate(out):
+        if not clear[len(prompt) - 1 + i]:
+            continue
         row = lg[len(prompt) - 1 + i]
         assert row.max() - row[t] <= margin, (i, t, int(row.argmax()))
 

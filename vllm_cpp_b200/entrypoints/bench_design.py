@@ -96,13 +96,15 @@ class KernelBench:
         from ..ops.bench import _time
         return _time(fn, iters=iters, warmup=3, flush=self.flush)
 
-    def add(self, name, whose, fn, nbytes=0.0, flops=0.0, note=None):
+    def add(self, name, whose, fn, nbytes=0.0, flops=0.0, note=None, full_us=None):
         """The roofline is the slower of the bytes at the measured copy rate and the tensor FLOPs at
-        the measured GEMM rate."""
+        the measured GEMM rate. ``full_us``: the roofline with work that ``flops`` leaves out."""
         ms = self.time(fn)
         best = max(nbytes / (self.hbm * 1e6), flops / (self.tflops * 1e9))
         row = {"kernel": name, "model": whose, "us": round(ms * 1e3, 1), "roofline_us": round(best * 1e3, 1),
                "fraction": round(best / ms, 3)}
+        if full_us is not None:
+            row.update(full_roofline_us=round(full_us, 1), full_fraction=round(full_us / (ms * 1e3), 3))
         if note:
             row["note"] = note
         self.rows.append(row)
@@ -131,9 +133,14 @@ class KernelBench:
         out = torch.empty(T, H * D, dtype=torch.bfloat16, device=self.dev)
         shape = dict(H=H, G=G, kw=kw, vdim=D, block_size=bs)
         kind = A.kernel_kind("prefill", q, pages, **shape)
+        # mixing the heads costs H multiply-adds per head and pair in fp32 (128 lanes an SM), or products
+        # kw wide instead of D; the cheaper of the two
+        sms, mhz = torch.cuda.get_device_properties(0).multi_processor_count, 1965.0
+        full = min(max(flops / self.tflops / 1e6, pairs * H * H / (sms * 128 * mhz)),
+                   2 * pairs * H * (kw + D) / self.tflops / 1e6)
         self.add(f"attention, {B} x {prompt} prompt", "nufusun",
                  lambda: A.prefill(q, pages, out, block_table=bt, seq_lens=sl, q_start=qs, num_reqs=B, tile_req=tr,
-                                   tile_q0=tq, bias=bias, null_entry=True, **shape), flops=flops,
+                                   tile_q0=tq, bias=bias, null_entry=True, **shape), flops=flops, full_us=full,
                  note=f"{kind}; multiplies {kw} + {D} wide, {(kw + D) / (2 * D):.2f} x the counted FLOPs")
         q2, kv = self.rnd(T, H * D), self.rnd(B * nb + 1, 2, bs, G, D)
         self.add(f"attention, {B} x {prompt} prompt", "qwen3-moe",
