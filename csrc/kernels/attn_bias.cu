@@ -741,7 +741,8 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
   uint8_t* sV = sK + p.k_slots * slot_bytes;
   BiasPrefillBars* bars = reinterpret_cast<BiasPrefillBars*>(sV + p.v_slots * nvc * kChunkBytes);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int tile = blockIdx.x, h = blockIdx.y, hkv = h / (p.H / p.G);
+  // late tiles of a prompt see the most keys: they go first, so that the last CTAs to run are short
+  const int tile = gridDim.x - 1 - blockIdx.x, h = blockIdx.y, hkv = h / (p.H / p.G);
   const int req = p.tile_req[tile], q0 = p.tile_q0[tile];
   const int q_begin = p.q_start[req], q_len = p.q_start[req + 1] - q_begin;
   const int seq_len = p.seq_lens[req], ctx_off = seq_len - q_len;

@@ -99,6 +99,25 @@ def small_case(name: str):
         slots = torch.arange(B, dtype=torch.int32, device=dev)
         out = torch.empty(B, Hv, 128, device=dev, dtype=torch.bfloat16)
         fn = lambda: G.packed_decode(xc, a, b, A_log, dtb, state, slots, out, Hk, Hv)
+    elif name in ("bias_prefill_small", "bias_decode_small"):
+        from . import bias_attn as A
+        H, G, Dh, bs_, bias = 32, 4, 128, 32, torch.randn(32, 1024, device=dev)
+        kw = G * Dh
+        B, n = (2, 2048) if "prefill" in name else (64, 2048)
+        nb = n // bs_
+        pages = torch.randn(B * nb + 1, bs_ * 2 * kw, device=dev).to(torch.bfloat16)
+        bt = torch.arange(B * nb, device=dev, dtype=torch.int32).reshape(B, nb)
+        sl = torch.full((B,), n, dtype=torch.int32, device=dev)
+        rows = B * n if "prefill" in name else B
+        q = (torch.randn(rows, H * kw, device=dev) * kw ** -0.5).to(torch.bfloat16)
+        out = torch.empty(rows, H * Dh, device=dev, dtype=torch.bfloat16)
+        kw_ = dict(block_table=bt, seq_lens=sl, H=H, G=G, kw=kw, vdim=Dh, block_size=bs_, bias=bias, null_entry=True)
+        if "prefill" in name:
+            treq, tq0 = (torch.tensor(x, dtype=torch.int32, device=dev) for x in ref.build_prefill_tiles([n] * B))
+            qs = torch.arange(B + 1, device=dev, dtype=torch.int32) * n
+            fn = lambda: A.prefill(q, pages, out, q_start=qs, num_reqs=B, tile_req=treq, tile_q0=tq0, **kw_)
+        else:
+            fn = lambda: A.decode(q, pages, out, splits=2, **kw_)
     elif name == "moe_small":
         from . import moe as M
         T, E, k, H, I = 2048, 128, 8, 2048, 768
