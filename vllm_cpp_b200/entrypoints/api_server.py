@@ -537,6 +537,7 @@ def build_arg_parser() -> argparse.ArgumentParser:
     ap.add_argument("--host", default="0.0.0.0")
     ap.add_argument("--port", type=int, default=8000)
     ap.add_argument("--served-model-name", default=None)
+    ap.add_argument("--dtype", default="auto", choices=["auto", "bfloat16", "float32"])
     ap.add_argument("--max-model-len", type=int, default=None)
     ap.add_argument("--max-num-seqs", type=int, default=256)
     ap.add_argument("--max-num-batched-tokens", type=int, default=None)
@@ -576,7 +577,7 @@ def main(argv=None) -> int:
     from ..config import EngineArgs, ParallelConfig
     from ..parallel.launch import launch_engine
     a = build_arg_parser().parse_args(argv)
-    kw = dict(model=a.model, tokenizer=a.tokenizer, device=a.device, block_size=a.block_size,
+    kw = dict(model=a.model, tokenizer=a.tokenizer, device=a.device, dtype=a.dtype, block_size=a.block_size,
               max_num_seqs=a.max_num_seqs, max_model_len=a.max_model_len,
               max_num_batched_tokens=a.max_num_batched_tokens,
               gpu_memory_utilization=a.gpu_memory_utilization, async_scheduling=a.async_scheduling,

@@ -209,7 +209,7 @@ def main():
                          "gemm_small | gemm_decode_small | prefill_small | decode_small | gdn_scan_small | "
                          "gdn_decode_small | moe_small | gemm_streamk_small | gemm_gated_small | "
                          "gemm_fp8_small | gemm_w4a16_small | gemm_nvfp4_small | gemm_nvfp4_prefill_small | "
-                         "decode_d256_small | mla_decode_small")
+                         "decode_d256_small | mla_decode_small | bias_prefill_small | bias_decode_small")
     args = ap.parse_args()
     if args.case:
         return small_case(args.case)
