@@ -58,6 +58,7 @@ struct alignas(8) DecodeTcBars {
   uint64_t s_full[2], s_empty[2];
   uint64_t p_full[2], p_empty[2];
   uint64_t pv_done;
+  uint64_t o_done;        // completes once, after the product of the last tile
   uint64_t grp;
   uint32_t tmem_base;
   float red_max[2][4][kNQ];
@@ -126,6 +127,7 @@ __global__ void __launch_bounds__(192, D == 128 ? 2 : 1)
       mbar_init(&bars->p_empty[i], 1);
     }
     mbar_init(&bars->pv_done, 1);
+    mbar_init(&bars->o_done, 1);
     mbar_init(&bars->grp, 4);
     mbar_fence_init();
   }
@@ -250,6 +252,7 @@ __global__ void __launch_bounds__(192, D == 128 ? 2 : 1)
             umma_commit(&bars->kv_empty[sl]);
             umma_commit(&bars->pv_done);      // before p_empty: whoever sees p_empty has this arrival too
             umma_commit(&bars->p_empty[pb]);
+            if (i == ntiles - 1) umma_commit(&bars->o_done);
           }
         }
       }
@@ -353,12 +356,9 @@ __global__ void __launch_bounds__(192, D == 128 ? 2 : 1)
         if (lane == 0) mbar_arrive(&bars->p_full[pb]);
       }
       // ---------------- epilogue: O^T / l ----------------
-      // pv_done completes once per tile and the loop only guarantees ntiles-2 completions seen
-      // (through p_empty), so observe the last two in order: a parity wait two phases ahead
-      // would be satisfied by the older phase.
-      if (ok && ntiles >= 2)
-        ok = __all_sync(0xffffffffu, mbar_wait(&bars->pv_done, (ntiles - 2) & 1, p.status));
-      if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->pv_done, (ntiles - 1) & 1, p.status));
+      // The last product has a barrier of its own: the final phases of pv_done may both have passed
+      // before a warp gets here, and a parity wait cannot tell two completions from none.
+      if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->o_done, 0, p.status));
       if (ok) {
         tc_fence_after_sync();
 #pragma unroll

@@ -62,6 +62,7 @@ struct alignas(8) MlaBars {
   uint64_t s_full[2], s_empty[2];
   uint64_t p_full[2], p_empty[2];
   uint64_t pv_done;
+  uint64_t o_done;        // completes once, after the product of the last tile
   uint64_t grp;
   uint32_t tmem_base;
   float red_max[2][4][kNQ];
@@ -126,6 +127,7 @@ __global__ void __launch_bounds__(192, 1)
       mbar_init(&bars->p_empty[i], 1);
     }
     mbar_init(&bars->pv_done, 1);
+    mbar_init(&bars->o_done, 1);
     mbar_init(&bars->grp, 4);
     mbar_fence_init();
   }
@@ -245,6 +247,7 @@ __global__ void __launch_bounds__(192, 1)
           }
           umma_commit(&bars->pv_done);    // before p_empty: whoever sees p_empty has this arrival too
           umma_commit(&bars->p_empty[pb]);
+          if (!next) umma_commit(&bars->o_done);
           if (next) {
             for (int pc = 1; pc < kVPieces && ok; ++pc) ok = s_piece(j + 1, pc, false);
             if (ok) umma_commit(&bars->s_full[(j + 1) & 1]);
@@ -340,10 +343,9 @@ __global__ void __launch_bounds__(192, 1)
         __syncwarp();
         if (lane == 0) mbar_arrive(&bars->p_full[pb]);
       }
-      // observe the last two completions in order (the loop only guarantees ntiles-2 seen)
-      if (ok && ntiles >= 2)
-        ok = __all_sync(0xffffffffu, mbar_wait(&bars->pv_done, (ntiles - 2) & 1, p.status));
-      if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->pv_done, (ntiles - 1) & 1, p.status));
+      // The last product has a barrier of its own: the final phases of pv_done may both have passed
+      // before a warp gets here, and a parity wait cannot tell two completions from none.
+      if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->o_done, 0, p.status));
       if (ok) {
         tc_fence_after_sync();
 #pragma unroll
