@@ -171,11 +171,12 @@ typedef struct B200MoeScatter {
   const void* op_counter;
 } B200MoeScatter;
 
-// Attention with a per-head distance bias, mixed heads and an optional null softmax entry over pages
-// [block_size][kw] keys | [block_size][G * vdim] values (attn_bias.cu). q rows carry the score scale;
-// every head reads the whole key row. bias: fp32 [H, bias_len], the entry of distance
-// min(i - j, bias_len - 1), or null. Decode: one row per request. Prefill: q_start [num_reqs + 1]
-// and the 128-row tile list. f32: fp32 q / out / cache instead of bf16.
+// Attention over pages [block_size][kw] keys | [block_size][G * vdim] values (attn_bias.cu). kw is the
+// whole key row; a head reads all of it (query rows kw wide, see b200_head_mix_kv) or, with ``grouped``, the
+// kw / G columns of its group (query rows that wide). Scores are multiplied by ``scale``. bias: fp32
+// [H, bias_len], the entry of distance min(i - j, bias_len - 1), or null. chunk > 0: position i sees j <= i
+// with i / chunk == j / chunk. null_entry: one softmax entry of score 0 without a value. Decode: one row per
+// request. Prefill: q_start [num_reqs + 1] and the 128-row tile list. f32: fp32 q / out / cache, not bf16.
 typedef struct B200BiasAttn {
   const void* q;
   long long ldq;
@@ -194,11 +195,49 @@ typedef struct B200BiasAttn {
   int max_blocks, num_reqs, rows;
   int H, G, kw, vdim, block_size;
   int bias_len, null_entry, f32, splits, num_tiles;
+  int grouped, chunk;
+  float scale;
 } B200BiasAttn;
+
+// Gated delta rule (delta.cu, delta_chunk.cu). Rows: nd decode rows, then the prompt portions listed by
+// q_start / tile_req / tile_q0 (relative to the portions). proj rows: q heads | k heads (G of D each) |
+// v heads (H of V) and, at ``gate``, the output gates (H of V). ab rows: a | b (H each). D, V: padded to
+// multiples of 16; dim, vdim: the sizes themselves. f32: fp32 proj / v / out / conv_state, not bf16.
+typedef struct B200Delta {
+  const void* proj;
+  const void* gate;
+  long long ldp;
+  const float* ab;
+  long long ldab;
+  const float* conv_w;         // [taps][2 G D + H V], the last row is the current token's
+  const float* A;              // [H] exp(A_log)
+  const float* dt;             // [H]
+  const float* norm_w;         // [V]
+  void* conv_state;            // [slots][taps - 1][2 G D + H V]
+  float* state;                // [slots][H][D][V]
+  float* q;                    // [T, G, D] unit, q also times q_scale
+  float* k;
+  void* v;                     // [T, H, V]
+  float* g;                    // [T, H] log of the decay
+  float* beta;                 // [T, H]
+  float* o;                    // [T, H, V] fp32 (chunked prompts, before the norm)
+  void* out;
+  long long ldo;
+  const int* seq_lens;         // per request, decode rows first
+  const int* slots;
+  const int* q_start;
+  const int* tile_req;
+  const int* tile_q0;
+  int nd, num_prefills, num_tiles, T;
+  int G, H, D, V, dim, vdim, taps, f32;
+  float eps, q_scale;
+} B200Delta;
 
 // fp32 residual stream update + RMSNorm in one pass per row (stream.cu):
 //   start:  stream = table[ids] * scale        (ids non-null)
 //   else:   stream += a + sum_j w_j y[pair_pos[j]]   (a, y each optional; pair_w null: w = 1)
+// post_w: the update is first divided by its own rms and multiplied by post_w + norm_offset. ident: rows that
+// stand for y where pair_pos < 0 (experts that return their input; may be ``out``).
 //   out = stream / rms(stream) * (norm_w + norm_offset)
 // Rows are `width` values in storage padded to `cols` (a multiple of 8, zeros). norm_w: fp32.
 typedef struct B200StreamNorm {
@@ -207,11 +246,13 @@ typedef struct B200StreamNorm {
   const void* table;
   const void* a;
   const void* y;
-  const void* pair_pos;        // int32 [T, k], < 0: skipped
+  const void* pair_pos;        // int32 [T, k], < 0: skipped (or ident)
   const float* pair_w;
   const float* norm_w;
+  const float* post_w;
+  const void* ident;
   void* out;
-  long long lds, lda, ldy, ldo, vocab;
+  long long lds, lda, ldy, ldi, ldo, vocab;
   int T, width, cols, k;
   int f32, a_f32;              // element type of table / y / out, and of a
   float scale, eps, norm_offset;
@@ -257,6 +298,7 @@ int b200_merge_attn_states(const void* a, const void* lse_a, const void* b, cons
 int b200_attn_decode_tc(const void* q, int ldq, void* out, int ldo, const void* kv_cache, int64_t num_blocks, int block_size, int Hq, int Hkv, int D, const void* block_table, int max_blocks, const void* seq_lens, int B, float scale, float softcap, int window, int splits, void* tmp_o, void* tmp_lse, cudaStream_t stream);
 // ---- attn_bias.cu
 int b200_head_mix_kv(const void* qkv, long long ld, const void* mix, void* q_out, long long ldq, const void* slots, void* cache, int H, int G, int dim, int vdim, int block_size, int T, int f32, cudaStream_t stream);
+int b200_rotate_kv(const void* qkv, long long ld, const void* positions, const void* cos_sin, int rot, float eps, void* q_out, long long ldq, const void* slots, void* cache, int H, int G, int D, int V, int dim, int block_size, int T, int f32, cudaStream_t stream);
 int b200_bias_attn_kernel(const B200BiasAttn* a, int phase);
 int b200_bias_attn_decode(const B200BiasAttn* a, int any_size, cudaStream_t stream);
 int b200_bias_attn_prefill(const B200BiasAttn* a, int any_size, cudaStream_t stream);
@@ -272,6 +314,10 @@ int b200_gdn_packed_decode(const void* xc, long ld, const void* a, const void* b
 int b200_rmsnorm_gated(const void* x, long ldx, const void* z, long ldz, const void* w, void* out, long ldo, long R, int D, float eps, int gate_kind, int heads, cudaStream_t stream);
 // ---- gdn_scan.cu
 int b200_gdn_chunk_scan(const void* q, const void* k, const void* v, long ldv, int v_col0, const float* g, const float* beta, int T, int Hk, int Hv, const int* chunk_tok0, const int* chunk_len, int NT, const int* seq_chunk0, const int* slots, const int* has_init, int n_seq, float* state, void* u, void* w, void* qs, void* pbuf, float* gc, void* out, cudaStream_t stream);
+// ---- delta.cu
+int b200_delta_prepare(const B200Delta* a, cudaStream_t stream);
+int b200_delta_rule(const B200Delta* a, int reqs, cudaStream_t stream);
+int b200_delta_norm(const B200Delta* a, int rows, cudaStream_t stream);
 // ---- gemm_bf16.cu
 int b200_gemm_bf16_gated(const void* A, int lda, const void* W, int ldw, void* out, int ldo, int M, int N, int K, int kind, int force_path, cudaStream_t stream);
 int b200_gemm_fp8_pair(const void* A, int lda, const void* W, int ldw, void* out, int ldo, const float* a_scale, const float* w_scale, int w_scale_per_channel, const void* bias, int M, int N, int K, cudaStream_t stream);
@@ -304,7 +350,7 @@ int b200_mla_assemble_kv(const void* kvb, const void* dense, void* cache, int N,
 int b200_mla_pad_q(const void* q, long ldq, void* out, int T, int H, cudaStream_t stream);
 int b200_mla_copy_qpe(const void* q, long ldq, void* qabs, int T, int H, cudaStream_t stream);
 // ---- moe.cu
-int b200_moe_router_topk(const void* logits_f32, int ld, int T, int E, int k, int renorm, int scoring, const void* e_bias, int n_group, int topk_group, float routed_scale, void* topk_ids, void* topk_w, cudaStream_t stream);
+int b200_moe_router_topk(const void* logits_f32, int ld, int T, int E, int k, int renorm, int scoring, const void* e_bias, int n_group, int topk_group, int group_best, float routed_scale, void* topk_ids, void* topk_w, cudaStream_t stream);
 int b200_moe_sort(const void* topk_ids, int T, int k, int e0, int e1, void* meta, void* sorted_token, void* pair_pos, void* chunk_expert, void* chunk_row0, void* chunk_n, int max_chunks, cudaStream_t stream);
 int b200_moe_gather(const void* x, int ldx, const void* sorted_token, const void* meta, int E, void* xs, int H, int max_rows, cudaStream_t stream);
 int b200_moe_grouped_gemm(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, cudaStream_t stream);
@@ -327,6 +373,7 @@ int b200_gather_rows(const void* x, const void* idx, void* out, int n_out, int n
 int b200_stream_norm(const B200StreamNorm* a, cudaStream_t stream);
 int b200_gemm_f32(const void* A, int lda, const void* W, int ldw, void* out, int ldo, const void* bias, int M, int N, int K, cudaStream_t stream);
 int b200_moe_grouped_gemm_f32(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, cudaStream_t stream);
+int b200_gated_act_f32(const void* gate_up, int ldg, void* out, int ldo, int T, int I, int kind, cudaStream_t stream);
 int b200_clamped_gate_f32(const void* gate_up, void* out, const void* meta, int E, int max_rows, int I, const B200ClampedGate* act, cudaStream_t stream);
 // ---- rope_cache.cu
 int b200_rope_kv(void* qkv, int ld, int q_off, int k_off, int v_off, int q_head_stride, int Hq, int Hkv, int D, int rot, const void* positions, const void* cos_sin, const void* q_norm_w, const void* k_norm_w, float eps, int gemma, int neox, const void* slot_mapping, void* kv_cache, int block_size, void* q_out, int T, cudaStream_t stream);

@@ -1,13 +1,15 @@
-// Attention whose scores carry a per-head distance bias and a mix of the heads, with an optional
-// null entry in the softmax, over a paged cache with separate key and value widths.
+// Attention over a paged cache with separate key and value widths: scores may carry a per-head distance
+// bias and a mix of the heads, the softmax a null entry, and a query may be limited to its own chunk of
+// positions.
 //
-//   s[h, i, j] = sum_g M[h, g] (q_g(i) . k_g(j)) + bias[h, min(i - j, L - 1)]
+//   s[h, i, j] = scale sum_g M[h, g] (q_g(i) . k_g(j)) + bias[h, min(i - j, L - 1)]
 //   p[h, i, j] = exp(s) / (null + sum_j exp(s)),   o[h, i] = sum_j p[h, i, j] v_{h / R}(j)
 //
 // A mix of heads before the softmax is linear in the queries, so it moves to the query side: head h
 // gets the query row  q'_h = [ sum_{g in group 0} M[h, g] q_g | sum_{g in group 1} ... ]  over the
 // concatenated key heads, one key row per token serves every head (b200_head_mix_kv builds the
-// rows and writes the cache), and the score is one dot product of the full key row.
+// rows and writes the cache), and the score is one dot product of the full key row. Without a mix
+// ("grouped") a head's query row meets the columns of its own group only.
 //
 // Cache of a layer: [num_blocks] pages of  [block_size][kw] keys | [block_size][vw] values,
 // kw = key row, vw = value row (all key / value heads), one element type.
@@ -29,6 +31,9 @@
 namespace b200 {
 
 static constexpr float kLog2e = 1.4426950408889634f;
+
+bool grouped_decode_fits(const B200BiasAttn* a);            // attn_grouped.cu
+int grouped_decode(const B200BiasAttn* a, cudaStream_t stream);
 
 __device__ __forceinline__ float to_f(float v) { return v; }
 __device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
@@ -187,6 +192,9 @@ struct BiasAttnParams {
   const int32_t* q_start;   // [num_reqs + 1] first row of each request; null: one row per request
   int num_reqs, rows;
   int H, G, kw, vdim, block_size;
+  int qw;                   // width of a head's query row: kw, or kw / G (grouped)
+  int chunk;                // > 0: keys of the query's own chunk of this many positions
+  float scale;
   const float* bias;        // [H, bias_len] or null
   int bias_len;
   int null_entry;           // softmax counts one entry of score 0 without a value
@@ -210,8 +218,8 @@ static constexpr int kAnyAcc = 16;     // outputs per thread: kAnyHeads * vdim <
 template <typename T>
 __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
   extern __shared__ float any_smem[];
-  float* sq = any_smem;                                  // [kAnyHeads][kw]
-  float* sc = sq + kAnyHeads * p.kw;                     // [kAnyHeads][kAnyKeys]
+  float* sq = any_smem;                                  // [kAnyHeads][qw]
+  float* sc = sq + kAnyHeads * p.qw;                     // [kAnyHeads][kAnyKeys]
   __shared__ long long krow[kAnyKeys], vrow[kAnyKeys];
   __shared__ float s_alpha[kAnyHeads], s_l[kAnyHeads];
   pdl_wait();
@@ -231,8 +239,8 @@ __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
   } else {
     pos = p.seq_lens[req] - 1;
   }
-  const T* q = reinterpret_cast<const T*>(p.q) + (size_t)row * p.ldq + (size_t)h0 * p.kw;
-  for (int i = tid; i < nh * p.kw; i += blockDim.x) sq[i] = to_f(q[i]);
+  const T* q = reinterpret_cast<const T*>(p.q) + (size_t)row * p.ldq + (size_t)h0 * p.qw;
+  for (int i = tid; i < nh * p.qw; i += blockDim.x) sq[i] = to_f(q[i]);
   const T* cache = reinterpret_cast<const T*>(p.cache);
   const int32_t* bt = p.block_table + (size_t)req * p.max_blocks;
   float acc[kAnyAcc];
@@ -240,7 +248,7 @@ __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
   for (int a = 0; a < kAnyAcc; ++a) acc[a] = 0.f;
   // warp w owns the softmax state of head h0 + w
   float m = p.null_entry ? 0.f : -INFINITY, l = p.null_entry ? 1.f : 0.f;
-  for (int base = 0; base <= pos; base += kAnyKeys) {
+  for (int base = p.chunk > 0 ? pos / p.chunk * p.chunk : 0; base <= pos; base += kAnyKeys) {
     const int key = base + tid;
     const bool valid = key <= pos;
     __syncthreads();
@@ -253,14 +261,23 @@ __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
 #pragma unroll
       for (int h = 0; h < kAnyHeads; ++h) s[h] = 0.f;
       const T* k = cache + krow[tid];
-      for (int i = 0; i < p.kw; ++i) {
-        const float kv = to_f(k[i]);
+      if (p.qw < p.kw) {
 #pragma unroll
-        for (int h = 0; h < kAnyHeads; ++h) s[h] = fmaf(sq[h * p.kw + i], kv, s[h]);
+        for (int h = 0; h < kAnyHeads; ++h) {
+          if (h >= nh) break;
+          const T* kg = k + (size_t)((h0 + h) / R) * p.qw;
+          for (int i = 0; i < p.qw; ++i) s[h] = fmaf(sq[h * p.qw + i], to_f(kg[i]), s[h]);
+        }
+      } else {
+        for (int i = 0; i < p.kw; ++i) {
+          const float kv = to_f(k[i]);
+#pragma unroll
+          for (int h = 0; h < kAnyHeads; ++h) s[h] = fmaf(sq[h * p.kw + i], kv, s[h]);
+        }
       }
       for (int h = 0; h < nh; ++h)
         sc[h * kAnyKeys + tid] =
-            s[h] + (p.bias ? p.bias[(size_t)(h0 + h) * p.bias_len + min(pos - key, p.bias_len - 1)] : 0.f);
+            s[h] * p.scale + (p.bias ? p.bias[(size_t)(h0 + h) * p.bias_len + min(pos - key, p.bias_len - 1)] : 0.f);
     } else {
       for (int h = 0; h < nh; ++h) sc[h * kAnyKeys + tid] = -INFINITY;
     }
@@ -734,7 +751,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                              const __grid_constant__ CUtensorMap tmV, BiasAttnParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const int nkc = (p.kw + 63) / 64, nvc = (p.vdim + 63) / 64;
+  const int nkc = (p.qw + 63) / 64, nvc = (p.vdim + 63) / 64;
   const int slot_bytes = p.q_stream ? 2 * kChunkBytes : kChunkBytes;      // [keys | queries]
   uint8_t* sQ = smem;
   uint8_t* sK = sQ + (p.q_stream ? 0 : nkc * kChunkBytes);
@@ -747,7 +764,10 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
   const int q_begin = p.q_start[req], q_len = p.q_start[req + 1] - q_begin;
   const int seq_len = p.seq_lens[req], ctx_off = seq_len - q_len;
   const int rows = min(kBQ, q_len - q0);
-  const int ntiles = (ctx_off + q0 + rows - 1) / kBKeys + 1;
+  // first key tile: that of the chunk start of the first row
+  const int lo_tile = p.chunk > 0 ? (ctx_off + q0) / p.chunk * p.chunk / kBKeys : 0;
+  const int ntiles = (ctx_off + q0 + rows - 1) / kBKeys + 1 - lo_tile;
+  const int k_col = p.qw < p.kw ? hkv * p.qw : 0;
   // TMEM columns: S buffers (128 each), then O, then two P buffers (64 each)
   const int s_bufs = p.vdim > 128 ? 1 : 2;
   const int o_cols = p.vdim > 128 ? 256 : 128;
@@ -779,7 +799,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
     const int32_t* bt = p.block_table + (size_t)req * p.max_blocks;
     const int nblk = (seq_len + p.block_size - 1) / p.block_size;
     auto page_of = [&](int j) {
-      const int bi = (j * kBKeys + lane * rpl) / p.block_size;
+      const int bi = ((lo_tile + j) * kBKeys + lane * rpl) / p.block_size;
       return max(lane < loads && bi < nblk ? bt[bi] : bt[0], 0);
     };
     if (lane == 0) {
@@ -789,7 +809,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
       if (!p.q_stream) {
         mbar_expect_tx(&bars->q_full, nkc * kChunkBytes);
         for (int c = 0; c < nkc; ++c)
-          tma_load_2d(sQ + c * kChunkBytes, &tmQ, &bars->q_full, h * p.kw + c * 64, q_begin + q0);
+          tma_load_2d(sQ + c * kChunkBytes, &tmQ, &bars->q_full, h * p.qw + c * 64, q_begin + q0);
       }
     }
     int sl = 0, blk = page_of(0), blk_prev = 0;
@@ -799,7 +819,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
     for (int j = 0; j <= ntiles && ok; ++j) {
       const int next = j + 1 < ntiles ? page_of(j + 1) : 0;
       if (j < ntiles) {
-        const int row = p.block_size > kBKeys ? (j * kBKeys) % p.block_size : 0;
+        const int row = p.block_size > kBKeys ? ((lo_tile + j) * kBKeys) % p.block_size : 0;
         for (int c = 0; c < nkc; ++c) {
           ok = __all_sync(0xffffffffu, mbar_wait(&bars->k_empty[sl], ph, p.status));
           if (!ok) break;
@@ -807,16 +827,16 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
           if (lane == 0) {
             mbar_expect_tx(&bars->k_full[sl], slot_bytes);
             if (p.q_stream)
-              tma_load_2d(dst + kChunkBytes, &tmQ, &bars->k_full[sl], h * p.kw + c * 64, q_begin + q0);
+              tma_load_2d(dst + kChunkBytes, &tmQ, &bars->k_full[sl], h * p.qw + c * 64, q_begin + q0);
           }
           __syncwarp();
-          if (lane < loads) tma_load_3d(dst + lane * rpl * 128, &tmK, &bars->k_full[sl], c * 64, row, blk);
+          if (lane < loads) tma_load_3d(dst + lane * rpl * 128, &tmK, &bars->k_full[sl], k_col + c * 64, row, blk);
           if (++sl == p.k_slots) { sl = 0; ph ^= 1; }
         }
       }
       if (j >= 1 && ok) {
         const int i = j - 1, vs = i % p.v_slots;
-        const int row = p.block_size > kBKeys ? (i * kBKeys) % p.block_size : 0;
+        const int row = p.block_size > kBKeys ? ((lo_tile + i) * kBKeys) % p.block_size : 0;
         ok = __all_sync(0xffffffffu, mbar_wait(&bars->v_empty[vs], ((i / p.v_slots) & 1) ^ 1, p.status));
         if (!ok) break;
         if (lane == 0) mbar_expect_tx(&bars->v_full[vs], nvc * kChunkBytes);
@@ -837,7 +857,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
       // descriptors advance by plain adds: 16 k elements are 32 bytes = 2 address units
       const uint64_t qd0 = umma_desc_k_sw128(smem_u32(sQ), 1024), kd0 = umma_desc_k_sw128(smem_u32(sK), 1024);
       const uint64_t vd0 = umma_desc_mn_sw128(smem_u32(sV), kChunkBytes, 1024);
-      const int tail = (p.kw - (nkc - 1) * 64 + 15) / 16;          // instructions of the last chunk
+      const int tail = (p.qw - (nkc - 1) * 64 + 15) / 16;          // instructions of the last chunk
       int ksl = 0;
       uint32_t kph = 0;
       for (int j = 0; j <= ntiles && ok; ++j) {
@@ -883,16 +903,19 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
     const int quarter = warp & 3, half = (warp - 2) >> 2, r = quarter * 32 + lane;
     const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
     const int q_pos = ctx_off + q0 + r, hi = min(q_pos, seq_len - 1);
+    const int lo = p.chunk > 0 ? q_pos / p.chunk * p.chunk : 0;
     const int warp_pos0 = ctx_off + q0 + quarter * 32;       // position of the warp's first row
+    const int warp_lo = p.chunk > 0 ? (warp_pos0 + 31) / p.chunk * p.chunk : 0;   // largest lo of its rows
     const int key0 = half * 64;                              // this thread's keys inside a tile
+    const float scale2 = p.scale * kLog2e;
     const float* bias = p.bias ? p.bias + (size_t)h * p.bias_len : nullptr;
     const int last = p.bias_len - 1;
     const float far = bias ? bias[last] * kLog2e : 0.f;
-    // Window entry e of tile j holds the bias of distance d0 - e, d0 = warp_pos0 + 31 - j * 128; key k
+    // Window entry e of tile j (from lo_tile) holds the bias of distance d0 - e, d0 = warp_pos0 + 31 - its first key; key k
     // of the tile is entry 31 - lane + k for this row. Tiles that lie wholly beyond the table need none.
-    auto tile_near = [&](int j) { return bias && warp_pos0 - (j * kBKeys + kBKeys - 1) < last; };
+    auto tile_near = [&](int j) { return bias && warp_pos0 - ((lo_tile + j) * kBKeys + kBKeys - 1) < last; };
     auto fill_window = [&](int j) {
-      const int d0 = warp_pos0 + 31 - j * kBKeys;
+      const int d0 = warp_pos0 + 31 - (lo_tile + j) * kBKeys;
 #pragma unroll
       for (int i = 0; i < 3; ++i) {
         const int e = half * 32 + lane + i * 64;
@@ -907,7 +930,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
     if (tile_near(0)) fill_window(0);
     pair_sync(quarter);
     for (int j = 0; j < ntiles; ++j) {
-      const int sb = j % s_bufs, pb = j & 1, kbase = j * kBKeys + key0;
+      const int sb = j % s_bufs, pb = j & 1, kbase = (lo_tile + j) * kBKeys + key0;
       // after a wait that ran out the warp goes through the motions without waiting, so that its
       // partner is never left at a barrier
       ok = ok && __all_sync(0xffffffffu, mbar_wait(&bars->s_full[sb], (j / s_bufs) & 1, p.status));
@@ -924,21 +947,21 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
         const float* w = bars->window[j & 1][quarter] + 31 - lane + key0;
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          s0[i] = __float_as_uint(fmaf(__uint_as_float(s0[i]), kLog2e, w[i]));
-          s1[i] = __float_as_uint(fmaf(__uint_as_float(s1[i]), kLog2e, w[i + 32]));
+          s0[i] = __float_as_uint(fmaf(__uint_as_float(s0[i]), scale2, w[i]));
+          s1[i] = __float_as_uint(fmaf(__uint_as_float(s1[i]), scale2, w[i + 32]));
         }
       } else {
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          s0[i] = __float_as_uint(fmaf(__uint_as_float(s0[i]), kLog2e, far));
-          s1[i] = __float_as_uint(fmaf(__uint_as_float(s1[i]), kLog2e, far));
+          s0[i] = __float_as_uint(fmaf(__uint_as_float(s0[i]), scale2, far));
+          s1[i] = __float_as_uint(fmaf(__uint_as_float(s1[i]), scale2, far));
         }
       }
-      if (kbase + 63 > min(warp_pos0, seq_len - 1)) {                    // (warp-uniform)
+      if (kbase + 63 > min(warp_pos0, seq_len - 1) || kbase < warp_lo) {                    // (warp-uniform)
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          if (kbase + i > hi) s0[i] = __float_as_uint(-INFINITY);
-          if (kbase + 32 + i > hi) s1[i] = __float_as_uint(-INFINITY);
+          if (kbase + i > hi || kbase + i < lo) s0[i] = __float_as_uint(-INFINITY);
+          if (kbase + 32 + i > hi || kbase + 32 + i < lo) s1[i] = __float_as_uint(-INFINITY);
         }
       }
       float mx0 = -INFINITY, mx1 = -INFINITY;
@@ -1034,6 +1057,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
 // Shapes the decode kernel serves. tk: keys per tile; cls: register class (0: 8 output tiles, 2 query
 // chunks and 4 heads per warp, 1: 16 tiles, 8 heads, queries in shared memory).
 static bool decode_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem, int& tk, int& cls) {
+  if (a->grouped || a->chunk || a->scale != 1.f) return false;           // (attn_grouped.cu)
   if (a->f32 || (a->kw & 7) || (a->vdim & 7) || (a->ldq & 7) || (a->ldo & 1)) return false;
   if (((uintptr_t)a->q | (uintptr_t)a->cache) & 15) return false;
   const int R = a->H / a->G, nkc = (a->kw + 63) / 64;
@@ -1076,7 +1100,9 @@ static bool prefill_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem)
   if (((uintptr_t)a->q | (uintptr_t)a->cache | (uintptr_t)a->out) & 15) return false;
   const int bs = a->block_size;
   if (bs < 8 || (bs & 7) || (bs < kBKeys && kBKeys % bs) || (bs > kBKeys && bs % kBKeys)) return false;
-  const int nkc = (a->kw + 63) / 64, nvc = (a->vdim + 63) / 64;
+  // a group's columns start on a 16-byte boundary and the last product of 16 reads none of the next group
+  if (a->grouped && (a->kw / a->G & 15)) return false;
+  const int nkc = ((a->grouped ? a->kw / a->G : a->kw) + 63) / 64, nvc = (a->vdim + 63) / 64;
   const int limit = 227 * 1024, fixed = (int)sizeof(BiasPrefillBars) + 1024;
   // the query tile stays in shared memory if enough of the key ring fits beside it
   for (p.q_stream = 0; p.q_stream < 2; ++p.q_stream) {
@@ -1143,6 +1169,7 @@ static BiasAttnParams common_params(const B200BiasAttn* a) {
   p.seq_lens = (const int32_t*)a->seq_lens; p.q_start = (const int32_t*)a->q_start;
   p.num_reqs = a->num_reqs; p.rows = a->rows;
   p.H = a->H; p.G = a->G; p.kw = a->kw; p.vdim = a->vdim; p.block_size = a->block_size;
+  p.qw = a->grouped ? a->kw / a->G : a->kw; p.chunk = a->chunk; p.scale = a->scale;
   p.bias = (const float*)a->bias; p.bias_len = a->bias_len; p.null_entry = a->null_entry;
   p.splits = a->splits < 1 ? 1 : a->splits; p.tmp_o = (float*)a->tmp_o; p.tmp_lse = (float*)a->tmp_lse;
   p.tile_req = (const int32_t*)a->tile_req; p.tile_q0 = (const int32_t*)a->tile_q0;
@@ -1153,7 +1180,7 @@ static BiasAttnParams common_params(const B200BiasAttn* a) {
 template <typename T>
 static int launch_any(const BiasAttnParams& p, cudaStream_t stream) {
   if ((long)kAnyHeads * p.vdim > 128l * kAnyAcc) return -4;
-  const size_t smem = (size_t)kAnyHeads * (p.kw + kAnyKeys) * 4;
+  const size_t smem = (size_t)kAnyHeads * (p.qw + kAnyKeys) * 4;
   if (smem > 200 * 1024) return -4;
   static PerDeviceOnce once;
   if (once.first()) cudaFuncSetAttribute(bias_attn_any_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
@@ -1222,7 +1249,7 @@ static int launch_mix_vec(const MixParams& p, cudaStream_t stream) {
 
 static bool valid_args(const B200BiasAttn* a) {
   return a->H > 0 && a->G > 0 && a->H % a->G == 0 && a->kw > 0 && a->vdim > 0 && a->block_size > 0 &&
-         (!a->bias || a->bias_len > 0);
+         (!a->bias || a->bias_len > 0) && (!a->grouped || a->kw % a->G == 0) && a->chunk >= 0;
 }
 
 }  // namespace b200
@@ -1253,7 +1280,8 @@ int b200_bias_attn_kernel(const B200BiasAttn* a, int phase) {
   size_t smem;
   int tk, cls;
   if (!valid_args(a)) return 0;
-  return (phase == 0 ? decode_plan(a, p, smem, tk, cls) : prefill_plan(a, p, smem)) ? 2 : 1;
+  if (phase == 0) return decode_plan(a, p, smem, tk, cls) || grouped_decode_fits(a) ? 2 : 1;
+  return prefill_plan(a, p, smem) ? 2 : 1;
 }
 
 int b200_bias_attn_decode(const B200BiasAttn* a, int any_size, cudaStream_t stream) {
@@ -1263,6 +1291,7 @@ int b200_bias_attn_decode(const B200BiasAttn* a, int any_size, cudaStream_t stre
   p.q_start = nullptr;
   size_t smem;
   int tk, cls;
+  if (!any_size && grouped_decode_fits(a)) return grouped_decode(a, stream);
   if (any_size || !decode_plan(a, p, smem, tk, cls))
     return a->f32 ? launch_any<float>(p, stream) : launch_any<__nv_bfloat16>(p, stream);
   if (p.splits > 1 && (!p.tmp_o || !p.tmp_lse)) return -1;
@@ -1283,7 +1312,7 @@ int b200_bias_attn_prefill(const B200BiasAttn* a, int any_size, cudaStream_t str
     return a->f32 ? launch_any<float>(p, stream) : launch_any<__nv_bfloat16>(p, stream);
   if (a->num_tiles <= 0) return 0;
   CUtensorMap tmQ, tmK, tmV;
-  if (!encode_tmap_2d(&tmQ, a->q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)a->rows, (uint64_t)a->H * a->kw,
+  if (!encode_tmap_2d(&tmQ, a->q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)a->rows, (uint64_t)a->H * p.qw,
                       (uint64_t)a->ldq, kBQ, 64, CU_TENSOR_MAP_SWIZZLE_128B) ||
       !page_maps(a, kBKeys, &tmK, &tmV))
     return -3;

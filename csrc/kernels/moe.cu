@@ -23,13 +23,13 @@ namespace b200 {
 
 // --------------------------------------------------------------------------- router top-k
 // One block per token. scoring: 0 softmax, 1 sigmoid. Grouped selection (n_group > 1): the
-// experts are split into n_group groups, a group's score is the sum of its two best
+// experts are split into n_group groups, a group's score is the sum of its group_best (1 or 2) best
 // (bias-corrected) scores, only the topk_group best groups stay eligible. Selection uses
 // score + bias, the returned weight is the unbiased score. Ties break to the lowest index.
 __global__ void __launch_bounds__(256)
     moe_router_topk_kernel(const float* __restrict__ logits, int ld, int E, int k, int renorm,
                            int scoring, const float* __restrict__ e_bias, int n_group,
-                           int topk_group, float routed_scale, int32_t* topk_ids, float* topk_w) {
+                           int topk_group, int group_best, float routed_scale, int32_t* topk_ids, float* topk_w) {
   extern __shared__ float sh[];   // E scores, E selection scores
   float* score = sh;
   float* sel = sh + E;
@@ -79,7 +79,7 @@ __global__ void __launch_bounds__(256)
         const float v = sel[threadIdx.x * per + i];
         if (v > b0) { b1 = b0; b0 = v; } else if (v > b1) { b1 = v; }
       }
-      gscore[threadIdx.x] = e_bias ? b0 + b1 : b0;
+      gscore[threadIdx.x] = group_best == 2 ? b0 + b1 : b0;
     }
     __syncthreads();
     if (threadIdx.x == 0) {
@@ -543,13 +543,13 @@ typedef __nv_bfloat16 bf16;
 extern "C" {
 
 int b200_moe_router_topk(const void* logits_f32, int ld, int T, int E, int k, int renorm,
-                         int scoring, const void* e_bias, int n_group, int topk_group,
+                         int scoring, const void* e_bias, int n_group, int topk_group, int group_best,
                          float routed_scale, void* topk_ids, void* topk_w, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (k > E || n_group > 64 || (n_group > 1 && E % n_group)) return -1;
   moe_router_topk_kernel<<<T, 256, (size_t)2 * E * sizeof(float), stream>>>(
       (const float*)logits_f32, ld, E, k, renorm, scoring, (const float*)e_bias, n_group,
-      topk_group, routed_scale, (int32_t*)topk_ids, (float*)topk_w);
+      topk_group, group_best, routed_scale, (int32_t*)topk_ids, (float*)topk_w);
   RETL;
 }
 

@@ -1,8 +1,9 @@
 // The fp32 residual stream of models that keep it in 32 bits, and true fp32 products (no reduced
 // precision mode) for running such a model in 32 bits throughout.
-//   stream_norm_kernel   embedding or residual update (+ expert outputs gathered per token) + RMSNorm
+//   stream_norm_kernel   embedding or residual update (+ expert outputs gathered per token, + norm of the
+//                        update) + RMSNorm
 //   gemm_f32_kernel      out = A W^T (+ bias), plain or per expert chunk
-//   clamped_gate_kernel  activation of [gate | up] rows
+//   clamped_gate_kernel, gated_act_kernel   activation of [gate | up] rows
 #include "api.h"
 #include "sm100.cuh"
 
@@ -43,8 +44,17 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(B200StreamNorm p, int*
   }
   const int32_t* pos = reinterpret_cast<const int32_t*>(p.pair_pos) + (size_t)t * p.k;
   float4 keep[kRegs];
-  float ss = 0.f;
-  auto value = [&](int i) {
+  auto row_sum = [&](float ss) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+    for (int w = 0; w < (int)(blockDim.x >> 5); ++w) ss += red[w];
+    return ss;
+  };
+  auto sq = [](float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; };
+  auto update = [&](int i) {             // what is added to the stream (or starts it)
     float4 v;
     if (p.ids) {
       v = src ? Vec4<T>::load(src + i * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -57,38 +67,57 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(B200StreamNorm p, int*
       else add4(v, Vec4<T>::load(reinterpret_cast<const T*>(p.a) + (size_t)t * p.lda + i * 4));
     }
     for (int j = 0; j < p.k; ++j) {
-      if (pos[j] < 0) continue;
-      float4 y = Vec4<T>::load(reinterpret_cast<const T*>(p.y) + (size_t)pos[j] * p.ldy + i * 4);
+      if (pos[j] < 0 && !p.ident) continue;
+      float4 y = pos[j] < 0 ? Vec4<T>::load(reinterpret_cast<const T*>(p.ident) + (size_t)t * p.ldi + i * 4)
+                            : Vec4<T>::load(reinterpret_cast<const T*>(p.y) + (size_t)pos[j] * p.ldy + i * 4);
       if (p.pair_w) {
         const float w = p.pair_w[(size_t)t * p.k + j];
         y.x *= w; y.y *= w; y.z *= w; y.w *= w;
       }
       add4(v, y);
     }
-    add4(v, Vec4<float>::load(s + i * 4));
     return v;
   };
+  float post = 1.f;                      // 1 / rms of the update
+  if (p.post_w) {
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < kRegs; ++c) {
+      const int i = threadIdx.x + c * blockDim.x;
+      if (i < nv) {
+        keep[c] = update(i);
+        ss += sq(keep[c]);
+      }
+    }
+    for (int i = threadIdx.x + kRegs * blockDim.x; i < nv; i += blockDim.x) ss += sq(update(i));
+    post = 1.f / sqrtf(row_sum(ss) / (float)p.width + p.eps);
+    __syncthreads();                     // (red is used again)
+  }
+  auto value = [&](int i, float4 v) {
+    if (p.post_w) {
+      const float4 w = Vec4<float>::load(p.post_w + i * 4);
+      v.x *= post * (w.x + p.norm_offset); v.y *= post * (w.y + p.norm_offset);
+      v.z *= post * (w.z + p.norm_offset); v.w *= post * (w.w + p.norm_offset);
+    }
+    if (!p.ids) add4(v, Vec4<float>::load(s + i * 4));
+    return v;
+  };
+  float ss = 0.f;
 #pragma unroll
   for (int c = 0; c < kRegs; ++c) {
     const int i = threadIdx.x + c * blockDim.x;
     if (i < nv) {
-      keep[c] = value(i);
+      keep[c] = value(i, p.post_w ? keep[c] : update(i));
       Vec4<float>::store(s + i * 4, keep[c]);
-      ss += keep[c].x * keep[c].x + keep[c].y * keep[c].y + keep[c].z * keep[c].z + keep[c].w * keep[c].w;
+      ss += sq(keep[c]);
     }
   }
   for (int i = threadIdx.x + kRegs * blockDim.x; i < nv; i += blockDim.x) {
-    const float4 v = value(i);
+    const float4 v = value(i, update(i));
     Vec4<float>::store(s + i * 4, v);
-    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    ss += sq(v);
   }
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
-  __syncthreads();
-  ss = 0.f;
-  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) ss += red[w];
-  const float inv = 1.f / sqrtf(ss / (float)p.width + p.eps);
+  const float inv = 1.f / sqrtf(row_sum(ss) / (float)p.width + p.eps);
   T* out = reinterpret_cast<T*>(p.out) + (size_t)t * p.ldo;
   auto finish = [&](int i, float4 v) {
     const float4 w = Vec4<float>::load(p.norm_w + i * 4);
@@ -186,6 +215,21 @@ __global__ void __launch_bounds__(128)
   }
 }
 
+// out = act(gate) * up of fp32 rows [gate (I) | up (I)]. kind: 0 SiLU, 1 GELU-tanh, 2 GELU-erf.
+__global__ void __launch_bounds__(128) gated_act_kernel(const float* gu, int ldg, float* out, int ldo, int I, int kind) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const float* g = gu + (size_t)blockIdx.x * ldg;
+  for (int i = threadIdx.x; i < I; i += blockDim.x) {
+    const float x = g[i];
+    float a;
+    if (kind == 0) a = x / (1.f + expf(-x));
+    else if (kind == 1) a = 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+    else a = 0.5f * x * (1.f + erff(x * 0.7071067811865476f));
+    out[(size_t)blockIdx.x * ldo + i] = a * g[I + i];
+  }
+}
+
 }  // namespace b200
 
 using namespace b200;
@@ -195,7 +239,7 @@ extern "C" {
 int b200_stream_norm(const B200StreamNorm* a, cudaStream_t stream) {
   if (a->T <= 0) return 0;
   if (!a->stream || !a->out || !a->norm_w || a->width <= 0 || a->cols < a->width || (a->cols & 7) || a->k < 0) return -1;
-  if ((a->lds & 3) || (a->lda & 3) || (a->ldy & 3) || (a->ldo & 3) || (a->ids && !a->table)) return -1;
+  if ((a->lds & 3) || (a->lda & 3) || (a->ldy & 3) || (a->ldi & 3) || (a->ldo & 3) || (a->ids && !a->table)) return -1;
   if (a->k > 0 && (!a->pair_pos || !a->y)) return -1;
   int threads = ((a->cols / 4 + 31) / 32) * 32;
   if (threads > 256) threads = 256;
@@ -225,6 +269,13 @@ int b200_moe_grouped_gemm_f32(const void* xs, int max_rows, const void* W, int E
             (const int32_t*)meta + 3 * E + 1};
   dim3 grid((N + kFT - 1) / kFT, 256 / kFT, max_chunks);     // a chunk has at most 256 rows
   return launch_pdl(gemm_f32_kernel, grid, dim3(256), 0, stream, p) == cudaSuccess ? 0 : -2;
+}
+
+int b200_gated_act_f32(const void* gate_up, int ldg, void* out, int ldo, int T, int I, int kind, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (I <= 0 || kind < 0 || kind > 2) return -1;
+  return launch_pdl(gated_act_kernel, dim3(T), dim3(128), 0, stream, (const float*)gate_up, ldg, (float*)out, ldo, I,
+                    kind) == cudaSuccess ? 0 : -2;
 }
 
 int b200_clamped_gate_f32(const void* gate_up, void* out, const void* meta, int E, int max_rows, int I,

@@ -453,7 +453,7 @@ void DenseModel::moe_cuda(const Layer& L, int T) {
   const int H = c.hidden, E = c.num_experts, k = c.experts_per_token, I = c.moe_inter, P = T * k;
   check(b200_gemm_bf16(normed_.data(), H, L.router.data(), H, router_logits_.data(), E, 1, nullptr, nullptr, 0, T, E,
                        H, gemm_ws_.data(), gemm_ws_.nbytes(), kConstW, s), "router");
-  check(b200_moe_router_topk(router_logits_.data(), E, T, E, k, c.norm_topk_prob ? 1 : 0, 0, nullptr, 1, 1, 1.0f,
+  check(b200_moe_router_topk(router_logits_.data(), E, T, E, k, c.norm_topk_prob ? 1 : 0, 0, nullptr, 1, 1, 1, 1.0f,
                              topk_ids_.data(), topk_w_.data(), s), "router_topk");
   check(b200_moe_sort(topk_ids_.data(), T, k, 0, E, moe_meta_.data(), sorted_token_.data(), pair_pos_.data(),
                       chunk_expert_.data(), chunk_row0_.data(), chunk_n_.data(), max_chunks_, s), "moe_sort");

@@ -42,29 +42,57 @@ class RopeConfig:
 
 @dataclass
 class AttentionSpec:
-    """Mixer of one decoder block: grouped heads with separate key and value sizes, a distance bias
-    that saturates at ``bias_max``."""
+    """Softmax mixer of one decoder block: grouped heads with separate key and value sizes. Positions
+    enter through a distance bias that saturates at ``bias_max`` (0: none) or a rotation of the first
+    ``rot_dims`` dimensions (0: none)."""
     heads: int
     kv_heads: int
     dim: int
     vdim: int
     scale: float
-    bias_max: int
+    bias_max: int = 0
+    rot_dims: int = 0
+    rot_base: float = 10000.0
+    chunk: int = 0                            # > 0: a query sees the keys of its own chunk of this many positions
+    kv_from: Optional[int] = None             # block whose keys and values are read (None: its own)
+
+
+@dataclass
+class DeltaSpec:
+    """Gated-delta-rule mixer of one decoder block: ``heads`` states of ``dim`` x ``vdim``, queries and
+    keys shared by ``heads / kv_heads`` heads each, short convolutions of ``conv`` taps."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+
+
+@dataclass
+class DenseSpec:
+    """Feed-forward of one decoder block: one gated unit."""
+    ff: int
 
 
 @dataclass
 class ExpertSpec:
-    """Feed-forward of one decoder block: ``top`` of ``experts`` clamped gated units."""
+    """Feed-forward of one decoder block: ``top`` of ``experts`` gated units (clamped at ``limit``) and
+    ``identity`` experts that return their input; the choice is made among the ``keep`` best of
+    ``groups`` groups of neighbours."""
     experts: int
     top: int
     ff: int
-    limit: float
+    limit: float = float("inf")
+    identity: int = 0
+    groups: int = 1
+    keep: int = 1
 
 
 @dataclass
 class BlockSpec:
-    attention: AttentionSpec
-    mlp: Optional[ExpertSpec] = None
+    attention: Optional[AttentionSpec] = None
+    mlp: "Optional[ExpertSpec | DenseSpec]" = None
+    delta: Optional[DeltaSpec] = None         # set instead of ``attention``
 
 
 @dataclass
@@ -301,60 +329,142 @@ def model_config_from_blocks(cfg: dict) -> ModelConfig:
     """ModelConfig of a config.json that names one ``architecture`` and lists its ``layers``, each
     with a mixer and a feed-forward (or null)."""
     arch = cfg["architecture"]
-    if arch != "Nufusun":
+    readers = {"Nufusun": _nufusun_block, "Diforax": _diforax_block}
+    if arch not in readers:
         raise ValueError(f"no reader for the layer list of architecture {arch!r}")
     blocks = []
     for i, l in enumerate(cfg["layers"]):
-        if l["type"] != "attention":
-            raise ValueError(f"layer {i}: unknown mixer {l['type']!r}")
-        m = l["mixer"]
-        att = AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]),
-                            vdim=int(m["vdim"]), scale=float(m["scale"]), bias_max=int(m["bias_max"]))
-        if att.heads % att.kv_heads:
-            raise ValueError(f"layer {i}: {att.heads} heads do not divide into {att.kv_heads} groups")
-        mlp = None
-        if l.get("mlp") is not None:
-            f = l["mlp"]
-            if f["kind"] != "moe":
-                raise ValueError(f"layer {i}: unknown feed-forward {f['kind']!r}")
-            mlp = ExpertSpec(experts=int(f["router"]["experts"]), top=int(f["router"]["top"]),
-                             ff=int(f["expert"]["ff"]), limit=float(f["expert"]["limit"]))
-            if not 1 <= mlp.top <= mlp.experts:
-                raise ValueError(f"layer {i}: {mlp.top} of {mlp.experts} experts")
-        blocks.append(BlockSpec(att, mlp))
-    m = model_config_of_blocks(arch, blocks, vocab=int(cfg["vocab"]), width=int(cfg["width"]),
-                               eps=float(cfg["norm"]["eps"]), embed_scale=float(cfg["embedding"]["scale"]), raw=cfg)
+        try:
+            blocks.append(_checked(readers[arch](l), blocks))
+        except ValueError as e:
+            raise ValueError(f"layer {i}: {e}") from None
+    kw = dict(vocab=int(cfg["vocab"]), width=int(cfg["width"]), eps=float(cfg["norm"]["eps"]), raw=cfg)
+    if arch == "Nufusun":
+        kw["embed_scale"] = float(cfg["embedding"]["scale"])
+    m = model_config_of_blocks(arch, blocks, **kw)
     m.eos_token_id, m.bos_token_id = cfg.get("eos_token_id"), cfg.get("bos_token_id")
     return m
 
 
-def model_config_of_blocks(arch: str, blocks: list, *, vocab: int, width: int, eps: float, embed_scale: float,
+def _nufusun_block(l: dict) -> BlockSpec:
+    if l["type"] != "attention":
+        raise ValueError(f"unknown mixer {l['type']!r}")
+    m, mlp = l["mixer"], None
+    att = AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                        scale=float(m["scale"]), bias_max=int(m["bias_max"]))
+    if l.get("mlp") is not None:
+        f = l["mlp"]
+        if f["kind"] != "moe":
+            raise ValueError(f"unknown feed-forward {f['kind']!r}")
+        mlp = ExpertSpec(experts=int(f["router"]["experts"]), top=int(f["router"]["top"]), ff=int(f["expert"]["ff"]),
+                         limit=float(f["expert"]["limit"]))
+    return BlockSpec(att, mlp)
+
+
+def _diforax_block(l: dict) -> BlockSpec:
+    m, f = l["mixer"], l.get("mlp")
+    sizes = {k: int(m[k]) for k in ("heads", "kv_heads", "dim", "vdim")}
+    att = delta = mlp = None
+    if l["type"] == "delta":
+        delta = DeltaSpec(**sizes, conv=int(m["conv"]))
+    elif l["type"] == "attention":
+        rot, mask = m.get("rot") or {}, m.get("mask") or {}
+        att = AttentionSpec(**sizes, scale=float(m["scale"]), rot_dims=int(rot.get("dims", 0)),
+                            rot_base=float(rot.get("base", 1.0)), chunk=int(mask.get("size", 0)),
+                            kv_from=None if m.get("kv_from") is None else int(m["kv_from"]))
+    else:
+        raise ValueError(f"unknown mixer {l['type']!r}")
+    if f is not None and f["kind"] == "dense":
+        mlp = DenseSpec(ff=int(f["ff"]))
+    elif f is not None and f["kind"] == "moe":
+        r = f["router"]
+        g = r.get("groups") or {"count": 1, "keep": 1}
+        mlp = ExpertSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(f["expert"]["ff"]),
+                         identity=int(r.get("identity") or 0), groups=int(g["count"]), keep=int(g["keep"]))
+    elif f is not None:
+        raise ValueError(f"unknown feed-forward {f['kind']!r}")
+    return BlockSpec(att, mlp, delta)
+
+
+def _checked(b: BlockSpec, before: list) -> BlockSpec:
+    """The sizes of a block fit together (``before``: the blocks ahead of it)."""
+    m, a, f = b.attention or b.delta, b.attention, b.mlp
+    if m.heads % m.kv_heads:
+        raise ValueError(f"{m.heads} heads do not divide into {m.kv_heads} groups")
+    if a is not None and (a.rot_dims % 2 or a.rot_dims > a.dim):
+        raise ValueError(f"{a.rot_dims} rotated dimensions of {a.dim}")
+    if b.delta is not None and b.delta.conv < 1:
+        raise ValueError("a convolution has at least one tap")
+    if a is not None and a.kv_from is not None:
+        src = before[a.kv_from].attention if 0 <= a.kv_from < len(before) else None
+        if src is None or src.kv_from is not None:
+            raise ValueError(f"block {a.kv_from} has no keys of its own to read")
+        if (src.kv_heads, src.dim, src.vdim) != (a.kv_heads, a.dim, a.vdim):
+            raise ValueError(f"the keys of block {a.kv_from} have other sizes")
+    if isinstance(f, ExpertSpec):
+        n = f.experts + f.identity
+        if n % f.groups or not 1 <= f.keep <= f.groups:
+            raise ValueError(f"{n} experts in {f.groups} groups, {f.keep} kept")
+        if not 1 <= f.top <= n // f.groups * f.keep:
+            raise ValueError(f"{f.top} of {n // f.groups * f.keep} experts")
+    return b
+
+
+def model_config_of_blocks(arch: str, blocks: list, *, vocab: int, width: int, eps: float, embed_scale: float = 1.0,
                            max_position: int = 32768, raw: Optional[dict] = None) -> ModelConfig:
-    att, moe = [b.attention for b in blocks], [b.mlp for b in blocks if b.mlp is not None]
-    return ModelConfig(
+    att = [b.attention for b in blocks if b.attention is not None]
+    moe = [b.mlp for b in blocks if isinstance(b.mlp, ExpertSpec)]
+    dense = [b.mlp.ff for b in blocks if isinstance(b.mlp, DenseSpec)]
+    m = ModelConfig(
         architecture=arch, vocab_size=vocab, hidden_size=width, num_layers=len(blocks),
-        intermediate_size=max([m.ff * m.top for m in moe], default=0), num_heads=max(a.heads for a in att),
-        num_kv_heads=max(a.kv_heads for a in att), head_dim=max(a.dim for a in att),
-        v_head_dim=max(a.vdim for a in att), rms_norm_eps=eps, embed_scale=embed_scale, gemma_norm=True,
-        attention_bias=True, hidden_act="clamped_gate", scoring_func="sigmoid", norm_topk_prob=False,
+        intermediate_size=max([m.ff * m.top for m in moe] + dense, default=0),
+        num_heads=max([a.heads for a in att], default=1), num_kv_heads=max([a.kv_heads for a in att], default=1),
+        head_dim=max([a.dim for a in att], default=8), v_head_dim=max([a.vdim for a in att], default=8),
+        rms_norm_eps=eps, embed_scale=embed_scale, norm_topk_prob=False,
         num_experts=max([m.experts for m in moe], default=0), num_experts_per_tok=max([m.top for m in moe], default=0),
         moe_intermediate_size=max([m.ff for m in moe], default=0), max_position_embeddings=max_position,
         blocks=blocks, raw=raw or {})
+    if arch == "Nufusun":
+        m.gemma_norm, m.attention_bias, m.hidden_act, m.scoring_func = True, True, "clamped_gate", "sigmoid"
+    else:
+        m.sandwich_norm, m.hidden_act = True, "gelu_tanh"
+        m.layer_types = ["linear_attention" if b.delta is not None else "chunked_attention" if b.attention.chunk
+                         else "full_attention" for b in blocks]
+    return m
 
 
 def block_config_dict(cfg: ModelConfig) -> dict:
     """config.json of a ModelConfig with ``blocks`` (the inverse of model_config_from_blocks)."""
     layers = []
     for b in cfg.blocks:
-        a, m = b.attention, b.mlp
-        layers.append({
-            "type": "attention",
-            "mixer": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale,
-                      "bias_max": a.bias_max},
-            "mlp": None if m is None else {"kind": "moe", "router": {"experts": m.experts, "top": m.top},
-                                           "expert": {"ff": m.ff, "limit": m.limit}}})
-    return {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_size,
-            "norm": {"eps": cfg.rms_norm_eps}, "embedding": {"scale": cfg.embed_scale}, "layers": layers}
+        m, a, f, mlp = b.attention or b.delta, b.attention, b.mlp, None
+        mixer = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim}
+        if b.delta is not None:
+            mixer["conv"] = m.conv
+        else:
+            mixer["scale"] = a.scale
+            if a.bias_max:
+                mixer["bias_max"] = a.bias_max
+            if a.rot_dims:
+                mixer["rot"] = {"base": a.rot_base, "dims": a.rot_dims}
+            if a.chunk:
+                mixer["mask"] = {"size": a.chunk}
+            if a.kv_from is not None:
+                mixer["kv_from"] = a.kv_from
+        if isinstance(f, DenseSpec):
+            mlp = {"kind": "dense", "ff": f.ff}
+        elif f is not None:
+            mlp = {"kind": "moe", "router": {"experts": f.experts, "top": f.top}, "expert": {"ff": f.ff}}
+            if cfg.architecture == "Nufusun":
+                mlp["expert"]["limit"] = f.limit
+            else:
+                mlp["router"].update(groups={"count": f.groups, "keep": f.keep}, identity=f.identity)
+        layers.append({"type": "attention" if b.delta is None else "delta", "mixer": mixer, "mlp": mlp})
+    out = {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_size,
+           "norm": {"eps": cfg.rms_norm_eps}, "layers": layers}
+    if cfg.architecture == "Nufusun":
+        out["embedding"] = {"scale": cfg.embed_scale}
+    return out
 
 
 def load_model_config(model_dir: str) -> ModelConfig:
@@ -432,6 +542,22 @@ def synthetic_config(name: str) -> ModelConfig:
                       ExpertSpec(experts=5, top=2, ff=64, limit=2.0))
         return model_config_of_blocks("Nufusun", [b, BlockSpec(b.attention), b], vocab=500, width=192, eps=1e-5,
                                       embed_scale=2.0, max_position=2048)
+    if n in ("diforax-30b-a3b",):
+        # width, attention heads and experts of qwen3-coder-30b-a3b, three delta layers to one attention layer
+        moe = ExpertSpec(experts=128, top=8, ff=768, identity=16, groups=8, keep=4)
+        delta = BlockSpec(None, moe, DeltaSpec(heads=32, kv_heads=16, dim=128, vdim=128, conv=4))
+        att = BlockSpec(AttentionSpec(heads=32, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, rot_dims=128,
+                                      rot_base=1e6, chunk=8192), moe)
+        return model_config_of_blocks("Diforax", [delta, delta, delta, att] * 12, vocab=151936, width=2048, eps=1e-6,
+                                      max_position=262144)
+    if n == "tiny-diforax":
+        att = AttentionSpec(heads=6, kv_heads=3, dim=24, vdim=40, scale=0.3, rot_dims=16, rot_base=5e3, chunk=50)
+        moe = ExpertSpec(experts=6, top=2, ff=64, identity=2, groups=4, keep=2)
+        delta = DeltaSpec(heads=4, kv_heads=2, dim=24, vdim=16, conv=3)
+        shared = AttentionSpec(**{**att.__dict__, "kv_from": 1, "chunk": 70})
+        return model_config_of_blocks("Diforax", [BlockSpec(None, DenseSpec(96), delta), BlockSpec(att, moe),
+                                                  BlockSpec(None, None, delta), BlockSpec(shared, DenseSpec(80))],
+                                      vocab=500, width=192, eps=1e-5, max_position=2048)
     if n.startswith("tiny"):
         # small shapes for tests: tiny-dense, tiny-moe, tiny-mla, tiny-gdn
         base = dict(vocab_size=512, hidden_size=256, intermediate_size=512, num_layers=2,

@@ -269,7 +269,7 @@ class CpuBackend(FusedLinearMixin):
             return out
         return y
 
-    # ---- fp32 residual stream, mixed-head attention with a distance bias, clamped experts
+    # ---- fp32 residual stream, attention over split pages, delta rule, gated units and experts
     def stream_norm(self, stream, norm_w, eps, out, **kw):
         from ..ops.stream import ref_stream_norm
         return ref_stream_norm(stream, norm_w, eps, out, **kw)
@@ -277,6 +277,29 @@ class CpuBackend(FusedLinearMixin):
     def head_mix_kv(self, qkv, mix, q_out, slots, cache, **kw):
         from ..ops.bias_attn import ref_head_mix_kv
         ref_head_mix_kv(qkv, mix, q_out, slots, cache, **kw)
+
+    def rotate_kv(self, qkv, positions, table, rot, eps, q_out, slots, cache, **kw):
+        from ..ops.bias_attn import ref_rotate_kv
+        ref_rotate_kv(qkv, positions, table, rot, eps, q_out, slots, cache, **kw)
+
+    def delta_mixer(self, proj, ab, w, shape, conv_state, state, ctx, bufs, out, eps):
+        from ..ops.delta import ref_delta_mixer
+        return ref_delta_mixer(proj, ab, w, shape, conv_state, state, ctx, bufs, out, eps)
+
+    def gated_unit(self, x, w, kind, out, scratch):
+        gu = self.gemm(x, w, out_dtype=torch.float32)
+        g, u = gu.chunk(2, -1)
+        act = {0: torch.nn.functional.silu, 1: lambda v: torch.nn.functional.gelu(v, approximate="tanh"),
+               2: torch.nn.functional.gelu}[kind]
+        return out.copy_(act(g) * u)
+
+    def routed_experts(self, x, logits, w_gate_up, w_down, ws, *, top, correction, groups, keep):
+        from ..ops import moe as M
+        ids, w = M.ref_router_topk(logits, top, renorm=False, e_bias=correction, n_group=groups, topk_group=keep,
+                                   group_best=1)
+        y = M.ref_clamped_experts(x, ids, None, w_gate_up, w_down)
+        pos = torch.arange(ids.numel(), dtype=torch.int32).view_as(ids)
+        return y, torch.where(ids < w_gate_up.shape[0], pos, torch.full_like(pos, -1)), w
 
     def bias_attention(self, q, cache, ctx, group, *, out, **kw):
         from ..ops.bias_attn import ref_bias_attention
@@ -575,6 +598,32 @@ class GpuBackend(FusedLinearMixin):
     def head_mix_kv(self, qkv, mix, q_out, slots, cache, **kw):
         from ..ops.bias_attn import head_mix_kv
         head_mix_kv(qkv, mix, q_out, slots, cache, **kw)
+
+    def rotate_kv(self, qkv, positions, table, rot, eps, q_out, slots, cache, **kw):
+        from ..ops.bias_attn import rotate_kv
+        rotate_kv(qkv, positions, table, rot, eps, q_out, slots, cache, **kw)
+
+    def delta_mixer(self, proj, ab, w, shape, conv_state, state, ctx, bufs, out, eps):
+        from ..ops.delta import delta_mixer
+        return delta_mixer(proj, ab, w, shape, conv_state, state, ctx, bufs, out, eps)
+
+    def gated_unit(self, x, w, kind, out, scratch):
+        """act(x W_gate^T) * (x W_up^T). bf16: ``w`` interleaved (ops.interleave_gate_up), fp32: ``w`` =
+        [gate | up] rows. ``scratch``: [T, 2 I] of the type of ``x``."""
+        if x.dtype == torch.float32:
+            from ..ops.stream import gated_act_f32
+            return gated_act_f32(self.gemm(x, w, out=scratch), kind, out)
+        return self.gemm_gated(x, w, kind, out=out, scratch=scratch)
+
+    def routed_experts(self, x, logits, w_gate_up, w_down, ws, *, top, correction, groups, keep):
+        """Softmax router over ``logits`` (experts, then identity experts), chosen by score + ``correction``
+        among the ``keep`` best of ``groups`` groups; -> (expert outputs in sorted order, the row of each
+        (token, choice) pair, -1 for identity experts, the weights)."""
+        from ..ops import moe as M
+        ids, w = M.router_topk(logits, top, renorm=False, e_bias=correction, n_group=groups, topk_group=keep,
+                               group_best=1)
+        y = M.clamped_experts(x, ids, None, w_gate_up, w_down, ws)
+        return y, ws.pair_pos[: ids.numel()].view_as(ids), w
 
     def bias_attention(self, q, cache, ctx, group, *, out, **kw):
         """Decode rows first (one token per request), then the prompt portions."""

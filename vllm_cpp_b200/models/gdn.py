@@ -22,6 +22,7 @@ from ..config import ModelConfig, ParallelConfig
 from .base import StepContext, shard_cols, shard_rows
 from .dense import ACT_KIND, DenseModel
 from .moe import MoeModel
+from .recurrent import RecurrentState
 
 
 def _round_up(a, b):
@@ -59,6 +60,7 @@ class Qwen35Model(DenseModel):
             self.shared_inter = c.shared_expert_intermediate_size // self.tp
             self.moe_ws = None
         self.gdn_ws = None
+        self.recurrent = RecurrentState()
         self.conv_state: dict[int, torch.Tensor] = {}
         self.ssm_state: dict[int, torch.Tensor] = {}
 
@@ -301,28 +303,10 @@ class Qwen35Model(DenseModel):
 
     # ---- recurrent state across a speculative step
     def snapshot_state(self, slots: list) -> None:
-        """Saves the convolution and recurrent state of the given request slots. A step that
-        verifies draft tokens advances the state over all of them; when some are rejected there is
-        nothing to subtract, so the runner restores this copy and has the kept tokens run again."""
-        if not slots or not self.gdn_layers:
-            return
-        if not getattr(self, "_snap", None):
-            self._snap = {l: (torch.empty_like(self.conv_state[l]), torch.empty_like(self.ssm_state[l]))
-                          for l in self.gdn_layers}
-        idx = torch.tensor(slots, dtype=torch.long, device=self.device)
-        for l in self.gdn_layers:
-            c, s = self._snap[l]
-            c.index_copy_(0, idx, self.conv_state[l].index_select(0, idx))
-            s.index_copy_(0, idx, self.ssm_state[l].index_select(0, idx))
+        self.recurrent.snapshot(slots)
 
     def restore_state(self, slots: list) -> None:
-        if not slots or not self.gdn_layers:
-            return
-        idx = torch.tensor(slots, dtype=torch.long, device=self.device)
-        for l in self.gdn_layers:
-            c, s = self._snap[l]
-            self.conv_state[l].index_copy_(0, idx, c.index_select(0, idx))
-            self.ssm_state[l].index_copy_(0, idx, s.index_select(0, idx))
+        self.recurrent.restore(slots)
 
     def state_bytes_per_request(self) -> int:
         return len(self.gdn_layers) * (self.conv_dim * 3 * 2 + self.gv * 128 * 128 * 4)
@@ -341,10 +325,10 @@ class Qwen35Model(DenseModel):
         self.bufs.reserve("last", max_reqs, c.hidden_size)
         self.bufs.reserve("logits", max_reqs, self.vocab_shard, torch.float32)
         self.bufs.reserve("argmax_cand", max_reqs, 2, torch.int32)
+        self.recurrent = RecurrentState()
         for l in self.gdn_layers:
-            self.conv_state[l] = torch.zeros((max_reqs, self.conv_dim, 3), dtype=self.dtype, device=self.device)
-            self.ssm_state[l] = torch.zeros((max_reqs, self.gv, 128, 128), dtype=torch.float32,
-                                            device=self.device)
+            self.conv_state[l] = self.recurrent.add((max_reqs, self.conv_dim, 3), self.dtype, self.device)
+            self.ssm_state[l] = self.recurrent.add((max_reqs, self.gv, 128, 128), torch.float32, self.device)
         if self.device.type == "cuda":
             from ..ops.gdn import GdnWorkspace
             self.gdn_ws = GdnWorkspace(self.device, max_tokens, max_reqs, self.gv)

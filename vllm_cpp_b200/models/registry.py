@@ -19,6 +19,7 @@ _REGISTRY.update({
     "Qwen3NextForCausalLM": ("gdn", "Qwen35Model"),
     "OPTForCausalLM": ("opt", "OPTModel"),
     "Nufusun": ("nufusun", "NufusunModel"),
+    "Diforax": ("diforax", "DiforaxModel"),
 })
 
 

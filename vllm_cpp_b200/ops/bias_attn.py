@@ -1,5 +1,6 @@
-"""Attention with a per-head distance bias, heads mixed before the softmax and an optional null
-softmax entry, over pages ``[block_size, kw] keys | [block_size, G * vdim] values``.
+"""Attention over pages ``[block_size, kw] keys | [block_size, G * vdim] values``: grouped heads (each reads
+the key columns of its group) or heads mixed before the softmax, with an optional distance bias, null
+softmax entry and limit to the query's chunk of positions.
 
 The mix of the heads is moved to the query side (``head_mix_kv``): head ``h`` reads the whole key
 row of a token with the query row ``[sum_{g in group 0} M[h, g] q_g | sum_{g in group 1} ... ]``."""
@@ -22,7 +23,7 @@ class BiasAttnArgs(ctypes.Structure):
                 ("tmp_lse", _P), ("tile_req", _P), ("tile_q0", _P),
                 ("max_blocks", _I), ("num_reqs", _I), ("rows", _I), ("H", _I), ("G", _I), ("kw", _I), ("vdim", _I),
                 ("block_size", _I), ("bias_len", _I), ("null_entry", _I), ("f32", _I), ("splits", _I),
-                ("num_tiles", _I)]
+                ("num_tiles", _I), ("grouped", _I), ("chunk", _I), ("scale", ctypes.c_float)]
 
 
 _declared = False
@@ -35,6 +36,7 @@ def _declare():
     P, I, L = _lib.P, _lib.I, ctypes.c_longlong
     A = ctypes.POINTER(BiasAttnArgs)
     _lib.declare("b200_head_mix_kv", [P, L, P, P, L, P, P, I, I, I, I, I, I, I, P], I)
+    _lib.declare("b200_rotate_kv", [P, L, P, P, I, _lib.F, P, L, P, P, I, I, I, I, I, I, I, I, P], I)
     _lib.declare("b200_bias_attn_kernel", [A, I], I)
     _lib.declare("b200_bias_attn_decode", [A, I, P], I)
     _lib.declare("b200_bias_attn_prefill", [A, I, P], I)
@@ -52,7 +54,19 @@ def head_mix_kv(qkv, mix, q_out, slots, cache, *, H, G, dim, vdim, block_size):
                                  int(q_out.dtype == torch.float32), stream_ptr()), "head_mix_kv")
 
 
-def _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry) -> BiasAttnArgs:
+def rotate_kv(qkv, positions, table, rot, eps, q_out, slots, cache, *, H, G, D, V, dim, block_size):
+    """Rows ``[q | k | v]`` (``G`` 0: q alone) -> q and k heads rotated over their first ``rot`` dimensions
+    (pairs half of ``rot`` apart, ``table`` [positions, cos | sin]) and divided by their root mean square
+    over ``dim``; q to ``q_out`` [T, H * D], k and v to ``cache`` (slot < 0: none)."""
+    _declare()
+    assert qkv.dtype == q_out.dtype and (cache is None or cache.dtype == q_out.dtype)
+    check(lib().b200_rotate_kv(ptr(qkv), qkv.stride(0), ptr(positions), ptr(table), rot, eps, ptr(q_out), q_out.stride(0),
+                               ptr(slots), ptr(cache), H, G, D, V, dim, block_size, qkv.shape[0],
+                               int(q_out.dtype == torch.float32), stream_ptr()), "rotate_kv")
+
+
+def _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry, scale, chunk,
+          grouped) -> BiasAttnArgs:
     a = BiasAttnArgs()
     a.q, a.ldq, a.out, a.ldo = ptr(q), q.stride(0), ptr(out), out.stride(0)
     a.cache, a.num_blocks = ptr(cache), cache.shape[0]
@@ -61,14 +75,15 @@ def _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias
     a.rows, a.num_reqs = q.shape[0], q.shape[0]
     a.H, a.G, a.kw, a.vdim, a.block_size = H, G, kw, vdim, block_size
     a.null_entry, a.f32, a.splits = int(null_entry), int(q.dtype == torch.float32), 1
+    a.scale, a.chunk, a.grouped = scale, chunk, int(grouped)
     return a
 
 
 def decode(q, cache, out, *, block_table, seq_lens, H, G, kw, vdim, block_size, bias=None, null_entry=False,
-           splits=1, tmp=None, any_size=False):
+           splits=1, tmp=None, any_size=False, scale=1.0, chunk=0, grouped=False):
     """One query row per request, at its last position."""
     _declare()
-    a = _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry)
+    a = _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry, scale, chunk, grouped)
     if splits > 1:
         if tmp is None:
             tmp = (torch.empty(a.rows * H * splits * vdim, dtype=torch.float32, device=q.device),
@@ -80,22 +95,23 @@ def decode(q, cache, out, *, block_table, seq_lens, H, G, kw, vdim, block_size, 
 
 
 def prefill(q, cache, out, *, block_table, seq_lens, q_start, num_reqs, tile_req, tile_q0, H, G, kw, vdim,
-            block_size, bias=None, null_entry=False, any_size=False):
+            block_size, bias=None, null_entry=False, any_size=False, scale=1.0, chunk=0, grouped=False):
     """Portions of prompts; ``tile_req`` / ``tile_q0`` list their 128-row query tiles."""
     _declare()
-    a = _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry)
+    a = _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry, scale, chunk, grouped)
     a.q_start, a.num_reqs = ptr(q_start), num_reqs
     a.tile_req, a.tile_q0, a.num_tiles = ptr(tile_req), ptr(tile_q0), tile_req.numel()
     check(lib().b200_bias_attn_prefill(ctypes.byref(a), int(any_size), stream_ptr()), "bias_attn_prefill")
     return out
 
 
-def kernel_kind(phase: str, q, cache, *, H, G, kw, vdim, block_size) -> str:
+def kernel_kind(phase: str, q, cache, *, H, G, kw, vdim, block_size, scale=1.0, chunk=0, grouped=False) -> str:
     """Which kernel serves a shape: "tensor-core" or "any-size"."""
     _declare()
     a = BiasAttnArgs()
     a.q, a.ldq, a.out, a.ldo, a.cache = ptr(q), q.stride(0), ptr(q), H * vdim, ptr(cache)
     a.H, a.G, a.kw, a.vdim, a.block_size = H, G, kw, vdim, block_size
+    a.scale, a.chunk, a.grouped = scale, chunk, int(grouped)
     a.f32, a.tile_req = int(q.dtype == torch.float32), ptr(q)
     return {2: "tensor-core", 1: "any-size"}[lib().b200_bias_attn_kernel(ctypes.byref(a), int(phase == "prefill"))]
 
@@ -152,8 +168,26 @@ def ref_head_mix_kv(qkv, mix, q_out, slots, cache, *, H, G, dim, vdim, block_siz
     vals[b, o] = qkv[ok, H * dim + kw: H * dim + kw + vw].to(cache.dtype)
 
 
+def ref_rotate_kv(qkv, positions, table, rot, eps, q_out, slots, cache, *, H, G, D, V, dim, block_size):
+    T, half = qkv.shape[0], rot // 2
+    x = qkv[:, : (H + G) * D].float().view(T, H + G, D).clone()
+    if table is not None:
+        cs = table[positions.long()]
+        c, s = cs[:, None, :half], cs[:, None, half:]
+        u, v = x[..., :half].clone(), x[..., half:rot].clone()
+        x[..., :half], x[..., half:rot] = u * c - v * s, v * c + u * s
+    x = x / torch.sqrt((x * x).sum(-1, keepdim=True) / dim + eps)
+    q_out[:T, : H * D] = x[:, :H].reshape(T, -1).to(q_out.dtype)
+    if G:
+        keys, vals = page_views(cache, block_size, G * D)
+        ok = slots >= 0
+        b, o = slots[ok] // block_size, slots[ok] % block_size
+        keys[b, o] = x[ok, H:].reshape(-1, G * D).to(cache.dtype)
+        vals[b, o] = qkv[ok, (H + G) * D: (H + G) * D + G * V].to(cache.dtype)
+
+
 def ref_bias_attention(q, cache, out, *, block_table, seq_lens, q_start, H, G, kw, vdim, block_size, bias=None,
-                       null_entry=False):
+                       null_entry=False, scale=1.0, chunk=0, grouped=False):
     keys, vals = page_views(cache, block_size, kw)
     qs = q_start.tolist()
     for r, sl in enumerate(seq_lens.tolist()):
@@ -163,11 +197,19 @@ def ref_bias_attention(q, cache, out, *, block_table, seq_lens, q_start, H, G, k
         blocks = block_table[r, : (sl + block_size - 1) // block_size].long()
         k = keys[blocks].reshape(-1, kw)[:sl].float()
         v = vals[blocks].reshape(-1, G, vdim)[:sl].float().repeat_interleave(H // G, 1)
-        s = torch.einsum("qhd,kd->hqk", q[t0:t1, : H * kw].float().view(t1 - t0, H, kw), k)
-        dist = torch.arange(sl - (t1 - t0), sl)[:, None] - torch.arange(sl)[None]
+        if grouped:
+            kg = k.view(sl, G, kw // G).repeat_interleave(H // G, 1)
+            s = torch.einsum("qhd,khd->hqk", q[t0:t1, : H * kw // G].float().view(t1 - t0, H, kw // G), kg) * scale
+        else:
+            s = torch.einsum("qhd,kd->hqk", q[t0:t1, : H * kw].float().view(t1 - t0, H, kw), k) * scale
+        at, key = torch.arange(sl - (t1 - t0), sl)[:, None], torch.arange(sl)[None]
+        dist = at - key
         if bias is not None:
             s = s + bias[:, dist.clamp(0, bias.shape[1] - 1)]
-        s = s.masked_fill(dist < 0, -math.inf)
+        hidden = dist < 0
+        if chunk:
+            hidden = hidden | (at // chunk != key // chunk)
+        s = s.masked_fill(hidden, -math.inf)
         m = s.amax(-1, keepdim=True)
         if null_entry:
             m = m.clamp(min=0)

@@ -26,7 +26,7 @@ def _declare():
     if _declared:
         return
     P, I, F = _lib.P, _lib.I, _lib.F
-    _lib.declare("b200_moe_router_topk", [P, I, I, I, I, I, I, P, I, I, F, P, P, P], I)
+    _lib.declare("b200_moe_router_topk", [P, I, I, I, I, I, I, P, I, I, I, F, P, P, P], I)
     _lib.declare("b200_moe_sort", [P, I, I, I, I, P, P, P, P, P, P, I, P], I)
     _lib.declare("b200_moe_gather", [P, I, P, P, I, P, I, I, P], I)
     _lib.declare("b200_moe_grouped_gemm", [P, I, P, I, I, I, P, P, P, P, P, I, P], I)
@@ -44,15 +44,16 @@ def _declare():
 
 def router_topk(logits: torch.Tensor, k: int, *, renorm: bool = True, scoring: str = "softmax",
                 e_bias: torch.Tensor | None = None, n_group: int = 1, topk_group: int = 1,
-                routed_scale: float = 1.0):
-    """logits: fp32 [T, E] -> (ids int32 [T, k], weights fp32 [T, k])."""
+                routed_scale: float = 1.0, group_best: int | None = None):
+    """logits: fp32 [T, E] -> (ids int32 [T, k], weights fp32 [T, k]). A group's score is the sum of its
+    ``group_best`` best scores (default: two with ``e_bias``, else one)."""
     _declare()
     T, E = logits.shape
     ids = torch.empty((T, k), dtype=torch.int32, device=logits.device)
     w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
     check(lib().b200_moe_router_topk(ptr(logits), logits.stride(0), T, E, k, int(renorm),
                                      0 if scoring == "softmax" else 1, ptr(e_bias), n_group,
-                                     topk_group, routed_scale, ptr(ids), ptr(w), stream_ptr()),
+                                     topk_group, group_best or (1 if e_bias is None else 2), routed_scale, ptr(ids), ptr(w), stream_ptr()),
           "moe_router_topk")
     return ids, w
 
@@ -123,18 +124,20 @@ def grouped_gemm_gated(xs: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Ten
     return out
 
 
-def clamped_experts(x, ids, w, w_gate_up, w_down, ws: MoeWorkspace, *, limit, alpha, up_offset):
+def clamped_experts(x, ids, w, w_gate_up, w_down, ws: MoeWorkspace, *, limit=float("inf"), alpha=1.0, up_offset=0.0):
     """Expert outputs in sorted order, ``ws.y[ws.pair_pos[t * k + j]]`` = W_down a(w_tj W_gate_up x_t)
-    with the clamped pair ``a`` (see :class:`ops.stream.ClampedGate`); the routing weight scales the
-    expert's input. bf16: tcgen05 grouped GEMMs, the weight and the activation in the epilogue of the
+    with the clamped pair ``a`` (see :class:`ops.stream.ClampedGate`; by default SiLU(gate) * up). The
+    routing weight scales the expert's input (``w`` None: not at all); ids past the last matrix have
+    no output, their ``pair_pos`` is -1. bf16: tcgen05 grouped GEMMs, the weight and the activation in the epilogue of the
     first; fp32: fp32 products."""
     T, k = ids.shape
     E, P = w_gate_up.shape[0], T * k
     chunks = min(ws.max_chunks, E + (P + 255) // 256)
     moe_sort(ids, 0, E, ws)
     moe_gather(x, ws, E, P)
-    check(lib().b200_moe_row_weights(ptr(ws.pair_pos), ptr(w), P, ptr(ws.row_w), stream_ptr()), "moe_row_weights")
-    act = ClampedGate(limit, alpha, up_offset, ptr(ws.row_w))
+    if w is not None:
+        check(lib().b200_moe_row_weights(ptr(ws.pair_pos), ptr(w), P, ptr(ws.row_w), stream_ptr()), "moe_row_weights")
+    act = ClampedGate(limit, alpha, up_offset, ptr(ws.row_w) if w is not None else None)
     N, K = w_gate_up.shape[1:]
     args = (ptr(ws.chunk_expert), ptr(ws.chunk_row0), ptr(ws.chunk_n), ptr(ws.meta), chunks)
     if x.dtype == torch.bfloat16:
@@ -175,7 +178,7 @@ def shared_gate(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
 
 # ------------------------------------------------------------------------------ references
 def ref_router_topk(logits, k, renorm=True, scoring="softmax", e_bias=None, n_group=1,
-                    topk_group=1, routed_scale=1.0):
+                    topk_group=1, routed_scale=1.0, group_best=None):
     x = logits.float()
     score = torch.softmax(x, -1) if scoring == "softmax" else torch.sigmoid(x)
     # (plain sigmoid scores are ranked by their logits, which do not tie where fp32 scores round to 1)
@@ -184,7 +187,8 @@ def ref_router_topk(logits, k, renorm=True, scoring="softmax", e_bias=None, n_gr
     T, E = x.shape
     if n_group > 1 and topk_group < n_group:
         g = sel.view(T, n_group, E // n_group)
-        gs = g.topk(2, dim=-1).values.sum(-1) if e_bias is not None else g.max(-1).values
+        best = group_best or (1 if e_bias is None else 2)
+        gs = g.topk(2, dim=-1).values.sum(-1) if best == 2 else g.max(-1).values
         keep = torch.zeros_like(gs, dtype=torch.bool)
         keep.scatter_(1, gs.topk(topk_group, dim=-1).indices, True)
         sel = sel.masked_fill(~keep[:, :, None].expand_as(g).reshape(T, E), float("-inf"))
@@ -203,15 +207,19 @@ def ref_router_topk(logits, k, renorm=True, scoring="softmax", e_bias=None, n_gr
     return ids.int(), w * routed_scale
 
 
-def ref_clamped_experts(x, ids, w, w_gate_up, w_down, *, limit, alpha, up_offset):
+def ref_clamped_experts(x, ids, w, w_gate_up, w_down, *, limit=float("inf"), alpha=1.0, up_offset=0.0):
     """-> outputs [T * k, H] in pair order (token-major), in the type of ``x``."""
     from .stream import ref_clamped_gate
     T, k = ids.shape
     y = torch.zeros((T * k, x.shape[1]), dtype=x.dtype, device=x.device)
-    flat, wt = ids.reshape(-1).long(), w.reshape(-1)
+    flat = ids.reshape(-1).long()
     for e in flat.unique().tolist():
+        if e >= w_gate_up.shape[0]:
+            continue
         rows = (flat == e).nonzero().flatten()
-        gu = (x[rows // k].float() @ w_gate_up[e].float().t()) * wt[rows, None]
+        gu = x[rows // k].float() @ w_gate_up[e].float().t()
+        if w is not None:
+            gu = gu * w.reshape(-1)[rows, None]
         a = ref_clamped_gate(gu, limit, alpha, up_offset).to(x.dtype)
         y[rows] = (a.float() @ w_down[e].float().t()).to(x.dtype)
     return y

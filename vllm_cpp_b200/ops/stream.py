@@ -14,7 +14,8 @@ _P, _L, _I, _F = ctypes.c_void_p, ctypes.c_longlong, ctypes.c_int, ctypes.c_floa
 
 class StreamNormArgs(ctypes.Structure):
     _fields_ = [("stream", _P), ("ids", _P), ("table", _P), ("a", _P), ("y", _P), ("pair_pos", _P), ("pair_w", _P),
-                ("norm_w", _P), ("out", _P), ("lds", _L), ("lda", _L), ("ldy", _L), ("ldo", _L), ("vocab", _L),
+                ("norm_w", _P), ("post_w", _P), ("ident", _P), ("out", _P), ("lds", _L), ("lda", _L), ("ldy", _L),
+                ("ldi", _L), ("ldo", _L), ("vocab", _L),
                 ("T", _I), ("width", _I), ("cols", _I), ("k", _I), ("f32", _I), ("a_f32", _I),
                 ("scale", _F), ("eps", _F), ("norm_offset", _F)]
 
@@ -33,22 +34,25 @@ def _declare():
         return
     P, I = _lib.P, _lib.I
     _lib.declare("b200_stream_norm", [ctypes.POINTER(StreamNormArgs), P], I)
+    _lib.declare("b200_gated_act_f32", [P, I, P, I, I, I, I, P], I)
     _lib.declare("b200_gemm_f32", [P, I, P, I, P, I, P, I, I, I, P], I)
     lib()
     _declared = True
 
 
 def stream_norm(stream, norm_w, eps, out, *, width, ids=None, table=None, scale=1.0, a=None, y=None,
-                pair_pos=None, pair_w=None, norm_offset=1.0):
+                pair_pos=None, pair_w=None, norm_offset=1.0, post_w=None, ident=None):
     """``stream`` [T, cols] fp32 starts as ``table[ids] * scale`` or takes ``+= a + sum_j w_j
-    y[pair_pos[:, j]]``; ``out`` = stream / rms(stream) * (norm_w + norm_offset). ``cols`` is
-    ``width`` padded with zeros."""
+    y[pair_pos[:, j]]`` (``ident`` rows where ``pair_pos`` < 0; may be ``out``), with ``post_w`` that sum
+    over its rms times (post_w + norm_offset); ``out`` = stream / rms(stream) * (norm_w + norm_offset).
+    ``cols`` is ``width`` padded with zeros."""
     _declare()
     T, cols = stream.shape
     s = StreamNormArgs()
     s.stream, s.norm_w, s.out = ptr(stream), ptr(norm_w), ptr(out)
     s.ids, s.table, s.a, s.y = ptr(ids), ptr(table), ptr(a), ptr(y)
     s.pair_pos, s.pair_w = ptr(pair_pos), ptr(pair_w)
+    s.post_w, s.ident, s.ldi = ptr(post_w), ptr(ident), ident.stride(0) if ident is not None else 0
     s.lds, s.ldo = stream.stride(0), out.stride(0)
     s.lda = a.stride(0) if a is not None else 0
     s.ldy = y.stride(0) if y is not None else 0
@@ -73,9 +77,18 @@ def gemm_f32(a, w, bias=None, out=None):
     return out
 
 
+def gated_act_f32(gate_up, kind, out):
+    """act(gate) * up of fp32 rows ``[gate | up]``; ``kind`` as in ``ops.act_and_mul``."""
+    _declare()
+    T, I = gate_up.shape[0], gate_up.shape[1] // 2
+    check(lib().b200_gated_act_f32(ptr(gate_up), gate_up.stride(0), ptr(out), out.stride(0), T, I, kind, stream_ptr()),
+          "gated_act_f32")
+    return out
+
+
 # ------------------------------------------------------------------------------ restatements
 def ref_stream_norm(stream, norm_w, eps, out, *, width, ids=None, table=None, scale=1.0, a=None, y=None,
-                    pair_pos=None, pair_w=None, norm_offset=1.0):
+                    pair_pos=None, pair_w=None, norm_offset=1.0, post_w=None, ident=None):
     if ids is not None:
         stream.copy_(table[ids].float() * scale)
     else:
@@ -85,7 +98,11 @@ def ref_stream_norm(stream, norm_w, eps, out, *, width, ids=None, table=None, sc
         if pair_pos is not None:
             for j in range(pair_pos.shape[1]):
                 yj = y[pair_pos[:, j].long().clamp(min=0)].float() * (pair_pos[:, j] >= 0)[:, None]
+                if ident is not None:
+                    yj = yj + ident.float() * (pair_pos[:, j] < 0)[:, None]
                 d += yj * pair_w[:, j, None] if pair_w is not None else yj
+        if post_w is not None:
+            d = d / torch.sqrt((d * d).sum(-1, keepdim=True) / width + eps) * (post_w + norm_offset)
         stream += d
     inv = 1.0 / torch.sqrt((stream * stream).sum(-1, keepdim=True) / width + eps)
     out.copy_(stream * inv * (norm_w + norm_offset))
