@@ -230,6 +230,7 @@ typedef struct B200Delta {
   const int* tile_q0;
   int nd, num_prefills, num_tiles, T;
   int G, H, D, V, dim, vdim, taps, f32;
+  int split;                   // q and k of the portions as bf16 pairs [hi (D) | lo (D)] instead of fp32
   float eps, q_scale;
 } B200Delta;
 
@@ -318,6 +319,9 @@ int b200_gdn_chunk_scan(const void* q, const void* k, const void* v, long ldv, i
 int b200_delta_prepare(const B200Delta* a, cudaStream_t stream);
 int b200_delta_rule(const B200Delta* a, int reqs, cudaStream_t stream);
 int b200_delta_norm(const B200Delta* a, int rows, cudaStream_t stream);
+// ---- delta_chunk.cu
+int b200_delta_chunk_fits(const B200Delta* a);
+int b200_delta_chunk(const B200Delta* a, void* tp, void* gc, cudaStream_t stream);
 // ---- gemm_bf16.cu
 int b200_gemm_bf16_gated(const void* A, int lda, const void* W, int ldw, void* out, int ldo, int M, int N, int K, int kind, int force_path, cudaStream_t stream);
 int b200_gemm_fp8_pair(const void* A, int lda, const void* W, int ldw, void* out, int ldo, const float* a_scale, const float* w_scale, int w_scale_per_channel, const void* bias, int M, int N, int K, cudaStream_t stream);

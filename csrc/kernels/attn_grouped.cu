@@ -1,5 +1,11 @@
 // Grouped-query attention over the pages of attn_bias.cu ([block_size][G * D] keys | [block_size][G * V]
 // values): query / key preparation and the decode kernel.
+//
+//   rotate_kv_kernel        rotation, unit norm, cache write
+//   grouped_decode_kernel   bf16, one query row per request: a CTA takes one kv group and one split of the
+//                           visible keys, its four warps every fourth tile of 16 keys, each through its own
+//                           ring of cp.async stages (no block barrier before the final merge); the group's
+//                           query heads are the 16 rows of mma.sync, because the kernel is bound by the cache read
 #include "api.h"
 #include "sm100.cuh"
 
@@ -91,8 +97,256 @@ __global__ void __launch_bounds__(128) rotate_kv_kernel(RotateParams p) {
   }
 }
 
-bool grouped_decode_fits(const B200BiasAttn* a) { return false; }
-int grouped_decode(const B200BiasAttn* a, cudaStream_t stream) { return -4; }
+// ---------------------------------------------------------------------------------------------- decode
+struct GroupedDecode {
+  const bf16* q;
+  long long ldq;
+  bf16* out;
+  long long ldo;
+  const bf16* cache;
+  const int32_t* block_table;
+  const int32_t* seq_lens;
+  int max_blocks, H, G, R, D, V, block_size, chunk, splits;
+  float scale2;                // score scale x log2(e)
+  float* tmp_o;                // [B, H, splits, V]
+  float* tmp_lse;              // [B, H, splits], log2
+};
+
+static constexpr int kGWarps = 4, kGKeys = 16, kGStages = 3;
+
+__device__ __forceinline__ void g_ldsm4(uint32_t* r, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void g_ldsm4t(uint32_t* r, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void g_mma(float* d, const uint32_t* a, const uint32_t* b) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+      "{%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+}
+__device__ __forceinline__ void g_cp16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ void g_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void g_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ float g_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+__host__ __device__ inline int g_stage_bytes(int D, int V) { return kGKeys * (D + 8 + V + 8) * 2; }
+
+// ND, NV: bounds of D / 16 and V / 16.
+template <int ND, int NV>
+__global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_decode_kernel(GroupedDecode p) {
+  extern __shared__ uint4 g_smem[];
+  __shared__ float s_m[kGWarps][16], s_l[kGWarps][16];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int b = blockIdx.x, g = blockIdx.y, split = blockIdx.z;
+  const int nd = p.D / 16, nv = p.V / 16, kw = p.G * p.D, vw = p.G * p.V;
+  const int ks = (p.D + 8) * 2, vs = (p.V + 8) * 2, stage = g_stage_bytes(p.D, p.V);
+  const uint32_t ring = smem_u32(g_smem) + warp * kGStages * stage;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int pos = p.seq_lens[b] - 1, lo = p.chunk > 0 && pos > 0 ? pos / p.chunk * p.chunk : 0;
+  // 16-key tiles of this split: a whole number per warp
+  const int first = lo / kGKeys, all = pos < 0 ? 0 : pos / kGKeys + 1 - first;
+  const int per = ((all + p.splits - 1) / p.splits + kGWarps - 1) / kGWarps * kGWarps;
+  const int ta = first + split * per, tb = min(first + all, ta + per);
+  const int n = tb - ta > warp ? (tb - ta - warp + kGWarps - 1) / kGWarps : 0;
+  const int32_t* bt = p.block_table + (size_t)b * p.max_blocks;
+
+  auto load = [&](int i) {                       // tile i of this warp into stage i % kGStages
+    if (i < n) {
+      const int key = (ta + warp + i * kGWarps) * kGKeys;
+      const int page = max(bt[key / p.block_size], 0), off = key % p.block_size;
+      const bf16* k = p.cache + (size_t)page * p.block_size * (kw + vw) + (size_t)off * kw + (size_t)g * p.D;
+      const bf16* v = p.cache + (size_t)page * p.block_size * (kw + vw) + (size_t)p.block_size * kw + (size_t)off * vw + (size_t)g * p.V;
+      const uint32_t dst = ring + (i % kGStages) * stage;
+      const int ku = p.D / 8, vu = p.V / 8;
+      for (int x = lane; x < kGKeys * ku; x += 32) {
+        const int r = x / ku, u = x - r * ku;
+        g_cp16(dst + r * ks + u * 16, k + (size_t)r * kw + u * 8);
+      }
+      for (int x = lane; x < kGKeys * vu; x += 32) {
+        const int r = x / vu, u = x - r * vu;
+        g_cp16(dst + kGKeys * ks + r * vs + u * 16, v + (size_t)r * vw + u * 8);
+      }
+    }
+    g_commit();
+  };
+#pragma unroll
+  for (int i = 0; i + 1 < kGStages; ++i) load(i);
+
+  const int r0 = lane >> 2, c0 = (lane & 3) * 2;
+  uint32_t qa[ND][4];
+#pragma unroll
+  for (int x = 0; x < ND; ++x)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = r0 + (e & 1) * 8, d = x * 16 + c0 + (e >> 1) * 8;
+      qa[x][e] = r < p.R && x < nd ? *reinterpret_cast<const uint32_t*>(p.q + (size_t)b * p.ldq + (size_t)(g * p.R + r) * p.D + d) : 0u;
+    }
+  float o[NV * 2][4];
+#pragma unroll
+  for (int x = 0; x < NV * 2; ++x) o[x][0] = o[x][1] = o[x][2] = o[x][3] = 0.f;
+  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+  const uint32_t k_off = ((lane & 7) + ((lane >> 4) << 3)) * ks + ((lane >> 3) & 1) * 16;
+  const uint32_t v_off = kGKeys * ks + (lane & 15) * vs + (lane >> 4) * 16;
+  for (int i = 0; i < n; ++i) {
+    g_wait<kGStages - 2>();
+    __syncwarp();
+    load(i + kGStages - 1);                      // (into the stage of the tile before)
+    const uint32_t st = ring + (i % kGStages) * stage;
+    float s[2][4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s[0][e] = s[1][e] = 0.f;
+#pragma unroll
+    for (int x = 0; x < ND; ++x) {
+      if (x < nd) {
+        uint32_t kb[4];
+        g_ldsm4(kb, st + k_off + x * 32);
+        g_mma(s[0], qa[x], kb);
+        g_mma(s[1], qa[x], kb + 2);
+      }
+    }
+    const int key = (ta + warp + i * kGWarps) * kGKeys;
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[t][e] *= p.scale2;
+    if (key < lo || key + kGKeys - 1 > pos) {
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int j = key + t * 8 + c0 + e;
+          if (j < lo || j > pos) s[t][e] = s[t][e + 2] = -INFINITY;
+        }
+    }
+    float x0 = fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1]));
+    float x1 = fmaxf(fmaxf(s[0][2], s[0][3]), fmaxf(s[1][2], s[1][3]));
+    x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1));
+    x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1));
+    x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
+    x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
+    // the reference maximum is raised lazily, by more than 2^8
+    const bool up0 = x0 > m0 + 8.f, up1 = x1 > m1 + 8.f;
+    if (__any_sync(0xffffffffu, up0 || up1)) {
+      const float a0 = up0 ? (m0 == -INFINITY ? 0.f : g_ex2(m0 - x0)) : 1.f, a1 = up1 ? (m1 == -INFINITY ? 0.f : g_ex2(m1 - x1)) : 1.f;
+      if (up0) m0 = x0;
+      if (up1) m1 = x1;
+      l0 *= a0;
+      l1 *= a1;
+#pragma unroll
+      for (int x = 0; x < NV * 2; ++x) { o[x][0] *= a0; o[x][1] *= a0; o[x][2] *= a1; o[x][3] *= a1; }
+    }
+#pragma unroll
+    for (int t = 0; t < 2; ++t) {
+      s[t][0] = g_ex2(s[t][0] - m0); s[t][1] = g_ex2(s[t][1] - m0);
+      s[t][2] = g_ex2(s[t][2] - m1); s[t][3] = g_ex2(s[t][3] - m1);
+      l0 += s[t][0] + s[t][1];
+      l1 += s[t][2] + s[t][3];
+    }
+    const uint32_t pa[4] = {pack_bf16x2(s[0][0], s[0][1]), pack_bf16x2(s[0][2], s[0][3]), pack_bf16x2(s[1][0], s[1][1]),
+                            pack_bf16x2(s[1][2], s[1][3])};
+#pragma unroll
+    for (int x = 0; x < NV; ++x) {
+      if (x < nv) {
+        uint32_t vb[4];
+        g_ldsm4t(vb, st + v_off + x * 32);
+        g_mma(o[2 * x], pa, vb);
+        g_mma(o[2 * x + 1], pa, vb + 2);
+      }
+    }
+  }
+  g_wait<0>();
+  l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
+  l0 += __shfl_xor_sync(0xffffffffu, l0, 2); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+  if ((lane & 3) == 0) {
+    s_m[warp][r0] = m0; s_m[warp][r0 + 8] = m1;
+    s_l[warp][r0] = l0; s_l[warp][r0 + 8] = l1;
+  }
+  __syncthreads();                               // (every ring is drained: its memory takes the partial sums)
+  float* so = reinterpret_cast<float*>(g_smem);  // [warp][16][V]
+  float t0 = -INFINITY, t1 = -INFINITY;
+#pragma unroll
+  for (int w = 0; w < kGWarps; ++w) { t0 = fmaxf(t0, s_m[w][r0]); t1 = fmaxf(t1, s_m[w][r0 + 8]); }
+  const float f0 = m0 == -INFINITY ? 0.f : g_ex2(m0 - t0), f1 = m1 == -INFINITY ? 0.f : g_ex2(m1 - t1);
+#pragma unroll
+  for (int x = 0; x < NV * 2; ++x) {
+    if (x < 2 * nv) {
+      float* d = so + (size_t)(warp * 16 + r0) * p.V + x * 8 + c0;
+      *reinterpret_cast<float2*>(d) = make_float2(o[x][0] * f0, o[x][1] * f0);
+      *reinterpret_cast<float2*>(d + 8 * p.V) = make_float2(o[x][2] * f1, o[x][3] * f1);
+    }
+  }
+  __syncthreads();
+  for (int i = tid; i < p.R * p.V / 2; i += kGWarps * 32) {
+    const int r = i * 2 / p.V, c = i * 2 - r * p.V;
+    float mx = -INFINITY, l = 0.f;
+#pragma unroll
+    for (int w = 0; w < kGWarps; ++w) mx = fmaxf(mx, s_m[w][r]);
+    float2 y = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int w = 0; w < kGWarps; ++w) {
+      if (s_m[w][r] != -INFINITY) l += s_l[w][r] * g_ex2(s_m[w][r] - mx);
+      const float2 v = *reinterpret_cast<const float2*>(so + (size_t)(w * 16 + r) * p.V + c);
+      y.x += v.x;
+      y.y += v.y;
+    }
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+    const size_t h = (size_t)g * p.R + r;
+    if (p.splits == 1) {
+      *reinterpret_cast<uint32_t*>(p.out + (size_t)b * p.ldo + h * p.V + c) = pack_bf16x2(y.x * inv, y.y * inv);
+    } else {
+      const size_t at = ((size_t)b * p.H + h) * p.splits + split;
+      *reinterpret_cast<float2*>(p.tmp_o + at * p.V + c) = make_float2(y.x * inv, y.y * inv);
+      if (c == 0) p.tmp_lse[at] = l > 0.f ? mx + log2f(l) : -INFINITY;
+    }
+  }
+}
+
+bool grouped_decode_fits(const B200BiasAttn* a) {
+  if (!a->grouped || a->f32 || a->bias || a->null_entry || a->kw % a->G) return false;
+  const int D = a->kw / a->G, V = a->vdim;
+  return !(D & 15) && !(V & 15) && D <= 256 && V <= 256 && a->H / a->G <= 16 && a->block_size % kGKeys == 0 &&
+         !(((uintptr_t)a->q | (uintptr_t)a->cache) & 15) && !(a->ldq & 7) && !(a->ldo & 1) && a->scale > 0.f;
+}
+
+template <int ND, int NV>
+static int launch_grouped(const GroupedDecode& p, int rows, cudaStream_t stream) {
+  size_t smem = (size_t)kGWarps * kGStages * g_stage_bytes(p.D, p.V);
+  const size_t merge = (size_t)kGWarps * 16 * p.V * 4;
+  if (smem < merge) smem = merge;
+  static PerDeviceOnce once;
+  if (once.first()) cudaFuncSetAttribute(grouped_decode_kernel<ND, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+  return launch_pdl(grouped_decode_kernel<ND, NV>, dim3(rows, p.G, p.splits), dim3(kGWarps * 32), smem, stream, p) ==
+                 cudaSuccess ? 0 : -2;
+}
+template <int ND>
+static int launch_grouped(const GroupedDecode& p, int rows, cudaStream_t stream) {
+  return p.V <= 64 ? launch_grouped<ND, 4>(p, rows, stream) : p.V <= 128 ? launch_grouped<ND, 8>(p, rows, stream)
+                                                                          : launch_grouped<ND, 16>(p, rows, stream);
+}
+
+int grouped_decode(const B200BiasAttn* a, cudaStream_t stream) {
+  GroupedDecode p{(const bf16*)a->q, a->ldq, (bf16*)a->out, a->ldo, (const bf16*)a->cache, (const int32_t*)a->block_table,
+                  (const int32_t*)a->seq_lens, a->max_blocks, a->H, a->G, a->H / a->G, a->kw / a->G, a->vdim, a->block_size,
+                  a->chunk, a->splits < 1 ? 1 : a->splits, a->scale * 1.4426950408889634f, (float*)a->tmp_o,
+                  (float*)a->tmp_lse};
+  if (p.splits > 1 && (!p.tmp_o || !p.tmp_lse)) return -1;
+  if (p.G > 65535 || p.splits > 65535) return -4;
+  const int rc = p.D <= 64 ? launch_grouped<4>(p, a->rows, stream) : p.D <= 128 ? launch_grouped<8>(p, a->rows, stream)
+                                                                                : launch_grouped<16>(p, a->rows, stream);
+  if (rc || p.splits == 1) return rc;
+  return b200_attn_decode_merge(p.tmp_o, p.tmp_lse, p.out, (int)p.ldo, a->rows, p.H, p.V, p.splits, stream);
+}
 
 }  // namespace b200
 

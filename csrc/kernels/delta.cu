@@ -146,8 +146,19 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(B200Delta p) {
       if (sec < p.G) inv *= p.q_scale;
       float* d = (sec < p.G ? p.q + (t * p.G + sec) * p.D : p.k + (t * p.G + sec - p.G) * p.D);
 #pragma unroll
-      for (int i = 0; i < NI; ++i)
-        if (i * 128 + lane * 4 < width) *reinterpret_cast<float4*>(d + i * 128 + lane * 4) = mul4(inv, y[i]);
+      for (int i = 0; i < NI; ++i) {
+        const int c = i * 128 + lane * 4;
+        if (c >= width) continue;
+        const float4 x = mul4(inv, y[i]);
+        if (p.split && (int)blockIdx.x >= p.nd) {        // x = hi + lo
+          bf16* b = reinterpret_cast<bf16*>(d) + c;
+          Ld4<bf16>::put(b, x);
+          const float4 hi = Ld4<bf16>::get(b);
+          Ld4<bf16>::put(b + p.D, make_float4(x.x - hi.x, x.y - hi.y, x.z - hi.z, x.w - hi.w));
+        } else {
+          *reinterpret_cast<float4*>(d + c) = x;
+        }
+      }
     }
   }
   if (at == 0) {
@@ -217,18 +228,23 @@ __global__ void __launch_bounds__(THREADS) delta_rule_kernel(B200Delta p, int sl
       sk[i] = p.k[((size_t)t * p.G + kv) * p.D + i];
       sq[i] = p.q[((size_t)t * p.G + kv) * p.D + i];
     }
-    const float decay = expf(p.g[(size_t)t * p.H + h]), beta = p.beta[(size_t)t * p.H + h];
+    const float lg = p.g[(size_t)t * p.H + h], beta = p.beta[(size_t)t * p.H + h];
+    // A factor near one, applied over thousands of tokens, must not be rounded to fp32 first: its
+    // distance from one is what is multiplied and added.
+    const bool slow = lg > -0.5f;
+    const float keep = slow ? 1.f : 0.f, rest = slow ? expm1f(lg) : expf(lg);
+    auto decayed = [&](float4 x) { return fma4(rest, x, mul4(keep, x)); };
     __syncthreads();
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
     if (MAXR) {
 #pragma unroll
       for (int r = 0; r < MAXR; ++r)
         if (r < nr) {
-          s[r] = mul4(decay, s[r]);
+          s[r] = decayed(s[r]);
           a = fma4(sk[r0 + r], s[r], a);
         }
     } else {
-      for (int r = 0; r < nr; ++r) a = fma4(sk[r0 + r], mul4(decay, S[(size_t)r * nv]), a);
+      for (int r = 0; r < nr; ++r) a = fma4(sk[r0 + r], decayed(S[(size_t)r * nv]), a);
     }
     if (on) red0[sl * nv + v4] = a;
     __syncthreads();
@@ -249,7 +265,7 @@ __global__ void __launch_bounds__(THREADS) delta_rule_kernel(B200Delta p, int sl
           }
       } else {
         for (int r = 0; r < nr; ++r) {
-          const float4 x = fma4(sk[r0 + r], u, mul4(decay, S[(size_t)r * nv]));
+          const float4 x = fma4(sk[r0 + r], u, decayed(S[(size_t)r * nv]));
           S[(size_t)r * nv] = x;
           a = fma4(sq[r0 + r], x, a);
         }

@@ -18,6 +18,7 @@ from __future__ import annotations
 import torch
 
 from ..config import DenseSpec, ExpertSpec, ModelConfig, ParallelConfig
+from ..ops.bias_attn import grouped_decode_splits
 from ..ops.delta import DeltaShape
 from .backend import make_backend
 from .base import BufferPool, StepContext
@@ -70,6 +71,7 @@ class DiforaxModel(DenseModel):
         self.kv_layers = [l for l, b in enumerate(cfg.blocks) if b.attention is not None and b.attention.kv_from is None]
         self.bufs = BufferPool(self.device)
         self.moe_ws: dict = {}
+        self.chunks = None                    # scratch of the chunked delta rule
         self.recurrent = RecurrentState()
         self.state: dict[int, tuple] = {}
         self.rope: dict[tuple, torch.Tensor] = {}
@@ -169,7 +171,7 @@ class DiforaxModel(DenseModel):
             if isinstance(f, DenseSpec):
                 ff = self._ff_padded(f.ff)
                 gate, up = (put(p["mlp." + n], ff, C) for n in ("gate", "up"))
-                if self._interleaved():
+                if self._bf16_kernels():
                     from ..ops import interleave_gate_up
                     L["gate_up"] = interleave_gate_up(gate, up).contiguous()
                 else:
@@ -182,12 +184,12 @@ class DiforaxModel(DenseModel):
             if k not in self.w:
                 raise ValueError(f"{k} is missing from the checkpoint")
 
-    def _interleaved(self) -> bool:
+    def _bf16_kernels(self) -> bool:
         return self.device.type == "cuda" and self.dtype == torch.bfloat16
 
     def _ff_padded(self, ff: int) -> int:
         """(the gated product takes gate and up rows in blocks of 128)"""
-        return _pad(ff, 128 if self._interleaved() else 8)
+        return _pad(ff, 128 if self._bf16_kernels() else 8)
 
     @staticmethod
     def _tensor_names(b) -> set:
@@ -279,7 +281,17 @@ class DiforaxModel(DenseModel):
 
     def decode_workspace(self, batch: int, max_seq_len: int, block_size: int):
         """(KV splits, split buffers) of a decode batch; one pair of buffers serves every block."""
-        return 1, None
+        att = [b.attention for b in self.cfg.blocks if b.attention is not None]
+        if self.device.type != "cuda" or not att:
+            return 1, None
+        from .. import ops
+        keys = max(min(a.chunk or max_seq_len, max_seq_len) for a in att)
+        s = grouped_decode_splits(batch, min(a.kv_heads for a in att), keys, ops.num_sms())
+        if s == 1:
+            return 1, None
+        heads, out = max(a.heads for a in att), max(a.heads * _pad(a.vdim, 16) for a in att)
+        return s, (torch.empty(batch * s * out, dtype=torch.float32, device=self.device),
+                   torch.empty(batch * s * heads, dtype=torch.float32, device=self.device))
 
     # ------------------------------------------------------------------ buffers
     def _delta_buffers(self, s: DeltaShape, T: int):
@@ -289,6 +301,7 @@ class DiforaxModel(DenseModel):
         sizes = {"q": (s.G * s.D, f32), "k": (s.G * s.D, f32), "v": (s.H * s.V, self.dtype), "g": (s.H, f32),
                  "beta": (s.H, f32), "o": (s.H * s.V, f32)}
         bufs = {n: self.bufs.get(f"delta_{n}{w}", T, w, t) for n, (w, t) in sizes.items()}
+        bufs["chunks"] = self.chunks
         return proj, ab, bufs, self.bufs.get(f"heads{s.H * s.V}", T, s.H * s.V, self.dtype)
 
     def _attention_buffers(self, a, T: int):
@@ -308,6 +321,10 @@ class DiforaxModel(DenseModel):
         self.bufs.reserve("last", max_reqs, self.cols, self.dtype)
         self.bufs.reserve("logits", max_reqs, _pad(self.cfg.vocab_size), torch.float32)
         self.recurrent = RecurrentState()
+        heads = max([self.cfg.blocks[l].delta.heads for l in self.delta_layers], default=0)
+        if heads and self._bf16_kernels():
+            from ..ops.delta import chunk_workspace
+            self.chunks = chunk_workspace(self.device, (max_tokens + 127) // 128 + max_reqs, heads)
         for l, b in enumerate(self.cfg.blocks):
             f = b.mlp
             if b.delta is not None:

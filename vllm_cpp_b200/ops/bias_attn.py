@@ -122,6 +122,11 @@ def decode_splits(batch: int, max_seq_len: int, num_sms: int) -> int:
     return max(1, min(num_sms // max(1, batch), -(-max_seq_len // 128), 32))
 
 
+def grouped_decode_splits(batch: int, groups: int, max_keys: int, num_sms: int) -> int:
+    """KV splits of a grouped decode batch: one wave of two CTAs per SM, no split below 128 keys."""
+    return max(1, min(2 * num_sms // max(1, batch * groups), -(-max_keys // 128), 32))
+
+
 # ------------------------------------------------------------------------- tables built at load time
 def bucket_of_distance(n: int, num_buckets: int, max_distance: int) -> int:
     """Distances below half the table have a bucket each; beyond, buckets are spaced evenly in the

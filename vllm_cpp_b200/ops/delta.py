@@ -42,7 +42,7 @@ class DeltaArgs(ctypes.Structure):
                 ("norm_w", _P), ("conv_state", _P), ("state", _P), ("q", _P), ("k", _P), ("v", _P), ("g", _P),
                 ("beta", _P), ("o", _P), ("out", _P), ("ldo", _L), ("seq_lens", _P), ("slots", _P), ("q_start", _P),
                 ("tile_req", _P), ("tile_q0", _P), ("nd", _I), ("num_prefills", _I), ("num_tiles", _I), ("T", _I),
-                ("G", _I), ("H", _I), ("D", _I), ("V", _I), ("dim", _I), ("vdim", _I), ("taps", _I), ("f32", _I),
+                ("G", _I), ("H", _I), ("D", _I), ("V", _I), ("dim", _I), ("vdim", _I), ("taps", _I), ("f32", _I), ("split", _I),
                 ("eps", _F), ("q_scale", _F)]
 
 
@@ -57,6 +57,8 @@ def _declare():
     _lib.declare("b200_delta_prepare", [A, _P], _I)
     _lib.declare("b200_delta_rule", [A, _I, _P], _I)
     _lib.declare("b200_delta_norm", [A, _I, _P], _I)
+    _lib.declare("b200_delta_chunk_fits", [A], _I)
+    _lib.declare("b200_delta_chunk", [A, _P, _P, _P], _I)
     lib()
     _declared = True
 
@@ -65,7 +67,9 @@ def delta_mixer(proj, ab, w, shape: DeltaShape, conv_state, state, rows, bufs, o
     """``proj`` [T, columns] and ``ab`` fp32 [T, >= 2 H] -> ``out`` [T, H * V]. ``w``: conv_w fp32
     [taps, channels], A, dt, norm fp32. ``conv_state`` [slots, taps - 1, channels] and ``state`` fp32
     [slots, H, D, V] are advanced; a request's first rows start from zero. ``rows``: the step's
-    :class:`StepContext`. ``bufs``: q, k, v, g, beta, o scratch of T rows."""
+    :class:`StepContext`. ``bufs``: q, k, v, g, beta, o scratch of T rows, and for prompts ``chunks``
+    (see :func:`chunk_workspace`). bf16 prompts run in chunks of 64 tokens on the tensor cores;
+    ``token_by_token``, fp32 and sizes beyond them walk the tokens."""
     _declare()
     a = DeltaArgs()
     s, es = shape, proj.element_size()
@@ -81,9 +85,26 @@ def delta_mixer(proj, ab, w, shape: DeltaShape, conv_state, state, rows, bufs, o
     a.nd, a.num_prefills, a.num_tiles, a.T = rows.num_decodes, rows.num_prefills, rows.num_tiles, proj.shape[0]
     a.G, a.H, a.D, a.V, a.dim, a.vdim, a.taps = s.G, s.H, s.D, s.V, s.dim, s.vdim, s.taps
     a.f32, a.eps, a.q_scale = int(proj.dtype == torch.float32), eps, s.dim ** -0.5
+    chunks = bufs.get("chunks")
+    a.split = int(chunks is not None and a.num_prefills > 0 and not token_by_token
+                  and lib().b200_delta_chunk_fits(ctypes.byref(a)))
     check(lib().b200_delta_prepare(ctypes.byref(a), stream_ptr()), "delta_prepare")
-    check(lib().b200_delta_rule(ctypes.byref(a), a.nd + a.num_prefills, stream_ptr()), "delta_rule")
+    check(lib().b200_delta_rule(ctypes.byref(a), a.nd + (0 if a.split else a.num_prefills), stream_ptr()), "delta_rule")
+    if a.split:
+        tp, gc = chunks
+        assert tp.numel() >= a.num_tiles * s.H * CHUNK_VALUES and gc.numel() >= a.num_tiles * s.H * 128
+        check(lib().b200_delta_chunk(ctypes.byref(a), ptr(tp), ptr(gc), stream_ptr()), "delta_chunk")
+        check(lib().b200_delta_norm(ctypes.byref(a), a.T - a.nd, stream_ptr()), "delta_norm")
     return out
+
+
+CHUNK_VALUES = 2 * 4 * 64 * 64          # bf16 values per 128-row tile and head
+
+
+def chunk_workspace(device, max_tiles: int, heads: int):
+    """Scratch of the chunk kernels: (pair matrices, decay sums) for up to ``max_tiles`` 128-row tiles."""
+    return (torch.empty(max_tiles * heads * CHUNK_VALUES, dtype=torch.bfloat16, device=device),
+            torch.empty(max_tiles * heads * 128, dtype=torch.float32, device=device))
 
 
 # ------------------------------------------------------------------------------ restatements
