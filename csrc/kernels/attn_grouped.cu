@@ -161,6 +161,10 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
   const int n = tb - ta > warp ? (tb - ta - warp + kGWarps - 1) / kGWarps : 0;
   const int32_t* bt = p.block_table + (size_t)b * p.max_blocks;
 
+  // 16-byte unit u of row r of a tile, this lane's first and the step to its next (32 units on)
+  const int ku = p.D / 8, vu = p.V / 8;
+  const int kr0 = lane / ku, ku0 = lane - kr0 * ku, krs = 32 / ku, kus = 32 - krs * ku;
+  const int vr0 = lane / vu, vu0 = lane - vr0 * vu, vrs = 32 / vu, vus = 32 - vrs * vu;
   auto load = [&](int i) {                       // tile i of this warp into stage i % kGStages
     if (i < n) {
       const int key = (ta + warp + i * kGWarps) * kGKeys;
@@ -168,14 +172,17 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
       const bf16* k = p.cache + (size_t)page * p.block_size * (kw + vw) + (size_t)off * kw + (size_t)g * p.D;
       const bf16* v = p.cache + (size_t)page * p.block_size * (kw + vw) + (size_t)p.block_size * kw + (size_t)off * vw + (size_t)g * p.V;
       const uint32_t dst = ring + (i % kGStages) * stage;
-      const int ku = p.D / 8, vu = p.V / 8;
-      for (int x = lane; x < kGKeys * ku; x += 32) {
-        const int r = x / ku, u = x - r * ku;
-        g_cp16(dst + r * ks + u * 16, k + (size_t)r * kw + u * 8);
+      for (int r = kr0, u = ku0; r < kGKeys;) {
+        g_cp16(dst + r * ks + u * 16, k + r * kw + u * 8);
+        r += krs;
+        u += kus;
+        if (u >= ku) { u -= ku; ++r; }
       }
-      for (int x = lane; x < kGKeys * vu; x += 32) {
-        const int r = x / vu, u = x - r * vu;
-        g_cp16(dst + kGKeys * ks + r * vs + u * 16, v + (size_t)r * vw + u * 8);
+      for (int r = vr0, u = vu0; r < kGKeys;) {
+        g_cp16(dst + kGKeys * ks + r * vs + u * 16, v + r * vw + u * 8);
+        r += vrs;
+        u += vus;
+        if (u >= vu) { u -= vu; ++r; }
       }
     }
     g_commit();
@@ -203,18 +210,20 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
     __syncwarp();
     load(i + kGStages - 1);                      // (into the stage of the tile before)
     const uint32_t st = ring + (i % kGStages) * stage;
-    float s[2][4];
+    float s[2][4], z[2][4];                      // (two sums each, to halve the chains of products)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) s[0][e] = s[1][e] = 0.f;
+    for (int e = 0; e < 4; ++e) s[0][e] = s[1][e] = z[0][e] = z[1][e] = 0.f;
 #pragma unroll
     for (int x = 0; x < ND; ++x) {
       if (x < nd) {
         uint32_t kb[4];
         g_ldsm4(kb, st + k_off + x * 32);
-        g_mma(s[0], qa[x], kb);
-        g_mma(s[1], qa[x], kb + 2);
+        g_mma(x & 1 ? z[0] : s[0], qa[x], kb);
+        g_mma(x & 1 ? z[1] : s[1], qa[x], kb + 2);
       }
     }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { s[0][e] += z[0][e]; s[1][e] += z[1][e]; }
     const int key = (ta + warp + i * kGWarps) * kGKeys;
 #pragma unroll
     for (int t = 0; t < 2; ++t)
@@ -312,6 +321,71 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
   }
 }
 
+// Heads of up to 128 values whose half rotation is a multiple of four: a lane holds four values, the partner's
+// come by shuffle; a warp takes kRotItems (token, head) pairs, loads first.
+static constexpr int kRotItems = 4;
+template <typename T>
+__global__ void __launch_bounds__(128) rotate_kv_vec_kernel(RotateParams p) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int lane = threadIdx.x & 31, heads = p.H + 2 * p.G, c = lane * 4, kw = p.G * p.D, vw = p.G * p.V;
+  const long long x0 = ((long long)blockIdx.x * 4 + (threadIdx.x >> 5)) * kRotItems, total = (long long)p.T * heads;
+  int t = (int)(x0 / heads), h = (int)(x0 - (long long)t * heads);
+  float4 v[kRotItems], cs[kRotItems], sn[kRotItems];
+  T* dst[kRotItems];
+  bool turn[kRotItems];
+  const int half = p.rot / 2;
+  const bool low = c < half, in_rot = p.cos_sin && c < p.rot;
+#pragma unroll
+  for (int i = 0; i < kRotItems; ++i) {
+    v[i] = cs[i] = sn[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    dst[i] = nullptr;
+    turn[i] = h < p.H + p.G;
+    if (x0 + i < total) {
+      const T* row = reinterpret_cast<const T*>(p.qkv) + (size_t)t * p.ld;
+      const int width = turn[i] ? p.D : p.V;
+      const int64_t slot = h < p.H ? 0 : p.slots[t];
+      if (slot >= 0 && c < width) {
+        v[i] = load4<T>(row + (turn[i] ? (size_t)h * p.D : (size_t)(p.H + p.G) * p.D + (size_t)(h - p.H - p.G) * p.V) + c);
+        if (h < p.H) {
+          dst[i] = reinterpret_cast<T*>(p.q_out) + (size_t)t * p.ldq + (size_t)h * p.D + c;
+        } else {
+          const int64_t page = slot / p.block_size, off = slot - page * p.block_size;
+          T* base = reinterpret_cast<T*>(p.cache) + page * p.block_size * (int64_t)(kw + vw);
+          dst[i] = turn[i] ? base + off * kw + (int64_t)(h - p.H) * p.D + c
+                           : base + (int64_t)p.block_size * kw + off * vw + (int64_t)(h - p.H - p.G) * p.V + c;
+        }
+        if (turn[i] && in_rot) {
+          const float* f = p.cos_sin + (size_t)p.positions[t] * p.rot + (low ? c : c - half);
+          cs[i] = *reinterpret_cast<const float4*>(f);
+          sn[i] = *reinterpret_cast<const float4*>(f + half);
+        }
+      }
+    }
+    if (++h == heads) { h = 0; ++t; }
+  }
+  const int partner = in_rot ? (low ? lane + half / 4 : lane - half / 4) : lane;
+#pragma unroll
+  for (int i = 0; i < kRotItems; ++i) {
+    float4 o;
+    o.x = __shfl_sync(0xffffffffu, v[i].x, partner);
+    o.y = __shfl_sync(0xffffffffu, v[i].y, partner);
+    o.z = __shfl_sync(0xffffffffu, v[i].z, partner);
+    o.w = __shfl_sync(0xffffffffu, v[i].w, partner);
+    float4 y = v[i];
+    if (turn[i] && in_rot) {
+      const float g = low ? -1.f : 1.f;
+      y = make_float4(y.x * cs[i].x + g * o.x * sn[i].x, y.y * cs[i].y + g * o.y * sn[i].y,
+                      y.z * cs[i].z + g * o.z * sn[i].z, y.w * cs[i].w + g * o.w * sn[i].w);
+    }
+    float ss = y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
+#pragma unroll
+    for (int k = 16; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+    const float inv = turn[i] ? 1.f / sqrtf(ss / (float)p.dim + p.eps) : 1.f;
+    if (dst[i]) store4(dst[i], make_float4(y.x * inv, y.y * inv, y.z * inv, y.w * inv));
+  }
+}
+
 bool grouped_decode_fits(const B200BiasAttn* a) {
   if (!a->grouped || a->f32 || a->bias || a->null_entry || a->kw % a->G) return false;
   const int D = a->kw / a->G, V = a->vdim;
@@ -363,6 +437,11 @@ int b200_rotate_kv(const void* qkv, long long ld, const void* positions, const v
     return -1;
   RotateParams p{qkv, ld, (const int64_t*)positions, (const float*)cos_sin, q_out, ldq, (const int64_t*)slots, cache,
                  rot, H, G, D, V, dim, block_size, T, eps};
+  if (D <= 128 && (!G || V <= 128) && (!cos_sin || !(rot & 7))) {
+    const dim3 vgrid((unsigned)(((long long)T * (H + 2 * G) + 4 * kRotItems - 1) / (4 * kRotItems)));
+    return (f32 ? launch_pdl(rotate_kv_vec_kernel<float>, vgrid, dim3(128), 0, stream, p)
+                : launch_pdl(rotate_kv_vec_kernel<bf16>, vgrid, dim3(128), 0, stream, p)) == cudaSuccess ? 0 : -2;
+  }
   const dim3 grid((unsigned)(((long long)T * (H + 2 * G) + 3) / 4));
   const size_t smem = (size_t)4 * D * 4;
   return (f32 ? launch_pdl(rotate_kv_kernel<float>, grid, dim3(128), smem, stream, p)

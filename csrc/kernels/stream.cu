@@ -26,6 +26,8 @@ template <> struct Vec4<__nv_bfloat16> {
 };
 __device__ __forceinline__ void add4(float4& x, float4 y) { x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w; }
 
+static constexpr int kMaxPairs = 128;    // expert outputs per row
+
 // One CTA per row; a thread keeps its four-value groups in registers between the two passes
 // (kRegs groups), wider rows are read again from the stream.
 template <typename T>
@@ -42,7 +44,16 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(B200StreamNorm p, int*
     if (id >= 0 && id < p.vocab) src = reinterpret_cast<const T*>(p.table) + (size_t)id * p.cols;
     else if (threadIdx.x == 0 && status) atomicExch(status, (int)kErrBadArg);
   }
-  const int32_t* pos = reinterpret_cast<const int32_t*>(p.pair_pos) + (size_t)t * p.k;
+  // the row's pairs; ident rows (or nothing) stand for y where there is no expert output
+  __shared__ const T* s_y[kMaxPairs];
+  __shared__ float s_w[kMaxPairs];
+  for (int x = threadIdx.x; x < p.k; x += blockDim.x) {
+    const int32_t at = reinterpret_cast<const int32_t*>(p.pair_pos)[(size_t)t * p.k + x];
+    s_y[x] = at >= 0 ? reinterpret_cast<const T*>(p.y) + (size_t)at * p.ldy
+                               : p.ident ? reinterpret_cast<const T*>(p.ident) + (size_t)t * p.ldi : nullptr;
+    s_w[x] = p.pair_w ? p.pair_w[(size_t)t * p.k + x] : 1.f;
+  }
+  if (p.k > 0) __syncthreads();
   float4 keep[kRegs];
   auto row_sum = [&](float ss) {
 #pragma unroll
@@ -66,15 +77,17 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(B200StreamNorm p, int*
       if (p.a_f32) add4(v, Vec4<float>::load(reinterpret_cast<const float*>(p.a) + (size_t)t * p.lda + i * 4));
       else add4(v, Vec4<T>::load(reinterpret_cast<const T*>(p.a) + (size_t)t * p.lda + i * 4));
     }
-    for (int j = 0; j < p.k; ++j) {
-      if (pos[j] < 0 && !p.ident) continue;
-      float4 y = pos[j] < 0 ? Vec4<T>::load(reinterpret_cast<const T*>(p.ident) + (size_t)t * p.ldi + i * 4)
-                            : Vec4<T>::load(reinterpret_cast<const T*>(p.y) + (size_t)pos[j] * p.ldy + i * 4);
-      if (p.pair_w) {
-        const float w = p.pair_w[(size_t)t * p.k + j];
-        y.x *= w; y.y *= w; y.z *= w; y.w *= w;
-      }
-      add4(v, y);
+    for (int j = 0; j < p.k; j += 4) {     // (four loads on the way at a time)
+      float4 y[4];
+#pragma unroll
+      for (int x = 0; x < 4; ++x)
+        y[x] = j + x < p.k && s_y[j + x] ? Vec4<T>::load(s_y[j + x] + i * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int x = 0; x < 4; ++x)
+        if (j + x < p.k) {
+          const float w = s_w[j + x];
+          v.x = fmaf(w, y[x].x, v.x); v.y = fmaf(w, y[x].y, v.y); v.z = fmaf(w, y[x].z, v.z); v.w = fmaf(w, y[x].w, v.w);
+        }
     }
     return v;
   };
@@ -241,6 +254,7 @@ int b200_stream_norm(const B200StreamNorm* a, cudaStream_t stream) {
   if (!a->stream || !a->out || !a->norm_w || a->width <= 0 || a->cols < a->width || (a->cols & 7) || a->k < 0) return -1;
   if ((a->lds & 3) || (a->lda & 3) || (a->ldy & 3) || (a->ldi & 3) || (a->ldo & 3) || (a->ids && !a->table)) return -1;
   if (a->k > 0 && (!a->pair_pos || !a->y)) return -1;
+  if (a->k > kMaxPairs) return -4;
   int threads = ((a->cols / 4 + 31) / 32) * 32;
   if (threads > 256) threads = 256;
   int* st = device_status_word();

@@ -3,7 +3,6 @@ implementation in ``nufusun_reference.py``; every test runs on the CPU back end 
 on the kernels."""
 import json
 import os
-import random
 import subprocess
 import sys
 
@@ -12,6 +11,7 @@ import torch
 
 import nufusun_case as C
 import nufusun_reference as R
+from replay import Replay, engine, greedy, random_steps, rel, tokens
 
 sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
@@ -21,11 +21,6 @@ both = pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 device = pytest.mark.parametrize("dev", DEVICES)
 CLOSE_CALL = 0.05       # router margin below which rounding to bf16 may change the chosen experts
 _logits: dict = {}
-
-
-def tokens(n, vocab, seed):
-    return [random.Random(seed).randrange(vocab) for _ in range(n)] if n < 2 else \
-        [random.Random(seed * 1000003 + i).randrange(vocab) for i in range(n)]
 
 
 def oracle(name, toks, seed=0):
@@ -61,42 +56,6 @@ def folder(tmp_path_factory):
             done[name, seed] = C.write(base / f"{name}{seed}", *C.case(name, seed))
         return done[name, seed]
     return get
-
-
-def rel(got, want):
-    """Row-wise error of the logits with their mean taken off."""
-    d = got.double() - want
-    d = d - d.mean(-1, keepdim=True)
-    w = want - want.mean(-1, keepdim=True)
-    return (d.norm(dim=-1) / w.norm(dim=-1)).max().item()
-
-
-class Replay:
-    """Steps of (request, count) pairs through the engine; collects the logits of every position."""
-
-    def __init__(self, model, dtype, dev, max_tokens, page=8, max_requests=4):
-        from vllm_cpp_b200.entrypoints.trace import TraceReplay
-        self.r = TraceReplay(model, dtype, max_tokens, dev, max_requests=max_requests, page=page)
-
-    def run(self, prompts, steps):
-        at, got = {}, {}
-        for step in steps:
-            entries, end = [], []
-            for rid, n in step:
-                lo = at.get(rid, 0)
-                entries.append({"id": rid, "tokens": prompts[rid][lo:lo + n], "want": list(range(n))})
-                at[rid] = lo + n
-                if at[rid] == len(prompts[rid]):
-                    end.append(rid)
-            rows = self.r.step(entries, end)
-            for e in entries:
-                got.setdefault(e["id"], []).extend(rows[:len(e["tokens"])])
-                rows = rows[len(e["tokens"]):]
-        assert all(len(v) == at[k] for k, v in got.items())
-        return {k: torch.stack(v) for k, v in got.items()}
-
-    def free_pages(self):
-        return self.r.llm.core.scheduler().num_free_blocks()
 
 
 # ------------------------------------------------------------------------------ one sequence
@@ -221,20 +180,7 @@ def test_mixed_batches(folder, name, dtype, dev):
     """Portions beside single tokens, requests that pause, unequal lengths."""
     vocab = C.CASES[name][0]["vocab"]
     prompts = {r: tokens(n, vocab, 20 + i) for i, (r, n) in enumerate([("a", 90), ("b", 17), ("c", 41), ("d", 3)])}
-    left = {r: len(p) for r, p in prompts.items()}
-    rnd, steps = random.Random(5), []
-    while left:
-        step = []
-        for r in list(left):
-            if rnd.random() < 0.25:
-                continue
-            n = min(left[r], rnd.choice([1, 1, 1, 2, 5, 16]))
-            step.append((r, n))
-            left[r] -= n
-            if not left[r]:
-                del left[r]
-        if step:
-            steps.append(step)
+    steps = random_steps({r: len(p) for r, p in prompts.items()}, 5)
     got = Replay(folder(name), dtype, dev, 176).run(prompts, steps)
     for r, p in prompts.items():
         agrees(got[r], name, p, dtype)
@@ -269,19 +215,6 @@ def test_pages_and_slots_are_used_again(folder, dtype, dev):
 
 
 # ------------------------------------------------------------------------------ generation
-def engine(model, dtype, dev, **kw):
-    from vllm_cpp_b200.config import EngineArgs
-    from vllm_cpp_b200.engine import LLM
-    args = dict(model=model, dtype=dtype, device=dev, block_size=8, num_blocks=80, max_model_len=256, max_num_seqs=4,
-                max_num_batched_tokens=64)
-    return LLM(EngineArgs(**{**args, **kw}))
-
-
-def greedy(n, **kw):
-    from vllm_cpp_b200.engine import SamplingParams
-    return SamplingParams(temperature=0.0, max_tokens=n, ignore_eos=True, **kw)
-
-
 def check_greedy(name, prompt, out, margin):
     """Every generated token is the oracle's choice, or within ``margin`` of it (with a bf16-sized
     margin: except where the choice of experts is a close call)."""

@@ -1,8 +1,9 @@
-"""Throughput of the Nufusun design beside the closest other model of this package (Qwen3-MoE) at equal
-layer sizes, and its kernels beside the like kernels of that model, each against its roofline.
+"""Throughput of a design with listed layers beside the closest other model of this package at equal layer
+sizes, and its kernels beside the like kernels of that model, each against its roofline.
 
-``bench.py --design nufusun`` runs it and prints one JSON line. Random weights; device time (CUDA
-events); kernels are timed with an L2 flush between iterations, median of several."""
+``bench.py --design nufusun`` (beside Qwen3-MoE) or ``--design diforax`` (beside the Qwen3.5 MoE hybrids) runs
+it and prints one JSON line. Random weights; device time (CUDA events); kernels are timed with an L2 flush
+between iterations, median of several."""
 from __future__ import annotations
 
 import json
@@ -11,7 +12,8 @@ import os
 import torch
 
 # name -> width, heads, kv heads, head size, experts, top, expert size, layers
-SIZES = {
+FIELDS = ("width", "heads", "kv_heads", "head", "experts", "top", "expert", "layers")
+NUFUSUN_SIZES = {
     "30b-a3b layers": (2048, 32, 4, 128, 128, 8, 768, 4),
     "small layers": (1024, 16, 4, 64, 32, 4, 512, 6),
     "8 kv heads": (2048, 32, 8, 64, 64, 4, 1024, 4),
@@ -19,7 +21,37 @@ SIZES = {
 }
 
 
-def configs(size):
+# name -> those, then delta value heads, delta key heads (of 128 x 128)
+DIFORAX_SIZES = {
+    "30b-a3b layers": (2048, 32, 4, 128, 128, 8, 768, 4, 32, 16),
+    "wide heads": (2048, 16, 2, 256, 64, 4, 1024, 4, 32, 16),
+    "small layers": (1024, 16, 4, 128, 32, 4, 512, 8, 16, 8),
+    "wide layers": (4096, 32, 8, 128, 16, 2, 2048, 4, 48, 16),
+}
+
+
+def diforax_configs(size):
+    """Three delta blocks to one attention block; chunks longer than the prompts, as the other model's
+    attention has no limit; an eighth as many identity experts, which the other model does not have."""
+    from ..config import AttentionSpec, BlockSpec, DeltaSpec, ExpertSpec, ModelConfig, RopeConfig, model_config_of_blocks
+    W, H, G, D, E, top, ff, layers, dh, dk = size
+    moe = ExpertSpec(experts=E, top=top, ff=ff, identity=E // 8, groups=4, keep=2)
+    att = AttentionSpec(heads=H, kv_heads=G, dim=D, vdim=D, scale=D ** -0.5, rot_dims=D, rot_base=1e6, chunk=1 << 15)
+    delta = BlockSpec(None, moe, DeltaSpec(heads=dh, kv_heads=dk, dim=128, vdim=128, conv=4))
+    blocks = [BlockSpec(att, moe) if l % 4 == 3 else delta for l in range(layers)]
+    mine = model_config_of_blocks("Diforax", blocks, vocab=32000, width=W, eps=1e-6)
+    other = ModelConfig(architecture="Qwen3_5MoeForConditionalGeneration", vocab_size=32000, hidden_size=W,
+                        intermediate_size=3 * W, num_layers=layers, num_heads=H, num_kv_heads=G, head_dim=D,
+                        max_position_embeddings=32768, qk_norm=True, gemma_norm=True, attn_output_gate=True,
+                        rope=RopeConfig(theta=1e6), layer_types=["full_attention" if l % 4 == 3 else "linear_attention"
+                                                                 for l in range(layers)],
+                        linear_num_key_heads=dk, linear_num_value_heads=dh, linear_key_head_dim=128,
+                        linear_value_head_dim=128, linear_conv_kernel_dim=4, num_experts=E, num_experts_per_tok=top,
+                        moe_intermediate_size=ff, norm_topk_prob=True)
+    return {"diforax": mine, "qwen3.5-moe": other}
+
+
+def nufusun_configs(size):
     from ..config import AttentionSpec, BlockSpec, ExpertSpec, ModelConfig, RopeConfig, model_config_of_blocks
     W, H, G, D, E, top, ff, layers = size
     block = BlockSpec(AttentionSpec(heads=H, kv_heads=G, dim=D, vdim=D, scale=D ** -0.5, bias_max=1024),
@@ -86,7 +118,7 @@ def _peaks():
 
 class KernelBench:
     def __init__(self, size):
-        self.W, self.H, self.G, self.D, self.E, self.top, self.ff, _ = size
+        self.W, self.H, self.G, self.D, self.E, self.top, self.ff = size[:7]
         self.dev = torch.device("cuda")
         self.hbm, self.tflops, _ = _peaks()
         self.flush = torch.empty(256 << 20, dtype=torch.uint8, device=self.dev)
@@ -114,6 +146,14 @@ class KernelBench:
 
     def i32(self, x):
         return torch.tensor(x, dtype=torch.int32, device=self.dev)
+
+
+class NufusunKernels(KernelBench):
+    def run(self):
+        self.attention(B=4, prompt=2048, decode_batch=64, ctx=4096)
+        self.attention(B=8, prompt=1024, decode_batch=8, ctx=16384)
+        for T in (64, 8192):
+            self.rest(T)
 
     def attention(self, B, prompt, decode_batch, ctx, bs=32):
         from .. import ops
@@ -216,15 +256,200 @@ class KernelBench:
                  note="two kernels")
 
 
-def run(sizes=None, kernels=True) -> dict:
+class DiforaxKernels(KernelBench):
+    def __init__(self, size):
+        super().__init__(size)
+        self.dh, self.dk = size[8:]
+
+    def run(self):
+        self.attention(B=4, prompt=2048, decode_batch=64, ctx=4096)
+        self.attention(B=8, prompt=1024, decode_batch=8, ctx=16384)
+        self.delta(B=4, n=2048)
+        self.delta(B=8, n=1024)
+        self.delta(B=1, n=8192)
+        for B in (16, 64, 256):
+            self.delta(B=B, n=1)
+        for T in (64, 8192):
+            self.rest(T)
+
+    def attention(self, B, prompt, decode_batch, ctx, bs=32):
+        from .. import ops
+        from ..ops import bias_attn as A
+        from ..ops.reference import build_prefill_tiles
+        H, G, D, kw = self.H, self.G, self.D, self.G * self.D
+        shape = dict(H=H, G=G, kw=kw, vdim=D, block_size=bs, grouped=True)
+        nb, T = prompt // bs, B * prompt
+        bt = torch.arange(1, B * nb + 1, device=self.dev, dtype=torch.int32).view(B, nb)
+        sl, qs = self.i32([prompt] * B), self.i32([i * prompt for i in range(B + 1)])
+        tr, tq = (self.i32(x) for x in build_prefill_tiles([prompt] * B))
+        q, pages = self.rnd(T, H * D), self.rnd(B * nb + 1, bs * 2 * kw)
+        kv, out = self.rnd(B * nb + 1, 2, bs, G, D), torch.empty(T, H * D, dtype=torch.bfloat16, device=self.dev)
+        for chunk in (0, 512):
+            n, last = divmod(prompt, chunk or prompt)
+            size = chunk or prompt
+            pairs = B * (n * size * (size + 1) / 2 + last * (last + 1) / 2)
+            self.add(f"attention, {B} x {prompt} prompt" + (f", chunks of {chunk}" if chunk else ""), "diforax",
+                     lambda: A.prefill(q, pages, out, block_table=bt, seq_lens=sl, q_start=qs, num_reqs=B, tile_req=tr,
+                                       tile_q0=tq, scale=D ** -0.5, chunk=chunk, **shape), flops=2 * pairs * H * 2 * D,
+                     note=A.kernel_kind("prefill", q, pages, scale=D ** -0.5, chunk=chunk, **shape))
+            self.add(f"attention, {B} x {prompt} prompt" + (f", chunks of {chunk}" if chunk else ""), "qwen3.5-moe",
+                     lambda: ops.attn_prefill(q, kv, block_table=bt, seq_lens=sl, q_start=qs, tile_req=tr, tile_q0=tq,
+                                              num_q_heads=H, num_kv_heads=G, head_dim=D, block_size=bs, scale=D ** -0.5,
+                                              window=-chunk, out=out), flops=2 * pairs * H * 2 * D)
+        qkv, pos = self.rnd(T, (H + 2 * G) * D), torch.arange(T, device=self.dev) % prompt
+        slots = (bt.long()[:, :, None] * bs + torch.arange(bs, device=self.dev)).reshape(-1)
+        table, nw = self.rnd(prompt, D, dtype=torch.float32), self.rnd(D)
+        nbytes = T * 2 * (H + 2 * G) * D * 2
+        self.add(f"query preparation + cache write, {T} tokens", "diforax",
+                 lambda: A.rotate_kv(qkv, pos, table, D, 1e-6, q, slots, pages, H=H, G=G, D=D, V=D, dim=D, block_size=bs),
+                 nbytes=nbytes)
+        self.add(f"query preparation + cache write, {T} tokens", "qwen3.5-moe",
+                 lambda: ops.rope_kv(qkv, pos, table, num_q_heads=H, num_kv_heads=G, head_dim=D, q_norm=nw, k_norm=nw,
+                                     slot_mapping=slots, kv_cache=kv, block_size=bs, q_out=q), nbytes=nbytes)
+        B, nb = decode_batch, ctx // bs
+        bt = torch.arange(1, B * nb + 1, device=self.dev, dtype=torch.int32).view(B, nb)
+        sl = self.i32([ctx] * B)
+        pages, kv, q = self.rnd(B * nb + 1, bs * 2 * kw), self.rnd(B * nb + 1, 2, bs, G, D), self.rnd(B, H * D)
+        out = torch.empty(B, H * D, dtype=torch.bfloat16, device=self.dev)
+        splits = A.grouped_decode_splits(B, G, ctx, ops.num_sms())
+        tmp = (torch.empty(B * H * splits * D, dtype=torch.float32, device=self.dev),
+               torch.empty(B * H * splits, dtype=torch.float32, device=self.dev))
+        nbytes = B * ctx * 2 * kw * 2
+        self.add(f"attention, decode {B} x {ctx}", "diforax",
+                 lambda: A.decode(q, pages, out, block_table=bt, seq_lens=sl, splits=splits, tmp=tmp, scale=D ** -0.5,
+                                  **shape), nbytes=nbytes, note=A.kernel_kind("decode", q, pages, scale=D ** -0.5, **shape))
+        self.add(f"attention, decode {B} x {ctx}", "qwen3.5-moe",
+                 lambda: ops.attn_decode(q, kv, block_table=bt, seq_lens=sl, num_q_heads=H, num_kv_heads=G, head_dim=D,
+                                         block_size=bs, scale=D ** -0.5, out=out), nbytes=nbytes)
+
+    def delta(self, B, n):
+        """``B`` prompts of ``n`` tokens, or (n 1) a decode batch: preparation, then recurrence with norm and gate."""
+        import ctypes
+        from types import SimpleNamespace
+        from ..ops import delta as X
+        from ..ops import gdn as Q
+        from ..ops.reference import build_prefill_tiles
+        G, H, D, T = self.dk, self.dh, 128, B * n
+        s = X.DeltaShape(G=G, H=H, D=D, V=D, dim=D, vdim=D, taps=4)
+        f32 = dict(dtype=torch.float32)
+        proj, ab = self.rnd(T, s.columns), self.rnd(T, 2 * H, **f32)
+        w = {"conv_w": self.rnd(4, s.channels, **f32), "A": self.rnd(H, **f32).abs(), "dt": self.rnd(H, **f32),
+             "norm": self.rnd(D, **f32)}
+        conv, state = self.rnd(B, 3, s.channels), torch.zeros(B, H, D, D, device=self.dev)
+        tr, tq = build_prefill_tiles([n] * B) if n > 1 else ([], [])
+        rows = SimpleNamespace(seq_lens=self.i32([n + 5] * B), state_slots=self.i32(list(range(B))),
+                               prefill_q_start=self.i32([i * n for i in range(B + 1)]), tile_req=self.i32(tr or [0]),
+                               tile_q0=self.i32(tq or [0]), num_decodes=B if n == 1 else 0, num_prefills=0 if n == 1 else B,
+                               num_tiles=len(tr))
+        bufs = {"q": self.rnd(T, G, D, **f32), "k": self.rnd(T, G, D, **f32), "v": self.rnd(T, H, D), "g": self.rnd(T, H, **f32),
+                "beta": self.rnd(T, H, **f32), "o": self.rnd(T, H, D, **f32), "chunks": X.chunk_workspace(self.dev, len(tr) + 1, H)}
+        out = torch.empty(T, H * D, dtype=torch.bfloat16, device=self.dev)
+        a = X.delta_args(proj, ab, w, s, conv, state, rows, bufs, out, 1e-6)
+        what = f"{B} x {n} prompt" if n > 1 else f"decode {B}"
+        prep = T * (2 * s.channels * 2 + 2 * H * 4)
+        step = T * (2 * G * D + 3 * H * D) * 2 + B * H * D * D * 4 * 2
+        flops = T * H * (6.0 * D * D + 4 * 64 * D) if n > 1 else 0
+        self.add(f"delta preparation, {what}", "diforax", lambda: X.run_prepare(a), nbytes=prep)
+        self.add(f"delta rule + gated norm, {what}", "diforax", lambda: X.run_rule(a, bufs), nbytes=step, flops=flops,
+                 note="state, q and k in 32 bits")
+        # the other model's kernels
+        cw, cst = w["conv_w"].t().contiguous().to(torch.bfloat16), self.rnd(B, s.channels, 3)
+        xc, st2 = self.rnd(T, s.channels), torch.zeros(B, H, D, D, device=self.dev)
+        mixed, z = proj[:, : s.channels], proj[:, s.channels:]
+        abb, slots, core = ab.to(torch.bfloat16), rows.state_slots, torch.empty_like(out)
+        a2, b2, nw = abb[:, :H], abb[:, H:], w["norm"].to(torch.bfloat16)
+        if n == 1:
+            self.add(f"delta preparation, {what}", "qwen3.5-moe", lambda: Q.conv1d_update(mixed, cw, cst, slots, xc), nbytes=prep,
+                     note="convolution only")
+
+            def theirs():
+                Q.packed_decode(xc, a2, b2, w["A"], w["dt"], st2, slots, core.view(T, H, D), G, H)
+                Q.rmsnorm_gated(core, z, nw, core, heads=H)
+        else:
+            q, k = self.rnd(T, G, D), self.rnd(T, G, D)
+            g, beta, init = self.rnd(T, H, **f32), self.rnd(T, H, **f32).abs(), self.i32([1] * B)
+            ws, qsl = Q.GdnWorkspace(self.dev, T, B, H), rows.prefill_q_start
+            host = [i * n for i in range(B + 1)]
+            t0, ln, s0 = Q.build_chunk_table(host)
+            table = (self.i32(t0.tolist()), self.i32(ln.tolist()), self.i32(s0.tolist()))
+
+            def theirs_prep():
+                Q.conv1d_fwd(mixed, cw, cst, qsl, slots, init, xc)
+                Q.post_conv(xc, G, H, a2, b2, w["A"], w["dt"], q, k, g, beta)
+            self.add(f"delta preparation, {what}", "qwen3.5-moe", theirs_prep, nbytes=prep)
+
+            def theirs():
+                Q.chunk_scan(q, k, xc, g, beta, st2, host, slots, init, core.view(T, H, D), ws, v_col0=2 * G * D, table=table)
+                Q.rmsnorm_gated(core, z, nw, core, heads=H)
+        self.add(f"delta rule + gated norm, {what}", "qwen3.5-moe", theirs, nbytes=step, flops=flops)
+
+    def rest(self, T):
+        import ctypes
+        from .. import ops
+        from ..ops import moe as M
+        from ..ops.stream import stream_norm
+        W, E, top, ff = self.W, self.E, self.top, self.ff
+        P, I = T * top, E // 8
+        ws = M.MoeWorkspace(self.dev, T, top, E, W, ff)
+        x, wgu, wd = self.rnd(T, W), self.rnd(E, 2 * ff, W, s=0.05), self.rnd(E, W, ff, s=0.05)
+        logits, corr = self.rnd(T, E + I, dtype=torch.float32), self.rnd(E + I, dtype=torch.float32, s=0.01)
+        choose = lambda: M.router_topk(logits, top, renorm=False, e_bias=corr, n_group=4, topk_group=2, group_best=1)  # noqa: E731
+        self.add(f"router, {T} tokens", "diforax", choose, nbytes=T * ((E + I) * 4 + top * 8))
+        plain = logits[:, :E].contiguous()
+        self.add(f"router, {T} tokens", "qwen3.5-moe", lambda: M.router_topk(plain, top), nbytes=T * (E * 4 + top * 8))
+        for who, (ids, w) in (("diforax", choose()), ("qwen3.5-moe", M.router_topk(plain, top))):
+            real = ids < E
+            used, pairs = int(ids[real].unique().numel()), int(real.sum())
+            chunks = min(ws.max_chunks, E + (P + 255) // 256)
+            M.moe_sort(ids, 0, E, ws)
+            M.moe_gather(x, ws, E, P)
+            nbytes, fl = used * 2 * ff * W * 2 + pairs * (W + ff) * 2, 2.0 * pairs * 2 * ff * W
+            if who == "diforax":
+                act = M.ClampedGate(float("inf"), 1.0, 0.0, None)
+                args = (M.ptr(ws.chunk_expert), M.ptr(ws.chunk_row0), M.ptr(ws.chunk_n), M.ptr(ws.meta), chunks)
+                fn = lambda: M.check(M.lib().b200_moe_grouped_gemm_clamped(M.ptr(ws.xs), P, M.ptr(wgu), E, 2 * ff, W,  # noqa: E731
+                                                                           M.ptr(ws.act), *args, ctypes.byref(act), M.stream_ptr()), "gemm")
+            else:
+                fn = lambda: M.grouped_gemm_gated(ws.xs, wgu, ws.act, ws, P, chunks)                    # noqa: E731
+            self.add(f"gated expert products, {T} tokens", who, fn, nbytes=nbytes, flops=fl)
+            self.add(f"down expert products, {T} tokens", who, lambda: M.grouped_gemm(ws.act, wd, ws.y, ws, P, chunks),
+                     nbytes=used * ff * W * 2 + pairs * (W + ff) * 2, flops=fl / 2)
+            out, stream = torch.empty_like(x), self.rnd(T, W, dtype=torch.float32)
+            nw = self.rnd(W, dtype=torch.float32)
+            if who == "diforax":
+                pos = ws.pair_pos[:P].view(T, top)
+                self.add(f"expert sum + norms + residual, {T} tokens", who,
+                         lambda: stream_norm(stream, nw, 1e-6, out, width=W, y=ws.y, pair_pos=pos, pair_w=w, post_w=nw, ident=out,
+                                             norm_offset=0.0), nbytes=T * W * (4 + 4 + 2 * top + 2), note="a norm more")
+                mixed = self.rnd(T, W, dtype=torch.float32)
+                self.add(f"norms + residual, {T} tokens", who,
+                         lambda: stream_norm(stream, nw, 1e-6, out, width=W, a=mixed, post_w=nw, norm_offset=0.0),
+                         nbytes=T * W * (4 + 4 + 4 + 2), note="a norm more")
+                continue
+            o2, res, nwb = torch.empty_like(x), self.rnd(T, W), nw.to(torch.bfloat16)
+
+            def two():
+                M.combine(ws.y, ws, w, o2)
+                ops.rmsnorm(o2, nwb, 1e-6, residual=res, out=out)
+            self.add(f"expert sum + norms + residual, {T} tokens", who, two, nbytes=T * W * 2 * (top + 1 + 1 + 2 + 1), note="two kernels")
+            self.add(f"norms + residual, {T} tokens", who, lambda: ops.rmsnorm(o2, nwb, 1e-6, residual=res, out=out),
+                     nbytes=T * W * 2 * 4)
+
+
+DESIGNS = {"nufusun": (NUFUSUN_SIZES, nufusun_configs, NufusunKernels), "diforax": (DIFORAX_SIZES, diforax_configs, DiforaxKernels)}
+
+
+def run(design="nufusun", sizes=None, kernels=True) -> dict:
+    table, configs, bench = DESIGNS[design]
     hbm, tf, how = _peaks()
-    res = {"metric": "design_layer_throughput", "unit": "tok/s", "impl": "ours", "dtype": "bf16",
+    res = {"metric": "design_layer_throughput", "unit": "tok/s", "impl": "ours", "design": design, "dtype": "bf16",
            "data": "synthetic (uniform-random prompt ids, random-init weights)",
            "roofline": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": how}, "models": {}, "kernels": {}}
-    for name, size in SIZES.items():
+    names = FIELDS + (("delta_heads", "delta_key_heads") if design == "diforax" else ())
+    for name, size in table.items():
         if sizes and name not in sizes:
             continue
-        res["models"][name] = {"layers": dict(zip(("width", "heads", "kv_heads", "head", "experts", "top", "expert", "layers"), size))}
+        res["models"][name] = {"layers": dict(zip(names, size))}
         for prompt, batch in ((1024, 64), (4096, 16)):
             r = {}
             for who, cfg in configs(size).items():
@@ -232,11 +457,8 @@ def run(sizes=None, kernels=True) -> dict:
                 torch.cuda.empty_cache()
             res["models"][name][f"prompt {prompt}, decode batch {batch}"] = r
         if kernels:
-            k = KernelBench(size)
-            k.attention(B=4, prompt=2048, decode_batch=64, ctx=4096)
-            k.attention(B=8, prompt=1024, decode_batch=8, ctx=16384)
-            for T in (64, 8192):
-                k.rest(T)
+            k = bench(size)
+            k.run()
             res["kernels"][name] = k.rows
             del k
             torch.cuda.empty_cache()

@@ -63,17 +63,10 @@ def _declare():
     _declared = True
 
 
-def delta_mixer(proj, ab, w, shape: DeltaShape, conv_state, state, rows, bufs, out, eps, *, token_by_token=False):
-    """``proj`` [T, columns] and ``ab`` fp32 [T, >= 2 H] -> ``out`` [T, H * V]. ``w``: conv_w fp32
-    [taps, channels], A, dt, norm fp32. ``conv_state`` [slots, taps - 1, channels] and ``state`` fp32
-    [slots, H, D, V] are advanced; a request's first rows start from zero. ``rows``: the step's
-    :class:`StepContext`. ``bufs``: q, k, v, g, beta, o scratch of T rows, and for prompts ``chunks``
-    (see :func:`chunk_workspace`). bf16 prompts run in chunks of 64 tokens on the tensor cores;
-    ``token_by_token``, fp32 and sizes beyond them walk the tokens."""
+def delta_args(proj, ab, w, shape: DeltaShape, conv_state, state, rows, bufs, out, eps, *, token_by_token=False) -> DeltaArgs:
     _declare()
-    a = DeltaArgs()
-    s, es = shape, proj.element_size()
-    a.proj, a.ldp, a.gate = ptr(proj), proj.stride(0), ptr(proj) + s.channels * es
+    a, s = DeltaArgs(), shape
+    a.proj, a.ldp, a.gate = ptr(proj), proj.stride(0), ptr(proj) + s.channels * proj.element_size()
     a.ab, a.ldab = ptr(ab), ab.stride(0)
     a.conv_w, a.A, a.dt, a.norm_w = ptr(w["conv_w"]), ptr(w["A"]), ptr(w["dt"]), ptr(w["norm"])
     a.conv_state, a.state = ptr(conv_state), ptr(state)
@@ -85,16 +78,34 @@ def delta_mixer(proj, ab, w, shape: DeltaShape, conv_state, state, rows, bufs, o
     a.nd, a.num_prefills, a.num_tiles, a.T = rows.num_decodes, rows.num_prefills, rows.num_tiles, proj.shape[0]
     a.G, a.H, a.D, a.V, a.dim, a.vdim, a.taps = s.G, s.H, s.D, s.V, s.dim, s.vdim, s.taps
     a.f32, a.eps, a.q_scale = int(proj.dtype == torch.float32), eps, s.dim ** -0.5
-    chunks = bufs.get("chunks")
-    a.split = int(chunks is not None and a.num_prefills > 0 and not token_by_token
+    a.split = int(bufs.get("chunks") is not None and a.num_prefills > 0 and not token_by_token
                   and lib().b200_delta_chunk_fits(ctypes.byref(a)))
+    return a
+
+
+def run_prepare(a: DeltaArgs) -> None:
     check(lib().b200_delta_prepare(ctypes.byref(a), stream_ptr()), "delta_prepare")
+
+
+def run_rule(a: DeltaArgs, bufs) -> None:
     check(lib().b200_delta_rule(ctypes.byref(a), a.nd + (0 if a.split else a.num_prefills), stream_ptr()), "delta_rule")
     if a.split:
-        tp, gc = chunks
-        assert tp.numel() >= a.num_tiles * s.H * CHUNK_VALUES and gc.numel() >= a.num_tiles * s.H * 128
+        tp, gc = bufs["chunks"]
+        assert tp.numel() >= a.num_tiles * a.H * CHUNK_VALUES and gc.numel() >= a.num_tiles * a.H * 128
         check(lib().b200_delta_chunk(ctypes.byref(a), ptr(tp), ptr(gc), stream_ptr()), "delta_chunk")
         check(lib().b200_delta_norm(ctypes.byref(a), a.T - a.nd, stream_ptr()), "delta_norm")
+
+
+def delta_mixer(proj, ab, w, shape: DeltaShape, conv_state, state, rows, bufs, out, eps, *, token_by_token=False):
+    """``proj`` [T, columns] and ``ab`` fp32 [T, >= 2 H] -> ``out`` [T, H * V]. ``w``: conv_w fp32
+    [taps, channels], A, dt, norm fp32. ``conv_state`` [slots, taps - 1, channels] and ``state`` fp32
+    [slots, H, D, V] are advanced; a request's first rows start from zero. ``rows``: the step's
+    :class:`StepContext`. ``bufs``: q, k, v, g, beta, o scratch of T rows, and for prompts ``chunks``
+    (see :func:`chunk_workspace`). bf16 prompts run in chunks of 64 tokens on the tensor cores;
+    ``token_by_token``, fp32 and sizes beyond them walk the tokens."""
+    a = delta_args(proj, ab, w, shape, conv_state, state, rows, bufs, out, eps, token_by_token=token_by_token)
+    run_prepare(a)
+    run_rule(a, bufs)
     return out
 
 
