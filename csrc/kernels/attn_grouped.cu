@@ -329,8 +329,8 @@ __global__ void __launch_bounds__(128) rotate_kv_vec_kernel(RotateParams p) {
   pdl_wait();
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31, heads = p.H + 2 * p.G, c = lane * 4, kw = p.G * p.D, vw = p.G * p.V;
-  const long long x0 = ((long long)blockIdx.x * 4 + (threadIdx.x >> 5)) * kRotItems, total = (long long)p.T * heads;
-  int t = (int)(x0 / heads), h = (int)(x0 - (long long)t * heads);
+  const int x0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * kRotItems, total = p.T * heads;   // (below 2^31: checked)
+  int t = x0 / heads, h = x0 - t * heads;
   float4 v[kRotItems], cs[kRotItems], sn[kRotItems];
   T* dst[kRotItems];
   bool turn[kRotItems];
@@ -350,8 +350,8 @@ __global__ void __launch_bounds__(128) rotate_kv_vec_kernel(RotateParams p) {
         if (h < p.H) {
           dst[i] = reinterpret_cast<T*>(p.q_out) + (size_t)t * p.ldq + (size_t)h * p.D + c;
         } else {
-          const int64_t page = slot / p.block_size, off = slot - page * p.block_size;
-          T* base = reinterpret_cast<T*>(p.cache) + page * p.block_size * (int64_t)(kw + vw);
+          const uint32_t page = (uint32_t)slot / (uint32_t)p.block_size, off = (uint32_t)slot - page * p.block_size;
+          T* base = reinterpret_cast<T*>(p.cache) + page * (p.block_size * (int64_t)(kw + vw));
           dst[i] = turn[i] ? base + off * kw + (int64_t)(h - p.H) * p.D + c
                            : base + (int64_t)p.block_size * kw + off * vw + (int64_t)(h - p.H - p.G) * p.V + c;
         }
@@ -437,7 +437,7 @@ int b200_rotate_kv(const void* qkv, long long ld, const void* positions, const v
     return -1;
   RotateParams p{qkv, ld, (const int64_t*)positions, (const float*)cos_sin, q_out, ldq, (const int64_t*)slots, cache,
                  rot, H, G, D, V, dim, block_size, T, eps};
-  if (D <= 128 && (!G || V <= 128) && (!cos_sin || !(rot & 7))) {
+  if (D <= 128 && (!G || V <= 128) && (!cos_sin || !(rot & 7)) && (long long)T * (H + 2 * G) < (1ll << 31) - 64) {
     const dim3 vgrid((unsigned)(((long long)T * (H + 2 * G) + 4 * kRotItems - 1) / (4 * kRotItems)));
     return (f32 ? launch_pdl(rotate_kv_vec_kernel<float>, vgrid, dim3(128), 0, stream, p)
                 : launch_pdl(rotate_kv_vec_kernel<bf16>, vgrid, dim3(128), 0, stream, p)) == cudaSuccess ? 0 : -2;

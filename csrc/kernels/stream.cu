@@ -30,9 +30,8 @@ static constexpr int kMaxPairs = 128;    // expert outputs per row
 
 // One CTA per row; a thread keeps its four-value groups in registers between the two passes
 // (kRegs groups), wider rows are read again from the stream.
-template <typename T>
+template <typename T, int kRegs>
 __global__ void __launch_bounds__(256) stream_norm_kernel(B200StreamNorm p, int* status) {
-  constexpr int kRegs = 4;
   __shared__ float red[8];
   pdl_wait();
   pdl_launch_dependents();
@@ -54,7 +53,12 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(B200StreamNorm p, int*
     s_w[x] = p.pair_w ? p.pair_w[(size_t)t * p.k + x] : 1.f;
   }
   if (p.k > 0) __syncthreads();
-  float4 keep[kRegs];
+  float4 keep[kRegs], old[kRegs];        // update, then new stream; old stream (asked for ahead of the sums)
+#pragma unroll
+  for (int c = 0; c < kRegs; ++c) {
+    const int i = threadIdx.x + c * blockDim.x;
+    if (i < nv && !p.ids) old[c] = Vec4<float>::load(s + i * 4);
+  }
   auto row_sum = [&](float ss) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
@@ -106,13 +110,13 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(B200StreamNorm p, int*
     post = 1.f / sqrtf(row_sum(ss) / (float)p.width + p.eps);
     __syncthreads();                     // (red is used again)
   }
-  auto value = [&](int i, float4 v) {
+  auto value = [&](int i, float4 v, float4 before) {
     if (p.post_w) {
       const float4 w = Vec4<float>::load(p.post_w + i * 4);
       v.x *= post * (w.x + p.norm_offset); v.y *= post * (w.y + p.norm_offset);
       v.z *= post * (w.z + p.norm_offset); v.w *= post * (w.w + p.norm_offset);
     }
-    if (!p.ids) add4(v, Vec4<float>::load(s + i * 4));
+    if (!p.ids) add4(v, before);
     return v;
   };
   float ss = 0.f;
@@ -120,13 +124,13 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(B200StreamNorm p, int*
   for (int c = 0; c < kRegs; ++c) {
     const int i = threadIdx.x + c * blockDim.x;
     if (i < nv) {
-      keep[c] = value(i, p.post_w ? keep[c] : update(i));
+      keep[c] = value(i, p.post_w ? keep[c] : update(i), old[c]);
       Vec4<float>::store(s + i * 4, keep[c]);
       ss += sq(keep[c]);
     }
   }
   for (int i = threadIdx.x + kRegs * blockDim.x; i < nv; i += blockDim.x) {
-    const float4 v = value(i, update(i));
+    const float4 v = value(i, update(i), Vec4<float>::load(s + i * 4));
     Vec4<float>::store(s + i * 4, v);
     ss += sq(v);
   }
@@ -143,6 +147,16 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(B200StreamNorm p, int*
     if (i < nv) finish(i, keep[c]);
   }
   for (int i = threadIdx.x + kRegs * blockDim.x; i < nv; i += blockDim.x) finish(i, Vec4<float>::load(s + i * 4));
+}
+
+template <typename T>
+static cudaError_t launch_stream_norm(const B200StreamNorm& a, int threads, cudaStream_t stream) {
+  const int groups = (a.cols / 4 + threads - 1) / threads;
+  const dim3 grid(a.T), block(threads);
+  int* st = device_status_word();
+  if (groups <= 1) return launch_pdl(stream_norm_kernel<T, 1>, grid, block, 0, stream, a, st);
+  if (groups <= 2) return launch_pdl(stream_norm_kernel<T, 2>, grid, block, 0, stream, a, st);
+  return launch_pdl(stream_norm_kernel<T, 4>, grid, block, 0, stream, a, st);
 }
 
 // ------------------------------------------------------------------------------------ fp32 products
@@ -257,10 +271,8 @@ int b200_stream_norm(const B200StreamNorm* a, cudaStream_t stream) {
   if (a->k > kMaxPairs) return -4;
   int threads = ((a->cols / 4 + 31) / 32) * 32;
   if (threads > 256) threads = 256;
-  int* st = device_status_word();
-  cudaError_t e = a->f32 ? launch_pdl(stream_norm_kernel<float>, dim3(a->T), dim3(threads), 0, stream, *a, st)
-                         : launch_pdl(stream_norm_kernel<__nv_bfloat16>, dim3(a->T), dim3(threads), 0, stream, *a, st);
-  return e == cudaSuccess ? 0 : -2;
+  return (a->f32 ? launch_stream_norm<float>(*a, threads, stream) : launch_stream_norm<__nv_bfloat16>(*a, threads, stream)) ==
+                 cudaSuccess ? 0 : -2;
 }
 
 int b200_gemm_f32(const void* A, int lda, const void* W, int ldw, void* out, int ldo, const void* bias, int M, int N,

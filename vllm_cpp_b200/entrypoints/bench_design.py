@@ -32,10 +32,10 @@ DIFORAX_SIZES = {
 
 def diforax_configs(size):
     """Three delta blocks to one attention block; chunks longer than the prompts, as the other model's
-    attention has no limit; an eighth as many identity experts, which the other model does not have."""
+    attention has no limit; an eighth as many identity experts (at least four), which the other model does not have."""
     from ..config import AttentionSpec, BlockSpec, DeltaSpec, ExpertSpec, ModelConfig, RopeConfig, model_config_of_blocks
     W, H, G, D, E, top, ff, layers, dh, dk = size
-    moe = ExpertSpec(experts=E, top=top, ff=ff, identity=E // 8, groups=4, keep=2)
+    moe = ExpertSpec(experts=E, top=top, ff=ff, identity=max(4, E // 8), groups=4, keep=2)
     att = AttentionSpec(heads=H, kv_heads=G, dim=D, vdim=D, scale=D ** -0.5, rot_dims=D, rot_base=1e6, chunk=1 << 15)
     delta = BlockSpec(None, moe, DeltaSpec(heads=dh, kv_heads=dk, dim=128, vdim=128, conv=4))
     blocks = [BlockSpec(att, moe) if l % 4 == 3 else delta for l in range(layers)]
@@ -389,7 +389,7 @@ class DiforaxKernels(KernelBench):
         from ..ops import moe as M
         from ..ops.stream import stream_norm
         W, E, top, ff = self.W, self.E, self.top, self.ff
-        P, I = T * top, E // 8
+        P, I = T * top, max(4, E // 8)
         ws = M.MoeWorkspace(self.dev, T, top, E, W, ff)
         x, wgu, wd = self.rnd(T, W), self.rnd(E, 2 * ff, W, s=0.05), self.rnd(E, W, ff, s=0.05)
         logits, corr = self.rnd(T, E + I, dtype=torch.float32), self.rnd(E + I, dtype=torch.float32, s=0.01)

@@ -99,6 +99,28 @@ def small_case(name: str):
         slots = torch.arange(B, dtype=torch.int32, device=dev)
         out = torch.empty(B, Hv, 128, device=dev, dtype=torch.bfloat16)
         fn = lambda: G.packed_decode(xc, a, b, A_log, dtb, state, slots, out, Hk, Hv)
+    elif name == "delta_small":
+        # 8 prompts of 2048 tokens at the head counts of gdn_scan_small
+        from types import SimpleNamespace
+        from . import delta as X
+        from .reference import build_prefill_tiles
+        B, n, s = 8, 2048, X.DeltaShape(G=2, H=6, D=128, V=128, dim=128, vdim=128, taps=4)
+        T, f32 = B * n, dict(device=dev, dtype=torch.float32)
+        i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)      # noqa: E731
+        tr, tq = build_prefill_tiles([n] * B)
+        rows_ = SimpleNamespace(seq_lens=i32([n] * B), state_slots=i32(list(range(B))),
+                                prefill_q_start=i32([i * n for i in range(B + 1)]), tile_req=i32(tr), tile_q0=i32(tq),
+                                num_decodes=0, num_prefills=B, num_tiles=len(tr))
+        w = {"conv_w": torch.randn(4, s.channels, **f32), "A": torch.rand(s.H, **f32), "dt": torch.randn(s.H, **f32),
+             "norm": torch.rand(s.V, **f32)}
+        bufs = {k: torch.empty(T, m, **f32) for k, m in (("q", s.G * s.D), ("k", s.G * s.D), ("g", s.H), ("beta", s.H),
+                                                        ("o", s.H * s.V))}
+        bufs["v"] = torch.empty(T, s.H * s.V, device=dev, dtype=torch.bfloat16)
+        bufs["chunks"] = X.chunk_workspace(dev, len(tr), s.H)
+        keep = (torch.randn(T, s.columns, device=dev).to(torch.bfloat16), torch.randn(T, 2 * s.H, **f32),
+                torch.zeros(B, 3, s.channels, device=dev, dtype=torch.bfloat16), torch.zeros(B, s.H, s.D, s.V, **f32),
+                torch.empty(T, s.H * s.V, device=dev, dtype=torch.bfloat16))
+        fn = lambda: X.delta_mixer(keep[0], keep[1], w, s, keep[2], keep[3], rows_, bufs, keep[4], 1e-6)
     elif name in ("bias_prefill_small", "bias_decode_small"):
         from . import bias_attn as A
         H, G, Dh, bs_, bias = 32, 4, 128, 32, torch.randn(32, 1024, device=dev)
@@ -209,7 +231,7 @@ def main():
                          "gemm_small | gemm_decode_small | prefill_small | decode_small | gdn_scan_small | "
                          "gdn_decode_small | moe_small | gemm_streamk_small | gemm_gated_small | "
                          "gemm_fp8_small | gemm_w4a16_small | gemm_nvfp4_small | gemm_nvfp4_prefill_small | "
-                         "decode_d256_small | mla_decode_small | bias_prefill_small | bias_decode_small")
+                         "decode_d256_small | mla_decode_small | bias_prefill_small | bias_decode_small | delta_small")
     args = ap.parse_args()
     if args.case:
         return small_case(args.case)
