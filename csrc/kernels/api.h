@@ -174,8 +174,8 @@ typedef struct B200MoeScatter {
 // Attention over pages [block_size][kw] keys | [block_size][G * vdim] values (attn_bias.cu). kw is the
 // whole key row; a head reads all of it (query rows kw wide, see b200_head_mix_kv) or, with ``grouped``, the
 // kw / G columns of its group (query rows that wide). Scores are multiplied by ``scale``. bias: fp32
-// [H, bias_len], the entry of distance min(i - j, bias_len - 1), or null. chunk > 0: position i sees j <= i
-// with i / chunk == j / chunk. null_entry: one softmax entry of score 0 without a value. Decode: one row per
+// [H, bias_len], the entry of distance min(i - j, bias_len - 1), or null. chunk > 0: a query
+// sees the keys of its own chunk of that many positions. null_entry: one softmax entry of score 0 without a value. Decode: one row per
 // request. Prefill: q_start [num_reqs + 1] and the 128-row tile list. f32: fp32 q / out / cache, not bf16.
 typedef struct B200BiasAttn {
   const void* q;

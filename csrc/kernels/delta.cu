@@ -2,9 +2,9 @@
 //
 //   delta_prep_kernel   short causal convolutions (any number of taps) + SiLU, unit q / k per head, log
 //                       decay and write strength, convolution state; prompt portions and decode rows
-//   delta_rule_kernel   S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, token by token with the
-//                       state in registers, then RMS norm of o, weight and SiLU gate. Serves decode rows and,
-//                       for any sizes and fp32 storage, whole prompt portions
+//   delta_rule_kernel   with F = e^g S the faded state:  S = F + k (x) beta (v - k F),  o = q S  token by token,
+//                       the state in registers, then RMS norm of o, weight and SiLU gate. Serves decode rows
+//                       and, for any sizes and fp32 storage, whole prompt portions
 //   delta_norm_kernel   the same norm and gate over rows of fp32 o (after the chunked prompt kernel)
 //
 // Sizes D, V are padded to multiples of 16 with zeros (weights, hence activations and state); ``dim`` and

@@ -1,6 +1,6 @@
 """Diforax decoders: delta-rule and chunked-attention blocks in any order over an fp32 residual stream.
 
-Every sublayer is normed before and after:  x += norm_b(mixer(norm(x)));  x += norm_b(ff(norm(x))).
+A sublayer f (mixer, then feed-forward) sits between two norms:  x += n2(f(n1(x))).
 
 * Delta mixer (``ops/delta.py``): short convolutions, unit q / k, one decay and one write strength per
   head; the fp32 state and the convolutions' last inputs are kept per request slot (``recurrent.py``).
