@@ -41,10 +41,29 @@ class RopeConfig:
 
 
 @dataclass
+class RotaryScaling:
+    """Frequencies divided by ``factor``; with ``original`` (the length before scaling) YaRN, which divides the
+    slow ones only: those of at most ``slow`` turns within it, ramped up to ``fast`` turns."""
+    factor: float
+    original: float = 0
+    fast: float = 32.0
+    slow: float = 1.0
+
+    def rope(self, base: float, dims: int) -> RopeConfig:
+        import math
+        if not self.original:
+            return RopeConfig(theta=base, rotary_dim=dims, scaling_type="linear", factor=self.factor)
+        return RopeConfig(theta=base, rotary_dim=dims, scaling_type="yarn", factor=self.factor,
+                          original_max_position=self.original, beta_fast=self.fast, beta_slow=self.slow,
+                          apply_yarn_scaling=False, attn_factor=0.1 * math.log(self.factor) + 1.0)
+
+
+@dataclass
 class AttentionSpec:
     """Softmax mixer of one decoder block: grouped heads with separate key and value sizes. Positions
     enter through a distance bias that saturates at ``bias_max`` (0: none) or a rotation of the first
-    ``rot_dims`` dimensions (0: none)."""
+    ``rot_dims`` dimensions (0: none). With ``diff`` every head has two maps over the same values and
+    subtracts the second, weighted by a learned number that starts around ``diff``."""
     heads: int
     kv_heads: int
     dim: int
@@ -55,6 +74,36 @@ class AttentionSpec:
     rot_base: float = 10000.0
     chunk: int = 0                            # > 0: a query sees the keys of its own chunk of this many positions
     kv_from: Optional[int] = None             # block whose keys and values are read (None: its own)
+    window: int = 0                           # > 0: a query sees itself and the window - 1 positions before it
+    rot_scaling: Optional[RotaryScaling] = None
+    diff: Optional[float] = None
+
+
+@dataclass
+class LatentSpec:
+    """Latent softmax mixer of one decoder block: ``heads`` heads whose keys (``dim``) and values (``vdim``)
+    are projections of one normed latent of ``kv_rank`` values per token, beside ``rot_dim`` rotated key
+    dimensions shared by the heads; queries come from a normed latent of ``q_rank`` values; each head's output
+    has a sigmoid gate."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    window: int = 0
+    rot_base: float = 10000.0
+    rot_scaling: Optional[RotaryScaling] = None
+
+
+@dataclass
+class RglruSpec:
+    """Real-gated linear recurrent mixer of one decoder block: ``width`` channels behind a short convolution of
+    ``conv`` taps, gates from ``blocks`` square matrices over equal parts of them."""
+    width: int
+    blocks: int
+    conv: int
 
 
 @dataclass
@@ -92,7 +141,14 @@ class ExpertSpec:
 class BlockSpec:
     attention: Optional[AttentionSpec] = None
     mlp: "Optional[ExpertSpec | DenseSpec]" = None
-    delta: Optional[DeltaSpec] = None         # set instead of ``attention``
+    delta: Optional[DeltaSpec] = None         # set instead of ``attention``, as the next two
+    latent: Optional[LatentSpec] = None
+    rglru: Optional[RglruSpec] = None
+    weights_of: Optional[int] = None          # block whose weights this one runs with (None: its own)
+
+    @property
+    def mixer(self):
+        return self.attention or self.delta or self.latent or self.rglru
 
 
 @dataclass
@@ -329,7 +385,7 @@ def model_config_from_blocks(cfg: dict) -> ModelConfig:
     """ModelConfig of a config.json that names one ``architecture`` and lists its ``layers``, each
     with a mixer and a feed-forward (or null)."""
     arch = cfg["architecture"]
-    readers = {"Nufusun": _nufusun_block, "Diforax": _diforax_block}
+    readers = {"Nufusun": _nufusun_block, "Diforax": _diforax_block, "Tabupel": _tabupel_block}
     if arch not in readers:
         raise ValueError(f"no reader for the layer list of architecture {arch!r}")
     blocks = []
@@ -338,9 +394,18 @@ def model_config_from_blocks(cfg: dict) -> ModelConfig:
             blocks.append(_checked(readers[arch](l), blocks))
         except ValueError as e:
             raise ValueError(f"layer {i}: {e}") from None
+    for i, b in enumerate(blocks):
+        if b.weights_of is not None:
+            src = blocks[b.weights_of] if 0 <= b.weights_of < len(blocks) else None
+            if src is None or src.weights_of is not None:
+                raise ValueError(f"layer {i}: block {b.weights_of} has no weights of its own")
+            if (src.mixer, src.mlp) != (b.mixer, b.mlp):
+                raise ValueError(f"layer {i}: block {b.weights_of}, whose weights it uses, has other sizes")
     kw = dict(vocab=int(cfg["vocab"]), width=int(cfg["width"]), eps=float(cfg["norm"]["eps"]), raw=cfg)
     if arch == "Nufusun":
         kw["embed_scale"] = float(cfg["embedding"]["scale"])
+    if arch == "Tabupel":
+        kw.update(residual_mult=float(cfg["residual_mult"]), logit_softcap=float(cfg["logit_softcap"]))
     m = model_config_of_blocks(arch, blocks, **kw)
     m.eos_token_id, m.bos_token_id = cfg.get("eos_token_id"), cfg.get("bos_token_id")
     return m
@@ -386,15 +451,46 @@ def _diforax_block(l: dict) -> BlockSpec:
     return BlockSpec(att, mlp, delta)
 
 
+def _tabupel_block(l: dict) -> BlockSpec:
+    m, f, att, latent, rglru, mlp = l["mixer"], l.get("mlp"), None, None, None, None
+    rot, mask = m.get("rot") or {}, m.get("mask") or {}
+    scaling = rot.get("scaling")
+    if scaling is not None:
+        scaling = RotaryScaling(**{k: float(v) for k, v in scaling.items() if k in ("factor", "original", "fast", "slow")})
+    where = dict(window=int(mask.get("size", 0)), rot_base=float(rot.get("base", 1.0)), rot_scaling=scaling)
+    if l["type"] == "attention":
+        att = AttentionSpec(**{k: int(m[k]) for k in ("heads", "kv_heads", "dim", "vdim")}, scale=float(m["scale"]),
+                            rot_dims=int(rot.get("dims", 0)), diff=float(m["diff"]), **where)
+    elif l["type"] == "latent_attention":
+        latent = LatentSpec(**{k: int(m[k]) for k in ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank")},
+                            scale=float(m["scale"]), **where)
+        if int(rot.get("dims", latent.rot_dim)) != latent.rot_dim:
+            raise ValueError(f"{rot['dims']} rotated dimensions of {latent.rot_dim}")
+    elif l["type"] == "rglru":
+        rglru = RglruSpec(**{k: int(m[k]) for k in ("width", "blocks", "conv")})
+    else:
+        raise ValueError(f"unknown mixer {l['type']!r}")
+    if f is not None:
+        if f["kind"] != "dense":
+            raise ValueError(f"unknown feed-forward {f['kind']!r}")
+        mlp = DenseSpec(ff=int(f["ff"]))
+    src = l.get("weights_of")
+    return BlockSpec(att, mlp, latent=latent, rglru=rglru, weights_of=None if src is None else int(src))
+
+
 def _checked(b: BlockSpec, before: list) -> BlockSpec:
     """The sizes of a block fit together (``before``: the blocks ahead of it)."""
-    m, a, f = b.attention or b.delta, b.attention, b.mlp
-    if m.heads % m.kv_heads:
+    m, a, f, lat = b.mixer, b.attention, b.mlp, b.latent
+    if (a or b.delta) is not None and m.heads % m.kv_heads:
         raise ValueError(f"{m.heads} heads do not divide into {m.kv_heads} groups")
     if a is not None and (a.rot_dims % 2 or a.rot_dims > a.dim):
         raise ValueError(f"{a.rot_dims} rotated dimensions of {a.dim}")
-    if b.delta is not None and b.delta.conv < 1:
+    if lat is not None and lat.rot_dim % 2:
+        raise ValueError(f"{lat.rot_dim} rotated dimensions")
+    if (b.delta or b.rglru) is not None and m.conv < 1:
         raise ValueError("a convolution has at least one tap")
+    if b.rglru is not None and m.width % m.blocks:
+        raise ValueError(f"{m.width} channels do not divide into {m.blocks} blocks")
     if a is not None and a.kv_from is not None:
         src = before[a.kv_from].attention if 0 <= a.kv_from < len(before) else None
         if src is None or src.kv_from is not None:
@@ -411,21 +507,27 @@ def _checked(b: BlockSpec, before: list) -> BlockSpec:
 
 
 def model_config_of_blocks(arch: str, blocks: list, *, vocab: int, width: int, eps: float, embed_scale: float = 1.0,
-                           max_position: int = 32768, raw: Optional[dict] = None) -> ModelConfig:
+                           residual_mult: float = 1.0, logit_softcap: float = 0.0, max_position: int = 32768,
+                           raw: Optional[dict] = None) -> ModelConfig:
     att = [b.attention for b in blocks if b.attention is not None]
+    lat = [b.latent for b in blocks if b.latent is not None]
     moe = [b.mlp for b in blocks if isinstance(b.mlp, ExpertSpec)]
     dense = [b.mlp.ff for b in blocks if isinstance(b.mlp, DenseSpec)]
     m = ModelConfig(
         architecture=arch, vocab_size=vocab, hidden_size=width, num_layers=len(blocks),
         intermediate_size=max([m.ff * m.top for m in moe] + dense, default=0),
-        num_heads=max([a.heads for a in att], default=1), num_kv_heads=max([a.kv_heads for a in att], default=1),
-        head_dim=max([a.dim for a in att], default=8), v_head_dim=max([a.vdim for a in att], default=8),
+        num_heads=max([a.heads for a in att + lat], default=1), num_kv_heads=max([a.kv_heads for a in att], default=1),
+        head_dim=max([a.dim for a in att + lat], default=8), v_head_dim=max([a.vdim for a in att + lat], default=8),
         rms_norm_eps=eps, embed_scale=embed_scale, norm_topk_prob=False,
         num_experts=max([m.experts for m in moe], default=0), num_experts_per_tok=max([m.top for m in moe], default=0),
         moe_intermediate_size=max([m.ff for m in moe], default=0), max_position_embeddings=max_position,
         blocks=blocks, raw=raw or {})
     if arch == "Nufusun":
         m.gemma_norm, m.attention_bias, m.hidden_act, m.scoring_func = True, True, "clamped_gate", "sigmoid"
+    elif arch == "Tabupel":
+        m.hidden_act, m.residual_multiplier, m.final_logit_softcap = "silu", residual_mult, logit_softcap
+        m.layer_types = ["linear_attention" if b.rglru is not None else "sliding_attention" if b.mixer.window
+                         else "full_attention" for b in blocks]
     else:
         m.sandwich_norm, m.hidden_act = True, "gelu_tanh"
         m.layer_types = ["linear_attention" if b.delta is not None else "chunked_attention" if b.attention.chunk
@@ -435,6 +537,8 @@ def model_config_of_blocks(arch: str, blocks: list, *, vocab: int, width: int, e
 
 def block_config_dict(cfg: ModelConfig) -> dict:
     """config.json of a ModelConfig with ``blocks`` (the inverse of model_config_from_blocks)."""
+    if cfg.architecture == "Tabupel":
+        return _tabupel_dict(cfg)
     layers = []
     for b in cfg.blocks:
         m, a, f, mlp = b.attention or b.delta, b.attention, b.mlp, None
@@ -465,6 +569,30 @@ def block_config_dict(cfg: ModelConfig) -> dict:
     if cfg.architecture == "Nufusun":
         out["embedding"] = {"scale": cfg.embed_scale}
     return out
+
+
+def _tabupel_dict(cfg: ModelConfig) -> dict:
+    from dataclasses import asdict
+    layers = []
+    for b in cfg.blocks:
+        m = {k: v for k, v in asdict(b.mixer).items() if v is not None}
+        kind = "rglru" if b.rglru is not None else "latent_attention" if b.latent is not None else "attention"
+        if b.rglru is None:
+            rot = {"base": m.pop("rot_base"), "dims": m.pop("rot_dims", m.get("rot_dim"))}
+            s = m.pop("rot_scaling", None)
+            if s is not None:
+                rot["scaling"] = s if s["original"] else {"factor": s["factor"]}
+            w = m.pop("window")
+            m.update(rot=rot, **({"mask": {"size": w}} if w else {}))
+            for k in ("bias_max", "chunk"):
+                m.pop(k, None)
+        l = {"type": kind, "mixer": m, "mlp": None if b.mlp is None else {"kind": "dense", "ff": b.mlp.ff}}
+        if b.weights_of is not None:
+            l["weights_of"] = b.weights_of
+        layers.append(l)
+    return {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_size,
+            "norm": {"eps": cfg.rms_norm_eps}, "residual_mult": cfg.residual_multiplier,
+            "logit_softcap": cfg.final_logit_softcap, "layers": layers}
 
 
 def load_model_config(model_dir: str) -> ModelConfig:
@@ -558,6 +686,26 @@ def synthetic_config(name: str) -> ModelConfig:
         return model_config_of_blocks("Diforax", [BlockSpec(None, DenseSpec(96), delta), BlockSpec(att, moe),
                                                   BlockSpec(None, None, delta), BlockSpec(shared, DenseSpec(80))],
                                       vocab=500, width=192, eps=1e-5, max_position=2048)
+    if n == "tabupel-3b":
+        # two recurrent layers to one attention layer, latent and differential attention in turn
+        ff, rec = DenseSpec(7680), RglruSpec(width=2560, blocks=10, conv=4)
+        lat = LatentSpec(heads=16, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, scale=192 ** -0.5, window=2048,
+                         rot_base=1e4, rot_scaling=RotaryScaling(40.0, 4096))
+        att = AttentionSpec(heads=10, kv_heads=2, dim=128, vdim=256, scale=128 ** -0.5, rot_dims=128, rot_base=1e6,
+                            rot_scaling=RotaryScaling(8.0), diff=0.6, window=2048)
+        r, a, d = (BlockSpec(None, ff, rglru=rec), BlockSpec(None, ff, latent=lat), BlockSpec(att, ff))
+        return model_config_of_blocks("Tabupel", [r, r, a, r, r, d] * 4 + [r, r], vocab=151936, width=2560, eps=1e-6,
+                                      residual_mult=0.5, logit_softcap=30.0, max_position=131072)
+    if n == "tiny-tabupel":
+        ff = DenseSpec(96)
+        rec = BlockSpec(None, ff, rglru=RglruSpec(width=80, blocks=5, conv=3))
+        lat = LatentSpec(heads=3, dim=40, rot_dim=16, vdim=24, q_rank=56, kv_rank=48, scale=0.15, window=50, rot_base=5e3,
+                         rot_scaling=RotaryScaling(3.0, 64))
+        att = AttentionSpec(heads=4, kv_heads=2, dim=24, vdim=40, scale=0.2, rot_dims=16, rot_base=5e3,
+                            rot_scaling=RotaryScaling(2.0), diff=0.4, window=33)
+        return model_config_of_blocks("Tabupel", [BlockSpec(None, None, latent=lat), rec, BlockSpec(att, DenseSpec(64)),
+                                                  BlockSpec(None, ff, rglru=rec.rglru, weights_of=1)],
+                                      vocab=500, width=192, eps=1e-5, residual_mult=0.7, logit_softcap=20.0, max_position=2048)
     if n.startswith("tiny"):
         # small shapes for tests: tiny-dense, tiny-moe, tiny-mla, tiny-gdn
         base = dict(vocab_size=512, hidden_size=256, intermediate_size=512, num_layers=2,

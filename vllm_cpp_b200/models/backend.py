@@ -282,6 +282,31 @@ class CpuBackend(FusedLinearMixin):
         from ..ops.bias_attn import ref_rotate_kv
         ref_rotate_kv(qkv, positions, table, rot, eps, q_out, slots, cache, **kw)
 
+    def diff_combine(self, maps, out, **kw):
+        from ..ops.bias_attn import ref_diff_combine
+        return ref_diff_combine(maps, out, **kw)
+
+    def latent_prepare(self, down, positions, table, w, shape, eps, cq, slots, cache):
+        from ..ops.latent import ref_prepare
+        ref_prepare(down, positions, table, w, shape, eps, cq, slots, cache)
+
+    def latent_attention(self, q, positions, table, cache, w, shape, ctx, group, *, scale, window, block_size, gate, out, **_):
+        from ..ops.latent import ref_latent_attention
+        return ref_latent_attention(q, positions, table, cache, w, shape, block_table=ctx.block_table[group],
+                                    seq_lens=ctx.seq_lens, q_start=ctx.query_start, scale=scale, window=window,
+                                    block_size=block_size, gate=gate, out=out)
+
+    def short_conv(self, x, w, bias, state, ctx, out, act=None):
+        from ..ops.rglru import ref_short_conv
+        return ref_short_conv(x, w, bias, state, ctx, out, act)
+
+    def rglru(self, u, y, w, shape, state, ctx, bufs, out):
+        from ..ops.rglru import ref_rglru
+        return ref_rglru(u, y, w, shape, state, ctx, bufs, out)
+
+    def softcap_f32(self, x, cap):
+        return x.copy_(cap * torch.tanh(x / cap))
+
     def delta_mixer(self, proj, ab, w, shape, conv_state, state, ctx, bufs, out, eps):
         from ..ops.delta import ref_delta_mixer
         return ref_delta_mixer(proj, ab, w, shape, conv_state, state, ctx, bufs, out, eps)
@@ -602,6 +627,62 @@ class GpuBackend(FusedLinearMixin):
     def rotate_kv(self, qkv, positions, table, rot, eps, q_out, slots, cache, **kw):
         from ..ops.bias_attn import rotate_kv
         rotate_kv(qkv, positions, table, rot, eps, q_out, slots, cache, **kw)
+
+    def diff_combine(self, maps, out, **kw):
+        from ..ops.bias_attn import diff_combine
+        return diff_combine(maps, out, **kw)
+
+    def latent_prepare(self, down, positions, table, w, shape, eps, cq, slots, cache):
+        from ..ops.latent import prepare
+        prepare(down, positions, table, w, shape, eps, cq, slots, cache)
+
+    def latent_attention(self, q, positions, table, cache, w, shape, ctx, group, *, scale, window, block_size, gate, out,
+                         pages, absorbed, scratch):
+        """Decode rows in the absorbed form; prompt portions over expanded keys and values (``pages``: their
+        visible pages, None: these too in the absorbed form). ``absorbed(n)``: (query, latent output) rows,
+        ``scratch(name, rows, cols)``: page rows. ``q`` is not rotated yet."""
+        from ..ops import latent as M
+        s, nd, T, bt = shape, ctx.num_decodes, q.shape[0], ctx.block_table[group]
+        tensor = q.dtype == torch.bfloat16 and s.tensor_decode
+        n_abs = nd if pages is not None else T
+        qa, lat = absorbed(n_abs)
+        M.queries(q, positions, table, s, qa, n_abs)
+        if n_abs:
+            M.heads_product(q, s.qw, w["uk_t"], qa, s.row, n_abs)
+        common = dict(scale=scale, window=window, block_size=block_size)
+        if nd and tensor:
+            M.decode(qa[:nd], cache, lat[:nd], s, block_table=bt[:nd], seq_lens=ctx.seq_lens[:nd], gate=gate[:nd],
+                     splits=ctx.decode_splits, tmp=ctx.extra.get("decode_tmp"), **common)
+        elif nd:
+            M.absorbed_any_size(qa[:nd], cache, lat[:nd], s, decode_rows=True, block_table=bt[:nd], seq_lens=ctx.seq_lens[:nd],
+                                gate=gate[:nd], **common)
+        P = ctx.num_prefills
+        rows = dict(seq_lens=ctx.seq_lens[nd:], q_start=ctx.prefill_q_start, num_reqs=P, tile_req=ctx.tile_req[:ctx.num_tiles],
+                    tile_q0=ctx.tile_q0[:ctx.num_tiles], gate=gate[nd:], **common)
+        if P and pages is None:
+            M.absorbed_any_size(qa[nd:], cache, lat[nd:], s, decode_rows=False, block_table=bt[nd:], **rows)
+        if n_abs:
+            M.heads_product(lat, s.rankp, w["uv"], out, s.V, n_abs)
+        if P and pages is not None:
+            v = pages()
+            n = v["total"] * block_size
+            dense, kv = scratch(f"latent{s.row}", n, s.row), scratch(f"expanded{s.H * (s.D + s.V)}", n, s.H * (s.D + s.V))
+            M.gather(cache, bt[nd:], ctx.seq_lens[nd:], v["first"], v["base"], block_size, dense, P, v["table"].shape[1])
+            self.gemm(dense[:, : s.rankp], w["kv"], out=kv)
+            M.prefill_expanded(q[nd:], kv, dense, out[nd:], s, block_table=v["table"], **rows)
+        return out
+
+    def short_conv(self, x, w, bias, state, ctx, out, act=None):
+        from ..ops.rglru import short_conv
+        return short_conv(x, w, bias, state, ctx, out, act)
+
+    def rglru(self, u, y, w, shape, state, ctx, bufs, out):
+        from ..ops.rglru import rglru
+        return rglru(u, y, w, shape, state, ctx, bufs, out)
+
+    def softcap_f32(self, x, cap):
+        from ..ops.stream import softcap_f32
+        return softcap_f32(x, cap)
 
     def delta_mixer(self, proj, ab, w, shape, conv_state, state, ctx, bufs, out, eps):
         from ..ops.delta import delta_mixer

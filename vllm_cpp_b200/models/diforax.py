@@ -17,66 +17,25 @@ from __future__ import annotations
 
 import torch
 
-from ..config import DenseSpec, ExpertSpec, ModelConfig, ParallelConfig
+from ..config import DenseSpec, ExpertSpec
 from ..ops.bias_attn import grouped_decode_splits
 from ..ops.delta import DeltaShape
-from .backend import make_backend
-from .base import BufferPool, StepContext
-from .dense import ACT_KIND, DenseModel
+from .base import StepContext
+from .listed import ListedModel, pad as _pad, pad_heads as _pad_heads
 from .recurrent import RecurrentState
-
-
-def _pad(n: int, m: int = 8) -> int:
-    return (n + m - 1) // m * m
-
-
-def _padded(t: torch.Tensor, *shape: int) -> torch.Tensor:
-    if tuple(t.shape) == shape:
-        return t
-    out = torch.zeros(shape, dtype=t.dtype, device=t.device)
-    out[tuple(slice(0, n) for n in t.shape)] = t
-    return out
-
-
-def _pad_heads(t: torch.Tensor, heads: int, padded: int, axis: int = 0) -> torch.Tensor:
-    """Each head's rows (or columns) padded with zeros."""
-    t = t.transpose(0, axis)
-    out = torch.zeros((heads, padded, *t.shape[1:]), dtype=t.dtype, device=t.device)
-    out[:, : t.shape[0] // heads] = t.reshape(heads, -1, *t.shape[1:])
-    return out.reshape(heads * padded, *t.shape[1:]).transpose(0, axis)
 
 
 def _delta_shape(d) -> DeltaShape:
     return DeltaShape(G=d.kv_heads, H=d.heads, D=_pad(d.dim, 16), V=_pad(d.vdim, 16), dim=d.dim, vdim=d.vdim, taps=d.conv)
 
 
-class DiforaxModel(DenseModel):
-    DTYPES = ("bfloat16", "float32")
-
-    def __init__(self, cfg: ModelConfig, device="cuda", parallel: ParallelConfig | None = None,
-                 comm=None, max_position: int | None = None):
-        # (the dense constructor sets up the one rotary table and the shards of uniform layers)
-        self.cfg, self.device = cfg, torch.device(device)
-        self.par = parallel or ParallelConfig()
-        if self.par.tensor_parallel_size > 1:
-            raise ValueError("Diforax runs on one rank")
-        self.tp, self.rank, self.comm = 1, 0, comm
-        self.be = make_backend(self.device)
-        self.dtype = torch.float32 if cfg.dtype == "float32" else torch.bfloat16
-        self.hq, self.hkv, self.D = cfg.num_heads, cfg.num_kv_heads, _pad(cfg.head_dim, 16)
-        self.max_position = max_position or cfg.max_position_embeddings
-        self.width, self.cols = cfg.hidden_size, _pad(cfg.hidden_size)
-        self.vocab_shard, self.vocab_start = cfg.vocab_size, 0
+class DiforaxModel(ListedModel):
+    def __init__(self, cfg, *args, **kw):
+        super().__init__(cfg, *args, **kw)
         self.delta_layers = [l for l, b in enumerate(cfg.blocks) if b.delta is not None]
         self.kv_layers = [l for l, b in enumerate(cfg.blocks) if b.attention is not None and b.attention.kv_from is None]
-        self.bufs = BufferPool(self.device)
         self.moe_ws: dict = {}
         self.chunks = None                    # scratch of the chunked delta rule
-        self.recurrent = RecurrentState()
-        self.state: dict[int, tuple] = {}
-        self.rope: dict[tuple, torch.Tensor] = {}
-        self.w: dict[str, torch.Tensor] = {}
-        self.layers: list[dict] = []
 
     # ------------------------------------------------------------------ weights
     def init_random(self, seed: int = 0, std: float = 0.02) -> None:
@@ -125,11 +84,7 @@ class DiforaxModel(DenseModel):
         self.load_weights(gen())
 
     def load_weights(self, named_tensors) -> None:
-        c, C, dev, dt = self.cfg, self.cols, self.device, self.dtype
-
-        def put(t, *shape, dtype=None):
-            return _padded(t.to(dev, dtype or dt), *(shape or t.shape)).contiguous()
-
+        c, C, dev, dt, put = self.cfg, self.cols, self.device, self.dtype, self.put
         self.layers = [dict() for _ in c.blocks]
         for L, b in zip(self.layers, c.blocks):
             if isinstance(b.mlp, ExpertSpec):
@@ -138,17 +93,8 @@ class DiforaxModel(DenseModel):
                 L["w_down"] = torch.zeros((b.mlp.experts, C, f8), dtype=dt, device=dev)
         pend: list[dict] = [dict() for _ in c.blocks]
         for name, t in named_tensors:
-            if name == "embed":
-                self.w["embed"] = put(t, t.shape[0], C)
-            elif name == "head":
-                self.w["lm_head"] = put(t, _pad(t.shape[0]), C)
-            elif name == "final.norm":
-                self.w["final_norm"] = put(t, C, dtype=torch.float32)
-            else:
-                layer, _, rest = name.partition(".")
-                if not (layer.startswith("l") and layer[1:].isdigit() and int(layer[1:]) < len(c.blocks)):
-                    raise ValueError(f"unexpected tensor {name!r}")
-                l = int(layer[1:])
+            if not self._take_shared(name, t):
+                l, rest = self._block_of(name)
                 L, f, part = self.layers[l], c.blocks[l].mlp, rest.split(".")
                 if isinstance(f, ExpertSpec) and part[0] == "mlp" and len(part) == 3:
                     e, f8 = int(part[1][1:]), _pad(f.ff)
@@ -159,37 +105,18 @@ class DiforaxModel(DenseModel):
                         L["w_gate_up"][e, r0: r0 + f.ff, : self.width] = t.to(dev, dt)
                 pend[l][rest] = None if "w_gate_up" in L and len(part) == 3 and part[0] == "mlp" else t
         for l, (L, b, p) in enumerate(zip(self.layers, c.blocks, pend)):
-            want = self._tensor_names(b)
-            if want != set(p):
-                raise ValueError(f"layer {l}: tensors missing from the checkpoint {sorted(want - set(p))}, "
-                                 f"unexpected {sorted(set(p) - want)}")
+            self._expect(l, self._tensor_names(b), set(p))
             for n in ("norm1", "norm1b", "norm2", "norm2b"):
                 if n in p:
                     L[n] = put(p[n], C, dtype=torch.float32)
             (self._load_delta if b.delta is not None else self._load_attention)(L, b, {n[4:]: t for n, t in p.items()}, put)
             f = b.mlp
             if isinstance(f, DenseSpec):
-                ff = self._ff_padded(f.ff)
-                gate, up = (put(p["mlp." + n], ff, C) for n in ("gate", "up"))
-                if self._bf16_kernels():
-                    from ..ops import interleave_gate_up
-                    L["gate_up"] = interleave_gate_up(gate, up).contiguous()
-                else:
-                    L["gate_up"] = torch.cat([gate, up], 0)
-                L["down"] = put(p["mlp.down"], C, ff)
+                self._load_dense(L, f, p)
             elif f is not None:
                 L["router"] = put(p["mlp.router"], _pad(f.experts + f.identity), C)
                 L["correction"] = put(p["mlp.correction"], dtype=torch.float32)
-        for k in ("embed", "lm_head", "final_norm"):
-            if k not in self.w:
-                raise ValueError(f"{k} is missing from the checkpoint")
-
-    def _bf16_kernels(self) -> bool:
-        return self.device.type == "cuda" and self.dtype == torch.bfloat16
-
-    def _ff_padded(self, ff: int) -> int:
-        """(the gated product takes gate and up rows in blocks of 128)"""
-        return _pad(ff, 128 if self._bf16_kernels() else 8)
+        self._expect_shared()
 
     @staticmethod
     def _tensor_names(b) -> set:
@@ -231,9 +158,6 @@ class DiforaxModel(DenseModel):
             i = torch.arange(0, a.rot_dims, 2, dtype=torch.float64)
             self.rope[key] = self.be.rope_table(a.rot_base ** (-i / a.rot_dims), self.max_position + 8)
 
-    def quantize_weights(self, method: str = "nvfp4") -> None:
-        raise ValueError("Diforax checkpoints are served in bfloat16 or float32")
-
     # ------------------------------------------------------------------ caches and state
     def _kv_row(self, l: int) -> int:
         a = self.cfg.blocks[l].attention
@@ -273,12 +197,6 @@ class DiforaxModel(DenseModel):
             n += (s.taps - 1) * s.channels * self.dtype.itemsize + s.H * s.D * s.V * 4
         return n
 
-    def snapshot_state(self, slots: list) -> None:
-        self.recurrent.snapshot(slots)
-
-    def restore_state(self, slots: list) -> None:
-        self.recurrent.restore(slots)
-
     def decode_workspace(self, batch: int, max_seq_len: int, block_size: int):
         """(KV splits, split buffers) of a decode batch; one pair of buffers serves every block."""
         att = [b.attention for b in self.cfg.blocks if b.attention is not None]
@@ -310,16 +228,8 @@ class DiforaxModel(DenseModel):
         return (self.bufs.get(f"proj{n}", T, n, self.dtype), self.bufs.get(f"q{a.heads * D}", T, a.heads * D, self.dtype),
                 self.bufs.get(f"heads{a.heads * V}", T, a.heads * V, self.dtype))
 
-    def _dense_buffers(self, f, T: int):
-        ff = self._ff_padded(f.ff)
-        return (self.bufs.get(f"act{ff}", T, ff, self.dtype), self.bufs.get(f"gate_up{ff}", T, 2 * ff, self.dtype))
-
     def reserve_buffers(self, max_tokens: int, max_reqs: int) -> None:
-        self.bufs.reserve("stream", max_tokens, self.cols, torch.float32)
-        self.bufs.reserve("mixed", max_tokens, self.cols, torch.float32)
-        self.bufs.reserve("normed", max_tokens, self.cols, self.dtype)
-        self.bufs.reserve("last", max_reqs, self.cols, self.dtype)
-        self.bufs.reserve("logits", max_reqs, _pad(self.cfg.vocab_size), torch.float32)
+        self._reserve_rows(max_tokens, max_reqs)
         self.recurrent = RecurrentState()
         heads = max([self.cfg.blocks[l].delta.heads for l in self.delta_layers], default=0)
         if heads and self._bf16_kernels():
@@ -343,9 +253,6 @@ class DiforaxModel(DenseModel):
                     from ..ops.moe import MoeWorkspace
                     self.moe_ws[key] = MoeWorkspace(self.device, max_tokens, f.top, f.experts, self.cols, _pad(f.ff),
                                                     self.dtype)
-
-    def fused_tp_supported(self) -> bool:
-        return False
 
     # ------------------------------------------------------------------ forward
     def _delta(self, h, l, L, ctx, T, out):
@@ -372,9 +279,7 @@ class DiforaxModel(DenseModel):
         """-> what ``stream_norm`` adds: a product, or expert outputs and where to find them."""
         be = self.be
         if isinstance(f, DenseSpec):
-            act, gate_up = self._dense_buffers(f, T)
-            be.gated_unit(h, L["gate_up"], ACT_KIND["gelu_tanh"], act, gate_up)
-            return dict(a=be.gemm(act, L["down"], out=out, out_dtype=torch.float32))
+            return dict(a=self._dense(h, L, f, "gelu_tanh", T, out))
         n = f.experts + f.identity
         logits = self.bufs.get(f"router{_pad(n)}", T, _pad(n), torch.float32)
         be.gemm(h, L["router"], out=logits, out_dtype=torch.float32)
@@ -401,11 +306,4 @@ class DiforaxModel(DenseModel):
             if b.mlp is not None:
                 add = self._feed_forward(h, L, b.mlp, T, mixed)
                 be.stream_norm(stream, nw, eps, h, post_w=L["norm2b"], **add, **norm)
-        if ctx.decode_only_full_logits:
-            n, last = T, h
-        else:
-            n = ctx.num_logits
-            last = be.gather_rows(h, ctx.logits_indices[:n], out=self.bufs.get("last", n, self.cols, self.dtype))
-        logits = self.bufs.get("logits", n, self.w["lm_head"].shape[0], torch.float32)
-        be.gemm(last, self.w["lm_head"], out=logits, out_dtype=torch.float32)
-        return logits[:, : c.vocab_size]
+        return self._logits(ctx, h)

@@ -20,6 +20,7 @@ _REGISTRY.update({
     "OPTForCausalLM": ("opt", "OPTModel"),
     "Nufusun": ("nufusun", "NufusunModel"),
     "Diforax": ("diforax", "DiforaxModel"),
+    "Tabupel": ("tabupel", "TabupelModel"),
 })
 
 

@@ -41,9 +41,7 @@ def _yarn_correction_range(low_rot, high_rot, dim, base, max_pos, truncate=True)
 
 
 def _yarn_linear_ramp(lo, hi, n):
-    if lo == hi:
-        hi += 0.001
-    r = (torch.arange(n, dtype=torch.float64) - lo) / (hi - lo)
+    r = (torch.arange(n, dtype=torch.float64) - lo) / max(hi - lo, 0.001)
     return r.clamp(0, 1)
 
 

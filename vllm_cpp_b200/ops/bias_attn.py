@@ -1,6 +1,7 @@
 """Attention over pages ``[block_size, kw] keys | [block_size, G * vdim] values``: grouped heads (each reads
 the key columns of its group) or heads mixed before the softmax, with an optional distance bias, null
-softmax entry and limit to the query's chunk of positions.
+softmax entry and limit to the query's chunk or window of positions. With two ``maps`` every head has two
+queries and every group two keys over the same values (``diff_combine`` joins the two outputs).
 
 The mix of the heads is moved to the query side (``head_mix_kv``): head ``h`` reads the whole key
 row of a token with the query row ``[sum_{g in group 0} M[h, g] q_g | sum_{g in group 1} ... ]``."""
@@ -8,6 +9,7 @@ from __future__ import annotations
 
 import ctypes
 import math
+from typing import NamedTuple, Optional
 
 import torch
 
@@ -23,7 +25,17 @@ class BiasAttnArgs(ctypes.Structure):
                 ("tmp_lse", _P), ("tile_req", _P), ("tile_q0", _P),
                 ("max_blocks", _I), ("num_reqs", _I), ("rows", _I), ("H", _I), ("G", _I), ("kw", _I), ("vdim", _I),
                 ("block_size", _I), ("bias_len", _I), ("null_entry", _I), ("f32", _I), ("splits", _I),
-                ("num_tiles", _I), ("grouped", _I), ("chunk", _I), ("scale", ctypes.c_float)]
+                ("num_tiles", _I), ("grouped", _I), ("chunk", _I), ("scale", ctypes.c_float),
+                ("window", _I), ("maps", _I), ("values_in_keys", _I), ("shared", _I), ("gate", _P), ("ldg", _L),
+                ("keys", _P), ("values", _P), ("shared_keys", _P), ("ldk", _L), ("ldv", _L), ("lds", _L)]
+
+
+class SplitRows(NamedTuple):
+    """Key and value rows outside a page tensor, ``block_size`` consecutive rows to a page, and key columns that
+    every head shares (a head's query row: its own columns padded to whole 64-wide chunks, then these)."""
+    keys: torch.Tensor
+    values: torch.Tensor
+    shared: Optional[torch.Tensor] = None
 
 
 _declared = False
@@ -36,7 +48,8 @@ def _declare():
     P, I, L = _lib.P, _lib.I, ctypes.c_longlong
     A = ctypes.POINTER(BiasAttnArgs)
     _lib.declare("b200_head_mix_kv", [P, L, P, P, L, P, P, I, I, I, I, I, I, I, P], I)
-    _lib.declare("b200_rotate_kv", [P, L, P, P, I, _lib.F, P, L, P, P, I, I, I, I, I, I, I, I, P], I)
+    _lib.declare("b200_rotate_kv", [P, L, P, P, I, _lib.F, P, P, P, L, P, P, I, I, I, I, I, I, I, I, I, P], I)
+    _lib.declare("b200_diff_combine", [P, L, P, L, I, I, I, I, _lib.F, _lib.F, _lib.F, I, P], I)
     _lib.declare("b200_bias_attn_kernel", [A, I], I)
     _lib.declare("b200_bias_attn_decode", [A, I, P], I)
     _lib.declare("b200_bias_attn_prefill", [A, I, P], I)
@@ -54,36 +67,58 @@ def head_mix_kv(qkv, mix, q_out, slots, cache, *, H, G, dim, vdim, block_size):
                                  int(q_out.dtype == torch.float32), stream_ptr()), "head_mix_kv")
 
 
-def rotate_kv(qkv, positions, table, rot, eps, q_out, slots, cache, *, H, G, D, V, dim, block_size):
+def rotate_kv(qkv, positions, table, rot, eps, q_out, slots, cache, *, H, G, D, V, dim, block_size, q_w=None, k_w=None,
+              value_heads=None):
     """Rows ``[q | k | v]`` (``G`` 0: q alone) -> q and k heads rotated over their first ``rot`` dimensions
     (pairs half of ``rot`` apart, ``table`` [positions, cos | sin]) and divided by their root mean square
-    over ``dim``; q to ``q_out`` [T, H * D], k and v to ``cache`` (slot < 0: none)."""
+    over ``dim``; q to ``q_out`` [T, H * D], k and v to ``cache`` (slot < 0: none). With weights ``q_w`` /
+    ``k_w`` fp32 [D] the heads are normed and weighted first, then rotated. ``value_heads``: as many as ``G``."""
     _declare()
     assert qkv.dtype == q_out.dtype and (cache is None or cache.dtype == q_out.dtype)
-    check(lib().b200_rotate_kv(ptr(qkv), qkv.stride(0), ptr(positions), ptr(table), rot, eps, ptr(q_out), q_out.stride(0),
-                               ptr(slots), ptr(cache), H, G, D, V, dim, block_size, qkv.shape[0],
-                               int(q_out.dtype == torch.float32), stream_ptr()), "rotate_kv")
+    check(lib().b200_rotate_kv(ptr(qkv), qkv.stride(0), ptr(positions), ptr(table), rot, eps, ptr(q_w), ptr(k_w), ptr(q_out),
+                               q_out.stride(0), ptr(slots), ptr(cache), H, G, G if value_heads is None else value_heads, D, V,
+                               dim, block_size, qkv.shape[0], int(q_out.dtype == torch.float32), stream_ptr()), "rotate_kv")
 
 
-def _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry, scale, chunk,
-          grouped) -> BiasAttnArgs:
+def diff_combine(maps, out, *, H, V, vdim, lam, eps, scale):
+    """``maps`` [T, H * 2 * V] -> per head o = first - ``lam`` second, over its root mean square over ``vdim``,
+    times ``scale``; ``out`` [T, H * V]."""
+    _declare()
+    check(lib().b200_diff_combine(ptr(maps), maps.stride(0), ptr(out), out.stride(0), H, V, vdim, maps.shape[0], lam, eps, scale,
+                                  int(out.dtype == torch.float32), stream_ptr()), "diff_combine")
+    return out
+
+
+def _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry, scale, chunk, window,
+          maps, grouped, gate, values_in_keys, rows=None) -> BiasAttnArgs:
     a = BiasAttnArgs()
     a.q, a.ldq, a.out, a.ldo = ptr(q), q.stride(0), ptr(out), out.stride(0)
-    a.cache, a.num_blocks = ptr(cache), cache.shape[0]
+    if rows is None:
+        a.cache, a.num_blocks = ptr(cache), cache.shape[0]
+    else:
+        a.num_blocks = rows.keys.shape[0] // block_size
+        a.keys, a.ldk, a.values, a.ldv = ptr(rows.keys), rows.keys.stride(0), ptr(rows.values), rows.values.stride(0)
+        if rows.shared is not None:
+            a.shared_keys, a.lds, a.shared = ptr(rows.shared), rows.shared.stride(0), q.shape[1] // H - -(-kw // G // 64) * 64
     a.block_table, a.max_blocks, a.seq_lens = ptr(block_table), block_table.stride(0), ptr(seq_lens)
     a.bias, a.bias_len = ptr(bias), bias.shape[1] if bias is not None else 0
     a.rows, a.num_reqs = q.shape[0], q.shape[0]
     a.H, a.G, a.kw, a.vdim, a.block_size = H, G, kw, vdim, block_size
     a.null_entry, a.f32, a.splits = int(null_entry), int(q.dtype == torch.float32), 1
-    a.scale, a.chunk, a.grouped = scale, chunk, int(grouped)
+    a.scale, a.chunk, a.window, a.maps, a.grouped = scale, chunk, window, maps, int(grouped)
+    a.values_in_keys = int(values_in_keys)
+    a.gate, a.ldg = ptr(gate), gate.stride(0) if gate is not None else 0
     return a
 
 
 def decode(q, cache, out, *, block_table, seq_lens, H, G, kw, vdim, block_size, bias=None, null_entry=False,
-           splits=1, tmp=None, any_size=False, scale=1.0, chunk=0, grouped=False):
-    """One query row per request, at its last position."""
+           splits=1, tmp=None, any_size=False, scale=1.0, chunk=0, window=0, maps=1, grouped=False, gate=None,
+           values_in_keys=False):
+    """One query row per request, at its last position. ``gate`` [rows, H]: the outputs times its sigmoid;
+    ``values_in_keys``: values are the first columns of the key rows (these two: any-size kernel)."""
     _declare()
-    a = _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry, scale, chunk, grouped)
+    a = _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry, scale, chunk, window, maps,
+              grouped, gate, values_in_keys)
     if splits > 1:
         if tmp is None:
             tmp = (torch.empty(a.rows * H * splits * vdim, dtype=torch.float32, device=q.device),
@@ -95,23 +130,27 @@ def decode(q, cache, out, *, block_table, seq_lens, H, G, kw, vdim, block_size, 
 
 
 def prefill(q, cache, out, *, block_table, seq_lens, q_start, num_reqs, tile_req, tile_q0, H, G, kw, vdim,
-            block_size, bias=None, null_entry=False, any_size=False, scale=1.0, chunk=0, grouped=False):
-    """Portions of prompts; ``tile_req`` / ``tile_q0`` list their 128-row query tiles."""
+            block_size, bias=None, null_entry=False, any_size=False, scale=1.0, chunk=0, window=0, maps=1, grouped=False,
+            gate=None, values_in_keys=False, rows=None):
+    """Portions of prompts; ``tile_req`` / ``tile_q0`` list their 128-row query tiles. ``rows``
+    (:class:`SplitRows`, tensor-core kernel only) stands for ``cache``."""
     _declare()
-    a = _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry, scale, chunk, grouped)
+    a = _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry, scale, chunk, window, maps,
+              grouped, gate, values_in_keys, rows)
     a.q_start, a.num_reqs = ptr(q_start), num_reqs
     a.tile_req, a.tile_q0, a.num_tiles = ptr(tile_req), ptr(tile_q0), tile_req.numel()
     check(lib().b200_bias_attn_prefill(ctypes.byref(a), int(any_size), stream_ptr()), "bias_attn_prefill")
     return out
 
 
-def kernel_kind(phase: str, q, cache, *, H, G, kw, vdim, block_size, scale=1.0, chunk=0, grouped=False) -> str:
+def kernel_kind(phase: str, q, cache, *, H, G, kw, vdim, block_size, scale=1.0, chunk=0, window=0, maps=1,
+                grouped=False) -> str:
     """Which kernel serves a shape: "tensor-core" or "any-size"."""
     _declare()
     a = BiasAttnArgs()
     a.q, a.ldq, a.out, a.ldo, a.cache = ptr(q), q.stride(0), ptr(q), H * vdim, ptr(cache)
     a.H, a.G, a.kw, a.vdim, a.block_size = H, G, kw, vdim, block_size
-    a.scale, a.chunk, a.grouped = scale, chunk, int(grouped)
+    a.scale, a.chunk, a.window, a.maps, a.grouped = scale, chunk, window, maps, int(grouped)
     a.f32, a.tile_req = int(q.dtype == torch.float32), ptr(q)
     return {2: "tensor-core", 1: "any-size"}[lib().b200_bias_attn_kernel(ctypes.byref(a), int(phase == "prefill"))]
 
@@ -173,38 +212,55 @@ def ref_head_mix_kv(qkv, mix, q_out, slots, cache, *, H, G, dim, vdim, block_siz
     vals[b, o] = qkv[ok, H * dim + kw: H * dim + kw + vw].to(cache.dtype)
 
 
-def ref_rotate_kv(qkv, positions, table, rot, eps, q_out, slots, cache, *, H, G, D, V, dim, block_size):
-    T, half = qkv.shape[0], rot // 2
+def ref_rotate_kv(qkv, positions, table, rot, eps, q_out, slots, cache, *, H, G, D, V, dim, block_size, q_w=None, k_w=None,
+                  value_heads=None):
+    T, half, GV = qkv.shape[0], rot // 2, G if value_heads is None else value_heads
     x = qkv[:, : (H + G) * D].float().view(T, H + G, D).clone()
+
+    def norm(x):
+        return x / torch.sqrt((x * x).sum(-1, keepdim=True) / dim + eps)
+    if q_w is not None:
+        x = norm(x) * torch.cat([q_w.expand(H, D), k_w.expand(G, D)], 0)
     if table is not None:
         cs = table[positions.long()]
         c, s = cs[:, None, :half], cs[:, None, half:]
         u, v = x[..., :half].clone(), x[..., half:rot].clone()
         x[..., :half], x[..., half:rot] = u * c - v * s, v * c + u * s
-    x = x / torch.sqrt((x * x).sum(-1, keepdim=True) / dim + eps)
+    if q_w is None:
+        x = norm(x)
     q_out[:T, : H * D] = x[:, :H].reshape(T, -1).to(q_out.dtype)
     if G:
         keys, vals = page_views(cache, block_size, G * D)
         ok = slots >= 0
         b, o = slots[ok] // block_size, slots[ok] % block_size
         keys[b, o] = x[ok, H:].reshape(-1, G * D).to(cache.dtype)
-        vals[b, o] = qkv[ok, (H + G) * D: (H + G) * D + G * V].to(cache.dtype)
+        vals[b, o] = qkv[ok, (H + G) * D: (H + G) * D + GV * V].to(cache.dtype)
+
+
+def ref_diff_combine(maps, out, *, H, V, vdim, lam, eps, scale):
+    T = maps.shape[0]
+    x = maps[:, : H * 2 * V].float().view(T, H, 2, V)
+    o = x[:, :, 0] - lam * x[:, :, 1]
+    o = o / torch.sqrt((o * o).sum(-1, keepdim=True) / vdim + eps) * scale
+    out[:T, : H * V] = o.reshape(T, -1).to(out.dtype)
+    return out
 
 
 def ref_bias_attention(q, cache, out, *, block_table, seq_lens, q_start, H, G, kw, vdim, block_size, bias=None,
-                       null_entry=False, scale=1.0, chunk=0, grouped=False):
+                       null_entry=False, scale=1.0, chunk=0, window=0, maps=1, grouped=False, gate=None, values_in_keys=False):
     keys, vals = page_views(cache, block_size, kw)
-    qs = q_start.tolist()
+    qs, R = q_start.tolist(), H // G
     for r, sl in enumerate(seq_lens.tolist()):
         t0, t1 = qs[r], qs[r + 1]
         if t1 <= t0 or sl <= 0:
             continue
         blocks = block_table[r, : (sl + block_size - 1) // block_size].long()
         k = keys[blocks].reshape(-1, kw)[:sl].float()
-        v = vals[blocks].reshape(-1, G, vdim)[:sl].float().repeat_interleave(H // G, 1)
-        if grouped:
-            kg = k.view(sl, G, kw // G).repeat_interleave(H // G, 1)
-            s = torch.einsum("qhd,khd->hqk", q[t0:t1, : H * kw // G].float().view(t1 - t0, H, kw // G), kg) * scale
+        v = k[:, :vdim].unsqueeze(1) if values_in_keys else vals[blocks].reshape(-1, G, vdim)[:sl].float()
+        v = v.repeat_interleave(R, 1)
+        if grouped:                          # (head h reads map h % maps of its group)
+            kg = k.view(sl, G, 1, maps, -1).expand(sl, G, R // maps, maps, kw // G // maps).reshape(sl, H, -1)
+            s = torch.einsum("qhd,khd->hqk", q[t0:t1, : H * kg.shape[-1]].float().view(t1 - t0, H, -1), kg) * scale
         else:
             s = torch.einsum("qhd,kd->hqk", q[t0:t1, : H * kw].float().view(t1 - t0, H, kw), k) * scale
         at, key = torch.arange(sl - (t1 - t0), sl)[:, None], torch.arange(sl)[None]
@@ -214,11 +270,16 @@ def ref_bias_attention(q, cache, out, *, block_table, seq_lens, q_start, H, G, k
         hidden = dist < 0
         if chunk:
             hidden = hidden | (at // chunk != key // chunk)
+        if window:
+            hidden = hidden | (dist >= window)
         s = s.masked_fill(hidden, -math.inf)
         m = s.amax(-1, keepdim=True)
         if null_entry:
             m = m.clamp(min=0)
         e = torch.exp(s - m)
         den = e.sum(-1, keepdim=True) + (torch.exp(-m) if null_entry else 0.0)
-        out[t0:t1, : H * vdim] = torch.einsum("hqk,khd->qhd", e / den, v).reshape(t1 - t0, H * vdim).to(out.dtype)
+        o = torch.einsum("hqk,khd->qhd", e / den, v)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[t0:t1, :H].float())[..., None]
+        out[t0:t1, : H * vdim] = o.reshape(t1 - t0, H * vdim).to(out.dtype)
     return out

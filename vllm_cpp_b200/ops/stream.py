@@ -17,7 +17,7 @@ class StreamNormArgs(ctypes.Structure):
                 ("norm_w", _P), ("post_w", _P), ("ident", _P), ("out", _P), ("lds", _L), ("lda", _L), ("ldy", _L),
                 ("ldi", _L), ("ldo", _L), ("vocab", _L),
                 ("T", _I), ("width", _I), ("cols", _I), ("k", _I), ("f32", _I), ("a_f32", _I),
-                ("scale", _F), ("eps", _F), ("norm_offset", _F)]
+                ("scale", _F), ("eps", _F), ("norm_offset", _F), ("mult", _F)]
 
 
 class ClampedGate(ctypes.Structure):
@@ -36,14 +36,15 @@ def _declare():
     _lib.declare("b200_stream_norm", [ctypes.POINTER(StreamNormArgs), P], I)
     _lib.declare("b200_gated_act_f32", [P, I, P, I, I, I, I, P], I)
     _lib.declare("b200_gemm_f32", [P, I, P, I, P, I, P, I, I, I, P], I)
+    _lib.declare("b200_softcap_f32", [P, ctypes.c_longlong, _lib.F, P], I)
     lib()
     _declared = True
 
 
 def stream_norm(stream, norm_w, eps, out, *, width, ids=None, table=None, scale=1.0, a=None, y=None,
-                pair_pos=None, pair_w=None, norm_offset=1.0, post_w=None, ident=None):
-    """``stream`` [T, cols] fp32 starts as ``table[ids] * scale`` or takes ``+= a + sum_j w_j
-    y[pair_pos[:, j]]`` (``ident`` rows where ``pair_pos`` < 0; may be ``out``), with ``post_w`` that sum
+                pair_pos=None, pair_w=None, norm_offset=1.0, post_w=None, ident=None, mult=1.0):
+    """``stream`` [T, cols] fp32 starts as ``table[ids] * scale`` or takes ``+= mult (a + sum_j w_j
+    y[pair_pos[:, j]])`` (``ident`` rows where ``pair_pos`` < 0; may be ``out``), with ``post_w`` that sum
     over its rms times (post_w + norm_offset); ``out`` = stream / rms(stream) * (norm_w + norm_offset).
     ``cols`` is ``width`` padded with zeros."""
     _declare()
@@ -60,7 +61,7 @@ def stream_norm(stream, norm_w, eps, out, *, width, ids=None, table=None, scale=
     s.T, s.width, s.cols, s.k = T, width, cols, pair_pos.shape[1] if pair_pos is not None else 0
     s.f32 = int(out.dtype == torch.float32)
     s.a_f32 = int(a is not None and a.dtype == torch.float32)
-    s.scale, s.eps, s.norm_offset = scale, eps, norm_offset
+    s.scale, s.eps, s.norm_offset, s.mult = scale, eps, norm_offset, mult
     check(lib().b200_stream_norm(ctypes.byref(s), stream_ptr()), "stream_norm")
     return out
 
@@ -77,6 +78,13 @@ def gemm_f32(a, w, bias=None, out=None):
     return out
 
 
+def softcap_f32(x, cap):
+    """cap * tanh(x / cap) in place over fp32 rows [n, cols]."""
+    _declare()
+    check(lib().b200_softcap_f32(ptr(x), x.numel(), cap, stream_ptr()), "softcap_f32")
+    return x
+
+
 def gated_act_f32(gate_up, kind, out):
     """act(gate) * up of fp32 rows ``[gate | up]``; ``kind`` as in ``ops.act_and_mul``."""
     _declare()
@@ -88,7 +96,7 @@ def gated_act_f32(gate_up, kind, out):
 
 # ------------------------------------------------------------------------------ restatements
 def ref_stream_norm(stream, norm_w, eps, out, *, width, ids=None, table=None, scale=1.0, a=None, y=None,
-                    pair_pos=None, pair_w=None, norm_offset=1.0, post_w=None, ident=None):
+                    pair_pos=None, pair_w=None, norm_offset=1.0, post_w=None, ident=None, mult=1.0):
     if ids is not None:
         stream.copy_(table[ids].float() * scale)
     else:
@@ -103,7 +111,7 @@ def ref_stream_norm(stream, norm_w, eps, out, *, width, ids=None, table=None, sc
                 d += yj * pair_w[:, j, None] if pair_w is not None else yj
         if post_w is not None:
             d = d / torch.sqrt((d * d).sum(-1, keepdim=True) / width + eps) * (post_w + norm_offset)
-        stream += d
+        stream += mult * d
     inv = 1.0 / torch.sqrt((stream * stream).sum(-1, keepdim=True) / width + eps)
     out.copy_(stream * inv * (norm_w + norm_offset))
     return out
