@@ -197,7 +197,80 @@ typedef struct B200BiasAttn {
   int bias_len, null_entry, f32, splits, num_tiles;
   int grouped, chunk;
   float scale;
+  int window;                  // > 0: a query sees itself and the window - 1 positions before it
+  int maps;                    // > 1 (grouped): a group's key columns hold that many keys, head h meets the h % maps-th
+  int values_in_keys;          // values are the first vdim columns of the key rows (any-size kernel)
+  int shared;                  // width of shared_keys in a query row
+  const void* gate;            // element (row, head): the output times its sigmoid (prefill and any-size kernels)
+  long long ldg;
+  // prefill on the tensor cores, instead of cache: rows of keys and values, block_size consecutive rows to a
+  // page, and key columns that every head shares (query rows: own columns in whole 64-wide chunks, then these)
+  const void* keys;
+  const void* values;
+  const void* shared_keys;
+  long long ldk, ldv, lds;
 } B200BiasAttn;
+
+// Latent attention (latent.cu): norms of the query and key latents, rotation of the shared key part, cache rows
+// [latent (rankp) | rotated part]. down rows: query latent | key latent at kv_col | rotated part at rot_col.
+typedef struct B200LatentPrep {
+  const void* down;
+  long long ldd;
+  const void* positions;
+  const float* cos_sin;        // [positions][cos rot / 2 | sin rot / 2]
+  const float* q_norm;
+  const float* kv_norm;
+  void* cq;
+  long long ldcq;
+  const void* slots;
+  void* cache;
+  int T, q_rank, rank, rot, kv_col, rot_col, rankp, row, f32;
+  float eps;
+} B200LatentPrep;
+
+// The rows of an engine step: nd decode rows (one per request), then the prompt portions listed by q_start /
+// tile_req / tile_q0 (128-row tiles, relative to the portions).
+typedef struct B200Rows {
+  const int* seq_lens;
+  const int* slots;
+  const int* q_start;
+  const int* tile_req;
+  const int* tile_q0;
+  int nd, num_prefills, num_tiles, T;
+} B200Rows;
+
+// Causal convolution per channel with carried inputs (rglru.cu). act: 0 none, 1 SiLU.
+typedef struct B200ShortConv {
+  B200Rows rows;
+  const void* x;
+  long long ldx;
+  const float* w;              // [taps][C], the last row is the current token's
+  const float* bias;           // [C] or null
+  void* state;                 // [slots][taps - 1][C]
+  void* out;
+  long long ldo;
+  int C, taps, act, f32;
+} B200ShortConv;
+
+// Real-gated linear recurrent unit (rglru.cu), see rglru.py.
+typedef struct B200Rglru {
+  B200Rows rows;
+  const void* u;
+  long long ldu;
+  const void* y;
+  long long ldy;
+  const void* gates;           // [blocks][2][M][B]
+  const float* gate_bias;      // [2][C]
+  const float* rate;           // [C]
+  float* state;                // [slots][C]
+  void* out;
+  long long ldo;
+  float* summary;              // [3][B200_RGLRU_SLICES][C]
+  float* a;                    // any-size kernels: [T][C]
+  float* b;
+  int blocks, B, M, slices, f32;
+} B200Rglru;
+#define B200_RGLRU_SLICES 64
 
 // Gated delta rule (delta.cu, delta_chunk.cu). Rows: nd decode rows, then the prompt portions listed by
 // q_start / tile_req / tile_q0 (relative to the portions). proj rows: q heads | k heads (G of D each) |
@@ -236,7 +309,7 @@ typedef struct B200Delta {
 
 // fp32 residual stream update + RMSNorm in one pass per row (stream.cu):
 //   start:  stream = table[ids] * scale        (ids non-null)
-//   else:   stream += a + sum_j w_j y[pair_pos[j]]   (a, y each optional; pair_w null: w = 1)
+//   else:   stream += mult (a + sum_j w_j y[pair_pos[j]])   (a, y each optional; pair_w null: w = 1)
 // post_w: the update is first divided by its own rms and multiplied by post_w + norm_offset. ident: rows that
 // stand for y where pair_pos < 0 (experts that return their input; may be ``out``).
 //   out = stream / rms(stream) * (norm_w + norm_offset)
@@ -256,7 +329,7 @@ typedef struct B200StreamNorm {
   long long lds, lda, ldy, ldi, ldo, vocab;
   int T, width, cols, k;
   int f32, a_f32;              // element type of table / y / out, and of a
-  float scale, eps, norm_offset;
+  float scale, eps, norm_offset, mult;
 } B200StreamNorm;
 
 // Activation of a gated pair with clamps: g = min(gate, limit), u = clamp(up, -limit, limit),
@@ -299,7 +372,8 @@ int b200_merge_attn_states(const void* a, const void* lse_a, const void* b, cons
 int b200_attn_decode_tc(const void* q, int ldq, void* out, int ldo, const void* kv_cache, int64_t num_blocks, int block_size, int Hq, int Hkv, int D, const void* block_table, int max_blocks, const void* seq_lens, int B, float scale, float softcap, int window, int splits, void* tmp_o, void* tmp_lse, cudaStream_t stream);
 // ---- attn_bias.cu
 int b200_head_mix_kv(const void* qkv, long long ld, const void* mix, void* q_out, long long ldq, const void* slots, void* cache, int H, int G, int dim, int vdim, int block_size, int T, int f32, cudaStream_t stream);
-int b200_rotate_kv(const void* qkv, long long ld, const void* positions, const void* cos_sin, int rot, float eps, void* q_out, long long ldq, const void* slots, void* cache, int H, int G, int D, int V, int dim, int block_size, int T, int f32, cudaStream_t stream);
+int b200_rotate_kv(const void* qkv, long long ld, const void* positions, const void* cos_sin, int rot, float eps, const float* q_w, const float* k_w, void* q_out, long long ldq, const void* slots, void* cache, int H, int G, int GV, int D, int V, int dim, int block_size, int T, int f32, cudaStream_t stream);
+int b200_diff_combine(const void* maps, long long ldm, void* out, long long ldo, int H, int V, int vdim, int T, float lam, float eps, float scale, int f32, cudaStream_t stream);
 int b200_bias_attn_kernel(const B200BiasAttn* a, int phase);
 int b200_bias_attn_decode(const B200BiasAttn* a, int any_size, cudaStream_t stream);
 int b200_bias_attn_prefill(const B200BiasAttn* a, int any_size, cudaStream_t stream);
@@ -349,10 +423,20 @@ void b200_tp_layers_abi(int* out2);
 int b200_dense_layers_tp(const B200DenseLayerWeights* w, int num_layers, const B200DenseStep* s, const B200TpLayers* c, cudaStream_t stream);
 // ---- mla.cu
 int b200_mla_decode(const void* qabs, void* out, int ldo, const void* cache, int64_t num_blocks, int block_size, int Hq, const void* block_table, int max_blocks, const void* seq_lens, int B, float scale, int splits, void* tmp_o, void* tmp_lse, cudaStream_t stream);
+int b200_latent_decode(const void* qabs, void* out, int ldo, const void* cache, int64_t num_blocks, int block_size, int H, int rank, int rot, const void* block_table, int max_blocks, const void* seq_lens, int B, float scale, int window, const void* gate, long long ldg, int splits, void* tmp_o, void* tmp_lse, cudaStream_t stream);
 int b200_mla_gather_latent(const void* cache, const void* block_table, int max_blocks, const void* seq_lens, const void* dense_base, int block_size, void* dense, int num_reqs, int max_req_blocks, cudaStream_t stream);
 int b200_mla_assemble_kv(const void* kvb, const void* dense, void* cache, int N, int H, int block_size, cudaStream_t stream);
 int b200_mla_pad_q(const void* q, long ldq, void* out, int T, int H, cudaStream_t stream);
 int b200_mla_copy_qpe(const void* q, long ldq, void* qabs, int T, int H, cudaStream_t stream);
+// ---- latent.cu
+int b200_latent_prepare(const B200LatentPrep* a, cudaStream_t stream);
+int b200_latent_queries(void* q, long long ldq, const void* positions, const float* cos_sin, int H, int qn, int qw, int rot, void* qabs, int rankp, int row, int absorbed, int T, int f32, cudaStream_t stream);
+int b200_latent_gather(const void* cache, const void* block_table, int max_blocks, const void* seq_lens, const void* first, const void* base, int block_size, int row_bytes, void* dense, int num_reqs, int max_pages, cudaStream_t stream);
+// ---- rglru.cu
+int b200_short_conv(const B200ShortConv* a, cudaStream_t stream);
+int b200_rglru_fits(const B200Rglru* a);
+int b200_rglru_slices(const B200Rglru* a);
+int b200_rglru(const B200Rglru* a, int any_size, cudaStream_t stream);
 // ---- moe.cu
 int b200_moe_router_topk(const void* logits_f32, int ld, int T, int E, int k, int renorm, int scoring, const void* e_bias, int n_group, int topk_group, int group_best, float routed_scale, void* topk_ids, void* topk_w, cudaStream_t stream);
 int b200_moe_sort(const void* topk_ids, int T, int k, int e0, int e1, void* meta, void* sorted_token, void* pair_pos, void* chunk_expert, void* chunk_row0, void* chunk_n, int max_chunks, cudaStream_t stream);
@@ -376,6 +460,8 @@ int b200_gather_rows(const void* x, const void* idx, void* out, int n_out, int n
 // ---- stream.cu
 int b200_stream_norm(const B200StreamNorm* a, cudaStream_t stream);
 int b200_gemm_f32(const void* A, int lda, const void* W, int ldw, void* out, int ldo, const void* bias, int M, int N, int K, cudaStream_t stream);
+int b200_gemm_f32_batched(const void* A, int lda, int a_batch, const void* W, int ldw, void* out, int ldo, long long out_batch, int M, int N, int K, int batch, cudaStream_t stream);
+int b200_softcap_f32(void* x, long long n, float cap, cudaStream_t stream);
 int b200_moe_grouped_gemm_f32(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, cudaStream_t stream);
 int b200_gated_act_f32(const void* gate_up, int ldg, void* out, int ldo, int T, int I, int kind, cudaStream_t stream);
 int b200_clamped_gate_f32(const void* gate_up, void* out, const void* meta, int E, int max_rows, int I, const B200ClampedGate* act, cudaStream_t stream);

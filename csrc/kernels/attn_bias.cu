@@ -1,6 +1,7 @@
 // Attention over a paged cache with separate key and value widths: scores may carry a per-head distance
-// bias and a mix of the heads, the softmax a null entry, and a query may be limited to its own chunk of
-// positions.
+// bias and a mix of the heads, the softmax a null entry, and a query may be limited to its own chunk or
+// window of positions. Grouped heads may come in maps: a group then holds that many keys per token beside one
+// value, and head h meets the h % maps-th.
 //
 //   s[h, i, j] = scale sum_g M[h, g] (q_g(i) . k_g(j)) + bias[h, min(i - j, L - 1)]
 //   p[h, i, j] = exp(s) / (null + sum_j exp(s)),   o[h, i] = sum_j p[h, i, j] v_{h / R}(j)
@@ -208,14 +209,23 @@ struct BiasAttnParams {
   const int32_t* tile_q0;
   int k_slots, v_slots, q_stream;
   int* status;
+  int window, maps, values_in_keys;
+  int own_chunks;           // 64-wide chunks of a query row that meet the head's own key columns
+  const void* gate;         // [rows, ldg]
+  long long ldg;
 };
 
-// ------------------------------------------------------------------------------- any-size attention
-static constexpr int kAnyHeads = 4;
-static constexpr int kAnyKeys = 128;
-static constexpr int kAnyAcc = 16;     // outputs per thread: kAnyHeads * vdim <= 128 * kAnyAcc
+// First position a query at pos sees.
+__device__ __forceinline__ int first_key(const BiasAttnParams& p, int pos) {
+  return p.chunk > 0 ? pos / p.chunk * p.chunk : p.window > 0 ? max(pos - p.window + 1, 0) : 0;
+}
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 
-template <typename T>
+// ------------------------------------------------------------------------------- any-size attention
+static constexpr int kAnyKeys = 128;
+static constexpr int kAnyAcc = 16;     // outputs per thread: heads * vdim <= 128 * kAnyAcc
+
+template <typename T, int kAnyHeads>
 __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
   extern __shared__ float any_smem[];
   float* sq = any_smem;                                  // [kAnyHeads][qw]
@@ -226,7 +236,7 @@ __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
   pdl_launch_dependents();
   const int row = blockIdx.x, h0 = blockIdx.y * kAnyHeads, nh = min(kAnyHeads, p.H - h0);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int vw = p.G * p.vdim, R = p.H / p.G;
+  const int vw = p.values_in_keys ? 0 : p.G * p.vdim, R = p.H / p.G;
   int req = row, pos;
   if (p.q_start) {
     int lo = 0, hi = p.num_reqs - 1;                     // last request whose first row is <= row
@@ -248,7 +258,7 @@ __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
   for (int a = 0; a < kAnyAcc; ++a) acc[a] = 0.f;
   // warp w owns the softmax state of head h0 + w
   float m = p.null_entry ? 0.f : -INFINITY, l = p.null_entry ? 1.f : 0.f;
-  for (int base = p.chunk > 0 ? pos / p.chunk * p.chunk : 0; base <= pos; base += kAnyKeys) {
+  for (int base = first_key(p, pos); base <= pos; base += kAnyKeys) {
     const int key = base + tid;
     const bool valid = key <= pos;
     __syncthreads();
@@ -256,7 +266,7 @@ __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
       const long long page = (long long)bt[key / p.block_size] * p.block_size * (p.kw + vw);
       const int off = key % p.block_size;
       krow[tid] = page + (long long)off * p.kw;
-      vrow[tid] = page + (long long)p.block_size * p.kw + (long long)off * vw;
+      vrow[tid] = p.values_in_keys ? krow[tid] : page + (long long)p.block_size * p.kw + (long long)off * vw;
       float s[kAnyHeads];
 #pragma unroll
       for (int h = 0; h < kAnyHeads; ++h) s[h] = 0.f;
@@ -265,7 +275,7 @@ __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
 #pragma unroll
         for (int h = 0; h < kAnyHeads; ++h) {
           if (h >= nh) break;
-          const T* kg = k + (size_t)((h0 + h) / R) * p.qw;
+          const T* kg = k + (size_t)((h0 + h) / R * p.maps + (h0 + h) % p.maps) * p.qw;
           for (int i = 0; i < p.qw; ++i) s[h] = fmaf(sq[h * p.qw + i], to_f(kg[i]), s[h]);
         }
       } else {
@@ -326,7 +336,9 @@ __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
     const int e = tid + a * 128;
     if (e < nh * p.vdim) {
       const float ls = s_l[e / p.vdim];
-      o[e] = from_f<T>(ls > 0.f ? acc[a] / ls : 0.f);
+      float x = ls > 0.f ? acc[a] / ls : 0.f;
+      if (p.gate) x *= sigmoid_f(to_f(reinterpret_cast<const T*>(p.gate)[(size_t)row * p.ldg + h0 + e / p.vdim]));
+      o[e] = from_f<T>(x);
     }
   }
 }
@@ -748,7 +760,8 @@ __device__ __forceinline__ void pair_sync(int quarter) {             // the two 
 
 __global__ void __launch_bounds__(kPrefillThreads, 1)
     bias_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                             const __grid_constant__ CUtensorMap tmV, BiasAttnParams p) {
+                             const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmS,
+                             BiasAttnParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int nkc = (p.qw + 63) / 64, nvc = (p.vdim + 63) / 64;
@@ -764,10 +777,10 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
   const int q_begin = p.q_start[req], q_len = p.q_start[req + 1] - q_begin;
   const int seq_len = p.seq_lens[req], ctx_off = seq_len - q_len;
   const int rows = min(kBQ, q_len - q0);
-  // first key tile: that of the chunk start of the first row
-  const int lo_tile = p.chunk > 0 ? (ctx_off + q0) / p.chunk * p.chunk / kBKeys : 0;
+  // first key tile: that of the first row's first key
+  const int lo_tile = first_key(p, ctx_off + q0) / kBKeys;
   const int ntiles = (ctx_off + q0 + rows - 1) / kBKeys + 1 - lo_tile;
-  const int k_col = p.qw < p.kw ? hkv * p.qw : 0;
+  const int k_col = p.own_chunks < nkc ? hkv * (p.kw / p.G) : p.qw < p.kw ? (hkv * p.maps + h % p.maps) * p.qw : 0;
   // TMEM columns: S buffers (128 each), then O, then two P buffers (64 each)
   const int s_bufs = p.vdim > 128 ? 1 : 2;
   const int o_cols = p.vdim > 128 ? 256 : 128;
@@ -830,7 +843,11 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
               tma_load_2d(dst + kChunkBytes, &tmQ, &bars->k_full[sl], h * p.qw + c * 64, q_begin + q0);
           }
           __syncwarp();
-          if (lane < loads) tma_load_3d(dst + lane * rpl * 128, &tmK, &bars->k_full[sl], k_col + c * 64, row, blk);
+          if (lane < loads) {
+            const bool own = c < p.own_chunks;
+            tma_load_3d(dst + lane * rpl * 128, own ? &tmK : &tmS, &bars->k_full[sl],
+                        own ? k_col + c * 64 : (c - p.own_chunks) * 64, row, blk);
+          }
           if (++sl == p.k_slots) { sl = 0; ph ^= 1; }
         }
       }
@@ -903,9 +920,9 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
     const int quarter = warp & 3, half = (warp - 2) >> 2, r = quarter * 32 + lane;
     const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
     const int q_pos = ctx_off + q0 + r, hi = min(q_pos, seq_len - 1);
-    const int lo = p.chunk > 0 ? q_pos / p.chunk * p.chunk : 0;
+    const int lo = first_key(p, q_pos);
     const int warp_pos0 = ctx_off + q0 + quarter * 32;       // position of the warp's first row
-    const int warp_lo = p.chunk > 0 ? (warp_pos0 + 31) / p.chunk * p.chunk : 0;   // largest lo of its rows
+    const int warp_lo = first_key(p, warp_pos0 + 31);        // largest lo of its rows
     const int key0 = half * 64;                              // this thread's keys inside a tile
     const float scale2 = p.scale * kLog2e;
     const float* bias = p.bias ? p.bias + (size_t)h * p.bias_len : nullptr;
@@ -1025,7 +1042,9 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
     if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->o_full, 0, p.status));
     if (ok) {
       tc_fence_after_sync();
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (p.gate && r < rows)
+        inv *= sigmoid_f(to_f(reinterpret_cast<const __nv_bfloat16*>(p.gate)[(size_t)(q_begin + q0 + r) * p.ldg + h]));
       __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(q_begin + q0 + r) * p.ldo + (size_t)h * p.vdim;
       for (int c = half; c < vcols; c += 2) {
         uint32_t rr[32];
@@ -1057,7 +1076,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
 // Shapes the decode kernel serves. tk: keys per tile; cls: register class (0: 8 output tiles, 2 query
 // chunks and 4 heads per warp, 1: 16 tiles, 8 heads, queries in shared memory).
 static bool decode_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem, int& tk, int& cls) {
-  if (a->grouped || a->chunk || a->scale != 1.f) return false;           // (attn_grouped.cu)
+  if (a->grouped || a->chunk || a->window || a->gate || a->scale != 1.f) return false;           // (attn_grouped.cu)
   if (a->f32 || (a->kw & 7) || (a->vdim & 7) || (a->ldq & 7) || (a->ldo & 1)) return false;
   if (((uintptr_t)a->q | (uintptr_t)a->cache) & 15) return false;
   const int R = a->H / a->G, nkc = (a->kw + 63) / 64;
@@ -1097,12 +1116,14 @@ static bool decode_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem, 
 
 static bool prefill_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem) {
   if (a->f32 || !a->tile_req || (a->kw & 7) || (a->vdim & 7) || a->vdim > 256 || (a->ldq & 7) || (a->ldo & 7)) return false;
-  if (((uintptr_t)a->q | (uintptr_t)a->cache | (uintptr_t)a->out) & 15) return false;
-  const int bs = a->block_size;
+  if (((uintptr_t)a->q | (uintptr_t)a->cache | (uintptr_t)a->out) & 15 || a->values_in_keys) return false;
+  if (((uintptr_t)a->keys | (uintptr_t)a->values | (uintptr_t)a->shared_keys) & 15 || (a->ldk | a->ldv | a->lds) & 7) return false;
+  const int bs = a->block_size, maps = a->maps > 1 ? a->maps : 1;
   if (bs < 8 || (bs & 7) || (bs < kBKeys && kBKeys % bs) || (bs > kBKeys && bs % kBKeys)) return false;
   // a group's columns start on a 16-byte boundary and the last product of 16 reads none of the next group
-  if (a->grouped && (a->kw / a->G & 15)) return false;
-  const int nkc = ((a->grouped ? a->kw / a->G : a->kw) + 63) / 64, nvc = (a->vdim + 63) / 64;
+  if (a->grouped && (a->kw / a->G / maps & 15)) return false;
+  if (a->shared && (!a->shared_keys || (a->shared & 15) || maps > 1 || !a->grouped)) return false;
+  const int nkc = ((a->grouped ? a->kw / a->G / maps : a->kw) + 63) / 64 + (a->shared + 63) / 64, nvc = (a->vdim + 63) / 64;
   const int limit = 227 * 1024, fixed = (int)sizeof(BiasPrefillBars) + 1024;
   // the query tile stays in shared memory if enough of the key ring fits beside it
   for (p.q_stream = 0; p.q_stream < 2; ++p.q_stream) {
@@ -1162,6 +1183,17 @@ static bool page_maps(const B200BiasAttn* a, int keys, CUtensorMap* mk, CUtensor
   return true;
 }
 
+// Tensor maps of key, value and shared rows outside a page tensor.
+static bool split_maps(const B200BiasAttn* a, int keys, CUtensorMap* mk, CUtensorMap* mv, CUtensorMap* ms) {
+  const uint32_t rows = a->block_size < keys ? a->block_size : keys;
+  auto map = [&](CUtensorMap* m, const void* base, long long cols, long long ld) {
+    return encode_tmap_3d(m, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, cols, a->block_size, a->num_blocks, (uint64_t)ld * 2,
+                          (uint64_t)ld * 2 * a->block_size, 64, rows, 1, CU_TENSOR_MAP_SWIZZLE_128B);
+  };
+  return map(mk, a->keys, a->kw, a->ldk) && map(mv, a->values, (long long)a->G * a->vdim, a->ldv) &&
+         (!a->shared || map(ms, a->shared_keys, a->shared, a->lds));
+}
+
 static BiasAttnParams common_params(const B200BiasAttn* a) {
   BiasAttnParams p{};
   p.q = a->q; p.ldq = a->ldq; p.out = a->out; p.ldo = a->ldo; p.cache = a->cache;
@@ -1169,7 +1201,11 @@ static BiasAttnParams common_params(const B200BiasAttn* a) {
   p.seq_lens = (const int32_t*)a->seq_lens; p.q_start = (const int32_t*)a->q_start;
   p.num_reqs = a->num_reqs; p.rows = a->rows;
   p.H = a->H; p.G = a->G; p.kw = a->kw; p.vdim = a->vdim; p.block_size = a->block_size;
-  p.qw = a->grouped ? a->kw / a->G : a->kw; p.chunk = a->chunk; p.scale = a->scale;
+  p.maps = a->maps > 1 ? a->maps : 1; p.window = a->window; p.values_in_keys = a->values_in_keys;
+  p.gate = a->gate; p.ldg = a->ldg;
+  p.qw = a->grouped ? a->kw / a->G / p.maps : a->kw; p.chunk = a->chunk; p.scale = a->scale;
+  p.own_chunks = (p.qw + 63) / 64;
+  if (a->shared) p.qw = p.own_chunks * 64 + a->shared;
   p.bias = (const float*)a->bias; p.bias_len = a->bias_len; p.null_entry = a->null_entry;
   p.splits = a->splits < 1 ? 1 : a->splits; p.tmp_o = (float*)a->tmp_o; p.tmp_lse = (float*)a->tmp_lse;
   p.tile_req = (const int32_t*)a->tile_req; p.tile_q0 = (const int32_t*)a->tile_q0;
@@ -1177,15 +1213,21 @@ static BiasAttnParams common_params(const B200BiasAttn* a) {
   return p;
 }
 
-template <typename T>
+template <typename T, int kAnyHeads>
 static int launch_any(const BiasAttnParams& p, cudaStream_t stream) {
   if ((long)kAnyHeads * p.vdim > 128l * kAnyAcc) return -4;
   const size_t smem = (size_t)kAnyHeads * (p.qw + kAnyKeys) * 4;
   if (smem > 200 * 1024) return -4;
   static PerDeviceOnce once;
-  if (once.first()) cudaFuncSetAttribute(bias_attn_any_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+  if (once.first())
+    cudaFuncSetAttribute(bias_attn_any_kernel<T, kAnyHeads>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
   dim3 grid(p.rows, (p.H + kAnyHeads - 1) / kAnyHeads);
-  return launch_pdl(bias_attn_any_kernel<T>, grid, dim3(128), smem, stream, p) == cudaSuccess ? 0 : -2;
+  return launch_pdl(bias_attn_any_kernel<T, kAnyHeads>, grid, dim3(128), smem, stream, p) == cudaSuccess ? 0 : -2;
+}
+template <typename T>
+static int launch_any(const BiasAttnParams& p, cudaStream_t stream) {
+  return 4l * p.vdim <= 128l * kAnyAcc && 16l * (p.qw + kAnyKeys) <= 200 * 1024 ? launch_any<T, 4>(p, stream)
+                                                                                : launch_any<T, 1>(p, stream);
 }
 
 template <int TK, int MAXI, int CPW, int HPW>
@@ -1249,7 +1291,9 @@ static int launch_mix_vec(const MixParams& p, cudaStream_t stream) {
 
 static bool valid_args(const B200BiasAttn* a) {
   return a->H > 0 && a->G > 0 && a->H % a->G == 0 && a->kw > 0 && a->vdim > 0 && a->block_size > 0 &&
-         (!a->bias || a->bias_len > 0) && (!a->grouped || a->kw % a->G == 0) && a->chunk >= 0;
+         (!a->bias || a->bias_len > 0) && (!a->grouped || a->kw % a->G == 0) && a->chunk >= 0 &&
+         a->window >= 0 && (a->maps <= 1 || (a->grouped && a->kw / a->G % a->maps == 0 && a->H / a->G % a->maps == 0)) &&
+         (!a->values_in_keys || (a->G == 1 && a->vdim <= a->kw));
 }
 
 }  // namespace b200
@@ -1308,17 +1352,21 @@ int b200_bias_attn_prefill(const B200BiasAttn* a, int any_size, cudaStream_t str
   if (!valid_args(a) || !a->q_start) return -1;
   BiasAttnParams p = common_params(a);
   size_t smem;
-  if (any_size || !prefill_plan(a, p, smem))
+  const bool split = a->keys != nullptr;
+  if (any_size || !prefill_plan(a, p, smem)) {
+    if (split || a->shared) return -4;
     return a->f32 ? launch_any<float>(p, stream) : launch_any<__nv_bfloat16>(p, stream);
+  }
   if (a->num_tiles <= 0) return 0;
-  CUtensorMap tmQ, tmK, tmV;
+  CUtensorMap tmQ, tmK, tmV, tmS;
   if (!encode_tmap_2d(&tmQ, a->q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)a->rows, (uint64_t)a->H * p.qw,
                       (uint64_t)a->ldq, kBQ, 64, CU_TENSOR_MAP_SWIZZLE_128B) ||
-      !page_maps(a, kBKeys, &tmK, &tmV))
+      !(split ? split_maps(a, kBKeys, &tmK, &tmV, &tmS) : page_maps(a, kBKeys, &tmK, &tmV)))
     return -3;
+  if (!a->shared) tmS = tmK;
   static PerDeviceOnce once;
   if (once.first()) cudaFuncSetAttribute(bias_attn_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
-  bias_attn_prefill_kernel<<<dim3(a->num_tiles, a->H), kPrefillThreads, smem, stream>>>(tmQ, tmK, tmV, p);
+  bias_attn_prefill_kernel<<<dim3(a->num_tiles, a->H), kPrefillThreads, smem, stream>>>(tmQ, tmK, tmV, tmS, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 

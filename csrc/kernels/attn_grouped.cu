@@ -1,7 +1,8 @@
 // Grouped-query attention over the pages of attn_bias.cu ([block_size][G * D] keys | [block_size][G * V]
 // values): query / key preparation and the decode kernel.
 //
-//   rotate_kv_kernel        rotation, unit norm, cache write
+//   rotate_kv_kernel        rotation and unit norm, or weighted norm and rotation; cache write
+//   diff_combine_kernel     difference of a head's two maps, its norm
 //   grouped_decode_kernel   bf16, one query row per request: a CTA takes one kv group and one split of the
 //                           visible keys, its four warps every fourth tile of 16 keys, each through its own
 //                           ring of cp.async stages (no block barrier before the final merge); the group's
@@ -15,9 +16,10 @@ typedef __nv_bfloat16 bf16;
 
 // ------------------------------------------------------------------- rotation, unit norm, cache write
 // Dimension i < rot / 2 of a q or k head is rotated with dimension i + rot / 2, then the head is divided by
-// its root mean square over dim; v is copied. One warp per (token, head).
+// its root mean square over dim (with weights: divided and weighted first, then rotated); v is copied. One warp
+// per (token, head).
 struct RotateParams {
-  const void* qkv;             // [T, ld]: q heads (H * D) | key heads (G * D) | value heads (G * V); G 0: q only
+  const void* qkv;             // [T, ld]: q heads (H * D) | key heads (G * D) | value heads (GV * V); G 0: q only
   long long ld;
   const int64_t* positions;
   const float* cos_sin;        // [positions][cos rot / 2 | sin rot / 2], null: no rotation
@@ -27,6 +29,9 @@ struct RotateParams {
   void* cache;
   int rot, H, G, D, V, dim, block_size, T;
   float eps;
+  int GV;
+  const float* q_w;            // [D], null: unit norm after the rotation
+  const float* k_w;
 };
 
 static constexpr int kRotMax = 512;
@@ -49,14 +54,14 @@ __global__ void __launch_bounds__(128) rotate_kv_kernel(RotateParams p) {
   extern __shared__ float rot_smem[];
   pdl_wait();
   pdl_launch_dependents();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, heads = p.H + 2 * p.G;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, heads = p.H + p.G + p.GV;
   const long long x = (long long)blockIdx.x * 4 + warp;
   if (x >= (long long)p.T * heads) return;
   const int t = (int)(x / heads), h = (int)(x % heads);
   const T* row = reinterpret_cast<const T*>(p.qkv) + (size_t)t * p.ld;
   const int64_t slot = h < p.H ? 0 : p.slots[t];
   if (slot < 0) return;
-  const int kw = p.G * p.D, vw = p.G * p.V;
+  const int kw = p.G * p.D, vw = p.GV * p.V;
   T* page = reinterpret_cast<T*>(p.cache);
   if (h >= p.H) page += slot / p.block_size * p.block_size * (int64_t)(kw + vw);
   const int off = (int)(slot % p.block_size);
@@ -71,6 +76,26 @@ __global__ void __launch_bounds__(128) rotate_kv_kernel(RotateParams p) {
   const T* src = row + (size_t)h * p.D;
   for (int i = lane * 4; i < p.D; i += 128) *reinterpret_cast<float4*>(b + i) = load4<T>(src + i);
   __syncwarp();
+  auto inv_rms = [&]() {
+    float ss = 0.f;
+    for (int i = lane * 4; i < p.D; i += 128) {
+      const float4 v = *reinterpret_cast<const float4*>(b + i);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    return 1.f / sqrtf(ss / (float)p.dim + p.eps);
+  };
+  float inv = 1.f;
+  if (p.q_w) {
+    const float* w = h < p.H ? p.q_w : p.k_w;
+    const float n = inv_rms();
+    for (int i = lane * 4; i < p.D; i += 128) {
+      const float4 v = *reinterpret_cast<const float4*>(b + i), g = *reinterpret_cast<const float4*>(w + i);
+      *reinterpret_cast<float4*>(b + i) = make_float4(v.x * n * g.x, v.y * n * g.y, v.z * n * g.z, v.w * n * g.w);
+    }
+    __syncwarp();
+  }
   const int half = p.rot / 2;
   if (p.cos_sin) {
     const float* cs = p.cos_sin + (size_t)p.positions[t] * p.rot;
@@ -81,14 +106,7 @@ __global__ void __launch_bounds__(128) rotate_kv_kernel(RotateParams p) {
     }
     __syncwarp();
   }
-  float ss = 0.f;
-  for (int i = lane * 4; i < p.D; i += 128) {
-    const float4 v = *reinterpret_cast<const float4*>(b + i);
-    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-  }
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  const float inv = 1.f / sqrtf(ss / (float)p.dim + p.eps);
+  if (!p.q_w) inv = inv_rms();
   T* dst = h < p.H ? reinterpret_cast<T*>(p.q_out) + (size_t)t * p.ldq + (size_t)h * p.D
                    : page + (int64_t)off * kw + (int64_t)(h - p.H) * p.D;
   for (int i = lane * 4; i < p.D; i += 128) {
@@ -106,7 +124,7 @@ struct GroupedDecode {
   const bf16* cache;
   const int32_t* block_table;
   const int32_t* seq_lens;
-  int max_blocks, H, G, R, D, V, block_size, chunk, splits;
+  int max_blocks, H, G, R, D, V, block_size, chunk, splits, window, maps;
   float scale2;                // score scale x log2(e)
   float* tmp_o;                // [B, H, splits, V]
   float* tmp_lse;              // [B, H, splits], log2
@@ -147,13 +165,15 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
   extern __shared__ uint4 g_smem[];
   __shared__ float s_m[kGWarps][16], s_l[kGWarps][16];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int b = blockIdx.x, g = blockIdx.y, split = blockIdx.z;
+  // (a group of more than 16 heads takes several CTAs)
+  const int b = blockIdx.x, g = blockIdx.y % p.G, head0 = blockIdx.y / p.G * 16, R = min(p.R - head0, 16), split = blockIdx.z;
   const int nd = p.D / 16, nv = p.V / 16, kw = p.G * p.D, vw = p.G * p.V;
   const int ks = (p.D + 8) * 2, vs = (p.V + 8) * 2, stage = g_stage_bytes(p.D, p.V);
   const uint32_t ring = smem_u32(g_smem) + warp * kGStages * stage;
   pdl_wait();
   pdl_launch_dependents();
-  const int pos = p.seq_lens[b] - 1, lo = p.chunk > 0 && pos > 0 ? pos / p.chunk * p.chunk : 0;
+  const int pos = p.seq_lens[b] - 1, 
+            lo = pos <= 0 ? 0 : p.chunk > 0 ? pos / p.chunk * p.chunk : p.window > 0 ? max(pos - p.window + 1, 0) : 0;
   // 16-key tiles of this split: a whole number per warp
   const int first = lo / kGKeys, all = pos < 0 ? 0 : pos / kGKeys + 1 - first;
   const int per = ((all + p.splits - 1) / p.splits + kGWarps - 1) / kGWarps * kGWarps;
@@ -191,13 +211,16 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
   for (int i = 0; i + 1 < kGStages; ++i) load(i);
 
   const int r0 = lane >> 2, c0 = (lane & 3) * 2;
+  // with maps the query row of a head is zero outside the columns of its own map
   uint32_t qa[ND][4];
+  const int dm = p.D / p.maps;
 #pragma unroll
   for (int x = 0; x < ND; ++x)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int r = r0 + (e & 1) * 8, d = x * 16 + c0 + (e >> 1) * 8;
-      qa[x][e] = r < p.R && x < nd ? *reinterpret_cast<const uint32_t*>(p.q + (size_t)b * p.ldq + (size_t)(g * p.R + r) * p.D + d) : 0u;
+      const int r = r0 + (e & 1) * 8, d = x * 16 + c0 + (e >> 1) * 8 - (head0 + r) % p.maps * dm;
+      qa[x][e] = r < R && x < nd && d >= 0 && d < dm
+                     ? *reinterpret_cast<const uint32_t*>(p.q + (size_t)b * p.ldq + (size_t)(g * p.R + head0 + r) * dm + d) : 0u;
     }
   float o[NV * 2][4];
 #pragma unroll
@@ -296,7 +319,7 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
     }
   }
   __syncthreads();
-  for (int i = tid; i < p.R * p.V / 2; i += kGWarps * 32) {
+  for (int i = tid; i < R * p.V / 2; i += kGWarps * 32) {
     const int r = i * 2 / p.V, c = i * 2 - r * p.V;
     float mx = -INFINITY, l = 0.f;
 #pragma unroll
@@ -310,7 +333,7 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
       y.y += v.y;
     }
     const float inv = l > 0.f ? 1.f / l : 0.f;
-    const size_t h = (size_t)g * p.R + r;
+    const size_t h = (size_t)g * p.R + head0 + r;
     if (p.splits == 1) {
       *reinterpret_cast<uint32_t*>(p.out + (size_t)b * p.ldo + h * p.V + c) = pack_bf16x2(y.x * inv, y.y * inv);
     } else {
@@ -328,12 +351,12 @@ template <typename T>
 __global__ void __launch_bounds__(128) rotate_kv_vec_kernel(RotateParams p) {
   pdl_wait();
   pdl_launch_dependents();
-  const int lane = threadIdx.x & 31, heads = p.H + 2 * p.G, c = lane * 4, kw = p.G * p.D, vw = p.G * p.V;
+  const int lane = threadIdx.x & 31, heads = p.H + p.G + p.GV, c = lane * 4, kw = p.G * p.D, vw = p.GV * p.V;
   const int x0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * kRotItems, total = p.T * heads;   // (below 2^31: checked)
   int t = x0 / heads, h = x0 - t * heads;
   float4 v[kRotItems], cs[kRotItems], sn[kRotItems];
   T* dst[kRotItems];
-  bool turn[kRotItems];
+  bool turn[kRotItems], is_q[kRotItems];
   const int half = p.rot / 2;
   const bool low = c < half, in_rot = p.cos_sin && c < p.rot;
 #pragma unroll
@@ -341,6 +364,7 @@ __global__ void __launch_bounds__(128) rotate_kv_vec_kernel(RotateParams p) {
     v[i] = cs[i] = sn[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     dst[i] = nullptr;
     turn[i] = h < p.H + p.G;
+    is_q[i] = h < p.H;
     if (x0 + i < total) {
       const T* row = reinterpret_cast<const T*>(p.qkv) + (size_t)t * p.ld;
       const int width = turn[i] ? p.D : p.V;
@@ -364,6 +388,25 @@ __global__ void __launch_bounds__(128) rotate_kv_vec_kernel(RotateParams p) {
     }
     if (++h == heads) { h = 0; ++t; }
   }
+  auto sum_sq = [](float4 y) {
+    float ss = y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
+#pragma unroll
+    for (int k = 16; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+    return ss;
+  };
+  if (p.q_w) {
+    float4 wq = make_float4(0.f, 0.f, 0.f, 0.f), wk = wq;
+    if (c < p.D) {
+      wq = *reinterpret_cast<const float4*>(p.q_w + c);
+      if (p.k_w) wk = *reinterpret_cast<const float4*>(p.k_w + c);
+    }
+#pragma unroll
+    for (int i = 0; i < kRotItems; ++i) {
+      const float inv = 1.f / sqrtf(sum_sq(v[i]) / (float)p.dim + p.eps);
+      const float4 w = is_q[i] ? wq : wk;
+      if (turn[i]) v[i] = make_float4(v[i].x * inv * w.x, v[i].y * inv * w.y, v[i].z * inv * w.z, v[i].w * inv * w.w);
+    }
+  }
   const int partner = in_rot ? (low ? lane + half / 4 : lane - half / 4) : lane;
 #pragma unroll
   for (int i = 0; i < kRotItems; ++i) {
@@ -378,18 +421,15 @@ __global__ void __launch_bounds__(128) rotate_kv_vec_kernel(RotateParams p) {
       y = make_float4(y.x * cs[i].x + g * o.x * sn[i].x, y.y * cs[i].y + g * o.y * sn[i].y,
                       y.z * cs[i].z + g * o.z * sn[i].z, y.w * cs[i].w + g * o.w * sn[i].w);
     }
-    float ss = y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
-#pragma unroll
-    for (int k = 16; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
-    const float inv = turn[i] ? 1.f / sqrtf(ss / (float)p.dim + p.eps) : 1.f;
+    const float inv = turn[i] && !p.q_w ? 1.f / sqrtf(sum_sq(y) / (float)p.dim + p.eps) : 1.f;
     if (dst[i]) store4(dst[i], make_float4(y.x * inv, y.y * inv, y.z * inv, y.w * inv));
   }
 }
 
 bool grouped_decode_fits(const B200BiasAttn* a) {
-  if (!a->grouped || a->f32 || a->bias || a->null_entry || a->kw % a->G) return false;
+  if (!a->grouped || a->f32 || a->bias || a->null_entry || a->kw % a->G || a->values_in_keys || a->gate) return false;
   const int D = a->kw / a->G, V = a->vdim;
-  return !(D & 15) && !(V & 15) && D <= 256 && V <= 256 && a->H / a->G <= 16 && a->block_size % kGKeys == 0 &&
+  return !(D / (a->maps > 1 ? a->maps : 1) & 15) && !(V & 15) && D <= 256 && V <= 256 && a->block_size % kGKeys == 0 &&
          !(((uintptr_t)a->q | (uintptr_t)a->cache) & 15) && !(a->ldq & 7) && !(a->ldo & 1) && a->scale > 0.f;
 }
 
@@ -400,7 +440,7 @@ static int launch_grouped(const GroupedDecode& p, int rows, cudaStream_t stream)
   if (smem < merge) smem = merge;
   static PerDeviceOnce once;
   if (once.first()) cudaFuncSetAttribute(grouped_decode_kernel<ND, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
-  return launch_pdl(grouped_decode_kernel<ND, NV>, dim3(rows, p.G, p.splits), dim3(kGWarps * 32), smem, stream, p) ==
+  return launch_pdl(grouped_decode_kernel<ND, NV>, dim3(rows, p.G * ((p.R + 15) / 16), p.splits), dim3(kGWarps * 32), smem, stream, p) ==
                  cudaSuccess ? 0 : -2;
 }
 template <int ND>
@@ -412,14 +452,56 @@ static int launch_grouped(const GroupedDecode& p, int rows, cudaStream_t stream)
 int grouped_decode(const B200BiasAttn* a, cudaStream_t stream) {
   GroupedDecode p{(const bf16*)a->q, a->ldq, (bf16*)a->out, a->ldo, (const bf16*)a->cache, (const int32_t*)a->block_table,
                   (const int32_t*)a->seq_lens, a->max_blocks, a->H, a->G, a->H / a->G, a->kw / a->G, a->vdim, a->block_size,
-                  a->chunk, a->splits < 1 ? 1 : a->splits, a->scale * 1.4426950408889634f, (float*)a->tmp_o,
+                  a->chunk, a->splits < 1 ? 1 : a->splits, a->window, a->maps > 1 ? a->maps : 1, a->scale * 1.4426950408889634f, (float*)a->tmp_o,
                   (float*)a->tmp_lse};
   if (p.splits > 1 && (!p.tmp_o || !p.tmp_lse)) return -1;
-  if (p.G > 65535 || p.splits > 65535) return -4;
+  if ((long)p.G * ((p.R + 15) / 16) > 65535 || p.splits > 65535) return -4;
   const int rc = p.D <= 64 ? launch_grouped<4>(p, a->rows, stream) : p.D <= 128 ? launch_grouped<8>(p, a->rows, stream)
                                                                                 : launch_grouped<16>(p, a->rows, stream);
   if (rc || p.splits == 1) return rc;
   return b200_attn_decode_merge(p.tmp_o, p.tmp_lse, p.out, (int)p.ldo, a->rows, p.H, p.V, p.splits, stream);
+}
+
+// ----------------------------------------------------------------------- difference of two maps
+// One warp per (token, head): o = first - lam second, over its root mean square over vdim, times scale.
+template <typename T>
+__global__ void __launch_bounds__(128) diff_combine_kernel(const T* maps, long long ldm, T* out, long long ldo, int H, int V,
+                                                           int vdim, long long items, float lam, float eps, float scale) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long x = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (x >= items) return;
+  const int lane = threadIdx.x & 31, h = (int)(x % H);
+  const long long t = x / H;
+  const T* src = maps + t * ldm + (size_t)h * 2 * V;
+  T* dst = out + t * ldo + (size_t)h * V;
+  auto diff = [&](int i) {
+    const float4 a = load4<T>(src + i), b = load4<T>(src + V + i);
+    return make_float4(a.x - lam * b.x, a.y - lam * b.y, a.z - lam * b.z, a.w - lam * b.w);
+  };
+  static constexpr int kKeep = 2;                // (groups kept between the passes)
+  float4 keep[kKeep];
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < kKeep; ++c) {
+    keep[c] = c * 128 + lane * 4 < V ? diff(c * 128 + lane * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    ss += keep[c].x * keep[c].x + keep[c].y * keep[c].y + keep[c].z * keep[c].z + keep[c].w * keep[c].w;
+  }
+  for (int i = kKeep * 128 + lane * 4; i < V; i += 128) {
+    const float4 v = diff(i);
+    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float f = scale / sqrtf(ss / (float)vdim + eps);
+#pragma unroll
+  for (int c = 0; c < kKeep; ++c)
+    if (c * 128 + lane * 4 < V)
+      store4(dst + c * 128 + lane * 4, make_float4(keep[c].x * f, keep[c].y * f, keep[c].z * f, keep[c].w * f));
+  for (int i = kKeep * 128 + lane * 4; i < V; i += 128) {
+    const float4 v = diff(i);
+    store4(dst + i, make_float4(v.x * f, v.y * f, v.z * f, v.w * f));
+  }
 }
 
 }  // namespace b200
@@ -429,23 +511,36 @@ using namespace b200;
 extern "C" {
 
 int b200_rotate_kv(const void* qkv, long long ld, const void* positions, const void* cos_sin, int rot, float eps,
-                   void* q_out, long long ldq, const void* slots, void* cache, int H, int G, int D, int V, int dim,
-                   int block_size, int T, int f32, cudaStream_t stream) {
+                   const float* q_w, const float* k_w, void* q_out, long long ldq, const void* slots, void* cache, int H, int G,
+                   int GV, int D, int V, int dim, int block_size, int T, int f32, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (H <= 0 || G < 0 || D <= 0 || (D & 3) || (G && (V <= 0 || (V & 3))) || D > kRotMax || dim <= 0 || dim > D ||
+  if (H <= 0 || G < 0 || GV < 0 || GV > G || (G && q_w && !k_w) || D <= 0 || (D & 3) || (G && (V <= 0 || (V & 3))) || D > kRotMax || dim <= 0 || dim > D ||
       (cos_sin && ((rot & 1) || rot > dim)) || (ld & 3) || (ldq & 3) || block_size <= 0)
     return -1;
   RotateParams p{qkv, ld, (const int64_t*)positions, (const float*)cos_sin, q_out, ldq, (const int64_t*)slots, cache,
-                 rot, H, G, D, V, dim, block_size, T, eps};
-  if (D <= 128 && (!G || V <= 128) && (!cos_sin || !(rot & 7)) && (long long)T * (H + 2 * G) < (1ll << 31) - 64) {
-    const dim3 vgrid((unsigned)(((long long)T * (H + 2 * G) + 4 * kRotItems - 1) / (4 * kRotItems)));
+                 rot, H, G, D, V, dim, block_size, T, eps, GV, q_w, k_w};
+  const long long items = (long long)T * (H + G + GV);
+  if (D <= 128 && (!G || V <= 128) && (!cos_sin || !(rot & 7)) && items < (1ll << 31) - 64) {
+    const dim3 vgrid((unsigned)((items + 4 * kRotItems - 1) / (4 * kRotItems)));
     return (f32 ? launch_pdl(rotate_kv_vec_kernel<float>, vgrid, dim3(128), 0, stream, p)
                 : launch_pdl(rotate_kv_vec_kernel<bf16>, vgrid, dim3(128), 0, stream, p)) == cudaSuccess ? 0 : -2;
   }
-  const dim3 grid((unsigned)(((long long)T * (H + 2 * G) + 3) / 4));
+  const dim3 grid((unsigned)((items + 3) / 4));
   const size_t smem = (size_t)4 * D * 4;
   return (f32 ? launch_pdl(rotate_kv_kernel<float>, grid, dim3(128), smem, stream, p)
               : launch_pdl(rotate_kv_kernel<bf16>, grid, dim3(128), smem, stream, p)) == cudaSuccess ? 0 : -2;
+}
+
+int b200_diff_combine(const void* maps, long long ldm, void* out, long long ldo, int H, int V, int vdim, int T, float lam,
+                      float eps, float scale, int f32, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || V <= 0 || (V & 3) || vdim <= 0 || vdim > V || (ldm & 3) || (ldo & 3)) return -1;
+  const long long items = (long long)T * H;
+  const dim3 grid((unsigned)((items + 3) / 4));
+  return (f32 ? launch_pdl(diff_combine_kernel<float>, grid, dim3(128), 0, stream, (const float*)maps, ldm, (float*)out, ldo, H,
+                           V, vdim, items, lam, eps, scale)
+              : launch_pdl(diff_combine_kernel<bf16>, grid, dim3(128), 0, stream, (const bf16*)maps, ldm, (bf16*)out, ldo, H, V,
+                           vdim, items, lam, eps, scale)) == cudaSuccess ? 0 : -2;
 }
 
 }  // extern "C"

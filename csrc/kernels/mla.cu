@@ -1,11 +1,14 @@
-// Multi-head latent attention (DeepSeek-V2 family) kernels.
+// Multi-head latent attention kernels (DeepSeek-V2 family; the decode kernel also serves other latent sizes,
+// windows and gated heads).
 //
-// Cache: one row of 512 latent + 64 rotary values per token, [num_blocks * block_size, 576].
+// Cache: one row of 512 latent + 64 rotary values per token, [num_blocks * block_size, 576]; other latents are
+// 1 to 4 pieces of 128 values.
 //
 // Decode ("absorbed" form, reference: src/vt/cuda/cuda_mla_decode.cu MlaDecodeStage1/2):
 // queries arrive already multiplied by W_UK, q' = [q_nope W_UK (512) | q_pe (64)], and all
 // heads attend to the same latent rows (multi-query); V is the first 512 columns of those
 // rows. tcgen05 with swapped operands, one CTA = one (sequence, kv split):
+// (more than 16 heads: one CTA per 16):
 //     S^T[128 tok, 16 heads] = C[128 tok, 576] * q'[16, 576]^T
 //     O^T[512, 16]          += C[128 tok, 0:512]^T * P^T          (four M = 128 products)
 // Every byte of the latent tile is loaded once. Its four 128-column value pieces go through a ring
@@ -33,14 +36,13 @@ typedef __nv_bfloat16 bf16;
 static constexpr int kTok = 128;
 static constexpr int kNQ = 16;
 static constexpr int kLat = 512, kRope = 64, kRow = kLat + kRope;   // 576
-static constexpr int kVPieces = 4;         // 128-column value pieces of a row (the rotary 64 columns follow)
+// (kVPieces, the kernel's parameter: 128-column value pieces of a row; the rotary 64 columns follow)
 static constexpr int kVSlots = 5;          // ring of the value pieces
 static constexpr int kRSlots = 2;          // ring of the rotary pieces
 static constexpr int kSlots = kVSlots + kRSlots;
 static constexpr int kSlotBytes = 128 * 128 * 2;
 static constexpr int kRopeBytes = 128 * 64 * 2;
 static constexpr int kRingBytes = kVSlots * kSlotBytes + kRSlots * kRopeBytes;
-static constexpr int kQBytes = 9 * 2048;   // 9 halves of [16 heads x 64 cols]
 
 struct MlaDecodeParams {
   bf16* out;            // [B, Hq, 512]
@@ -54,6 +56,9 @@ struct MlaDecodeParams {
   float* tmp_o;         // [B, Hq, splits, 512]
   float* tmp_lse;       // [B, Hq, splits] log2 domain
   int* status;
+  int window;           // > 0: only the last that many positions
+  const bf16* gate;     // [B, ldg] or null: each head's output times sigmoid(gate)
+  long long ldg;
 };
 
 struct alignas(8) MlaBars {
@@ -67,6 +72,7 @@ struct alignas(8) MlaBars {
   uint32_t tmem_base;
   float red_max[2][4][kNQ];
   float red_sum[4][kNQ];
+  float gate[kNQ];
 };
 
 __device__ __forceinline__ void mla_tmem_st_x16(uint32_t taddr, const uint32_t* r) {
@@ -93,10 +99,13 @@ __device__ __forceinline__ float mla_exp2(float x) {
 
 // Ring order shared by producer and consumer: S pieces of tile 0; then for every later tile j
 // its S pieces followed by the O pieces of tile j-1; last the O pieces of the final tile.
+template <int kVPieces>
 __global__ void __launch_bounds__(192, 1)
     mla_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmC,
                       MlaDecodeParams p) {
   extern __shared__ uint8_t smem_raw[];
+  constexpr int kLat = kVPieces * 128;
+  constexpr int kQHalves = 2 * kVPieces + 1, kQBytes = kQHalves * 2048;   // halves of [16 heads x 64 cols]
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sKV = smem;
   uint8_t* sRope = sKV + kVSlots * kSlotBytes;
@@ -106,13 +115,14 @@ __global__ void __launch_bounds__(192, 1)
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int b = blockIdx.x, split = blockIdx.y;
-  const int G = p.Hq;
+  const int head0 = blockIdx.z * kNQ, G = min(p.Hq - head0, kNQ);
   const int seq_len = p.seq_lens[b];
-  const int tiles_total = (seq_len + kTok - 1) / kTok;
+  const int first_tok = p.window > 0 ? max(seq_len - p.window, 0) : 0, first_tile = first_tok / kTok;
+  const int tiles_total = (seq_len + kTok - 1) / kTok - first_tile;
   const int tiles_per_split = (tiles_total + p.splits - 1) / p.splits;
   const int tile0 = split * tiles_per_split;
   const int ntiles = max(0, min(tiles_total, tile0 + tiles_per_split) - tile0);
-  const int tok_base = tile0 * kTok;
+  const int tok_base = (first_tile + tile0) * kTok;
 
   if (threadIdx.x == 0) {
     mbar_init(&bars->q_full, 1);
@@ -151,7 +161,7 @@ __global__ void __launch_bounds__(192, 1)
         tma_prefetch_desc(&tmQ);
         tma_prefetch_desc(&tmC);
         mbar_expect_tx(&bars->q_full, kQBytes);
-        for (int h = 0; h < 9; ++h) tma_load_3d(sQ + h * 2048, &tmQ, &bars->q_full, h * 64, 0, b);
+        for (int h = 0; h < kQHalves; ++h) tma_load_3d(sQ + h * 2048, &tmQ, &bars->q_full, h * 64, head0, b);
         const int32_t* bt = p.block_table + (size_t)b * p.max_blocks;
         const int nblk_valid = (seq_len + p.block_size - 1) / p.block_size;
         const int rows_per_load = min(p.block_size, kTok);
@@ -275,7 +285,7 @@ __global__ void __launch_bounds__(192, 1)
         __syncwarp();
         if (lane == 0) mbar_arrive(&bars->s_empty[sb]);
         const int tok = tok_base + j * kTok + t;
-        const bool valid = tok < seq_len;
+        const bool valid = tok < seq_len && tok >= first_tok;
         float s[kNQ];
 #pragma unroll
         for (int g = 0; g < kNQ; ++g) s[g] = valid ? __uint_as_float(r[g]) * p.scale_log2 : -INFINITY;
@@ -348,6 +358,8 @@ __global__ void __launch_bounds__(192, 1)
       if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->o_done, 0, p.status));
       if (ok) {
         tc_fence_after_sync();
+        if (quarter == 0 && lane < kNQ)
+          bars->gate[lane] = p.gate && lane < G ? 1.f / (1.f + expf(-__bfloat162float(p.gate[(size_t)b * p.ldg + head0 + lane]))) : 1.f;
 #pragma unroll
         for (int g = 0; g < kNQ; ++g) {
           float v = lsum[g];
@@ -368,11 +380,11 @@ __global__ void __launch_bounds__(192, 1)
           for (int g = 0; g < kNQ; ++g) {
             if (g < G) {
               const float l = bars->red_sum[0][g] + bars->red_sum[1][g] + bars->red_sum[2][g] + bars->red_sum[3][g];
-              const float v = l > 0.f ? __uint_as_float(o[g]) / l : 0.f;
+              const float v = l > 0.f ? __uint_as_float(o[g]) / l * bars->gate[g] : 0.f;
               if (p.splits == 1) {
-                p.out[(size_t)b * p.ldo + (size_t)g * kLat + d] = __float2bfloat16(v);
+                p.out[(size_t)b * p.ldo + (size_t)(head0 + g) * kLat + d] = __float2bfloat16(v);
               } else {
-                const size_t row = ((size_t)b * p.Hq + g) * p.splits + split;
+                const size_t row = ((size_t)b * p.Hq + head0 + g) * p.splits + split;
                 p.tmp_o[row * kLat + d] = v;
                 if (d == 0) p.tmp_lse[row] = l > 0.f ? m[g] + log2f(l) : -INFINITY;
               }
@@ -387,9 +399,9 @@ __global__ void __launch_bounds__(192, 1)
       for (int pc = 0; pc < kVPieces; ++pc) {
         const int d = pc * 128 + t;
         if (p.splits == 1) {
-          p.out[(size_t)b * p.ldo + (size_t)g * kLat + d] = __float2bfloat16(0.f);
+          p.out[(size_t)b * p.ldo + (size_t)(head0 + g) * kLat + d] = __float2bfloat16(0.f);
         } else {
-          const size_t row = ((size_t)b * p.Hq + g) * p.splits + split;
+          const size_t row = ((size_t)b * p.Hq + head0 + g) * p.splits + split;
           p.tmp_o[row * kLat + d] = 0.f;
           if (d == 0) p.tmp_lse[row] = -INFINITY;
         }
@@ -485,42 +497,45 @@ extern "C" int b200_attn_decode_merge(const void* tmp_o, const void* tmp_lse, vo
 
 extern "C" {
 
-// qabs: [B, Hq, 576] bf16 contiguous; cache: [num_blocks * block_size, 576]; out: [B, Hq, 512]
-// (row stride ldo). Hq <= 16.
-int b200_mla_decode(const void* qabs, void* out, int ldo, const void* cache, int64_t num_blocks,
-                    int block_size, int Hq, const void* block_table, int max_blocks,
-                    const void* seq_lens, int B, float scale, int splits, void* tmp_o, void* tmp_lse,
-                    cudaStream_t stream) {
+// qabs: [B, H, rank + 64] bf16 contiguous; cache: [num_blocks * block_size, rank + 64]; out: [B, H, rank]
+// (row stride ldo). rank: 128 to 512 in steps of 128.
+int b200_latent_decode(const void* qabs, void* out, int ldo, const void* cache, int64_t num_blocks, int block_size, int H,
+                       int rank, int rot, const void* block_table, int max_blocks, const void* seq_lens, int B, float scale,
+                       int window, const void* gate, long long ldg, int splits, void* tmp_o, void* tmp_lse,
+                       cudaStream_t stream) {
   if (B <= 0) return 0;
-  if (Hq < 1 || Hq > kNQ) return -1;
+  if (H < 1 || rank < 128 || rank > 512 || rank % 128 || rot != kRope || window < 0) return -1;
   if (block_size < 8 || (block_size & 7) || (block_size < kTok && kTok % block_size) ||
       (block_size > kTok && block_size % kTok) || kTok / (block_size < kTok ? block_size : kTok) > 16)
     return -1;
   if (splits < 1) splits = 1;
   if (splits > 1 && (!tmp_o || !tmp_lse)) return -1;
+  const int hgroups = (H + kNQ - 1) / kNQ, row = rank + kRope;
+  if (splits > 65535 || hgroups > 65535) return -4;
   static std::mutex mu;
   static std::unordered_map<MKey, CUtensorMap, MKeyHash> maps;
   CUtensorMap tmQ, tmC;
   {
     std::lock_guard<std::mutex> lock(mu);
-    MKey kq{qabs, (uint64_t)B, (uint64_t)Hq};
+    MKey kq{qabs, (uint64_t)B, (uint64_t)H << 16 | row};
     auto it = maps.find(kq);
     if (it == maps.end()) {
+      if (maps.size() > 4096) maps.clear();
       CUtensorMap m;
-      if (!encode_tmap_3d(&m, qabs, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)kRow, (uint64_t)Hq,
-                          (uint64_t)B, (uint64_t)kRow * 2, (uint64_t)Hq * kRow * 2, 64, kNQ, 1,
+      if (!encode_tmap_3d(&m, qabs, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (uint64_t)row, (uint64_t)H,
+                          (uint64_t)B, (uint64_t)row * 2, (uint64_t)H * row * 2, 64, kNQ, 1,
                           CU_TENSOR_MAP_SWIZZLE_128B))
         return -3;
       it = maps.emplace(kq, m).first;
     }
     tmQ = it->second;
     const uint32_t box_rows = block_size < kTok ? block_size : kTok;
-    MKey kc{cache, (uint64_t)num_blocks * block_size, (uint64_t)box_rows + 99991};
+    MKey kc{cache, (uint64_t)num_blocks * block_size, (uint64_t)1 << 48 | (uint64_t)box_rows << 16 | row};
     it = maps.find(kc);
     if (it == maps.end()) {
       CUtensorMap m;
       if (!encode_tmap_2d(&m, cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2,
-                          (uint64_t)num_blocks * block_size, kRow, kRow, box_rows, 64,
+                          (uint64_t)num_blocks * block_size, row, row, box_rows, 64,
                           CU_TENSOR_MAP_SWIZZLE_128B))
         return -3;
       it = maps.emplace(kc, m).first;
@@ -530,19 +545,37 @@ int b200_mla_decode(const void* qabs, void* out, int ldo, const void* cache, int
   MlaDecodeParams p;
   p.out = (bf16*)out; p.ldo = ldo;
   p.block_table = (const int32_t*)block_table; p.max_blocks = max_blocks;
-  p.seq_lens = (const int32_t*)seq_lens; p.Hq = Hq; p.block_size = block_size;
+  p.seq_lens = (const int32_t*)seq_lens; p.Hq = H; p.block_size = block_size;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.splits = splits; p.tmp_o = (float*)tmp_o; p.tmp_lse = (float*)tmp_lse;
   p.status = device_status_word();
-  constexpr size_t smem = (size_t)kRingBytes + kQBytes + 8192 + 1024 + sizeof(MlaBars);
-  static PerDeviceOnce attr_once;
-  if (attr_once.first()) {
-    cudaFuncSetAttribute(mla_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  p.window = window; p.gate = (const bf16*)gate; p.ldg = ldg;
+  auto launch = [&](auto kernel, PerDeviceOnce& attr_once, int pieces) {
+    const size_t smem = (size_t)kRingBytes + (2 * pieces + 1) * 2048 + 8192 + 1024 + sizeof(MlaBars);
+    if (attr_once.first()) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    kernel<<<dim3(B, splits, hgroups), 192, smem, stream>>>(tmQ, tmC, p);
+  };
+  static PerDeviceOnce once[4];
+  switch (rank / 128) {
+    case 1: launch(mla_decode_kernel<1>, once[0], 1); break;
+    case 2: launch(mla_decode_kernel<2>, once[1], 2); break;
+    case 3: launch(mla_decode_kernel<3>, once[2], 3); break;
+    default: launch(mla_decode_kernel<4>, once[3], 4); break;
   }
-  mla_decode_kernel<<<dim3(B, splits), 192, smem, stream>>>(tmQ, tmC, p);
   if (cudaGetLastError() != cudaSuccess) return -2;
-  if (splits > 1) return b200_attn_decode_merge(tmp_o, tmp_lse, out, ldo, B, Hq, kLat, splits, stream);
+  if (splits > 1) return b200_attn_decode_merge(tmp_o, tmp_lse, out, ldo, B, H, rank, splits, stream);
   return 0;
+}
+
+// qabs: [B, Hq, 576] bf16 contiguous; cache: [num_blocks * block_size, 576]; out: [B, Hq, 512]
+// (row stride ldo). Hq <= 16.
+int b200_mla_decode(const void* qabs, void* out, int ldo, const void* cache, int64_t num_blocks,
+                    int block_size, int Hq, const void* block_table, int max_blocks,
+                    const void* seq_lens, int B, float scale, int splits, void* tmp_o, void* tmp_lse,
+                    cudaStream_t stream) {
+  if (Hq > kNQ) return -1;
+  return b200_latent_decode(qabs, out, ldo, cache, num_blocks, block_size, Hq, kLat, kRope, block_table, max_blocks, seq_lens,
+                            B, scale, 0, nullptr, 0, splits, tmp_o, tmp_lse, stream);
 }
 
 int b200_mla_gather_latent(const void* cache, const void* block_table, int max_blocks,

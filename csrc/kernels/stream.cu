@@ -3,6 +3,7 @@
 //   stream_norm_kernel   embedding or residual update (+ expert outputs gathered per token, + norm of the
 //                        update) + RMSNorm
 //   gemm_f32_kernel      out = A W^T (+ bias), plain or per expert chunk
+//   softcap_kernel      cap tanh(x / cap) of fp32 logits
 //   clamped_gate_kernel, gated_act_kernel   activation of [gate | up] rows
 #include "api.h"
 #include "sm100.cuh"
@@ -116,7 +117,10 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(B200StreamNorm p, int*
       v.x *= post * (w.x + p.norm_offset); v.y *= post * (w.y + p.norm_offset);
       v.z *= post * (w.z + p.norm_offset); v.w *= post * (w.w + p.norm_offset);
     }
-    if (!p.ids) add4(v, before);
+    if (!p.ids) {
+      v.x *= p.mult; v.y *= p.mult; v.z *= p.mult; v.w *= p.mult;
+      add4(v, before);
+    }
     return v;
   };
   float ss = 0.f;
@@ -166,6 +170,8 @@ struct F32Gemm {
   const float* bias;
   float* out;
   int lda, ldw, ldo, M, N, K;
+  // batched (blockIdx.z): columns of A, rows of W, columns of out
+  long long a_batch, w_batch, out_batch;
   // grouped: chunk c covers rows [row0[c], row0[c] + n[c]) of A / out with the matrix of expert[c]
   const int32_t* chunk_expert;
   const int32_t* chunk_row0;
@@ -181,12 +187,18 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(F32Gemm p) {
   pdl_wait();
   pdl_launch_dependents();
   const float* W = p.W;
+  const float* A = p.A;
+  float* out = p.out;
   int row_base = 0, rows = p.M;
   if (p.chunk_expert) {
     if ((int)blockIdx.z >= *p.num_chunks) return;
     W += (size_t)p.chunk_expert[blockIdx.z] * p.N * p.ldw;
     row_base = p.chunk_row0[blockIdx.z];
     rows = p.chunk_n[blockIdx.z];
+  } else {
+    A += blockIdx.z * p.a_batch;
+    W += blockIdx.z * p.w_batch;
+    out += blockIdx.z * p.out_batch;
   }
   const int m0 = blockIdx.y * kFT, n0 = blockIdx.x * kFT;
   if (m0 >= rows) return;
@@ -200,7 +212,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(F32Gemm p) {
     for (int x = threadIdx.x; x < kFT * kFK; x += 256) {
       const int r = x >> 4, k = x & 15;
       const bool kin = k0 + k < p.K;
-      sa[k][r] = (kin && m0 + r < rows) ? p.A[(size_t)(row_base + m0 + r) * p.lda + k0 + k] : 0.f;
+      sa[k][r] = (kin && m0 + r < rows) ? A[(size_t)(row_base + m0 + r) * p.lda + k0 + k] : 0.f;
       sw[k][r] = (kin && n0 + r < p.N) ? W[(size_t)(n0 + r) * p.ldw + k0 + k] : 0.f;
     }
     __syncthreads();
@@ -223,7 +235,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(F32Gemm p) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < p.N) p.out[(size_t)(row_base + m) * p.ldo + n] = acc[i][j] + (p.bias ? p.bias[n] : 0.f);
+      if (n < p.N) out[(size_t)(row_base + m) * p.ldo + n] = acc[i][j] + (p.bias ? p.bias[n] : 0.f);
     }
   }
 }
@@ -257,6 +269,13 @@ __global__ void __launch_bounds__(128) gated_act_kernel(const float* gu, int ldg
   }
 }
 
+__global__ void __launch_bounds__(256) softcap_kernel(float* x, long long n, float cap) {
+  pdl_wait();
+  pdl_launch_dependents();
+  for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < n; i += (long long)gridDim.x * 256)
+    x[i] = cap * tanhf(x[i] / cap);
+}
+
 }  // namespace b200
 
 using namespace b200;
@@ -279,10 +298,29 @@ int b200_gemm_f32(const void* A, int lda, const void* W, int ldw, void* out, int
                   int K, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   F32Gemm p{(const float*)A, (const float*)W, (const float*)bias, (float*)out, lda, ldw, ldo, M, N, K,
-            nullptr, nullptr, nullptr, nullptr};
+            0, 0, 0, nullptr, nullptr, nullptr, nullptr};
   dim3 grid((N + kFT - 1) / kFT, (M + kFT - 1) / kFT);
   if (grid.y > 65535) return -4;
   return launch_pdl(gemm_f32_kernel, grid, dim3(256), 0, stream, p) == cudaSuccess ? 0 : -2;
+}
+
+// out[m, b * out_batch + n] = sum_k A[m, b * a_batch + k] W[b * N + n, k]
+int b200_gemm_f32_batched(const void* A, int lda, int a_batch, const void* W, int ldw, void* out, int ldo,
+                          long long out_batch, int M, int N, int K, int batch, cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
+  F32Gemm p{(const float*)A, (const float*)W, nullptr, (float*)out, lda, ldw, ldo, M, N, K,
+            a_batch, (long long)N * ldw, out_batch, nullptr, nullptr, nullptr, nullptr};
+  dim3 grid((N + kFT - 1) / kFT, (M + kFT - 1) / kFT, batch);
+  if (grid.y > 65535 || grid.z > 65535) return -4;
+  return launch_pdl(gemm_f32_kernel, grid, dim3(256), 0, stream, p) == cudaSuccess ? 0 : -2;
+}
+
+int b200_softcap_f32(void* x, long long n, float cap, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f)) return -1;
+  const long long blocks = (n + 255) / 256;
+  return launch_pdl(softcap_kernel, dim3((unsigned)(blocks < 16384 ? blocks : 16384)), dim3(256), 0, stream, (float*)x, n,
+                    cap) == cudaSuccess ? 0 : -2;
 }
 
 int b200_moe_grouped_gemm_f32(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out,
@@ -291,7 +329,7 @@ int b200_moe_grouped_gemm_f32(const void* xs, int max_rows, const void* W, int E
   if (max_rows <= 0) return 0;
   if (max_chunks > 65535) return -4;
   F32Gemm p{(const float*)xs, (const float*)W, nullptr, (float*)out, K, K, N, max_rows, N, K,
-            (const int32_t*)chunk_expert, (const int32_t*)chunk_row0, (const int32_t*)chunk_n,
+            0, 0, 0, (const int32_t*)chunk_expert, (const int32_t*)chunk_row0, (const int32_t*)chunk_n,
             (const int32_t*)meta + 3 * E + 1};
   dim3 grid((N + kFT - 1) / kFT, 256 / kFT, max_chunks);     // a chunk has at most 256 rows
   return launch_pdl(gemm_f32_kernel, grid, dim3(256), 0, stream, p) == cudaSuccess ? 0 : -2;

@@ -173,7 +173,7 @@ class TabupelModel(ListedModel):
         dkv = p["dkv"]
         parts = ((p["dq"], q8), (dkv[: s.rank], k8), (pairs_apart(dkv[s.rank:], 1, 0, s.rot), r8), (p["g"], g8))
         L["down_proj"] = torch.cat([self.put(t, n, self.cols) for t, n in parts], 0)
-        L["q_norm"], L["kv_norm"] = (self.put(p[n], **f32) for n in ("dq.norm", "dkv.norm"))
+        L["q_norm"], L["kv_norm"] = (self.put(p[n], w, **f32) for n, w in (("dq.norm", q8), ("dkv.norm", k8)))
         uq = p["uq"].reshape(H, s.dim + s.rot, -1)
         turned = pairs_apart(uq[:, s.dim:].reshape(H * s.rot, -1), H, 0, s.rot).reshape(H, s.rot, -1)
         uq = torch.cat([self.put(uq[:, : s.dim], H, s.qn, q8), self.put(turned, H, s.qw - s.qn, q8)], 1)
