@@ -1,7 +1,7 @@
 // Grouped-query attention over the pages of attn_bias.cu ([block_size][G * D] keys | [block_size][G * V]
 // values): query / key preparation and the decode kernel.
 //
-//   rotate_kv_kernel        rotation and unit norm, or weighted norm and rotation; cache write
+//   rotate_kv kernels       rotation and unit norm, or weighted norm and rotation; cache write
 //   diff_combine_kernel     difference of a head's two maps, its norm
 //   grouped_decode_kernel   bf16, one query row per request: a CTA takes one kv group and one split of the
 //                           visible keys, its four warps every fourth tile of 16 keys, each through its own
@@ -426,6 +426,125 @@ __global__ void __launch_bounds__(128) rotate_kv_vec_kernel(RotateParams p) {
   }
 }
 
+// Head sizes that are multiples of 8 (up to 256) whose half rotation is one too: a lane holds eight values, a head
+// is a group of LANES lanes. One CTA per token, its warps take the heads in turn, so that a lane needs the
+// token's cosines only once. The value row is copied in pieces as wide as a head.
+template <typename T> struct Ld8;
+template <> struct Ld8<float> {
+  static __device__ __forceinline__ void get(const float* p, float* v) {
+    *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
+    *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(p + 4);
+  }
+  static __device__ __forceinline__ void put(float* p, const float* v) {
+    *reinterpret_cast<float4*>(p) = *reinterpret_cast<const float4*>(v);
+    *reinterpret_cast<float4*>(p + 4) = *reinterpret_cast<const float4*>(v + 4);
+  }
+};
+template <> struct Ld8<bf16> {
+  static __device__ __forceinline__ void get(const bf16* p, float* v) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 f = unpack_bf16x2(w[i]);
+      v[2 * i] = f.x;
+      v[2 * i + 1] = f.y;
+    }
+  }
+  static __device__ __forceinline__ void put(bf16* p, const float* v) {
+    *reinterpret_cast<uint4*>(p) =
+        make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+  }
+};
+
+template <typename T, int LANES>
+__global__ void __launch_bounds__(128) rotate_kv_row_kernel(RotateParams p) {
+  static constexpr int kHeads = 32 / LANES;              // heads of a warp at a time
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane % LANES, c = sub * 8;
+  const int kw = p.G * p.D, vw = p.GV * p.V, turned = p.H + p.G, heads = turned + (vw + p.D - 1) / p.D;
+  const T* row = reinterpret_cast<const T*>(p.qkv) + (size_t)t * p.ld;
+  const int64_t slot = p.G ? p.slots[t] : -1;
+  T* page = nullptr;
+  int off = 0;
+  if (slot >= 0) {
+    page = reinterpret_cast<T*>(p.cache) + slot / p.block_size * p.block_size * (int64_t)(kw + vw);
+    off = (int)(slot % p.block_size);
+  }
+  const int half = p.rot / 2;
+  const bool in = c < p.D, low = c < half, in_rot = p.cos_sin && c < p.rot;
+  float cs[8], sn[8], wq[8], wk[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) { cs[i] = 1.f; sn[i] = 0.f; wq[i] = wk[i] = 1.f; }
+  if (in_rot) {
+    const float* f = p.cos_sin + (size_t)p.positions[t] * p.rot + (low ? c : c - half);
+    Ld8<float>::get(f, cs);
+    Ld8<float>::get(f + half, sn);
+    if (low) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) sn[i] = -sn[i];
+    }
+  }
+  if (p.q_w && in) {
+    Ld8<float>::get(p.q_w + c, wq);
+    if (p.k_w) Ld8<float>::get(p.k_w + c, wk);
+  }
+  const int partner = in_rot ? (low ? lane + half / 8 : lane - half / 8) : lane;
+  auto inv_rms = [&](const float* v) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss = fmaf(v[i], v[i], ss);
+#pragma unroll
+    for (int k = LANES / 2; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+    return 1.f / sqrtf(ss / (float)p.dim + p.eps);
+  };
+#pragma unroll 2
+  for (int h0 = warp * kHeads; h0 < heads; h0 += 4 * kHeads) {
+    const int h = h0 + lane / LANES;
+    const bool on = in && h < heads && (h < p.H || page) && (h < turned || (h - turned) * p.D + c < vw);
+    float v[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = 0.f;
+    if (on) Ld8<T>::get(row + (size_t)h * p.D + c, v);
+    if (h0 < turned) {                                   // (warp-uniform)
+      float inv = 1.f;
+      if (p.q_w) {
+        inv = inv_rms(v);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] *= h < turned ? inv * (h < p.H ? wq[i] : wk[i]) : 1.f;
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const float o = __shfl_sync(0xffffffffu, v[i], partner);
+        if (h < turned) v[i] = fmaf(v[i], cs[i], o * sn[i]);
+      }
+      if (!p.q_w) {
+        inv = inv_rms(v);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] *= h < turned ? inv : 1.f;
+      }
+    }
+    if (!on) continue;
+    T* dst = h < p.H ? reinterpret_cast<T*>(p.q_out) + (size_t)t * p.ldq + (size_t)h * p.D
+             : h < turned ? page + (int64_t)off * kw + (int64_t)(h - p.H) * p.D
+                          : page + (int64_t)p.block_size * kw + (int64_t)off * vw + (int64_t)(h - turned) * p.D;
+    Ld8<T>::put(dst + c, v);
+  }
+}
+
+template <typename T>
+static int launch_rotate_rows(const RotateParams& p, cudaStream_t stream) {
+  const dim3 grid(p.T), block(128);
+  cudaError_t e;
+  if (p.D <= 16) e = launch_pdl(rotate_kv_row_kernel<T, 2>, grid, block, 0, stream, p);
+  else if (p.D <= 32) e = launch_pdl(rotate_kv_row_kernel<T, 4>, grid, block, 0, stream, p);
+  else if (p.D <= 64) e = launch_pdl(rotate_kv_row_kernel<T, 8>, grid, block, 0, stream, p);
+  else if (p.D <= 128) e = launch_pdl(rotate_kv_row_kernel<T, 16>, grid, block, 0, stream, p);
+  else e = launch_pdl(rotate_kv_row_kernel<T, 32>, grid, block, 0, stream, p);
+  return e == cudaSuccess ? 0 : -2;
+}
+
 bool grouped_decode_fits(const B200BiasAttn* a) {
   if (!a->grouped || a->f32 || a->bias || a->null_entry || a->kw % a->G || a->values_in_keys || a->gate) return false;
   const int D = a->kw / a->G, V = a->vdim;
@@ -520,6 +639,10 @@ int b200_rotate_kv(const void* qkv, long long ld, const void* positions, const v
   RotateParams p{qkv, ld, (const int64_t*)positions, (const float*)cos_sin, q_out, ldq, (const int64_t*)slots, cache,
                  rot, H, G, D, V, dim, block_size, T, eps, GV, q_w, k_w};
   const long long items = (long long)T * (H + G + GV);
+  const int es = f32 ? 4 : 2;
+  const bool aligned = !(((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)cache) & 15) && !((ld * es | ldq * es) & 15);
+  if (aligned && !(D & 7) && D <= 256 && (!cos_sin || !(rot & 15)) && !(GV * V & 7))
+    return f32 ? launch_rotate_rows<float>(p, stream) : launch_rotate_rows<bf16>(p, stream);
   if (D <= 128 && (!G || V <= 128) && (!cos_sin || !(rot & 7)) && items < (1ll << 31) - 64) {
     const dim3 vgrid((unsigned)((items + 4 * kRotItems - 1) / (4 * kRotItems)));
     return (f32 ? launch_pdl(rotate_kv_vec_kernel<float>, vgrid, dim3(128), 0, stream, p)

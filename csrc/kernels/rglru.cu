@@ -194,15 +194,17 @@ __global__ void __launch_bounds__(128) rglru_scan_any_kernel(B200Rglru p) {
 // One CTA: 128 channels of a block (blockIdx.x) and one slice of the units (blockIdx.y). A unit is up to 64
 // rows: decode rows, or rows of one portion (half of a 128-row tile). Gate logits come out transposed, channels
 // as the 128 rows of the product and tokens as its 64 columns, so that a thread holds one channel and walks
-// its tokens in registers. Warps 0-7: recurrence, lane quarter = channels, warps 4-7 the later half of the
-// tokens; both halves reduce theirs to (decay, end state), exchange these, and run through once more from the
-// state they start with. Warp 8: TMA, warp 9: MMA; the product of the next unit runs under the recurrence of this one.
-static constexpr int kUnit = 64, kHalf = 32, kMaxUStages = 4, kRgThreads = 320;
+// its tokens in registers. Warps 0-15: recurrence, lane quarter = channels, four parts of 16 tokens; every part
+// reduces its tokens to (decay, end state), the parts exchange these, and each runs through once more from the
+// state it starts with. Warp 16: TMA, warp 17: MMA; the product of the next unit, its rows of y and the look-up of
+// where its rows are run under the recurrence of this one.
+static constexpr int kUnit = 64, kParts = 4, kPart = kUnit / kParts, kMaxUStages = 4;
+static constexpr int kRgWarps = 4 * kParts, kRgThreads = (kRgWarps + 2) * 32;
 
 struct alignas(8) RgBars {
   uint64_t w_full, u_full[kMaxUStages], u_empty[kMaxUStages], d_full[2], d_empty[2];
   uint32_t tmem_base;
-  float2 xch[2][2][128];                 // [unit parity][half][channel]: decay, end state
+  float2 xch[2][kParts][128];            // [unit parity][part][channel]: decay, end state
 };
 
 struct RgUnit {
@@ -259,16 +261,16 @@ __global__ void __launch_bounds__(kRgThreads, 1)
 
   if (threadIdx.x == 0) {
     mbar_init(&bars->w_full, 1);
-    for (int i = 0; i < stages; ++i) { mbar_init(&bars->u_full[i], 1); mbar_init(&bars->u_empty[i], 8); }
-    for (int i = 0; i < 2; ++i) { mbar_init(&bars->d_full[i], 1); mbar_init(&bars->d_empty[i], 8); }
+    for (int i = 0; i < stages; ++i) { mbar_init(&bars->u_full[i], 1); mbar_init(&bars->u_empty[i], kRgWarps); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&bars->d_full[i], 1); mbar_init(&bars->d_empty[i], kRgWarps); }
     mbar_fence_init();
   }
-  if (warp == 9) { tmem_alloc(&bars->tmem_base, 256); tmem_relinquish(); }
+  if (warp == kRgWarps + 1) { tmem_alloc(&bars->tmem_base, 256); tmem_relinquish(); }
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
   const uint32_t tmem = bars->tmem_base;                // buffer b: r logits at 128 b, i logits at 128 b + 64
-  if (warp == 8 && lane == 0) {                         // (weights: written by no kernel of the step)
+  if (warp == kRgWarps && lane == 0) {                  // (weights: written by no kernel of the step)
     tma_prefetch_desc(&tmW);
     tma_prefetch_desc(&tmU);
     mbar_expect_tx(&bars->w_full, 2 * kc * 16384);
@@ -291,7 +293,7 @@ __global__ void __launch_bounds__(kRgThreads, 1)
     if (!runs_on || unit1 >= units) last = first;
   }
 
-  if (warp == 8) {
+  if (warp == kRgWarps) {
     if (lane == 0) {
       int k = 0;
       for (int i = first; i < last; ++i) {
@@ -307,7 +309,7 @@ __global__ void __launch_bounds__(kRgThreads, 1)
       // (the weights must not be on their way when the block ends)
       if (k == 0) mbar_wait(&bars->w_full, 0, status);
     }
-  } else if (warp == 9) {
+  } else if (warp == kRgWarps + 1) {
     if (lane == 0 && first < last) {
       const uint32_t idesc = umma_idesc_bf16(128, kUnit, 0, 0);
       const uint64_t wd0 = umma_desc_k_sw128(smem_u32(sW), 1024), ud0 = umma_desc_k_sw128(smem_u32(sU), 1024);
@@ -330,7 +332,7 @@ __global__ void __launch_bounds__(kRgThreads, 1)
       }
     }
   } else {
-    const int quarter = warp & 3, half = warp >> 2, ch = quarter * 32 + lane;       // channel of the tile
+    const int quarter = warp & 3, piece = warp >> 2, ch = quarter * 32 + lane;      // channel of the tile
     const int cb = part * 128 + ch, c = blk * p.B + cb;                             // of the block, of all
     const bool live = cb < p.B;
     const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
@@ -341,39 +343,54 @@ __global__ void __launch_bounds__(kRgThreads, 1)
     const bf16* y = reinterpret_cast<const bf16*>(p.y) + c;
     bf16* out = reinterpret_cast<bf16*>(p.out) + c;
     const int uc = min(cb >> 6, kc - 1), ux = (cb & 63) >> 3, uo = (cb & 7) * 2;    // u of this channel in a stage
+    const int t0 = piece * kPart;
     float carry = 0.f, decay = 1.f;                         // state before the unit; kSummary: decay since the slice's start
     bool ok = true;
     int k = 0;
+    bf16 yv[kPart];
+    auto load_y = [&](const RgUnit& u) {
+#pragma unroll
+      for (int t = 0; t < kPart; ++t)
+        yv[t] = live && t0 + t < u.n ? y[(size_t)(u.row0 + t0 + t) * p.ldy] : __float2bfloat16(0.f);
+    };
+    RgUnit next = {};
+    if (first < last) {
+      next = rg_unit(R, first, decode_units);
+      if (!kSummary) load_y(next);
+    }
     for (int i = first; i < last; ++i) {
-      const RgUnit u = rg_unit(R, i, decode_units);
-      if (u.n <= 0) continue;
-      const int st = k % stages, buf = k & 1, t0 = half * kHalf, n = min(max(u.n - t0, 0), kHalf);
-      bf16 yv[kHalf];
-      float before[kHalf];                                  // decode: the rows' states
-      if (!kSummary) {
-#pragma unroll
-        for (int t = 0; t < kHalf; ++t) yv[t] = live && t < n ? y[(size_t)(u.row0 + t0 + t) * p.ldy] : __float2bfloat16(0.f);
+      const RgUnit u = next;
+      if (i + 1 < last) next = rg_unit(R, i + 1, decode_units);
+      if (u.n <= 0) {
+        if (!kSummary && i + 1 < last) load_y(next);
+        continue;
       }
+      const int st = k % stages, buf = k & 1, n = min(max(u.n - t0, 0), kPart);
+      float before[kPart];                                  // decode: the rows' states
+      int slot = -1;                                        // decode: that of row t0 + lane
       if (!kSummary && u.decode) {
+        bool fresh = true;
+        if (lane < n) {
+          slot = R.slots[u.row0 + t0 + lane];
+          fresh = R.seq_lens[u.row0 + t0 + lane] <= 1;
+        }
+        const int from = fresh ? -1 : slot;
 #pragma unroll
-        for (int t = 0; t < kHalf; ++t) {
-          before[t] = 0.f;
-          if (live && t < n) {
-            const int row = u.row0 + t0 + t, slot = R.slots[row];
-            if (slot >= 0 && R.seq_lens[row] > 1) before[t] = p.state[(size_t)slot * C + c];
-          }
+        for (int t = 0; t < kPart; ++t) {
+          const int s = __shfl_sync(0xffffffffu, from, t);
+          before[t] = live && s >= 0 ? p.state[(size_t)s * C + c] : 0.f;
         }
       } else if (u.at == 0) {                               // a portion starts
-        const int slot = R.slots[u.req];
+        const int s = R.slots[u.req];
         carry = 0.f;
-        if (live && slot >= 0 && R.seq_lens[u.req] > u.len) {
+        if (live && s >= 0 && R.seq_lens[u.req] > u.len) {
           // (a later slice may already have written the state of a portion that runs on: the first pass kept it)
           const bool runs_on = (i + (u.len + kUnit - 1) / kUnit) > unit1;
-          carry = !kSummary && runs_on ? sum[2 * kind + (size_t)slice * C] : p.state[(size_t)slot * C + c];
+          carry = !kSummary && runs_on ? sum[2 * kind + (size_t)slice * C] : p.state[(size_t)s * C + c];
         }
         if (kSummary) {
           decay = 0.f;
-          if (live && half == 0) sum[2 * kind + (size_t)slice * C] = carry;
+          if (live && piece == 0) sum[2 * kind + (size_t)slice * C] = carry;
         }
       } else if (i == first && !kSummary && live) {         // a portion of earlier slices goes on
         const int from = (i - u.at / kUnit) / per_slice;
@@ -382,9 +399,9 @@ __global__ void __launch_bounds__(kRgThreads, 1)
       }
       ok = ok && __all_sync(0xffffffffu, mbar_wait(&bars->d_full[buf], (k >> 1) & 1, status));
       tc_fence_after_sync();
-      uint32_t lr[kHalf], li[kHalf];
-      tmem_ld_32x32b_x32(tmem + buf * 128 + t0 + lane_off, lr);
-      tmem_ld_32x32b_x32(tmem + buf * 128 + 64 + t0 + lane_off, li);
+      uint32_t lr[kPart], li[kPart];
+      tmem_ld_32x32b_x16(tmem + buf * 128 + t0 + lane_off, lr);
+      tmem_ld_32x32b_x16(tmem + buf * 128 + 64 + t0 + lane_off, li);
       tmem_ld_wait();
       tc_fence_before_sync();
       __syncwarp();
@@ -392,56 +409,60 @@ __global__ void __launch_bounds__(kRgThreads, 1)
       const uint8_t* us = sU + (st * kc + uc) * 8192 + t0 * 128 + uo;
       float D = 1.f, S = 0.f;
 #pragma unroll
-      for (int t = 0; t < kHalf; ++t) {
+      for (int t = 0; t < kPart; ++t) {
         const float r = rg_sigmoid(__uint_as_float(lr[t]) + bias_r), g = rg_sigmoid(__uint_as_float(li[t]) + bias_i);
         const float x = __bfloat162float(*reinterpret_cast<const bf16*>(us + t * 128 + ((ux ^ (t & 7)) << 4)));
         const float la = rate * r, a = __expf(la);
         const float b = rg_sqrt(rg_one_minus_exp(2.f * la, a * a)) * g * x;
         lr[t] = __float_as_uint(t < n ? a : 1.f);
         li[t] = __float_as_uint(t < n ? b : 0.f);
-        D *= t < n ? a : 1.f;
-        S = t < n ? fmaf(a, S, b) : S;
+        D *= __uint_as_float(lr[t]);
+        S = fmaf(__uint_as_float(lr[t]), S, __uint_as_float(li[t]));
       }
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->u_empty[st]);
-      auto gelu = [&](bf16 v) {                             // z / (1 + exp(-2 x)) is z (1 + tanh x) / 2
-        const float z = __bfloat162float(v);
-        return __fdividef(z, 1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+      auto gelu = [&](bf16 v) {                             // w / (1 + exp(-2 x)) is w (1 + tanh x) / 2
+        const float w = __bfloat162float(v);
+        return __fdividef(w, 1.f + __expf(-1.5957691216057308f * (w + 0.044715f * w * w * w)));
       };
       if (!kSummary && u.decode) {
 #pragma unroll
-        for (int t = 0; t < kHalf; ++t) {
+        for (int t = 0; t < kPart; ++t) {
+          const int to = __shfl_sync(0xffffffffu, slot, t);
           if (live && t < n) {
-            const int row = u.row0 + t0 + t, slot = R.slots[row];
             const float s = fmaf(__uint_as_float(lr[t]), before[t], __uint_as_float(li[t]));
-            out[(size_t)row * p.ldo] = __float2bfloat16(s * gelu(yv[t]));
-            if (slot >= 0) p.state[(size_t)slot * C + c] = s;
+            out[(size_t)(u.row0 + t0 + t) * p.ldo] = __float2bfloat16(s * gelu(yv[t]));
+            if (to >= 0) p.state[(size_t)to * C + c] = s;
           }
         }
       } else {
-        bars->xch[k & 1][half][ch] = make_float2(D, S);
-        asm volatile("bar.sync 1, 256;" ::: "memory");
-        const float2 h0 = bars->xch[k & 1][0][ch], h1 = bars->xch[k & 1][1][ch];
-        const float mid = fmaf(h0.x, carry, h0.y), end = fmaf(h1.x, mid, h1.y);
-        if (kSummary) {
-          decay *= h0.x * h1.x;
-        } else {
-          float s = half ? mid : carry;
+        bars->xch[k & 1][piece][ch] = make_float2(D, S);
+        asm volatile("bar.sync 1, %0;" ::"n"(kRgWarps * 32) : "memory");
+        float s = carry, end = carry;
 #pragma unroll
-          for (int t = 0; t < kHalf; ++t) {
+        for (int q = 0; q < kParts; ++q) {
+          const float2 h = bars->xch[k & 1][q][ch];
+          if (q == piece) s = end;
+          end = fmaf(h.x, end, h.y);
+          if (kSummary) decay *= h.x;
+        }
+        if (!kSummary) {
+#pragma unroll
+          for (int t = 0; t < kPart; ++t) {
             s = fmaf(__uint_as_float(lr[t]), s, __uint_as_float(li[t]));
             if (live && t < n) out[(size_t)(u.row0 + t0 + t) * p.ldo] = __float2bfloat16(s * gelu(yv[t]));
           }
-          if (live && half == 0 && u.at + u.n >= u.len) {
-            const int slot = R.slots[u.req];
-            if (slot >= 0) p.state[(size_t)slot * C + c] = end;
+          if (live && piece == 0 && u.at + u.n >= u.len) {
+            const int to = R.slots[u.req];
+            if (to >= 0) p.state[(size_t)to * C + c] = end;
           }
         }
         carry = end;
       }
+      if (!kSummary && i + 1 < last) load_y(next);          // (used at the end of the next unit)
       ++k;
     }
-    if (kSummary && live && half == 0 && first < last) {
+    if (kSummary && live && piece == 0 && first < last) {
       sum[(size_t)slice * C] = carry;
       sum[kind + (size_t)slice * C] = decay;
     }
@@ -449,7 +470,7 @@ __global__ void __launch_bounds__(kRgThreads, 1)
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
-  if (warp == 9) tmem_dealloc(tmem, 256);
+  if (warp == kRgWarps + 1) tmem_dealloc(tmem, 256);
 }
 
 static size_t rg_smem(int B, int stages) {

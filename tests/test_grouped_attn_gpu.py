@@ -178,7 +178,7 @@ def test_rotation_unit_norm_and_cache(dtype, shape):
     only_q = torch.empty_like(q)
     A.rotate_kv(qkv[:, : H * D].contiguous().to(DEV), pos.to(DEV), table, rot, eps, only_q, slots.to(DEV), cache, H=H, G=0, D=D,
                 V=V, dim=dim, block_size=bs)
-    assert torch.equal(only_q, q)
+    assert (only_q.double() - q.double()).abs().max() < tol
 
 
 @pytest.mark.parametrize("width", [40, 37, 1024, 5000])

@@ -1,8 +1,9 @@
 """Throughput of a design with listed layers beside the closest other model of this package at equal layer
 sizes, and its kernels beside the like kernels of that model, each against its roofline.
 
-``bench.py --design nufusun`` (beside Qwen3-MoE) or ``--design diforax`` (beside the Qwen3.5 MoE hybrids) runs
-it and prints one JSON line. Random weights; device time (CUDA events); kernels are timed with an L2 flush
+``bench.py --design nufusun`` (beside Qwen3-MoE), ``--design diforax`` (beside the Qwen3.5 MoE hybrids) or
+``--design tabupel`` (beside the dense Qwen3.5 hybrids, its latent kernels beside DeepSeek-V2's) runs it and
+prints one JSON line. Random weights; device time (CUDA events); kernels are timed with an L2 flush
 between iterations, median of several."""
 from __future__ import annotations
 
@@ -28,6 +29,41 @@ DIFORAX_SIZES = {
     "small layers": (1024, 16, 4, 128, 32, 4, 512, 8, 16, 8),
     "wide layers": (4096, 32, 8, 128, 16, 2, 2048, 4, 48, 16),
 }
+
+
+# width, dense size, layers; differential heads, kv heads, size (values twice as wide); latent heads, query and
+# key latent; recurrent width, its blocks
+TABUPEL_FIELDS = ("width", "ff", "layers", "heads", "kv_heads", "head", "latent_heads", "q_rank", "kv_rank", "recurrent", "blocks")
+TABUPEL_SIZES = {
+    "2b layers": (2560, 7680, 6, 20, 4, 64, 16, 1536, 512, 2560, 10),
+    "wide heads": (2048, 6144, 6, 8, 2, 128, 16, 1024, 512, 2048, 8),
+    "small layers": (1024, 3072, 12, 8, 4, 64, 8, 512, 512, 1024, 8),
+    "wide layers": (4096, 12288, 6, 32, 8, 64, 16, 1536, 512, 4096, 16),
+}
+
+
+def tabupel_configs(size):
+    """Two recurrent layers to one attention layer, latent and differential in turn; windows longer than the
+    prompts, as the other model's attention has no limit. The other model: the same pattern of delta-rule layers
+    and attention layers with heads as wide as a head's two maps."""
+    from ..config import (AttentionSpec, BlockSpec, DenseSpec, LatentSpec, ModelConfig, RglruSpec, RopeConfig, RotaryScaling,
+                          model_config_of_blocks)
+    W, ff, layers, H, G, D, LH, qr, kr, rec, nb = size
+    mlp, win = DenseSpec(ff), 1 << 15
+    r = BlockSpec(None, mlp, rglru=RglruSpec(width=rec, blocks=nb, conv=4))
+    a = BlockSpec(None, mlp, latent=LatentSpec(heads=LH, dim=128, rot_dim=64, vdim=128, q_rank=qr, kv_rank=kr, scale=192 ** -0.5,
+                                               window=win, rot_base=1e4, rot_scaling=RotaryScaling(40.0, 4096)))
+    d = BlockSpec(AttentionSpec(heads=H, kv_heads=G, dim=D, vdim=2 * D, scale=D ** -0.5, rot_dims=D, rot_base=1e6,
+                                rot_scaling=RotaryScaling(8.0), window=win, diff=0.5), mlp)
+    mine = model_config_of_blocks("Tabupel", [(r, r, a, r, r, d)[l % 6] for l in range(layers)], vocab=32000, width=W, eps=1e-6,
+                                  residual_mult=0.5, logit_softcap=30.0)
+    other = ModelConfig(architecture="Qwen3_5ForConditionalGeneration", vocab_size=32000, hidden_size=W, intermediate_size=ff,
+                        num_layers=layers, num_heads=H, num_kv_heads=G, head_dim=2 * D, max_position_embeddings=32768, qk_norm=True,
+                        gemma_norm=True, attn_output_gate=True, rope=RopeConfig(theta=1e6),
+                        layer_types=["full_attention" if l % 3 == 2 else "linear_attention" for l in range(layers)],
+                        linear_num_key_heads=max(1, rec // 256), linear_num_value_heads=max(2, rec // 128), linear_key_head_dim=128,
+                        linear_value_head_dim=128, linear_conv_kernel_dim=4)
+    return {"tabupel": mine, "qwen3.5": other}
 
 
 def diforax_configs(size):
@@ -436,7 +472,239 @@ class DiforaxKernels(KernelBench):
                      nbytes=T * W * 2 * 4)
 
 
-DESIGNS = {"nufusun": (NUFUSUN_SIZES, nufusun_configs, NufusunKernels), "diforax": (DIFORAX_SIZES, diforax_configs, DiforaxKernels)}
+class TabupelKernels(KernelBench):
+    def __init__(self, size):
+        super().__init__((size[0], *size[3:6], 1, 1, size[1]))
+        self.LH, self.qr, self.kr, self.rec, self.nb = size[6:]
+
+    def run(self):
+        self.attention(B=4, prompt=2048, decode_batch=64, ctx=4096)
+        self.attention(B=8, prompt=1024, decode_batch=8, ctx=16384)
+        self.latent(B=4, prompt=2048, decode_batch=64, ctx=4096)
+        self.latent(B=8, prompt=1024, decode_batch=8, ctx=16384)
+        for B, n in ((4, 2048), (8, 1024), (1, 8192), (16, 1), (64, 1), (256, 1)):
+            self.recurrence(B, n)
+        for T in (64, 8192):
+            self.rest(T)
+
+    def step_rows(self, B, prompt, bs):
+        from ..ops.reference import build_prefill_tiles
+        nb = prompt // bs
+        bt = torch.arange(1, B * nb + 1, device=self.dev, dtype=torch.int32).view(B, nb)
+        tr, tq = (self.i32(x) for x in build_prefill_tiles([prompt] * B))
+        return bt, dict(seq_lens=self.i32([prompt] * B), q_start=self.i32([i * prompt for i in range(B + 1)]), tile_req=tr, tile_q0=tq)
+
+    @staticmethod
+    def pairs(B, n, window):
+        w = min(window or n, n)
+        return B * (w * (w + 1) / 2 + (n - w) * w)
+
+    def attention(self, B, prompt, decode_batch, ctx, bs=32):
+        from .. import ops
+        from ..ops import bias_attn as A
+        H, G, D = self.H, self.G, self.D
+        V, T = 2 * D, B * prompt
+        row = G * (2 * D + V)
+        bt, rows = self.step_rows(B, prompt, bs)
+        shape = dict(H=2 * H, G=G, kw=2 * G * D, vdim=V, block_size=bs, grouped=True, maps=2, scale=D ** -0.5)
+        q, pages = self.rnd(T, 2 * H * D), self.rnd(B * prompt // bs + 1, bs * row)
+        maps = torch.empty(T, 2 * H * V, dtype=torch.bfloat16, device=self.dev)
+        q2, kv = self.rnd(T, H * V), self.rnd(B * prompt // bs + 1, 2, bs, G, V)
+        out = torch.empty(T, H * V, dtype=torch.bfloat16, device=self.dev)
+        for window in (0, 512):
+            what = f"attention, {B} x {prompt} prompt" + (f", window {window}" if window else "")
+            n = self.pairs(B, prompt, window)
+            self.add(what, "tabupel", lambda: A.prefill(q, pages, maps, block_table=bt, num_reqs=B, window=window, **rows, **shape),
+                     flops=2 * n * 2 * H * (D + V), note=A.kernel_kind("prefill", q, pages, window=window, **shape))
+            self.add(what, "qwen3.5", lambda: ops.attn_prefill(q2, kv, block_table=bt, num_q_heads=H, num_kv_heads=G, head_dim=V,
+                                                               block_size=bs, scale=V ** -0.5, window=window, out=out, **rows),
+                     flops=2 * n * H * 2 * V)
+        qkv, pos = self.rnd(T, 2 * (H + G) * D + G * V), torch.arange(T, device=self.dev) % prompt
+        slots = (bt.long()[:, :, None] * bs + torch.arange(bs, device=self.dev)).reshape(-1)
+        table, nw = self.rnd(prompt, D, dtype=torch.float32), self.rnd(D, dtype=torch.float32)
+        nbytes = T * 2 * (2 * (H + G) * D + G * V) * 2
+        self.add(f"query preparation + cache write, {T} tokens", "tabupel",
+                 lambda: A.rotate_kv(qkv, pos, table, D, 1e-6, q, slots, pages, H=2 * H, G=2 * G, value_heads=G, D=D, V=V, dim=D,
+                                     block_size=bs, q_w=nw, k_w=nw), nbytes=nbytes)
+        qkv2, nw2 = self.rnd(T, (H + 2 * G) * V), self.rnd(V)
+        table2 = self.rnd(prompt, V, dtype=torch.float32)
+        self.add(f"query preparation + cache write, {T} tokens", "qwen3.5",
+                 lambda: ops.rope_kv(qkv2, pos, table2, num_q_heads=H, num_kv_heads=G, head_dim=V, q_norm=nw2, k_norm=nw2,
+                                     slot_mapping=slots, kv_cache=kv, block_size=bs, q_out=q2), nbytes=T * 2 * (H + 2 * G) * V * 2)
+        from ..ops import gdn as Q
+        self.add(f"difference of the maps + norm, {T} tokens", "tabupel",
+                 lambda: A.diff_combine(maps, out, H=H, V=V, vdim=V, lam=0.4, eps=1e-6, scale=0.5), nbytes=T * 3 * H * V * 2)
+        a, b = self.rnd(T, H * 128), self.rnd(T, H * 128)
+        core, nw3 = torch.empty_like(a), self.rnd(128)
+        self.add(f"difference of the maps + norm, {T} tokens", "qwen3.5",
+                 lambda: Q.rmsnorm_gated(a, b, nw3, core, heads=H), nbytes=T * 3 * H * 128 * 2, note="norm and gate of two rows")
+        B, nb = decode_batch, ctx // bs
+        bt = torch.arange(1, B * nb + 1, device=self.dev, dtype=torch.int32).view(B, nb)
+        sl = self.i32([ctx] * B)
+        pages, kv, q, q2 = self.rnd(B * nb + 1, bs * row), self.rnd(B * nb + 1, 2, bs, G, V), self.rnd(B, 2 * H * D), self.rnd(B, H * V)
+        maps, out = (torch.empty(B, n * H * V, dtype=torch.bfloat16, device=self.dev) for n in (2, 1))
+        splits = A.grouped_decode_splits(B, G, ctx, ops.num_sms())
+        tmp = (torch.empty(B * 2 * H * splits * V, dtype=torch.float32, device=self.dev),
+               torch.empty(B * 2 * H * splits, dtype=torch.float32, device=self.dev))
+        nbytes = B * ctx * row * 2
+        self.add(f"attention, decode {B} x {ctx}", "tabupel",
+                 lambda: A.decode(q, pages, maps, block_table=bt, seq_lens=sl, splits=splits, tmp=tmp, **shape), nbytes=nbytes,
+                 note=A.kernel_kind("decode", q, pages, **shape))
+        self.add(f"attention, decode {B} x {ctx}", "qwen3.5",
+                 lambda: ops.attn_decode(q2, kv, block_table=bt, seq_lens=sl, num_q_heads=H, num_kv_heads=G, head_dim=V,
+                                         block_size=bs, scale=V ** -0.5, out=out), nbytes=nbytes)
+
+    def latent(self, B, prompt, decode_batch, ctx, bs=32):
+        from .. import ops
+        from ..ops import latent as L
+        from ..ops import mla as M
+        H, T = self.LH, B * prompt
+        s = L.LatentShape(H=H, dim=128, rot=64, vdim=128, q_rank=self.qr, rank=self.kr)
+        scale, gate = 192 ** -0.5, self.rnd(T, s.down[3])
+        bt, rows = self.step_rows(B, prompt, bs)
+        cache, q = self.rnd(B * prompt // bs + 1, bs * s.row), self.rnd(T, H * s.qw)
+        out = torch.empty(T, H * s.V, dtype=torch.bfloat16, device=self.dev)
+        wkv = self.rnd(H * (s.D + s.V), s.rankp, s=0.05)
+        dense, kvb = self.rnd(T, s.row), self.rnd(T, H * (s.D + s.V))
+        n = self.pairs(B, prompt, 0)
+        first, base, total, table = L.visible_pages([prompt] * B, [prompt] * B, 0, bs)
+        first, base, table = self.i32(first.tolist()), self.i32(base.tolist()), torch.from_numpy(table).to(self.dev)
+        flops = 2 * n * H * (192 + 128)
+        self.add(f"latent attention, {B} x {prompt} prompt", "tabupel",
+                 lambda: L.prefill_expanded(q, kvb, dense, out, s, block_table=table, num_reqs=B, scale=scale, window=0,
+                                            block_size=bs, gate=gate, **rows), flops=flops)
+        qpad, pages = self.rnd(T, H * 256), self.rnd(T // bs, 2, bs, H, 256)
+        attn = torch.empty(T, H * 256, dtype=torch.bfloat16, device=self.dev)
+        sl, qs, tr, tq = (rows[k] for k in ("seq_lens", "q_start", "tile_req", "tile_q0"))
+        ident = torch.arange(T // bs, device=self.dev, dtype=torch.int32).view(B, -1)
+        theirs = H <= 16 and self.kr == 512
+        self.add(f"latent attention, {B} x {prompt} prompt", "deepseek-v2",
+                 lambda: ops.attn_prefill(qpad, pages, block_table=ident, num_q_heads=H, num_kv_heads=H, head_dim=256, block_size=bs,
+                                          scale=scale, out=attn, **rows), flops=flops, note="heads padded to 256")
+
+        def expand():
+            L.gather(cache, bt, sl, first, base, bs, dense, B, table.shape[1])
+            ops.gemm(dense[:, : s.rankp], wkv, out=kvb, const_w=True)
+
+        def their_expand():
+            M.gather_latent(cache, bt, sl, base * bs, bs, dense, B, prompt // bs)
+            ops.gemm(dense[:, :512], wkv, out=kvb)
+            M.assemble_kv(kvb, dense, pages, T, H, bs)
+            M.pad_q(q, qpad, T, H)
+        nbytes = T * (2 * s.row + H * (s.D + s.V)) * 2
+        fl = 2.0 * T * s.rankp * H * (s.D + s.V)
+        self.add(f"latent rows to keys and values, {T} tokens", "tabupel", expand, nbytes=nbytes, flops=fl, note="gather, product")
+        if theirs:
+            self.add(f"latent rows to keys and values, {T} tokens", "deepseek-v2", their_expand, nbytes=nbytes, flops=fl,
+                     note="gather, product, assembly of keys, padding of queries")
+        # ---- preparation
+        down, cq = self.rnd(T, sum(s.down)), torch.empty(T, s.down[0], dtype=torch.bfloat16, device=self.dev)
+        f32 = dict(dtype=torch.float32)
+        w = {"q_norm": self.rnd(s.down[0], **f32), "kv_norm": self.rnd(s.down[1], **f32)}
+        pos, tab = torch.arange(T, device=self.dev) % prompt, self.rnd(prompt, 64, **f32)
+        slots = (bt.long()[:, :, None] * bs + torch.arange(bs, device=self.dev)).reshape(-1)
+        self.add(f"latent preparation, {T} tokens", "tabupel",
+                 lambda: L.prepare(down, pos, tab, w, s, 1e-6, cq, slots, cache), nbytes=T * 2 * (sum(s.down[:3]) * 2))
+        self.add(f"latent queries, {T} tokens", "tabupel", lambda: L.queries(q, pos, tab, s, None, 0), nbytes=T * H * 64 * 2 * 2)
+        qa = self.rnd(T, H * 192 + 576)
+        kvn, cache3 = self.rnd(512), self.rnd(B * prompt // bs + 1, bs, 576)
+        kvc, kpe = qa[:, H * 192: H * 192 + 512], qa[:, H * 192 + 512:]
+
+        def their_prep():
+            ops.rope_kv(qa, pos, tab, num_q_heads=H, num_kv_heads=1, head_dim=64, rot_dim=64, neox=False, q_head_stride=192,
+                        offsets=(128, H * 192 + 512, 0))
+            ops.rmsnorm(kvc, kvn, 1e-6, out=kvc)
+            ops.concat_and_cache_mla(kvc, kpe, slots, cache3)
+        self.add(f"latent preparation and queries, {T} tokens", "deepseek-v2", their_prep, nbytes=T * 2 * (H * 64 * 2 + 576 * 2),
+                 note="three kernels, no query latent")
+        # ---- decode
+        B, nb = decode_batch, ctx // bs
+        bt = torch.arange(1, B * nb + 1, device=self.dev, dtype=torch.int32).view(B, nb)
+        sl, cache = self.i32([ctx] * B), self.rnd(B * nb + 1, bs * s.row)
+        qabs, olat = self.rnd(B, H * s.row), torch.empty(B, H * s.rankp, dtype=torch.bfloat16, device=self.dev)
+        splits = L.decode_splits(B, H, ctx, ops.num_sms())
+        tmp = (torch.empty(B * H * splits * s.rankp, dtype=torch.float32, device=self.dev),
+               torch.empty(B * H * splits, dtype=torch.float32, device=self.dev))
+        for window in (0, 1024):
+            keys = min(window or ctx, ctx)
+            what = f"latent attention, decode {B} x {ctx}" + (f", window {window}" if window else "")
+            self.add(what, "tabupel", lambda: L.decode(qabs, cache, olat, s, block_table=bt, seq_lens=sl, scale=scale, window=window,
+                                                       block_size=bs, gate=gate[:B], splits=splits, tmp=tmp),
+                     nbytes=B * keys * s.row * 2)
+        if theirs:
+            q3, c3 = qabs.view(B, H, 576), cache.view(-1, bs, 576)
+            self.add(f"latent attention, decode {B} x {ctx}", "deepseek-v2",
+                     lambda: M.mla_decode(q3, c3, bt, sl, olat, scale, bs, splits=splits,
+                                          tmp=(tmp[0].view(B, H, splits, 512), tmp[1].view(B, H, splits))), nbytes=B * ctx * 576 * 2)
+
+    def recurrence(self, B, n):
+        """``B`` prompts of ``n`` tokens, or (n 1) a decode batch: convolution, then gates and recurrence."""
+        from types import SimpleNamespace
+        from ..ops import gdn as Q
+        from ..ops import rglru as G
+        from ..ops.reference import build_prefill_tiles
+        s, T, C = G.RglruShape(blocks=self.nb, size=self.rec // self.nb, taps=4), B * n, self.rec
+        f32 = dict(dtype=torch.float32)
+        tr, tq = build_prefill_tiles([n] * B) if n > 1 else ([], [])
+        rows = SimpleNamespace(seq_lens=self.i32([n + 5] * B), state_slots=self.i32(list(range(B))),
+                               prefill_q_start=self.i32([i * n for i in range(B + 1)]), tile_req=self.i32(tr or [0]),
+                               tile_q0=self.i32(tq or [0]), num_decodes=B if n == 1 else 0, num_prefills=0 if n == 1 else B,
+                               num_tiles=len(tr))
+        proj, u, out = self.rnd(T, 2 * C), self.rnd(T, C), torch.empty(T, C, dtype=torch.bfloat16, device=self.dev)
+        w = {"gates": self.rnd(s.blocks, 2, s.M, s.B, s=0.05), "gate_bias": self.rnd(2, C, **f32), "rate": -self.rnd(C, **f32).abs()}
+        cw, cb, conv = self.rnd(4, C, **f32), self.rnd(C, **f32), self.rnd(B, 3, C)
+        state, bufs = torch.zeros(B, C, device=self.dev), {"summary": torch.empty(G.summary_values(s), device=self.dev)}
+        what = f"{B} x {n} prompt" if n > 1 else f"decode {B}"
+        self.add(f"convolution, {what}", "tabupel", lambda: G.short_conv(proj[:, C:], cw, cb, conv, rows, u),
+                 nbytes=(T * 2 + B * 6) * C * 2)
+        a = G.rglru_args(u, proj[:, :C], w, s, state, rows, bufs, out)
+        self.add(f"gates + recurrence, {what}", "tabupel", lambda: G.run_rglru(a),
+                 nbytes=T * C * 6 + B * C * 8 + 2 * C * s.B * 2, flops=2.0 * T * C * 2 * s.B)
+        # the delta rule of as many channels
+        H, K, D = max(2, C // 128), max(1, C // 256), 128
+        CC = 2 * K * D + H * D
+        x, xc, cw2, cst = self.rnd(T, CC), self.rnd(T, CC), self.rnd(CC, 4), self.rnd(B, CC, 3)
+        st2, z, core = torch.zeros(B, H, D, D, device=self.dev), self.rnd(T, H * D), torch.empty(T, H * D, dtype=torch.bfloat16, device=self.dev)
+        slots, init, nw = rows.state_slots, self.i32([1] * B), self.rnd(D)
+        A, dt = self.rnd(H, **f32).abs(), self.rnd(H, **f32)
+        if n == 1:
+            ab = self.rnd(T, 2 * H)
+            self.add(f"convolution, {what}", "qwen3.5", lambda: Q.conv1d_update(x, cw2, cst, slots, xc), nbytes=(T * 2 + B * 6) * CC * 2)
+
+            def theirs():
+                Q.packed_decode(xc, ab[:, :H], ab[:, H:], A, dt, st2, slots, core.view(T, H, D), K, H)
+                Q.rmsnorm_gated(core, z, nw, core, heads=H)
+        else:
+            q, k = self.rnd(T, K, D), self.rnd(T, K, D)
+            g, beta = -self.rnd(T, H, **f32).abs(), self.rnd(T, H, **f32).abs()
+            ws, host = Q.GdnWorkspace(self.dev, T, B, H), [i * n for i in range(B + 1)]
+            table = tuple(self.i32(x.tolist()) for x in Q.build_chunk_table(host))
+            self.add(f"convolution, {what}", "qwen3.5", lambda: Q.conv1d_fwd(x, cw2, cst, rows.prefill_q_start, slots, init, xc),
+                     nbytes=(T * 2 + B * 6) * CC * 2)
+
+            def theirs():
+                Q.chunk_scan(q, k, xc, g, beta, st2, host, slots, init, core.view(T, H, D), ws, v_col0=2 * K * D, table=table)
+                Q.rmsnorm_gated(core, z, nw, core, heads=H)
+        self.add(f"gates + recurrence, {what}", "qwen3.5", theirs,
+                 nbytes=T * (2 * K * D + 3 * H * D) * 2 + B * H * D * D * 8, flops=T * H * (6.0 * D * D + 4 * 64 * D) if n > 1 else 0,
+                 note="delta rule + norm")
+
+    def rest(self, T):
+        from .. import ops
+        from ..ops.stream import softcap_f32, stream_norm
+        W = self.W
+        out, stream, mixed, nw = self.rnd(T, W), self.rnd(T, W, dtype=torch.float32), self.rnd(T, W, dtype=torch.float32), self.rnd(W, dtype=torch.float32)
+        self.add(f"residual + norm, {T} tokens", "tabupel",
+                 lambda: stream_norm(stream, nw, 1e-6, out, width=W, a=mixed, norm_offset=0.0, mult=0.5), nbytes=T * W * (4 + 4 + 4 + 2))
+        o2, res, nwb = torch.empty_like(out), self.rnd(T, W), nw.to(torch.bfloat16)
+        self.add(f"residual + norm, {T} tokens", "qwen3.5", lambda: ops.rmsnorm(o2, nwb, 1e-6, residual=res, out=out), nbytes=T * W * 2 * 4)
+        if T <= 64:
+            logits = self.rnd(T, 32000, dtype=torch.float32)
+            self.add(f"logit cap, {T} rows", "tabupel", lambda: softcap_f32(logits, 30.0), nbytes=T * 32000 * 8)
+
+
+DESIGNS = {"nufusun": (NUFUSUN_SIZES, nufusun_configs, NufusunKernels), "diforax": (DIFORAX_SIZES, diforax_configs, DiforaxKernels),
+           "tabupel": (TABUPEL_SIZES, tabupel_configs, TabupelKernels)}
 
 
 def run(design="nufusun", sizes=None, kernels=True) -> dict:
@@ -445,7 +713,7 @@ def run(design="nufusun", sizes=None, kernels=True) -> dict:
     res = {"metric": "design_layer_throughput", "unit": "tok/s", "impl": "ours", "design": design, "dtype": "bf16",
            "data": "synthetic (uniform-random prompt ids, random-init weights)",
            "roofline": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": how}, "models": {}, "kernels": {}}
-    names = FIELDS + (("delta_heads", "delta_key_heads") if design == "diforax" else ())
+    names = TABUPEL_FIELDS if design == "tabupel" else FIELDS + (("delta_heads", "delta_key_heads") if design == "diforax" else ())
     for name, size in table.items():
         if sizes and name not in sizes:
             continue

@@ -55,10 +55,12 @@ class TabupelModel(ListedModel):
     # ------------------------------------------------------------------ weights
     def init_random(self, seed: int = 0, std: float = 0.02) -> None:
         c, W = self.cfg, self.width
-        g = torch.Generator().manual_seed(seed)
+        big = sum(b.mlp.ff * 3 * W for b in c.blocks if b.mlp is not None) > 2e8
+        gdev = self.device if (self.device.type == "cuda" and big) else torch.device("cpu")
+        g = torch.Generator(device=gdev).manual_seed(seed)
 
         def full(*shape, s=std, mean=0.0):
-            return torch.empty(shape, dtype=torch.float32).normal_(mean, s, generator=g).to(torch.bfloat16)
+            return torch.empty(shape, dtype=torch.float32, device=gdev).normal_(mean, s, generator=g).to(torch.bfloat16)
 
         def norm(n):
             return full(n, s=0.1, mean=1.0)
