@@ -230,17 +230,34 @@ __device__ __forceinline__ RgUnit rg_unit(const B200Rows& R, int i, int decode_u
   return u;
 }
 
-__device__ __forceinline__ float rg_sigmoid(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+static constexpr float kRgLog2e = 1.4426950408889634f;
+
+__device__ __forceinline__ float rg_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rg_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ float rg_sqrt(float x) {
   float y;
   asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// 1 - exp(x) for x <= 0: near 0 the series of expm1
+// 1 - exp(x) for x <= 0, ex = exp(x): near 0 the series of expm1
 __device__ __forceinline__ float rg_one_minus_exp(float x, float ex) {
-  const float series = -x * (1.f + x * (0.5f + x * (1.f / 6.f + x * (1.f / 24.f + x * (1.f / 120.f)))));
-  return x > -0.1f ? series : 1.f - ex;
+  const float series = -x * fmaf(x, fmaf(x, fmaf(x, 1.f / 24.f, 1.f / 6.f), 0.5f), 1.f);
+  return x > -0.02f ? series : 1.f - ex;
 }
+// w (1 + tanh z) / 2 with z = sqrt(2 / pi) (w + 0.044715 w^3), as w / (1 + exp(-2 z))
+__device__ __forceinline__ float rg_gelu(float w) {
+  const float k = -2.f * 0.7978845608028654f * kRgLog2e;
+  return w * rg_rcp(1.f + rg_ex2(w * fmaf(w * w, 0.044715f * k, k)));
+}
+template <bool B> struct RgFlag { static constexpr bool value = B; };
 
 template <bool kSummary>
 __global__ void __launch_bounds__(kRgThreads, 1)
@@ -336,12 +353,14 @@ __global__ void __launch_bounds__(kRgThreads, 1)
     const int cb = part * 128 + ch, c = blk * p.B + cb;                             // of the block, of all
     const bool live = cb < p.B;
     const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
-    const float bias_r = live ? p.gate_bias[c] : 0.f, bias_i = live ? p.gate_bias[C + c] : 0.f;
-    const float rate = live ? p.rate[c] : 0.f;
+    // (sigmoid(x + bias) as 1 / (1 + 2^(-log2(e) (x + bias))))
+    const float bias_r = live ? -kRgLog2e * p.gate_bias[c] : 0.f, bias_i = live ? -kRgLog2e * p.gate_bias[C + c] : 0.f;
+    const float rate = live ? p.rate[c] : 0.f, rate_l2 = rate * kRgLog2e;
     float* sum = p.summary + c;
     const size_t kind = (size_t)B200_RGLRU_SLICES * C;      // summary: end states | decays | starting states
-    const bf16* y = reinterpret_cast<const bf16*>(p.y) + c;
-    bf16* out = reinterpret_cast<bf16*>(p.out) + c;
+    const bf16* y = reinterpret_cast<const bf16*>(p.y);
+    bf16* out = reinterpret_cast<bf16*>(p.out);
+    const uint32_t ldy = (uint32_t)p.ldy, ldo = (uint32_t)p.ldo;                    // (offsets below 2^31: checked)
     const int uc = min(cb >> 6, kc - 1), ux = (cb & 63) >> 3, uo = (cb & 7) * 2;    // u of this channel in a stage
     const int t0 = piece * kPart;
     float carry = 0.f, decay = 1.f;                         // state before the unit; kSummary: decay since the slice's start
@@ -349,9 +368,14 @@ __global__ void __launch_bounds__(kRgThreads, 1)
     int k = 0;
     bf16 yv[kPart];
     auto load_y = [&](const RgUnit& u) {
+      const uint32_t at = (uint32_t)(u.row0 + t0) * ldy + c;
+      if (live && t0 + kPart <= u.n) {
 #pragma unroll
-      for (int t = 0; t < kPart; ++t)
-        yv[t] = live && t0 + t < u.n ? y[(size_t)(u.row0 + t0 + t) * p.ldy] : __float2bfloat16(0.f);
+        for (int t = 0; t < kPart; ++t) yv[t] = y[at + t * ldy];
+      } else {
+#pragma unroll
+        for (int t = 0; t < kPart; ++t) yv[t] = live && t0 + t < u.n ? y[at + t * ldy] : __float2bfloat16(0.f);
+      }
     };
     RgUnit next = {};
     if (first < last) {
@@ -408,30 +432,32 @@ __global__ void __launch_bounds__(kRgThreads, 1)
       if (lane == 0) mbar_arrive(&bars->d_empty[buf]);
       const uint8_t* us = sU + (st * kc + uc) * 8192 + t0 * 128 + uo;
       float D = 1.f, S = 0.f;
+      auto reduce = [&](auto full) {                        // decays to lr, inputs to li
 #pragma unroll
-      for (int t = 0; t < kPart; ++t) {
-        const float r = rg_sigmoid(__uint_as_float(lr[t]) + bias_r), g = rg_sigmoid(__uint_as_float(li[t]) + bias_i);
-        const float x = __bfloat162float(*reinterpret_cast<const bf16*>(us + t * 128 + ((ux ^ (t & 7)) << 4)));
-        const float la = rate * r, a = __expf(la);
-        const float b = rg_sqrt(rg_one_minus_exp(2.f * la, a * a)) * g * x;
-        lr[t] = __float_as_uint(t < n ? a : 1.f);
-        li[t] = __float_as_uint(t < n ? b : 0.f);
-        D *= __uint_as_float(lr[t]);
-        S = fmaf(__uint_as_float(lr[t]), S, __uint_as_float(li[t]));
-      }
+        for (int t = 0; t < kPart; ++t) {
+          const float r = rg_rcp(1.f + rg_ex2(fmaf(__uint_as_float(lr[t]), -kRgLog2e, bias_r)));
+          const float g = rg_rcp(1.f + rg_ex2(fmaf(__uint_as_float(li[t]), -kRgLog2e, bias_i)));
+          const float x = __bfloat162float(*reinterpret_cast<const bf16*>(us + t * 128 + ((ux ^ (t & 7)) << 4)));
+          float a = rg_ex2(rate_l2 * r), b = rg_sqrt(rg_one_minus_exp(2.f * rate * r, a * a)) * (g * x);
+          if (!decltype(full)::value && t >= n) { a = 1.f; b = 0.f; }
+          lr[t] = __float_as_uint(a);
+          li[t] = __float_as_uint(b);
+          D *= a;
+          S = fmaf(a, S, b);
+        }
+      };
+      if (n == kPart) reduce(RgFlag<true>());
+      else reduce(RgFlag<false>());
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->u_empty[st]);
-      auto gelu = [&](bf16 v) {                             // w / (1 + exp(-2 x)) is w (1 + tanh x) / 2
-        const float w = __bfloat162float(v);
-        return __fdividef(w, 1.f + __expf(-1.5957691216057308f * (w + 0.044715f * w * w * w)));
-      };
+      const uint32_t at = (uint32_t)(u.row0 + t0) * ldo + c;
       if (!kSummary && u.decode) {
 #pragma unroll
         for (int t = 0; t < kPart; ++t) {
           const int to = __shfl_sync(0xffffffffu, slot, t);
           if (live && t < n) {
             const float s = fmaf(__uint_as_float(lr[t]), before[t], __uint_as_float(li[t]));
-            out[(size_t)(u.row0 + t0 + t) * p.ldo] = __float2bfloat16(s * gelu(yv[t]));
+            out[at + t * ldo] = __float2bfloat16(s * rg_gelu(__bfloat162float(yv[t])));
             if (to >= 0) p.state[(size_t)to * C + c] = s;
           }
         }
@@ -447,10 +473,18 @@ __global__ void __launch_bounds__(kRgThreads, 1)
           if (kSummary) decay *= h.x;
         }
         if (!kSummary) {
+          if (live && n == kPart) {
 #pragma unroll
-          for (int t = 0; t < kPart; ++t) {
-            s = fmaf(__uint_as_float(lr[t]), s, __uint_as_float(li[t]));
-            if (live && t < n) out[(size_t)(u.row0 + t0 + t) * p.ldo] = __float2bfloat16(s * gelu(yv[t]));
+            for (int t = 0; t < kPart; ++t) {
+              s = fmaf(__uint_as_float(lr[t]), s, __uint_as_float(li[t]));
+              out[at + t * ldo] = __float2bfloat16(s * rg_gelu(__bfloat162float(yv[t])));
+            }
+          } else if (live) {
+#pragma unroll
+            for (int t = 0; t < kPart; ++t) {
+              s = fmaf(__uint_as_float(lr[t]), s, __uint_as_float(li[t]));
+              if (t < n) out[at + t * ldo] = __float2bfloat16(s * rg_gelu(__bfloat162float(yv[t])));
+            }
           }
           if (live && piece == 0 && u.at + u.n >= u.len) {
             const int to = R.slots[u.req];
@@ -504,7 +538,7 @@ int b200_short_conv(const B200ShortConv* a, cudaStream_t stream) {
 // 1: the tensor-core kernel serves this shape.
 int b200_rglru_fits(const B200Rglru* a) {
   return !a->f32 && a->B > 0 && a->B <= 256 && !(a->B & 15) && a->M % 128 == 0 && a->M >= a->B && !(a->ldu & 7) &&
-         !(((uintptr_t)a->u | (uintptr_t)a->gates) & 15) && a->summary;
+         a->rows.T * a->ldy < (1ll << 31) && a->rows.T * a->ldo < (1ll << 31) && !(((uintptr_t)a->u | (uintptr_t)a->gates) & 15) && a->summary;
 }
 
 // Slices of the rows: one wave of CTAs over all channels.
