@@ -269,11 +269,23 @@ __global__ void __launch_bounds__(128) gated_act_kernel(const float* gu, int ldg
   }
 }
 
-__global__ void __launch_bounds__(256) softcap_kernel(float* x, long long n, float cap) {
+// x = cap tanh(x / cap), as cap (1 - 2 / (1 + exp(2 x / cap))); near 0, where that cancels, by tanhf.
+__global__ void __launch_bounds__(256) softcap_kernel(float* x, long long n4, long long n, float cap) {
   pdl_wait();
   pdl_launch_dependents();
-  for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < n; i += (long long)gridDim.x * 256)
-    x[i] = cap * tanhf(x[i] / cap);
+  const float inv = 1.f / cap;
+  auto f = [&](float v) {
+    const float z = v * inv;
+    return cap * (fabsf(z) < 0.5f ? tanhf(z) : 1.f - 2.f / (1.f + expf(2.f * z)));
+  };
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i < n4) {
+    float4 v = reinterpret_cast<float4*>(x)[i];
+    v = make_float4(f(v.x), f(v.y), f(v.z), f(v.w));
+    reinterpret_cast<float4*>(x)[i] = v;
+  } else if (n4 * 4 + (i - n4) < n) {
+    x[n4 * 4 + (i - n4)] = f(x[n4 * 4 + (i - n4)]);
+  }
 }
 
 }  // namespace b200
@@ -318,9 +330,9 @@ int b200_gemm_f32_batched(const void* A, int lda, int a_batch, const void* W, in
 int b200_softcap_f32(void* x, long long n, float cap, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (!(cap > 0.f)) return -1;
-  const long long blocks = (n + 255) / 256;
-  return launch_pdl(softcap_kernel, dim3((unsigned)(blocks < 16384 ? blocks : 16384)), dim3(256), 0, stream, (float*)x, n,
-                    cap) == cudaSuccess ? 0 : -2;
+  const long long n4 = ((uintptr_t)x & 15) ? 0 : n / 4, items = n4 + (n - n4 * 4);
+  return launch_pdl(softcap_kernel, dim3((unsigned)((items + 255) / 256)), dim3(256), 0, stream, (float*)x, n4, n, cap) ==
+                 cudaSuccess ? 0 : -2;
 }
 
 int b200_moe_grouped_gemm_f32(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out,
