@@ -67,34 +67,38 @@ __global__ void __launch_bounds__(128) short_conv_kernel(B200ShortConv p) {
     row0 = R.nd + b + at;
     n = min(kConvRun, len - at);
   }
-  const int slot = R.slots[req];
   if (c >= p.C) return;
+  // (what does not depend on the slot is asked for ahead of it)
+  const int slot = R.slots[req];
+  const bool init = R.seq_lens[req] > len;
+  const T* x = reinterpret_cast<const T*>(p.x) + (size_t)(row0 - at) * p.ldx + c;      // the portion's first row
+  const float* w = p.w + c;
+  float4 hist[TAPS > 1 ? TAPS - 1 : 1], wt[TAPS ? TAPS : 1];
+  if (TAPS) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wt[j] = *reinterpret_cast<const float4*>(w + (size_t)j * p.C);
+  }
+  const float4 first = Rg4<T>::get(x + (size_t)at * p.ldx);
   T* out = reinterpret_cast<T*>(p.out) + (size_t)row0 * p.ldo + c;
   if (slot < 0) {                        // (a padding row: its values only have to be finite)
     for (int r = 0; r < n; ++r) Rg4<T>::put(out + (size_t)r * p.ldo, make_float4(0.f, 0.f, 0.f, 0.f));
     return;
   }
-  const bool init = R.seq_lens[req] > len;
-  const T* x = reinterpret_cast<const T*>(p.x) + (size_t)(row0 - at) * p.ldx + c;      // the portion's first row
   T* st = reinterpret_cast<T*>(p.state) + (size_t)slot * (taps - 1) * p.C + c;
   auto input = [&](int pos) {            // input of the portion's row pos (before it: the carried ones)
     if (pos >= 0) return Rg4<T>::get(x + (size_t)pos * p.ldx);
     if (!init) return make_float4(0.f, 0.f, 0.f, 0.f);
     return Rg4<T>::get(st + (size_t)(taps - 1 + pos) * p.C);
   };
-  const float* w = p.w + c;
   const float4 bias = p.bias ? *reinterpret_cast<const float4*>(p.bias + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-  float4 hist[TAPS > 1 ? TAPS - 1 : 1], wt[TAPS ? TAPS : 1];
   if (TAPS) {
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) wt[j] = *reinterpret_cast<const float4*>(w + (size_t)j * p.C);
 #pragma unroll
     for (int j = 0; j + 1 < TAPS; ++j) hist[j] = input(at - (TAPS - 1) + j);
   }
   for (int r = 0; r < n; ++r) {
     float4 a = bias;
     if (TAPS) {
-      const float4 xin = input(at + r);
+      const float4 xin = r == 0 ? first : input(at + r);
 #pragma unroll
       for (int j = 0; j + 1 < TAPS; ++j) a = rg_fma(wt[j], hist[j], a);
       a = rg_fma(wt[TAPS ? TAPS - 1 : 0], xin, a);
