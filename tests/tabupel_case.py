@@ -93,9 +93,9 @@ def write(path, cfg, tensors):
 # name -> (config, weight options). Sizes differ from layer to layer; some take the tensor-core kernels,
 # some the any-size kernels.
 CASES = {
-    "mixed": (config([rglru(96, 3, 4, 72), latent(3, 48, 16, 32, 40, 56, 0.2, 40, 4e3, (6.0, 100, 24.0, 1.5), 130),
+    "mixed": (config([rglru(96, 3, 4, 72), latent(3, 48, 16, 32, 40, 56, 0.2, 43, 4e3, (6.0, 100, 24.0, 1.5), 130),
                       attention(4, 2, 32, 48, 0.25, 24, 7e3, 20, 3.0, 0.45, 64), rglru(64, 1, 2), rglru(96, 3, 4, 72, weights_of=0),
-                      latent(3, 48, 16, 32, 40, 56, 0.2, 40, 4e3, (6.0, 100, 24.0, 1.5), 130, weights_of=1),
+                      latent(3, 48, 16, 32, 40, 56, 0.2, 43, 4e3, (6.0, 100, 24.0, 1.5), 130, weights_of=1),
                       attention(6, 1, 16, 64, 0.4, 33, 900.0, 16, 1.5, 0.2), rglru(64, 1, 2, weights_of=3)], width=64, vocab=96), {}),
     "odd": (config([latent(2, 10, 6, 7, 9, 11, 0.4, 13, 50.0, (2.5, 30, 8.0, 0.5), 11), rglru(21, 3, 3),
                     attention(3, 1, 10, 7, 0.5, 17, 700.0, 6, 2.0, 0.7, 9), rglru(10, 10, 5, 13),

@@ -13,7 +13,7 @@ pytestmark = pytest.mark.gpu
 DEV = "cuda"
 BF, F32 = torch.bfloat16, torch.float32
 # blocks, channels of one, taps: blocks below, at and above one 128-row product, and beyond the tensor-core form
-SHAPES = [(2, 64, 4), (5, 16, 3), (3, 21, 2), (1, 130, 1), (2, 256, 4), (1, 1, 6), (4, 128, 4), (1, 300, 4)]
+SHAPES = [(3, 64, 4), (5, 16, 3), (3, 21, 2), (1, 130, 1), (2, 256, 4), (1, 1, 6), (4, 128, 4), (1, 300, 4)]
 TOL = {BF: 1.5e-2, F32: 2e-5}
 
 
@@ -110,7 +110,7 @@ def test_whole_and_portions(shape, dtype):
         assert worst(run(s, x, y, w, dtype, cuts), want) < TOL[dtype], cuts
 
 
-@pytest.mark.parametrize("shape", [(2, 64, 4), (2, 256, 4), (3, 100, 4)])
+@pytest.mark.parametrize("shape", [(3, 64, 4), (2, 256, 4), (3, 100, 4)])
 @pytest.mark.parametrize("T", [3000, 64, 65, 128, 129])
 def test_long_prompts_run_in_slices(shape, T):
     """A portion over many slices of rows and one that follows it in the same step."""
@@ -145,7 +145,7 @@ def test_an_early_token_is_read_far_away():
         assert err(run(s, x, y, w, F32, cuts)[[599]], want[[599]]) < 3e-5
 
 
-@pytest.mark.parametrize("shape", [(2, 64, 4), (3, 21, 3), (1, 256, 2)])
+@pytest.mark.parametrize("shape", [(3, 64, 4), (3, 21, 3), (1, 256, 2)])
 @pytest.mark.parametrize("dtype", [F32, BF])
 def test_unequal_requests_and_reused_slots(shape, dtype):
     """Decode rows beside portions of unequal requests, in slots that others have used; a step's other
@@ -172,7 +172,7 @@ def test_unequal_requests_and_reused_slots(shape, dtype):
 
 def test_many_decode_rows():
     """More decode rows than one product takes, beside a portion."""
-    s, x, y, w = make(2, 64, 4, 200, seed=6, dtype=BF)
+    s, x, y, w = make(3, 64, 4, 200, seed=6, dtype=BF)
     a, b = (Engine(s, w, BF, 151, any_size=v) for v in (False, True))
     for at in (0, 1, 2):
         items = [(i, at, x[[(i + at) % 200]], y[[(i + at) % 200]]) for i in range(150)] + [(150, 200 * at, x, y)]

@@ -108,9 +108,9 @@ def run_rglru(a: RglruArgs, any_size: bool = False) -> None:
 
 
 def rglru(u, y, w, s: RglruShape, state, ctx, bufs, out, *, any_size=False):
-    """Channels ``u`` [T, C] and gate branch ``y`` (before its GELU) -> ``out`` = S gelu_tanh(y) with
-    S_t = a S_(t-1) + sqrt(1 - a^2) i u, a = exp(rate r); r and i are sigmoids of ``gates``
-    [blocks, 2, M, B] over each block's channels plus ``gate_bias`` fp32 [2, C]. ``state`` fp32 [slots, C] is
+    """Channels ``u`` [T, C] and gate branch ``y`` (before its GELU) -> ``out`` = state * gelu_tanh(y), the
+    state fading by d = exp(rate * g0) and taking in g1 * u with weight sqrt(1 - d * d); g0 and g1 are sigmoids of
+    ``gates`` [blocks, 2, M, B] over each block's channels plus ``gate_bias`` fp32 [2, C]. ``state`` fp32 [slots, C] is
     advanced; a request's first rows start from zero. ``bufs``: ``summary`` fp32 scratch (see
     :func:`summary_values`), or ``a`` / ``b`` fp32 [T, C] for the any-size kernels."""
     run_rglru(rglru_args(u, y, w, s, state, ctx, bufs, out), any_size)
