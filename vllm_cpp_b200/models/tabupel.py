@@ -33,6 +33,8 @@ RATE = 8.0                                # log a = -RATE r softplus(lam)
 
 def pairs_apart(t: torch.Tensor, heads: int, at: int, dims: int) -> torch.Tensor:
     """Rows ``at`` + 2i of each head to ``at`` + i, rows ``at`` + 2i + 1 to ``at`` + dims / 2 + i."""
+    if not dims:
+        return t
     x = t.reshape(heads, -1, *t.shape[1:]).clone()
     x[:, at: at + dims] = torch.cat([x[:, at: at + dims: 2], x[:, at + 1: at + dims: 2]], 1)
     return x.reshape(t.shape)
@@ -177,7 +179,7 @@ class TabupelModel(ListedModel):
         L["down_proj"] = torch.cat([self.put(t, n, self.cols) for t, n in parts], 0)
         L["q_norm"], L["kv_norm"] = (self.put(p[n], w, **f32) for n, w in (("dq.norm", q8), ("dkv.norm", k8)))
         uq = p["uq"].reshape(H, s.dim + s.rot, -1)
-        turned = pairs_apart(uq[:, s.dim:].reshape(H * s.rot, -1), H, 0, s.rot).reshape(H, s.rot, -1)
+        turned = pairs_apart(uq[:, s.dim:].reshape(H * s.rot, uq.shape[2]), H, 0, s.rot).reshape(H, s.rot, uq.shape[2])
         uq = torch.cat([self.put(uq[:, : s.dim], H, s.qn, q8), self.put(turned, H, s.qw - s.qn, q8)], 1)
         L["uq"] = uq.reshape(H * s.qw, q8).contiguous()
         uk, uv = p["uk"].reshape(H, s.dim, -1), p["uv"].reshape(H, s.vdim, -1)
