@@ -63,7 +63,9 @@ class AttentionSpec:
     """Softmax mixer of one decoder block: grouped heads with separate key and value sizes. Positions
     enter through a distance bias that saturates at ``bias_max`` (0: none) or a rotation of the first
     ``rot_dims`` dimensions (0: none). With ``diff`` every head has two maps over the same values and
-    subtracts the second, weighted by a learned number that starts around ``diff``."""
+    subtracts the second, weighted by a learned number that starts around ``diff``. ``sink``: a learned
+    number per head whose exponential joins the softmax's denominator; ``tied``: the values are the keys
+    before their rotation."""
     heads: int
     kv_heads: int
     dim: int
@@ -77,6 +79,8 @@ class AttentionSpec:
     window: int = 0                           # > 0: a query sees itself and the window - 1 positions before it
     rot_scaling: Optional[RotaryScaling] = None
     diff: Optional[float] = None
+    sink: bool = False
+    tied: bool = False
 
 
 @dataclass
@@ -118,9 +122,35 @@ class DeltaSpec:
 
 
 @dataclass
+class GlaSpec:
+    """Gated-linear-attention mixer of one decoder block: ``heads`` states of ``dim`` x ``vdim`` whose key
+    channels fade by sigmoid(z)^(1 / ``tau``), z a product of rank ``rank`` (a checkpoint's tensors say which)."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    rank: int = 16
+
+
+@dataclass
+class SsmSpec:
+    """State-space mixer (Mamba-2) of one decoder block: ``heads`` states of ``state`` x ``vdim``, input and
+    output vectors shared by ``heads / groups`` heads each, a short convolution of ``conv`` taps, the gated output
+    normed in ``norm_groups`` equal parts."""
+    heads: int
+    groups: int
+    state: int
+    vdim: int
+    conv: int
+    norm_groups: int
+
+
+@dataclass
 class DenseSpec:
-    """Feed-forward of one decoder block: one gated unit."""
+    """Feed-forward of one decoder block: one gated unit, or with ``plain`` one ungated unit with that
+    activation."""
     ff: int
+    plain: Optional[str] = None
 
 
 @dataclass
@@ -135,6 +165,7 @@ class ExpertSpec:
     identity: int = 0
     groups: int = 1
     keep: int = 1
+    plain: Optional[str] = None
 
 
 @dataclass
@@ -145,10 +176,31 @@ class BlockSpec:
     latent: Optional[LatentSpec] = None
     rglru: Optional[RglruSpec] = None
     weights_of: Optional[int] = None          # block whose weights this one runs with (None: its own)
+    gla: Optional[GlaSpec] = None             # set instead of ``attention``
+    ssm: Optional[SsmSpec] = None             # beside ``attention``: the sum of both, times ``scales``
+    scales: tuple = (1.0, 1.0)
+    layer: Optional[int] = None               # number of its tensors in the checkpoint (None: its place)
 
     @property
     def mixer(self):
-        return self.attention or self.delta or self.latent or self.rglru
+        return self.attention or self.delta or self.latent or self.rglru or self.gla or self.ssm
+
+
+@dataclass
+class BigramSpec:
+    """Embedding of token pairs: row (before * ``mul_prev`` + token * ``mul_cur``) mod ``buckets`` of a table, row
+    ``buckets`` for a first token."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
+@dataclass
+class LoopSpec:
+    """Layers ``start`` .. ``stop`` - 1 run ``times`` times in a row with the same weights."""
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass
@@ -219,6 +271,10 @@ class ModelConfig:
     bos_token_id: Optional[int] = None
     # block-by-block sizes of the families whose config.json lists every layer (None: uniform)
     blocks: Optional[list] = None
+    norm_groups: int = 1                      # norms divide this many equal parts of a row each by its own rms
+    input_conv: int = 0                       # taps of the convolution over what a sublayer reads (0: none)
+    bigram: Optional[BigramSpec] = None
+    loop: Optional[LoopSpec] = None           # (already unrolled in ``blocks``)
     raw: dict = field(default_factory=dict)
 
     @property
@@ -385,7 +441,7 @@ def model_config_from_blocks(cfg: dict) -> ModelConfig:
     """ModelConfig of a config.json that names one ``architecture`` and lists its ``layers``, each
     with a mixer and a feed-forward (or null)."""
     arch = cfg["architecture"]
-    readers = {"Nufusun": _nufusun_block, "Diforax": _diforax_block, "Tabupel": _tabupel_block}
+    readers = {"Nufusun": _nufusun_block, "Diforax": _diforax_block, "Tabupel": _tabupel_block, "Kubolorn": _kubolorn_block}
     if arch not in readers:
         raise ValueError(f"no reader for the layer list of architecture {arch!r}")
     blocks = []
@@ -394,6 +450,9 @@ def model_config_from_blocks(cfg: dict) -> ModelConfig:
             blocks.append(_checked(readers[arch](l), blocks))
         except ValueError as e:
             raise ValueError(f"layer {i}: {e}") from None
+    loop = LoopSpec(**{k: int(cfg["loop"][k]) for k in ("start", "stop", "times")}) if cfg.get("loop") else None
+    if loop is not None:
+        blocks = unrolled(blocks, loop)
     for i, b in enumerate(blocks):
         if b.weights_of is not None:
             src = blocks[b.weights_of] if 0 <= b.weights_of < len(blocks) else None
@@ -402,8 +461,13 @@ def model_config_from_blocks(cfg: dict) -> ModelConfig:
             if (src.mixer, src.mlp) != (b.mixer, b.mlp):
                 raise ValueError(f"layer {i}: block {b.weights_of}, whose weights it uses, has other sizes")
     kw = dict(vocab=int(cfg["vocab"]), width=int(cfg["width"]), eps=float(cfg["norm"]["eps"]), raw=cfg)
-    if arch == "Nufusun":
+    if arch in ("Nufusun", "Kubolorn"):
         kw["embed_scale"] = float(cfg["embedding"]["scale"])
+    if arch == "Kubolorn":
+        bigram = cfg["embedding"].get("bigram")
+        kw.update(norm_groups=int(cfg["norm"].get("groups") or 1), loop=loop,
+                  input_conv=int((cfg.get("canon") or {}).get("taps") or 0),
+                  bigram=BigramSpec(**{k: int(bigram[k]) for k in ("buckets", "mul_prev", "mul_cur")}) if bigram else None)
     if arch == "Tabupel":
         kw.update(residual_mult=float(cfg["residual_mult"]), logit_softcap=float(cfg["logit_softcap"]))
     m = model_config_of_blocks(arch, blocks, **kw)
@@ -478,6 +542,42 @@ def _tabupel_block(l: dict) -> BlockSpec:
     return BlockSpec(att, mlp, latent=latent, rglru=rglru, weights_of=None if src is None else int(src))
 
 
+def _kubolorn_block(l: dict) -> BlockSpec:
+    m, f, mlp = l["mixer"], l.get("mlp"), None
+    if f is not None and f["kind"] == "dense":
+        mlp = DenseSpec(ff=int(f["ff"]), plain="gelu_tanh")
+    elif f is not None and f["kind"] == "moe":
+        mlp = ExpertSpec(experts=int(f["router"]["experts"]), top=int(f["router"]["top"]), ff=int(f["expert"]["ff"]), plain="relu2")
+    elif f is not None:
+        raise ValueError(f"unknown feed-forward {f['kind']!r}")
+    if l["type"] == "gla":
+        return BlockSpec(None, mlp, gla=GlaSpec(**{k: int(m[k]) for k in ("heads", "dim", "vdim")}, tau=float(m["tau"])))
+    if l["type"] != "parallel":
+        raise ValueError(f"unknown mixer {l['type']!r}")
+    a, r, rot = m["left"], m["right"], m["left"].get("rot") or {}
+    if int(a.get("vdim", a["dim"])) != int(a["dim"]):
+        raise ValueError(f"values that are keys of {a['dim']} cannot have {a['vdim']}")
+    scaling = rot.get("scaling")
+    if scaling is not None:
+        scaling = RotaryScaling(**{k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")})
+    att = AttentionSpec(**{k: int(a[k]) for k in ("heads", "kv_heads", "dim")}, vdim=int(a["dim"]), scale=float(a["scale"]),
+                        rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 1.0)), rot_scaling=scaling, sink=True,
+                        tied=True)
+    ssm = SsmSpec(**{k: int(r[k]) for k in ("heads", "groups", "state", "vdim", "conv", "norm_groups")})
+    return BlockSpec(att, mlp, ssm=ssm, scales=(float(m["left_scale"]), float(m["right_scale"])))
+
+
+def unrolled(blocks: list, loop: LoopSpec) -> list:
+    """The blocks in the order they run; a pass after the first runs with the first one's weights."""
+    from dataclasses import replace
+    a, b, n = loop.start, loop.stop, loop.times
+    if not (0 <= a < b <= len(blocks) and n >= 1):
+        raise ValueError(f"layers {a} .. {b - 1} of {len(blocks)} cannot run {n} times")
+    order = list(range(a)) + list(range(a, b)) * n + list(range(b, len(blocks)))
+    first = {l: order.index(l) for l in order}
+    return [replace(blocks[l], layer=l, weights_of=None if first[l] == i else first[l]) for i, l in enumerate(order)]
+
+
 def _checked(b: BlockSpec, before: list) -> BlockSpec:
     """The sizes of a block fit together (``before``: the blocks ahead of it)."""
     m, a, f, lat = b.mixer, b.attention, b.mlp, b.latent
@@ -487,8 +587,11 @@ def _checked(b: BlockSpec, before: list) -> BlockSpec:
         raise ValueError(f"{a.rot_dims} rotated dimensions of {a.dim}")
     if lat is not None and lat.rot_dim % 2:
         raise ValueError(f"{lat.rot_dim} rotated dimensions")
-    if (b.delta or b.rglru) is not None and m.conv < 1:
+    if (b.delta or b.rglru or b.ssm) is not None and (b.ssm or m).conv < 1:
         raise ValueError("a convolution has at least one tap")
+    r = b.ssm
+    if r is not None and (r.heads % r.groups or r.heads * r.vdim % r.norm_groups):
+        raise ValueError(f"{r.heads} heads of {r.vdim} do not divide into {r.groups} groups and {r.norm_groups} normed parts")
     if b.rglru is not None and m.width % m.blocks:
         raise ValueError(f"{m.width} channels do not divide into {m.blocks} blocks")
     if a is not None and a.kv_from is not None:
@@ -508,7 +611,8 @@ def _checked(b: BlockSpec, before: list) -> BlockSpec:
 
 def model_config_of_blocks(arch: str, blocks: list, *, vocab: int, width: int, eps: float, embed_scale: float = 1.0,
                            residual_mult: float = 1.0, logit_softcap: float = 0.0, max_position: int = 32768,
-                           raw: Optional[dict] = None) -> ModelConfig:
+                           norm_groups: int = 1, input_conv: int = 0, bigram: Optional[BigramSpec] = None,
+                           loop: Optional[LoopSpec] = None, raw: Optional[dict] = None) -> ModelConfig:
     att = [b.attention for b in blocks if b.attention is not None]
     lat = [b.latent for b in blocks if b.latent is not None]
     moe = [b.mlp for b in blocks if isinstance(b.mlp, ExpertSpec)]
@@ -521,8 +625,14 @@ def model_config_of_blocks(arch: str, blocks: list, *, vocab: int, width: int, e
         rms_norm_eps=eps, embed_scale=embed_scale, norm_topk_prob=False,
         num_experts=max([m.experts for m in moe], default=0), num_experts_per_tok=max([m.top for m in moe], default=0),
         moe_intermediate_size=max([m.ff for m in moe], default=0), max_position_embeddings=max_position,
-        blocks=blocks, raw=raw or {})
-    if arch == "Nufusun":
+        blocks=blocks, norm_groups=norm_groups, input_conv=input_conv, bigram=bigram, loop=loop, raw=raw or {})
+    if width % norm_groups:
+        raise ValueError(f"a width of {width} does not divide into {norm_groups} normed parts")
+    if arch == "Kubolorn":
+        # (every block carries the last inputs of its convolutions, the embedding the last token)
+        m.tie_word_embeddings, m.norm_topk_prob, m.hidden_act = True, True, "gelu_tanh"
+        m.layer_types = ["linear_attention"] * len(blocks)
+    elif arch == "Nufusun":
         m.gemma_norm, m.attention_bias, m.hidden_act, m.scoring_func = True, True, "clamped_gate", "sigmoid"
     elif arch == "Tabupel":
         m.hidden_act, m.residual_multiplier, m.final_logit_softcap = "silu", residual_mult, logit_softcap
@@ -537,8 +647,8 @@ def model_config_of_blocks(arch: str, blocks: list, *, vocab: int, width: int, e
 
 def block_config_dict(cfg: ModelConfig) -> dict:
     """config.json of a ModelConfig with ``blocks`` (the inverse of model_config_from_blocks)."""
-    if cfg.architecture == "Tabupel":
-        return _tabupel_dict(cfg)
+    if cfg.architecture in ("Tabupel", "Kubolorn"):
+        return (_tabupel_dict if cfg.architecture == "Tabupel" else _kubolorn_dict)(cfg)
     layers = []
     for b in cfg.blocks:
         m, a, f, mlp = b.attention or b.delta, b.attention, b.mlp, None
@@ -593,6 +703,39 @@ def _tabupel_dict(cfg: ModelConfig) -> dict:
     return {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_size,
             "norm": {"eps": cfg.rms_norm_eps}, "residual_mult": cfg.residual_multiplier,
             "logit_softcap": cfg.final_logit_softcap, "layers": layers}
+
+
+def _kubolorn_dict(cfg: ModelConfig) -> dict:
+    from dataclasses import asdict
+    layers = []
+    for b in cfg.blocks:
+        if b.weights_of is not None:
+            continue
+        f, mlp = b.mlp, None
+        if isinstance(f, DenseSpec):
+            mlp = {"kind": "dense", "ff": f.ff}
+        elif f is not None:
+            mlp = {"kind": "moe", "router": {"experts": f.experts, "top": f.top}, "expert": {"ff": f.ff}}
+        if b.gla is not None:
+            g = b.gla
+            m = {"heads": g.heads, "dim": g.dim, "vdim": g.vdim, "tau": g.tau}
+        else:
+            a = b.attention
+            left = {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale}
+            if a.rot_dims:
+                left["rot"] = {"base": a.rot_base, "dims": a.rot_dims}
+                if a.rot_scaling is not None:
+                    left["rot"]["scaling"] = asdict(a.rot_scaling)
+            m = {"left": left, "right": asdict(b.ssm), "left_scale": b.scales[0], "right_scale": b.scales[1]}
+        layers.append({"type": "gla" if b.gla is not None else "parallel", "mixer": m, "mlp": mlp})
+    out = {"architecture": cfg.architecture, "vocab": cfg.vocab_size, "width": cfg.hidden_size, "layers": layers,
+           "norm": {"eps": cfg.rms_norm_eps, "groups": cfg.norm_groups}, "embedding": {"scale": cfg.embed_scale},
+           "canon": {"taps": cfg.input_conv}}
+    if cfg.bigram is not None:
+        out["embedding"]["bigram"] = asdict(cfg.bigram)
+    if cfg.loop is not None:
+        out["loop"] = asdict(cfg.loop)
+    return out
 
 
 def load_model_config(model_dir: str) -> ModelConfig:

@@ -326,6 +326,35 @@ class CpuBackend(FusedLinearMixin):
         pos = torch.arange(ids.numel(), dtype=torch.int32).view_as(ids)
         return y, torch.where(ids < w_gate_up.shape[0], pos, torch.full_like(pos, -1)), w
 
+    def embed_pairs(self, stream, ids, table, ctx, **kw):
+        from ..ops.conv_norm import ref_embed_pairs
+        return ref_embed_pairs(stream, ids, table, ctx, **kw)
+
+    def norm_conv(self, src, ctx, weights, outs, **kw):
+        from ..ops.conv_norm import ref_norm_conv
+        ref_norm_conv(src, ctx, weights, outs, **kw)
+
+    def rotate_tied(self, qk, positions, table, q_out, slots, cache, shape, **kw):
+        from ..ops.bias_attn import ref_rotate_tied
+        ref_rotate_tied(qk, positions, table, q_out, slots, cache, shape, **kw)
+
+    def gated_linear_attention(self, *args, **kw):
+        from ..ops.outer import ref_gated_linear_attention
+        return ref_gated_linear_attention(*args, **kw)
+
+    def state_space(self, *args, **kw):
+        from ..ops.outer import ref_state_space
+        return ref_state_space(*args, **kw)
+
+    def plain_unit(self, x, w, act, out):
+        from ..ops.moe import plain_act
+        return out.copy_(plain_act(self.gemm(x, w, out_dtype=torch.float32), act))
+
+    def plain_experts(self, x, logits, w_up, w_down, ws, *, top, act):
+        from ..ops import moe as M
+        ids, w = M.ref_router_topk(logits, top)
+        return M.ref_plain_experts(x, ids, w_up, w_down, act), torch.arange(ids.numel(), dtype=torch.int32).view_as(ids), w
+
     def bias_attention(self, q, cache, ctx, group, *, out, **kw):
         from ..ops.bias_attn import ref_bias_attention
         return ref_bias_attention(q, cache, out, block_table=ctx.block_table[group], seq_lens=ctx.seq_lens,
@@ -705,6 +734,41 @@ class GpuBackend(FusedLinearMixin):
                                group_best=1)
         y = M.clamped_experts(x, ids, None, w_gate_up, w_down, ws)
         return y, ws.pair_pos[: ids.numel()].view_as(ids), w
+
+    def embed_pairs(self, stream, ids, table, ctx, **kw):
+        from ..ops.conv_norm import embed_pairs
+        return embed_pairs(stream, ids, table, ctx, **kw)
+
+    def norm_conv(self, src, ctx, weights, outs, **kw):
+        from ..ops.conv_norm import norm_conv
+        norm_conv(src, ctx, weights, outs, **kw)
+
+    def rotate_tied(self, qk, positions, table, q_out, slots, cache, shape, **kw):
+        from ..ops.bias_attn import rotate_tied
+        rotate_tied(qk, positions, table, q_out, slots, cache, shape, **kw)
+
+    def gated_linear_attention(self, *args, **kw):
+        from ..ops.outer import gated_linear_attention
+        return gated_linear_attention(*args, **kw)
+
+    def state_space(self, *args, **kw):
+        from ..ops.outer import state_space
+        return state_space(*args, **kw)
+
+    def plain_unit(self, x, w, act, out):
+        """act(x W^T), the activation in the product's epilogue."""
+        from ..ops.moe import PLAIN
+        if x.dtype == torch.float32:
+            from ..ops.stream import gemm_f32
+            return gemm_f32(x, w, out=out, act=PLAIN[act])
+        return self.ops.gemm(x, w, out=out, const_w=True, act=PLAIN[act])
+
+    def plain_experts(self, x, logits, w_up, w_down, ws, *, top, act):
+        """The ``top`` experts with the largest ``logits``, weighted by the softmax over those; results as
+        :meth:`routed_experts`."""
+        from ..ops import moe as M
+        ids, w = M.router_topk(logits, top)
+        return M.plain_experts(x, ids, w_up, w_down, ws, act), ws.pair_pos[: ids.numel()].view_as(ids), w
 
     def bias_attention(self, q, cache, ctx, group, *, out, **kw):
         """Decode rows first (one token per request), then the prompt portions."""

@@ -4,11 +4,12 @@ from __future__ import annotations
 
 import torch
 
-from ..config import ModelConfig, ParallelConfig
+from ..config import ModelConfig, ParallelConfig, RopeConfig
 from .backend import make_backend
 from .base import BufferPool, StepContext
 from .dense import ACT_KIND, DenseModel
 from .recurrent import RecurrentState
+from .rope import rope_parameters
 
 
 def pad(n: int, m: int = 8) -> int:
@@ -112,6 +113,17 @@ class ListedModel(DenseModel):
         else:
             L["gate_up"] = torch.cat([gate, up], 0)
         L["down"] = self.put(p["mlp.down"], self.cols, ff)
+
+    def _rope_table(self, base, dims, scaling):
+        """Table of one rotation; blocks with the same rotation share it."""
+        if not dims:
+            return None
+        key = (base, dims, repr(scaling))
+        if key not in self.rope:
+            cfg = scaling.rope(base, dims) if scaling is not None else RopeConfig(theta=base, rotary_dim=dims)
+            inv, magnitude, _ = rope_parameters(cfg, dims, self.max_position)
+            self.rope[key] = self.be.rope_table(inv, self.max_position + 8, magnitude)
+        return self.rope[key]
 
     # ------------------------------------------------------------------ state
     def snapshot_state(self, slots: list) -> None:

@@ -21,6 +21,7 @@ _REGISTRY.update({
     "Nufusun": ("nufusun", "NufusunModel"),
     "Diforax": ("diforax", "DiforaxModel"),
     "Tabupel": ("tabupel", "TabupelModel"),
+    "Kubolorn": ("kubolorn", "KubolornModel"),
 })
 
 

@@ -26,7 +26,6 @@ from ..ops.rglru import RglruShape, summary_values, tensor_core_size
 from .base import StepContext
 from .listed import ListedModel, pad, pad_heads
 from .recurrent import RecurrentState
-from .rope import rope_parameters
 
 RATE = 8.0                                # log a = -RATE r softplus(lam)
 
@@ -145,18 +144,6 @@ class TabupelModel(ListedModel):
             if b.weights_of is not None:
                 self.layers[l] = self.layers[b.weights_of]
         self._expect_shared()
-
-    def _rope_table(self, base, dims, scaling):
-        """Table of one rotation; blocks with the same rotation share it."""
-        if not dims:
-            return None
-        key = (base, dims, repr(scaling))
-        if key not in self.rope:
-            from ..config import RopeConfig
-            cfg = scaling.rope(base, dims) if scaling is not None else RopeConfig(theta=base, rotary_dim=dims)
-            inv, magnitude, _ = rope_parameters(cfg, dims, self.max_position)
-            self.rope[key] = self.be.rope_table(inv, self.max_position + 8, magnitude)
-        return self.rope[key]
 
     def _load_attention(self, L, a, p) -> None:
         D, V, f32 = pad(a.dim, 16), pad(a.vdim, 16), dict(dtype=torch.float32)

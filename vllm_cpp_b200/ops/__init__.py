@@ -57,8 +57,9 @@ GEMM_WS_BYTES = 64 << 20
 def gemm(a: torch.Tensor, w: torch.Tensor, *, bias: torch.Tensor | None = None,
          residual: torch.Tensor | None = None, out: torch.Tensor | None = None,
          out_dtype: torch.dtype = torch.bfloat16, force_path: int = 0,
-         const_w: bool = False) -> torch.Tensor:
-    """``out[M,N] = a[M,K] @ w[N,K]^T (+ bias) (+ residual)``; bf16 inputs, fp32 accumulate.
+         const_w: bool = False, act: int = 0) -> torch.Tensor:
+    """``out[M,N] = act(a[M,K] @ w[N,K]^T (+ bias) (+ residual))``; bf16 inputs, fp32 accumulate.
+    ``act``: 0 none, 1 SiLU, 2 GELU-tanh, 3 GELU-erf, 4 squared ReLU, on the fp32 sums.
     ``const_w``: ``w`` is a model weight that no kernel in the stream writes, so the GEMM may
     fetch its first tiles while the previous kernel is still running."""
     if not (a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and a.dim() == 2 and w.dim() == 2
@@ -75,7 +76,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, *, bias: torch.Tensor | None = None,
         ptr(a), a.stride(0), ptr(w), w.stride(0), ptr(out), out.stride(0),
         1 if out.dtype == torch.float32 else 0, ptr(bias), ptr(residual),
         residual.stride(0) if residual is not None else 0, M, N, K, ptr(ws), ws.numel(),
-        force_path | (0x100 if const_w else 0), stream_ptr())
+        force_path | (0x100 if const_w else 0) | act << 9, stream_ptr())
     check(rc, f"gemm M={M} N={N} K={K}")
     return out
 

@@ -27,7 +27,8 @@ class BiasAttnArgs(ctypes.Structure):
                 ("block_size", _I), ("bias_len", _I), ("null_entry", _I), ("f32", _I), ("splits", _I),
                 ("num_tiles", _I), ("grouped", _I), ("chunk", _I), ("scale", ctypes.c_float),
                 ("window", _I), ("maps", _I), ("values_in_keys", _I), ("shared", _I), ("gate", _P), ("ldg", _L),
-                ("keys", _P), ("values", _P), ("shared_keys", _P), ("ldk", _L), ("ldv", _L), ("lds", _L)]
+                ("keys", _P), ("values", _P), ("shared_keys", _P), ("ldk", _L), ("ldv", _L), ("lds", _L),
+                ("sink", _P), ("key_at", _I), ("out_scale", ctypes.c_float)]
 
 
 class SplitRows(NamedTuple):
@@ -49,6 +50,7 @@ def _declare():
     A = ctypes.POINTER(BiasAttnArgs)
     _lib.declare("b200_head_mix_kv", [P, L, P, P, L, P, P, I, I, I, I, I, I, I, P], I)
     _lib.declare("b200_rotate_kv", [P, L, P, P, I, _lib.F, P, P, P, L, P, P, I, I, I, I, I, I, I, I, I, P], I)
+    _lib.declare("b200_rotate_tied", [P, L, P, P, I, P, L, P, P, I, I, I, I, I, I, P], I)
     _lib.declare("b200_diff_combine", [P, L, P, L, I, I, I, I, _lib.F, _lib.F, _lib.F, I, P], I)
     _lib.declare("b200_bias_attn_kernel", [A, I], I)
     _lib.declare("b200_bias_attn_decode", [A, I, P], I)
@@ -80,6 +82,44 @@ def rotate_kv(qkv, positions, table, rot, eps, q_out, slots, cache, *, H, G, D, 
                                dim, block_size, qkv.shape[0], int(q_out.dtype == torch.float32), stream_ptr()), "rotate_kv")
 
 
+class TiedShape(NamedTuple):
+    """Keys and values from one projection: a group's cache row is ``[first, not rotated | rest | first, rotated]``, the value
+    is its first ``D`` columns and the key its last ``D``. ``rot`` dimensions are rotated, ``r8`` is that padded to 8s."""
+    H: int
+    G: int
+    dim: int
+    rot: int
+
+    @property
+    def r8(self) -> int:
+        return (self.rot + 7) // 8 * 8
+
+    @property
+    def D(self) -> int:
+        return (self.r8 + self.dim - self.rot + 15) // 16 * 16
+
+    @property
+    def pitch(self) -> int:
+        return self.D + self.r8
+
+    def spread(self, t: torch.Tensor, heads: int, axis: int = 0) -> torch.Tensor:
+        """Each head's rows (or columns) of a projection in the order ``[first | rest]`` with the padding in place."""
+        t = t.transpose(0, axis).reshape(heads, self.dim, -1)
+        out = torch.zeros((heads, self.D, t.shape[2]), dtype=t.dtype, device=t.device)
+        out[:, : self.rot], out[:, self.r8: self.r8 + self.dim - self.rot] = t[:, : self.rot], t[:, self.rot:]
+        return out.reshape(heads * self.D, -1).transpose(0, axis)
+
+
+def rotate_tied(qk, positions, table, q_out, slots, cache, s: TiedShape, *, block_size):
+    """Rows ``[q heads | k heads]`` of ``s.D`` columns each (:meth:`TiedShape.spread`) -> rotated queries ``[rest | first]`` to
+    ``q_out`` [T, H * D] and this step's cache rows (slot < 0: none). The rotated pairs lie half of ``rot`` apart."""
+    _declare()
+    assert qk.dtype == q_out.dtype == cache.dtype
+    check(lib().b200_rotate_tied(ptr(qk), qk.stride(0), ptr(positions), ptr(table), s.rot, ptr(q_out), q_out.stride(0), ptr(slots),
+                                 ptr(cache), s.H, s.G, s.D, block_size, qk.shape[0], int(q_out.dtype == torch.float32),
+                                 stream_ptr()), "rotate_tied")
+
+
 def diff_combine(maps, out, *, H, V, vdim, lam, eps, scale):
     """``maps`` [T, H * 2 * V] -> per head o = first - ``lam`` second, over its root mean square over ``vdim``,
     times ``scale``; ``out`` [T, H * V]."""
@@ -90,8 +130,9 @@ def diff_combine(maps, out, *, H, V, vdim, lam, eps, scale):
 
 
 def _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry, scale, chunk, window,
-          maps, grouped, gate, values_in_keys, rows=None) -> BiasAttnArgs:
+          maps, grouped, gate, values_in_keys, rows=None, sink=None, key_at=0, out_scale=1.0) -> BiasAttnArgs:
     a = BiasAttnArgs()
+    a.sink, a.key_at, a.out_scale = ptr(sink), key_at, out_scale
     a.q, a.ldq, a.out, a.ldo = ptr(q), q.stride(0), ptr(out), out.stride(0)
     if rows is None:
         a.cache, a.num_blocks = ptr(cache), cache.shape[0]
@@ -113,12 +154,14 @@ def _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias
 
 def decode(q, cache, out, *, block_table, seq_lens, H, G, kw, vdim, block_size, bias=None, null_entry=False,
            splits=1, tmp=None, any_size=False, scale=1.0, chunk=0, window=0, maps=1, grouped=False, gate=None,
-           values_in_keys=False):
-    """One query row per request, at its last position. ``gate`` [rows, H]: the outputs times its sigmoid;
-    ``values_in_keys``: values are the first columns of the key rows (these two: any-size kernel)."""
+           values_in_keys=False, sink=None, key_at=0, out_scale=1.0):
+    """One query row per request, at its last position. ``gate`` [rows, H]: the outputs times its sigmoid (any-size
+    kernel); ``values_in_keys``: values are the first ``vdim`` columns of a group's key row, its key the columns from
+    ``key_at`` on. ``sink`` fp32 [H]: the softmax counts one more entry of that score without a value. The outputs are
+    multiplied by ``out_scale``."""
     _declare()
     a = _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry, scale, chunk, window, maps,
-              grouped, gate, values_in_keys)
+              grouped, gate, values_in_keys, None, sink, key_at, out_scale)
     if splits > 1:
         if tmp is None:
             tmp = (torch.empty(a.rows * H * splits * vdim, dtype=torch.float32, device=q.device),
@@ -131,12 +174,12 @@ def decode(q, cache, out, *, block_table, seq_lens, H, G, kw, vdim, block_size, 
 
 def prefill(q, cache, out, *, block_table, seq_lens, q_start, num_reqs, tile_req, tile_q0, H, G, kw, vdim,
             block_size, bias=None, null_entry=False, any_size=False, scale=1.0, chunk=0, window=0, maps=1, grouped=False,
-            gate=None, values_in_keys=False, rows=None):
+            gate=None, values_in_keys=False, rows=None, sink=None, key_at=0, out_scale=1.0):
     """Portions of prompts; ``tile_req`` / ``tile_q0`` list their 128-row query tiles. ``rows``
     (:class:`SplitRows`, tensor-core kernel only) stands for ``cache``."""
     _declare()
     a = _args(q, cache, out, block_table, seq_lens, H, G, kw, vdim, block_size, bias, null_entry, scale, chunk, window, maps,
-              grouped, gate, values_in_keys, rows)
+              grouped, gate, values_in_keys, rows, sink, key_at, out_scale)
     a.q_start, a.num_reqs = ptr(q_start), num_reqs
     a.tile_req, a.tile_q0, a.num_tiles = ptr(tile_req), ptr(tile_q0), tile_req.numel()
     check(lib().b200_bias_attn_prefill(ctypes.byref(a), int(any_size), stream_ptr()), "bias_attn_prefill")
@@ -144,7 +187,7 @@ def prefill(q, cache, out, *, block_table, seq_lens, q_start, num_reqs, tile_req
 
 
 def kernel_kind(phase: str, q, cache, *, H, G, kw, vdim, block_size, scale=1.0, chunk=0, window=0, maps=1,
-                grouped=False) -> str:
+                grouped=False, values_in_keys=False, key_at=0) -> str:
     """Which kernel serves a shape: "tensor-core" or "any-size"."""
     _declare()
     a = BiasAttnArgs()
@@ -152,6 +195,7 @@ def kernel_kind(phase: str, q, cache, *, H, G, kw, vdim, block_size, scale=1.0, 
     a.H, a.G, a.kw, a.vdim, a.block_size = H, G, kw, vdim, block_size
     a.scale, a.chunk, a.window, a.maps, a.grouped = scale, chunk, window, maps, int(grouped)
     a.f32, a.tile_req = int(q.dtype == torch.float32), ptr(q)
+    a.values_in_keys, a.key_at, a.out_scale = int(values_in_keys), key_at, 1.0
     return {2: "tensor-core", 1: "any-size"}[lib().b200_bias_attn_kernel(ctypes.byref(a), int(phase == "prefill"))]
 
 
@@ -237,6 +281,23 @@ def ref_rotate_kv(qkv, positions, table, rot, eps, q_out, slots, cache, *, H, G,
         vals[b, o] = qkv[ok, (H + G) * D: (H + G) * D + GV * V].to(cache.dtype)
 
 
+def ref_rotate_tied(qk, positions, table, q_out, slots, cache, s: TiedShape, *, block_size):
+    T, half = qk.shape[0], s.rot // 2
+    x = qk[:, : (s.H + s.G) * s.D].float().view(T, s.H + s.G, s.D)
+    first, rest = x[..., : s.r8], x[..., s.r8:]
+    turned = first.clone()
+    if table is not None:
+        cs = table[positions.long()]
+        c, n = cs[:, None, :half], cs[:, None, half:]
+        u, v = first[..., :half], first[..., half: s.rot]
+        turned[..., :half], turned[..., half: s.rot] = u * c - v * n, v * c + u * n
+    key = torch.cat([rest, turned], -1)
+    q_out[:T, : s.H * s.D] = key[:, : s.H].reshape(T, -1).to(q_out.dtype)
+    page = cache.view(cache.shape[0], -1)[:, : block_size * s.G * s.pitch].view(cache.shape[0], block_size, s.G * s.pitch)
+    ok = slots >= 0
+    page[slots[ok] // block_size, slots[ok] % block_size] = torch.cat([first, key], -1)[ok, s.H:].reshape(-1, s.G * s.pitch).to(cache.dtype)
+
+
 def ref_diff_combine(maps, out, *, H, V, vdim, lam, eps, scale):
     T = maps.shape[0]
     x = maps[:, : H * 2 * V].float().view(T, H, 2, V)
@@ -247,7 +308,8 @@ def ref_diff_combine(maps, out, *, H, V, vdim, lam, eps, scale):
 
 
 def ref_bias_attention(q, cache, out, *, block_table, seq_lens, q_start, H, G, kw, vdim, block_size, bias=None,
-                       null_entry=False, scale=1.0, chunk=0, window=0, maps=1, grouped=False, gate=None, values_in_keys=False):
+                       null_entry=False, scale=1.0, chunk=0, window=0, maps=1, grouped=False, gate=None, values_in_keys=False,
+                       sink=None, key_at=0, out_scale=1.0):
     keys, vals = page_views(cache, block_size, kw)
     qs, R = q_start.tolist(), H // G
     for r, sl in enumerate(seq_lens.tolist()):
@@ -256,10 +318,12 @@ def ref_bias_attention(q, cache, out, *, block_table, seq_lens, q_start, H, G, k
             continue
         blocks = block_table[r, : (sl + block_size - 1) // block_size].long()
         k = keys[blocks].reshape(-1, kw)[:sl].float()
-        v = k[:, :vdim].unsqueeze(1) if values_in_keys else vals[blocks].reshape(-1, G, vdim)[:sl].float()
+        v = k.view(sl, G, -1)[..., :vdim] if values_in_keys else vals[blocks].reshape(-1, G, vdim)[:sl].float()
+        if key_at:
+            k = k.view(sl, G, -1)[..., key_at:].reshape(sl, -1)
         v = v.repeat_interleave(R, 1)
         if grouped:                          # (head h reads map h % maps of its group)
-            kg = k.view(sl, G, 1, maps, -1).expand(sl, G, R // maps, maps, kw // G // maps).reshape(sl, H, -1)
+            kg = k.view(sl, G, 1, maps, -1).expand(-1, -1, R // maps, -1, -1).reshape(sl, H, -1)
             s = torch.einsum("qhd,khd->hqk", q[t0:t1, : H * kg.shape[-1]].float().view(t1 - t0, H, -1), kg) * scale
         else:
             s = torch.einsum("qhd,kd->hqk", q[t0:t1, : H * kw].float().view(t1 - t0, H, kw), k) * scale
@@ -276,9 +340,13 @@ def ref_bias_attention(q, cache, out, *, block_table, seq_lens, q_start, H, G, k
         m = s.amax(-1, keepdim=True)
         if null_entry:
             m = m.clamp(min=0)
+        if sink is not None:
+            m = torch.maximum(m, sink.view(-1, 1, 1))
         e = torch.exp(s - m)
         den = e.sum(-1, keepdim=True) + (torch.exp(-m) if null_entry else 0.0)
-        o = torch.einsum("hqk,khd->qhd", e / den, v)
+        if sink is not None:
+            den = den + torch.exp(sink.view(-1, 1, 1) - m)
+        o = torch.einsum("hqk,khd->qhd", e / den, v) * out_scale
         if gate is not None:
             o = o * torch.sigmoid(gate[t0:t1, :H].float())[..., None]
         out[t0:t1, : H * vdim] = o.reshape(t1 - t0, H * vdim).to(out.dtype)

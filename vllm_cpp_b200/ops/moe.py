@@ -37,6 +37,8 @@ def _declare():
     _lib.declare("b200_moe_grouped_gemm_clamped", [P, I, P, I, I, I, P, P, P, P, P, I, C, P], I)
     _lib.declare("b200_moe_row_weights", [P, P, I, P, P], I)
     _lib.declare("b200_moe_grouped_gemm_f32", [P, I, P, I, I, I, P, P, P, P, P, I, P], I)
+    for n in ("b200_moe_grouped_gemm_act", "b200_moe_grouped_gemm_f32_act"):
+        _lib.declare(n, [P, I, P, I, I, I, P, P, P, P, P, I, I, P], I)
     _lib.declare("b200_clamped_gate_f32", [P, P, P, I, I, I, C, P], I)
     lib()
     _declared = True
@@ -154,6 +156,26 @@ def clamped_experts(x, ids, w, w_gate_up, w_down, ws: MoeWorkspace, *, limit=flo
     return ws.y
 
 
+PLAIN = {"gelu_tanh": 2, "relu2": 4}           # activations of ungated units, as the products' epilogues number them
+
+
+def plain_experts(x, ids, w_up, w_down, ws: MoeWorkspace, act: str):
+    """Expert outputs in sorted order, ``ws.y[ws.pair_pos[t * k + j]]`` = W_down act(W_up x_t); the activation runs in the
+    epilogue of the first grouped product."""
+    _declare()
+    T, k = ids.shape
+    E, P = w_up.shape[0], T * k
+    chunks = min(ws.max_chunks, E + (P + 255) // 256)
+    moe_sort(ids, 0, E, ws)
+    moe_gather(x, ws, E, P)
+    args = (ptr(ws.chunk_expert), ptr(ws.chunk_row0), ptr(ws.chunk_n), ptr(ws.meta), chunks)
+    run, kind = ((lib().b200_moe_grouped_gemm_act, "moe_grouped_gemm_act") if x.dtype == torch.bfloat16 else
+                 (lib().b200_moe_grouped_gemm_f32_act, "moe_grouped_gemm_f32_act"))
+    for src, w, out, a in ((ws.xs, w_up, ws.act, PLAIN[act]), (ws.act, w_down, ws.y, 0)):
+        check(run(ptr(src), P, ptr(w), E, w.shape[1], w.shape[2], ptr(out), *args, a, stream_ptr()), kind)
+    return ws.y
+
+
 def combine(y: torch.Tensor, ws: MoeWorkspace, topk_w: torch.Tensor, out: torch.Tensor | None,
             shared: torch.Tensor | None = None, shared_gate: torch.Tensor | None = None,
             scatter: B200MoeScatter | None = None):
@@ -221,6 +243,24 @@ def ref_clamped_experts(x, ids, w, w_gate_up, w_down, *, limit=float("inf"), alp
         if w is not None:
             gu = gu * w.reshape(-1)[rows, None]
         a = ref_clamped_gate(gu, limit, alpha, up_offset).to(x.dtype)
+        y[rows] = (a.float() @ w_down[e].float().t()).to(x.dtype)
+    return y
+
+
+def plain_act(x, act: str):
+    if act == "relu2":
+        return torch.relu(x) ** 2
+    return torch.nn.functional.gelu(x, approximate="tanh")
+
+
+def ref_plain_experts(x, ids, w_up, w_down, act: str):
+    """-> outputs [T * k, H] in pair order (token-major), in the type of ``x``."""
+    T, k = ids.shape
+    y = torch.zeros((T * k, x.shape[1]), dtype=x.dtype, device=x.device)
+    flat = ids.reshape(-1).long()
+    for e in flat.unique().tolist():
+        rows = (flat == e).nonzero().flatten()
+        a = plain_act(x[rows // k].float() @ w_up[e].float().t(), act).to(x.dtype)
         y[rows] = (a.float() @ w_down[e].float().t()).to(x.dtype)
     return y
 

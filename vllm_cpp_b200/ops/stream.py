@@ -35,7 +35,7 @@ def _declare():
     P, I = _lib.P, _lib.I
     _lib.declare("b200_stream_norm", [ctypes.POINTER(StreamNormArgs), P], I)
     _lib.declare("b200_gated_act_f32", [P, I, P, I, I, I, I, P], I)
-    _lib.declare("b200_gemm_f32", [P, I, P, I, P, I, P, I, I, I, P], I)
+    _lib.declare("b200_gemm_f32", [P, I, P, I, P, I, P, I, I, I, I, P], I)
     _lib.declare("b200_softcap_f32", [P, ctypes.c_longlong, _lib.F, P], I)
     lib()
     _declared = True
@@ -66,15 +66,15 @@ def stream_norm(stream, norm_w, eps, out, *, width, ids=None, table=None, scale=
     return out
 
 
-def gemm_f32(a, w, bias=None, out=None):
-    """``a @ w.T (+ bias)`` in fp32 multiply-adds."""
+def gemm_f32(a, w, bias=None, out=None, act=0):
+    """``act(a @ w.T (+ bias))`` in fp32 multiply-adds; ``act`` as in ``ops.gemm``."""
     _declare()
     M, K = a.shape
     N = w.shape[0]
     if out is None:
         out = torch.empty((M, N), dtype=torch.float32, device=a.device)
     check(lib().b200_gemm_f32(ptr(a), a.stride(0), ptr(w), w.stride(0), ptr(out), out.stride(0), ptr(bias), M, N, K,
-                              stream_ptr()), f"gemm_f32 M={M} N={N} K={K}")
+                              act, stream_ptr()), f"gemm_f32 M={M} N={N} K={K}")
     return out
 
 
