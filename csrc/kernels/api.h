@@ -20,7 +20,8 @@ void* b200_status_ptr();
 const char* b200_kernel_arch();
 
 // C[M,N] = A[M,K] * W[N,K]^T (+bias[N]) (+residual[M,N]); bf16 in, bf16 or f32 out.
-// force_path: 0 auto, 1 tiled kernel, 2 swap-AB split-K kernel, 3 BN=128, 4 BN=256.
+// force_path: 0 auto, 1 tiled kernel, 2 swap-AB split-K kernel, 3 BN=128, 4 BN=256; + 0x100: W is never written by a
+// kernel; + act << 9: activation of the result (act_epilogue in sm100.cuh).
 int b200_gemm_bf16(const void* A, int lda, const void* W, int ldw, void* out, int ldo,
                    int out_f32, const void* bias, const void* residual, int ldr, int M, int N,
                    int K, void* workspace, size_t ws_bytes, int force_path, cudaStream_t stream);
@@ -199,7 +200,7 @@ typedef struct B200BiasAttn {
   float scale;
   int window;                  // > 0: a query sees itself and the window - 1 positions before it
   int maps;                    // > 1 (grouped): a group's key columns hold that many keys, head h meets the h % maps-th
-  int values_in_keys;          // values are the first vdim columns of the key rows (any-size kernel)
+  int values_in_keys;          // values are the first vdim columns of a group's key row
   int shared;                  // width of shared_keys in a query row
   const void* gate;            // element (row, head): the output times its sigmoid (prefill and any-size kernels)
   long long ldg;
@@ -209,6 +210,9 @@ typedef struct B200BiasAttn {
   const void* values;
   const void* shared_keys;
   long long ldk, ldv, lds;
+  const float* sink;           // [H] or null: the softmax counts one more entry of that score without a value
+  int key_at;                  // values_in_keys: a group's key is its columns from here on
+  float out_scale;             // the outputs are multiplied by this
 } B200BiasAttn;
 
 // Latent attention (latent.cu): norms of the query and key latents, rotation of the shared key part, cache rows
@@ -238,6 +242,80 @@ typedef struct B200Rows {
   const int* tile_q0;
   int nd, num_prefills, num_tiles, T;
 } B200Rows;
+
+// Start of the fp32 stream (conv_norm.cu): stream = norm(table[ids] * scale + bigram[row]), row = (token before *
+// mul_prev + token * mul_cur) mod buckets, or buckets for a request's first token (bigram null: none). The norm divides
+// ``groups`` equal parts of width each by its own rms. Rows are width values in storage padded to cols.
+typedef struct B200EmbedPairs {
+  B200Rows rows;
+  float* stream;
+  long long lds;
+  const void* ids;             // int64 [T]
+  const void* table;           // [vocab][cols]
+  const void* bigram;          // [buckets + 1][cols]
+  long long* prev;             // [slots]: each request's last token
+  const float* norm_w;
+  long long vocab, buckets, mul_prev, mul_cur;
+  int width, cols, groups, f32;
+  float scale, eps;
+} B200EmbedPairs;
+
+// Stream update, norm in equal parts and causal convolutions over the normed rows (conv_norm.cu), see conv_norm.py:
+// dst = src + a + sum_j pair_w[j] y[pair_pos[j]];  out_i[t] = sum_j w_i[j] xhat[t - taps + 1 + j].
+typedef struct B200NormConv {
+  B200Rows rows;
+  const float* src;
+  float* dst;                  // another buffer than src, or null
+  long long lds;
+  const float* a;
+  long long lda;
+  const void* y;
+  long long ldy;
+  const void* pair_pos;        // int32 [T][k], < 0: nothing
+  const float* pair_w;
+  const float* w1;             // [taps][cols]
+  const float* w2;
+  void* out1;
+  void* out2;                  // null: one convolution
+  long long ldo;
+  float* state;                // [slots][taps - 1][cols]
+  int width, cols, groups, taps, k, f32;
+  float eps;
+} B200NormConv;
+
+// Recurrences over outer products (outer.cu, outer_chunk.cu), see outer.py: S <- decay S + k v^T, o = S^T q with fp32
+// states [slots][H][D][V]; key and query heads are shared by H / G states each. Rows of q, k, v lie ld apart.
+//   kind 0: decay per key channel, sigmoid(a2 a1 + a2b)^inv_tau; out = norm(o) * norm_w * silu(gate) per head
+//   kind 1: decay per head, exp(-A dt), dt = softplus(dt + dt_bias), k scaled by dt; out = out_scale *
+//           norm((o + skip v) silu(gate)) * norm_w, the norm in ``parts`` equal parts of the H * vdim values
+typedef struct B200Outer {
+  B200Rows rows;
+  const void* q;               // [T][G * D]
+  const void* k;
+  const void* v;               // [T][H * V]
+  long long ld;
+  const void* a1;              // [T][rank]
+  const void* a2;              // [H * D][rank]
+  const float* a2b;
+  long long lda1;
+  const void* dt;              // [T][H]
+  const float* dt_bias;
+  const float* A;
+  long long lddt;
+  float* state;
+  float* o;                    // [T][H * V], before norm and gate
+  float* ws;                   // [segments][H][D][V], [segments][H][D]: portions cut in segments
+  float* ws_decay;
+  const void* gate;            // [T][H * V]
+  long long ldg;
+  const float* norm_w;         // [V] or [H * V]
+  const float* skip;           // [H]
+  void* out;
+  long long ldo;
+  int kind, H, G, D, V, dim, vdim, rank, f32, parts;
+  int seg_tiles, multi;        // 128-row tiles per segment; some portion has more than one segment
+  float q_scale, inv_tau, eps, out_scale;
+} B200Outer;
 
 // Causal convolution per channel with carried inputs (rglru.cu). act: 0 none, 1 SiLU.
 typedef struct B200ShortConv {
@@ -373,6 +451,7 @@ int b200_attn_decode_tc(const void* q, int ldq, void* out, int ldo, const void* 
 // ---- attn_bias.cu
 int b200_head_mix_kv(const void* qkv, long long ld, const void* mix, void* q_out, long long ldq, const void* slots, void* cache, int H, int G, int dim, int vdim, int block_size, int T, int f32, cudaStream_t stream);
 int b200_rotate_kv(const void* qkv, long long ld, const void* positions, const void* cos_sin, int rot, float eps, const float* q_w, const float* k_w, void* q_out, long long ldq, const void* slots, void* cache, int H, int G, int GV, int D, int V, int dim, int block_size, int T, int f32, cudaStream_t stream);
+int b200_rotate_tied(const void* qk, long long ld, const void* positions, const void* cos_sin, int rot, void* q_out, long long ldq, const void* slots, void* cache, int H, int G, int D, int block_size, int T, int f32, cudaStream_t stream);
 int b200_diff_combine(const void* maps, long long ldm, void* out, long long ldo, int H, int V, int vdim, int T, float lam, float eps, float scale, int f32, cudaStream_t stream);
 int b200_bias_attn_kernel(const B200BiasAttn* a, int phase);
 int b200_bias_attn_decode(const B200BiasAttn* a, int any_size, cudaStream_t stream);
@@ -381,6 +460,15 @@ int b200_bias_attn_prefill(const B200BiasAttn* a, int any_size, cudaStream_t str
 int b200_attn_prefill(const void* q, int ldq, void* out, int ldo, void* lse, const void* kv_cache, int64_t num_blocks, int block_size, int Hq, int Hkv, int D, const void* block_table, int max_blocks, const void* seq_lens, const void* q_start, const void* tile_req, const void* tile_q0, int num_tiles, int total_q, float scale, float softcap, int window, int causal, cudaStream_t stream);
 // ---- common.cu
 long long b200_set_peer_wait_cycles(long long cycles);
+// ---- conv_norm.cu
+int b200_embed_pairs(const B200EmbedPairs* a, cudaStream_t stream);
+int b200_norm_conv(const B200NormConv* a, cudaStream_t stream);
+// ---- outer.cu
+int b200_outer_step(const B200Outer* a, int reqs, cudaStream_t stream);
+int b200_outer_norm(const B200Outer* a, int reqs, int chunks, cudaStream_t stream);
+// ---- outer_chunk.cu
+int b200_outer_fits(const B200Outer* a);
+int b200_outer_chunk(const B200Outer* a, cudaStream_t stream);
 // ---- gdn.cu
 int b200_gdn_conv1d_fwd(const void* x, long ldx, const void* w, void* conv_state, const int* qsl, const int* slots, const int* has_init, void* out, long ldo, int n_seq, int total_tokens, int C, cudaStream_t stream);
 int b200_gdn_conv1d_update(const void* x, long ldx, const void* w, void* conv_state, const int* slots, void* out, long ldo, int B, int C, cudaStream_t stream);
@@ -444,6 +532,7 @@ int b200_moe_gather(const void* x, int ldx, const void* sorted_token, const void
 int b200_moe_grouped_gemm(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, cudaStream_t stream);
 int b200_moe_grouped_gemm_gated(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, int kind, cudaStream_t stream);
 int b200_moe_grouped_gemm_clamped(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, const B200ClampedGate* act, cudaStream_t stream);
+int b200_moe_grouped_gemm_act(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, int act, cudaStream_t stream);
 int b200_moe_row_weights(const void* pair_pos, const void* topk_w, int P, void* row_w, cudaStream_t stream);
 int b200_moe_combine(const void* y, const void* pair_pos, const void* topk_w, int T, int k, int H, const void* shared, const void* shared_gate, void* out, const B200MoeScatter* sc, cudaStream_t stream);
 int b200_shared_gate(const void* x, int ldx, const void* w, int T, int H, void* out, cudaStream_t stream);
@@ -459,10 +548,11 @@ int b200_embedding(const void* ids, const void* table, void* out, int T, int H, 
 int b200_gather_rows(const void* x, const void* idx, void* out, int n_out, int n_src, int row_bytes, cudaStream_t stream);
 // ---- stream.cu
 int b200_stream_norm(const B200StreamNorm* a, cudaStream_t stream);
-int b200_gemm_f32(const void* A, int lda, const void* W, int ldw, void* out, int ldo, const void* bias, int M, int N, int K, cudaStream_t stream);
+int b200_gemm_f32(const void* A, int lda, const void* W, int ldw, void* out, int ldo, const void* bias, int M, int N, int K, int act, cudaStream_t stream);
 int b200_gemm_f32_batched(const void* A, int lda, int a_batch, const void* W, int ldw, void* out, int ldo, long long out_batch, int M, int N, int K, int batch, cudaStream_t stream);
 int b200_softcap_f32(void* x, long long n, float cap, cudaStream_t stream);
 int b200_moe_grouped_gemm_f32(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, cudaStream_t stream);
+int b200_moe_grouped_gemm_f32_act(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out, const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta, int max_chunks, int act, cudaStream_t stream);
 int b200_gated_act_f32(const void* gate_up, int ldg, void* out, int ldo, int T, int I, int kind, cudaStream_t stream);
 int b200_clamped_gate_f32(const void* gate_up, void* out, const void* meta, int E, int max_rows, int I, const B200ClampedGate* act, cudaStream_t stream);
 // ---- rope_cache.cu

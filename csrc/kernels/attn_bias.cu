@@ -213,6 +213,9 @@ struct BiasAttnParams {
   int own_chunks;           // 64-wide chunks of a query row that meet the head's own key columns
   const void* gate;         // [rows, ldg]
   long long ldg;
+  const float* sink;        // [H]: one more entry of the softmax, without a value
+  int key_at, pitch, vpitch;   // first key column and columns of a group's key row; columns from value head to value head
+  float out_scale;
 };
 
 // First position a query at pos sees.
@@ -258,6 +261,7 @@ __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
   for (int a = 0; a < kAnyAcc; ++a) acc[a] = 0.f;
   // warp w owns the softmax state of head h0 + w
   float m = p.null_entry ? 0.f : -INFINITY, l = p.null_entry ? 1.f : 0.f;
+  if (p.sink && warp < nh) { m = p.sink[h0 + warp]; l = 1.f; }
   for (int base = first_key(p, pos); base <= pos; base += kAnyKeys) {
     const int key = base + tid;
     const bool valid = key <= pos;
@@ -275,7 +279,7 @@ __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
 #pragma unroll
         for (int h = 0; h < kAnyHeads; ++h) {
           if (h >= nh) break;
-          const T* kg = k + (size_t)((h0 + h) / R * p.maps + (h0 + h) % p.maps) * p.qw;
+          const T* kg = k + (size_t)((h0 + h) / R) * p.pitch + p.key_at + (size_t)((h0 + h) % p.maps) * p.qw;
           for (int i = 0; i < p.qw; ++i) s[h] = fmaf(sq[h * p.qw + i], to_f(kg[i]), s[h]);
         }
       } else {
@@ -321,7 +325,7 @@ __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
       const int e = tid + a * 128;
       if (e < nh * p.vdim) {
         const int h = e / p.vdim, d = e - h * p.vdim;
-        const T* v = cache + (size_t)((h0 + h) / R) * p.vdim + d;
+        const T* v = cache + (size_t)((h0 + h) / R) * p.vpitch + d;
         float x = acc[a] * s_alpha[h];
         for (int kk = 0; kk < nk; ++kk) x = fmaf(sc[h * kAnyKeys + kk], to_f(v[vrow[kk]]), x);
         acc[a] = x;
@@ -336,7 +340,7 @@ __global__ void __launch_bounds__(128) bias_attn_any_kernel(BiasAttnParams p) {
     const int e = tid + a * 128;
     if (e < nh * p.vdim) {
       const float ls = s_l[e / p.vdim];
-      float x = ls > 0.f ? acc[a] / ls : 0.f;
+      float x = ls > 0.f ? acc[a] / ls * p.out_scale : 0.f;
       if (p.gate) x *= sigmoid_f(to_f(reinterpret_cast<const T*>(p.gate)[(size_t)row * p.ldg + h0 + e / p.vdim]));
       o[e] = from_f<T>(x);
     }
@@ -780,7 +784,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
   // first key tile: that of the first row's first key
   const int lo_tile = first_key(p, ctx_off + q0) / kBKeys;
   const int ntiles = (ctx_off + q0 + rows - 1) / kBKeys + 1 - lo_tile;
-  const int k_col = p.own_chunks < nkc ? hkv * (p.kw / p.G) : p.qw < p.kw ? (hkv * p.maps + h % p.maps) * p.qw : 0;
+  const int k_col = p.own_chunks < nkc ? hkv * p.pitch : p.qw < p.kw ? hkv * p.pitch + p.key_at + h % p.maps * p.qw : 0;
   // TMEM columns: S buffers (128 each), then O, then two P buffers (64 each)
   const int s_bufs = p.vdim > 128 ? 1 : 2;
   const int o_cols = p.vdim > 128 ? 256 : 128;
@@ -861,7 +865,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
         if (lane < loads)
           for (int c = 0; c < nvc; ++c)
             tma_load_3d(sV + (vs * nvc + c) * kChunkBytes + lane * rpl * 128, &tmV, &bars->v_full[vs],
-                        hkv * p.vdim + c * 64, row, blk_prev);
+                        hkv * p.vpitch + c * 64, row, blk_prev);
       }
       blk_prev = blk;
       blk = next;
@@ -941,7 +945,8 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
     };
     // m: reference maximum of the row in the log2 domain (the same in both threads of a row), raised
     // lazily, by more than 2^8. The null entry is the state before the first key: score 0, weight 1.
-    float m = p.null_entry ? 0.f : -INFINITY, l = p.null_entry && half == 0 ? 1.f : 0.f;
+    float m = p.null_entry ? 0.f : -INFINITY, l = (p.null_entry || p.sink) && half == 0 ? 1.f : 0.f;
+    if (p.sink) m = p.sink[h] * kLog2e;
     bool ok = true;
     const int vcols = (p.vdim + 31) / 32;
     if (tile_near(0)) fill_window(0);
@@ -1042,7 +1047,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
     if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->o_full, 0, p.status));
     if (ok) {
       tc_fence_after_sync();
-      float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? p.out_scale / l : 0.f;
       if (p.gate && r < rows)
         inv *= sigmoid_f(to_f(reinterpret_cast<const __nv_bfloat16*>(p.gate)[(size_t)(q_begin + q0 + r) * p.ldg + h]));
       __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)(q_begin + q0 + r) * p.ldo + (size_t)h * p.vdim;
@@ -1076,7 +1081,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
 // Shapes the decode kernel serves. tk: keys per tile; cls: register class (0: 8 output tiles, 2 query
 // chunks and 4 heads per warp, 1: 16 tiles, 8 heads, queries in shared memory).
 static bool decode_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem, int& tk, int& cls) {
-  if (a->grouped || a->chunk || a->window || a->gate || a->scale != 1.f) return false;           // (attn_grouped.cu)
+  if (a->grouped || a->chunk || a->window || a->gate || a->scale != 1.f || a->sink || a->out_scale != 1.f) return false;           // (attn_grouped.cu)
   if (a->f32 || (a->kw & 7) || (a->vdim & 7) || (a->ldq & 7) || (a->ldo & 1)) return false;
   if (((uintptr_t)a->q | (uintptr_t)a->cache) & 15) return false;
   const int R = a->H / a->G, nkc = (a->kw + 63) / 64;
@@ -1116,14 +1121,14 @@ static bool decode_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem, 
 
 static bool prefill_plan(const B200BiasAttn* a, BiasAttnParams& p, size_t& smem) {
   if (a->f32 || !a->tile_req || (a->kw & 7) || (a->vdim & 7) || a->vdim > 256 || (a->ldq & 7) || (a->ldo & 7)) return false;
-  if (((uintptr_t)a->q | (uintptr_t)a->cache | (uintptr_t)a->out) & 15 || a->values_in_keys) return false;
+  if (((uintptr_t)a->q | (uintptr_t)a->cache | (uintptr_t)a->out) & 15 || (a->values_in_keys && !a->grouped)) return false;
   if (((uintptr_t)a->keys | (uintptr_t)a->values | (uintptr_t)a->shared_keys) & 15 || (a->ldk | a->ldv | a->lds) & 7) return false;
   const int bs = a->block_size, maps = a->maps > 1 ? a->maps : 1;
   if (bs < 8 || (bs & 7) || (bs < kBKeys && kBKeys % bs) || (bs > kBKeys && bs % kBKeys)) return false;
   // a group's columns start on a 16-byte boundary and the last product of 16 reads none of the next group
-  if (a->grouped && (a->kw / a->G / maps & 15)) return false;
+  if (a->grouped && (((a->kw / a->G - a->key_at) / maps & 15) || (a->kw / a->G & 7) || (a->key_at & 7))) return false;
   if (a->shared && (!a->shared_keys || (a->shared & 15) || maps > 1 || !a->grouped)) return false;
-  const int nkc = ((a->grouped ? a->kw / a->G / maps : a->kw) + 63) / 64 + (a->shared + 63) / 64, nvc = (a->vdim + 63) / 64;
+  const int nkc = ((a->grouped ? (a->kw / a->G - a->key_at) / maps : a->kw) + 63) / 64 + (a->shared + 63) / 64, nvc = (a->vdim + 63) / 64;
   const int limit = 227 * 1024, fixed = (int)sizeof(BiasPrefillBars) + 1024;
   // the query tile stays in shared memory if enough of the key ring fits beside it
   for (p.q_stream = 0; p.q_stream < 2; ++p.q_stream) {
@@ -1161,7 +1166,7 @@ struct PageMapHash {
 static bool page_maps(const B200BiasAttn* a, int keys, CUtensorMap* mk, CUtensorMap* mv) {
   static std::mutex mu;
   static std::unordered_map<PageMapKey, std::pair<CUtensorMap, CUtensorMap>, PageMapHash> maps;
-  const int vw = a->G * a->vdim;
+  const int vw = a->values_in_keys ? 0 : a->G * a->vdim;
   const uint32_t rows = a->block_size < keys ? a->block_size : keys;
   PageMapKey key{a->cache, (uint64_t)a->num_blocks, a->block_size, a->kw, vw, (int)rows};
   std::lock_guard<std::mutex> lock(mu);
@@ -1173,9 +1178,10 @@ static bool page_maps(const B200BiasAttn* a, int keys, CUtensorMap* mk, CUtensor
     CUtensorMap k, v;
     if (!encode_tmap_3d(&k, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a->kw, a->block_size, a->num_blocks,
                         (uint64_t)a->kw * 2, page, 64, rows, 1, CU_TENSOR_MAP_SWIZZLE_128B) ||
-        !encode_tmap_3d(&v, base + (size_t)a->block_size * a->kw * 2, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, vw,
-                        a->block_size, a->num_blocks, (uint64_t)vw * 2, page, 64, rows, 1, CU_TENSOR_MAP_SWIZZLE_128B))
+        (vw && !encode_tmap_3d(&v, base + (size_t)a->block_size * a->kw * 2, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, vw,
+                               a->block_size, a->num_blocks, (uint64_t)vw * 2, page, 64, rows, 1, CU_TENSOR_MAP_SWIZZLE_128B)))
       return false;
+    if (!vw) v = k;
     it = maps.emplace(key, std::make_pair(k, v)).first;
   }
   *mk = it->second.first;
@@ -1202,8 +1208,9 @@ static BiasAttnParams common_params(const B200BiasAttn* a) {
   p.num_reqs = a->num_reqs; p.rows = a->rows;
   p.H = a->H; p.G = a->G; p.kw = a->kw; p.vdim = a->vdim; p.block_size = a->block_size;
   p.maps = a->maps > 1 ? a->maps : 1; p.window = a->window; p.values_in_keys = a->values_in_keys;
-  p.gate = a->gate; p.ldg = a->ldg;
-  p.qw = a->grouped ? a->kw / a->G / p.maps : a->kw; p.chunk = a->chunk; p.scale = a->scale;
+  p.gate = a->gate; p.ldg = a->ldg; p.sink = a->sink; p.out_scale = a->out_scale;
+  p.pitch = a->kw / a->G; p.key_at = a->key_at; p.vpitch = a->values_in_keys ? p.pitch : a->vdim;
+  p.qw = a->grouped ? (p.pitch - p.key_at) / p.maps : a->kw; p.chunk = a->chunk; p.scale = a->scale;
   p.own_chunks = (p.qw + 63) / 64;
   if (a->shared) p.qw = p.own_chunks * 64 + a->shared;
   p.bias = (const float*)a->bias; p.bias_len = a->bias_len; p.null_entry = a->null_entry;
@@ -1293,7 +1300,8 @@ static bool valid_args(const B200BiasAttn* a) {
   return a->H > 0 && a->G > 0 && a->H % a->G == 0 && a->kw > 0 && a->vdim > 0 && a->block_size > 0 &&
          (!a->bias || a->bias_len > 0) && (!a->grouped || a->kw % a->G == 0) && a->chunk >= 0 &&
          a->window >= 0 && (a->maps <= 1 || (a->grouped && a->kw / a->G % a->maps == 0 && a->H / a->G % a->maps == 0)) &&
-         (!a->values_in_keys || (a->G == 1 && a->vdim <= a->kw));
+         (!a->values_in_keys || a->vdim <= a->kw / a->G) && !(a->sink && a->null_entry) &&
+         (!a->key_at || (a->values_in_keys && a->grouped && a->maps <= 1 && a->key_at > 0 && a->key_at < a->kw / a->G));
 }
 
 }  // namespace b200

@@ -128,6 +128,10 @@ struct GroupedDecode {
   float scale2;                // score scale x log2(e)
   float* tmp_o;                // [B, H, splits, V]
   float* tmp_lse;              // [B, H, splits], log2
+  // values inside the key rows: a group's row is ``pitch`` columns, the value its first V, the key those from key_at on
+  int pitch, key_at, tied;
+  const float* sink;
+  float out_scale;
 };
 
 static constexpr int kGWarps = 4, kGKeys = 16, kGStages = 3;
@@ -158,6 +162,8 @@ __device__ __forceinline__ float g_ex2(float x) {
 }
 
 __host__ __device__ inline int g_stage_bytes(int D, int V) { return kGKeys * (D + 8 + V + 8) * 2; }
+// (rows of an odd number of 16-byte units)
+__host__ __device__ inline int g_tied_row(int pitch) { return (pitch / 8 | 1) * 16; }
 
 // ND, NV: bounds of D / 16 and V / 16.
 template <int ND, int NV>
@@ -167,8 +173,9 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   // (a group of more than 16 heads takes several CTAs)
   const int b = blockIdx.x, g = blockIdx.y % p.G, head0 = blockIdx.y / p.G * 16, R = min(p.R - head0, 16), split = blockIdx.z;
-  const int nd = p.D / 16, nv = p.V / 16, kw = p.G * p.D, vw = p.G * p.V;
-  const int ks = (p.D + 8) * 2, vs = (p.V + 8) * 2, stage = g_stage_bytes(p.D, p.V);
+  const int nd = p.D / 16, nv = p.V / 16, kw = p.G * p.pitch, vw = p.tied ? 0 : p.G * p.V;
+  const int ks = p.tied ? g_tied_row(p.pitch) : (p.D + 8) * 2, vs = p.tied ? ks : (p.V + 8) * 2;
+  const int stage = p.tied ? kGKeys * ks : g_stage_bytes(p.D, p.V);
   const uint32_t ring = smem_u32(g_smem) + warp * kGStages * stage;
   pdl_wait();
   pdl_launch_dependents();
@@ -182,14 +189,14 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
   const int32_t* bt = p.block_table + (size_t)b * p.max_blocks;
 
   // 16-byte unit u of row r of a tile, this lane's first and the step to its next (32 units on)
-  const int ku = p.D / 8, vu = p.V / 8;
+  const int ku = p.pitch / 8, vu = p.V / 8;
   const int kr0 = lane / ku, ku0 = lane - kr0 * ku, krs = 32 / ku, kus = 32 - krs * ku;
   const int vr0 = lane / vu, vu0 = lane - vr0 * vu, vrs = 32 / vu, vus = 32 - vrs * vu;
   auto load = [&](int i) {                       // tile i of this warp into stage i % kGStages
     if (i < n) {
       const int key = (ta + warp + i * kGWarps) * kGKeys;
       const int page = max(bt[key / p.block_size], 0), off = key % p.block_size;
-      const bf16* k = p.cache + (size_t)page * p.block_size * (kw + vw) + (size_t)off * kw + (size_t)g * p.D;
+      const bf16* k = p.cache + (size_t)page * p.block_size * (kw + vw) + (size_t)off * kw + (size_t)g * p.pitch;
       const bf16* v = p.cache + (size_t)page * p.block_size * (kw + vw) + (size_t)p.block_size * kw + (size_t)off * vw + (size_t)g * p.V;
       const uint32_t dst = ring + (i % kGStages) * stage;
       for (int r = kr0, u = ku0; r < kGKeys;) {
@@ -198,7 +205,7 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
         u += kus;
         if (u >= ku) { u -= ku; ++r; }
       }
-      for (int r = vr0, u = vu0; r < kGKeys;) {
+      for (int r = p.tied ? kGKeys : vr0, u = vu0; r < kGKeys;) {
         g_cp16(dst + kGKeys * ks + r * vs + u * 16, v + r * vw + u * 8);
         r += vrs;
         u += vus;
@@ -226,8 +233,12 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
 #pragma unroll
   for (int x = 0; x < NV * 2; ++x) o[x][0] = o[x][1] = o[x][2] = o[x][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-  const uint32_t k_off = ((lane & 7) + ((lane >> 4) << 3)) * ks + ((lane >> 3) & 1) * 16;
-  const uint32_t v_off = kGKeys * ks + (lane & 15) * vs + (lane >> 4) * 16;
+  if (p.sink && warp == 0 && split == 0) {       // (counted once; a lane's l is a part of its row's)
+    if (r0 < R) { m0 = p.sink[g * p.R + head0 + r0] * 1.4426950408889634f; l0 = (lane & 3) == 0 ? 1.f : 0.f; }
+    if (r0 + 8 < R) { m1 = p.sink[g * p.R + head0 + r0 + 8] * 1.4426950408889634f; l1 = (lane & 3) == 0 ? 1.f : 0.f; }
+  }
+  const uint32_t k_off = ((lane & 7) + ((lane >> 4) << 3)) * ks + ((lane >> 3) & 1) * 16 + p.key_at * 2;
+  const uint32_t v_off = (p.tied ? 0 : kGKeys * ks) + (lane & 15) * vs + (lane >> 4) * 16;
   for (int i = 0; i < n; ++i) {
     g_wait<kGStages - 2>();
     __syncwarp();
@@ -332,7 +343,7 @@ __global__ void __launch_bounds__(kGWarps * 32, ND + NV <= 16 ? 2 : 1) grouped_d
       y.x += v.x;
       y.y += v.y;
     }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    const float inv = l > 0.f ? p.out_scale / l : 0.f;
     const size_t h = (size_t)g * p.R + head0 + r;
     if (p.splits == 1) {
       *reinterpret_cast<uint32_t*>(p.out + (size_t)b * p.ldo + h * p.V + c) = pack_bf16x2(y.x * inv, y.y * inv);
@@ -546,15 +557,16 @@ static int launch_rotate_rows(const RotateParams& p, cudaStream_t stream) {
 }
 
 bool grouped_decode_fits(const B200BiasAttn* a) {
-  if (!a->grouped || a->f32 || a->bias || a->null_entry || a->kw % a->G || a->values_in_keys || a->gate) return false;
-  const int D = a->kw / a->G, V = a->vdim;
+  if (!a->grouped || a->f32 || a->bias || a->null_entry || a->kw % a->G || a->gate) return false;
+  if (a->values_in_keys && (a->maps > 1 || (a->kw / a->G & 7) || (a->key_at & 7))) return false;
+  const int D = a->kw / a->G - a->key_at, V = a->vdim;
   return !(D / (a->maps > 1 ? a->maps : 1) & 15) && !(V & 15) && D <= 256 && V <= 256 && a->block_size % kGKeys == 0 &&
          !(((uintptr_t)a->q | (uintptr_t)a->cache) & 15) && !(a->ldq & 7) && !(a->ldo & 1) && a->scale > 0.f;
 }
 
 template <int ND, int NV>
 static int launch_grouped(const GroupedDecode& p, int rows, cudaStream_t stream) {
-  size_t smem = (size_t)kGWarps * kGStages * g_stage_bytes(p.D, p.V);
+  size_t smem = (size_t)kGWarps * kGStages * (p.tied ? kGKeys * g_tied_row(p.pitch) : g_stage_bytes(p.D, p.V));
   const size_t merge = (size_t)kGWarps * 16 * p.V * 4;
   if (smem < merge) smem = merge;
   static PerDeviceOnce once;
@@ -570,15 +582,90 @@ static int launch_grouped(const GroupedDecode& p, int rows, cudaStream_t stream)
 
 int grouped_decode(const B200BiasAttn* a, cudaStream_t stream) {
   GroupedDecode p{(const bf16*)a->q, a->ldq, (bf16*)a->out, a->ldo, (const bf16*)a->cache, (const int32_t*)a->block_table,
-                  (const int32_t*)a->seq_lens, a->max_blocks, a->H, a->G, a->H / a->G, a->kw / a->G, a->vdim, a->block_size,
+                  (const int32_t*)a->seq_lens, a->max_blocks, a->H, a->G, a->H / a->G, a->kw / a->G - a->key_at, a->vdim, a->block_size,
                   a->chunk, a->splits < 1 ? 1 : a->splits, a->window, a->maps > 1 ? a->maps : 1, a->scale * 1.4426950408889634f, (float*)a->tmp_o,
-                  (float*)a->tmp_lse};
+                  (float*)a->tmp_lse, a->kw / a->G, a->key_at, a->values_in_keys, a->sink, a->out_scale};
   if (p.splits > 1 && (!p.tmp_o || !p.tmp_lse)) return -1;
   if ((long)p.G * ((p.R + 15) / 16) > 65535 || p.splits > 65535) return -4;
   const int rc = p.D <= 64 ? launch_grouped<4>(p, a->rows, stream) : p.D <= 128 ? launch_grouped<8>(p, a->rows, stream)
                                                                                 : launch_grouped<16>(p, a->rows, stream);
   if (rc || p.splits == 1) return rc;
   return b200_attn_decode_merge(p.tmp_o, p.tmp_lse, p.out, (int)p.ldo, a->rows, p.H, p.V, p.splits, stream);
+}
+
+// --------------------------------------------------------- rotation where values are unrotated keys
+// One CTA per token. A head of the projection is [first r8 | rest], of which rot are rotated (pairs half of rot apart); the
+// query row becomes [rest | first rotated], a group's cache row [first | rest | first rotated]. A thread copies VEC values
+// of the rest or turns VEC pairs; the padding after rot is zeros.
+struct TiedRotate {
+  const void* qk;
+  long long ld;
+  const int64_t* positions;
+  const float* cos_sin;
+  void* q_out;
+  long long ldq;
+  const int64_t* slots;
+  void* cache;
+  int rot, r8, H, G, D, block_size;
+};
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128) rotate_tied_kernel(TiedRotate p) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x, half = p.rot / 2, rest = p.D - p.r8, pitch = p.D + p.r8;
+  const int copies = rest / VEC, turns = half / VEC, units = copies + turns, pads = VEC == 1 ? p.r8 - p.rot : 0;
+  const T* row = reinterpret_cast<const T*>(p.qk) + (size_t)t * p.ld;
+  const int64_t slot = p.slots[t];
+  T* line = slot < 0 ? nullptr : reinterpret_cast<T*>(p.cache) + slot * p.G * pitch;   // (pages hold rows only)
+  const float* cs = p.cos_sin ? p.cos_sin + (size_t)p.positions[t] * p.rot : nullptr;
+  for (int x = threadIdx.x; x < (p.H + p.G) * (units + pads); x += blockDim.x) {
+    const int h = x / (units + pads), u = x - h * (units + pads);
+    const bool is_q = h < p.H;
+    if (!is_q && !line) continue;
+    const T* src = row + (size_t)h * p.D;
+    T* head = is_q ? reinterpret_cast<T*>(p.q_out) + (size_t)t * p.ldq + (size_t)h * p.D : line + (size_t)(h - p.H) * pitch;
+    T* key = is_q ? head : head + p.r8;              // [rest | first rotated]
+    if (u < copies) {
+      if (VEC == 8) *reinterpret_cast<uint4*>(key + u * 8) = *reinterpret_cast<const uint4*>(src + p.r8 + u * 8);
+      else key[u] = src[p.r8 + u];
+    } else if (u < units) {
+      const int i = (u - copies) * VEC;
+      float a[VEC], b[VEC], y[VEC], z[VEC];
+      if constexpr (VEC == 8) {
+        Ld8<T>::get(src + i, a);
+        Ld8<T>::get(src + half + i, b);
+      } else {
+        a[0] = (float)src[i];
+        b[0] = (float)src[half + i];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        const float c = cs[i + e], s = cs[half + i + e];
+        y[e] = a[e] * c - b[e] * s;
+        z[e] = b[e] * c + a[e] * s;
+      }
+      T* turned = key + rest;
+      if constexpr (VEC == 8) {
+        Ld8<T>::put(turned + i, y);
+        Ld8<T>::put(turned + half + i, z);
+        if (!is_q) {
+          Ld8<T>::put(head + i, a);
+          Ld8<T>::put(head + half + i, b);
+        }
+      } else {
+        turned[i] = (T)y[0];
+        turned[half + i] = (T)z[0];
+        if (!is_q) {
+          head[i] = src[i];
+          head[half + i] = src[half + i];
+        }
+      }
+    } else {
+      const int i = p.rot + u - units;
+      key[rest + i] = (T)0.f;
+      if (!is_q) head[i] = (T)0.f;
+    }
+  }
 }
 
 // ----------------------------------------------------------------------- difference of two maps
@@ -652,6 +739,23 @@ int b200_rotate_kv(const void* qkv, long long ld, const void* positions, const v
   const size_t smem = (size_t)4 * D * 4;
   return (f32 ? launch_pdl(rotate_kv_kernel<float>, grid, dim3(128), smem, stream, p)
               : launch_pdl(rotate_kv_kernel<bf16>, grid, dim3(128), smem, stream, p)) == cudaSuccess ? 0 : -2;
+}
+
+int b200_rotate_tied(const void* qk, long long ld, const void* positions, const void* cos_sin, int rot, void* q_out, long long ldq,
+                     const void* slots, void* cache, int H, int G, int D, int block_size, int T, int f32, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  const int r8 = (rot + 7) / 8 * 8;
+  if (H <= 0 || G <= 0 || D <= 0 || rot < 0 || (rot & 1) || r8 > D || (D & 7) || (rot && !cos_sin) || block_size <= 0) return -1;
+  const TiedRotate p{qk, ld, (const int64_t*)positions, (const float*)cos_sin, q_out, ldq, (const int64_t*)slots, cache, rot, r8,
+                     H, G, D, block_size};
+  const int es = f32 ? 4 : 2;
+  const bool vec = !(((uintptr_t)qk | (uintptr_t)q_out | (uintptr_t)cache | (uintptr_t)(ld * es) | (uintptr_t)(ldq * es)) & 15) &&
+                   !(rot & 15) && !f32;
+  cudaError_t e;
+  if (vec) e = launch_pdl(rotate_tied_kernel<bf16, 8>, dim3(T), dim3(128), 0, stream, p);
+  else if (f32) e = launch_pdl(rotate_tied_kernel<float, 1>, dim3(T), dim3(128), 0, stream, p);
+  else e = launch_pdl(rotate_tied_kernel<bf16, 1>, dim3(T), dim3(128), 0, stream, p);
+  return e == cudaSuccess ? 0 : -2;
 }
 
 int b200_diff_combine(const void* maps, long long ldm, void* out, long long ldo, int H, int V, int vdim, int T, float lam,

@@ -74,6 +74,7 @@ struct GemmParams {
   // so a tile holds both halves of 128 outputs; out[M, N / 2] = act(gate) * up. 0 = off,
   // otherwise activation kind + 1 (1 SiLU, 2 GELU-tanh, 3 GELU-erf).
   int act_fuse;
+  int act;                        // activation of the result (act_epilogue)
   // fp8 (e4m3 x e4m3) instantiation of the pair kernel: out = acc * a_scale * w_scale[(n)]
   const float* scale_a;
   const float* scale_w;
@@ -417,6 +418,10 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
               }
             }
           }
+          if (p.act) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) v[i] = act_epilogue(v[i], p.act);
+          }
           if (p.tp_world > 1 && p.peer_recv[0]) {
             const int owner = row / p.rows_per_rank;
             const uint32_t par = *p.op_counter & 1;
@@ -521,6 +526,10 @@ __device__ __forceinline__ void epilogue_store_chunk(const GemmParams& p, float 
         f = unpack_bf16x2(b.w); v[i + 6] += f.x; v[i + 7] += f.y;
       }
     }
+  }
+  if (p.act) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) v[i] = act_epilogue(v[i], p.act);
   }
   if (p.out_f32) {
     float* o = reinterpret_cast<float*>(p.out) + (size_t)row * p.ldo + col0;
@@ -1033,6 +1042,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
               } else {
                 v += bias_v;
                 if (p.residual) v += __bfloat162float(p.residual[(size_t)m * p.ldr + n]);
+                v = act_epilogue(v, p.act);
                 const size_t o = (size_t)bz * p.batch_out_stride + (size_t)m * p.ldo + n;
                 if (p.out_f32)
                   reinterpret_cast<float*>(p.out)[o] = v;
@@ -1067,7 +1077,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
 __global__ void splitk_reduce_kernel(const float* __restrict__ ws, int splits, int M, int N,
                                      void* out, int ldo, int out_f32,
                                      const __nv_bfloat16* __restrict__ bias,
-                                     const __nv_bfloat16* __restrict__ residual, int ldr) {
+                                     const __nv_bfloat16* __restrict__ residual, int ldr, int act) {
   pdl_wait();                 // predecessor grid complete, its writes visible
   pdl_launch_dependents();    // the successor may become resident (it waits the same way)
   const int n4 = N >> 2;
@@ -1090,6 +1100,10 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ ws, int splits, i
       uint2 b = *reinterpret_cast<const uint2*>(residual + (size_t)m * ldr + n);
       float2 f0 = unpack_bf16x2(b.x), f1 = unpack_bf16x2(b.y);
       acc.x += f0.x; acc.y += f0.y; acc.z += f1.x; acc.w += f1.y;
+    }
+    if (act) {
+      acc.x = act_epilogue(acc.x, act); acc.y = act_epilogue(acc.y, act);
+      acc.z = act_epilogue(acc.z, act); acc.w = act_epilogue(acc.w, act);
     }
     if (out_f32) {
       *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + (size_t)m * ldo + n) = acc;
@@ -1416,8 +1430,9 @@ static int gemm_bf16_impl(const void* A, int lda, const void* W, int ldw, void* 
                           const B200TpGemm* tp, cudaStream_t stream, int act_fuse) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   // bit 8 of force_path: W is a constant weight (nothing in the stream writes it)
-  const int w_early = (force_path >> 8) & 1;
+  const int w_early = (force_path >> 8) & 1, act = (force_path >> 9) & 7;
   force_path &= 0xff;
+  if (act > 4 || (act && (tp || act_fuse))) return -1;
   if (act_fuse && ((tp && tp->scatter) || M <= 128 || (N & 255) || bias || residual || out_f32)) return -1;
   if (act_fuse && force_path == 0) force_path = 9;      // the gated epilogue lives in the pair kernel
   if ((K & 7) || (lda & 7) || (ldw & 7) || (N & 7) || (ldo & 7) || (residual && (ldr & 7))) return -1;
@@ -1428,7 +1443,7 @@ static int gemm_bf16_impl(const void* A, int lda, const void* W, int ldw, void* 
   GemmParams p{};
   p.w_early = (w_early && !tp) ? 1 : 0;
   p.M = M; p.N = N; p.K = K;
-  p.out = out; p.ldo = ldo; p.out_f32 = out_f32;
+  p.out = out; p.ldo = ldo; p.out_f32 = out_f32; p.act = act;
   p.bias = reinterpret_cast<const __nv_bfloat16*>(bias);
   p.residual = reinterpret_cast<const __nv_bfloat16*>(residual);
   p.ldr = ldr;
@@ -1527,10 +1542,10 @@ static int gemm_bf16_impl(const void* A, int lda, const void* W, int ldw, void* 
       if (blocks > sms * 8) blocks = sms * 8;
       if (tp) {
         splitk_reduce_kernel<<<blocks, 256, 0, stream>>>(p.workspace, splits, M, N, out, ldo,
-                                                         out_f32, p.bias, p.residual, ldr);
+                                                         out_f32, p.bias, p.residual, ldr, act);
         if (cudaGetLastError() != cudaSuccess) return -2;
       } else if (launch_pdl(splitk_reduce_kernel, dim3(blocks), dim3(256), 0, stream, (const float*)p.workspace,
-                            splits, M, N, out, ldo, out_f32, p.bias, p.residual, ldr) != cudaSuccess) {
+                            splits, M, N, out, ldo, out_f32, p.bias, p.residual, ldr, act) != cudaSuccess) {
         return -2;
       }
     }
@@ -1787,7 +1802,7 @@ extern "C" int b200_gemm_bf16_smallm_static(const void* A, int lda, const void* 
     int blocks = (int)((total + 255) / 256);
     if (blocks > sms * 8) blocks = sms * 8;
     splitk_reduce_kernel<<<blocks, 256, 0, stream>>>(sd.scratch, splits, M, N, out, ldo, 0,
-                                                     nullptr, nullptr, 0);
+                                                     nullptr, nullptr, 0, 0);
     if (cudaGetLastError() != cudaSuccess) { g_static_err = "reduce launch failed"; return -2; }
   }
   return 0;

@@ -276,6 +276,7 @@ struct GroupedParams {
   // activation kernel would see them.
   int act_fuse;
   B200ClampedGate clamp;    // act_fuse == 4: clamped pair, applied to the fp32 accumulators
+  int act;                  // not gated: activation of the result (act_epilogue)
   int* status;
 };
 struct alignas(8) GroupedBars {
@@ -423,7 +424,7 @@ __global__ void __launch_bounds__(192, 1)
           for (int i = 0; i < 16; ++i) {
             const int m = c * 16 + i;
             if (m < rows)
-              p.out[(size_t)(row0 + m) * p.N + n] = __float2bfloat16(__uint_as_float(r[i]));
+              p.out[(size_t)(row0 + m) * p.N + n] = __float2bfloat16(act_epilogue(__uint_as_float(r[i]), p.act));
           }
         }
       }
@@ -589,9 +590,9 @@ int b200_moe_gather(const void* x, int ldx, const void* sorted_token, const void
 static int moe_grouped_gemm_impl(const void* xs, int max_rows, const void* W, int E, int N, int K,
                                  void* out, const void* chunk_expert, const void* chunk_row0,
                                  const void* chunk_n, const void* meta, int max_chunks, int act_fuse,
-                                 cudaStream_t stream, const B200ClampedGate* clamp = nullptr) {
+                                 cudaStream_t stream, const B200ClampedGate* clamp = nullptr, int act = 0) {
   if (max_rows <= 0) return 0;
-  if ((K & 7) || (N & 7)) return -1;
+  if ((K & 7) || (N & 7) || act < 0 || act > 4) return -1;
   if (act_fuse && ((N & 1) || ((N / 2) & 7) || act_fuse < 1 || act_fuse > 4 || (act_fuse == 4) != (clamp != nullptr)))
     return -1;
   static std::mutex mu;
@@ -612,7 +613,7 @@ static int moe_grouped_gemm_impl(const void* xs, int max_rows, const void* W, in
   if (stages > kGMaxStages) stages = kGMaxStages;
   const int nkb = (K + kGBK - 1) / kGBK;
   if (stages > nkb) stages = nkb < 2 ? 2 : nkb;
-  p.stages = stages; p.act_fuse = act_fuse; p.status = device_status_word();
+  p.stages = stages; p.act_fuse = act_fuse; p.act = act; p.status = device_status_word();
   if (clamp) p.clamp = *clamp;
   const size_t smem = (size_t)stages * stage + 1024 + sizeof(GroupedBars);
   static PerDeviceOnce attr_once;
@@ -650,6 +651,14 @@ int b200_moe_grouped_gemm_clamped(const void* xs, int max_rows, const void* W, i
   if (!act) return -1;
   return moe_grouped_gemm_impl(xs, max_rows, W, E, N, K, out, chunk_expert, chunk_row0, chunk_n, meta, max_chunks, 4,
                                stream, act);
+}
+// The plain product with an activation of the result (act_epilogue).
+int b200_moe_grouped_gemm_act(const void* xs, int max_rows, const void* W, int E, int N, int K,
+                              void* out, const void* chunk_expert, const void* chunk_row0,
+                              const void* chunk_n, const void* meta, int max_chunks, int act,
+                              cudaStream_t stream) {
+  return moe_grouped_gemm_impl(xs, max_rows, W, E, N, K, out, chunk_expert, chunk_row0, chunk_n, meta, max_chunks, 0,
+                               stream, nullptr, act);
 }
 int b200_moe_row_weights(const void* pair_pos, const void* topk_w, int P, void* row_w, cudaStream_t stream) {
   if (P <= 0) return 0;

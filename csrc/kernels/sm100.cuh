@@ -512,4 +512,13 @@ inline cudaError_t launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, s
   return cudaLaunchKernelEx(&cfg, kernel, KArgs(static_cast<Args&&>(args))...);
 }
 #endif
+// Activations in the epilogue of a product: 0 none, 1 SiLU, 2 GELU-tanh, 3 GELU-erf, 4 squared ReLU.
+__device__ __forceinline__ float act_epilogue(float x, int act) {
+  if (act == 4) { x = fmaxf(x, 0.f); return x * x; }
+  if (act == 2) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+  if (act == 1) return x / (1.f + expf(-x));
+  if (act == 3) return 0.5f * x * (1.f + erff(x * 0.7071067811865476f));
+  return x;
+}
+
 }  // namespace b200

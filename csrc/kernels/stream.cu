@@ -177,6 +177,7 @@ struct F32Gemm {
   const int32_t* chunk_row0;
   const int32_t* chunk_n;
   const int32_t* num_chunks;
+  int act;
 };
 
 static constexpr int kFT = 64, kFK = 16;
@@ -235,7 +236,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(F32Gemm p) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < p.N) out[(size_t)(row_base + m) * p.ldo + n] = acc[i][j] + (p.bias ? p.bias[n] : 0.f);
+      if (n < p.N) out[(size_t)(row_base + m) * p.ldo + n] = act_epilogue(acc[i][j] + (p.bias ? p.bias[n] : 0.f), p.act);
     }
   }
 }
@@ -307,10 +308,10 @@ int b200_stream_norm(const B200StreamNorm* a, cudaStream_t stream) {
 }
 
 int b200_gemm_f32(const void* A, int lda, const void* W, int ldw, void* out, int ldo, const void* bias, int M, int N,
-                  int K, cudaStream_t stream) {
+                  int K, int act, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   F32Gemm p{(const float*)A, (const float*)W, (const float*)bias, (float*)out, lda, ldw, ldo, M, N, K,
-            0, 0, 0, nullptr, nullptr, nullptr, nullptr};
+            0, 0, 0, nullptr, nullptr, nullptr, nullptr, act};
   dim3 grid((N + kFT - 1) / kFT, (M + kFT - 1) / kFT);
   if (grid.y > 65535) return -4;
   return launch_pdl(gemm_f32_kernel, grid, dim3(256), 0, stream, p) == cudaSuccess ? 0 : -2;
@@ -321,7 +322,7 @@ int b200_gemm_f32_batched(const void* A, int lda, int a_batch, const void* W, in
                           long long out_batch, int M, int N, int K, int batch, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
   F32Gemm p{(const float*)A, (const float*)W, nullptr, (float*)out, lda, ldw, ldo, M, N, K,
-            a_batch, (long long)N * ldw, out_batch, nullptr, nullptr, nullptr, nullptr};
+            a_batch, (long long)N * ldw, out_batch, nullptr, nullptr, nullptr, nullptr, 0};
   dim3 grid((N + kFT - 1) / kFT, (M + kFT - 1) / kFT, batch);
   if (grid.y > 65535 || grid.z > 65535) return -4;
   return launch_pdl(gemm_f32_kernel, grid, dim3(256), 0, stream, p) == cudaSuccess ? 0 : -2;
@@ -338,11 +339,18 @@ int b200_softcap_f32(void* x, long long n, float cap, cudaStream_t stream) {
 int b200_moe_grouped_gemm_f32(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out,
                               const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta,
                               int max_chunks, cudaStream_t stream) {
+  return b200_moe_grouped_gemm_f32_act(xs, max_rows, W, E, N, K, out, chunk_expert, chunk_row0, chunk_n, meta, max_chunks, 0,
+                                       stream);
+}
+
+int b200_moe_grouped_gemm_f32_act(const void* xs, int max_rows, const void* W, int E, int N, int K, void* out,
+                                  const void* chunk_expert, const void* chunk_row0, const void* chunk_n, const void* meta,
+                                  int max_chunks, int act, cudaStream_t stream) {
   if (max_rows <= 0) return 0;
   if (max_chunks > 65535) return -4;
   F32Gemm p{(const float*)xs, (const float*)W, nullptr, (float*)out, K, K, N, max_rows, N, K,
             0, 0, 0, (const int32_t*)chunk_expert, (const int32_t*)chunk_row0, (const int32_t*)chunk_n,
-            (const int32_t*)meta + 3 * E + 1};
+            (const int32_t*)meta + 3 * E + 1, act};
   dim3 grid((N + kFT - 1) / kFT, 256 / kFT, max_chunks);     // a chunk has at most 256 rows
   return launch_pdl(gemm_f32_kernel, grid, dim3(256), 0, stream, p) == cudaSuccess ? 0 : -2;
 }

@@ -85,7 +85,8 @@ def segment_tiles(num_tiles: int, portions: int, ctas: int, num_sms: int) -> int
 
 def workspace_values(s: OuterShape, max_tokens: int) -> tuple[int, int]:
     """fp32 values of (states, decays) of the cut portions of a step."""
-    segments = 2 * (max_tokens // (128 * MIN_SEGMENT) + 1)
+    # (a cut portion has 2 MIN_SEGMENT tiles at least, the last of them partly filled)
+    segments = 2 * (max_tokens * 8 // (7 * 128 * MIN_SEGMENT) + 2)
     return segments * s.H * s.D * s.V, segments * s.H * s.D
 
 
