@@ -327,7 +327,7 @@ def main() -> int:
                     help="skip the extra keys (the whole offline batch and the concurrency sweep)")
     ap.add_argument("--sync-scheduling", action="store_true",
                     help="schedule step N+1 only after step N's tokens are on the host")
-    ap.add_argument("--design", default=None, choices=["nufusun", "diforax", "tabupel"],
+    ap.add_argument("--design", default=None, choices=["nufusun", "diforax", "tabupel", "kubolorn"],
                     help="instead of the serving workload: prefill and decode throughput of this design and the "
                          "roofline fractions of its kernels beside the closest other model at equal layer sizes")
     ap.add_argument("--design-size", action="append", help="one of the --design sizes (default: all)")

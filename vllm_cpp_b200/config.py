@@ -849,6 +849,27 @@ def synthetic_config(name: str) -> ModelConfig:
         return model_config_of_blocks("Tabupel", [BlockSpec(None, None, latent=lat), rec, BlockSpec(att, DenseSpec(64)),
                                                   BlockSpec(None, ff, rglru=rec.rglru, weights_of=1)],
                                       vocab=500, width=192, eps=1e-5, residual_mult=0.7, logit_softcap=20.0, max_position=2048)
+    if n == "kubolorn-3b":
+        # three linear-attention layers to one parallel layer; the parallel layers carry the experts
+        g = BlockSpec(None, DenseSpec(8192, plain="gelu_tanh"), gla=GlaSpec(heads=16, dim=128, vdim=128, tau=16.0))
+        att = AttentionSpec(heads=32, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, rot_dims=64, rot_base=1e6,
+                            rot_scaling=RotaryScaling(8.0, 8192), sink=True, tied=True)
+        p = BlockSpec(att, ExpertSpec(experts=64, top=4, ff=1024, plain="relu2"), scales=(0.7, 0.7),
+                      ssm=SsmSpec(heads=32, groups=4, state=128, vdim=64, conv=4, norm_groups=4))
+        loop = LoopSpec(start=8, stop=16, times=2)
+        return model_config_of_blocks("Kubolorn", unrolled([g, g, g, p] * 6, loop), vocab=151936, width=2048, eps=1e-6, embed_scale=45.0,
+                                      norm_groups=4, input_conv=4, bigram=BigramSpec(65521, 31337, 7919), loop=loop,
+                                      max_position=65536)
+    if n == "tiny-kubolorn":
+        att = AttentionSpec(heads=6, kv_heads=2, dim=40, vdim=40, scale=0.2, rot_dims=24, rot_base=5e3,
+                            rot_scaling=RotaryScaling(3.0, 64), sink=True, tied=True)
+        p = BlockSpec(att, ExpertSpec(experts=4, top=2, ff=48, plain="relu2"), scales=(0.9, 1.1),
+                      ssm=SsmSpec(heads=6, groups=2, state=24, vdim=32, conv=3, norm_groups=4))
+        g = BlockSpec(None, DenseSpec(96, plain="gelu_tanh"), gla=GlaSpec(heads=3, dim=24, vdim=40, tau=8.0, rank=8))
+        loop = LoopSpec(start=0, stop=2, times=2)
+        return model_config_of_blocks("Kubolorn", unrolled([g, p, BlockSpec(None, None, gla=g.gla)], loop), vocab=500, width=192, eps=1e-5,
+                                      embed_scale=2.0, norm_groups=3, input_conv=2, bigram=BigramSpec(101, 7, 3), loop=loop,
+                                      max_position=2048)
     if n.startswith("tiny"):
         # small shapes for tests: tiny-dense, tiny-moe, tiny-mla, tiny-gdn
         base = dict(vocab_size=512, hidden_size=256, intermediate_size=512, num_layers=2,

@@ -1,9 +1,9 @@
 """Throughput of a design with listed layers beside the closest other model of this package at equal layer
 sizes, and its kernels beside the like kernels of that model, each against its roofline.
 
-``bench.py --design nufusun`` (beside Qwen3-MoE), ``--design diforax`` (beside the Qwen3.5 MoE hybrids) or
-``--design tabupel`` (beside the dense Qwen3.5 hybrids, its latent kernels beside DeepSeek-V2's) runs it and
-prints one JSON line. Random weights; device time (CUDA events); kernels are timed with an L2 flush
+``bench.py --design nufusun`` (beside Qwen3-MoE), ``--design diforax`` (beside the Qwen3.5 MoE hybrids),
+``--design tabupel`` (beside the dense Qwen3.5 hybrids, its latent kernels beside DeepSeek-V2's) or ``--design kubolorn``
+(beside the Qwen3.5 hybrids, dense or with experts) runs it and prints one JSON line. Random weights; device time (CUDA events); kernels are timed with an L2 flush
 between iterations, median of several."""
 from __future__ import annotations
 
@@ -40,6 +40,42 @@ TABUPEL_SIZES = {
     "small layers": (1024, 3072, 12, 8, 4, 64, 8, 512, 512, 1024, 8),
     "wide layers": (4096, 12288, 6, 32, 8, 64, 16, 1536, 512, 4096, 16),
 }
+
+
+# width, attention heads, kv heads, size, experts (0: dense), top, expert or dense size, layers, linear-attention heads and
+# state-space heads (states of 128 x 128 and 128 x 64)
+KUBOLORN_FIELDS = FIELDS + ("gla_heads", "ssm_heads")
+KUBOLORN_SIZES = {
+    "2b layers": (2048, 16, 4, 128, 0, 0, 8192, 8, 16, 32),
+    "30b-a3b layers": (2048, 32, 4, 128, 128, 8, 768, 4, 16, 32),
+    "small layers": (1024, 16, 4, 64, 32, 4, 512, 8, 8, 16),
+    "wide layers": (4096, 32, 8, 128, 0, 0, 12288, 4, 32, 64),
+}
+
+
+def kubolorn_configs(size):
+    """Three linear-attention layers to one layer with attention beside a state-space mixer. The other model: as many
+    delta-rule heads of 128 x 128, one attention layer in four; its gated units are two thirds as wide, so that the
+    feed-forwards hold as many weights."""
+    from ..config import (AttentionSpec, BigramSpec, BlockSpec, DenseSpec, ExpertSpec, GlaSpec, ModelConfig, RopeConfig, RotaryScaling,
+                          SsmSpec, model_config_of_blocks)
+    W, H, G, D, E, top, ff, layers, gh, sh = size
+    mlp = ExpertSpec(experts=E, top=top, ff=ff * 3 // 2, plain="relu2") if E else DenseSpec(ff, plain="gelu_tanh")
+    g = BlockSpec(None, mlp, gla=GlaSpec(heads=gh, dim=128, vdim=128, tau=16.0))
+    a = AttentionSpec(heads=H, kv_heads=G, dim=D, vdim=D, scale=D ** -0.5, rot_dims=D // 2, rot_base=1e6, rot_scaling=RotaryScaling(8.0, 8192),
+                      sink=True, tied=True)
+    p = BlockSpec(a, mlp, ssm=SsmSpec(heads=sh, groups=4, state=128, vdim=64, conv=4, norm_groups=4), scales=(0.7, 0.7))
+    mine = model_config_of_blocks("Kubolorn", [p if l % 4 == 3 else g for l in range(layers)], vocab=32000, width=W, eps=1e-6,
+                                  embed_scale=1.0, norm_groups=4, input_conv=4, bigram=BigramSpec(32749, 31337, 7919))
+    dense = dict(architecture="Qwen3_5ForConditionalGeneration", intermediate_size=ff * 2 // 3 // 128 * 128)
+    moe = dict(architecture="Qwen3_5MoeForConditionalGeneration", intermediate_size=3 * W, num_experts=E, num_experts_per_tok=top,
+               moe_intermediate_size=ff, norm_topk_prob=True)
+    other = ModelConfig(vocab_size=32000, hidden_size=W, num_layers=layers, num_heads=H, num_kv_heads=G, head_dim=D,
+                        max_position_embeddings=32768, qk_norm=True, gemma_norm=True, attn_output_gate=True, rope=RopeConfig(theta=1e6),
+                        layer_types=["full_attention" if l % 4 == 3 else "linear_attention" for l in range(layers)],
+                        linear_num_key_heads=gh, linear_num_value_heads=gh, linear_key_head_dim=128, linear_value_head_dim=128,
+                        linear_conv_kernel_dim=4, **(moe if E else dense))
+    return {"kubolorn": mine, "qwen3.5": other}
 
 
 def tabupel_configs(size):
@@ -703,8 +739,204 @@ class TabupelKernels(KernelBench):
             self.add(f"logit cap, {T} rows", "tabupel", lambda: softcap_f32(logits, 30.0), nbytes=T * 32000 * 8)
 
 
+class KubolornKernels(KernelBench):
+    def __init__(self, size):
+        super().__init__(size)
+        self.gh, self.sh = size[8:]
+
+    def run(self):
+        self.attention(B=4, prompt=2048, decode_batch=64, ctx=4096)
+        self.attention(B=8, prompt=1024, decode_batch=8, ctx=16384)
+        for B, n in ((4, 2048), (8, 1024), (1, 8192), (16, 1), (64, 1), (256, 1)):
+            self.recurrences(B, n)
+        for T in (64, 8192):
+            self.rest(T)
+
+    def attention(self, B, prompt, decode_batch, ctx, bs=32):
+        from .. import ops
+        from ..ops import bias_attn as A
+        from ..ops.reference import build_prefill_tiles
+        H, G, D = self.H, self.G, self.D
+        s, T, nb, scale = A.TiedShape(H, G, D, D // 2), B * prompt, prompt // bs, D ** -0.5
+        row = G * s.pitch
+        shape = dict(H=H, G=G, kw=row, vdim=s.D, block_size=bs, grouped=True, values_in_keys=True, key_at=s.r8, scale=scale)
+        sink = self.rnd(H, dtype=torch.float32)
+        bt = torch.arange(1, B * nb + 1, device=self.dev, dtype=torch.int32).view(B, nb)
+        tr, tq = (self.i32(x) for x in build_prefill_tiles([prompt] * B))
+        rows = dict(seq_lens=self.i32([prompt] * B), q_start=self.i32([i * prompt for i in range(B + 1)]), tile_req=tr, tile_q0=tq)
+        q, pages, kv = self.rnd(T, H * D), self.rnd(B * nb + 1, bs * row), self.rnd(B * nb + 1, 2, bs, G, D)
+        out = torch.empty(T, H * D, dtype=torch.bfloat16, device=self.dev)
+        flops = 2 * B * (prompt * (prompt + 1) / 2) * H * 2 * D
+        what = f"attention, {B} x {prompt} prompt"
+        self.add(what, "kubolorn", lambda: A.prefill(q, pages, out, block_table=bt, num_reqs=B, sink=sink, **rows, **shape), flops=flops,
+                 note=A.kernel_kind("prefill", q, pages, **shape))
+        self.add(what, "qwen3.5", lambda: ops.attn_prefill(q, kv, block_table=bt, num_q_heads=H, num_kv_heads=G, head_dim=D, block_size=bs,
+                                                           scale=scale, out=out, **rows), flops=flops)
+        qk, pos = self.rnd(T, (H + G) * D), torch.arange(T, device=self.dev) % prompt
+        slots = (bt.long()[:, :, None] * bs + torch.arange(bs, device=self.dev)).reshape(-1)
+        table, qkv, nw = self.rnd(prompt, D, dtype=torch.float32), self.rnd(T, (H + 2 * G) * D), self.rnd(D)
+        half = table[:, : D // 2].contiguous()
+        what = f"query preparation + cache write, {T} tokens"
+        self.add(what, "kubolorn", lambda: A.rotate_tied(qk, pos, half, q, slots, pages, s, block_size=bs),
+                 nbytes=T * 2 * ((H + G) * D + H * D + row))
+        self.add(what, "qwen3.5", lambda: ops.rope_kv(qkv, pos, table, num_q_heads=H, num_kv_heads=G, head_dim=D, q_norm=nw, k_norm=nw,
+                                                      slot_mapping=slots, kv_cache=kv, block_size=bs, q_out=q), nbytes=T * 2 * (H + 2 * G) * D * 2)
+        B, nb = decode_batch, ctx // bs
+        bt = torch.arange(1, B * nb + 1, device=self.dev, dtype=torch.int32).view(B, nb)
+        sl, pages, kv, q = self.i32([ctx] * B), self.rnd(B * nb + 1, bs * row), self.rnd(B * nb + 1, 2, bs, G, D), self.rnd(B, H * D)
+        out = torch.empty(B, H * D, dtype=torch.bfloat16, device=self.dev)
+        splits = A.grouped_decode_splits(B, G, ctx, ops.num_sms())
+        tmp = (torch.empty(B * H * splits * D, dtype=torch.float32, device=self.dev), torch.empty(B * H * splits, dtype=torch.float32, device=self.dev))
+        what = f"attention, decode {B} x {ctx}"
+        self.add(what, "kubolorn", lambda: A.decode(q, pages, out, block_table=bt, seq_lens=sl, splits=splits, tmp=tmp, sink=sink, **shape),
+                 nbytes=B * ctx * row * 2, note=A.kernel_kind("decode", q, pages, **shape))
+        self.add(what, "qwen3.5", lambda: ops.attn_decode(q, kv, block_table=bt, seq_lens=sl, num_q_heads=H, num_kv_heads=G, head_dim=D,
+                                                          block_size=bs, scale=scale, out=out), nbytes=B * ctx * 2 * G * D * 2)
+
+    def recurrences(self, B, n):
+        """``B`` prompts of ``n`` tokens, or (n 1) a decode batch: both recurrences with their norms, and the convolution of the
+        state-space mixer; beside the delta rule of as many heads."""
+        from types import SimpleNamespace
+        from ..ops import gdn as Q
+        from ..ops import outer as O
+        from ..ops import rglru as R
+        from ..ops.reference import build_prefill_tiles
+        T, f32, H = B * n, dict(dtype=torch.float32), self.gh
+        tr, tq = build_prefill_tiles([n] * B) if n > 1 else ([], [])
+        rows = SimpleNamespace(seq_lens=self.i32([n + 5] * B), state_slots=self.i32(list(range(B))),
+                               prefill_q_start=self.i32([i * n for i in range(B + 1)]), tile_req=self.i32(tr or [0]),
+                               tile_q0=self.i32(tq or [0]), num_decodes=B if n == 1 else 0, num_prefills=0 if n == 1 else B, num_tiles=len(tr))
+        what = f"{B} x {n} prompt" if n > 1 else f"decode {B}"
+
+        def buffers(s):
+            a, b = O.workspace_values(s, T)
+            return {"o": self.rnd(T, s.inner, **f32), "states": torch.empty(a, device=self.dev), "decays": torch.empty(b, device=self.dev)}
+        # (a chunk of 64: products with the state, pairs of tokens, their products with v, the update)
+        flops = lambda s: T * s.H * (4.0 * s.D * s.V + 64.0 * (s.D + s.V)) if n > 1 else 0.0                # noqa: E731
+        s = O.OuterShape(H=H, G=H, dim=128, vdim=128, rank=16)
+        proj = self.rnd(T, 4 * H * 128 + 16)
+        parts = torch.split(proj, [H * 128] * 4 + [16], 1)
+        w = {"a2": self.rnd(H * 128, 16, s=0.25), "a2_bias": self.rnd(H * 128, **f32), "norm": self.rnd(128, **f32)}
+        state, out, bufs = torch.zeros(B, H, 128, 128, device=self.dev), self.rnd(T, H * 128), buffers(s)
+        self.add(f"linear attention + gated norm, {what}", "kubolorn",
+                 lambda: O.gated_linear_attention(*parts, w, s, state, rows, bufs, out, tau=16.0, eps=1e-6),
+                 nbytes=T * (5 * H * 128 + 16) * 2 + B * H * 128 * 128 * 8, flops=flops(s))
+        m = O.OuterShape(H=self.sh, G=4, dim=128, vdim=64)
+        C = m.inner + 2 * m.G * m.D
+        row, u, z = self.rnd(T, C + m.inner + 64), self.rnd(T, C), self.rnd(T, m.inner)
+        cw, cb, conv = self.rnd(4, C, **f32), self.rnd(C, **f32), self.rnd(B, 3, C)
+        self.add(f"convolution, {what}", "kubolorn", lambda: R.short_conv(row[:, m.inner: m.inner + C], cw, cb, conv, rows, u, act="silu"),
+                 nbytes=(T * 2 + B * 6) * C * 2)
+        wm = {"dt_bias": self.rnd(m.H, **f32), "A": self.rnd(m.H, **f32).abs(), "D": self.rnd(m.H, **f32), "norm": self.rnd(m.inner, **f32)}
+        stm, outm, bufm, dt = torch.zeros(B, m.H, 128, 64, device=self.dev), self.rnd(T, m.inner), buffers(m), row[:, -64:]
+        self.add(f"state space + gated norm, {what}", "kubolorn",
+                 lambda: O.state_space(u, z, dt, wm, m, stm, rows, bufm, outm, parts=4, eps=1e-6),
+                 nbytes=T * (C + 2 * m.inner + m.H) * 2 + B * m.H * 128 * 64 * 8, flops=flops(m))
+        K, D = H, 128                                        # the delta rule
+        CC = 2 * K * D + H * D
+        x, xc, cw2, cst = self.rnd(T, CC), self.rnd(T, CC), self.rnd(CC, 4), self.rnd(B, CC, 3)
+        st2, z2, core = torch.zeros(B, H, D, D, device=self.dev), self.rnd(T, H * D), self.rnd(T, H * D)
+        slots, init, nw = rows.state_slots, self.i32([1] * B), self.rnd(D)
+        A, dtb = self.rnd(H, **f32).abs(), self.rnd(H, **f32)
+        if n == 1:
+            ab = self.rnd(T, 2 * H)
+            self.add(f"convolution, {what}", "qwen3.5", lambda: Q.conv1d_update(x, cw2, cst, slots, xc), nbytes=(T * 2 + B * 6) * CC * 2)
+
+            def theirs():
+                Q.packed_decode(xc, ab[:, :H], ab[:, H:], A, dtb, st2, slots, core.view(T, H, D), K, H)
+                Q.rmsnorm_gated(core, z2, nw, core, heads=H)
+        else:
+            q, k = self.rnd(T, K, D), self.rnd(T, K, D)
+            g, beta = -self.rnd(T, H, **f32).abs(), self.rnd(T, H, **f32).abs()
+            ws, host = Q.GdnWorkspace(self.dev, T, B, H), [i * n for i in range(B + 1)]
+            table = tuple(self.i32(x.tolist()) for x in Q.build_chunk_table(host))
+            self.add(f"convolution, {what}", "qwen3.5", lambda: Q.conv1d_fwd(x, cw2, cst, rows.prefill_q_start, slots, init, xc),
+                     nbytes=(T * 2 + B * 6) * CC * 2)
+
+            def theirs():
+                Q.chunk_scan(q, k, xc, g, beta, st2, host, slots, init, core.view(T, H, D), ws, v_col0=2 * K * D, table=table)
+                Q.rmsnorm_gated(core, z2, nw, core, heads=H)
+        self.add(f"delta rule + gated norm, {what}", "qwen3.5", theirs,
+                 nbytes=T * (2 * K * D + 3 * H * D) * 2 + B * H * D * D * 8, flops=T * H * (6.0 * D * D + 4 * 64 * D) if n > 1 else 0)
+
+    def rest(self, T):
+        from types import SimpleNamespace
+        from .. import ops
+        from ..config import BigramSpec
+        from ..models.backend import GpuBackend
+        from ..ops import conv_norm as N
+        from ..ops import moe as M
+        from ..ops.reference import build_prefill_tiles
+        W, f32, be = self.W, dict(dtype=torch.float32), GpuBackend()
+        B, n = (T, 1) if T <= 64 else (4, T // 4)
+        tr, tq = build_prefill_tiles([n] * B) if n > 1 else ([], [])
+        rows = SimpleNamespace(seq_lens=self.i32([n + 5] * B), state_slots=self.i32(list(range(B))),
+                               prefill_q_start=self.i32([i * n for i in range(B + 1)]), tile_req=self.i32(tr or [0]),
+                               tile_q0=self.i32(tq or [0]), num_decodes=B if n == 1 else 0, num_prefills=0 if n == 1 else B, num_tiles=len(tr))
+        src, dst, mixed = (self.rnd(T, W, **f32) for _ in range(3))
+        outs, taps = [self.rnd(T, W), self.rnd(T, W)], [self.rnd(4, W, **f32), self.rnd(4, W, **f32)]
+        state = self.rnd(B, 3, W, **f32)
+        norm = dict(width=W, groups=4, eps=1e-6)
+        o2, res, nwb = self.rnd(T, W), self.rnd(T, W), self.rnd(W)
+        what = f"residual + norm, {T} tokens"
+        self.add(what, "kubolorn", lambda: N.norm_conv(src, rows, taps, outs, state=state, dst=dst, a=mixed, **norm),
+                 nbytes=T * W * (4 + 4 + 4 + 4) + B * W * 24, note="two convolutions more")
+        self.add(what, "qwen3.5", lambda: ops.rmsnorm(o2, nwb, 1e-6, residual=res, out=outs[0]), nbytes=T * W * 2 * 4)
+        ids, table, big = torch.randint(0, 32000, (T,), device=self.dev), self.rnd(32000, W), self.rnd(32750, W)
+        prev, nw = torch.zeros(B, dtype=torch.int64, device=self.dev), self.rnd(W, **f32)
+        self.add(f"embedding, {T} tokens", "kubolorn",
+                 lambda: N.embed_pairs(src, ids, table, rows, scale=1.0, norm_w=nw, bigram=big, prev=prev, spec=BigramSpec(32749, 31337, 7919),
+                                       **norm), nbytes=T * W * 8, note="token pairs and norm")
+        self.add(f"embedding, {T} tokens", "qwen3.5", lambda: ops.embedding(ids, table, out=o2), nbytes=T * W * 4)
+        x = self.rnd(T, W)
+        if not self.E:
+            ff, fg = self.ff, self.ff * 2 // 3 // 128 * 128
+            up, cat, gu = self.rnd(ff, W, s=0.05), self.rnd(T, ff + W), self.rnd(2 * fg, W, s=0.05)
+            act, scratch = self.rnd(T, fg), self.rnd(T, 2 * fg)
+            what = f"feed-forward, first product, {T} tokens"
+            self.add(what, "kubolorn", lambda: be.plain_unit(x, up, "gelu_tanh", cat[:, W:]), nbytes=(ff * W + T * (W + ff)) * 2, flops=2.0 * T * ff * W)
+            self.add(what, "qwen3.5", lambda: be.gated_unit(x, gu, 0, act, scratch), nbytes=(2 * fg * W + T * (W + fg)) * 2, flops=2.0 * T * 2 * fg * W)
+            wo, out = self.rnd(W, ff + W, s=0.05), self.rnd(T, W, **f32)
+            what = f"feed-forward, second product, {T} tokens"
+            self.add(what, "kubolorn", lambda: be.gemm(cat, wo, out=out, out_dtype=torch.float32), nbytes=((ff + W) * W + T * (W + ff)) * 2 + T * W * 4,
+                     flops=2.0 * T * (ff + W) * W, note="with the mixer's, fp32")
+            wd = self.rnd(W, fg, s=0.05)
+            self.add(what, "qwen3.5", lambda: be.gemm(act, wd, out=o2), nbytes=(fg * W + T * (W + fg)) * 2, flops=2.0 * T * fg * W)
+            return
+        E, top, ff = self.E, self.top, self.ff
+        P, fp = T * top, ff * 3 // 2
+        ws, wg = M.MoeWorkspace(self.dev, T, top, E, W, fp), M.MoeWorkspace(self.dev, T, top, E, W, ff)
+        ids, w = M.router_topk(self.rnd(T, E, **f32), top)
+        used, chunks = int(ids.unique().numel()), min(ws.max_chunks, E + (P + 255) // 256)
+        wu, wd, wgu, wgd = self.rnd(E, fp, W, s=0.05), self.rnd(E, W, fp, s=0.05), self.rnd(E, 2 * ff, W, s=0.05), self.rnd(E, W, ff, s=0.05)
+        for z in (ws, wg):
+            M.moe_sort(ids, 0, E, z)
+            M.moe_gather(x, z, E, P)
+        args = (M.ptr(ws.chunk_expert), M.ptr(ws.chunk_row0), M.ptr(ws.chunk_n), M.ptr(ws.meta), chunks, M.PLAIN["relu2"], M.stream_ptr())
+        what = f"experts, first products, {T} tokens"
+        self.add(what, "kubolorn", lambda: M.check(M.lib().b200_moe_grouped_gemm_act(M.ptr(ws.xs), P, M.ptr(wu), E, fp, W, M.ptr(ws.act), *args), "gemm"),
+                 nbytes=(used * fp * W + P * (W + fp)) * 2, flops=2.0 * P * fp * W)
+        self.add(what, "qwen3.5", lambda: M.grouped_gemm_gated(wg.xs, wgu, wg.act, wg, P, chunks), nbytes=(used * 2 * ff * W + P * (W + ff)) * 2,
+                 flops=2.0 * P * 2 * ff * W)
+        what = f"experts, second products, {T} tokens"
+        self.add(what, "kubolorn", lambda: M.grouped_gemm(ws.act, wd, ws.y, ws, P, chunks), nbytes=(used * fp * W + P * (W + fp)) * 2,
+                 flops=2.0 * P * fp * W)
+        self.add(what, "qwen3.5", lambda: M.grouped_gemm(wg.act, wgd, wg.y, wg, P, chunks), nbytes=(used * ff * W + P * (W + ff)) * 2,
+                 flops=2.0 * P * ff * W)
+        pos = ws.pair_pos[:P].view(T, top)
+        what = f"expert sum + residual + norm, {T} tokens"
+        self.add(what, "kubolorn", lambda: N.norm_conv(src, rows, taps, outs, state=state, dst=dst, a=mixed, y=ws.y, pair_pos=pos, pair_w=w, **norm),
+                 nbytes=T * W * (4 + 4 + 4 + 4 + 2 * top) + B * W * 24, note="two convolutions more")
+
+        def two():
+            M.combine(wg.y, wg, w, o2)
+            ops.rmsnorm(o2, nwb, 1e-6, residual=res, out=outs[0])
+        self.add(what, "qwen3.5", two, nbytes=T * W * 2 * (top + 1 + 1 + 2 + 1), note="two kernels")
+
+
 DESIGNS = {"nufusun": (NUFUSUN_SIZES, nufusun_configs, NufusunKernels), "diforax": (DIFORAX_SIZES, diforax_configs, DiforaxKernels),
-           "tabupel": (TABUPEL_SIZES, tabupel_configs, TabupelKernels)}
+           "tabupel": (TABUPEL_SIZES, tabupel_configs, TabupelKernels),
+           "kubolorn": (KUBOLORN_SIZES, kubolorn_configs, KubolornKernels)}
 
 
 def run(design="nufusun", sizes=None, kernels=True) -> dict:
@@ -713,7 +945,7 @@ def run(design="nufusun", sizes=None, kernels=True) -> dict:
     res = {"metric": "design_layer_throughput", "unit": "tok/s", "impl": "ours", "design": design, "dtype": "bf16",
            "data": "synthetic (uniform-random prompt ids, random-init weights)",
            "roofline": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": how}, "models": {}, "kernels": {}}
-    names = TABUPEL_FIELDS if design == "tabupel" else FIELDS + (("delta_heads", "delta_key_heads") if design == "diforax" else ())
+    names = TABUPEL_FIELDS if design == "tabupel" else KUBOLORN_FIELDS if design == "kubolorn" else FIELDS + (("delta_heads", "delta_key_heads") if design == "diforax" else ())
     for name, size in table.items():
         if sizes and name not in sizes:
             continue
