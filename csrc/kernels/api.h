@@ -304,6 +304,8 @@ typedef struct B200Outer {
   long long lddt;
   float* state;
   float* o;                    // [T][H * V], before norm and gate
+  void* pairs;                 // workspace of the chunk kernels (b200_outer_workspace values per chunk and state)
+  float* factors;
   float* ws;                   // [segments][H][D][V], [segments][H][D]: portions cut in segments
   float* ws_decay;
   const void* gate;            // [T][H * V]
@@ -468,6 +470,7 @@ int b200_outer_step(const B200Outer* a, int reqs, cudaStream_t stream);
 int b200_outer_norm(const B200Outer* a, int reqs, int chunks, cudaStream_t stream);
 // ---- outer_chunk.cu
 int b200_outer_fits(const B200Outer* a);
+void b200_outer_workspace(int kind, int D, int* values);
 int b200_outer_chunk(const B200Outer* a, cudaStream_t stream);
 // ---- gdn.cu
 int b200_gdn_conv1d_fwd(const void* x, long ldx, const void* w, void* conv_state, const int* qsl, const int* slots, const int* has_init, void* out, long ldo, int n_seq, int total_tokens, int C, cudaStream_t stream);

@@ -92,7 +92,15 @@ __global__ void __launch_bounds__(256) embed_pairs_kernel(B200EmbedPairs p, int*
   float* part = row_smem + p.cols;               // [groups][warps], then [groups]
   for (int g = 0; g < p.groups; ++g) {
     float ss = 0.f;
-    for (int i = tid; i < gs; i += blockDim.x) ss = fmaf(row_smem[g * gs + i], row_smem[g * gs + i], ss);
+    if (!(gs & 3))
+      for (int i = tid * 4; i < gs; i += blockDim.x * 4) {
+        float v[4];
+        Vals<float, 4>::get(row_smem + g * gs + i, v);
+#pragma unroll
+        for (int x = 0; x < 4; ++x) ss = fmaf(v[x], v[x], ss);
+      }
+    else
+      for (int i = tid; i < gs; i += blockDim.x) ss = fmaf(row_smem[g * gs + i], row_smem[g * gs + i], ss);
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     if (lane == 0) part[g * nw + warp] = ss;
@@ -106,6 +114,20 @@ __global__ void __launch_bounds__(256) embed_pairs_kernel(B200EmbedPairs p, int*
   }
   __syncthreads();
   float* out = p.stream + (size_t)t * p.lds;
+  if (!(gs & 3)) {
+    for (int i = tid * 4; i < p.cols; i += blockDim.x * 4) {
+      float v[4] = {0.f, 0.f, 0.f, 0.f}, w[4];
+      if (i < p.width) {
+        const float f = inv[i / gs];
+        Vals<float, 4>::get(row_smem + i, v);
+        Vals<float, 4>::get(p.norm_w + i, w);
+#pragma unroll
+        for (int x = 0; x < 4; ++x) v[x] *= f * w[x];
+      }
+      Vals<float, 4>::put(out + i, v);
+    }
+    return;
+  }
   for (int i = tid; i < p.cols; i += blockDim.x) out[i] = i < p.width ? row_smem[i] * inv[i / gs] * p.norm_w[i] : 0.f;
 }
 
@@ -152,12 +174,13 @@ __global__ void __launch_bounds__(512) norm_conv_kernel(B200NormConv p) {
   auto normed = [&](int pos, int count, bool keep, float (&x)[kBatch][NV][VEC]) {
     if (p.k > 0) {
       __syncthreads();                           // (the last batch's pairs have been read)
-      for (int i = tid; i < count * p.k; i += nt) {
-        const int r = i / p.k, j = i - r * p.k;
-        const size_t pair = (size_t)(first + pos + r) * p.k + j;
+      const int k4 = (p.k + 3) & ~3;             // (entries without an output: weight 0, and some row that is there)
+      for (int i = tid; i < count * k4; i += nt) {
+        const int r = i / k4, j = i - r * k4;
+        const size_t pair = (size_t)(first + pos + r) * p.k + min(j, p.k - 1);
         const int32_t y = reinterpret_cast<const int32_t*>(p.pair_pos)[pair];
-        s_y[r][j] = y >= 0 ? reinterpret_cast<const T*>(p.y) + (size_t)y * p.ldy : nullptr;
-        s_w[r][j] = p.pair_w[pair];
+        s_y[r][j] = reinterpret_cast<const T*>(p.y) + (size_t)max(y, 0) * p.ldy;
+        s_w[r][j] = y >= 0 && j < p.k ? p.pair_w[pair] : 0.f;
       }
       __syncthreads();
     }
@@ -181,20 +204,29 @@ __global__ void __launch_bounds__(512) norm_conv_kernel(B200NormConv p) {
             for (int e = 0; e < VEC; ++e) x[r][c][e] += a[e];
           }
     }
-    for (int j = 0; j < p.k; ++j)
+    // (the loads of four pairs of every row are on the way at a time)
+    constexpr int kAhead = NV * VEC <= 4 ? 4 : 1;
+    for (int j0 = 0; j0 < p.k; j0 += kAhead) {
+      float y[kAhead][kBatch][NV][VEC];
 #pragma unroll
-      for (int r = 0; r < kBatch; ++r)
-        if (r < count && s_y[r][j]) {
-          const float w = s_w[r][j];
+      for (int j = 0; j < kAhead; ++j)
+#pragma unroll
+        for (int r = 0; r < kBatch; ++r)
 #pragma unroll
           for (int c = 0; c < NV; ++c)
-            if (on[c]) {
-              float y[VEC];
-              Vals<T, VEC>::get(s_y[r][j] + col[c], y);
+            if (r < count && on[c]) Vals<T, VEC>::get(s_y[r][j0 + j] + col[c], y[j][r][c]);
 #pragma unroll
-              for (int e = 0; e < VEC; ++e) x[r][c][e] = fmaf(w, y[e], x[r][c][e]);
+      for (int j = 0; j < kAhead; ++j)
+#pragma unroll
+        for (int r = 0; r < kBatch; ++r)
+#pragma unroll
+          for (int c = 0; c < NV; ++c)
+            if (r < count && on[c]) {
+              const float w = s_w[r][j0 + j];
+#pragma unroll
+              for (int e = 0; e < VEC; ++e) x[r][c][e] = fmaf(w, y[j][r][c][e], x[r][c][e]);
             }
-        }
+    }
 #pragma unroll
     for (int r = 0; r < kBatch; ++r) {
       float ss = 0.f;

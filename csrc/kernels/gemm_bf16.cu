@@ -418,10 +418,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
               }
             }
           }
-          if (p.act) {
-#pragma unroll
-            for (int i = 0; i < 32; ++i) v[i] = act_epilogue(v[i], p.act);
-          }
+          act_epilogue<true>(v, p.act);
           if (p.tp_world > 1 && p.peer_recv[0]) {
             const int owner = row / p.rows_per_rank;
             const uint32_t par = *p.op_counter & 1;
@@ -527,10 +524,7 @@ __device__ __forceinline__ void epilogue_store_chunk(const GemmParams& p, float 
       }
     }
   }
-  if (p.act) {
-#pragma unroll
-    for (int i = 0; i < 32; ++i) v[i] = act_epilogue(v[i], p.act);
-  }
+  act_epilogue<true>(v, p.act);
   if (p.out_f32) {
     float* o = reinterpret_cast<float*>(p.out) + (size_t)row * p.ldo + col0;
 #pragma unroll
@@ -1042,7 +1036,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
               } else {
                 v += bias_v;
                 if (p.residual) v += __bfloat162float(p.residual[(size_t)m * p.ldr + n]);
-                v = act_epilogue(v, p.act);
+                v = act_epilogue<true>(v, p.act);
                 const size_t o = (size_t)bz * p.batch_out_stride + (size_t)m * p.ldo + n;
                 if (p.out_f32)
                   reinterpret_cast<float*>(p.out)[o] = v;
@@ -1102,8 +1096,8 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ ws, int splits, i
       acc.x += f0.x; acc.y += f0.y; acc.z += f1.x; acc.w += f1.y;
     }
     if (act) {
-      acc.x = act_epilogue(acc.x, act); acc.y = act_epilogue(acc.y, act);
-      acc.z = act_epilogue(acc.z, act); acc.w = act_epilogue(acc.w, act);
+      acc.x = act_epilogue<true>(acc.x, act); acc.y = act_epilogue<true>(acc.y, act);
+      acc.z = act_epilogue<true>(acc.z, act); acc.w = act_epilogue<true>(acc.w, act);
     }
     if (out_f32) {
       *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + (size_t)m * ldo + n) = acc;

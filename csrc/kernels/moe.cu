@@ -420,11 +420,15 @@ __global__ void __launch_bounds__(192, 1)
         tmem_ld_32x32b_x16(ta + c * 16, r);
         tmem_ld_wait();
         if (n < p.N) {
+          float v[16];
+#pragma unroll
+          for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]);
+          act_epilogue<true>(v, p.act);
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
             const int m = c * 16 + i;
             if (m < rows)
-              p.out[(size_t)(row0 + m) * p.N + n] = __float2bfloat16(act_epilogue(__uint_as_float(r[i]), p.act));
+              p.out[(size_t)(row0 + m) * p.N + n] = __float2bfloat16(v[i]);
           }
         }
       }

@@ -512,13 +512,34 @@ inline cudaError_t launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, s
   return cudaLaunchKernelEx(&cfg, kernel, KArgs(static_cast<Args&&>(args))...);
 }
 #endif
-// Activations in the epilogue of a product: 0 none, 1 SiLU, 2 GELU-tanh, 3 GELU-erf, 4 squared ReLU.
+// Activations in the epilogue of a product: 0 none, 1 SiLU, 2 GELU-tanh, 3 GELU-erf, 4 squared ReLU. FAST (results that are
+// rounded to bf16): 0.5 (1 + tanh u) = 1 / (1 + e^(-2 u)) with the approximate exponential and quotient.
+template <bool FAST>
 __device__ __forceinline__ float act_epilogue(float x, int act) {
   if (act == 4) { x = fmaxf(x, 0.f); return x * x; }
-  if (act == 2) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
-  if (act == 1) return x / (1.f + expf(-x));
+  if (act == 2) {
+    const float u = 0.7978845608028654f * (x + 0.044715f * x * x * x);
+    return FAST ? __fdividef(x, 1.f + __expf(-2.f * u)) : 0.5f * x * (1.f + tanhf(u));
+  }
+  if (act == 1) return FAST ? __fdividef(x, 1.f + __expf(-x)) : x / (1.f + expf(-x));
   if (act == 3) return 0.5f * x * (1.f + erff(x * 0.7071067811865476f));
   return x;
+}
+template <bool FAST, int N>
+__device__ __forceinline__ void act_epilogue(float (&v)[N], int act) {
+  if (act == 2) {                                // (one loop per activation, so that none tests which it is)
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = act_epilogue<FAST>(v[i], 2);
+  } else if (act == 4) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = act_epilogue<FAST>(v[i], 4);
+  } else if (act == 1) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = act_epilogue<FAST>(v[i], 1);
+  } else if (act == 3) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = act_epilogue<FAST>(v[i], 3);
+  }
 }
 
 }  // namespace b200

@@ -236,7 +236,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(F32Gemm p) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < p.N) out[(size_t)(row_base + m) * p.ldo + n] = act_epilogue(acc[i][j] + (p.bias ? p.bias[n] : 0.f), p.act);
+      if (n < p.N) out[(size_t)(row_base + m) * p.ldo + n] = act_epilogue<false>(acc[i][j] + (p.bias ? p.bias[n] : 0.f), p.act);
     }
   }
 }

@@ -106,9 +106,10 @@ class Engine:
                                                                          ("gate", H, V, s.V)))
         nan = float("nan")
         out = torch.full((T, s.inner), nan, dtype=dtype, device=DEV)
-        tiles = len(tr) + 2
-        bufs = {"o": torch.full((T, s.inner), nan, device=DEV), "states": torch.full((2 * tiles * H * s.D * s.V,), nan, device=DEV),
-                "decays": torch.full((2 * tiles * H * s.D,), nan, device=DEV)}
+        work = O.Workspace(DEV, T, len(items))
+        work.segments = 2 * (len(tr) + 2)                                          # (tests cut portions finer than the model does)
+        work.reserve(s, O.CHANNEL if kind == "channel" else O.HEAD)
+        bufs = {"o": torch.full((T, s.inner), nan, device=DEV), **{k: t.fill_(nan) for k, t in work.allocate().items()}}
         if kind == "channel":
             a1 = self.spread(cat("a1"), 1, x, s.rank)
             row = torch.cat([q, k, v, gate, a1], 1).to(dtype).to(DEV)

@@ -808,16 +808,17 @@ class KubolornKernels(KernelBench):
                                tile_q0=self.i32(tq or [0]), num_decodes=B if n == 1 else 0, num_prefills=0 if n == 1 else B, num_tiles=len(tr))
         what = f"{B} x {n} prompt" if n > 1 else f"decode {B}"
 
-        def buffers(s):
-            a, b = O.workspace_values(s, T)
-            return {"o": self.rnd(T, s.inner, **f32), "states": torch.empty(a, device=self.dev), "decays": torch.empty(b, device=self.dev)}
+        def buffers(s, kind):
+            work = O.Workspace(self.dev, T, B)
+            work.reserve(s, kind)
+            return {"o": self.rnd(T, s.inner, **f32), **work.allocate()}
         # (a chunk of 64: products with the state, pairs of tokens, their products with v, the update)
         flops = lambda s: T * s.H * (4.0 * s.D * s.V + 64.0 * (s.D + s.V)) if n > 1 else 0.0                # noqa: E731
         s = O.OuterShape(H=H, G=H, dim=128, vdim=128, rank=16)
         proj = self.rnd(T, 4 * H * 128 + 16)
         parts = torch.split(proj, [H * 128] * 4 + [16], 1)
         w = {"a2": self.rnd(H * 128, 16, s=0.25), "a2_bias": self.rnd(H * 128, **f32), "norm": self.rnd(128, **f32)}
-        state, out, bufs = torch.zeros(B, H, 128, 128, device=self.dev), self.rnd(T, H * 128), buffers(s)
+        state, out, bufs = torch.zeros(B, H, 128, 128, device=self.dev), self.rnd(T, H * 128), buffers(s, O.CHANNEL)
         self.add(f"linear attention + gated norm, {what}", "kubolorn",
                  lambda: O.gated_linear_attention(*parts, w, s, state, rows, bufs, out, tau=16.0, eps=1e-6),
                  nbytes=T * (5 * H * 128 + 16) * 2 + B * H * 128 * 128 * 8, flops=flops(s))
@@ -828,7 +829,7 @@ class KubolornKernels(KernelBench):
         self.add(f"convolution, {what}", "kubolorn", lambda: R.short_conv(row[:, m.inner: m.inner + C], cw, cb, conv, rows, u, act="silu"),
                  nbytes=(T * 2 + B * 6) * C * 2)
         wm = {"dt_bias": self.rnd(m.H, **f32), "A": self.rnd(m.H, **f32).abs(), "D": self.rnd(m.H, **f32), "norm": self.rnd(m.inner, **f32)}
-        stm, outm, bufm, dt = torch.zeros(B, m.H, 128, 64, device=self.dev), self.rnd(T, m.inner), buffers(m), row[:, -64:]
+        stm, outm, bufm, dt = torch.zeros(B, m.H, 128, 64, device=self.dev), self.rnd(T, m.inner), buffers(m, O.HEAD), row[:, -64:]
         self.add(f"state space + gated norm, {what}", "kubolorn",
                  lambda: O.state_space(u, z, dt, wm, m, stm, rows, bufm, outm, parts=4, eps=1e-6),
                  nbytes=T * (C + 2 * m.inner + m.H) * 2 + B * m.H * 128 * 64 * 8, flops=flops(m))

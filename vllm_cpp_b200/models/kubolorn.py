@@ -23,7 +23,7 @@ import torch
 from ..config import DenseSpec, ExpertSpec
 from ..ops.bias_attn import TiedShape, grouped_decode_splits
 from ..ops.conv_norm import conv_weights
-from ..ops.outer import OuterShape, workspace_values
+from ..ops.outer import CHANNEL, HEAD, OuterShape, Workspace
 from .base import StepContext
 from .listed import ListedModel, pad, pad_heads, padded
 from .recurrent import RecurrentState
@@ -283,7 +283,7 @@ class KubolornModel(ListedModel):
             self.bufs.reserve(n, max_tokens, self.cols, t)
         self.recurrent = RecurrentState()
         self.prev = self.recurrent.add((max_reqs,), torch.int64, self.device) if self.cfg.bigram is not None else None
-        states = decays = 0
+        work = Workspace(self.device, max_tokens, max_reqs) if self._bf16_kernels() else None
         for l, b in enumerate(self.cfg.blocks):
             L, f = self.layers[l], b.mlp
             s = L["shape"]
@@ -297,17 +297,16 @@ class KubolornModel(ListedModel):
                 rows = self.recurrent.add((max_reqs, self.cfg.input_conv - 1, self.cols), torch.float32, self.device)
             self.state[l] = (rows, self.recurrent.add((max_reqs, *conv), self.dtype, self.device) if conv else None,
                              self.recurrent.add((max_reqs, *state), torch.float32, self.device))
-            n, d = workspace_values(s, max_tokens)
-            states, decays = max(states, n), max(decays, d)
+            if work is not None:
+                work.reserve(s, CHANNEL if b.gla is not None else HEAD)
             if isinstance(f, ExpertSpec):
                 n, key = pad(f.experts), (f.experts, f.top, f.ff)
                 self.bufs.reserve(f"router{n}", max_tokens, n, torch.float32)
                 if self.device.type == "cuda" and key not in self.moe_ws:
                     from ..ops.moe import MoeWorkspace
                     self.moe_ws[key] = MoeWorkspace(self.device, max_tokens, f.top, f.experts, self.cols, pad(f.ff), self.dtype)
-        if self._bf16_kernels():
-            self.scratch = {"states": torch.empty(states, dtype=torch.float32, device=self.device),
-                            "decays": torch.empty(decays, dtype=torch.float32, device=self.device)}
+        if work is not None:
+            self.scratch = work.allocate()
 
     # ------------------------------------------------------------------ forward
     def _gla(self, h, l, L, g, ctx, T, proj, out):

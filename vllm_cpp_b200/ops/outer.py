@@ -45,7 +45,7 @@ class OuterArgs(ctypes.Structure):
     _fields_ = [("rows", RowArgs), ("q", _P), ("k", _P), ("v", _P), ("ld", _L),
                 ("a1", _P), ("a2", _P), ("a2b", _P), ("lda1", _L),
                 ("dt", _P), ("dt_bias", _P), ("A", _P), ("lddt", _L),
-                ("state", _P), ("o", _P), ("ws", _P), ("ws_decay", _P), ("gate", _P), ("ldg", _L), ("norm_w", _P), ("skip", _P),
+                ("state", _P), ("o", _P), ("pairs", _P), ("factors", _P), ("ws", _P), ("ws_decay", _P), ("gate", _P), ("ldg", _L), ("norm_w", _P), ("skip", _P),
                 ("out", _P), ("ldo", _L),
                 ("kind", _I), ("H", _I), ("G", _I), ("D", _I), ("V", _I), ("dim", _I), ("vdim", _I), ("rank", _I), ("f32", _I),
                 ("parts", _I), ("seg_tiles", _I), ("multi", _I), ("q_scale", _F), ("inv_tau", _F), ("eps", _F), ("out_scale", _F)]
@@ -60,6 +60,7 @@ def _declare():
         return
     A = ctypes.POINTER(OuterArgs)
     _lib.declare("b200_outer_fits", [A], _I)
+    _lib.declare("b200_outer_workspace", [_I, _I, ctypes.POINTER(_I)], None)
     _lib.declare("b200_outer_step", [A, _I, _P], _I)
     _lib.declare("b200_outer_chunk", [A, _P], _I)
     _lib.declare("b200_outer_norm", [A, _I, _I, _P], _I)
@@ -83,11 +84,29 @@ def segment_tiles(num_tiles: int, portions: int, ctas: int, num_sms: int) -> int
     return max(MIN_SEGMENT, -(-per // cuts))
 
 
-def workspace_values(s: OuterShape, max_tokens: int) -> tuple[int, int]:
-    """fp32 values of (states, decays) of the cut portions of a step."""
-    # (a cut portion has 2 MIN_SEGMENT tiles at least, the last of them partly filled)
-    segments = 2 * (max_tokens * 8 // (7 * 128 * MIN_SEGMENT) + 2)
-    return segments * s.H * s.D * s.V, segments * s.H * s.D
+class Workspace:
+    """Scratch of the chunk kernels for steps of up to ``max_tokens`` rows in ``max_portions`` portions; it serves every shape
+    that :meth:`reserve` has seen."""
+
+    def __init__(self, device, max_tokens: int, max_portions: int):
+        self.device, self.chunks = device, max_tokens // 64 + max_portions
+        # (a cut portion has 2 MIN_SEGMENT tiles at least, the last of them partly filled)
+        self.segments = 2 * (max_tokens * 8 // (7 * 128 * MIN_SEGMENT) + 2)
+        self.sizes = [0, 0, 0, 0]
+        self.buffers: dict = {}
+
+    def reserve(self, s: OuterShape, kind: int) -> None:
+        _declare()
+        v = (_I * 2)()
+        lib().b200_outer_workspace(kind, s.D, v)
+        need = (self.chunks * s.H * v[0], self.chunks * s.H * v[1], self.segments * s.H * s.D * s.V, self.segments * s.H * s.D)
+        self.sizes = [max(a, b) for a, b in zip(self.sizes, need)]
+
+    def allocate(self) -> dict:
+        f32 = torch.float32
+        self.buffers = {n: torch.empty(z, dtype=t, device=self.device) for n, z, t in
+                        zip(("pairs", "factors", "states", "decays"), self.sizes, (torch.bfloat16, f32, f32, f32))}
+        return self.buffers
 
 
 def outer_args(s: OuterShape, q, k, v, state, ctx, bufs, out, *, eps, q_scale=1.0, out_scale=1.0, channel=None, head=None, gate=None,
@@ -105,6 +124,7 @@ def outer_args(s: OuterShape, q, k, v, state, ctx, bufs, out, *, eps, q_scale=1.
         dt, bias, A = head
         a.kind, a.dt, a.lddt, a.dt_bias, a.A = HEAD, ptr(dt), dt.stride(0), ptr(bias), ptr(A)
     a.state, a.o, a.ws, a.ws_decay = ptr(state), ptr(bufs["o"]), ptr(bufs.get("states")), ptr(bufs.get("decays"))
+    a.pairs, a.factors = ptr(bufs.get("pairs")), ptr(bufs.get("factors"))
     a.gate, a.ldg, a.norm_w, a.skip = ptr(gate), gate.stride(0), ptr(norm_w), ptr(skip)
     a.out, a.ldo = ptr(out), out.stride(0)
     a.H, a.G, a.D, a.V, a.dim, a.vdim, a.rank = s.H, s.G, s.D, s.V, s.dim, s.vdim, s.rank
@@ -126,6 +146,10 @@ def run(a: OuterArgs, ctx, bufs, *, token_by_token=False, seg_tiles=None) -> Non
         if a.multi:
             most = 2 * (a.rows.num_tiles // seg_tiles + 1)
             assert bufs["states"].numel() >= most * a.H * a.D * a.V and bufs["decays"].numel() >= most * a.H * a.D
+        v = (_I * 2)()
+        lib().b200_outer_workspace(a.kind, a.D, v)
+        most = a.H * ((a.rows.T - a.rows.nd) // 64 + a.rows.num_prefills)
+        assert bufs["pairs"].numel() >= most * v[0] and bufs["factors"].numel() >= most * v[1]
         check(lib().b200_outer_chunk(ctypes.byref(a), stream_ptr()), "outer_chunk")
     # (decode rows of the channel kind are normed by the step kernel where it holds whole heads)
     check(lib().b200_outer_norm(ctypes.byref(a), reqs, int(chunks), stream_ptr()), "outer_norm")
@@ -136,7 +160,7 @@ def gated_linear_attention(q, k, v, gate, a1, w, s: OuterShape, state, ctx, bufs
     """``q`` / ``k`` [T, H * D], ``v`` / ``gate`` [T, H * V], ``a1`` [T, rank] (columns of one projection) -> ``out`` [T, H * V].
     The state fades per key channel by sigmoid(a2 a1 + bias)^(1 / tau), ``w``: a2 [H * D, rank], a2_bias fp32 [H * D],
     norm fp32 [V]. ``state`` fp32 [slots, H, D, V] is advanced; a request's first rows start from zero. ``bufs``: o fp32
-    [T, H * V], and for prompts states / decays (see :func:`workspace_values`). bf16 prompts run in chunks of 64 tokens
+    [T, H * V], and for prompts the buffers of a :class:`Workspace`. bf16 prompts run in chunks of 64 tokens
     on the tensor cores; ``token_by_token``, fp32 and sizes beyond them walk the tokens."""
     a = outer_args(s, q, k, v, state, ctx, bufs, out, eps=eps, q_scale=s.dim ** -0.5, channel=(a1, w["a2"], w["a2_bias"], tau),
                    gate=gate, norm_w=w["norm"])
