@@ -16,27 +16,36 @@ typedef __nv_bfloat16 bf16;
 static constexpr int kRun = 16;          // rows of a portion that one CTA walks
 static constexpr int kBatch = 4;         // rows on the way at a time
 static constexpr int kPairs = 64;        // expert outputs per row
+static constexpr int kAhead = 4;         // of a row on the way at a time
 
+// VEC values in memory (Raw) and as floats
 template <typename T, int VEC> struct Vals;
 template <> struct Vals<float, 4> {
+  typedef float4 Raw;
+  static __device__ __forceinline__ void open(Raw r, float* v) { *reinterpret_cast<float4*>(v) = r; }
   static __device__ __forceinline__ void get(const float* p, float* v) { *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p); }
   static __device__ __forceinline__ void put(float* p, const float* v) { *reinterpret_cast<float4*>(p) = *reinterpret_cast<const float4*>(v); }
 };
 template <> struct Vals<bf16, 4> {
-  static __device__ __forceinline__ void get(const bf16* p, float* v) {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
+  typedef uint2 Raw;
+  static __device__ __forceinline__ void open(Raw u, float* v) {
     const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
     v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
   }
+  static __device__ __forceinline__ void get(const bf16* p, float* v) { open(*reinterpret_cast<const uint2*>(p), v); }
   static __device__ __forceinline__ void put(bf16* p, const float* v) {
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
   }
 };
 template <> struct Vals<float, 1> {
+  typedef float Raw;
+  static __device__ __forceinline__ void open(Raw r, float* v) { *v = r; }
   static __device__ __forceinline__ void get(const float* p, float* v) { *v = *p; }
   static __device__ __forceinline__ void put(float* p, const float* v) { *p = *v; }
 };
 template <> struct Vals<bf16, 1> {
+  typedef bf16 Raw;
+  static __device__ __forceinline__ void open(Raw r, float* v) { *v = __bfloat162float(r); }
   static __device__ __forceinline__ void get(const bf16* p, float* v) { *v = __bfloat162float(*p); }
   static __device__ __forceinline__ void put(bf16* p, const float* v) { *p = __float2bfloat16(*v); }
 };
@@ -133,13 +142,11 @@ __global__ void __launch_bounds__(256) embed_pairs_kernel(B200EmbedPairs p, int*
 
 // ------------------------------------------------------------------- update, norm, convolutions
 // grid (runs, parts). VEC consecutive values a thread at a time, NV of those; TAPS 0: any number, carried rows of the run in
-// shared memory and taps read from memory.
-template <typename T, int VEC, int NV, int TAPS>
-__global__ void __launch_bounds__(512) norm_conv_kernel(B200NormConv p) {
-  extern __shared__ float hist_smem[];           // TAPS 0: [taps - 1][NV][threads][VEC]
+// shared memory and taps read from memory. PAIRS: with expert outputs. MT: most threads.
+template <typename T, int VEC, int NV, int TAPS, bool PAIRS, int MT>
+__global__ void __launch_bounds__(MT, MT > 128 ? 1 : PAIRS ? 4 : 5) norm_conv_kernel(B200NormConv p) {
+  extern __shared__ float4 nc_smem[];            // PAIRS: [rows][pairs] rows of y, weights; TAPS 0: [taps - 1][NV][threads][VEC]
   __shared__ float red[kBatch][16];
-  __shared__ const T* s_y[kBatch][kPairs];
-  __shared__ float s_w[kBatch][kPairs];
   pdl_wait();
   pdl_launch_dependents();
   const int tid = threadIdx.x, nt = blockDim.x, warp = tid >> 5, lane = tid & 31, taps = TAPS ? TAPS : p.taps;
@@ -170,20 +177,24 @@ __global__ void __launch_bounds__(512) norm_conv_kernel(B200NormConv p) {
     on[c] = i < gs;
     col[c] = base + (on[c] ? i : 0);
   }
+  // the expert outputs of every row that this CTA looks at: its run with the taps - 1 rows ahead, and the portion's last taps - 1
+  // (no output: weight 0, and some row that is there)
+  const int k4 = PAIRS ? (p.k + kAhead - 1) / kAhead * kAhead : 0, ahead = at == 0 ? 0 : taps - 1;
+  const int run = ahead + n, tail = at == 0 && len > n ? taps - 1 : 0;
+  int32_t* s_y = reinterpret_cast<int32_t*>(nc_smem);                  // [kRun + 2 (taps - 1)][k4]
+  float* s_w = reinterpret_cast<float*>(s_y + (kRun + 2 * (taps - 1)) * k4);
+  if (PAIRS) {
+    for (int i = tid; i < (run + tail) * k4; i += nt) {
+      const int r = i / k4, j = i - r * k4, pos = r < run ? at - ahead + r : len - tail + (r - run);
+      const size_t pair = (size_t)(first + pos) * p.k + min(j, p.k - 1);
+      const int32_t y = reinterpret_cast<const int32_t*>(p.pair_pos)[pair];
+      s_y[i] = max(y, 0);
+      s_w[i] = y >= 0 && j < p.k ? p.pair_w[pair] : 0.f;
+    }
+    __syncthreads();
+  }
   // Rows pos .. pos + count - 1 of the portion over their rms; those of this run (keep) also go to dst.
   auto normed = [&](int pos, int count, bool keep, float (&x)[kBatch][NV][VEC]) {
-    if (p.k > 0) {
-      __syncthreads();                           // (the last batch's pairs have been read)
-      const int k4 = (p.k + 3) & ~3;             // (entries without an output: weight 0, and some row that is there)
-      for (int i = tid; i < count * k4; i += nt) {
-        const int r = i / k4, j = i - r * k4;
-        const size_t pair = (size_t)(first + pos + r) * p.k + min(j, p.k - 1);
-        const int32_t y = reinterpret_cast<const int32_t*>(p.pair_pos)[pair];
-        s_y[r][j] = reinterpret_cast<const T*>(p.y) + (size_t)max(y, 0) * p.ldy;
-        s_w[r][j] = y >= 0 && j < p.k ? p.pair_w[pair] : 0.f;
-      }
-      __syncthreads();
-    }
 #pragma unroll
     for (int r = 0; r < kBatch; ++r)
 #pragma unroll
@@ -204,28 +215,38 @@ __global__ void __launch_bounds__(512) norm_conv_kernel(B200NormConv p) {
             for (int e = 0; e < VEC; ++e) x[r][c][e] += a[e];
           }
     }
-    // (the loads of four pairs of every row are on the way at a time)
-    constexpr int kAhead = NV * VEC <= 4 ? 4 : 1;
-    for (int j0 = 0; j0 < p.k; j0 += kAhead) {
-      float y[kAhead][kBatch][NV][VEC];
-#pragma unroll
-      for (int j = 0; j < kAhead; ++j)
-#pragma unroll
-        for (int r = 0; r < kBatch; ++r)
-#pragma unroll
-          for (int c = 0; c < NV; ++c)
-            if (r < count && on[c]) Vals<T, VEC>::get(s_y[r][j0 + j] + col[c], y[j][r][c]);
-#pragma unroll
-      for (int j = 0; j < kAhead; ++j)
+    if (PAIRS) {
+      const int e0 = (keep ? pos - (at - ahead) : run + pos - (len - tail)) * k4;
+      const T* y0 = reinterpret_cast<const T*>(p.y);
+      constexpr int AH = NV * VEC <= 4 ? kAhead : 1;
+      for (int j0 = 0; j0 < k4; j0 += AH) {      // (the loads of AH outputs of every row are on the way at a time)
+        typename Vals<T, VEC>::Raw y[AH][kBatch][NV];
 #pragma unroll
         for (int r = 0; r < kBatch; ++r)
+          if (r < count) {
 #pragma unroll
-          for (int c = 0; c < NV; ++c)
-            if (r < count && on[c]) {
-              const float w = s_w[r][j0 + j];
+            for (int j = 0; j < AH; ++j) {
+              const T* from = y0 + (size_t)s_y[e0 + r * k4 + j0 + j] * p.ldy;
 #pragma unroll
-              for (int e = 0; e < VEC; ++e) x[r][c][e] = fmaf(w, y[j][r][c][e], x[r][c][e]);
+              for (int c = 0; c < NV; ++c) y[j][r][c] = *reinterpret_cast<const typename Vals<T, VEC>::Raw*>(from + col[c]);
             }
+          }
+#pragma unroll
+        for (int r = 0; r < kBatch; ++r)
+          if (r < count) {
+#pragma unroll
+            for (int j = 0; j < AH; ++j) {
+              const float w = s_w[e0 + r * k4 + j0 + j];
+#pragma unroll
+              for (int c = 0; c < NV; ++c) {
+                float v[VEC];
+                Vals<T, VEC>::open(y[j][r][c], v);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) x[r][c][e] = on[c] ? fmaf(w, v[e], x[r][c][e]) : 0.f;
+              }
+            }
+          }
+      }
     }
 #pragma unroll
     for (int r = 0; r < kBatch; ++r) {
@@ -265,7 +286,7 @@ __global__ void __launch_bounds__(512) norm_conv_kernel(B200NormConv p) {
         if (p.out2) Vals<float, VEC>::get(p.w2 + (size_t)j * p.cols + col[c], wt[TAPS + j][c]);
       }
   }
-  float* mine = hist_smem + tid * VEC;           // entry j, piece c: mine + (j * NV + c) * nt * VEC
+  float* mine = s_w + (kRun + 2 * (taps - 1)) * k4 + tid * VEC;   // entry j, piece c: mine + (j * NV + c) * nt * VEC
   const int step = nt * VEC;
   auto carried = [&](int i, int c, float* v) {   // entry i of the state
     if (init && on[c]) {
@@ -381,27 +402,35 @@ __global__ void __launch_bounds__(512) norm_conv_kernel(B200NormConv p) {
   }
 }
 
-template <typename T, int VEC, int NV, int TAPS>
+template <typename T, int VEC, int NV, int TAPS, bool PAIRS, int MT>
 static int run_norm_conv(const B200NormConv& a, int threads, cudaStream_t stream) {
   const dim3 grid(a.rows.nd + a.rows.num_tiles * (128 / kRun), a.groups);
-  const size_t smem = TAPS ? 0 : (size_t)(a.taps - 1) * NV * VEC * threads * 4;
+  const size_t k4 = PAIRS ? (a.k + kAhead - 1) / kAhead * kAhead : 0;
+  const size_t smem = (kRun + 2 * (a.taps - 1)) * k4 * 8 + (TAPS ? 0 : (size_t)(a.taps - 1) * NV * VEC * threads * 4);
   if (smem > 160 * 1024) return -4;
   if (!TAPS) {
     static PerDeviceOnce once;
     if (once.first())
-      cudaFuncSetAttribute(norm_conv_kernel<T, VEC, NV, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+      cudaFuncSetAttribute(norm_conv_kernel<T, VEC, NV, TAPS, PAIRS, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
   }
-  return launch_pdl(norm_conv_kernel<T, VEC, NV, TAPS>, grid, dim3(threads), smem, stream, a) == cudaSuccess ? 0 : -2;
+  return launch_pdl(norm_conv_kernel<T, VEC, NV, TAPS, PAIRS, MT>, grid, dim3(threads), smem, stream, a) == cudaSuccess ? 0 : -2;
+}
+template <typename T, int VEC, int NV, int TAPS>
+static int pick_pairs(const B200NormConv& a, int threads, cudaStream_t stream) {
+  if constexpr (TAPS > 0 && NV == 1)
+    if (threads <= 128)
+      return a.k ? run_norm_conv<T, VEC, NV, TAPS, true, 128>(a, threads, stream) : run_norm_conv<T, VEC, NV, TAPS, false, 128>(a, threads, stream);
+  return a.k ? run_norm_conv<T, VEC, NV, TAPS, true, 512>(a, threads, stream) : run_norm_conv<T, VEC, NV, TAPS, false, 512>(a, threads, stream);
 }
 template <typename T, int VEC, int NV>
 static int pick_taps(const B200NormConv& a, int threads, cudaStream_t stream) {
   if constexpr (NV <= 2 && VEC == 4) {
-    if (a.taps == 1) return run_norm_conv<T, VEC, NV, 1>(a, threads, stream);
-    if (a.taps == 2) return run_norm_conv<T, VEC, NV, 2>(a, threads, stream);
-    if (a.taps == 3) return run_norm_conv<T, VEC, NV, 3>(a, threads, stream);
-    if (a.taps == 4) return run_norm_conv<T, VEC, NV, 4>(a, threads, stream);
+    if (a.taps == 1) return pick_pairs<T, VEC, NV, 1>(a, threads, stream);
+    if (a.taps == 2) return pick_pairs<T, VEC, NV, 2>(a, threads, stream);
+    if (a.taps == 3) return pick_pairs<T, VEC, NV, 3>(a, threads, stream);
+    if (a.taps == 4) return pick_pairs<T, VEC, NV, 4>(a, threads, stream);
   }
-  return run_norm_conv<T, VEC, NV, 0>(a, threads, stream);
+  return pick_pairs<T, VEC, NV, 0>(a, threads, stream);
 }
 template <typename T>
 static int pick_width(const B200NormConv& a, cudaStream_t stream) {
