@@ -3,7 +3,7 @@
 //   outer_step_kernel   token by token, the state in registers: decode rows and, for any sizes and fp32 storage, whole
 //                       prompt portions. Decay per key channel: with its low-rank product, output norm and gate. Decay per
 //                       head: with the step size
-//   outer_head_norm_kernel   norm per head, weight and SiLU gate over rows of fp32 o
+//   outer_head_norm kernels  norm per head, weight and SiLU gate over rows of fp32 o
 //   outer_part_norm_kernel   skip, SiLU gate, norm in equal parts over rows of fp32 o
 //
 // D and V are multiples of 16 padded with zeros; ``vdim`` is what the norms divide by.
@@ -179,6 +179,38 @@ __global__ void __launch_bounds__(THREADS) outer_step_kernel(B200Outer p, int sl
 }
 
 // ------------------------------------------------------------------------------------------- norms
+// Heads of up to 128 values: a warp takes kNormItems (row, head) pairs, loads first.
+static constexpr int kNormItems = 4;
+template <typename T>
+__global__ void __launch_bounds__(128) outer_head_norm_vec_kernel(B200Outer p, int row0, long items) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const long x0 = ((long)blockIdx.x * 4 + (threadIdx.x >> 5)) * kNormItems;
+  const int c = (threadIdx.x & 31) * 4;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 o[kNormItems], z[kNormItems];
+  const float4 w = c < p.V ? *reinterpret_cast<const float4*>(p.norm_w + c) : zero;
+  T* to[kNormItems];
+#pragma unroll
+  for (int i = 0; i < kNormItems; ++i) {
+    o[i] = z[i] = zero;
+    to[i] = nullptr;
+    if (x0 + i >= items || c >= p.V) continue;
+    const size_t t = row0 + (x0 + i) / p.H, h = (x0 + i) % p.H;
+    o[i] = *reinterpret_cast<const float4*>(p.o + (t * p.H + h) * p.V + c);
+    z[i] = Ou4<T>::get(reinterpret_cast<const T*>(p.gate) + t * p.ldg + h * p.V + c);
+    to[i] = reinterpret_cast<T*>(p.out) + t * p.ldo + h * p.V + c;
+  }
+#pragma unroll
+  for (int i = 0; i < kNormItems; ++i) {
+    const float ss = ou_sum(o[i].x * o[i].x + o[i].y * o[i].y + o[i].z * o[i].z + o[i].w * o[i].w);
+    const float inv = 1.f / sqrtf(ss / (float)p.vdim + p.eps);
+    const float4 g = ou_silu(z[i]);
+    if (to[i])
+      Ou4<T>::put(to[i], make_float4(o[i].x * inv * w.x * g.x, o[i].y * inv * w.y * g.y, o[i].z * inv * w.z * g.z, o[i].w * inv * w.w * g.w));
+  }
+}
+
 // One warp per (row, head).
 template <typename T>
 __global__ void __launch_bounds__(128) outer_head_norm_kernel(B200Outer p, int row0, int rows) {
@@ -334,6 +366,12 @@ int b200_outer_norm(const B200Outer* a, int reqs, int chunks, cudaStream_t strea
   }
   const int rows = chunks ? a->rows.T - a->rows.nd : 0;
   if (rows <= 0) return 0;
+  if (a->V <= 128) {
+    const long items = (long)rows * a->H;
+    const dim3 vgrid((unsigned)((items + 4 * kNormItems - 1) / (4 * kNormItems)));
+    return (a->f32 ? launch_pdl(outer_head_norm_vec_kernel<float>, vgrid, dim3(128), 0, stream, *a, a->rows.nd, items)
+                   : launch_pdl(outer_head_norm_vec_kernel<bf16>, vgrid, dim3(128), 0, stream, *a, a->rows.nd, items)) == cudaSuccess ? 0 : -2;
+  }
   const dim3 grid((unsigned)(((long)rows * a->H + 3) / 4));
   return (a->f32 ? launch_pdl(outer_head_norm_kernel<float>, grid, dim3(128), 0, stream, *a, a->rows.nd, rows)
                  : launch_pdl(outer_head_norm_kernel<bf16>, grid, dim3(128), 0, stream, *a, a->rows.nd, rows)) == cudaSuccess ? 0 : -2;

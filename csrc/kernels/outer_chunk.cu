@@ -11,7 +11,7 @@
 //
 //   outer_pairs_channel_kernel, outer_pairs_head_kernel   what does not depend on the state, parallel over chunks.
 //       Decay per channel (kind 0): q' = q e^G, k' = k e^(G_last - G) and P as pairs, G_last. P is the product of q' and
-//       k e^-G while no channel fades by more than e^-60 inside the chunk, else summed term by term. Decay per head
+//       k e^-G while no channel fades by more than 2^-86 inside the chunk, else summed term by term. Decay per head
 //       (kind 1): P = q k^T times e^(G_i - G_j) dt_j as pairs, e^G and dt e^(G_last - G); q k^T once for the heads that
 //       share it
 //   outer_scan_kernel   per (64 value columns, head, segment of a portion): walks the chunks with S in registers, as the
@@ -36,8 +36,9 @@ static constexpr int kC = 64;                    // tokens per chunk
 static constexpr int kVs = 64;                   // value columns per CTA of the scan
 static constexpr int kPairThreads = 256, kScanThreads = 512;
 static constexpr int kPlane = kC * 128;          // bytes of a 64 x 64 bf16 plane
-static constexpr float kMostDecay = 60.f;        // of a chunk whose factors are taken apart
-static constexpr float kTokenDecay = 30.f;       // of one token: beyond, nothing of the state is left either way
+static constexpr float kLog2e = 1.4426950408889634f;
+// kind 0, in powers of two: of a chunk whose factors are taken apart; of one token (beyond, nothing of the state is left)
+static constexpr float kMostDecay = 86.f, kTokenDecay = 44.f;
 static constexpr int kHeadsPerPair = 8;          // heads that one CTA of the head pairs serves
 
 __device__ __forceinline__ void oc_ldsm4(uint32_t* r, uint32_t addr) {
@@ -70,6 +71,11 @@ __device__ __forceinline__ void oc_cp16(uint32_t dst, const void* src, bool real
 }
 __device__ __forceinline__ void oc_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void oc_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ float oc_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ float oc_softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 // byte offset of 16-byte unit ``u`` of row ``r`` in a plane of 128-byte rows (units xored by the row)
@@ -80,7 +86,7 @@ __device__ __forceinline__ uint32_t oc_b(uint32_t base, int k0, int n0, int lane
 }
 
 // Workspace of one chunk and head, in bf16 values: kind 0: q' hi | lo | k' hi | lo ([64][D] each) | P hi | lo ([64][64]),
-// kind 1: P hi | lo. Factors in fp32: kind 0: G_last [D], kind 1: e^G [64] | dt e^(G_last - G) [64].
+// kind 1: P hi | lo. Factors in fp32: kind 0: G_last (to base 2) [D], kind 1: e^G [64] | dt e^(G_last - G) [64].
 __host__ __device__ inline size_t pair_values(int kind, int D) { return (kind == 0 ? (size_t)4 * kC * D : 0) + 2 * kC * kC; }
 __host__ __device__ inline int factor_values(int kind, int D) { return kind == 0 ? D : 2 * kC; }
 
@@ -94,14 +100,15 @@ __device__ __forceinline__ int chunks_ahead(const B200Rows& R, int req, int lane
 }
 
 // ------------------------------------------------------------------------------------- pairs, decay per channel
-struct ChannelSmem { int q, k, a1, total; };
+struct ChannelSmem { int q, k, a1, e, total; };
 __host__ __device__ inline ChannelSmem channel_smem(int D, int rank) {
   ChannelSmem m;
   const int rows = kC * (D + 8) * 2;             // a plane of q' or k e^-G rows
   m.q = 0;
   m.k = 2 * rows;                                // (over both, where P is summed term by term: fp32 [64][D] and [4][D])
   m.a1 = 4 * rows;
-  m.total = m.a1 + kC * (rank + 8) * 2;
+  m.e = m.a1 + kC * (rank + 8) * 2;              // 2^(G_last) [D]
+  m.total = m.e + D * 4;
   return m;
 }
 
@@ -139,7 +146,9 @@ __global__ void __launch_bounds__(kPairThreads, 3) outer_pairs_channel_kernel(B2
   const int col = (lane & 3) * 2, row = lane >> 2;
   float* sg = reinterpret_cast<float*>(smem);                     // term by term: sums inside blocks of 16 rows [64][D],
   float* st = sg + kC * D;                                       // sums of the blocks [4][D]
-  // Log decays, summed inside blocks of 16 rows; q', k' and k e^-G (``terms``: those sums alone, to shared memory).
+  float* se = reinterpret_cast<float*>(smem + L.e);
+  // Log decays (to base 2), summed inside blocks of 16 rows; q' and k e^-G (``terms``: those sums, and k' to the workspace).
+  const float scale = p.inv_tau * kLog2e;
   auto strips = [&](bool terms) {
     int far = 0;
     for (int u = warp * 2; u < D / 8; u += u & 1 ? 2 * (kPairThreads / 32) - 1 : 1) {    // (neighbours one after the other)
@@ -176,7 +185,7 @@ __global__ void __launch_bounds__(kPairThreads, 3) outer_pairs_channel_kernel(B2
 #pragma unroll
           for (int half = 0; half < 2; ++half) {
             float x = z[mb][half * 2 + e];
-            x = mb * 16 + half * 8 + row < n ? fmaxf(-oc_softplus(-x) * p.inv_tau, -kTokenDecay) : 0.f;
+            x = mb * 16 + half * 8 + row < n ? fmaxf(-(fmaxf(-x, 0.f) + log1pf(__expf(-fabsf(x)))) * scale, -kTokenDecay) : 0.f;
 #pragma unroll
             for (int o = 4; o < 32; o <<= 1) {
               const float y = __shfl_up_sync(0xffffffffu, x, o);
@@ -191,9 +200,20 @@ __global__ void __launch_bounds__(kPairThreads, 3) outer_pairs_channel_kernel(B2
       if (terms) {
 #pragma unroll
         for (int mb = 0; mb < 4; ++mb) {
+          float after[2] = {0.f, 0.f};           // (sums of the blocks behind, not a difference of sums)
 #pragma unroll
-          for (int half = 0; half < 2; ++half)
-            *reinterpret_cast<float2*>(sg + (mb * 16 + half * 8 + row) * D + cb) = make_float2(z[mb][half * 2], z[mb][half * 2 + 1]);
+          for (int x = mb + 1; x < 4; ++x) { after[0] += block[x][0]; after[1] += block[x][1]; }
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int r = mb * 16 + half * 8 + row;
+            const float g0 = z[mb][half * 2], g1 = z[mb][half * 2 + 1];
+            const float2 kk = unpack_bf16x2(kv[mb][half]);
+            *reinterpret_cast<float2*>(sg + r * D + cb) = make_float2(g0, g1);
+            uint32_t hi, lo;
+            oc_split(kk.x * oc_ex2(block[mb][0] - g0 + after[0]), kk.y * oc_ex2(block[mb][1] - g1 + after[1]), hi, lo);
+            *reinterpret_cast<uint32_t*>(wk + (size_t)r * D + cb) = hi;
+            *reinterpret_cast<uint32_t*>(wk + kC * D + (size_t)r * D + cb) = lo;
+          }
           if (lane < 4) *reinterpret_cast<float2*>(st + mb * D + cb) = make_float2(block[mb][0], block[mb][1]);
         }
         continue;
@@ -201,29 +221,22 @@ __global__ void __launch_bounds__(kPairThreads, 3) outer_pairs_channel_kernel(B2
       float before[2] = {0.f, 0.f};
       const float all0 = block[0][0] + block[1][0] + block[2][0] + block[3][0], all1 = block[0][1] + block[1][1] + block[2][1] + block[3][1];
       if (all0 < -kMostDecay || all1 < -kMostDecay) far = 1;
-      if (lane < 4) *reinterpret_cast<float2*>(p.factors + at * D + cb) = make_float2(all0, all1);
+      if (lane < 4) {
+        *reinterpret_cast<float2*>(p.factors + at * D + cb) = make_float2(all0, all1);
+        *reinterpret_cast<float2*>(se + cb) = make_float2(oc_ex2(all0), oc_ex2(all1));
+      }
 #pragma unroll
       for (int mb = 0; mb < 4; ++mb) {
-        float after[2] = {0.f, 0.f};             // (sums of the blocks behind, not a difference of sums)
-#pragma unroll
-        for (int x = mb + 1; x < 4; ++x) { after[0] += block[x][0]; after[1] += block[x][1]; }
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
-          const int r = mb * 16 + half * 8 + row;
-          const float g0 = z[mb][half * 2], g1 = z[mb][half * 2 + 1], s0 = before[0] + g0, s1 = before[1] + g1;
+          const float s0 = before[0] + z[mb][half * 2], s1 = before[1] + z[mb][half * 2 + 1];
           const float2 kk = unpack_bf16x2(kv[mb][half]), qq = unpack_bf16x2(qv[mb][half]);
           uint32_t hi, lo;
-          const size_t to = (size_t)r * D + cb;
-          oc_split(kk.x * expf(block[mb][0] - g0 + after[0]), kk.y * expf(block[mb][1] - g1 + after[1]), hi, lo);
-          *reinterpret_cast<uint32_t*>(wk + to) = hi;
-          *reinterpret_cast<uint32_t*>(wk + kC * D + to) = lo;
-          uint8_t* dst = smem + r * stride + cb * 2;
-          oc_split(kk.x * expf(-s0), kk.y * expf(-s1), hi, lo);
+          uint8_t* dst = smem + (mb * 16 + half * 8 + row) * stride + cb * 2;
+          oc_split(kk.x * oc_ex2(-s0), kk.y * oc_ex2(-s1), hi, lo);
           *reinterpret_cast<uint32_t*>(dst + L.k) = hi;
           *reinterpret_cast<uint32_t*>(dst + L.k + plane) = lo;
-          oc_split(p.q_scale * qq.x * expf(s0), p.q_scale * qq.y * expf(s1), hi, lo);
-          *reinterpret_cast<uint32_t*>(wq + to) = hi;
-          *reinterpret_cast<uint32_t*>(wq + kC * D + to) = lo;
+          oc_split(p.q_scale * qq.x * oc_ex2(s0), p.q_scale * qq.y * oc_ex2(s1), hi, lo);
           *reinterpret_cast<uint32_t*>(dst + L.q) = hi;
           *reinterpret_cast<uint32_t*>(dst + L.q + plane) = lo;
         }
@@ -233,7 +246,29 @@ __global__ void __launch_bounds__(kPairThreads, 3) outer_pairs_channel_kernel(B2
     }
     return far;
   };
-  if (!__syncthreads_or(strips(false))) {
+  const bool far = __syncthreads_or(strips(false));
+  // To the workspace in whole rows: q', and k' as k e^-G times e^(G_last).
+  for (int x = tid; x < kC * (D / 8); x += kPairThreads) {
+    const int r = x / (D / 8), u = x - r * (D / 8);
+    const uint8_t* from = smem + r * stride + u * 16;
+    const size_t to = (size_t)r * D + u * 8;
+    *reinterpret_cast<uint4*>(wq + to) = *reinterpret_cast<const uint4*>(from + L.q);
+    *reinterpret_cast<uint4*>(wq + kC * D + to) = *reinterpret_cast<const uint4*>(from + L.q + plane);
+    if (far) continue;
+    const uint4 a = *reinterpret_cast<const uint4*>(from + L.k), b = *reinterpret_cast<const uint4*>(from + L.k + plane);
+    const float4 e0 = *reinterpret_cast<const float4*>(se + u * 8), e1 = *reinterpret_cast<const float4*>(se + u * 8 + 4);
+    const float e[8] = {e0.x, e0.y, e0.z, e0.w, e1.x, e1.y, e1.z, e1.w};
+    const uint32_t h[4] = {a.x, a.y, a.z, a.w}, l[4] = {b.x, b.y, b.z, b.w};
+    uint32_t hi[4], lo[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 y = unpack_bf16x2(h[i]), z = unpack_bf16x2(l[i]);
+      oc_split((y.x + z.x) * e[2 * i], (y.y + z.y) * e[2 * i + 1], hi[i], lo[i]);
+    }
+    *reinterpret_cast<uint4*>(wk + to) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+    *reinterpret_cast<uint4*>(wk + kC * D + to) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+  }
+  if (!far) {
     const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * 32;
     if (n0 > m0) return;                         // (blocks above the diagonal are not needed)
     float px[4][4];
@@ -289,7 +324,7 @@ __global__ void __launch_bounds__(kPairThreads, 3) outer_pairs_channel_kernel(B2
           g += st[bj * D + d] - sg[j * D + d];
           for (int b = bj + 1; b < bi; ++b) g += st[b * D + d];
         }
-        s = fmaf(__bfloat162float(gq[(size_t)i * p.ld + d]) * __bfloat162float(gk[(size_t)j * p.ld + d]), expf(g), s);
+        s = fmaf(__bfloat162float(gq[(size_t)i * p.ld + d]) * __bfloat162float(gk[(size_t)j * p.ld + d]), oc_ex2(g), s);
       }
     s *= p.q_scale;
     const bf16 hi = __float2bfloat16(s);
@@ -499,7 +534,7 @@ __global__ void __launch_bounds__(kScanThreads, 1) outer_scan_kernel(B200Outer p
   const size_t size = (size_t)D * V;
   float* state = p.state + ((size_t)slot * p.H + h) * size + v0;
   float hs[MI][4][4];
-  float total[MI][2];                            // log decay of the rows of this thread's pieces since the segment's start
+  float total[MI][2];                            // log2 of the decay of the rows of this thread's pieces since the segment's start
   auto each_state = [&](auto f) {                // f(value, value, row, column) for pairs of columns
 #pragma unroll
     for (int i = 0; i < MI; ++i) {
@@ -534,7 +569,7 @@ __global__ void __launch_bounds__(kScanThreads, 1) outer_scan_kernel(B200Outer p
       const float* w = p.ws_decay + at * D;
       each_state([&](float& x, float& y, int d, int c) {
         const float2 u = *reinterpret_cast<const float2*>(s + (size_t)d * V + c);
-        const float f = i == 0 ? 0.f : expf(w[d]);
+        const float f = i == 0 ? 0.f : exp2f(w[d]);
         x = fmaf(f, x, u.x);
         y = fmaf(f, y, u.y);
       });
@@ -635,15 +670,15 @@ __global__ void __launch_bounds__(kScanThreads, 1) outer_scan_kernel(B200Outer p
         const float g0 = f[d0 + (lane >> 2)], g1 = f[d0 + (lane >> 2) + 8];
         total[i][0] += g0;
         total[i][1] += g1;
-        f0 = expf(g0);
-        f1 = expf(g1);
+        f0 = exp2f(g0);
+        f1 = exp2f(g1);
       }
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         hs[i][x][0] *= f0; hs[i][x][1] *= f0;
         hs[i][x][2] *= f1; hs[i][x][3] *= f1;
       }
-      if (KIND == 1) total[i][0] += logf(f0);
+      if (KIND == 1) total[i][0] += log2f(f0);
 #pragma unroll
       for (int k0 = 0; k0 < kC; k0 += 16) {
         uint32_t kh[4], kl[4], bh[8], bl[8];
