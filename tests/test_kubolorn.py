@@ -279,6 +279,15 @@ def test_pages_and_slots_are_used_again(folder, name, dtype, dev):
     assert r.free_pages() == total
 
 
+@device
+def test_an_id_is_used_again(folder, dev):
+    """A finished request's id at once for another one."""
+    r = Replay(folder("mixed"), "float32", dev, 64, max_requests=2)
+    for i in range(3):
+        toks = tokens(30 + i, 96, 160 + i)
+        agrees(r.run({"a": toks}, [[("a", 29)], [("a", 1 + i)]])["a"], "mixed", toks, "float32")
+
+
 # ------------------------------------------------------------------------------ generation
 def check_greedy(name, prompt, out, dtype="float32"):
     """Every generated token is the oracle's choice, or (rounding) next to it."""

@@ -694,7 +694,7 @@ def _tabupel_dict(cfg: ModelConfig) -> dict:
                 rot["scaling"] = s if s["original"] else {"factor": s["factor"]}
             w = m.pop("window")
             m.update(rot=rot, **({"mask": {"size": w}} if w else {}))
-            for k in ("bias_max", "chunk"):
+            for k in ("bias_max", "chunk", "sink", "tied"):
                 m.pop(k, None)
         l = {"type": kind, "mixer": m, "mlp": None if b.mlp is None else {"kind": "dense", "ff": b.mlp.ff}}
         if b.weights_of is not None:

@@ -35,13 +35,19 @@ class TraceReplay:
                                   max_num_batched_tokens=pages * page, max_score_rows=pages * page,
                                   enable_prefix_caching=False))
         self.length: dict[str, int] = {}
+        self.name: dict[str, str] = {}       # of a live request in the engine (a trace may use an id again)
+        self.count = 0
 
     def step(self, entries: list, end: list):
         """-> the wanted logits rows, in the order of the entries and their ``want``."""
         from ..engine import SamplingParams
         llm, order, total = self.llm, [], 0
         for e in entries:
-            rid, toks, at = e["id"], e["tokens"], self.length.get(e["id"], 0)
+            if e["id"] not in self.name:
+                self.count += 1
+                self.name[e["id"]] = f"{e['id']}.{self.count}"
+            rid, toks = self.name[e["id"]], e["tokens"]
+            at = self.length.get(rid, 0)
             want = [at + w for w in e.get("want", [])]
             if want:
                 llm.score_positions(rid, sorted(set(want)))
@@ -58,7 +64,7 @@ class TraceReplay:
             if ran != total:
                 raise RuntimeError(f"the engine ran {ran} of the step's {total} tokens")
         rows = {(rid, p): row for rid, items in llm.take_scores().items() for p, row in items}
-        for rid in end:
+        for rid in (self.name.pop(i) for i in end if i in self.name):
             llm.abort_request(rid)
             self.length.pop(rid, None)
         return [rows[k] for k in order]
