@@ -182,10 +182,10 @@ __global__ void __launch_bounds__(THREADS) outer_step_kernel(B200Outer p, int sl
 // Heads of up to 128 values: a warp takes kNormItems (row, head) pairs, loads first.
 static constexpr int kNormItems = 4;
 template <typename T>
-__global__ void __launch_bounds__(128) outer_head_norm_vec_kernel(B200Outer p, int row0, long items) {
+__global__ void __launch_bounds__(128) outer_head_norm_vec_kernel(B200Outer p, int row0, uint32_t items) {
   pdl_wait();
   pdl_launch_dependents();
-  const long x0 = ((long)blockIdx.x * 4 + (threadIdx.x >> 5)) * kNormItems;
+  const uint32_t x0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * kNormItems, H = p.H;
   const int c = (threadIdx.x & 31) * 4;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   float4 o[kNormItems], z[kNormItems];
@@ -196,7 +196,8 @@ __global__ void __launch_bounds__(128) outer_head_norm_vec_kernel(B200Outer p, i
     o[i] = z[i] = zero;
     to[i] = nullptr;
     if (x0 + i >= items || c >= p.V) continue;
-    const size_t t = row0 + (x0 + i) / p.H, h = (x0 + i) % p.H;
+    const uint32_t r = (x0 + i) / H, h = x0 + i - r * H;
+    const size_t t = row0 + r;
     o[i] = *reinterpret_cast<const float4*>(p.o + (t * p.H + h) * p.V + c);
     z[i] = Ou4<T>::get(reinterpret_cast<const T*>(p.gate) + t * p.ldg + h * p.V + c);
     to[i] = reinterpret_cast<T*>(p.out) + t * p.ldo + h * p.V + c;
@@ -246,7 +247,7 @@ __global__ void __launch_bounds__(256) outer_part_norm_kernel(B200Outer p) {
   const float* o = p.o + t * inner;
   const bool dense = p.V == p.vdim;
   for (int i = tid * 4; i < inner; i += 256 * 4) {
-    const int h = i / p.V, c = i - h * p.V;
+    const int h = (unsigned)i / (unsigned)p.V, c = i - h * p.V;
     const float d = p.skip[h];
     const float4 a = *reinterpret_cast<const float4*>(o + i), x = Ou4<T>::get(v + i), g = ou_silu(Ou4<T>::get(z + i));
     const float4 y = make_float4(fmaf(d, x.x, a.x) * g.x, fmaf(d, x.y, a.y) * g.y, fmaf(d, x.z, a.z) * g.z, fmaf(d, x.w, a.w) * g.w);
@@ -284,7 +285,7 @@ __global__ void __launch_bounds__(256) outer_part_norm_kernel(B200Outer p) {
   T* out = reinterpret_cast<T*>(p.out) + t * p.ldo;
   if (dense && !(ps & 3)) {
     for (int i = tid * 4; i < inner; i += 256 * 4) {
-      const float f = inv[i / ps];
+      const float f = inv[(unsigned)i / (unsigned)ps];
       const float4 y = *reinterpret_cast<const float4*>(part_smem + i), w = *reinterpret_cast<const float4*>(p.norm_w + i);
       Ou4<T>::put(out + i, make_float4(y.x * f * w.x, y.y * f * w.y, y.z * f * w.z, y.w * f * w.w));
     }
@@ -366,9 +367,9 @@ int b200_outer_norm(const B200Outer* a, int reqs, int chunks, cudaStream_t strea
   }
   const int rows = chunks ? a->rows.T - a->rows.nd : 0;
   if (rows <= 0) return 0;
-  if (a->V <= 128) {
-    const long items = (long)rows * a->H;
-    const dim3 vgrid((unsigned)((items + 4 * kNormItems - 1) / (4 * kNormItems)));
+  if (a->V <= 128 && (long)rows * a->H < (1l << 31)) {
+    const uint32_t items = (uint32_t)rows * a->H;
+    const dim3 vgrid((items + 4 * kNormItems - 1) / (4 * kNormItems));
     return (a->f32 ? launch_pdl(outer_head_norm_vec_kernel<float>, vgrid, dim3(128), 0, stream, *a, a->rows.nd, items)
                    : launch_pdl(outer_head_norm_vec_kernel<bf16>, vgrid, dim3(128), 0, stream, *a, a->rows.nd, items)) == cudaSuccess ? 0 : -2;
   }
